@@ -112,9 +112,38 @@ def cuda_sources():
     return sorted(os.path.join(CUDA_DIR, f) for f in os.listdir(CUDA_DIR) if f.endswith(".cu"))
 
 
-def build_cuda(force=False):
+# Kernel sources that a model type needs, for programs that serve one model and compile at their first call.
+MODEL_SOURCES = {
+    "movolorn": ("attention_decode_tma", "attention_prefill_tc", "attention_simt", "gemm_bf16", "gemm_bf16_2cta", "gemm_simt",
+                 "host_util", "moe", "sampling", "sandwich_norm"),
+}
+
+
+def _newer_than_sources(target, srcs, hdrs):
+    return os.path.exists(target) and not _newer(list(srcs) + list(hdrs), target)
+
+
+def build_for_model(model_type):
+    """What one model needs: the host runtime and its kernels, compiled side by side.  Returns the kernel library: the full
+    one when it is there and up to date, else a library of this model's kernels only."""
+    import fcntl
     os.makedirs(BUILD_DIR, exist_ok=True)
-    srcs = cuda_sources()
+    with open(os.path.join(BUILD_DIR, "lock"), "w") as lock:
+        fcntl.flock(lock, fcntl.LOCK_EX)
+        hdrs = [os.path.join(CUDA_DIR, f) for f in os.listdir(CUDA_DIR) if f.endswith((".cuh", ".h"))]
+        with ThreadPoolExecutor(max_workers=2) as ex:
+            core = ex.submit(build_core)
+            if model_type not in MODEL_SOURCES or _newer_than_sources(KERNELS_SO, cuda_sources(), hdrs):
+                out = build_cuda()
+            else:
+                out = build_cuda(only=MODEL_SOURCES[model_type], target=os.path.join(HERE, f"libxllm_kernels_{model_type}.so"))
+            core.result()
+    return out
+
+
+def build_cuda(force=False, only=None, target=KERNELS_SO):
+    os.makedirs(BUILD_DIR, exist_ok=True)
+    srcs = [s for s in cuda_sources() if only is None or os.path.basename(s)[:-3] in only]
     hdrs = [os.path.join(CUDA_DIR, f) for f in os.listdir(CUDA_DIR) if f.endswith((".cuh", ".h"))]
     objs, jobs = [], []
     for s in srcs:
@@ -127,9 +156,9 @@ def build_cuda(force=False):
         _run([NVCC, *NVCC_FLAGS, "-I", CUDA_DIR, "-c", s, "-o", o], log=o + ".log")
     with ThreadPoolExecutor(max_workers=min(8, max(1, len(jobs)))) as ex:
         list(ex.map(compile_one, jobs))
-    if jobs or not os.path.exists(KERNELS_SO):
-        _run([NVCC, "-shared", "-o", KERNELS_SO, *objs, "-lcuda", "-L/usr/local/cuda/lib64/stubs", "-lcudart"])
-    return KERNELS_SO
+    if jobs or not os.path.exists(target) or _newer(objs, target):
+        _run([NVCC, "-shared", "-o", target, *objs, "-lcuda", "-L/usr/local/cuda/lib64/stubs", "-lcudart"])
+    return target
 
 
 def build_all(force=False, core=True, cuda=True):

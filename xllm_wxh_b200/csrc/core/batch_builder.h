@@ -66,7 +66,7 @@ inline long build_batch(const Batch& b, const BatchLayout& L, int32_t* buf, int 
   auto as_f = [](float f) { int32_t i; std::memcpy(&i, &f, 4); return i; };
   const int n_seq = static_cast<int>(b.entries.size());
   int n_rows = 0;
-  for (auto& e : b.entries) if (e.sample) n_rows += 1 + e.n_spec;
+  for (auto& e : b.entries) n_rows += e.num_rows();
   if (b.num_tokens > L.T_cap || n_seq > L.B_cap || n_rows > L.S_cap) return -1;
   int32_t* H = buf + L.header;
   std::memset(H, 0, 32 * 4);
@@ -104,11 +104,11 @@ inline long build_batch(const Batch& b, const BatchLayout& L, int32_t* buf, int 
     n_spec = std::max(n_spec, e.n_spec);
     const bool is_dec = (real == 1 && e.sample && e.kv_before > 0);
     if (!is_dec) n_prefill_tokens += e.n_tokens;
-    if (e.sample) {
+    if (e.num_rows() > 0) {
       const SamplingParams& sp = s->req->sampling;
-      const int rows = 1 + e.n_spec;
+      const int rows = e.num_rows();
       for (int j = 0; j < rows; ++j) {
-        sidx[row] = t - rows + j;
+        sidx[row] = e.replay ? t - e.n_tokens + e.want[j] : t - rows + j;
         buf[L.temperature + row] = as_f(sp.temperature);
         buf[L.top_p + row] = as_f(sp.top_p);
         buf[L.top_k + row] = sp.top_k;

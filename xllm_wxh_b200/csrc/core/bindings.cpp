@@ -143,7 +143,7 @@ PYBIND11_MODULE(_core, m) {
       .def_property_readonly("num_sample_rows",
                              [](const Batch& b) {
                                int r = 0;
-                               for (auto& e : b.entries) if (e.sample) r += 1 + e.n_spec;
+                               for (auto& e : b.entries) r += e.num_rows();
                                return r;
                              })
       .def_property_readonly("max_blocks",
@@ -171,11 +171,16 @@ PYBIND11_MODULE(_core, m) {
         std::vector<std::tuple<int64_t, int, int, int>> v;
         int row = 0;
         for (auto& e : b.entries) {
-          if (!e.sample) continue;
+          if (e.num_rows() == 0) continue;
           const auto& sp = e.seq->req->sampling;
           if (sp.logprobs && sp.top_logprobs > 0) v.emplace_back(e.seq->req->id, e.seq->index, row, sp.top_logprobs);
-          row += 1 + e.n_spec;
+          row += e.num_rows();
         }
+        return v;
+      })
+      .def("rows_per_entry", [](const Batch& b) {
+        std::vector<int> v;
+        for (auto& e : b.entries) v.push_back(e.num_rows());
         return v;
       })
       .def("seq_tokens", [](const Batch& b, int i) { return b.entries.at(i).seq->tokens; })
@@ -310,6 +315,15 @@ PYBIND11_MODULE(_core, m) {
       .def_property_readonly("num_running", &Scheduler::num_running)
       .def_property_readonly("num_pending", &Scheduler::num_pending)
       .def("schedule", &Scheduler::schedule, py::return_value_policy::reference_internal)
+      // portions: [(request id, tokens, wanted places)]
+      .def("schedule_portions",
+           [](Scheduler& s, const std::vector<std::tuple<int64_t, std::vector<int32_t>, std::vector<int>>>& portions) {
+             std::vector<Portion> ps;
+             for (auto& p : portions) ps.push_back({std::get<0>(p), std::get<1>(p), std::get<2>(p)});
+             return s.schedule_portions(ps);
+           },
+           py::return_value_policy::reference_internal)
+      .def("complete_portions", &Scheduler::complete_portions)
       .def("process_output",
            [](Scheduler& s, int64_t batch_id, py::array_t<int32_t, py::array::c_style | py::array::forcecast> tokens,
               py::object logprobs) {

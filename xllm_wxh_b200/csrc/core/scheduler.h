@@ -64,6 +64,19 @@ struct BatchEntry {
   int kv_before = 0;   // seq->kv_tokens when scheduled
   int sample_slot = -1;  // index among the sampling entries of the batch
   int placeholder_pos = -1;  // position in seq->tokens of the overlap placeholder
+  // Replayed portion: the step samples nothing, the logits of these places among the entry's tokens are read instead
+  bool replay = false;
+  std::vector<int> want;
+  // rows of the step whose logits are computed for this entry
+  int num_rows() const { return replay ? static_cast<int>(want.size()) : (sample ? 1 + n_spec : 0); }
+};
+
+// The next `tokens.size()` tokens of a request whose steps are dictated from outside (replay), and the places among them
+// whose logits the caller wants.
+struct Portion {
+  int64_t request_id = 0;
+  std::vector<int32_t> tokens;
+  std::vector<int> want;
 };
 
 struct Batch {
@@ -348,6 +361,64 @@ class Scheduler {
     }
     ++stats_.steps;
     return out;
+  }
+
+  // Build a step from given portions instead of a policy (replay of recorded token streams): every portion's tokens are
+  // appended to its request and scheduled whole, all portions in one batch, with the blocks, slots and entry order of any
+  // other step.  A request is admitted with its first portion (its prompt must be empty) and may be left out of steps.
+  // Call `complete_portions` once the step has run.  Throws when the cache has no room; nothing is evicted or preempted.
+  std::vector<Batch*> schedule_portions(const std::vector<Portion>& portions) {
+    if (opt_.dp_size != 1) throw std::runtime_error("portions need one attention-DP rank");
+    drain_incoming();
+    reap_finished();
+    current_.clear();
+    std::vector<Sequence*> seqs;
+    int need = 0;
+    for (const Portion& p : portions) {
+      Request* r = find_request(p.request_id);
+      if (!r || r->finished() || r->cancelled) throw std::runtime_error("portion of an unknown or finished request");
+      Sequence* s = r->seqs[0].get();
+      if (p.tokens.empty() || s->remaining() != 0 || std::find(seqs.begin(), seqs.end(), s) != seqs.end())
+        throw std::runtime_error("a request has one non-empty portion per step, after its earlier ones have run");
+      for (int w : p.want)
+        if (w < 0 || w >= static_cast<int>(p.tokens.size())) throw std::runtime_error("wanted place outside its portion");
+      seqs.push_back(s);
+      need += blocks_needed(s, s->num_tokens() + static_cast<int>(p.tokens.size()));
+    }
+    if (need > pool_.at(0).num_available_blocks()) throw std::runtime_error("the KV cache has no room for this step's portions");
+    batches_storage_.emplace_back();
+    std::vector<Batch>& bs = batches_storage_.back();
+    bs.resize(1);
+    bs[0].id = next_batch_id_++;
+    budget_tokens_.assign(1, 1 << 30);
+    budget_seqs_.assign(1, 1 << 30);
+    for (size_t i = 0; i < portions.size(); ++i) {
+      Sequence* s = seqs[i];
+      s->dp_rank = 0;
+      s->tokens.insert(s->tokens.end(), portions[i].tokens.begin(), portions[i].tokens.end());
+      if (!is_running(s->req)) {
+        remove_from_queues(s->req);
+        running_.push_back(s->req);
+      }
+      if (!ensure_blocks(s, s->num_tokens())) throw std::runtime_error("block allocation failed");
+      add_entry(bs, s, static_cast<int>(portions[i].tokens.size()), 0);
+      bs[0].entries.back().replay = true;
+      bs[0].entries.back().want = portions[i].want;
+    }
+    finalize(bs[0]);
+    live_batches_[bs[0].id] = &bs[0];
+    while (batches_storage_.size() > 4) {
+      for (auto& b : batches_storage_.front()) live_batches_.erase(b.id);
+      batches_storage_.pop_front();
+    }
+    ++stats_.steps;
+    return {&bs[0]};
+  }
+  void complete_portions(int64_t batch_id) {
+    Batch* b = find_batch(batch_id);
+    if (!b) return;
+    for (auto& e : b->entries)
+      if (e.replay && !e.seq->finished) e.seq->kv_tokens = e.kv_before + e.n_tokens;
   }
 
   // Apply sampled tokens.  `tokens` is [num_sample, width]; width = 1 + n_spec, -1 marks a

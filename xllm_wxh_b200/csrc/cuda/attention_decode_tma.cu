@@ -12,6 +12,10 @@
 // engine removes the per-chunk address arithmetic and block-table lookups from the compute warps, which is what
 // bounds a decode kernel whose arithmetic intensity is a few FLOP per byte.
 //
+// Template parameters: DK / DV = query-key / value head dimension padded to 64 or 128 (the TMA loads fill the padding with
+// zeros), EXT = score extensions (per-head distance bias, per-head sink, chunk mask) and head dimensions below the padded
+// ones.
+//
 // Role: the reference's FlashInfer `batch_decode_with_kv_cache` (xllm/core/kernels/cuda/batch_decode.cpp:26-85).
 #include "common.cuh"
 
@@ -58,6 +62,11 @@ struct DecParams {
   const int* dyn_end = nullptr;   // optional device scalar that replaces seq_end (launch sized for a capacity)
   int ws_rows = 0;                // > 0: row capacity of a fixed-size workspace; sequences that do not fit it (or have more
                                   // than 16 query rows x heads per kv head) are skipped and XL_ERR_BOUNDS is recorded
+  // score extensions (EXT): see xl_prefill_attention_ext
+  int dk = 0, dv = 0;
+  int chunk = 0;
+  const float* slopes = nullptr;
+  const float* sinks = nullptr;
 };
 
 constexpr int kStages = 3;
@@ -68,19 +77,23 @@ struct DecBarriers {
   uint64_t empty[kStages];
 };
 
-template <int D>
+template <int DK, int DV, bool EXT>
 __global__ void __launch_bounds__(160) decode_attn_tma_kernel(const __grid_constant__ CUtensorMap tmK,
                                                               const __grid_constant__ CUtensorMap tmV, DecParams p) {
-  constexpr int HALVES = D / 64;                  // 128-byte column slabs per row
+  constexpr int KH = DK / 64, VH = DV / 64;       // 128-byte column slabs per row
   constexpr int SLAB = kTile * 128;               // bytes of one slab of a 64-token tile
-  constexpr int KV_BYTES = HALVES * SLAB;         // K (or V) bytes per stage
-  constexpr int STAGE_BYTES = 2 * KV_BYTES;
-  constexpr int CH = D / 8;
+  constexpr int K_BYTES = KH * SLAB;              // K bytes per stage (V behind it)
+  constexpr int STAGE_BYTES = (KH + VH) * SLAB;
+  constexpr int CH = DK / 8;
+  constexpr float kL2e = 1.4426950408889634f;
+  const int dk = EXT ? p.dk : DK, dv = EXT ? p.dv : DV;
   extern __shared__ uint8_t smem_raw[];
   uint8_t* smem = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(smem_raw) + 1023) & ~uintptr_t(1023));
   uint8_t* ring = smem;                                          // kStages * STAGE_BYTES, 1024-aligned
-  uint8_t* sQ = smem + kStages * STAGE_BYTES;                    // 16 x D bf16, 16-byte-chunk XOR swizzle
-  DecBarriers* bars = reinterpret_cast<DecBarriers*>(sQ + 16 * D * 2);
+  constexpr int MERGE_BYTES = 4 * 16 * DV * 4 + 128 * 4;         // partials of the four warps, in the ring's memory
+  constexpr int RING_BYTES = kStages * STAGE_BYTES > MERGE_BYTES ? kStages * STAGE_BYTES : MERGE_BYTES;
+  uint8_t* sQ = smem + RING_BYTES;                               // 16 x DK bf16, 16-byte-chunk XOR swizzle
+  DecBarriers* bars = reinterpret_cast<DecBarriers*>(sQ + 16 * DK * 2);
 
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const int seq = p.seq_begin + blockIdx.x;
@@ -99,8 +112,10 @@ __global__ void __launch_bounds__(160) decode_attn_tma_kernel(const __grid_const
   const int rows = min(16, q_len * group);
   const int* bt = p.block_tables + size_t(seq) * p.max_blocks;
 
-  const int per_split = ((kv_len + p.num_splits - 1) / p.num_splits + kTile - 1) / kTile * kTile;
-  int s_begin = split * per_split;
+  int r_begin = 0;                                // first key that any row may see, rounded down to a tile
+  if (EXT && p.chunk > 0) r_begin = (kv_len - q_len) / p.chunk * p.chunk / kTile * kTile;
+  const int per_split = ((kv_len - r_begin + p.num_splits - 1) / p.num_splits + kTile - 1) / kTile * kTile;
+  int s_begin = r_begin + split * per_split;
   const int s_end = min(kv_len, s_begin + per_split);
   if (p.window > 0) s_begin = max(s_begin, (max(0, kv_len - q_len - p.window + 1)) / kTile * kTile);
   const int n_tiles = s_end > s_begin ? (s_end - s_begin + kTile - 1) / kTile : 0;
@@ -115,18 +130,18 @@ __global__ void __launch_bounds__(160) decode_attn_tma_kernel(const __grid_const
   // Q rows -> smem (zero beyond `rows`); row m = qtok * group + g
   for (int i = threadIdx.x; i < 16 * CH; i += blockDim.x) {
     const int r = i / CH, c = i % CH;
-    const bool ok = r < rows;
+    const bool ok = r < rows && (!EXT || c * 8 < dk);
     const int qt = ok ? r / group : 0, g = ok ? r % group : 0;
-    const __nv_bfloat16* src = p.q + size_t(q_start + qt) * p.q_stride + (kvh * group + g) * D + c * 8;
-    cp_async_16(sQ + uint32_t(r) * (D * 2) + (uint32_t(c ^ (r & 7)) << 4), src, ok);
+    const __nv_bfloat16* src = p.q + size_t(q_start + qt) * p.q_stride + (kvh * group + g) * dk + (ok ? c * 8 : 0);
+    cp_async_16(sQ + uint32_t(r) * (DK * 2) + (uint32_t(c ^ (r & 7)) << 4), src, ok);
   }
   cp_async_commit();
   cp_async_wait_all();
   __syncthreads();
 
-  float o[D / 8][4];
+  float o[DV / 8][4];
 #pragma unroll
-  for (int i = 0; i < D / 8; ++i) o[i][0] = o[i][1] = o[i][2] = o[i][3] = 0.f;
+  for (int i = 0; i < DV / 8; ++i) o[i][0] = o[i][1] = o[i][2] = o[i][3] = 0.f;
   float m_run[2] = {-INFINITY, -INFINITY}, l_run[2] = {0.f, 0.f};
   const int row_a = lane >> 2, row_b = row_a + 8;
 
@@ -149,18 +164,18 @@ __global__ void __launch_bounds__(160) decode_attn_tma_kernel(const __grid_const
         const int base = s_begin + t * kTile;
         const int n_tok = min(kTile, s_end - base);
         const int n_boxes = (n_tok + bt_tok - 1) / bt_tok;
-        mbar_arrive_expect_tx(&bars->full[s], uint32_t(n_boxes) * bt_tok * 128 * HALVES * 2);
+        mbar_arrive_expect_tx(&bars->full[s], uint32_t(n_boxes) * bt_tok * 128 * (KH + VH));
         uint8_t* dK = ring + s * STAGE_BYTES;
-        uint8_t* dV = dK + KV_BYTES;
+        uint8_t* dV = dK + K_BYTES;
         for (int b = 0; b < n_boxes; ++b) {
           const int tok = base + b * bt_tok;
           int blk = bt[tok / p.block_size];
           if (blk < 0 || blk >= p.num_blocks_total) blk = 0;     // never form an address outside the cache
           const int z = blk * p.block_size + tok % p.block_size;
 #pragma unroll
-          for (int h = 0; h < HALVES; ++h) {
-            tma_load_3d(dK + h * SLAB + b * bt_tok * 128, &tmK, &bars->full[s], h * 64, kvh, z);
-            tma_load_3d(dV + h * SLAB + b * bt_tok * 128, &tmV, &bars->full[s], h * 64, kvh, z);
+          for (int h = 0; h < (KH > VH ? KH : VH); ++h) {
+            if (h < KH) tma_load_3d(dK + h * SLAB + b * bt_tok * 128, &tmK, &bars->full[s], h * 64, kvh, z);
+            if (h < VH) tma_load_3d(dV + h * SLAB + b * bt_tok * 128, &tmV, &bars->full[s], h * 64, kvh, z);
           }
         }
       }
@@ -171,17 +186,29 @@ __global__ void __launch_bounds__(160) decode_attn_tma_kernel(const __grid_const
     }
   } else {
     // ------------------------------------------------------------ consumers
-    uint32_t qf[D / 16][4];
+    uint32_t qf[DK / 16][4];
     {
       const int r = (lane & 7) + ((lane >> 3) & 1) * 8;
 #pragma unroll
-      for (int ks = 0; ks < D / 16; ++ks) {
+      for (int ks = 0; ks < DK / 16; ++ks) {
         const int c = ks * 2 + (lane >> 4);
-        ldsm_x4(smem_u32(sQ + uint32_t(r) * (D * 2) + (uint32_t(c ^ (r & 7)) << 4)), qf[ks][0], qf[ks][1], qf[ks][2], qf[ks][3]);
+        ldsm_x4(smem_u32(sQ + uint32_t(r) * (DK * 2) + (uint32_t(c ^ (r & 7)) << 4)), qf[ks][0], qf[ks][1], qf[ks][2], qf[ks][3]);
       }
     }
     const int lim_a = kv_len - q_len + (row_a < rows ? row_a / group : 0);
     const int lim_b = kv_len - q_len + (row_b < rows ? row_b / group : 0);
+    int lo_a = 0, lo_b = 0;                                // first visible key of the row's chunk
+    float slope_a = 0.f, slope_b = 0.f;
+    if (EXT) {
+      if (p.chunk > 0) {
+        lo_a = lim_a / p.chunk * p.chunk;
+        lo_b = lim_b / p.chunk * p.chunk;
+      }
+      if (p.slopes) {
+        slope_a = p.slopes[kvh * group + (row_a < rows ? row_a % group : 0)] * kL2e;
+        slope_b = p.slopes[kvh * group + (row_b < rows ? row_b % group : 0)] * kL2e;
+      }
+    }
     const int rk = (lane & 7) + (lane >> 4) * 8;           // K fragment row (token) of this lane
     const int rv = (lane & 7) + ((lane >> 3) & 1) * 8;     // V fragment row (token) of this lane
     for (int t = 0; t < n_tiles; ++t) {
@@ -194,12 +221,12 @@ __global__ void __launch_bounds__(160) decode_attn_tma_kernel(const __grid_const
       const int base = s_begin + t * kTile + warp * 16;
       if (base < s_end) {
         const uint8_t* tK = ring + s * STAGE_BYTES + warp * 2048;
-        const uint8_t* tV = tK + KV_BYTES;
+        const uint8_t* tV = tK + K_BYTES;
         float sc[2][4];
 #pragma unroll
         for (int i = 0; i < 2; ++i) sc[i][0] = sc[i][1] = sc[i][2] = sc[i][3] = 0.f;
 #pragma unroll
-        for (int ks = 0; ks < D / 16; ++ks) {
+        for (int ks = 0; ks < DK / 16; ++ks) {
           uint32_t b0, b1, b2, b3;
           const int c = (ks & 3) * 2 + ((lane >> 3) & 1);
           ldsm_x4(smem_u32(tK + (ks >> 2) * SLAB + rk * 128 + ((c ^ (rk & 7)) << 4)), b0, b1, b2, b3);
@@ -215,7 +242,12 @@ __global__ void __launch_bounds__(160) decode_attn_tma_kernel(const __grid_const
             const int lim = (e < 2) ? lim_a : lim_b;
             bool ok = tok <= lim && tok < s_end;
             if (p.window > 0) ok = ok && tok > lim - p.window;
-            const float v = ok ? sc[i][e] * p.scale_log2 : -INFINITY;
+            float x = sc[i][e] * p.scale_log2;
+            if (EXT) {
+              ok = ok && tok >= ((e < 2) ? lo_a : lo_b);
+              x += ((e < 2) ? slope_a : slope_b) * float(tok - lim);
+            }
+            const float v = ok ? x : -INFINITY;
             sc[i][e] = v;
             mx[e >> 1] = fmaxf(mx[e >> 1], v);
           }
@@ -246,7 +278,7 @@ __global__ void __launch_bounds__(160) decode_attn_tma_kernel(const __grid_const
                                 pack_bf16x2(sc[1][0], sc[1][1]), pack_bf16x2(sc[1][2], sc[1][3])};
         const bool rescale = (alpha[0] != 1.f) || (alpha[1] != 1.f);
 #pragma unroll
-        for (int dt = 0; dt < D / 16; ++dt) {
+        for (int dt = 0; dt < DV / 16; ++dt) {
           if (rescale) {
             o[2 * dt][0] *= alpha[0]; o[2 * dt][1] *= alpha[0]; o[2 * dt][2] *= alpha[1]; o[2 * dt][3] *= alpha[1];
             o[2 * dt + 1][0] *= alpha[0]; o[2 * dt + 1][1] *= alpha[0]; o[2 * dt + 1][2] *= alpha[1]; o[2 * dt + 1][3] *= alpha[1];
@@ -269,15 +301,15 @@ __global__ void __launch_bounds__(160) decode_attn_tma_kernel(const __grid_const
   }
   __syncthreads();   // ring no longer needed: reuse it for the merge
 
-  float* sO = reinterpret_cast<float*>(ring);     // [4][16][D]
-  float* sM = sO + 4 * 16 * D;                    // [4][16]
+  float* sO = reinterpret_cast<float*>(ring);     // [4][16][DV]
+  float* sM = sO + 4 * 16 * DV;                   // [4][16]
   float* sL = sM + 64;
   if (warp < 4) {
 #pragma unroll
-    for (int i = 0; i < D / 8; ++i) {
+    for (int i = 0; i < DV / 8; ++i) {
       const int col = i * 8 + (lane & 3) * 2;
-      *reinterpret_cast<float2*>(sO + (warp * 16 + row_a) * D + col) = make_float2(o[i][0], o[i][1]);
-      *reinterpret_cast<float2*>(sO + (warp * 16 + row_b) * D + col) = make_float2(o[i][2], o[i][3]);
+      *reinterpret_cast<float2*>(sO + (warp * 16 + row_a) * DV + col) = make_float2(o[i][0], o[i][1]);
+      *reinterpret_cast<float2*>(sO + (warp * 16 + row_b) * DV + col) = make_float2(o[i][2], o[i][3]);
     }
     if ((lane & 3) == 0) {
       sM[warp * 16 + row_a] = m_run[0]; sL[warp * 16 + row_a] = l_run[0];
@@ -293,18 +325,20 @@ __global__ void __launch_bounds__(160) decode_attn_tma_kernel(const __grid_const
       float w2 = (sM[32 + r] == -INFINITY) ? 0.f : exp2f(sM[32 + r] - m);
       float w3 = (sM[48 + r] == -INFINITY) ? 0.f : exp2f(sM[48 + r] - m);
       const float l = w0 * sL[r] + w1 * sL[16 + r] + w2 * sL[32 + r] + w3 * sL[48 + r];
-      const float inv = l > 0.f ? 1.f / l : 0.f;
       const int qt = r / group, g = r % group;
       const int hq = kvh * group + g;
+      float den = l;                              // the sink joins once: here, or in the merge of the splits
+      if (EXT && p.sinks && p.num_splits == 1 && m != -INFINITY) den += exp2f(p.sinks[hq] * kL2e - m);
+      const float inv = den > 0.f ? 1.f / den : 0.f;
       const size_t tok = size_t(q_start + qt);
-      for (int c = lane * 2; c < D; c += 64) {
-        const float a = w0 * sO[r * D + c] + w1 * sO[(16 + r) * D + c] + w2 * sO[(32 + r) * D + c] + w3 * sO[(48 + r) * D + c];
-        const float b = w0 * sO[r * D + c + 1] + w1 * sO[(16 + r) * D + c + 1] + w2 * sO[(32 + r) * D + c + 1] +
-                        w3 * sO[(48 + r) * D + c + 1];
+      for (int c = lane * 2; c < dv; c += 64) {
+        const float a = w0 * sO[r * DV + c] + w1 * sO[(16 + r) * DV + c] + w2 * sO[(32 + r) * DV + c] + w3 * sO[(48 + r) * DV + c];
+        const float b = w0 * sO[r * DV + c + 1] + w1 * sO[(16 + r) * DV + c + 1] + w2 * sO[(32 + r) * DV + c + 1] +
+                        w3 * sO[(48 + r) * DV + c + 1];
         if (p.num_splits == 1) {
-          *reinterpret_cast<uint32_t*>(p.out + tok * (size_t(p.n_q) * D) + hq * D + c) = pack_bf16x2(a * inv, b * inv);
+          *reinterpret_cast<uint32_t*>(p.out + tok * (size_t(p.n_q) * dv) + hq * dv + c) = pack_bf16x2(a * inv, b * inv);
         } else {
-          float* po = p.part_o + ((tok * p.n_q + hq) * p.num_splits + split) * D;
+          float* po = p.part_o + ((tok * p.n_q + hq) * p.num_splits + split) * dv;
           *reinterpret_cast<float2*>(po + c) = make_float2(a * inv, b * inv);
         }
       }
@@ -365,15 +399,15 @@ XL_API int xl_decode_attention_tma_dyn(const void* q, const void* k_cache, const
     const size_t merge = 4 * 16 * 128 * 4 + 128 * 4;
     const size_t smem = (ring > merge ? ring : merge) + 16 * 128 * 2 + sizeof(DecBarriers) + 1024;
     static bool set = false;
-    if (!set) { cudaFuncSetAttribute(decode_attn_tma_kernel<128>, cudaFuncAttributeMaxDynamicSharedMemorySize, int(smem)); set = true; }
-    decode_attn_tma_kernel<128><<<grid, 160, smem, st>>>(*tk, *tv, p);
+    if (!set) { cudaFuncSetAttribute(decode_attn_tma_kernel<128, 128, false>, cudaFuncAttributeMaxDynamicSharedMemorySize, int(smem)); set = true; }
+    decode_attn_tma_kernel<128, 128, false><<<grid, 160, smem, st>>>(*tk, *tv, p);
   } else {
     const size_t ring = size_t(kStages) * 2 * 1 * kTile * 128;
     const size_t merge = 4 * 16 * 64 * 4 + 128 * 4;
     const size_t smem = (ring > merge ? ring : merge) + 16 * 64 * 2 + sizeof(DecBarriers) + 1024;
     static bool set = false;
-    if (!set) { cudaFuncSetAttribute(decode_attn_tma_kernel<64>, cudaFuncAttributeMaxDynamicSharedMemorySize, int(smem)); set = true; }
-    decode_attn_tma_kernel<64><<<grid, 160, smem, st>>>(*tk, *tv, p);
+    if (!set) { cudaFuncSetAttribute(decode_attn_tma_kernel<64, 64, false>, cudaFuncAttributeMaxDynamicSharedMemorySize, int(smem)); set = true; }
+    decode_attn_tma_kernel<64, 64, false><<<grid, 160, smem, st>>>(*tk, *tv, p);
   }
   return cudaGetLastError() == cudaSuccess ? 0 : -1;
 }
@@ -462,6 +496,106 @@ XL_API int xl_decode_split_merge_dyn(const void* part_o, const void* part_lse, v
 XL_API int xl_decode_split_merge(const void* part_o, const void* part_lse, void* out, const void* q_cu, int seq_begin,
                                  int seq_end, int n_q, int head_dim, int splits, long max_rows, void* stream) {
   return xl_decode_split_merge_dyn(part_o, part_lse, out, q_cu, seq_begin, seq_end, n_q, head_dim, splits, max_rows, nullptr, stream);
+}
+
+// ============================================================================ score extensions
+namespace xl_dec {
+template <int DK, int DV>
+static int launch_ext(const CUtensorMap* tk, const CUtensorMap* tv, const DecParams& p, dim3 grid, cudaStream_t st) {
+  const size_t ring = size_t(kStages) * (DK / 64 + DV / 64) * kTile * 128;
+  const size_t merge = 4 * 16 * DV * 4 + 128 * 4;
+  const size_t smem = (ring > merge ? ring : merge) + 16 * DK * 2 + sizeof(DecBarriers) + 1024;
+  static bool set = false;
+  if (!set) {
+    cudaFuncSetAttribute(decode_attn_tma_kernel<DK, DV, true>, cudaFuncAttributeMaxDynamicSharedMemorySize, int(smem));
+    set = true;
+  }
+  decode_attn_tma_kernel<DK, DV, true><<<grid, 160, smem, st>>>(*tk, *tv, p);
+  return cudaGetLastError() == cudaSuccess ? 0 : -1;
+}
+
+// merge of split-KV partials for any value head dimension, with the sink's share of the denominator: one warp per
+// (token, head)
+__global__ void split_merge_ext_kernel(const float* __restrict__ part_o, const float* __restrict__ part_lse,
+                                       __nv_bfloat16* __restrict__ out, const int* __restrict__ q_cu, int seq_begin, int seq_end,
+                                       int n_q, int dv, int splits, const float* __restrict__ sinks, const int* dyn_end) {
+  const int lane = threadIdx.x & 31;
+  const long gw = (blockIdx.x * long(blockDim.x) + threadIdx.x) >> 5;
+  if (dyn_end) seq_end = *dyn_end;
+  if (seq_end <= seq_begin) return;
+  const int t0 = q_cu[seq_begin], t1 = q_cu[seq_end];
+  if (gw >= long(t1 - t0) * n_q) return;
+  const size_t tok = size_t(t0) + size_t(gw / n_q);
+  const int h = int(gw % n_q);
+  const float* lse = part_lse + (tok * n_q + h) * splits;
+  const float sink = sinks ? sinks[h] * 1.4426950408889634f : -INFINITY;
+  float m = sink;
+  for (int s = 0; s < splits; ++s) m = fmaxf(m, lse[s]);
+  float den = sinks ? exp2f(sink - m) : 0.f;
+  for (int s = 0; s < splits; ++s) den += lse[s] == -INFINITY ? 0.f : exp2f(lse[s] - m);
+  const float inv = den > 0.f ? 1.f / den : 0.f;
+  for (int c = lane; c < dv; c += 32) {
+    float acc = 0.f;
+    for (int s = 0; s < splits; ++s) {
+      const float w = lse[s] == -INFINITY ? 0.f : exp2f(lse[s] - m);
+      if (w != 0.f) acc += w * part_o[((tok * n_q + h) * splits + s) * dv + c];
+    }
+    out[tok * (size_t(n_q) * dv) + h * dv + c] = __float2bfloat16(acc * inv);
+  }
+}
+}  // namespace xl_dec
+
+// Decode attention with the score extensions of xl_prefill_attention_ext (head dimensions: multiples of 8, at most 128).
+// With num_splits > 1 the partials are merged by a second kernel; `max_rows` bounds the query tokens of the launch.
+XL_API int xl_decode_attention_ext(const void* q, const void* k_cache, const void* v_cache, void* out, const void* q_cu,
+                                   const void* kv_lens, const void* block_tables, int seq_begin, int seq_end, int max_blocks,
+                                   int block_size, int num_blocks_total, int n_q, int n_kv, int dk, int dv, int q_stride,
+                                   float scale, int window, int chunk, const void* slopes, const void* sinks, int num_splits,
+                                   void* part_o, void* part_lse, long max_rows, const void* dyn_end, void* stream) {
+  using namespace xl_dec;
+  if (seq_end <= seq_begin) return 0;
+  if (dk < 8 || dk > 128 || dk % 8 || dv < 8 || dv > 128 || dv % 8) return -3;
+  if (block_size % 16 != 0 || (block_size > 64 && block_size % 64 != 0) || (block_size < 64 && 64 % block_size != 0)) return -3;
+  if (n_q % n_kv || n_q / n_kv > 16) return -3;
+  if ((q_stride % 8) || (reinterpret_cast<uintptr_t>(q) & 15)) return -3;
+  if ((reinterpret_cast<uintptr_t>(k_cache) & 127) || (reinterpret_cast<uintptr_t>(v_cache) & 127)) return -3;
+  const int box_tokens = block_size < 64 ? block_size : 64;
+  const uint64_t slots = uint64_t(num_blocks_total) * block_size;
+  const CUtensorMap* tk = xl_host::tmap_3d(k_cache, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 2, slots, n_kv, dk, box_tokens, 1, 64,
+                                           CU_TENSOR_MAP_SWIZZLE_128B);
+  const CUtensorMap* tv = xl_host::tmap_3d(v_cache, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 2, slots, n_kv, dv, box_tokens, 1, 64,
+                                           CU_TENSOR_MAP_SWIZZLE_128B);
+  if (!tk || !tv) return -3;
+  DecParams p;
+  p.q = static_cast<const __nv_bfloat16*>(q);
+  p.out = static_cast<__nv_bfloat16*>(out);
+  p.q_cu = static_cast<const int*>(q_cu);
+  p.kv_lens = static_cast<const int*>(kv_lens);
+  p.block_tables = static_cast<const int*>(block_tables);
+  p.seq_begin = seq_begin; p.seq_end = seq_end;
+  p.max_blocks = max_blocks; p.block_size = block_size; p.n_q = n_q; p.n_kv = n_kv; p.q_stride = q_stride;
+  p.scale_log2 = scale * 1.4426950408889634f;
+  p.window = window;
+  p.num_splits = num_splits < 1 ? 1 : num_splits;
+  p.part_o = static_cast<float*>(part_o);
+  p.part_lse = static_cast<float*>(part_lse);
+  p.num_blocks_total = num_blocks_total;
+  p.box_tokens = box_tokens;
+  p.status = xl_host::status_word();
+  p.dyn_end = static_cast<const int*>(dyn_end);
+  p.dk = dk; p.dv = dv; p.chunk = chunk;
+  p.slopes = static_cast<const float*>(slopes);
+  p.sinks = static_cast<const float*>(sinks);
+  if (p.num_splits > 1 && (!part_o || !part_lse)) return -2;
+  cudaStream_t st = static_cast<cudaStream_t>(stream);
+  const dim3 grid(seq_end - seq_begin, n_kv, p.num_splits);
+  int rc;
+  if (dk > 64) rc = dv > 64 ? launch_ext<128, 128>(tk, tv, p, grid, st) : launch_ext<128, 64>(tk, tv, p, grid, st);
+  else rc = dv > 64 ? launch_ext<64, 128>(tk, tv, p, grid, st) : launch_ext<64, 64>(tk, tv, p, grid, st);
+  if (rc != 0 || p.num_splits == 1) return rc;
+  split_merge_ext_kernel<<<int((max_rows * n_q + 3) / 4), 128, 0, st>>>(p.part_o, p.part_lse, p.out, p.q_cu, seq_begin, seq_end, n_q, dv,
+                                                                        p.num_splits, p.sinks, p.dyn_end);
+  return cudaGetLastError() == cudaSuccess ? 0 : -1;
 }
 
 // ============================================================================ allocation-free entry point
@@ -555,16 +689,16 @@ XL_API int xl_decode_attention_noalloc(const void* q, const void* k_cache, const
   if (head_dim == 128) {
     const size_t ring = size_t(kStages) * 2 * 2 * kTile * 128;
     const size_t smem = ring + 16 * 128 * 2 + sizeof(DecBarriers) + 1024;
-    cudaFuncSetAttribute(decode_attn_tma_kernel<128>, cudaFuncAttributeMaxDynamicSharedMemorySize, int(smem));
-    decode_attn_tma_kernel<128><<<grid, 160, smem, st>>>(tk, tv, p);
+    cudaFuncSetAttribute(decode_attn_tma_kernel<128, 128, false>, cudaFuncAttributeMaxDynamicSharedMemorySize, int(smem));
+    decode_attn_tma_kernel<128, 128, false><<<grid, 160, smem, st>>>(tk, tv, p);
     if (num_splits > 1)
       split_merge_kernel<128><<<int((long(max_rows) * n_q + 3) / 4), 128, 0, st>>>(p.part_o, p.part_lse, p.out, p.q_cu, 0, n_seqs, n_q,
                                                                                   num_splits, nullptr, p.ws_rows, n_q / n_kv, p.status);
   } else {
     const size_t ring = size_t(kStages) * 2 * 1 * kTile * 128;
     const size_t smem = ring + 16 * 64 * 2 + sizeof(DecBarriers) + 1024;
-    cudaFuncSetAttribute(decode_attn_tma_kernel<64>, cudaFuncAttributeMaxDynamicSharedMemorySize, int(smem));
-    decode_attn_tma_kernel<64><<<grid, 160, smem, st>>>(tk, tv, p);
+    cudaFuncSetAttribute(decode_attn_tma_kernel<64, 64, false>, cudaFuncAttributeMaxDynamicSharedMemorySize, int(smem));
+    decode_attn_tma_kernel<64, 64, false><<<grid, 160, smem, st>>>(tk, tv, p);
     if (num_splits > 1)
       split_merge_kernel<64><<<int((long(max_rows) * n_q + 3) / 4), 128, 0, st>>>(p.part_o, p.part_lse, p.out, p.q_cu, 0, n_seqs, n_q,
                                                                                  num_splits, nullptr, p.ws_rows, n_q / n_kv, p.status);

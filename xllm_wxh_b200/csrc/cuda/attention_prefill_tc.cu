@@ -16,6 +16,9 @@
 //                   shared-memory tile that the second MMA reads, O rescaled in TMEM only when a row maximum grew
 //                   by more than 2^8 (otherwise the stale maximum is kept, which is exact after the final division
 //                   by the row sum), final O / l stored as bf16.
+// Template parameters: QS / VS = 64-column slabs of the query-key / value head dimension (a dimension that does not fill
+// its slabs is padded with zeros by the TMA loads), EXT = score extensions: per-head linear distance bias, per-head sink
+// (a score that joins the denominator and has no value), chunk mask (a query sees keys of its own position chunk only).
 // QK^T of tile j+1 is issued before P V of tile j, so the tensor pipe works while the softmax warps are busy.
 // Every wait is bounded; on expiry the kernel records a status code and leaves.
 #include <string.h>
@@ -27,18 +30,18 @@ using namespace xl;
 
 constexpr int BQ = 128;          // query rows per CTA (= TMEM lanes)
 constexpr int BKV = 64;          // kv tokens per tile
-constexpr int D = 128;           // head dimension
-template <int NH> struct Cfg {
+constexpr int Q_SLAB = BQ * 128;               // 16 KB: [128 rows][64 columns]
+constexpr int KV_SLAB = BKV * 128;             // 8 KB: [64 tokens][64 columns]
+constexpr int P_BYTES = BQ * BKV * 2;          // 16 KB: [128][64] K-major
+template <int NH, int QS, int VS> struct Cfg {
   static constexpr int kStages = NH == 2 ? 4 : 5;
   static constexpr int kThreads = 64 + 128 * NH;
-  static constexpr uint32_t kTmemCols = NH == 2 ? 512 : 256;   // per head: S0, S1 (64 columns each) and O (128)
+  static constexpr uint32_t kTmemCols = NH == 2 ? 512 : 256;   // per head: S0, S1 (64 columns each) and O (up to 128)
+  static constexpr int DK = 64 * QS, DV = 64 * VS;             // padded head dimensions
+  static constexpr int Q_BYTES = QS * Q_SLAB;
+  static constexpr int K_BYTES = QS * KV_SLAB, V_BYTES = VS * KV_SLAB;
+  static constexpr int STAGE_BYTES = K_BYTES + V_BYTES;        // K then V
 };
-constexpr int Q_BYTES = BQ * D * 2;            // 32 KB: two 64-column slabs of [128][64]
-constexpr int Q_SLAB = BQ * 128;               // 16 KB
-constexpr int KV_SLAB = BKV * 128;             // 8 KB: [64 tokens][64 columns]
-constexpr int K_BYTES = 2 * KV_SLAB;           // 16 KB
-constexpr int STAGE_BYTES = 2 * K_BYTES;       // K then V
-constexpr int P_BYTES = BQ * BKV * 2;          // 16 KB: [128][64] K-major
 constexpr int kMaxStages = 5;
 
 struct Barriers {
@@ -54,7 +57,11 @@ struct Barriers {
 };
 
 struct Params {
-  __nv_bfloat16* out;          // [T, Hq*D]
+  __nv_bfloat16* out;          // [T, Hq*dv]
+  int dv;                      // value head dimension (<= 64 * VS)
+  const float* slopes;         // EXT: [Hq] distance-bias slopes (null: none): score -= slope * (query pos - key pos)
+  const float* sinks;          // EXT: [Hq] sink scores (null: none): denominator += exp(sink)
+  int chunk;                   // EXT: positions per chunk (<= 0: no chunk mask)
   const int* q_cu;
   const int* kv_lens;
   const int* block_tables;
@@ -106,12 +113,14 @@ __device__ __forceinline__ float fast_exp2(float x) {
   return y;
 }
 
-template <int NH>
-__global__ void __launch_bounds__(Cfg<NH>::kThreads, 1)
+template <int NH, int QS, int VS, bool EXT>
+__global__ void __launch_bounds__(Cfg<NH, QS, VS>::kThreads, 1)
 prefill_attn_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__ CUtensorMap tmK,
                        const __grid_constant__ CUtensorMap tmV, const Params p) {
-  constexpr int kStages = Cfg<NH>::kStages;
-  constexpr uint32_t kTmemCols = Cfg<NH>::kTmemCols;
+  using C = Cfg<NH, QS, VS>;
+  constexpr int kStages = C::kStages;
+  constexpr uint32_t kTmemCols = C::kTmemCols;
+  constexpr int DK = C::DK, DV = C::DV, Q_BYTES = C::Q_BYTES, K_BYTES = C::K_BYTES, STAGE_BYTES = C::STAGE_BYTES;
   // The swizzled tiles need a 1024-byte aligned base, which the declared alignment of the dynamic array provides;
   // a CTA that finds it otherwise reports and leaves.
   extern __shared__ __align__(1024) uint8_t smem[];
@@ -154,6 +163,7 @@ prefill_attn_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_con
   const int kv_end = min(kv_len, pos0 + rows);
   int kv_begin = 0;
   if (p.window > 0) kv_begin = max(0, pos0 - p.window + 1) / BKV * BKV;
+  if (EXT && p.chunk > 0) kv_begin = max(kv_begin, pos0 / p.chunk * p.chunk / BKV * BKV);
   const int n_tiles_all = (kv_end - kv_begin + BKV - 1) / BKV;
   // this CTA's share of the key tiles (all of them without a split); short key ranges are left whole
   int n_eff = 1;
@@ -201,14 +211,18 @@ prefill_attn_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_con
       mbar_arrive_expect_tx(&bars->q_full, NH * Q_BYTES);
 #pragma unroll
       for (int h = 0; h < NH; ++h) {
-        tma_load_2d(sQ + h * Q_BYTES, &tmQ, &bars->q_full, (head0 + h) * D, q_start + q0);
-        tma_load_2d(sQ + h * Q_BYTES + Q_SLAB, &tmQ, &bars->q_full, (head0 + h) * D + 64, q_start + q0);
+#pragma unroll
+        for (int sl = 0; sl < QS; ++sl) {
+          if (EXT) tma_load_3d(sQ + h * Q_BYTES + sl * Q_SLAB, &tmQ, &bars->q_full, sl * 64, head0 + h, q_start + q0);
+          else tma_load_2d(sQ + h * Q_BYTES + sl * Q_SLAB, &tmQ, &bars->q_full, (head0 + h) * DK + sl * 64, q_start + q0);
+        }
       }
     }
     const int boxes = BKV / p.box_tokens;            // boxes per 64-token slab (1, 2 or 4)
-    const int per_tile = boxes * 4;                  // x 2 slabs x {K, V}
-    const int which = lane / (boxes * 2);            // 0 = K, 1 = V
-    const int slab = (lane / boxes) & 1;
+    const int per_tile = boxes * (QS + VS);          // x slabs of K, then of V
+    const int sl_all = lane / boxes;
+    const int which = sl_all >= QS ? 1 : 0;          // 0 = K, 1 = V
+    const int slab = which ? sl_all - QS : sl_all;
     const int bx = lane % boxes;
     bool ok = true;
     for (int j = 0; j < n_tiles && ok; ++j) {
@@ -243,7 +257,7 @@ prefill_attn_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_con
     // ------------------------------------------------------------ MMA issuer
     if (elect_one_sync()) {
       const uint32_t idesc_s = umma_idesc_f16(BQ, BKV, 1);
-      const uint32_t idesc_o = umma_idesc_f16(BQ, D, 1) | (1u << 16);       // B operand (V) is MN-major
+      const uint32_t idesc_o = umma_idesc_f16(BQ, DV, 1) | (1u << 16);       // B operand (V) is MN-major
       const uint32_t q_addr = smem_u32(sQ), p_addr = smem_u32(sP);
       bool ok = mbar_wait(&bars->q_full, 0);
       if (!ok) atomicExch(p.status, XL_ERR_WAIT_FULL);
@@ -282,7 +296,7 @@ prefill_attn_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_con
           }
           tc_fence_after();
 #pragma unroll
-          for (int k = 0; k < D / 16; ++k)
+          for (int k = 0; k < DK / 16; ++k)
             tc_mma_f16(tmem_base + h * 256 + b * 64, umma_desc_sw128(q_addr + h * Q_BYTES + (k >> 2) * Q_SLAB, (k & 3) * 32),
                        umma_desc_sw128(k_addr + (k >> 2) * KV_SLAB, (k & 3) * 32), idesc_s, k != 0);
           tc_commit(&bars->s_full[h][b]);
@@ -301,8 +315,12 @@ prefill_attn_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_con
     uint8_t* prow = sP + h * P_BYTES + r * 128;
     const int pos = pos0 + r;
     const int hi = min(pos, kv_len - 1);                     // last visible kv index of this row
-    const int lo = p.window > 0 ? max(0, pos - p.window + 1) : 0;
-    const float sc = p.scale_log2;
+    int lo = p.window > 0 ? max(0, pos - p.window + 1) : 0;
+    if (EXT && p.chunk > 0) lo = max(lo, pos / p.chunk * p.chunk);
+    const int lo_last = EXT && p.chunk > 0 ? (pos0 + BQ - 1) / p.chunk * p.chunk : 0;   // first key that every row's chunk may hold
+    const float slope2 = EXT && p.slopes ? p.slopes[head0 + h] * 1.4426950408889634f : 0.f;
+    // with the extensions v[] holds finished scores in the log2 domain, otherwise raw products that `sc` scales
+    const float sc = EXT ? 1.f : p.scale_log2;
     float m_ref = -INFINITY, l_run = 0.f;                    // m_ref: reference maximum of the raw scores
     bool ok = true;
     for (int j = 0; j < n_tiles && ok; ++j) {
@@ -321,12 +339,17 @@ prefill_attn_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_con
       __syncwarp();
       if (lane == 0) mbar_arrive(&bars->s_free[h][b]);
       const int kv0 = kv_begin + j * BKV;
-      const bool need_mask = (kv0 + BKV - 1 > pos0) || (kv0 + BKV > kv_len) || (p.window > 0);
+      const bool need_mask = (kv0 + BKV - 1 > pos0) || (kv0 + BKV > kv_len) || (p.window > 0) || (EXT && kv0 < lo_last);
       float v[64];
 #pragma unroll
       for (int c = 0; c < 32; ++c) {
         v[c] = __uint_as_float(s0[c]);
         v[32 + c] = __uint_as_float(s1[c]);
+      }
+      if (EXT) {
+        const float b0 = slope2 * float(kv0 - pos);
+#pragma unroll
+        for (int c = 0; c < 64; ++c) v[c] = fmaf(v[c], p.scale_log2, fmaf(slope2, float(c), b0));
       }
       if (need_mask) {
 #pragma unroll
@@ -368,7 +391,7 @@ prefill_attn_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_con
       tc_fence_after();
       if (j > 0 && __any_sync(0xffffffffu, rescale)) {
 #pragma unroll
-        for (int c = 0; c < D; c += 32) {
+        for (int c = 0; c < DV; c += 32) {
           uint32_t o[32];
           tmem_ld_32x32(t_o + c, o);
           tc_wait_ld();
@@ -397,9 +420,9 @@ prefill_attn_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_con
       // partial of this key range: O relative to m_ref, with m_ref and the row sum beside it
       tc_fence_after();
       const size_t unit = (size_t(tile_ord) * gridDim.y + blockIdx.y) * NH + h;
-      float4* wo = reinterpret_cast<float4*>(p.ws_o) + (unit * p.splits + blockIdx.z) * (D / 4) * BQ;
+      float4* wo = reinterpret_cast<float4*>(p.ws_o) + (unit * p.splits + blockIdx.z) * (DV / 4) * BQ;
 #pragma unroll
-      for (int c = 0; c < D; c += 32) {
+      for (int c = 0; c < DV; c += 32) {
         uint32_t o[32];
         tmem_ld_32x32(t_o + c, o);
         tc_wait_ld();
@@ -412,10 +435,12 @@ prefill_attn_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_con
       __threadfence();
     } else if (ok) {
       tc_fence_after();
+      if (EXT && p.sinks && m_ref != -INFINITY) l_run += fast_exp2(p.sinks[head0 + h] * 1.4426950408889634f - m_ref);
       const float inv = l_run > 0.f ? 1.f / l_run : 0.f;
-      __nv_bfloat16* dst = p.out + size_t(q_start + q0 + r) * (size_t(p.n_q) * D) + (head0 + h) * D;
+      const int dv = EXT ? p.dv : DV;
+      __nv_bfloat16* dst = p.out + size_t(q_start + q0 + r) * (size_t(p.n_q) * dv) + (head0 + h) * dv;
 #pragma unroll
-      for (int c = 0; c < D; c += 32) {
+      for (int c = 0; c < DV; c += 32) {
         uint32_t o[32];
         tmem_ld_32x32(t_o + c, o);
         tc_wait_ld();
@@ -426,7 +451,7 @@ prefill_attn_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_con
 #pragma unroll
             for (int e = 0; e < 4; ++e)
               w[e] = pack_bf16x2(__uint_as_float(o[8 * i + 2 * e]) * inv, __uint_as_float(o[8 * i + 2 * e + 1]) * inv);
-            *reinterpret_cast<uint4*>(dst + c + 8 * i) = make_uint4(w[0], w[1], w[2], w[3]);
+            if (!EXT || c + 8 * i < dv) *reinterpret_cast<uint4*>(dst + c + 8 * i) = make_uint4(w[0], w[1], w[2], w[3]);
           }
         }
       }
@@ -474,16 +499,18 @@ prefill_attn_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_con
         l_all += w[z] * v.y;
       }
     }
+    if (EXT && p.sinks && m_all != -INFINITY) l_all += fast_exp2(p.sinks[head0 + h] * 1.4426950408889634f - m_all);
     const float inv = l_all > 0.f ? 1.f / l_all : 0.f;
     if (r < rows) {
-      const float4* wo = reinterpret_cast<const float4*>(p.ws_o) + unit * p.splits * (D / 4) * BQ + r;
-      __nv_bfloat16* dst = p.out + size_t(q_start + q0 + r) * (size_t(p.n_q) * D) + (head0 + h) * D;
-      for (int c4 = 0; c4 < D / 4; c4 += 2) {
+      const int dv = EXT ? p.dv : DV;
+      const float4* wo = reinterpret_cast<const float4*>(p.ws_o) + unit * p.splits * (DV / 4) * BQ + r;
+      __nv_bfloat16* dst = p.out + size_t(q_start + q0 + r) * (size_t(p.n_q) * dv) + (head0 + h) * dv;
+      for (int c4 = 0; c4 < dv / 4; c4 += 2) {
         float4 a = make_float4(0.f, 0.f, 0.f, 0.f), b = a;
 #pragma unroll
         for (int z = 0; z < 8; ++z) {
           if (z < n_valid && w[z] != 0.f) {
-            const float4 x = __ldcg(wo + (size_t(z) * (D / 4) + c4) * BQ), y = __ldcg(wo + (size_t(z) * (D / 4) + c4 + 1) * BQ);
+            const float4 x = __ldcg(wo + (size_t(z) * (DV / 4) + c4) * BQ), y = __ldcg(wo + (size_t(z) * (DV / 4) + c4 + 1) * BQ);
             a.x += w[z] * x.x; a.y += w[z] * x.y; a.z += w[z] * x.z; a.w += w[z] * x.w;
             b.x += w[z] * y.x; b.y += w[z] * y.y; b.z += w[z] * y.z; b.w += w[z] * y.w;
           }
@@ -515,13 +542,14 @@ static uint8_t* split_workspace(cudaStream_t stream) {
   return ws[dev];
 }
 
-template <int NH>
+template <int NH, int QS, int VS, bool EXT>
 static int launch_prefill(const CUtensorMap* tq, const CUtensorMap* tk, const CUtensorMap* tv, const Params& p_in, int q_tiles_cap,
                           int total_q_rows, cudaStream_t stream) {
-  const size_t smem = size_t(NH) * (Q_BYTES + P_BYTES) + Cfg<NH>::kStages * STAGE_BYTES + sizeof(Barriers);
+  using C = Cfg<NH, QS, VS>;
+  const size_t smem = size_t(NH) * (C::Q_BYTES + P_BYTES) + C::kStages * C::STAGE_BYTES + sizeof(Barriers);
   static bool set = false;
   if (!set) {
-    cudaFuncSetAttribute(prefill_attn_tc_kernel<NH>, cudaFuncAttributeMaxDynamicSharedMemorySize, int(smem));
+    cudaFuncSetAttribute(prefill_attn_tc_kernel<NH, QS, VS, EXT>, cudaFuncAttributeMaxDynamicSharedMemorySize, int(smem));
     set = true;
   }
   Params p = p_in;
@@ -539,7 +567,7 @@ static int launch_prefill(const CUtensorMap* tq, const CUtensorMap* tk, const CU
   p.ws_tiles = 0;
   if (splits > 1) {
     uint8_t* w = split_workspace(stream);
-    const size_t per_tile = size_t(p.n_q) * splits * (size_t(BQ) * D * 4 + size_t(BQ) * 8);
+    const size_t per_tile = size_t(p.n_q) * splits * (size_t(BQ) * C::DV * 4 + size_t(BQ) * 8);
     size_t tiles = kSplitWsBytes / per_tile;
     const size_t cnt_cap = kSplitCntBytes / 4 / size_t(p.n_q / NH);
     if (tiles > cnt_cap) tiles = cnt_cap;
@@ -547,12 +575,12 @@ static int launch_prefill(const CUtensorMap* tq, const CUtensorMap* tk, const CU
       p.splits = splits;
       p.ws_tiles = int(tiles < size_t(q_tiles_cap) ? tiles : size_t(q_tiles_cap));
       p.ws_o = reinterpret_cast<float*>(w);
-      p.ws_ml = reinterpret_cast<float2*>(w + size_t(p.ws_tiles) * p.n_q * splits * size_t(BQ) * D * 4);
+      p.ws_ml = reinterpret_cast<float2*>(w + size_t(p.ws_tiles) * p.n_q * splits * size_t(BQ) * C::DV * 4);
       p.ws_cnt = reinterpret_cast<int*>(w + kSplitWsBytes);
     }
   }
   dim3 grid(q_tiles_cap, p.n_q / NH, p.splits);
-  prefill_attn_tc_kernel<NH><<<grid, Cfg<NH>::kThreads, smem, stream>>>(*tq, *tk, *tv, p);
+  prefill_attn_tc_kernel<NH, QS, VS, EXT><<<grid, C::kThreads, smem, stream>>>(*tq, *tk, *tv, p);
   return cudaGetLastError() == cudaSuccess ? 0 : -1;
 }
 
@@ -570,6 +598,7 @@ XL_API int xl_prefill_attention_tc(const void* q, const void* k_cache, const voi
                                    int total_q_rows, float scale, int window, int q_tiles_cap, const void* dyn_begin,
                                    const void* dyn_end, void* stream) {
   using namespace xl_pf;
+  constexpr int D = 128;
   if (head_dim != D) return -3;
   if (block_size % 16 != 0 || (block_size > 64 && block_size % 64 != 0) || (block_size < 64 && 64 % block_size != 0)) return -3;
   if (n_q % n_kv) return -3;
@@ -600,6 +629,58 @@ XL_API int xl_prefill_attention_tc(const void* q, const void* k_cache, const voi
   p.window = window;
   p.status = xl_host::status_word();
   cudaStream_t st = static_cast<cudaStream_t>(stream);
-  if ((n_q / n_kv) % 2 == 0) return launch_prefill<2>(tq, tk, tv, p, q_tiles_cap, total_q_rows, st);
-  return launch_prefill<1>(tq, tk, tv, p, q_tiles_cap, total_q_rows, st);
+  if ((n_q / n_kv) % 2 == 0) return launch_prefill<2, 2, 2, false>(tq, tk, tv, p, q_tiles_cap, total_q_rows, st);
+  return launch_prefill<1, 2, 2, false>(tq, tk, tv, p, q_tiles_cap, total_q_rows, st);
+}
+
+// The same with the score extensions and separate query-key / value head dimensions (multiples of 8, at most 128):
+//   score(i, j) = scale * q_i . k_j - slopes[h] * (i - j), visible when j <= i, within `window` (> 0) and in the same
+//   chunk of `chunk` positions (> 0); out = sum_j exp(score) v_j / (sum_j exp(score) + exp(sinks[h])).
+// `slopes` / `sinks` [n_q] fp32, null when absent.  Returns -3 when the shape is not covered.
+XL_API int xl_prefill_attention_ext(const void* q, const void* k_cache, const void* v_cache, void* out, const void* q_cu,
+                                    const void* kv_lens, const void* block_tables, int seq_begin, int seq_end, int max_blocks,
+                                    int block_size, int num_blocks_total, int n_q, int n_kv, int dk, int dv, int q_stride,
+                                    int total_q_rows, float scale, int window, int chunk, const void* slopes, const void* sinks,
+                                    int q_tiles_cap, const void* dyn_begin, const void* dyn_end, void* stream) {
+  using namespace xl_pf;
+  if (dk < 8 || dk > 128 || dk % 8 || dv < 8 || dv > 128 || dv % 8) return -3;
+  if (block_size % 16 != 0 || (block_size > 64 && block_size % 64 != 0) || (block_size < 64 && 64 % block_size != 0)) return -3;
+  if (n_q % n_kv) return -3;
+  if ((q_stride % 8) || (reinterpret_cast<uintptr_t>(q) & 15) || (reinterpret_cast<uintptr_t>(out) & 15)) return -3;
+  if ((reinterpret_cast<uintptr_t>(k_cache) & 127) || (reinterpret_cast<uintptr_t>(v_cache) & 127)) return -3;
+  if (q_tiles_cap <= 0 || seq_end <= seq_begin) return 0;
+  const int box_tokens = block_size < 64 ? block_size : 64;
+  const uint64_t slots = uint64_t(num_blocks_total) * block_size;
+  // boxes of 64 columns: columns past the head dimension come back as zeros and add nothing to the products
+  const CUtensorMap* tq = xl_host::tmap_3d(q, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 2, total_q_rows, n_q, dk, BQ, 1, 64,
+                                           CU_TENSOR_MAP_SWIZZLE_128B, q_stride);
+  const CUtensorMap* tk = xl_host::tmap_3d(k_cache, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 2, slots, n_kv, dk, box_tokens, 1, 64,
+                                           CU_TENSOR_MAP_SWIZZLE_128B);
+  const CUtensorMap* tv = xl_host::tmap_3d(v_cache, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 2, slots, n_kv, dv, box_tokens, 1, 64,
+                                           CU_TENSOR_MAP_SWIZZLE_128B);
+  if (!tq || !tk || !tv) return -3;
+  Params p;
+  memset(&p, 0, sizeof(p));
+  p.out = static_cast<__nv_bfloat16*>(out);
+  p.dv = dv;
+  p.slopes = static_cast<const float*>(slopes);
+  p.sinks = static_cast<const float*>(sinks);
+  p.chunk = chunk;
+  p.q_cu = static_cast<const int*>(q_cu);
+  p.kv_lens = static_cast<const int*>(kv_lens);
+  p.block_tables = static_cast<const int*>(block_tables);
+  p.seq_begin = seq_begin; p.seq_end = seq_end;
+  p.dyn_begin = static_cast<const int*>(dyn_begin);
+  p.dyn_end = static_cast<const int*>(dyn_end);
+  p.max_blocks = max_blocks; p.block_size = block_size; p.box_tokens = box_tokens; p.n_q = n_q; p.n_kv = n_kv;
+  p.num_slots = long(slots);
+  p.scale_log2 = scale * 1.4426950408889634f;
+  p.window = window;
+  p.status = xl_host::status_word();
+  cudaStream_t st = static_cast<cudaStream_t>(stream);
+  const bool pair = (n_q / n_kv) % 2 == 0, k2 = dk > 64, v2 = dv > 64;
+#define XL_PF_EXT(NH, QS, VS) launch_prefill<NH, QS, VS, true>(tq, tk, tv, p, q_tiles_cap, total_q_rows, st)
+  if (pair) return k2 ? (v2 ? XL_PF_EXT(2, 2, 2) : XL_PF_EXT(2, 2, 1)) : (v2 ? XL_PF_EXT(2, 1, 2) : XL_PF_EXT(2, 1, 1));
+  return k2 ? (v2 ? XL_PF_EXT(1, 2, 2) : XL_PF_EXT(1, 2, 1)) : (v2 ? XL_PF_EXT(1, 1, 2) : XL_PF_EXT(1, 1, 1));
+#undef XL_PF_EXT
 }

@@ -210,6 +210,15 @@ __device__ __forceinline__ float warp_max(float v) {
   for (int o = 16; o > 0; o >>= 1) v = fmaxf(v, __shfl_xor_sync(0xffffffffu, v, o));
   return v;
 }
+// Gate activations of a gated feed-forward: z * sigmoid(z), and the tanh form of gelu written with the identity
+// (1 + tanh(u)) / 2 = 1 / (1 + exp(-2u)), u = sqrt(2 / pi) (z + 0.044715 z^3).
+enum : int { ACT_SILU = 0, ACT_GELU_TANH = 1 };
+__device__ __forceinline__ float act_silu(float z) { return z / (1.f + __expf(-z)); }
+__device__ __forceinline__ float act_gelu_tanh(float z) {
+  const float u2 = -1.5957691216057308f * (z + 0.044715f * z * z * z);
+  return z / (1.f + __expf(u2));
+}
+__device__ __forceinline__ float gate_act(float z, int act) { return act == ACT_GELU_TANH ? act_gelu_tanh(z) : act_silu(z); }
 __device__ __forceinline__ uint32_t pack_bf16x2(float lo, float hi) {
   __nv_bfloat162 v = __floats2bfloat162_rn(lo, hi);
   return *reinterpret_cast<uint32_t*>(&v);
@@ -229,7 +238,7 @@ CUresult encode_tiled(CUtensorMap* map, CUtensorMapDataType dt, uint32_t rank, c
 const CUtensorMap* tmap_2d(const void* base, CUtensorMapDataType dt, int elem_bytes, uint64_t rows, uint64_t cols, uint64_t ld,
                            uint32_t box_rows, uint32_t box_cols, CUtensorMapSwizzle swz);
 const CUtensorMap* tmap_3d(const void* base, CUtensorMapDataType dt, int elem_bytes, uint64_t d2, uint64_t d1, uint64_t d0,
-                           uint32_t b2, uint32_t b1, uint32_t b0, CUtensorMapSwizzle swz);
+                           uint32_t b2, uint32_t b1, uint32_t b0, CUtensorMapSwizzle swz, uint64_t pitch = 0);
 int sm_count();
 int* status_word();   // device int, zero-initialised, one per process and device
 }  // namespace xl_host

@@ -33,7 +33,9 @@ struct GemmSmemBarriers {
   int abort_flag;
 };
 
-enum { EPI_NONE = 0, EPI_BIAS = 1, EPI_SWIGLU = 2, EPI_RS_PUSH = 3 };
+// EPI_GEGLU: as EPI_SWIGLU with the tanh form of gelu; EPI_F32: the accumulators are stored as fp32 (C is float).
+enum { EPI_NONE = 0, EPI_BIAS = 1, EPI_SWIGLU = 2, EPI_RS_PUSH = 3, EPI_GEGLU = 4, EPI_F32 = 5 };
+__host__ __device__ constexpr bool epi_gated(int epi) { return epi == EPI_SWIGLU || epi == EPI_GEGLU; }
 
 // EPI_RS_PUSH (tensor-parallel row-parallel linear): this rank's partial tile is not stored locally; each row is
 // pushed over NVLink straight from the epilogue registers into the receive buffer of the rank that owns the row
@@ -211,7 +213,7 @@ gemm_bf16_kernel(const __grid_constant__ CUtensorMap tmA, const __grid_constant_
         tc_wait_ld();
         const int width = (c + 32 <= BN) ? 32 : 16;
         const int n = n0 + c;
-        if (EPI == EPI_SWIGLU) {
+        if (epi_gated(EPI)) {
           // columns [0,16) gate, [16,32) up of output columns (n/2 .. n/2+16)
           if (row < row_lim && n < N) {
             uint32_t o[8];
@@ -219,13 +221,28 @@ gemm_bf16_kernel(const __grid_constant__ CUtensorMap tmA, const __grid_constant_
             for (int j = 0; j < 8; ++j) {
               float g0 = __uint_as_float(r[2 * j]), g1 = __uint_as_float(r[2 * j + 1]);
               float u0 = __uint_as_float(r[16 + 2 * j]), u1 = __uint_as_float(r[16 + 2 * j + 1]);
-              float a0 = g0 / (1.f + __expf(-g0)) * u0;
-              float a1 = g1 / (1.f + __expf(-g1)) * u1;
+              float a0 = (EPI == EPI_GEGLU ? act_gelu_tanh(g0) : act_silu(g0)) * u0;
+              float a1 = (EPI == EPI_GEGLU ? act_gelu_tanh(g1) : act_silu(g1)) * u1;
               o[j] = pack_bf16x2(a0, a1);
             }
             uint4* dst = reinterpret_cast<uint4*>(C + size_t(row - c_row_off) * ldc + c_col_off + (n >> 1));
             dst[0] = make_uint4(o[0], o[1], o[2], o[3]);
             dst[1] = make_uint4(o[4], o[5], o[6], o[7]);
+          }
+        } else if (EPI == EPI_F32) {
+          if (row < row_lim && n < N) {
+            float* dst = reinterpret_cast<float*>(C) + size_t(row - c_row_off) * ldc + c_col_off + n;
+            if (n + width <= N && (ldc & 3) == 0) {
+#pragma unroll
+              for (int j = 0; j < 8; ++j)
+                if (j * 4 < width)
+                  reinterpret_cast<float4*>(dst)[j] = make_float4(__uint_as_float(r[4 * j]), __uint_as_float(r[4 * j + 1]),
+                                                                  __uint_as_float(r[4 * j + 2]), __uint_as_float(r[4 * j + 3]));
+            } else {
+#pragma unroll
+              for (int j = 0; j < 32; ++j)
+                if (j < width && n + j < N) dst[j] = __uint_as_float(r[j]);
+            }
           }
         } else {
           if (row < row_lim && n < N) {
@@ -295,7 +312,7 @@ static double g_last_score = 0;
 static int pick_bn(int M, int N, int sms, int epi) {
   if (g_force_bn > 0) return g_force_bn;
   const int m_tiles = (M + kBM - 1) / kBM;
-  const int step = (epi == EPI_SWIGLU) ? 32 : 16;
+  const int step = epi_gated(epi) ? 32 : 16;
   int best = 128;
   double best_score = -1;
   for (int bn = 32; bn <= 256; bn += step) {
@@ -320,13 +337,13 @@ static int launch(const void* A, const void* W, void* C, const void* bias, int M
                   cudaStream_t stream, const RsPush* rs_in = nullptr, const Grouped* grp_in = nullptr, int num_experts = 1,
                   int max_m_tiles = 0) {
   if (M <= 0 || N <= 0 || K <= 0) return 0;
-  if ((lda % 8) || (ldw % 8) || (ldc % 8) || (reinterpret_cast<uintptr_t>(A) & 15) || (reinterpret_cast<uintptr_t>(W) & 15) ||
+  if ((lda % 8) || (ldw % 8) || (EPI != EPI_F32 && (ldc % 8)) || (reinterpret_cast<uintptr_t>(A) & 15) || (reinterpret_cast<uintptr_t>(W) & 15) ||
       ((EPI != EPI_RS_PUSH || (rs_in && rs_in->local)) && (reinterpret_cast<uintptr_t>(C) & 15)))
     return -2;  // TMA and 16-byte stores need 16-byte aligned rows
-  if (EPI == EPI_SWIGLU && (N % 32)) return -2;
+  if (epi_gated(EPI) && (N % 32)) return -2;
   const int sms = xl_host::sm_count();
   const int BN = pick_bn(M, N, sms, EPI);
-  if (!grp_in && g_mode != 1 && (M > kBM || K >= 2048) && g_force_bn == 0) {
+  if (EPI != EPI_F32 && !grp_in && g_mode != 1 && (M > kBM || K >= 2048) && g_force_bn == 0) {
     // A pair of CTAs per 256-row tile moves a third less shared-memory traffic per FLOP; it wins unless its coarser
     // tiles fill the SMs much worse than single-CTA tiles do.
     const double pair_score = xl_gemm_bf16_pair_score(EPI, M, N, K, !(EPI == EPI_RS_PUSH && !(rs_in && rs_in->local)));
@@ -347,7 +364,7 @@ static int launch(const void* A, const void* W, void* C, const void* bias, int M
   const CUtensorMap* tb = xl_host::tmap_2d(W, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 2, uint64_t(N) * num_experts, K, ldw, BN, kBK,
                                            CU_TENSOR_MAP_SWIZZLE_128B);
   if (!ta || !tb) return -4;
-  static bool attr_set[4] = {false, false, false, false};
+  static bool attr_set[6] = {false, false, false, false, false, false};
   RsPush rs;
   memset(&rs, 0, sizeof(rs));
   if (rs_in) rs = *rs_in;
@@ -381,9 +398,22 @@ XL_API int xl_gemm_bf16_swiglu(const void* A, const void* W, void* C, int M, int
   return xl::launch<xl::EPI_SWIGLU>(A, W, C, nullptr, M, N, K, lda, ldw, ldc, static_cast<cudaStream_t>(stream));
 }
 
+// Same with a chosen gate activation (ACT_SILU / ACT_GELU_TANH).
+XL_API int xl_gemm_bf16_gated(const void* A, const void* W, void* C, int M, int N, int K, int lda, int ldw, int ldc, int act,
+                              void* stream) {
+  if (act == xl::ACT_GELU_TANH)
+    return xl::launch<xl::EPI_GEGLU>(A, W, C, nullptr, M, N, K, lda, ldw, ldc, static_cast<cudaStream_t>(stream));
+  return xl::launch<xl::EPI_SWIGLU>(A, W, C, nullptr, M, N, K, lda, ldw, ldc, static_cast<cudaStream_t>(stream));
+}
+
+// fp32 C[M,N] = A[M,K] W[N,K]^T: the fp32 accumulators leave unrounded (router logits).
+XL_API int xl_gemm_bf16_f32(const void* A, const void* W, void* C, int M, int N, int K, int lda, int ldw, int ldc, void* stream) {
+  return xl::launch<xl::EPI_F32>(A, W, C, nullptr, M, N, K, lda, ldw, ldc, static_cast<cudaStream_t>(stream));
+}
+
 // Grouped GEMM over expert-sorted rows: C[r, :] = A[r, :] * W[expert(r)]^T for the rows listed in the tile table
 // (`tile_*` arrays and `num_m_tiles` live on the device; `max_m_tiles` bounds them for the launch).
-// swiglu != 0: W holds interleaved gate/up rows and C has N/2 columns.
+// swiglu != 0: W holds interleaved gate/up rows and C has N/2 columns (1: silu gate, 2: tanh-gelu gate).
 XL_API int xl_grouped_gemm_bf16(const void* A, const void* W, void* C, int M_cap, int N, int K, int lda, int ldc, int num_experts,
                                 const void* tile_expert, const void* tile_row0, const void* tile_row_end,
                                 const void* num_m_tiles, int max_m_tiles, int swiglu, int c_rows_per_expert, int c_col_stride,
@@ -397,6 +427,9 @@ XL_API int xl_grouped_gemm_bf16(const void* A, const void* W, void* C, int M_cap
   g.num_m_tiles = static_cast<const int*>(num_m_tiles);
   g.enabled = 1;
   if (max_m_tiles <= 0) return 0;
+  if (swiglu == 2)
+    return xl::launch<xl::EPI_GEGLU>(A, W, C, nullptr, M_cap, N, K, lda, K, ldc, static_cast<cudaStream_t>(stream), nullptr, &g,
+                                     num_experts, max_m_tiles);
   if (swiglu)
     return xl::launch<xl::EPI_SWIGLU>(A, W, C, nullptr, M_cap, N, K, lda, K, ldc, static_cast<cudaStream_t>(stream), nullptr, &g,
                                       num_experts, max_m_tiles);

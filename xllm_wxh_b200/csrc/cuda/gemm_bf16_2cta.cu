@@ -37,7 +37,8 @@ constexpr int kMaxStages = 8;
 constexpr int kThreads = 192;
 constexpr int kOutStageBytes = 4 * 2 * 2048;   // 4 epilogue warps x 2 buffers x (32 rows x 64 bytes)
 
-enum { EPI_NONE = 0, EPI_BIAS = 1, EPI_SWIGLU = 2, EPI_RS_PUSH = 3 };
+enum { EPI_NONE = 0, EPI_BIAS = 1, EPI_SWIGLU = 2, EPI_RS_PUSH = 3, EPI_GEGLU = 4 };
+__host__ __device__ constexpr bool epi_gated(int epi) { return epi == EPI_SWIGLU || epi == EPI_GEGLU; }
 
 struct Barriers {
   uint64_t full[kMaxStages];
@@ -146,12 +147,13 @@ __device__ __forceinline__ void emit_chunk(float (&v)[32], int row, int n, int w
                                            __nv_bfloat16* __restrict__ C, const __nv_bfloat16* __restrict__ bias,
                                            const RsPush& rs) {
   if (row >= M || n >= N) return;
-  if (EPI == EPI_SWIGLU) {
+  if (epi_gated(EPI)) {
     uint32_t o[8];
 #pragma unroll
     for (int j = 0; j < 8; ++j) {
       const float g0 = v[2 * j], g1 = v[2 * j + 1], u0 = v[16 + 2 * j], u1 = v[16 + 2 * j + 1];
-      o[j] = pack_bf16x2(g0 / (1.f + __expf(-g0)) * u0, g1 / (1.f + __expf(-g1)) * u1);
+      if (EPI == EPI_GEGLU) o[j] = pack_bf16x2(act_gelu_tanh(g0) * u0, act_gelu_tanh(g1) * u1);
+      else o[j] = pack_bf16x2(act_silu(g0) * u0, act_silu(g1) * u1);
     }
     uint4* dst = reinterpret_cast<uint4*>(C + size_t(row) * ldc + (n >> 1));
     dst[0] = make_uint4(o[0], o[1], o[2], o[3]);
@@ -200,12 +202,13 @@ __device__ __forceinline__ void store_chunk_tma(float (&v)[32], uint8_t* stage, 
   // the store issued two chunks ago read this buffer: it must be done with it
   if (lane == 0) tma_store_wait_read<1>();
   __syncwarp();
-  if (EPI == EPI_SWIGLU) {
+  if (epi_gated(EPI)) {
     uint32_t o[8];
 #pragma unroll
     for (int j = 0; j < 8; ++j) {
       const float g0 = v[2 * j], g1 = v[2 * j + 1], u0 = v[16 + 2 * j], u1 = v[16 + 2 * j + 1];
-      o[j] = pack_bf16x2(g0 / (1.f + __expf(-g0)) * u0, g1 / (1.f + __expf(-g1)) * u1);
+      if (EPI == EPI_GEGLU) o[j] = pack_bf16x2(act_gelu_tanh(g0) * u0, act_gelu_tanh(g1) * u1);
+      else o[j] = pack_bf16x2(act_silu(g0) * u0, act_silu(g1) * u1);
     }
     const int sw = (lane >> 2) & 1;                     // 32-byte swizzle: piece ^= address bit 7
     *reinterpret_cast<uint4*>(stage + lane * 32 + ((0 ^ sw) << 4)) = make_uint4(o[0], o[1], o[2], o[3]);
@@ -226,7 +229,7 @@ __device__ __forceinline__ void store_chunk_tma(float (&v)[32], uint8_t* stage, 
   fence_proxy_async_smem();
   __syncwarp();
   if (lane == 0) {
-    tma_store_2d(tmC, stage, EPI == EPI_SWIGLU ? (n >> 1) : n, row0);
+    tma_store_2d(tmC, stage, epi_gated(EPI) ? (n >> 1) : n, row0);
     tma_store_commit();
   }
 }
@@ -683,7 +686,7 @@ static int launch_pair(const void* A, const void* W, void* C, const void* bias, 
   // the rows stay in C (the row-push epilogue addresses other ranks' buffers per row).
   const CUtensorMap* tc = nullptr;
   if (g_tma_out && !pushes_rows && (reinterpret_cast<uintptr_t>(C) & 15) == 0 && (size_t(ldc) * 2) % 16 == 0) {
-    if (EPI == EPI_SWIGLU)
+    if (epi_gated(EPI))
       tc = xl_host::tmap_2d(C, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 2, M, N / 2, ldc, 32, 16, CU_TENSOR_MAP_SWIZZLE_32B);
     else
       tc = xl_host::tmap_2d(C, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 2, M, N, ldc, 32, 32, CU_TENSOR_MAP_SWIZZLE_64B);
@@ -723,7 +726,8 @@ static int launch_pair(const void* A, const void* W, void* C, const void* bias, 
 
 }  // namespace xl2
 
-// Entry points used by gemm_bf16.cu's dispatch.  `epi`: 0 none, 1 bias, 2 SwiGLU (interleaved W), 3 row push (TP).
+// Entry points used by gemm_bf16.cu's dispatch.  `epi`: 0 none, 1 bias, 2 SwiGLU (interleaved W), 3 row push (TP),
+// 4 gelu-gated (interleaved W).
 // `score` (may be null) receives the wave-fill score of the chosen tile width, comparable with the single-CTA one.
 extern "C" int xl_gemm_bf16_pair_launch(int epi, const void* A, const void* W, void* C, const void* bias, int M, int N, int K,
                                         int lda, int ldw, int ldc, void* stream, const void* rs) {
@@ -734,6 +738,7 @@ extern "C" int xl_gemm_bf16_pair_launch(int epi, const void* A, const void* W, v
     case 1: return xl2::launch_pair<xl2::EPI_BIAS>(A, W, C, bias, M, N, K, lda, ldw, ldc, st, nullptr);
     case 2: return xl2::launch_pair<xl2::EPI_SWIGLU>(A, W, C, bias, M, N, K, lda, ldw, ldc, st, nullptr);
     case 3: return xl2::launch_pair<xl2::EPI_RS_PUSH>(A, W, C, bias, M, N, K, lda, ldw, ldc, st, r);
+    case 4: return xl2::launch_pair<xl2::EPI_GEGLU>(A, W, C, bias, M, N, K, lda, ldw, ldc, st, nullptr);
   }
   return -2;
 }

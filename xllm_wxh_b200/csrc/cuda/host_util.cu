@@ -38,9 +38,10 @@ struct Key {
   uint64_t rows, cols, ld;
   uint32_t br, bc;
   int dt, swz;
+  uint64_t pitch = 0;
   bool operator==(const Key& o) const {
     return base == o.base && rows == o.rows && cols == o.cols && ld == o.ld && br == o.br && bc == o.bc && dt == o.dt &&
-           swz == o.swz;
+           swz == o.swz && pitch == o.pitch;
   }
 };
 struct KeyHash {
@@ -77,12 +78,14 @@ const CUtensorMap* tmap_2d(const void* base, CUtensorMapDataType dt, int elem_by
   return m;
 }
 
-// cached 3-D map of a [d2, d1, d0] row-major tensor (d0 innermost, contiguous), box = [b2, b1, b0]
+// cached 3-D map of a [d2, d1, d0] row-major tensor (d0 innermost, contiguous), box = [b2, b1, b0]; consecutive d2 slices
+// are `pitch` elements apart (0: d0 * d1)
 const CUtensorMap* tmap_3d(const void* base, CUtensorMapDataType dt, int elem_bytes, uint64_t d2, uint64_t d1, uint64_t d0,
-                           uint32_t b2, uint32_t b1, uint32_t b0, CUtensorMapSwizzle swz) {
+                           uint32_t b2, uint32_t b1, uint32_t b0, CUtensorMapSwizzle swz, uint64_t pitch) {
+  if (pitch == 0) pitch = d0 * d1;
   static std::mutex mu;
   static std::unordered_map<Key, CUtensorMap*, KeyHash> cache;
-  Key k{base, d2, d1 * 1000003ULL + b1, d0, b2, b0, int(dt), int(swz)};
+  Key k{base, d2, d1 * 1000003ULL + b1, d0, b2, b0, int(dt), int(swz), pitch};
   std::lock_guard<std::mutex> g(mu);
   auto it = cache.find(k);
   if (it != cache.end()) return it->second;
@@ -92,7 +95,7 @@ const CUtensorMap* tmap_3d(const void* base, CUtensorMapDataType dt, int elem_by
   }
   CUtensorMap* m = new CUtensorMap;
   uint64_t dims[3] = {d0, d1, d2};
-  uint64_t strides[2] = {d0 * uint64_t(elem_bytes), d0 * d1 * uint64_t(elem_bytes)};
+  uint64_t strides[2] = {d0 * uint64_t(elem_bytes), pitch * uint64_t(elem_bytes)};
   uint32_t box[3] = {b0, b1, b2};
   CUresult r = encode_tiled(m, dt, 3, base, dims, strides, box, swz);
   if (r != CUDA_SUCCESS) {

@@ -13,7 +13,7 @@ namespace xl {
 template <typename T>
 __global__ void moe_router_kernel(const T* __restrict__ logits, const float* __restrict__ bias, float* __restrict__ out_w,
                                   int* __restrict__ out_id, long long* __restrict__ load_hist, int T_tokens, int E, int top_k,
-                                  int sigmoid, int renorm, int n_group, int topk_group, float route_scale) {
+                                  int sigmoid, int renorm, int n_group, int topk_group, int group_top2, float route_scale) {
   constexpr int MAXV = 16;   // values per lane -> E <= 512
   const int lane = threadIdx.x & 31;
   const long t = (blockIdx.x * long(blockDim.x) + threadIdx.x) >> 5;
@@ -77,7 +77,7 @@ __global__ void moe_router_kernel(const T* __restrict__ logits, const float* __r
         const float n2 = fmaxf(fminf(b1, o1), fmaxf(b2, o2));
         b1 = n1; b2 = n2;
       }
-      const float gs = bias ? (b1 + (b2 == -INFINITY ? 0.f : b2)) : b1;   // noaux_tc: sum of the top-2; else group max
+      const float gs = group_top2 ? (b1 + (b2 == -INFINITY ? 0.f : b2)) : b1;   // noaux_tc: sum of the top-2; else group max
       if (lane == g) gscore_mine = gs;
     }
     // pick topk_group groups (iterative arg-max over lanes 0..n_group-1)
@@ -239,10 +239,11 @@ __global__ void moe_combine_kernel(const __nv_bfloat16* __restrict__ y, const in
 
 using namespace xl;
 
-// dtype: 0 fp32 logits, 1 bf16 logits
+// dtype: 0 fp32 logits, 1 bf16 logits.  group_top2: a group's score is the sum of its two best selection scores instead of
+// the best one.
 XL_API int xl_moe_router(const void* logits, int dtype, const void* bias, void* out_w, void* out_id, void* load_hist, int T,
-                         int E, int top_k, int sigmoid, int renorm, int n_group, int topk_group, float route_scale,
-                         void* stream) {
+                         int E, int top_k, int sigmoid, int renorm, int n_group, int topk_group, int group_top2,
+                         float route_scale, void* stream) {
   if (T <= 0) return 0;
   if (E > 512 || top_k > 32 || top_k < 1 || n_group > 32 || (n_group > 1 && E % n_group)) return -2;
   const int blocks = (T + 7) / 8;
@@ -251,12 +252,12 @@ XL_API int xl_moe_router(const void* logits, int dtype, const void* bias, void* 
     moe_router_kernel<float><<<blocks, 256, 0, st>>>(static_cast<const float*>(logits), static_cast<const float*>(bias),
                                                      static_cast<float*>(out_w), static_cast<int*>(out_id),
                                                      static_cast<long long*>(load_hist), T, E, top_k, sigmoid, renorm, n_group,
-                                                     topk_group, route_scale);
+                                                     topk_group, group_top2, route_scale);
   else
     moe_router_kernel<__nv_bfloat16><<<blocks, 256, 0, st>>>(
         static_cast<const __nv_bfloat16*>(logits), static_cast<const float*>(bias), static_cast<float*>(out_w),
         static_cast<int*>(out_id), static_cast<long long*>(load_hist), T, E, top_k, sigmoid, renorm, n_group, topk_group,
-        route_scale);
+        group_top2, route_scale);
   return cudaGetLastError() == cudaSuccess ? 0 : -1;
 }
 

@@ -1,0 +1,435 @@
+// Fused steps of a decoder whose sublayers are normed before and after and whose residual stream is fp32:
+//
+//   x += rms(y) * w_post;  h = rms(x) * w_next                      (one kernel between a sublayer and the next one)
+//
+// with three sources of the first line:
+//   SRC_ROWS   y is a tensor (the output of o_proj / down_proj);
+//   SRC_MOE    y is assembled here: weighted sum of the chosen experts' rows, identity experts (whose output is the
+//              sublayer's input itself, times the weight) and a shared expert, so that it never exists in memory;
+//   SRC_EMBED  there is no y: x = table[token] * scale starts the residual stream.
+// Also the kernel that follows the qkv projection where positions do not rotate anything: per-head q / k RMSNorm and the
+// write of k and v into the paged cache (q is normed in place); and the gated activation of an unfused feed-forward.
+//
+// All arithmetic is fp32; tensors are bf16, or fp32 when the model runs in 32-bit.
+#include <type_traits>
+
+#include "vec8.cuh"
+
+namespace xl_sn {
+using namespace xl;
+
+enum { SRC_ROWS = 0, SRC_MOE = 1, SRC_EMBED = 2 };
+
+template <typename T>
+struct NormParams {
+  float* x;                  // [rows, H] fp32 residual stream, updated in place (SRC_EMBED: written)
+  const T* w_post;           // [H] weight of the norm behind the sublayer
+  const T* w_next;           // [H] weight of the norm ahead of the next sublayer
+  T* h;                      // [rows, H] its output
+  int H;
+  float eps;
+  const T* y;                // SRC_ROWS: [rows, H]
+  // SRC_MOE
+  const T* y_exp;            // [*, H] expert outputs, row dst_of[t * k + j] belongs to choice j of token t (-1: none)
+  const int* dst_of;
+  const int* ids;            // [rows, k] chosen experts; ids >= first_identity are identity experts
+  const float* weights;      // [rows, k]
+  const T* h_in;             // [rows, H] the sublayer's input (identity experts)
+  const T* shared;           // [rows, H] or null
+  int k, first_identity;
+  // SRC_EMBED
+  const int* tokens;
+  const T* table;            // [V, H]
+  int V;
+  float scale;
+};
+
+// sum over the block of one value per thread; `red` holds one float per warp
+__device__ __forceinline__ float block_sum(float v, float* red) {
+  v = warp_sum(v);
+  if ((threadIdx.x & 31) == 0) red[threadIdx.x >> 5] = v;
+  __syncthreads();
+  float t = 0.f;
+  const int warps = (blockDim.x + 31) >> 5;
+  for (int i = 0; i < warps; ++i) t += red[i];
+  return t;
+}
+
+__device__ __forceinline__ int clamp_id(int id, int V) { return id < 0 ? 0 : (id >= V ? V - 1 : id); }
+
+// Register-resident rows: thread i owns the 8-element vectors i, i + blockDim, ... (VPT of them).
+template <typename T, int VPT, int SRC>
+__global__ void __launch_bounds__(256) sandwich_norm_kernel(const NormParams<T> p) {
+  __shared__ float red_a[8], red_b[8];
+  const int row = blockIdx.x, H = p.H, nvec = H / 8;
+  float y[VPT][8];
+  float ss = 0.f;
+  float w_id = 0.f;          // summed weight of this token's identity choices
+  if (SRC == SRC_MOE) {
+    for (int j = 0; j < p.k; ++j)
+      if (p.ids[row * p.k + j] >= p.first_identity) w_id += p.weights[row * p.k + j];
+  }
+#pragma unroll
+  for (int i = 0; i < VPT; ++i) {
+    const int v = threadIdx.x + i * blockDim.x;
+    if (v < nvec) {
+      if (SRC == SRC_ROWS) {
+        load8(p.y + size_t(row) * H + v * 8, y[i]);
+      } else if (SRC == SRC_EMBED) {
+        load8(p.table + size_t(clamp_id(p.tokens[row], p.V)) * H + v * 8, y[i]);
+#pragma unroll
+        for (int e = 0; e < 8; ++e) y[i][e] *= p.scale;
+      } else {
+        float f[8];
+#pragma unroll
+        for (int e = 0; e < 8; ++e) y[i][e] = 0.f;
+        if (p.shared) load8(p.shared + size_t(row) * H + v * 8, y[i]);
+        if (w_id != 0.f) {
+          load8(p.h_in + size_t(row) * H + v * 8, f);
+#pragma unroll
+          for (int e = 0; e < 8; ++e) y[i][e] += w_id * f[e];
+        }
+        for (int j = 0; j < p.k; ++j) {
+          const int r = p.dst_of[row * p.k + j];
+          if (r < 0) continue;
+          const float wj = p.weights[row * p.k + j];
+          load8(p.y_exp + size_t(r) * H + v * 8, f);
+#pragma unroll
+          for (int e = 0; e < 8; ++e) y[i][e] += wj * f[e];
+        }
+      }
+#pragma unroll
+      for (int e = 0; e < 8; ++e) ss += y[i][e] * y[i][e];
+    }
+  }
+  if (SRC != SRC_EMBED) {
+    const float r_post = rsqrtf(block_sum(ss, red_a) / float(H) + p.eps);
+    ss = 0.f;
+#pragma unroll
+    for (int i = 0; i < VPT; ++i) {
+      const int v = threadIdx.x + i * blockDim.x;
+      if (v < nvec) {
+        float w[8], x[8];
+        load8(p.w_post + v * 8, w);
+        load8(p.x + size_t(row) * H + v * 8, x);
+#pragma unroll
+        for (int e = 0; e < 8; ++e) {
+          y[i][e] = x[e] + y[i][e] * r_post * w[e];
+          ss += y[i][e] * y[i][e];
+        }
+      }
+    }
+  }
+  const float r_next = rsqrtf(block_sum(ss, red_b) / float(H) + p.eps);
+#pragma unroll
+  for (int i = 0; i < VPT; ++i) {
+    const int v = threadIdx.x + i * blockDim.x;
+    if (v < nvec) {
+      float w[8];
+      load8(p.w_next + v * 8, w);
+      store8(p.x + size_t(row) * H + v * 8, y[i]);
+#pragma unroll
+      for (int e = 0; e < 8; ++e) w[e] = y[i][e] * r_next * w[e];
+      store8(p.h + size_t(row) * H + v * 8, w);
+    }
+  }
+}
+
+// Any width: one element at a time, the row kept in shared memory.
+template <typename T, int SRC>
+__global__ void __launch_bounds__(256) sandwich_norm_any_kernel(const NormParams<T> p) {
+  extern __shared__ float row_cache[];
+  __shared__ float red_a[8], red_b[8];
+  const int row = blockIdx.x, H = p.H;
+  float ss = 0.f, w_id = 0.f;
+  if (SRC == SRC_MOE) {
+    for (int j = 0; j < p.k; ++j)
+      if (p.ids[row * p.k + j] >= p.first_identity) w_id += p.weights[row * p.k + j];
+  }
+  for (int i = threadIdx.x; i < H; i += blockDim.x) {
+    float y = 0.f;
+    if (SRC == SRC_ROWS) {
+      y = to_f32(p.y[size_t(row) * H + i]);
+    } else if (SRC == SRC_EMBED) {
+      y = to_f32(p.table[size_t(clamp_id(p.tokens[row], p.V)) * H + i]) * p.scale;
+    } else {
+      if (p.shared) y = to_f32(p.shared[size_t(row) * H + i]);
+      if (w_id != 0.f) y += w_id * to_f32(p.h_in[size_t(row) * H + i]);
+      for (int j = 0; j < p.k; ++j) {
+        const int r = p.dst_of[row * p.k + j];
+        if (r >= 0) y += p.weights[row * p.k + j] * to_f32(p.y_exp[size_t(r) * H + i]);
+      }
+    }
+    row_cache[i] = y;
+    ss += y * y;
+  }
+  if (SRC != SRC_EMBED) {
+    const float r_post = rsqrtf(block_sum(ss, red_a) / float(H) + p.eps);
+    ss = 0.f;
+    for (int i = threadIdx.x; i < H; i += blockDim.x) {
+      const float x = p.x[size_t(row) * H + i] + row_cache[i] * r_post * to_f32(p.w_post[i]);
+      row_cache[i] = x;
+      ss += x * x;
+    }
+  }
+  const float r_next = rsqrtf(block_sum(ss, red_b) / float(H) + p.eps);
+  for (int i = threadIdx.x; i < H; i += blockDim.x) {
+    p.x[size_t(row) * H + i] = row_cache[i];
+    from_f32(p.h + size_t(row) * H + i, row_cache[i] * r_next * to_f32(p.w_next[i]));
+  }
+}
+
+template <typename T, int SRC>
+static int launch_norm(const NormParams<T>& p, int rows, bool aligned, cudaStream_t st) {
+  if (rows <= 0) return 0;
+  const int nvec = p.H / 8;
+  if (aligned && p.H % 8 == 0 && nvec <= 1024) {
+    const int vpt = nvec <= 256 ? 1 : nvec <= 512 ? 2 : 4;
+    const int threads = ((nvec + vpt - 1) / vpt + 31) / 32 * 32;
+    if (vpt == 1) sandwich_norm_kernel<T, 1, SRC><<<rows, threads, 0, st>>>(p);
+    else if (vpt == 2) sandwich_norm_kernel<T, 2, SRC><<<rows, threads, 0, st>>>(p);
+    else sandwich_norm_kernel<T, 4, SRC><<<rows, threads, 0, st>>>(p);
+  } else {
+    const size_t smem = size_t(p.H) * sizeof(float);
+    if (smem > 200 * 1024) return -2;
+    static bool set = false;
+    if (!set) {
+      cudaFuncSetAttribute(sandwich_norm_any_kernel<T, SRC>, cudaFuncAttributeMaxDynamicSharedMemorySize, 200 * 1024);
+      set = true;
+    }
+    sandwich_norm_any_kernel<T, SRC><<<rows, 256, smem, st>>>(p);
+  }
+  return cudaGetLastError() == cudaSuccess ? 0 : -1;
+}
+
+static bool al16(const void* a, const void* b = nullptr, const void* c = nullptr, const void* d = nullptr) {
+  return !((reinterpret_cast<uintptr_t>(a) | reinterpret_cast<uintptr_t>(b) | reinterpret_cast<uintptr_t>(c) |
+            reinterpret_cast<uintptr_t>(d)) & 15);
+}
+
+template <typename T>
+static NormParams<T> base_params(void* x, const void* w_post, const void* w_next, void* h, int H, float eps) {
+  NormParams<T> p = {};
+  p.x = static_cast<float*>(x);
+  p.w_post = static_cast<const T*>(w_post);
+  p.w_next = static_cast<const T*>(w_next);
+  p.h = static_cast<T*>(h);
+  p.H = H;
+  p.eps = eps;
+  return p;
+}
+
+// ---------------------------------------------------------------- q / k norm + cache write
+// LPH lanes per (token, head), 8 elements per lane; heads as laid out by the fused qkv projection:
+// n_q query heads of dk, n_kv key heads of dk, n_kv value heads of dv.
+template <typename T>
+__global__ void __launch_bounds__(256) qknorm_kvwrite_vec_kernel(T* __restrict__ qkv, const int* __restrict__ slots,
+                                                                 const T* __restrict__ q_w, const T* __restrict__ k_w,
+                                                                 T* __restrict__ k_cache, T* __restrict__ v_cache, int T_rows,
+                                                                 int n_q, int n_kv, int dk, int dv, int lph, float eps,
+                                                                 long cache_slots) {
+  const int heads = n_q + 2 * n_kv;
+  const long gt = blockIdx.x * long(blockDim.x) + threadIdx.x;
+  const long item = gt / lph;
+  const int sub = int(gt % lph);
+  const bool active = item < long(T_rows) * heads;
+  const int t = active ? int(item / heads) : 0, h = active ? int(item % heads) : 0;
+  const size_t row = size_t(t) * (size_t(n_q + n_kv) * dk + size_t(n_kv) * dv);
+  const bool is_v = h >= n_q + n_kv;
+  const int dim = is_v ? dv : dk;
+  T* src = qkv + row + (is_v ? size_t(n_q + n_kv) * dk + size_t(h - n_q - n_kv) * dv : size_t(h) * dk);
+  const bool mine = active && sub * 8 < dim;
+  float f[8] = {0, 0, 0, 0, 0, 0, 0, 0};
+  if (mine) load8(src + sub * 8, f);
+  float ss = 0.f;
+#pragma unroll
+  for (int e = 0; e < 8; ++e) ss += f[e] * f[e];
+  for (int o = lph / 2; o > 0; o >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, o);
+  if (!mine) return;
+  if (!is_v) {
+    const T* w = h >= n_q ? k_w : q_w;
+    if (w) {
+      const float r = rsqrtf(ss / float(dk) + eps);
+      float wf[8];
+      load8(w + sub * 8, wf);
+#pragma unroll
+      for (int e = 0; e < 8; ++e) f[e] = f[e] * r * wf[e];
+    }
+  }
+  if (h < n_q) {
+    store8(src + sub * 8, f);
+    return;
+  }
+  const int slot = slots[t];
+  if (slot < 0 || slot >= cache_slots) return;
+  T* dst = is_v ? v_cache + (size_t(slot) * n_kv + (h - n_q - n_kv)) * dv : k_cache + (size_t(slot) * n_kv + (h - n_q)) * dk;
+  store8(dst + sub * 8, f);
+}
+
+// Any head dimension: one warp per (token, head).
+template <typename T>
+__global__ void __launch_bounds__(256) qknorm_kvwrite_any_kernel(T* __restrict__ qkv, const int* __restrict__ slots,
+                                                                 const T* __restrict__ q_w, const T* __restrict__ k_w,
+                                                                 T* __restrict__ k_cache, T* __restrict__ v_cache, int T_rows,
+                                                                 int n_q, int n_kv, int dk, int dv, float eps, long cache_slots) {
+  const int heads = n_q + 2 * n_kv, lane = threadIdx.x & 31;
+  const long item = (blockIdx.x * long(blockDim.x) + threadIdx.x) >> 5;
+  if (item >= long(T_rows) * heads) return;
+  const int t = int(item / heads), h = int(item % heads);
+  const size_t row = size_t(t) * (size_t(n_q + n_kv) * dk + size_t(n_kv) * dv);
+  const bool is_v = h >= n_q + n_kv;
+  const int dim = is_v ? dv : dk;
+  T* src = qkv + row + (is_v ? size_t(n_q + n_kv) * dk + size_t(h - n_q - n_kv) * dv : size_t(h) * dk);
+  const T* w = is_v ? nullptr : (h >= n_q ? k_w : q_w);
+  float r = 1.f;
+  if (w) {
+    float ss = 0.f;
+    for (int i = lane; i < dim; i += 32) ss += to_f32(src[i]) * to_f32(src[i]);
+    r = rsqrtf(warp_sum(ss) / float(dim) + eps);
+  }
+  const int slot = slots[t];
+  T* dst = src;
+  if (h >= n_q) {
+    if (slot < 0 || slot >= cache_slots) return;
+    dst = is_v ? v_cache + (size_t(slot) * n_kv + (h - n_q - n_kv)) * dv : k_cache + (size_t(slot) * n_kv + (h - n_q)) * dk;
+  }
+  for (int i = lane; i < dim; i += 32) {
+    const float v = to_f32(src[i]);
+    from_f32(dst + i, w ? v * r * to_f32(w[i]) : v);
+  }
+}
+
+template <typename T>
+static int launch_qknorm(void* qkv, const void* slots, const void* q_w, const void* k_w, void* k_cache, void* v_cache, int rows, int n_q,
+                         int n_kv, int dk, int dv, float eps, long cache_slots, cudaStream_t st) {
+  const long items = long(rows) * (n_q + 2 * n_kv);
+  const int dmax = dk > dv ? dk : dv;
+  if (dk % 8 == 0 && dv % 8 == 0 && dmax <= 256 && al16(qkv, k_cache, v_cache, q_w) && al16(k_w)) {
+    int lph = 1;
+    while (lph * 8 < dmax) lph *= 2;
+    qknorm_kvwrite_vec_kernel<T><<<int((items * lph + 255) / 256), 256, 0, st>>>(
+        static_cast<T*>(qkv), static_cast<const int*>(slots), static_cast<const T*>(q_w), static_cast<const T*>(k_w),
+        static_cast<T*>(k_cache), static_cast<T*>(v_cache), rows, n_q, n_kv, dk, dv, lph, eps, cache_slots);
+  } else {
+    qknorm_kvwrite_any_kernel<T><<<int((items + 7) / 8), 256, 0, st>>>(
+        static_cast<T*>(qkv), static_cast<const int*>(slots), static_cast<const T*>(q_w), static_cast<const T*>(k_w),
+        static_cast<T*>(k_cache), static_cast<T*>(v_cache), rows, n_q, n_kv, dk, dv, eps, cache_slots);
+  }
+  return cudaGetLastError() == cudaSuccess ? 0 : -1;
+}
+
+// ---------------------------------------------------------------- gated activation: out[t, i] = act(x[t, i]) * x[t, I + i]
+template <typename T>
+__global__ void gated_act_kernel(const T* __restrict__ x, T* __restrict__ out, long total, int I, int act) {
+  for (long idx = blockIdx.x * long(blockDim.x) + threadIdx.x; idx < total; idx += long(gridDim.x) * blockDim.x) {
+    const long t = idx / I;
+    const int i = int(idx % I);
+    const T* row = x + t * 2 * I;
+    from_f32(out + idx, gate_act(to_f32(row[i]), act) * to_f32(row[I + i]));
+  }
+}
+template <typename T>
+__global__ void gated_act_vec_kernel(const T* __restrict__ x, T* __restrict__ out, long total, int nvec, int act) {
+  for (long idx = blockIdx.x * long(blockDim.x) + threadIdx.x; idx < total; idx += long(gridDim.x) * blockDim.x) {
+    const long t = idx / nvec;
+    const int v = int(idx % nvec);
+    const T* row = x + t * 16 * nvec;
+    float g[8], u[8];
+    load8(row + v * 8, g);
+    load8(row + (nvec + v) * 8, u);
+#pragma unroll
+    for (int e = 0; e < 8; ++e) g[e] = gate_act(g[e], act) * u[e];
+    store8(out + idx * 8, g);
+  }
+}
+template <typename T>
+static int launch_gated_act(const void* x, void* out, int rows, int I, int act, cudaStream_t st) {
+  const bool vec = I % 8 == 0 && al16(x, out);
+  const long total = long(rows) * (vec ? I / 8 : I);
+  long blocks = (total + 255) / 256;
+  if (blocks > 148 * 16) blocks = 148 * 16;
+  if (vec) gated_act_vec_kernel<T><<<int(blocks), 256, 0, st>>>(static_cast<const T*>(x), static_cast<T*>(out), total, I / 8, act);
+  else gated_act_kernel<T><<<int(blocks), 256, 0, st>>>(static_cast<const T*>(x), static_cast<T*>(out), total, I, act);
+  return cudaGetLastError() == cudaSuccess ? 0 : -1;
+}
+
+}  // namespace xl_sn
+
+using namespace xl_sn;
+
+// `f32` in the entry points below: 1 when the model's tensors are fp32, 0 for bf16 (the residual x is fp32 either way).
+
+// x[t] = table[tokens[t]] * scale;  h = rms(x) * w_next
+XL_API int xl_embed_rms_norm(const void* tokens, const void* table, float scale, void* x, const void* w_next, void* h, int rows, int H,
+                             int V, float eps, int f32, void* stream) {
+  cudaStream_t st = static_cast<cudaStream_t>(stream);
+  const bool al = al16(table, x, w_next, h);
+  if (f32) {
+    auto p = base_params<float>(x, nullptr, w_next, h, H, eps);
+    p.tokens = static_cast<const int*>(tokens); p.table = static_cast<const float*>(table); p.V = V; p.scale = scale;
+    return launch_norm<float, SRC_EMBED>(p, rows, al, st);
+  }
+  auto p = base_params<__nv_bfloat16>(x, nullptr, w_next, h, H, eps);
+  p.tokens = static_cast<const int*>(tokens); p.table = static_cast<const __nv_bfloat16*>(table); p.V = V; p.scale = scale;
+  return launch_norm<__nv_bfloat16, SRC_EMBED>(p, rows, al, st);
+}
+
+// x += rms(y) * w_post;  h = rms(x) * w_next
+XL_API int xl_post_norm_add_norm(const void* y, void* x, const void* w_post, const void* w_next, void* h, int rows, int H, float eps,
+                                 int f32, void* stream) {
+  cudaStream_t st = static_cast<cudaStream_t>(stream);
+  const bool al = al16(y, x, w_post, w_next) && al16(h);
+  if (f32) {
+    auto p = base_params<float>(x, w_post, w_next, h, H, eps);
+    p.y = static_cast<const float*>(y);
+    return launch_norm<float, SRC_ROWS>(p, rows, al, st);
+  }
+  auto p = base_params<__nv_bfloat16>(x, w_post, w_next, h, H, eps);
+  p.y = static_cast<const __nv_bfloat16*>(y);
+  return launch_norm<__nv_bfloat16, SRC_ROWS>(p, rows, al, st);
+}
+
+// y[t] = sum_j weights[t, j] * expert output (an expert's row of y_exp, or h_in[t] for ids >= first_identity) + shared[t];
+// then as above.
+XL_API int xl_moe_combine_post_norm_add_norm(const void* y_exp, const void* dst_of, const void* ids, const void* weights,
+                                             const void* h_in, const void* shared, int k, int first_identity, void* x,
+                                             const void* w_post, const void* w_next, void* h, int rows, int H, float eps, int f32,
+                                             void* stream) {
+  cudaStream_t st = static_cast<cudaStream_t>(stream);
+  const bool al = al16(y_exp, x, w_post, w_next) && al16(h, h_in, shared);
+  auto fill = [&](auto& p, auto* tag) {
+    using E = std::remove_pointer_t<decltype(tag)>;
+    p.y_exp = static_cast<const E*>(y_exp);
+    p.dst_of = static_cast<const int*>(dst_of);
+    p.ids = static_cast<const int*>(ids);
+    p.weights = static_cast<const float*>(weights);
+    p.h_in = static_cast<const E*>(h_in);
+    p.shared = static_cast<const E*>(shared);
+    p.k = k;
+    p.first_identity = first_identity;
+  };
+  if (f32) {
+    auto p = base_params<float>(x, w_post, w_next, h, H, eps);
+    fill(p, static_cast<float*>(nullptr));
+    return launch_norm<float, SRC_MOE>(p, rows, al, st);
+  }
+  auto p = base_params<__nv_bfloat16>(x, w_post, w_next, h, H, eps);
+  fill(p, static_cast<__nv_bfloat16*>(nullptr));
+  return launch_norm<__nv_bfloat16, SRC_MOE>(p, rows, al, st);
+}
+
+// Per-head RMSNorm of q (in place) and k (null weight: none), k and v to the cache slots [cache_slots, n_kv, dk | dv].
+XL_API int xl_qknorm_kvwrite(void* qkv, const void* slots, const void* q_w, const void* k_w, void* k_cache, void* v_cache, int rows,
+                             int n_q, int n_kv, int dk, int dv, float eps, long cache_slots, int f32, void* stream) {
+  if (rows <= 0) return 0;
+  cudaStream_t st = static_cast<cudaStream_t>(stream);
+  if (f32) return launch_qknorm<float>(qkv, slots, q_w, k_w, k_cache, v_cache, rows, n_q, n_kv, dk, dv, eps, cache_slots, st);
+  return launch_qknorm<__nv_bfloat16>(qkv, slots, q_w, k_w, k_cache, v_cache, rows, n_q, n_kv, dk, dv, eps, cache_slots, st);
+}
+
+// x [rows, 2 I] = [gate | up] -> act(gate) * up; act: 0 silu, 1 tanh-gelu
+XL_API int xl_gated_act(const void* x, void* out, int rows, int I, int act, int f32, void* stream) {
+  if (rows <= 0) return 0;
+  cudaStream_t st = static_cast<cudaStream_t>(stream);
+  return f32 ? launch_gated_act<float>(x, out, rows, I, act, st) : launch_gated_act<__nv_bfloat16>(x, out, rows, I, act, st);
+}

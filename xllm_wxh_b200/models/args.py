@@ -13,6 +13,7 @@ import json
 import os
 from typing import Any, Dict, List, Optional
 
+from .layer_spec import AttentionSpec, FeedForwardSpec, LayerSpec, run_order
 
 @dataclasses.dataclass
 class QuantArgs:
@@ -88,6 +89,10 @@ class ModelArgs:
     # MTP
     num_nextn_predict_layers: int = 0
     quant: QuantArgs = dataclasses.field(default_factory=QuantArgs)
+    # designs that list their layers one by one (models/movolorn.py); the flat sizes above then hold maxima over the layers
+    layer_specs: List[LayerSpec] = dataclasses.field(default_factory=list)
+    layer_runs: List[int] = dataclasses.field(default_factory=list)      # layer of every run, in order (layers may repeat)
+    embedding_scale: float = 1.0
 
     # ------------------------------------------------------------------ derived
     @property
@@ -126,7 +131,63 @@ def _first(cfg: Dict[str, Any], *names, default=None):
     return default
 
 
+def _movolorn_layer(i: int, cfg: Dict[str, Any]) -> LayerSpec:
+    if cfg.get("type") != "attention":
+        raise ValueError(f"layer {i}: mixer '{cfg.get('type')}' is not supported")
+    m = cfg["mixer"]
+    H, G = int(m["heads"]), int(m["kv_heads"])
+    if H < 1 or G < 1 or H % G:
+        raise ValueError(f"layer {i}: {H} heads do not divide over {G} key/value heads")
+    mixer = AttentionSpec(heads=H, kv_heads=G, dim=int(m["dim"]), vdim=int(m["vdim"]), scale=float(m["scale"]),
+                          chunk=int((m.get("mask") or {}).get("size") or 0), distance_bias=True, sink=0.0, qk_norm=True)
+    f = cfg.get("mlp")
+    if not f:
+        return LayerSpec(mixer, None)
+    if f["kind"] == "dense":
+        return LayerSpec(mixer, FeedForwardSpec(ff=int(f["ff"]), act="gelu_tanh"))
+    if f["kind"] != "moe":
+        raise ValueError(f"layer {i}: feed-forward '{f['kind']}' is not supported")
+    r = f["router"]
+    g = r.get("groups") or {}
+    mlp = FeedForwardSpec(ff=int(f["expert"]["ff"]), act="silu", experts=int(r["experts"]), identity_experts=int(r.get("identity") or 0),
+                          top_k=int(r["top"]), n_group=int(g.get("count") or 1), topk_group=int(g.get("keep") or g.get("count") or 1),
+                          shared_ff=int((f.get("shared") or {}).get("ff") or 0))
+    outputs = mlp.experts + mlp.identity_experts
+    if outputs % mlp.n_group or mlp.topk_group > mlp.n_group or mlp.top_k > mlp.topk_group * (outputs // mlp.n_group):
+        raise ValueError(f"layer {i}: {outputs} router outputs, {mlp.n_group} groups of which {mlp.topk_group} are kept, top {mlp.top_k}")
+    return LayerSpec(mixer, mlp)
+
+
+def args_from_layer_list(specs: List[LayerSpec], runs: List[int], **kw) -> ModelArgs:
+    """ModelArgs of a design given layer by layer; the flat sizes that the engine plans with are maxima over the layers."""
+    mix = [s.mixer for s in specs]
+    ffs = [s.mlp for s in specs if s.mlp is not None]
+    inner = [f.shared_ff + f.ff * (f.top_k if f.is_moe else 1) for f in ffs]
+    return ModelArgs(layer_specs=specs, layer_runs=runs, n_layers=len(runs), n_heads=max(m.heads for m in mix),
+                     n_kv_heads=max(m.kv_heads for m in mix), head_dim=max(m.dim for m in mix), v_head_dim=max(m.vdim for m in mix),
+                     intermediate_size=max(inner, default=0), n_routed_experts=max((f.experts for f in ffs), default=0),
+                     num_experts_per_tok=max((f.top_k for f in ffs), default=0), qk_norm=any(m.qk_norm for m in mix), **kw)
+
+
+def _movolorn_args(cfg: Dict[str, Any]) -> ModelArgs:
+    specs = [_movolorn_layer(i, c) for i, c in enumerate(cfg["layers"])]
+    loop = cfg.get("loop") or {}
+    runs = run_order(len(specs), int(loop.get("start", 0)), int(loop.get("stop", 0)), int(loop.get("times", 1)))
+    dt = str(_first(cfg, "torch_dtype", "dtype", default="bfloat16"))
+    return args_from_layer_list(
+        specs, runs, model_type="movolorn", dtype=dt if dt in _DTYPES else "bfloat16", vocab_size=int(cfg["vocab"]),
+        hidden_size=int(cfg["width"]), rms_norm_eps=float(cfg["norm"]["eps"]),
+        embedding_scale=float((cfg.get("embedding") or {}).get("scale", 1.0)),
+        max_position_embeddings=int(_first(cfg, "max_position_embeddings", default=131072)),
+        eos_token_id=int(_first(cfg, "eos_token_id", default=-1)))
+
+
+_DTYPES = ("float32", "bfloat16")
+
+
 def args_from_hf_config(cfg: Dict[str, Any]) -> ModelArgs:
+    if str(cfg.get("architecture", "")).lower() == "movolorn":
+        return _movolorn_args(cfg)
     mt = _first(cfg, "model_type", "model_name", default="qwen3")
     a = ModelArgs(model_type=mt)
     a.dtype = {"float32": "float32", "float16": "float16"}.get(str(_first(cfg, "torch_dtype", "dtype", default="bfloat16")),
@@ -281,4 +342,17 @@ def preset(name: str) -> ModelArgs:
                          rope_mscale=1.0, rope_mscale_all_dim=1.0, max_position_embeddings=163840,
                          num_nextn_predict_layers=1,
                          quant=QuantArgs(method="fp8", weight_block_size=[128, 128]))
+    if name in ("movolorn-30b-a3b", "movolorn_30b_a3b"):
+        # layer sizes of qwen3-30b-a3b: the same attention, experts and active experts in the Movolorn block
+        mixer = dict(heads=32, kv_heads=4, dim=128, vdim=128, scale=128 ** -0.5, chunk=8192, distance_bias=True, sink=0.0, qk_norm=True)
+        spec = [LayerSpec(AttentionSpec(**mixer), FeedForwardSpec(ff=768, act="silu", experts=124, identity_experts=4, top_k=8, n_group=8,
+                                                                  topk_group=4)) for _ in range(48)]
+        return args_from_layer_list(spec, run_order(48), model_type="movolorn", vocab_size=151936, hidden_size=2048,
+                                    max_position_embeddings=40960)
+    if name in ("movolorn-8b", "movolorn_8b"):
+        # layer sizes of qwen3-8b in the Movolorn block (dense)
+        mixer = dict(heads=32, kv_heads=8, dim=128, vdim=128, scale=128 ** -0.5, chunk=8192, distance_bias=True, sink=0.0, qk_norm=True)
+        spec = [LayerSpec(AttentionSpec(**mixer), FeedForwardSpec(ff=12288, act="gelu_tanh")) for _ in range(36)]
+        return args_from_layer_list(spec, run_order(36), model_type="movolorn", vocab_size=151936, hidden_size=4096,
+                                    max_position_embeddings=40960)
     raise KeyError(name)

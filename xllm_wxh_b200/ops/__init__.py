@@ -45,6 +45,16 @@ def paged_attention(q, k_cache, v_cache, inp, scale, sliding_window=-1):
                                sliding_window)
 
 
+def paged_attention_ext(q, k_cache, v_cache, inp, scale, window=-1, chunk=0, slopes=None, sinks=None):
+    """Paged attention with a per-head linear distance bias (`slopes` [Hq] fp32), a per-head sink score in the softmax
+    denominator (`sinks` [Hq] fp32), keys limited to the query's chunk of `chunk` positions, and a value head dimension of
+    its own.  q [T, Hq, dk] -> [T, Hq * dv]."""
+    if q.is_cuda:
+        return _cuda().paged_attention_ext(q, k_cache, v_cache, inp, scale, window, chunk, slopes, sinks)
+    return ref.paged_attention(q, k_cache, v_cache, inp.q_cu, inp.kv_lens, inp.block_tables, inp.n_seqs, scale, window, chunk,
+                               slopes, sinks)
+
+
 def sample(logits, inp):
     """Penalties -> temperature -> top-k/top-p -> sample/argmax (+logprobs).  Returns
     (tokens int32 [S], logprobs | None, top_vals | None, top_ids | None)."""
@@ -67,9 +77,11 @@ def topk_candidates(logits, inp, id_offset: int, width: int):
     return ref.topk_candidates(logits, inp.temperature[:S], inp.top_k[:S], id_offset, width)
 
 
-def moe_router(logits, top_k, scoring="softmax", renorm=True, bias=None, n_group=1, topk_group=1, route_scale=1.0):
+def moe_router(logits, top_k, scoring="softmax", renorm=True, bias=None, n_group=1, topk_group=1, route_scale=1.0, group_score=None):
+    """`group_score`: how a group of experts is ranked, "max" or "top2" (sum of its two best); None: top2 with a bias, else max."""
     f = _cuda().moe_router if logits.is_cuda else ref.moe_router
-    return f(logits, top_k, scoring, renorm, bias, n_group, topk_group, route_scale)
+    extra = {} if group_score is None else {"group_score": group_score}
+    return f(logits, top_k, scoring, renorm, bias, n_group, topk_group, route_scale, **extra)
 
 
 def moe_experts(x, w13, w2, weights, ids, expert_offset=0, interleaved=False):
@@ -86,6 +98,47 @@ def gate_up_swiglu(x, w, interleaved=False):
         return _cuda().linear_swiglu(x, w)
     assert not interleaved
     return silu_and_mul(linear(x, w))
+
+
+# ----------------------------------------------------------------------------- sublayers normed before and after, fp32 residual
+def embed_rms_norm(ids, table, scale, w_next, eps):
+    """(fp32 residual x = table[ids] * scale, rms(x) * w_next in the table's dtype)."""
+    return (_cuda() if table.is_cuda else ref).embed_rms_norm(ids, table, scale, w_next, eps)
+
+
+def post_norm_add_norm(y, x, w_post, w_next, eps):
+    """x += rms(y) * w_post (x fp32, in place); returns rms(x) * w_next."""
+    return (_cuda() if y.is_cuda else ref).post_norm_add_norm(y, x, w_post, w_next, eps)
+
+
+def qknorm_kvwrite(qkv, slots, q_w, k_w, eps, k_cache, v_cache, n_q, n_kv):
+    """Per-head RMSNorm of q and k without any rotation; k and v into the paged caches.  Returns q [T, n_q * dk]."""
+    return (_cuda() if qkv.is_cuda else ref).qknorm_kvwrite(qkv, slots, q_w, k_w, eps, k_cache, v_cache, n_q, n_kv)
+
+
+def linear_f32(x, w):
+    """x w^T in fp32 (router logits)."""
+    return (_cuda() if x.is_cuda else ref).linear_f32(x, w)
+
+
+def gated_linear(x, w, act="silu", interleaved=False):
+    """act(x Wg^T) * (x Wu^T) with W = [gate rows; up rows], or the interleaved layout on CUDA (applied in the GEMM epilogue).
+    act: "silu" | "gelu_tanh"."""
+    if not x.is_cuda:
+        return ref.gated_act(linear(x, w), act)
+    return _cuda().linear_gated(x, w, act) if interleaved else _cuda().gated_act(linear(x, w), act)
+
+
+def moe_post_norm_add_norm(h_in, w13, w2, weights, ids, shared, first_identity, x, w_post, w_next, eps, act="silu", interleaved=False):
+    """Mixture sublayer from its routing to the next sublayer's input: y = sum_j weights_j expert_j(h_in) (ids from
+    `first_identity` on are identity experts: weight times h_in) + shared (or None); x += rms(y) * w_post (fp32, in place);
+    returns rms(x) * w_next."""
+    if h_in.is_cuda:
+        from . import moe_cuda
+        y, dst_of = moe_cuda.expert_rows(h_in, w13, w2, ids, act, interleaved)
+        return moe_cuda.combine_post_norm_add_norm(y, dst_of, ids, weights, h_in, shared, first_identity, x, w_post, w_next, eps)
+    y = ref.moe_mixture(h_in, w13, w2, weights, ids, shared, first_identity, act)
+    return ref.post_norm_add_norm(y, x, w_post, w_next, eps)
 
 
 # ----------------------------------------------------------------------------- MLA (DeepSeek)

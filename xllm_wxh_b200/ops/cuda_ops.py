@@ -12,7 +12,7 @@ from typing import Dict, Optional, Tuple
 import torch
 
 _HERE = os.path.dirname(os.path.abspath(__file__))
-_LIB_PATH = os.path.join(os.path.dirname(_HERE), "libxllm_kernels.so")
+_LIB_PATH = os.environ.get("XLLM_KERNELS_SO") or os.path.join(os.path.dirname(_HERE), "libxllm_kernels.so")
 _lib = None
 launch_count = 0          # kernels launched through this module (reported by bench.py as `gpu_launches`)
 
@@ -104,8 +104,51 @@ def sm_count() -> int:
 
 
 # ----------------------------------------------------------------------------- GEMM
+def _tc_gemm_ok(x: torch.Tensor, w: torch.Tensor, n_align: int = 8) -> bool:
+    """Whether the tensor-core GEMMs serve x [M, K] and w [..., N, K]: bf16, rows on 16-byte boundaries, N a multiple of
+    `n_align`."""
+    return (x.dtype == torch.bfloat16 and w.dtype == torch.bfloat16 and w.shape[-1] % 8 == 0 and w.shape[-2] % n_align == 0 and
+            x.stride(0) % 8 == 0 and (x.data_ptr() | w.data_ptr()) % 16 == 0)
+
+
+def _gemm_simt(x2: torch.Tensor, w: torch.Tensor, out_dtype: torch.dtype) -> torch.Tensor:
+    """The fp32-pipe GEMM: fp32 operands, or bf16 ones of any shape."""
+    global launch_count
+    assert x2.dtype == w.dtype and x2.dtype in (torch.float32, torch.bfloat16) and w.stride(-1) == 1
+    M, K = x2.shape
+    N = w.shape[0]
+    out = torch.empty((M, N), dtype=out_dtype, device=x2.device)
+    if M > 0:
+        _check(lib().xl_gemm_simt(_ptr(x2), _ptr(w), _ptr(out), c_int(M), c_int(N), c_int(K), c_long(x2.stride(0)), c_long(w.stride(0)),
+                                  c_long(N), c_int(int(x2.dtype == torch.float32)), c_int(int(out_dtype == torch.float32)), _stream()),
+               "xl_gemm_simt")
+        launch_count += 1
+    return out
+
+
+def linear_f32(x: torch.Tensor, w: torch.Tensor) -> torch.Tensor:
+    """x w^T with the fp32 sums kept (router logits); x and w bf16 or fp32."""
+    global launch_count
+    if x.stride(-1) != 1:
+        x = x.contiguous()
+    M, K = x.shape
+    N = w.shape[0]
+    if not _tc_gemm_ok(x, w, 1):
+        return _gemm_simt(x, w, torch.float32)
+    out = torch.empty((M, N), dtype=torch.float32, device=x.device)
+    if M > 0:
+        _check(lib().xl_gemm_bf16_f32(_ptr(x), _ptr(w), _ptr(out), c_int(M), c_int(N), c_int(K), c_int(x.stride(0)), c_int(w.stride(0)),
+                                      c_int(N), _stream()), "xl_gemm_bf16_f32")
+        launch_count += 1
+    return out
+
+
 def linear(x: torch.Tensor, w: torch.Tensor, bias: Optional[torch.Tensor] = None, out: Optional[torch.Tensor] = None) -> torch.Tensor:
     global launch_count
+    if x.dtype == torch.float32 or (bias is None and out is None and not _tc_gemm_ok(x.reshape(-1, x.shape[-1]), w)):
+        assert bias is None and out is None
+        x2 = x.reshape(-1, x.shape[-1])
+        return _gemm_simt(x2 if x2.stride(-1) == 1 else x2.contiguous(), w, x.dtype).reshape(x.shape[:-1] + (w.shape[0],))
     assert x.dtype == torch.bfloat16 and w.dtype == torch.bfloat16, "GEMM kernel is bf16"
     x2 = x.reshape(-1, x.shape[-1])
     if x2.stride(-1) != 1:
@@ -121,6 +164,37 @@ def linear(x: torch.Tensor, w: torch.Tensor, bias: Optional[torch.Tensor] = None
         _check(rc, "xl_gemm_bf16")
         launch_count += 1
     return out.reshape(x.shape[:-1] + (N,))
+
+
+ACTS = {"silu": 0, "gelu_tanh": 1}
+
+
+def linear_gated(x: torch.Tensor, w_interleaved: torch.Tensor, act: str) -> torch.Tensor:
+    """gate_up GEMM whose epilogue applies act(gate) * up; `w_interleaved` from `interleave_gate_up`."""
+    global launch_count
+    if x.stride(-1) != 1:
+        x = x.contiguous()
+    M, K = x.shape
+    N = w_interleaved.shape[0]
+    out = torch.empty((M, N // 2), dtype=torch.bfloat16, device=x.device)
+    if M > 0:
+        _check(lib().xl_gemm_bf16_gated(_ptr(x), _ptr(w_interleaved), _ptr(out), c_int(M), c_int(N), c_int(K), c_int(x.stride(0)),
+                                        c_int(w_interleaved.stride(0)), c_int(out.stride(0)), c_int(ACTS[act]), _stream()),
+               "xl_gemm_bf16_gated")
+        launch_count += 1
+    return out
+
+
+def gated_act(x: torch.Tensor, act: str) -> torch.Tensor:
+    """[T, 2I] = [gate | up] -> act(gate) * up (bf16 or fp32, any I)."""
+    global launch_count
+    T, I2 = x.shape
+    assert x.is_contiguous()
+    out = torch.empty((T, I2 // 2), dtype=x.dtype, device=x.device)
+    _check(lib().xl_gated_act(_ptr(x), _ptr(out), c_int(T), c_int(I2 // 2), c_int(ACTS[act]), c_int(int(x.dtype == torch.float32)),
+                              _stream()), "xl_gated_act")
+    launch_count += 1
+    return out
 
 
 def linear_swiglu(x: torch.Tensor, w_interleaved: torch.Tensor) -> torch.Tensor:
@@ -215,6 +289,50 @@ def rope_qknorm_kvwrite(qkv, positions, slots, cos_sin, q_w, k_w, eps, k_cache, 
     return qkv[:, :n_q * head_dim]
 
 
+# ----------------------------------------------------------------------------- norms before and after a sublayer, fp32 residual
+def _f32flag(t: torch.Tensor):
+    assert t.dtype in (torch.float32, torch.bfloat16)
+    return c_int(int(t.dtype == torch.float32))
+
+
+def embed_rms_norm(ids: torch.Tensor, table: torch.Tensor, scale: float, w_next: torch.Tensor, eps: float):
+    """(fp32 residual x = table[ids] * scale, rms(x) * w_next)."""
+    global launch_count
+    T = ids.numel()
+    V, H = table.shape
+    x = torch.empty((T, H), dtype=torch.float32, device=table.device)
+    h = torch.empty((T, H), dtype=table.dtype, device=table.device)
+    _check(lib().xl_embed_rms_norm(_ptr(ids), _ptr(table), c_float(scale), _ptr(x), _ptr(w_next), _ptr(h), c_int(T), c_int(H), c_int(V),
+                                   c_float(eps), _f32flag(table), _stream()), "xl_embed_rms_norm")
+    launch_count += 1
+    return x, h
+
+
+def post_norm_add_norm(y: torch.Tensor, x: torch.Tensor, w_post: torch.Tensor, w_next: torch.Tensor, eps: float) -> torch.Tensor:
+    """x += rms(y) * w_post in place; returns rms(x) * w_next."""
+    global launch_count
+    T, H = y.shape
+    assert y.is_contiguous() and x.is_contiguous() and x.dtype == torch.float32
+    h = torch.empty_like(y)
+    _check(lib().xl_post_norm_add_norm(_ptr(y), _ptr(x), _ptr(w_post), _ptr(w_next), _ptr(h), c_int(T), c_int(H), c_float(eps),
+                                       _f32flag(y), _stream()), "xl_post_norm_add_norm")
+    launch_count += 1
+    return h
+
+
+def qknorm_kvwrite(qkv, slots, q_w, k_w, eps, k_cache, v_cache, n_q, n_kv):
+    """Per-head RMSNorm of q (in place) and k, k and v into the paged caches; returns q [T, n_q * dk] (a view of qkv)."""
+    global launch_count
+    T = qkv.shape[0]
+    dk, dv = k_cache.shape[-1], v_cache.shape[-1]
+    assert qkv.is_contiguous() and qkv.shape[1] == (n_q + n_kv) * dk + n_kv * dv and k_cache.dtype == qkv.dtype
+    _check(lib().xl_qknorm_kvwrite(_ptr(qkv), _ptr(slots), _ptr(q_w), _ptr(k_w), _ptr(k_cache), _ptr(v_cache), c_int(T), c_int(n_q),
+                                   c_int(n_kv), c_int(dk), c_int(dv), c_float(eps), c_long(k_cache.shape[0] * k_cache.shape[1]),
+                                   _f32flag(qkv), _stream()), "xl_qknorm_kvwrite")
+    launch_count += 1
+    return qkv[:, :n_q * dk]
+
+
 # ----------------------------------------------------------------------------- attention
 decode_kernel = "tma"     # "tma" | "cp_async" (the fallback kernel; selectable for tests and comparisons)
 
@@ -298,6 +416,68 @@ def paged_attention(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tenso
     return out
 
 
+def paged_attention_ext(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tensor, inp, scale: float, window: int = -1, chunk: int = 0,
+                        slopes: Optional[torch.Tensor] = None, sinks: Optional[torch.Tensor] = None) -> torch.Tensor:
+    """Paged attention with score extensions and a value dimension of its own: q [T, Hq, dk] (may be a view of the qkv
+    buffer), caches [blocks, block, Hkv, dk | dv] -> [T, Hq * dv].  score = scale q.k - slopes[h] * distance; keys of the
+    query's own chunk of `chunk` positions only (0: all); exp(sinks[h]) joins the softmax denominator.  bf16 tensors with
+    head dimensions up to 128 (multiples of 8) run on the tensor-core kernels, anything else on the fp32-pipe kernel."""
+    global launch_count
+    from ..framework.step_input import H_NUM_DECODE, H_NUM_SEQS
+    T, Hq, dk = q.shape
+    block_size, n_kv, dv = k_cache.shape[1], k_cache.shape[2], v_cache.shape[3]
+    L, padded = inp.layout, inp.padded
+    for t in (slopes, sinks):
+        assert t is None or (t.dtype == torch.float32 and t.numel() == Hq and t.is_contiguous())
+    out = (torch.zeros if padded else torch.empty)((T, Hq * dv), dtype=q.dtype, device=q.device)
+    n_dec = inp.B if padded else inp.n_decode
+    n_all = inp.B if padded else inp.n_seqs
+    has_prefill = inp.has_prefill if padded else n_all > n_dec
+    q_stride = q.stride(0)
+
+    def simt():
+        _check(lib().xl_attention_simt(_ptr(q), _ptr(k_cache), _ptr(v_cache), _ptr(out), _ptr(inp.token_seq), _ptr(inp.positions),
+                                       _ptr(inp.block_tables), c_int(T), c_int(n_all), c_int(L.MB_cap), c_int(block_size),
+                                       c_long(k_cache.shape[0] * block_size), c_int(Hq), c_int(n_kv), c_int(dk), c_int(dv),
+                                       c_long(q_stride), c_float(scale), c_int(window), c_int(chunk), _ptr(slopes), _ptr(sinks),
+                                       _f32flag(q), _stream()), "xl_attention_simt")
+        return out
+    if q.dtype == torch.float32 or dk % 8 or dv % 8 or dk > 128 or dv > 128 or q.stride(1) != dk or Hq // n_kv > 16:
+        launch_count += 1
+        return simt()
+    hdr = getattr(inp, "header_dev", None)
+    dyn_dec = c_void_p(hdr.data_ptr() + 4 * H_NUM_DECODE) if padded else c_void_p(0)
+    dyn_all = c_void_p(hdr.data_ptr() + 4 * H_NUM_SEQS) if padded else c_void_p(0)
+    common = (_ptr(q), _ptr(k_cache), _ptr(v_cache), _ptr(out), _ptr(inp.q_cu), _ptr(inp.kv_lens), _ptr(inp.block_tables))
+    shape = (c_int(L.MB_cap), c_int(block_size), c_int(k_cache.shape[0]), c_int(Hq), c_int(n_kv), c_int(dk), c_int(dv), c_int(q_stride))
+    if n_dec > 0:
+        max_kv = (L.MB_cap * block_size) if padded else inp.max_kv
+        splits = decode_splits(n_dec, n_kv, min(max_kv, chunk) if chunk > 0 else max_kv)
+        po = pl = None
+        rows = max(T, n_dec)
+        if splits > 1:
+            po = torch.empty((rows, Hq, splits, dv), dtype=torch.float32, device=q.device)
+            pl = torch.empty((rows, Hq, splits), dtype=torch.float32, device=q.device)
+        rc = lib().xl_decode_attention_ext(*common, c_int(0), c_int(n_dec), *shape, c_float(scale), c_int(window), c_int(chunk),
+                                           _ptr(slopes), _ptr(sinks), c_int(splits), _ptr(po), _ptr(pl), c_long(rows), dyn_dec, _stream())
+        if rc == -3:            # a block size outside the tensor-core kernels' limits
+            launch_count += 1
+            return simt()
+        _check(rc, "xl_decode_attention_ext")
+        launch_count += 1 + (1 if splits > 1 else 0)
+    if has_prefill:
+        tiles = (T + 127) // 128 + n_all if padded else (inp.n_prefill_tokens + 127) // 128 + (n_all - n_dec)
+        rc = lib().xl_prefill_attention_ext(*common, c_int(0 if padded else n_dec), c_int(n_all), *shape, c_int(T), c_float(scale),
+                                            c_int(window), c_int(chunk), _ptr(slopes), _ptr(sinks), c_int(tiles), dyn_dec, dyn_all,
+                                            _stream())
+        if rc == -3:
+            launch_count += 1
+            return simt()
+        _check(rc, "xl_prefill_attention_ext")
+        launch_count += 1
+    return out
+
+
 # ----------------------------------------------------------------------------- sampling
 def sample(logits: torch.Tensor, inp):
     global launch_count
@@ -344,9 +524,9 @@ def topk_candidates(logits: torch.Tensor, inp, id_offset: int, width: int):
 
 
 # ----------------------------------------------------------------------------- MoE
-def moe_router(logits, top_k, scoring="softmax", renorm=True, bias=None, n_group=1, topk_group=1, route_scale=1.0):
+def moe_router(logits, top_k, scoring="softmax", renorm=True, bias=None, n_group=1, topk_group=1, route_scale=1.0, group_score=None):
     from . import moe_cuda
-    return moe_cuda.moe_router(logits, top_k, scoring, renorm, bias, n_group, topk_group, route_scale)
+    return moe_cuda.moe_router(logits, top_k, scoring, renorm, bias, n_group, topk_group, route_scale, group_score=group_score)
 
 
 def moe_experts(x, w13, w2, weights, ids, expert_offset=0, interleaved=False):

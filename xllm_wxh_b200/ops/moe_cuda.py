@@ -22,8 +22,10 @@ from .cuda_ops import _check, _ptr, _stream, c_float, c_int, c_void_p, lib
 
 def moe_router(logits: torch.Tensor, top_k: int, scoring: str = "softmax", renorm: bool = True,
                bias: Optional[torch.Tensor] = None, n_group: int = 1, topk_group: int = 1, route_scale: float = 1.0,
-               load_hist: Optional[torch.Tensor] = None) -> Tuple[torch.Tensor, torch.Tensor]:
+               load_hist: Optional[torch.Tensor] = None, group_score: Optional[str] = None) -> Tuple[torch.Tensor, torch.Tensor]:
+    """`group_score`: "top2" (sum of a group's two best selection scores) or "max"; default: top2 with a bias, else max."""
     T, E = logits.shape
+    top2 = (bias is not None) if group_score is None else group_score == "top2"
     assert logits.is_contiguous() and logits.dtype in (torch.float32, torch.bfloat16)
     w = torch.empty((T, top_k), dtype=torch.float32, device=logits.device)
     ids = torch.empty((T, top_k), dtype=torch.int32, device=logits.device)
@@ -31,7 +33,7 @@ def moe_router(logits: torch.Tensor, top_k: int, scoring: str = "softmax", renor
         bias = bias.float()
     _check(lib().xl_moe_router(_ptr(logits), c_int(0 if logits.dtype == torch.float32 else 1), _ptr(bias), _ptr(w), _ptr(ids),
                                _ptr(load_hist), c_int(T), c_int(E), c_int(top_k), c_int(int(scoring == "sigmoid")),
-                               c_int(int(renorm)), c_int(n_group), c_int(topk_group), c_float(route_scale), _stream()),
+                               c_int(int(renorm)), c_int(n_group), c_int(topk_group), c_int(int(top2)), c_float(route_scale), _stream()),
            "xl_moe_router")
     cuda_ops.launch_count += 1
     return w, ids
@@ -74,9 +76,10 @@ def moe_sort(ids: torch.Tensor, expert_offset: int, E_local: int, max_rows: Opti
     return SortedRouting(work, sorted_src, dst_of, E_local, max_tiles, rows)
 
 
-def grouped_gemm(a: torch.Tensor, w: torch.Tensor, r, swiglu: bool = False, out: Optional[torch.Tensor] = None,
+def grouped_gemm(a: torch.Tensor, w: torch.Tensor, r, swiglu: int = 0, out: Optional[torch.Tensor] = None,
                  c_rows_per_expert: int = 0, c_col_stride: int = 0) -> torch.Tensor:
-    """a [R_cap, K] rows sorted by expert; w [E_local, N, K]; returns [R_cap, N] (or [R_cap, N/2] with the SwiGLU epilogue).
+    """a [R_cap, K] rows sorted by expert; w [E_local, N, K]; returns [R_cap, N] (or [R_cap, N/2] with a gated epilogue:
+    `swiglu` 1 = silu gate, 2 = tanh-gelu gate).
     `r` provides the device-side tile table (`tile_expert`, `tile_row0`, `tile_row_end`, `num_m_tiles`, `max_tiles`).
     With `out` given, row `row - expert * c_rows_per_expert` / column offset `expert * c_col_stride` place each tile."""
     R_cap, K = a.shape
@@ -135,3 +138,46 @@ def moe_experts(x: torch.Tensor, w13: torch.Tensor, w2: torch.Tensor, weights: t
         h = cuda_ops.silu_and_mul(grouped_gemm(xs, w13, r))
     y = grouped_gemm(h, w2, r)
     return combine(y, r, weights, T, add)
+
+
+def grouped_gemm_simt(a: torch.Tensor, w: torch.Tensor, r: SortedRouting, gather_k: int = 0) -> torch.Tensor:
+    """The fp32-pipe grouped GEMM (fp32 operands, or bf16 ones of any shape).  `gather_k` > 0: `a` holds the unsorted token
+    rows and sorted row i reads row sorted_src[i] // gather_k of it."""
+    E, N, K = w.shape
+    assert a.shape[1] == K and w.is_contiguous() and a.stride(-1) == 1 and a.dtype == w.dtype
+    out = torch.empty((max(r.n, 1), N), dtype=a.dtype, device=a.device)
+    _check(lib().xl_grouped_gemm_simt(_ptr(a), _ptr(w), _ptr(out), c_int(N), c_int(K), ctypes.c_long(a.stride(0)), ctypes.c_long(N),
+                                      _ptr(r.tile_expert), _ptr(r.tile_row0), _ptr(r.tile_row_end), _ptr(r.num_m_tiles), c_int(r.max_tiles),
+                                      _ptr(r.sorted_src) if gather_k else c_void_p(0), c_int(max(gather_k, 1)),
+                                      c_int(int(a.dtype == torch.float32)), _stream()), "xl_grouped_gemm_simt")
+    cuda_ops.launch_count += 1
+    return out
+
+
+def expert_rows(x: torch.Tensor, w13: torch.Tensor, w2: torch.Tensor, ids: torch.Tensor, act: str = "silu", interleaved: bool = False):
+    """Outputs of the chosen experts before their weighted sum: (rows [*, H], dst_of [T * k] with -1 for ids outside the
+    experts of w13)."""
+    k = ids.shape[1]
+    r = moe_sort(ids, 0, w13.shape[0])
+    if interleaved:
+        y = grouped_gemm(grouped_gemm(gather_rows(x, r, k), w13, r, swiglu=1 + cuda_ops.ACTS[act]), w2, r)
+    elif cuda_ops._tc_gemm_ok(x, w13) and cuda_ops._tc_gemm_ok(x, w2) and x.shape[1] % 8 == 0:
+        y = grouped_gemm(cuda_ops.gated_act(grouped_gemm(gather_rows(x, r, k), w13, r), act), w2, r)
+    else:
+        y = grouped_gemm_simt(cuda_ops.gated_act(grouped_gemm_simt(x, w13, r, k), act), w2, r)
+    return y, r.dst_of
+
+
+def combine_post_norm_add_norm(y_exp, dst_of, ids, weights, h_in, shared, first_identity, x, w_post, w_next, eps) -> torch.Tensor:
+    """y = sum of the chosen experts' rows times their weights + identity choices (ids >= first_identity: weight times h_in)
+    + shared; then x += rms(y) * w_post in place; returns rms(x) * w_next.  One kernel; y is not stored."""
+    T, H = h_in.shape
+    assert h_in.is_contiguous() and x.is_contiguous() and x.dtype == torch.float32 and y_exp.shape[1] == H
+    assert shared is None or shared.is_contiguous()
+    h = torch.empty_like(h_in)
+    _check(lib().xl_moe_combine_post_norm_add_norm(_ptr(y_exp), _ptr(dst_of), _ptr(ids), _ptr(weights), _ptr(h_in), _ptr(shared),
+                                                   c_int(ids.shape[1]), c_int(first_identity), _ptr(x), _ptr(w_post), _ptr(w_next), _ptr(h),
+                                                   c_int(T), c_int(H), c_float(eps), c_int(int(h_in.dtype == torch.float32)), _stream()),
+           "xl_moe_combine_post_norm_add_norm")
+    cuda_ops.launch_count += 1
+    return h

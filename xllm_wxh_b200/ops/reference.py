@@ -143,10 +143,12 @@ def rope_qknorm_kvwrite(qkv: torch.Tensor, positions: torch.Tensor, slots: torch
 
 def paged_attention(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tensor, q_cu: torch.Tensor,
                     kv_lens: torch.Tensor, block_tables: torch.Tensor, n_seqs: int, scale: float,
-                    sliding_window: int = -1) -> torch.Tensor:
+                    sliding_window: int = -1, chunk: int = 0, slopes: Optional[torch.Tensor] = None,
+                    sinks: Optional[torch.Tensor] = None) -> torch.Tensor:
     """Causal attention of ragged query rows over paged KV.
     q [T, Hq, D]; caches [n_blocks, block, Hkv, D]; sequence i owns q rows q_cu[i]:q_cu[i+1], which are the
-    last rows of its kv_lens[i] tokens."""
+    last rows of its kv_lens[i] tokens.  `chunk` > 0: a query sees keys of its own chunk of positions only; `slopes` [Hq]:
+    slopes[h] * (query position - key position) is taken off the scores; `sinks` [Hq]: exp(sinks[h]) joins the denominator."""
     T, Hq, D = q.shape
     block = k_cache.shape[1]
     Hkv = k_cache.shape[2]
@@ -174,8 +176,16 @@ def paged_attention(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tenso
         mask = kpos <= qpos
         if sliding_window > 0:
             mask &= kpos > qpos - sliding_window
+        if chunk > 0:
+            mask &= torch.div(kpos, chunk, rounding_mode="floor") == torch.div(qpos, chunk, rounding_mode="floor")
+        if slopes is not None:
+            s = s - slopes.float()[:, None, None] * (qpos - kpos).float()[None]
         s = s.masked_fill(~mask[None], float("-inf"))
-        p = torch.softmax(s, dim=-1)
+        if sinks is not None:
+            s = torch.cat([s, sinks.float()[:, None, None].expand(Hq, n, 1)], dim=-1)
+            p = torch.softmax(s, dim=-1)[..., :-1]
+        else:
+            p = torch.softmax(s, dim=-1)
         out[qs:qe] = torch.einsum("hnl,lhd->nhd", p, v).to(q.dtype)
     return out.reshape(T, Hq * Dv)
 
@@ -288,7 +298,7 @@ def sample(logits: torch.Tensor, temperature: torch.Tensor, top_k: torch.Tensor,
 # ----------------------------------------------------------------------------- MoE
 def moe_router(logits: torch.Tensor, top_k: int, scoring: str = "softmax", renorm: bool = True,
                bias: Optional[torch.Tensor] = None, n_group: int = 1, topk_group: int = 1,
-               route_scale: float = 1.0) -> Tuple[torch.Tensor, torch.Tensor]:
+               route_scale: float = 1.0, group_score: Optional[str] = None) -> Tuple[torch.Tensor, torch.Tensor]:
     """Router (reference: moe_topk_softmax_kernels.cuh:324-611, moe_topk_sigmoid_kernels.cuh:165-383,
     group-limited rule of the MLU `moe_active_topk` op, param.h:402-442).
     Returns (weights fp32 [T, k], expert ids int32 [T, k])."""
@@ -298,7 +308,8 @@ def moe_router(logits: torch.Tensor, top_k: int, scoring: str = "softmax", renor
     T, E = scores.shape
     if n_group > 1:
         g = sel.view(T, n_group, E // n_group)
-        gscore = g.topk(2, dim=-1).values.sum(-1) if bias is not None else g.max(-1).values
+        top2 = (bias is not None) if group_score is None else group_score == "top2"
+        gscore = g.topk(2, dim=-1).values.sum(-1) if top2 else g.max(-1).values
         keep = gscore.topk(topk_group, dim=-1).indices
         gmask = torch.zeros(T, n_group, dtype=torch.bool, device=logits.device).scatter_(1, keep, True)
         sel = sel.masked_fill(~gmask[:, :, None].expand(T, n_group, E // n_group).reshape(T, E), float("-inf"))
@@ -327,6 +338,60 @@ def moe_experts(x: torch.Tensor, w13: torch.Tensor, w2: torch.Tensor, weights: t
         y = linear(h, w2[e])
         out.index_add_(0, tok, y.float() * wk[:, None])
     return out.to(x.dtype)
+
+
+def linear_f32(x: torch.Tensor, w: torch.Tensor) -> torch.Tensor:
+    return torch.nn.functional.linear(x.float(), w.float())
+
+
+def gated_act(x: torch.Tensor, act: str) -> torch.Tensor:
+    """[T, 2I] = [gate | up] -> act(gate) * up, act "silu" or "gelu_tanh"."""
+    d = x.shape[-1] // 2
+    g, u = x[..., :d].float(), x[..., d:].float()
+    g = torch.nn.functional.silu(g) if act == "silu" else torch.nn.functional.gelu(g, approximate="tanh")
+    return (g * u).to(x.dtype)
+
+
+def moe_mixture(h: torch.Tensor, w13: torch.Tensor, w2: torch.Tensor, weights: torch.Tensor, ids: torch.Tensor,
+                shared: Optional[torch.Tensor], first_identity: int, act: str) -> torch.Tensor:
+    """fp32 sum of the chosen experts' outputs times their weights, identity choices (ids >= first_identity) and `shared`."""
+    out = torch.zeros(h.shape, dtype=torch.float32, device=h.device)
+    for e in range(w13.shape[0]):
+        hit = ids == e
+        tok = hit.any(-1).nonzero().squeeze(-1)
+        if tok.numel():
+            y = linear(gated_act(linear(h[tok], w13[e]), act), w2[e])
+            out.index_add_(0, tok, y.float() * (weights * hit).sum(-1)[tok][:, None])
+    out += (weights * (ids >= first_identity)).sum(-1, keepdim=True) * h.float()
+    return out if shared is None else out + shared.float()
+
+
+# norms before and after a sublayer around an fp32 residual stream
+def _rms_f32(x: torch.Tensor, w: torch.Tensor, eps: float) -> torch.Tensor:
+    xf = x.float()
+    return xf * torch.rsqrt(xf.pow(2).mean(-1, keepdim=True) + eps) * w.float()
+
+
+def embed_rms_norm(ids: torch.Tensor, table: torch.Tensor, scale: float, w_next: torch.Tensor, eps: float):
+    x = embedding(ids, table).float() * scale
+    return x, _rms_f32(x, w_next, eps).to(table.dtype)
+
+
+def post_norm_add_norm(y: torch.Tensor, x: torch.Tensor, w_post: torch.Tensor, w_next: torch.Tensor, eps: float) -> torch.Tensor:
+    x += _rms_f32(y, w_post, eps)
+    return _rms_f32(x, w_next, eps).to(w_next.dtype)
+
+
+def qknorm_kvwrite(qkv, slots, q_w, k_w, eps, k_cache, v_cache, n_q, n_kv):
+    T = qkv.shape[0]
+    dk, dv = k_cache.shape[-1], v_cache.shape[-1]
+    q, k, v = qkv.split([n_q * dk, n_kv * dk, n_kv * dv], dim=-1)
+    q, k = q.reshape(T, n_q, dk), k.reshape(T, n_kv, dk)
+    if q_w is not None:
+        q, k = _rms_f32(q, q_w, eps).to(qkv.dtype), _rms_f32(k, k_w, eps).to(qkv.dtype)
+    k_cache.view(-1, n_kv, dk).index_copy_(0, slots.long(), k.to(k_cache.dtype))
+    v_cache.view(-1, n_kv, dv).index_copy_(0, slots.long(), v.reshape(T, n_kv, dv).to(v_cache.dtype))
+    return q.reshape(T, n_q * dk)
 
 
 def moe_experts_fp8(x, w13_deq, w2_deq, weights, ids, expert_offset=0):

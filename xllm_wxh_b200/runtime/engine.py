@@ -370,7 +370,7 @@ class LLMEngine:
                 continue
             decode_only = b.forward_type == 2 and b.num_spec == 0
             T, B, MB, S, P, padded = self.worker.choose_caps(b.num_tokens, b.num_seqs, b.max_blocks, b.num_sample_rows,
-                                                            decode_only, graphable=b.num_spec == 0 and not want_emb)
+                                                            decode_only, graphable=b.num_spec == 0 and want_emb in (0, 3))
             L = self.worker.layout_for(T, B, MB, S, P)
             specs.append([L, padded, total])
             total += L.total_words
@@ -657,6 +657,29 @@ class LLMEngine:
         self.host_trace.append(((t_sched - t0) * 1e3, (self._t_pack - t_sched) * 1e3, (self._t_issue - self._t_pack) * 1e3,
                                 (t_end - self._t_issue) * 1e3))
         return sch.take_outputs()
+
+    def step_portions(self, portions: Sequence[Tuple[int, Sequence[int], Sequence[int]]]) -> List[np.ndarray]:
+        """Run one step whose content is given: (request id, its next tokens, places among them whose logits are wanted) for
+        every request that takes part.  Blocks, packing, kernels and graphs are those of generation; nothing is sampled.
+        Requests are added with an empty prompt (`add_request([])`) and ended with `cancel`.  Returns one fp32
+        [wanted, vocab] array per portion."""
+        self.bind_thread()
+        if self.world_size != 1 or self._inflight:
+            raise RuntimeError("replayed steps run on an engine of one process with no step in flight")
+        batches = self.scheduler.schedule_portions([(int(r), list(t), list(w)) for r, t, w in portions])
+        b = batches[0]
+        if b.empty:
+            return []
+        res = self._publish(batches, patch=False, want_emb=3)
+        self.scheduler.complete_portions(b.id)
+        self.scheduler.take_outputs()
+        self.step_count += 1
+        rows = res.embeddings.numpy()
+        by_request, at = {}, 0
+        for e, n in zip(b.entries(), b.rows_per_entry()):       # the batch orders decode rows first
+            by_request[e[1]] = rows[at:at + n]
+            at += n
+        return [by_request[int(r)] for r, _, _ in portions]
 
     def export_chrome_trace(self, path: str, last: int = 0) -> int:
         """Write the host phases of the recorded steps as a Chrome / Perfetto trace (`chrome://tracing`): one track, four

@@ -225,7 +225,8 @@ class Worker:
                 want_embeddings: int = 0) -> StepResult:
         """Run one step whose packed inputs are already in `self._host[:layout.total_words]`.  `want_embeddings`: 0 = sample
         tokens; 1 = return the pooled embedding of every sampling row instead; 2 = return, in the same place, the
-        probability of the "yes" token against the "no" token at every sampling row (`self.yes_no_ids`)."""
+        probability of the "yes" token against the "no" token at every sampling row (`self.yes_no_ids`); 3 = the fp32
+        logits of every row, nothing is sampled (replayed steps)."""
         L = layout
         host = self._host
         header = host[L.header:L.header + 32].numpy().copy()
@@ -305,6 +306,9 @@ class Worker:
     def _finish(self, inp: StepInput, hidden, logits, want_embeddings: int, sharded_logits: bool = False) -> StepResult:
         S = inp.S
         batch_id = int(np.uint32(inp.header[12])) | (int(np.uint32(inp.header[13])) << 32)
+        if want_embeddings == 3:
+            rows = logits[:inp.n_sample].float().cpu()
+            return StepResult(batch_id, inp.n_sample, 1, torch.zeros(max(S, 1), dtype=torch.int32), None, None, None, None, rows)
         if want_embeddings == 2:
             # Qwen3-reranker scoring (sampler.cpp:78-90 of the reference): softmax over the logits of "no" and "yes" at
             # the position that would generate the answer; the score is the probability of "yes"
