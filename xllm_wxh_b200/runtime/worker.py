@@ -308,6 +308,8 @@ class Worker:
         batch_id = int(np.uint32(inp.header[12])) | (int(np.uint32(inp.header[13])) << 32)
         if want_embeddings == 3:
             rows = logits[:inp.n_sample].float().cpu()
+            if self.is_cuda and inp.n_sample == 0:      # nothing was copied back: the pinned inputs are free only after the step
+                torch.cuda.current_stream(self.device).synchronize()
             return StepResult(batch_id, inp.n_sample, 1, torch.zeros(max(S, 1), dtype=torch.int32), None, None, None, None, rows)
         if want_embeddings == 2:
             # Qwen3-reranker scoring (sampler.cpp:78-90 of the reference): softmax over the logits of "no" and "yes" at
