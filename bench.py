@@ -59,6 +59,8 @@ def parse():
     p.add_argument("--eplb", action="store_true", help="MoE: expert-parallel load balancing with one redundant slot per rank")
     p.add_argument("--tp-mlp-mode", type=str, default="auto", choices=["auto", "tp", "rows"],
                    help="dense MLP under tensor parallelism: sharded weights (tp), replicated weights run by rows, or auto")
+    p.add_argument("--compare-design", type=str, default="", help="instead of the serving workload: prefill and decode throughput of a "
+                   "model design's layers and its kernels, beside the closest other model at equal sizes (movolorn)")
     p.add_argument("--seed", type=int, default=0)
     return p.parse_args()
 
@@ -203,8 +205,29 @@ def pd_arm(a):
     os._exit(0)
 
 
+def compare_arm(a):
+    """Layers and kernels of one design beside its closest relative, one GPU; one JSON line."""
+    json_fd = os.dup(1)
+    os.dup2(2, 1)
+    import torch
+    from xllm_wxh_b200.ops import bench_design
+    if a.compare_design not in bench_design.PAIRS:
+        os.write(json_fd, (json.dumps({"unavailable": f"--compare-design takes {sorted(bench_design.PAIRS)}"}) + "\n").encode())
+        return 0
+    torch.cuda.set_device(0)
+    torch.manual_seed(a.seed)
+    sampler = ClockSampler(0)
+    sampler.start()
+    out = bench_design.run(a.compare_design, layers=a.layers or 4, block=a.block_size)
+    out["clocks"] = sampler.stop()
+    os.write(json_fd, (json.dumps(out) + "\n").encode())
+    return 0
+
+
 def main():
     a = parse()
+    if a.compare_design:
+        return compare_arm(a)
     if a.impl == "reference":
         return reference_arm(a)
     world = int(os.environ.get("WORLD_SIZE", "1"))
