@@ -197,6 +197,7 @@ class Options:
     # ---- python-side conveniences
     max_model_len: int = _flag(0, "Context limit (0 = model's).", "model")
     num_kv_blocks: int = _flag(0, "Force the number of KV blocks (0 = derive).", "kv")
+    num_state_slots: int = _flag(0, "Sequences that can hold recurrent state at a time, for models that keep any (0 = derive from max_seqs_per_batch and free memory).", "kv")
 
     def validate(self) -> "Options":
         """The reference's `validate_flags` (xllm/xllm.cpp:59-109) plus range checks."""

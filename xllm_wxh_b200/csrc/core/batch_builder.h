@@ -20,7 +20,8 @@ namespace xl {
 struct BatchLayout {
   int T_cap, B_cap, MB_cap, S_cap, P_cap;
   // offsets in int32 words
-  int header, tokens, positions, slots, token_seq, next_tokens, q_cu, kv_lens, block_tables, sample_idx, temperature, top_p, top_k,
+  int header, tokens, positions, slots, token_seq, next_tokens, q_cu, kv_lens, state_slots, block_tables, sample_idx, temperature,
+      top_p, top_k,
       rep_pen, freq_pen, pres_pen, seed_lo, seed_hi, want_logprobs, pen_cu, pen_ids, pen_counts, total_words;
   static int align(int x) { return (x + 31) & ~31; }
   BatchLayout(int T, int B, int MB, int S, int P) : T_cap(T), B_cap(B), MB_cap(MB), S_cap(S), P_cap(P) {
@@ -34,6 +35,7 @@ struct BatchLayout {
     next_tokens = sec(T);
     q_cu = sec(B + 1);
     kv_lens = sec(B);
+    state_slots = sec(B);
     block_tables = sec(B * MB);
     sample_idx = sec(S);
     temperature = sec(S);
@@ -72,7 +74,7 @@ inline long build_batch(const Batch& b, const BatchLayout& L, int32_t* buf, int 
   std::memset(H, 0, 32 * 4);
   int32_t *tok = buf + L.tokens, *pos = buf + L.positions, *slot = buf + L.slots, *tseq = buf + L.token_seq;
   int32_t* nxt = buf + L.next_tokens;   // token that follows each position (-1: not known yet = the one sampled this step)
-  int32_t *qcu = buf + L.q_cu, *kvl = buf + L.kv_lens, *bt = buf + L.block_tables, *sidx = buf + L.sample_idx;
+  int32_t *qcu = buf + L.q_cu, *kvl = buf + L.kv_lens, *sst = buf + L.state_slots, *bt = buf + L.block_tables, *sidx = buf + L.sample_idx;
   int t = 0, row = 0, max_q = 0, max_kv = 0, n_spec = 0, pen_total = 0, n_prefill_tokens = 0;
   bool any_pen = false, all_greedy = true, any_lp = false;
   int max_top_lp = 0, max_top_k = 0;
@@ -97,6 +99,7 @@ inline long build_batch(const Batch& b, const BatchLayout& L, int32_t* buf, int 
     }
     qcu[i + 1] = t;
     kvl[i] = kv_after;
+    sst[i] = s->state_slot;
     std::memcpy(bt + size_t(i) * L.MB_cap, s->blocks.data(), size_t(used_blocks) * 4);
     for (int j = used_blocks; j < L.MB_cap; ++j) bt[size_t(i) * L.MB_cap + j] = 0;
     max_q = std::max(max_q, e.n_tokens);
@@ -171,6 +174,7 @@ inline long build_batch(const Batch& b, const BatchLayout& L, int32_t* buf, int 
   for (int i = n_seq; i < L.B_cap; ++i) {
     qcu[i + 1] = t;
     kvl[i] = 0;
+    sst[i] = 0;
   }
   for (int i = row; i < L.S_cap; ++i) {
     sidx[i] = 0;

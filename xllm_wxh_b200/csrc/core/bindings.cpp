@@ -91,7 +91,8 @@ PYBIND11_MODULE(_core, m) {
       .def_readwrite("starve_threshold", &SchedulerOptions::starve_threshold)
       .def_readwrite("enable_starve_prevent", &SchedulerOptions::enable_starve_prevent)
       .def_readwrite("min_prefill_chunk", &SchedulerOptions::min_prefill_chunk)
-      .def_readwrite("host_blocks_factor", &SchedulerOptions::host_blocks_factor);
+      .def_readwrite("host_blocks_factor", &SchedulerOptions::host_blocks_factor)
+      .def_readwrite("num_state_slots", &SchedulerOptions::num_state_slots);
 
   py::class_<StepTimeModel>(m, "StepTimeModel")
       .def(py::init<>())
@@ -125,7 +126,7 @@ PYBIND11_MODULE(_core, m) {
            py::arg("P_cap"))
 #define RO(f) .def_readonly(#f, &BatchLayout::f)
       RO(T_cap) RO(B_cap) RO(MB_cap) RO(S_cap) RO(P_cap) RO(header) RO(tokens) RO(positions) RO(slots) RO(token_seq) RO(next_tokens)
-      RO(q_cu) RO(kv_lens) RO(block_tables) RO(sample_idx) RO(temperature) RO(top_p) RO(top_k) RO(rep_pen) RO(freq_pen)
+      RO(q_cu) RO(kv_lens) RO(state_slots) RO(block_tables) RO(sample_idx) RO(temperature) RO(top_p) RO(top_k) RO(rep_pen) RO(freq_pen)
       RO(pres_pen) RO(seed_lo) RO(seed_hi) RO(want_logprobs) RO(pen_cu) RO(pen_ids) RO(pen_counts) RO(total_words)
 #undef RO
       ;
@@ -312,6 +313,7 @@ PYBIND11_MODULE(_core, m) {
       .def("set_clock_override", &Scheduler::set_clock_override)
       .def("mix_order", &Scheduler::mix_order)
       .def("mix_latency_budget", &Scheduler::mix_latency_budget)
+      .def_property_readonly("num_free_state_slots", &Scheduler::num_free_state_slots)
       .def_property_readonly("num_running", &Scheduler::num_running)
       .def_property_readonly("num_pending", &Scheduler::num_pending)
       .def("schedule", &Scheduler::schedule, py::return_value_policy::reference_internal)

@@ -54,6 +54,7 @@ struct Sequence {
   std::vector<float> logprobs;  // one per generated token when requested
   int num_prompt_tokens = 0;
   std::vector<int> blocks;
+  int state_slot = 0;           // slot of recurrent state (0: none held)
   int kv_tokens = 0;            // tokens whose KV is in the cache
   int num_cached_tokens = 0;    // prompt tokens served by the prefix cache at admission
   int dp_rank = -1;

@@ -23,6 +23,7 @@
 
 #include "block_manager.h"
 #include "request.h"
+#include "state_slots.h"
 #include "step_time_model.h"
 
 namespace xl {
@@ -52,6 +53,9 @@ struct SchedulerOptions {
   int min_prefill_chunk = 50;  // a latency-bounded chunk smaller than this is not worth a step
   // host-memory tier of the prefix cache: host blocks = host_blocks_factor x device blocks (global_flags.cpp:439-442)
   double host_blocks_factor = 0.0;
+  // slots of recurrent state per DP rank (0: the model keeps none).  A sequence runs only while it holds one; a cached
+  // prefix has no state to continue from, so the prefix cache stays off.
+  int num_state_slots = 0;
 };
 
 enum class ForwardType : int { PREFILL = 0, CHUNKED_PREFILL = 1, DECODE = 2, MIXED = 3, EMPTY = 4 };
@@ -125,6 +129,11 @@ class Scheduler {
   Scheduler(const SchedulerOptions& opt, int num_blocks, int block_size, bool enable_prefix_cache, uint64_t seed = 1024)
       : opt_(opt), pool_(opt.dp_size, num_blocks, block_size, enable_prefix_cache, seed) {
     if (opt_.max_tokens_per_chunk_for_prefill <= 0) opt_.max_tokens_per_chunk_for_prefill = opt_.max_tokens_per_batch;
+    if (opt_.num_state_slots > 0) {
+      if (enable_prefix_cache) throw std::invalid_argument("recurrent state and the prefix cache do not go together");
+      if (opt_.num_speculative_tokens > 0) throw std::invalid_argument("recurrent state cannot take back rejected draft tokens");
+      for (int i = 0; i < opt_.dp_size; ++i) slots_.emplace_back(opt_.num_state_slots);
+    }
     const int host_blocks = static_cast<int>(opt_.host_blocks_factor * (num_blocks - 1));
     if (enable_prefix_cache && host_blocks >= 1) {
       for (int i = 0; i < opt_.dp_size; ++i) host_.emplace_back(host_blocks + 1, block_size, true, seed);
@@ -207,6 +216,7 @@ class Scheduler {
   const SchedulerOptions& options() const { return opt_; }
   BlockManagerPool& pool() { return pool_; }
   const SchedulerStats& stats() const { return stats_; }
+  int num_free_state_slots() const { return slots_.empty() ? 0 : slots_[0].num_free(); }
 
   // Thread-safe: API threads enqueue, the scheduler thread drains.
   int64_t add_request(std::unique_ptr<Request> r) {
@@ -373,7 +383,7 @@ class Scheduler {
     reap_finished();
     current_.clear();
     std::vector<Sequence*> seqs;
-    int need = 0;
+    int need = 0, need_slots = 0;
     for (const Portion& p : portions) {
       Request* r = find_request(p.request_id);
       if (!r || r->finished() || r->cancelled) throw std::runtime_error("portion of an unknown or finished request");
@@ -384,7 +394,9 @@ class Scheduler {
         if (w < 0 || w >= static_cast<int>(p.tokens.size())) throw std::runtime_error("wanted place outside its portion");
       seqs.push_back(s);
       need += blocks_needed(s, s->num_tokens() + static_cast<int>(p.tokens.size()));
+      need_slots += s->state_slot == 0;
     }
+    if (!slots_.empty() && need_slots > slots_[0].num_free()) throw std::runtime_error("no state slot is free for this step's new requests");
     if (need > pool_.at(0).num_available_blocks()) throw std::runtime_error("the KV cache has no room for this step's portions");
     batches_storage_.emplace_back();
     std::vector<Batch>& bs = batches_storage_.back();
@@ -591,7 +603,13 @@ class Scheduler {
     }
   }
 
+  void release_slot(Sequence* s) {
+    if (s->state_slot == 0) return;
+    slots_[s->dp_rank].release(s->state_slot);
+    s->state_slot = 0;
+  }
   void release_blocks(Sequence* s, bool publish) {
+    release_slot(s);
     if (s->blocks.empty()) return;
     BlockManager& bm = pool_.at(s->dp_rank);
     if (publish && s->num_placeholders == 0) {
@@ -828,10 +846,13 @@ class Scheduler {
     }
   }
 
+  // Blocks for `upto_tokens` tokens, and the sequence's state slot if the model keeps state.
   bool ensure_blocks(Sequence* s, int upto_tokens) {
-    int need = blocks_needed(s, upto_tokens);
-    if (need == 0) return true;
-    return pool_.at(s->dp_rank).allocate(need, s->blocks);
+    const bool want_slot = !slots_.empty() && s->state_slot == 0;
+    if (want_slot && slots_[s->dp_rank].num_free() == 0) return false;
+    if (!pool_.at(s->dp_rank).allocate(blocks_needed(s, upto_tokens), s->blocks)) return false;
+    if (want_slot) s->state_slot = slots_[s->dp_rank].acquire();
+    return true;
   }
 
   void preempt(Request* r) {
@@ -970,6 +991,7 @@ class Scheduler {
   }
   // A sequence that was matched against the prefix cache but not admitted must not pin blocks.
   void undo_match(Sequence* s) {
+    release_slot(s);
     if (s->blocks.empty()) return;
     drop_loads_into(s);
     pool_.at(s->dp_rank).release(s->blocks);
@@ -1334,6 +1356,7 @@ class Scheduler {
   StepTimeModel model_;
   double clock_override_ = -1.0;
   BlockManagerPool pool_;
+  std::vector<StateSlots> slots_;                               // one per DP rank (empty: no recurrent state)
   std::mutex mu_;
   std::deque<std::unique_ptr<Request>> incoming_;
   std::vector<int64_t> cancels_;

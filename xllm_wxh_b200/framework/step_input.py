@@ -56,6 +56,7 @@ class StepInput:
         self.next_tokens = buf[L.next_tokens:L.next_tokens + T]
         self.q_cu = buf[L.q_cu:L.q_cu + B + 1]
         self.kv_lens = buf[L.kv_lens:L.kv_lens + B]
+        self.state_slots = buf[L.state_slots:L.state_slots + B]     # slot of recurrent state per sequence (0: none / padding)
         self.block_tables = buf[L.block_tables:L.block_tables + L.B_cap * L.MB_cap].view(L.B_cap, L.MB_cap)[:B]
         self.sample_idx = buf[L.sample_idx:L.sample_idx + S]
         f = lambda off: buf[off:off + S].view(torch.float32)
@@ -68,6 +69,7 @@ class StepInput:
         self.pen_cu = buf[L.pen_cu:L.pen_cu + S + 1]
         self.pen_ids = buf[L.pen_ids:L.pen_ids + L.P_cap]
         self.pen_counts = buf[L.pen_counts:L.pen_counts + L.P_cap]
+        self.states = ()          # per layer run: its recurrent state records [slots, ...] (set by the worker)
         self.header_dev = buf[L.header:L.header + 32]
 
     @property

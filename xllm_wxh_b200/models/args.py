@@ -13,7 +13,8 @@ import json
 import os
 from typing import Any, Dict, List, Optional
 
-from .layer_spec import AttentionSpec, FeedForwardSpec, LayerSpec, run_order
+from .layer_spec import (AttentionSpec, FeedForwardSpec, LayerSpec, ParallelSpec, SelectiveScanSpec, TimeMixSpec, attention_of,
+                         pass_starts, run_order)
 
 @dataclasses.dataclass
 class QuantArgs:
@@ -89,10 +90,13 @@ class ModelArgs:
     # MTP
     num_nextn_predict_layers: int = 0
     quant: QuantArgs = dataclasses.field(default_factory=QuantArgs)
-    # designs that list their layers one by one (models/movolorn.py); the flat sizes above then hold maxima over the layers
+    # designs that list their layers one by one (models/movolorn.py, models/falalix.py); the flat sizes above then hold maxima
+    # over the layers
     layer_specs: List[LayerSpec] = dataclasses.field(default_factory=list)
     layer_runs: List[int] = dataclasses.field(default_factory=list)      # layer of every run, in order (layers may repeat)
+    pass_starts: List[int] = dataclasses.field(default_factory=list)     # run that opens pass t of a looped range
     embedding_scale: float = 1.0
+    residual_mult: float = 1.0          # factor of every sublayer's output on its way into the residual
 
     # ------------------------------------------------------------------ derived
     @property
@@ -160,7 +164,7 @@ def _movolorn_layer(i: int, cfg: Dict[str, Any]) -> LayerSpec:
 
 def args_from_layer_list(specs: List[LayerSpec], runs: List[int], **kw) -> ModelArgs:
     """ModelArgs of a design given layer by layer; the flat sizes that the engine plans with are maxima over the layers."""
-    mix = [s.mixer for s in specs]
+    mix = [a for a in (attention_of(s.mixer) for s in specs) if a is not None] or [AttentionSpec(1, 1, 1, 1, 1.0)]
     ffs = [s.mlp for s in specs if s.mlp is not None]
     inner = [f.shared_ff + f.ff * (f.top_k if f.is_moe else 1) for f in ffs]
     return ModelArgs(layer_specs=specs, layer_runs=runs, n_layers=len(runs), n_heads=max(m.heads for m in mix),
@@ -182,12 +186,52 @@ def _movolorn_args(cfg: Dict[str, Any]) -> ModelArgs:
         eos_token_id=int(_first(cfg, "eos_token_id", default=-1)))
 
 
+def _falalix_layer(i: int, cfg: Dict[str, Any]) -> LayerSpec:
+    kind, m = cfg.get("type"), cfg["mixer"]
+    if kind == "mamba1":
+        mixer = SelectiveScanSpec(inner=int(m["inner"]), state=int(m["state"]), conv=int(m["conv"]), dt_rank=int(m["dt_rank"]))
+        if min(mixer.inner, mixer.state, mixer.conv, mixer.dt_rank) < 1:
+            raise ValueError(f"layer {i}: sizes of a selective scan must be positive")
+    elif kind == "parallel":
+        a, t = m["left"], m["right"]
+        H, G = int(a["heads"]), int(a["kv_heads"])
+        if H < 1 or G < 1 or H % G:
+            raise ValueError(f"layer {i}: {H} heads do not divide over {G} key/value heads")
+        mask = a.get("mask") or {}
+        mixer = ParallelSpec(
+            AttentionSpec(heads=H, kv_heads=G, dim=int(a["dim"]), vdim=int(a["vdim"]), scale=float(a["scale"]),
+                          window=int(mask.get("size") or 0), keep_first=int(mask.get("keep_first") or 0), qk_norm_all=True, qkv_bias=True,
+                          output_gate=True),
+            TimeMixSpec(heads=int(t["heads"]), dim=int(t["dim"])), float(m.get("left_scale", 1.0)), float(m.get("right_scale", 1.0)))
+    else:
+        raise ValueError(f"layer {i}: mixer '{kind}' is not supported")
+    f = cfg.get("mlp")
+    if f and f["kind"] != "dense":
+        raise ValueError(f"layer {i}: feed-forward '{f['kind']}' is not supported")
+    return LayerSpec(mixer, FeedForwardSpec(ff=int(f["ff"]), act="relu2") if f else None)
+
+
+def _falalix_args(cfg: Dict[str, Any]) -> ModelArgs:
+    specs = [_falalix_layer(i, c) for i, c in enumerate(cfg["layers"])]
+    loop = cfg.get("loop") or {}
+    span = (int(loop.get("start", 0)), int(loop.get("stop", 0)), int(loop.get("times", 1)))
+    dt = str(_first(cfg, "torch_dtype", "dtype", default="bfloat16"))
+    return args_from_layer_list(
+        specs, run_order(len(specs), *span), model_type="falalix", dtype=dt if dt in _DTYPES else "bfloat16",
+        pass_starts=pass_starts(len(specs), *span), vocab_size=int(cfg["vocab"]), hidden_size=int(cfg["width"]),
+        rms_norm_eps=float(cfg["norm"]["eps"]), residual_mult=float(cfg.get("residual_mult", 1.0)),
+        max_position_embeddings=int(_first(cfg, "max_position_embeddings", default=131072)),
+        eos_token_id=int(_first(cfg, "eos_token_id", default=-1)))
+
+
 _DTYPES = ("float32", "bfloat16")
+_LAYER_LISTS = {"movolorn": _movolorn_args, "falalix": _falalix_args}     # designs that are named by "architecture"
 
 
 def args_from_hf_config(cfg: Dict[str, Any]) -> ModelArgs:
-    if str(cfg.get("architecture", "")).lower() == "movolorn":
-        return _movolorn_args(cfg)
+    by_layer = _LAYER_LISTS.get(str(cfg.get("architecture", "")).lower())
+    if by_layer is not None:
+        return by_layer(cfg)
     mt = _first(cfg, "model_type", "model_name", default="qwen3")
     a = ModelArgs(model_type=mt)
     a.dtype = {"float32": "float32", "float16": "float16"}.get(str(_first(cfg, "torch_dtype", "dtype", default="bfloat16")),
@@ -354,5 +398,16 @@ def preset(name: str) -> ModelArgs:
         mixer = dict(heads=32, kv_heads=8, dim=128, vdim=128, scale=128 ** -0.5, chunk=8192, distance_bias=True, sink=0.0, qk_norm=True)
         spec = [LayerSpec(AttentionSpec(**mixer), FeedForwardSpec(ff=12288, act="gelu_tanh")) for _ in range(36)]
         return args_from_layer_list(spec, run_order(36), model_type="movolorn", vocab_size=151936, hidden_size=4096,
+                                    max_position_embeddings=40960)
+    if name in ("falalix-8b", "falalix_8b"):
+        # the attention and feed-forward sizes of qwen3-8b beside a time mixing branch of the same width; every second layer a
+        # selective scan of twice the width
+        par = LayerSpec(ParallelSpec(AttentionSpec(heads=32, kv_heads=8, dim=128, vdim=128, scale=128 ** -0.5, window=4096, keep_first=128,
+                                                   qk_norm_all=True, qkv_bias=True, output_gate=True),
+                                     TimeMixSpec(heads=64, dim=64, decay_rank=64), 0.5, 0.5),
+                        FeedForwardSpec(ff=12288, act="relu2"))
+        scan = LayerSpec(SelectiveScanSpec(inner=8192, state=16, conv=4, dt_rank=256), None)
+        spec = [par, scan] * 18
+        return args_from_layer_list(spec, run_order(36), model_type="falalix", vocab_size=151936, hidden_size=4096,
                                     max_position_embeddings=40960)
     raise KeyError(name)

@@ -3,7 +3,7 @@ for designs whose configuration lists the layers one by one instead of giving on
 from __future__ import annotations
 
 import dataclasses
-from typing import List, Optional
+from typing import List, Optional, Union
 
 
 @dataclasses.dataclass
@@ -15,9 +15,13 @@ class AttentionSpec:
     scale: float                  # factor of q . k
     chunk: int = 0                # positions per chunk that a query may look at (0: all earlier ones)
     window: int = 0               # sliding window in positions (0: none)
+    keep_first: int = 0           # first positions of the sequence that stay visible behind the window
     distance_bias: bool = False   # take slope_h * (i - j) off the scores, slopes from `head_slopes`
     sink: Optional[float] = None  # score of a key without a value that joins the softmax denominator (None: no sink)
     qk_norm: bool = False         # RMS norm over every query and key head
+    qk_norm_all: bool = False     # RMS norm over the whole query and the whole key projection, ahead of the split into heads
+    qkv_bias: bool = False        # biases on the query, key and value projections
+    output_gate: bool = False     # the heads' outputs times sigmoid of a projection of the layer's input
 
     def head_slopes(self) -> List[float]:
         """Geometric slopes 2^(-8 (h + 1) / H), h = 0 .. H - 1."""
@@ -25,9 +29,47 @@ class AttentionSpec:
 
 
 @dataclasses.dataclass
+class TimeMixSpec:
+    """Linear attention with a matrix state per head, a data-dependent decay per key channel and a bonus for the current
+    token; its inputs are blends of every token with the one before it."""
+    heads: int
+    dim: int                      # key and value size of a head
+    decay_rank: int = 0           # inner size of the decay's low-rank projection (0: the checkpoint's tensors tell)
+
+
+@dataclasses.dataclass
+class SelectiveScanSpec:
+    """Diagonal state space layer with data-dependent step sizes, input and output vectors, behind a short causal
+    convolution."""
+    inner: int                    # channels
+    state: int                    # states per channel
+    conv: int                     # taps of the convolution
+    dt_rank: int                  # inner size of the step sizes' low-rank projection
+
+
+@dataclasses.dataclass
+class ParallelSpec:
+    """Two mixers side by side on the same input; their outputs are added with a factor each."""
+    left: AttentionSpec
+    right: TimeMixSpec
+    left_scale: float = 1.0
+    right_scale: float = 1.0
+
+
+Mixer = Union[AttentionSpec, SelectiveScanSpec, ParallelSpec]
+
+
+def attention_of(mixer: Mixer) -> Optional[AttentionSpec]:
+    """The attention part of a mixer: what its layer keeps in the paged cache (None: nothing)."""
+    if isinstance(mixer, ParallelSpec):
+        return mixer.left
+    return mixer if isinstance(mixer, AttentionSpec) else None
+
+
+@dataclasses.dataclass
 class FeedForwardSpec:
     ff: int                       # inner size (of one expert in a mixture)
-    act: str                      # gate activation: "silu" | "gelu_tanh"
+    act: str                      # gate activation "silu" | "gelu_tanh", or "relu2": squared relu without a gate
     experts: int = 0              # experts with weights (0: a dense feed-forward)
     identity_experts: int = 0     # router outputs behind them whose expert is the identity
     top_k: int = 0
@@ -45,7 +87,7 @@ class FeedForwardSpec:
 
 @dataclasses.dataclass
 class LayerSpec:
-    mixer: AttentionSpec
+    mixer: Mixer
     mlp: Optional[FeedForwardSpec]      # None: the layer has no feed-forward sublayer
 
 
@@ -54,3 +96,9 @@ def run_order(n_layers: int, start: int = 0, stop: int = 0, times: int = 1) -> L
     if not 0 <= start <= stop <= n_layers or times < 1:
         raise ValueError(f"bad layer loop: start {start}, stop {stop}, times {times} with {n_layers} layers")
     return list(range(start)) + list(range(start, stop)) * times + list(range(stop, n_layers))
+
+
+def pass_starts(n_layers: int, start: int = 0, stop: int = 0, times: int = 1) -> List[int]:
+    """Index in `run_order` of the first run of every pass through the loop (empty: no loop)."""
+    run_order(n_layers, start, stop, times)
+    return [start + t * (stop - start) for t in range(times)] if stop > start else []

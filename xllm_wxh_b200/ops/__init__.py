@@ -45,14 +45,14 @@ def paged_attention(q, k_cache, v_cache, inp, scale, sliding_window=-1):
                                sliding_window)
 
 
-def paged_attention_ext(q, k_cache, v_cache, inp, scale, window=-1, chunk=0, slopes=None, sinks=None):
+def paged_attention_ext(q, k_cache, v_cache, inp, scale, window=-1, chunk=0, slopes=None, sinks=None, keep_first=0):
     """Paged attention with a per-head linear distance bias (`slopes` [Hq] fp32), a per-head sink score in the softmax
-    denominator (`sinks` [Hq] fp32), keys limited to the query's chunk of `chunk` positions, and a value head dimension of
-    its own.  q [T, Hq, dk] -> [T, Hq * dv]."""
+    denominator (`sinks` [Hq] fp32), keys limited to the query's chunk of `chunk` positions, first positions that stay
+    visible behind the window (`keep_first`), and a value head dimension of its own.  q [T, Hq, dk] -> [T, Hq * dv]."""
     if q.is_cuda:
-        return _cuda().paged_attention_ext(q, k_cache, v_cache, inp, scale, window, chunk, slopes, sinks)
+        return _cuda().paged_attention_ext(q, k_cache, v_cache, inp, scale, window, chunk, slopes, sinks, keep_first)
     return ref.paged_attention(q, k_cache, v_cache, inp.q_cu, inp.kv_lens, inp.block_tables, inp.n_seqs, scale, window, chunk,
-                               slopes, sinks)
+                               slopes, sinks, keep_first)
 
 
 def sample(logits, inp):
@@ -139,6 +139,77 @@ def moe_post_norm_add_norm(h_in, w13, w2, weights, ids, shared, first_identity, 
         return moe_cuda.combine_post_norm_add_norm(y, dst_of, ids, weights, h_in, shared, first_identity, x, w_post, w_next, eps)
     y = ref.moe_mixture(h_in, w13, w2, weights, ids, shared, first_identity, act)
     return ref.post_norm_add_norm(y, x, w_post, w_next, eps)
+
+
+# ----------------------------------------------------------------------------- sublayers normed before only, fp32 residual
+def add_norm(y, x, mult, w_next, eps):
+    """x += mult * y (x fp32, in place); returns rms(x) * w_next."""
+    return (_cuda() if y.is_cuda else ref).add_norm(y, x, mult, w_next, eps)
+
+
+def replace_norm(y, vec, x, w_next, eps):
+    """x = y + vec (y, x fp32; vec one row); returns rms(x) * w_next."""
+    return (_cuda() if y.is_cuda else ref).replace_norm(y, vec, x, w_next, eps)
+
+
+def split_rows(x, x0):
+    """Rows [x, x0] for a product with `split_columns` of its weight.  In a bf16 model the fp32 x enters as two bf16 parts
+    (its rounded value and the rest), so that a product of the residual stream does not round it to 8 bits."""
+    return (_cuda() if x.is_cuda else ref).split_rows(x, x0)
+
+
+def split_columns(w, width):
+    """Weight [N, 2 width] of a product of [x, x0] in the column layout of `split_rows`."""
+    import torch
+    return w if w.dtype == torch.float32 else torch.cat([w[:, :width], w], 1).contiguous()
+
+
+def act_linear(x, w, act):
+    """act(x w^T), applied to the fp32 sums: "relu2" (squared relu) | "tanh"."""
+    return (_cuda() if x.is_cuda else ref).act_linear(x, w, act)
+
+
+def qknorm_all_kvwrite(qkv, slots, q_w, k_w, eps, k_cache, v_cache, n_q, n_kv):
+    """RMSNorm over the whole query and the whole key projection; k and v into the paged caches.  Rows of qkv may be longer
+    than q, k and v.  Returns q [T, n_q * dk]."""
+    return (_cuda() if qkv.is_cuda else ref).qknorm_all_kvwrite(qkv, slots, q_w, k_w, eps, k_cache, v_cache, n_q, n_kv)
+
+
+def gate_into(o, gate, scale, out):
+    """out = o * sigmoid(gate) * scale (gate and out may be strided views)."""
+    (_cuda() if o.is_cuda else ref).gate_into(o, gate, scale, out)
+
+
+# ----------------------------------------------------------------------------- recurrent layers
+# State tensors hold one record per state slot; `inp.state_slots` names each sequence's, and it is updated in place.
+def _seqs(inp):
+    return inp.q_cu, inp.kv_lens, inp.state_slots, inp.n_seqs
+
+
+def token_shift(h, mu, last, inp):
+    """[n, T, W]: every row of h blended with its predecessor by each of the n rows of mu; `last` [slots, W] is the state."""
+    return _cuda().token_shift(h, mu, last, inp) if h.is_cuda else ref.token_shift(h, mu, last, *_seqs(inp))
+
+
+def time_mix(r, k, v, z, w0, u, gate, norm_w, scale, eps, state, inp, out):
+    """Matrix-state recurrence with a decay exp(-exp(z + w0)) per key channel and the bonus u for the current token; per-head
+    RMS, weight, silu gate and `scale` on its output, which goes to `out` (may be a strided view)."""
+    if r.is_cuda:
+        _cuda().time_mix(r, k, v, z, w0, u, gate, norm_w, scale, eps, state, inp, out)
+    else:
+        ref.time_mix(r, k, v, z, w0, u, gate, norm_w, scale, eps, state, *_seqs(inp), out)
+
+
+def conv_silu(x, w, b, state, inp):
+    """silu of a causal convolution per channel over each sequence; x may be a strided view; state [slots, taps - 1, C]."""
+    return _cuda().conv_silu(x, w, b, state, inp) if x.is_cuda else ref.conv_silu(x, w, b, state, *_seqs(inp))
+
+
+def selective_scan(x, dt, dt_bias, A, B, C, D, z, state, inp):
+    """Diagonal state space recurrence with data-dependent steps softplus(dt + dt_bias); returns (scan + D x) silu(z)."""
+    if x.is_cuda:
+        return _cuda().selective_scan(x, dt, dt_bias, A, B, C, D, z, state, inp)
+    return ref.selective_scan(x, dt, dt_bias, A, B, C, D, z, state, *_seqs(inp))
 
 
 # ----------------------------------------------------------------------------- MLA (DeepSeek)

@@ -144,11 +144,12 @@ def rope_qknorm_kvwrite(qkv: torch.Tensor, positions: torch.Tensor, slots: torch
 def paged_attention(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tensor, q_cu: torch.Tensor,
                     kv_lens: torch.Tensor, block_tables: torch.Tensor, n_seqs: int, scale: float,
                     sliding_window: int = -1, chunk: int = 0, slopes: Optional[torch.Tensor] = None,
-                    sinks: Optional[torch.Tensor] = None) -> torch.Tensor:
+                    sinks: Optional[torch.Tensor] = None, keep_first: int = 0) -> torch.Tensor:
     """Causal attention of ragged query rows over paged KV.
     q [T, Hq, D]; caches [n_blocks, block, Hkv, D]; sequence i owns q rows q_cu[i]:q_cu[i+1], which are the
     last rows of its kv_lens[i] tokens.  `chunk` > 0: a query sees keys of its own chunk of positions only; `slopes` [Hq]:
-    slopes[h] * (query position - key position) is taken off the scores; `sinks` [Hq]: exp(sinks[h]) joins the denominator."""
+    slopes[h] * (query position - key position) is taken off the scores; `sinks` [Hq]: exp(sinks[h]) joins the denominator;
+    `keep_first`: so many first positions stay visible behind the window."""
     T, Hq, D = q.shape
     block = k_cache.shape[1]
     Hkv = k_cache.shape[2]
@@ -175,7 +176,7 @@ def paged_attention(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tenso
         kpos = torch.arange(L, device=q.device)[None, :]
         mask = kpos <= qpos
         if sliding_window > 0:
-            mask &= kpos > qpos - sliding_window
+            mask &= (kpos > qpos - sliding_window) | (kpos < keep_first)
         if chunk > 0:
             mask &= torch.div(kpos, chunk, rounding_mode="floor") == torch.div(qpos, chunk, rounding_mode="floor")
         if slopes is not None:
@@ -392,6 +393,110 @@ def qknorm_kvwrite(qkv, slots, q_w, k_w, eps, k_cache, v_cache, n_q, n_kv):
     k_cache.view(-1, n_kv, dk).index_copy_(0, slots.long(), k.to(k_cache.dtype))
     v_cache.view(-1, n_kv, dv).index_copy_(0, slots.long(), v.reshape(T, n_kv, dv).to(v_cache.dtype))
     return q.reshape(T, n_q * dk)
+
+
+# norms ahead of a sublayer only, around an fp32 residual stream
+def add_norm(y: torch.Tensor, x: torch.Tensor, mult: float, w_next: torch.Tensor, eps: float) -> torch.Tensor:
+    x += mult * y.float()
+    return _rms_f32(x, w_next, eps).to(w_next.dtype)
+
+
+def replace_norm(y: torch.Tensor, vec: torch.Tensor, x: torch.Tensor, w_next: torch.Tensor, eps: float) -> torch.Tensor:
+    x.copy_(y + vec.float())
+    return _rms_f32(x, w_next, eps).to(w_next.dtype)
+
+
+def split_rows(x: torch.Tensor, x0: torch.Tensor) -> torch.Tensor:
+    """[x, x0] as the input of a product; an fp32 x in a bf16 model enters as its bf16 value and what that leaves."""
+    if x0.dtype == torch.float32:
+        return torch.cat([x, x0], -1)
+    hi = x.to(x0.dtype)
+    return torch.cat([hi, (x - hi.float()).to(x0.dtype), x0], -1)
+
+
+def act_linear(x: torch.Tensor, w: torch.Tensor, act: str) -> torch.Tensor:
+    y = torch.nn.functional.linear(x.float(), w.float())
+    return (torch.relu(y) ** 2 if act == "relu2" else torch.tanh(y)).to(x.dtype)
+
+
+def qknorm_all_kvwrite(qkv, slots, q_w, k_w, eps, k_cache, v_cache, n_q, n_kv):
+    dk, dv = k_cache.shape[-1], v_cache.shape[-1]
+    q, k, v = qkv[:, :(n_q + n_kv) * dk + n_kv * dv].split([n_q * dk, n_kv * dk, n_kv * dv], dim=-1)
+    k_cache.view(-1, n_kv * dk).index_copy_(0, slots.long(), _rms_f32(k, k_w, eps).to(k_cache.dtype))
+    v_cache.view(-1, n_kv * dv).index_copy_(0, slots.long(), v.to(v_cache.dtype))
+    return _rms_f32(q, q_w, eps).to(qkv.dtype)
+
+
+def gate_into(o: torch.Tensor, gate: torch.Tensor, scale: float, out: torch.Tensor) -> None:
+    out.copy_(o.float() * torch.sigmoid(gate.float()) * scale)
+
+
+# ----------------------------------------------------------------------------- recurrent layers
+# `q_cu`, `kv_lens` as for attention: sequence i owns rows q_cu[i]:q_cu[i + 1], the last ones of its kv_lens[i] tokens, and
+# record slots[i] of the state tensors, which are updated in place; a sequence at its first token starts from zero.
+def _spans(q_cu, kv_lens, slots, n_seqs):
+    a, k, s = q_cu.tolist(), kv_lens.tolist(), slots.tolist()
+    return [(a[i], a[i + 1], k[i] > a[i + 1] - a[i], s[i]) for i in range(n_seqs) if a[i + 1] > a[i]]
+
+
+def token_shift(h, mu, last, q_cu, kv_lens, slots, n_seqs):
+    """[n, T, W]: h + (previous row of the sequence - h) * mu[i] for every row of mu; `last` [slots, W] keeps the last row."""
+    prev = torch.zeros_like(h)
+    for lo, hi, cont, s in _spans(q_cu, kv_lens, slots, n_seqs):
+        prev[lo + 1:hi] = h[lo:hi - 1]
+        if cont:
+            prev[lo] = last[s]
+        last[s] = h[hi - 1]
+    hf = h.float()
+    return (hf + (prev.float() - hf) * mu.float()[:, None]).to(h.dtype)
+
+
+def time_mix(r, k, v, z, w0, u, gate, norm_w, scale, eps, state, q_cu, kv_lens, slots, n_seqs, out):
+    """r, k, v, gate [T, H * d]; z [T, H * d] fp32: decay = exp(-exp(z + w0)); u [H, d] fp32; state [slots, H, d, d] fp32 (key,
+    value).  out [T, H * d] = o / rms(o per head) * norm_w * silu(gate) * scale."""
+    H, d = u.shape
+    T = r.shape[0]
+    R, K, V = (t.float().view(T, H, d) for t in (r, k, v))
+    W = torch.exp(-torch.exp(z + w0)).view(T, H, d)
+    o = torch.zeros(T, H, d)
+    for lo, hi, cont, s in _spans(q_cu, kv_lens, slots, n_seqs):
+        S = state[s].clone() if cont else torch.zeros_like(state[s])
+        for t in range(lo, hi):
+            kv = K[t][:, :, None] * V[t][:, None, :]
+            o[t] = torch.einsum("hk,hkv->hv", R[t], S + u[:, :, None] * kv)
+            S = W[t][:, :, None] * S + kv
+        state[s] = S
+    o = o * torch.rsqrt(o.pow(2).mean(-1, keepdim=True) + eps)
+    out.copy_(o.view(T, H * d) * norm_w.float() * torch.nn.functional.silu(gate.float()) * scale)
+
+
+def conv_silu(x, w, b, state, q_cu, kv_lens, slots, n_seqs):
+    """Causal convolution of every channel (w [C, taps], last column the current row) + b, then silu; state [slots, taps - 1, C]
+    keeps the last rows."""
+    taps = w.shape[1]
+    y = torch.zeros(x.shape, dtype=torch.float32)
+    for lo, hi, cont, s in _spans(q_cu, kv_lens, slots, n_seqs):
+        rows = torch.cat([state[s] if cont else torch.zeros_like(state[s]), x[lo:hi]])
+        y[lo:hi] = sum(rows[i:i + hi - lo].float() * w[:, i].float() for i in range(taps)) + b.float()
+        if taps > 1:
+            state[s] = rows[1 - taps:]
+    return torch.nn.functional.silu(y).to(x.dtype)
+
+
+def selective_scan(x, dt, dt_bias, A, B, C, D, z, state, q_cu, kv_lens, slots, n_seqs):
+    """x, z [T, c]; dt [T, c] fp32 (ahead of bias and softplus); A [c, n] fp32 (negative); B, C [T, n]; state [slots, c, n]
+    fp32.  Returns (scan + D x) silu(z)."""
+    T = x.shape[0]
+    xf, Bf, Cf = x.float(), B.float(), C.float()
+    step = torch.nn.functional.softplus(dt + dt_bias)
+    y = torch.zeros(T, x.shape[1])
+    for lo, hi, cont, s in _spans(q_cu, kv_lens, slots, n_seqs):
+        S = state[s].clone() if cont else torch.zeros_like(state[s])
+        for t in range(lo, hi):
+            S = torch.exp(step[t][:, None] * A) * S + (step[t] * xf[t])[:, None] * Bf[t]
+            y[t] = S @ Cf[t]
+        state[s] = S
+    return ((y + D * xf) * torch.nn.functional.silu(z.float())).to(x.dtype)
 
 
 def moe_experts_fp8(x, w13_deq, w2_deq, weights, ids, expert_offset=0):

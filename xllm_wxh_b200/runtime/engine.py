@@ -80,6 +80,7 @@ class LLMEngine:
             self._load_model()
         self._setup_parallel_kernels()
         self.block_size = self.opt.block_size
+        n_slots = self._plan_state()
         nb = self.worker.profile_kv_blocks()
         if self.world_size > 1:
             t = torch.tensor([nb], dtype=torch.int64, device=self.device)
@@ -89,6 +90,7 @@ class LLMEngine:
         # the cache that another instance maps: the decode side's when KV is pushed, the prefill side's when it is pulled
         mapped_role = "PREFILL" if self.opt.kv_cache_transfer_mode == "PULL" else "DECODE"
         self.worker.allocate_kv_cache(nb, ipc=self.opt.enable_disagg_pd and self.opt.instance_role == mapped_role)
+        self.worker.allocate_state_cache()
         self.worker._ensure_staging(self._max_message_words() // max(1, self.opt.dp_size))
         # host-memory tier of the prefix cache (every rank keeps the host copy of its own shard of each block)
         self.host_tier = None
@@ -141,6 +143,7 @@ class LLMEngine:
             so.chunked_match_frequency = self.opt.chunked_match_frequency
             so.dp_size = self.opt.dp_size
             so.handoff_after_prefill = self.opt.enable_disagg_pd and self.opt.instance_role == "PREFILL"
+            so.num_state_slots = n_slots
             so.host_blocks_factor = self.opt.host_blocks_factor if self.host_tier is not None else 0.0
             so.use_mix_scheduler = self.opt.use_mix_scheduler
             so.enable_latency_aware_schedule = self.opt.enable_latency_aware_schedule
@@ -213,6 +216,24 @@ class LLMEngine:
             m.load_weights(CheckpointReader(self.model_dir))
         if hasattr(m, "finalize_weights"):
             m.finalize_weights()
+
+    def _plan_state(self) -> int:
+        """Slots of recurrent state (0: the model keeps none).  A state belongs to one position of one sequence: it cannot be
+        shared between prompts, rolled back behind rejected draft tokens or sent on block by block, so the features that
+        rest on those are switched off or refused."""
+        n = self.worker.plan_state_slots()
+        if n == 0:
+            return 0
+        if self.world_size > 1 or self.opt.dp_size > 1:
+            raise ValueError("models with recurrent state run on one device")
+        if self.opt.num_speculative_tokens > 0:
+            raise ValueError("speculative decoding is not possible with recurrent state")
+        if self.opt.enable_disagg_pd:
+            raise ValueError("disaggregated prefill is not implemented for models with recurrent state")
+        if self.opt.enable_prefix_cache:
+            log.info("prefix cache off: the model keeps recurrent state")
+            self.opt.enable_prefix_cache = False
+        return n
 
     def _setup_parallel_kernels(self):
         if self.world_size > 1 and self.device.type == "cuda":

@@ -113,11 +113,12 @@ def sleep_rank(engine, level: int) -> int:
     if w._graphs is not None:
         w._graphs.invalidate()
         w._graphs = None
-    freed = sum(t.numel() * t.element_size() for layer in w.kv_caches for t in layer)
+    freed = sum(t.numel() * t.element_size() for layer in w.kv_caches + w.state_caches for t in layer)
     if engine.host_tier is not None:
         engine.host_tier.drain()
         engine.host_tier.detach()
     w.kv_caches = []
+    w.state_caches = []
     aliases: Dict[Tuple, Any] = {}                 # tied weights (lm_head = embedding) stay one tensor
     order: Dict[Tuple, int] = {}
     st.manifest, st.slots = [], []
@@ -178,6 +179,7 @@ def wakeup_rank(engine, source=None) -> None:
     else:
         engine._load_model()
     w.allocate_kv_cache(engine.num_blocks, ipc=engine.opt.enable_disagg_pd and engine.opt.instance_role == "DECODE")
+    w.allocate_state_cache()
     if engine.host_tier is not None:
         engine.host_tier.attach(w.kv_caches)
     if dev.type == "cuda":

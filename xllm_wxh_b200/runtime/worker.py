@@ -76,7 +76,9 @@ class Worker:
         dtype = {"auto": None, "bfloat16": torch.bfloat16, "float16": torch.float16, "float32": torch.float32}[options.dtype]
         self.model = model if model is not None else get_model_class(args.model_type)(args, self.comm, self.device, dtype)
         self.kv_caches: List[Tuple[torch.Tensor, ...]] = []
+        self.state_caches: List[Tuple[torch.Tensor, ...]] = []     # per layer run, records of `num_state_slots` + 1 slots
         self.num_blocks = 0
+        self.num_state_slots = 0
         self.block_size = options.block_size
         self._layouts: Dict[Tuple[int, int, int, int, int], "_core.BatchLayout"] = {}
         self._host: Optional[torch.Tensor] = None
@@ -103,7 +105,7 @@ class Worker:
         """How many KV blocks fit (reference: llm_engine.cpp:375-530 estimate_kv_cache_capacity)."""
         if self.opt.num_kv_blocks > 0:
             return self.opt.num_kv_blocks
-        per_block = self.kv_bytes_per_block()
+        per_block = max(1, self.kv_bytes_per_block())
         if self.opt.max_cache_size > 0:
             return max(2, int(self.opt.max_cache_size // per_block))
         if self.is_cuda:
@@ -114,9 +116,38 @@ class Worker:
             act = self.opt.max_tokens_per_batch * (a.hidden_size * 12 + a.intermediate_size // max(1, self.comm.tp_size) * 6 +
                                                    0) * 2
             act += 1024 * a.vocab_size * 4 // max(1, self.comm.tp_size) * 3
-            budget -= act + (2 << 30)
-            return max(2, int(budget // per_block))
+            budget -= act + (2 << 30) + (self.num_state_slots + 1) * self.state_bytes_per_slot()
+            # no more than every sequence at full length can use (a model may have few attention layers, or none)
+            useful = self.opt.max_seqs_per_batch * (a.max_position_embeddings // self.block_size + 1) + 1
+            return max(2, int(min(budget // per_block, max(useful, 2)) if self.state_bytes_per_slot() else budget // per_block))
         return 1024
+
+    # ------------------------------------------------------------------ recurrent state
+    def _state_shapes(self, slots: int):
+        f = getattr(self.model, "state_cache_shapes", None)
+        return f(slots) if f is not None else []
+
+    def state_bytes_per_slot(self) -> int:
+        """Bytes of recurrent state that one sequence holds over all layers (0: the model keeps none)."""
+        return sum(int(np.prod(s)) * torch.empty((), dtype=dt).element_size() for run in self._state_shapes(1) for s, dt in run)
+
+    def plan_state_slots(self) -> int:
+        """How many sequences can hold state at a time: as many as a batch has, within a quarter of the free memory."""
+        per = self.state_bytes_per_slot()
+        n = 0 if per == 0 else self.opt.num_state_slots
+        if per and n <= 0:
+            n = self.opt.max_seqs_per_batch
+            if self.is_cuda:
+                n = max(1, min(n, int(torch.cuda.mem_get_info(self.device)[0] // 4 // per)))
+        self.num_state_slots = n
+        return n
+
+    def allocate_state_cache(self):
+        """Records of every slot and of the padding slot 0.  They need no clearing: a sequence starts from zero, not from
+        what its slot holds (zeroed here once so that nothing is ever undefined)."""
+        if self.num_state_slots > 0:
+            self.state_caches = [tuple(torch.zeros(s, dtype=dt, device=self.device) for s, dt in run)
+                                 for run in self._state_shapes(self.num_state_slots + 1)]
 
     def kv_bytes_per_block(self) -> int:
         shapes = self.model.kv_cache_shapes(1, self.block_size)
@@ -234,6 +265,7 @@ class Worker:
             self._dev[:L.total_words].copy_(host[:L.total_words], non_blocking=True)
             self.h2d_bytes += L.total_words * 4
         inp = StepInput(self._dev, L, header, padded=padded)
+        inp.states = self.state_caches
         if patch_placeholders and self._last_tokens is not None:
             # token id -(j+1) stands for "j-th sample of the previous step"
             tok = inp.tokens

@@ -8,7 +8,7 @@ Every input line is one engine step:
 
 Its entries run as one batch: the next tokens of each named request, behind what earlier steps left in the cache.  `want`
 lists places among those tokens; their logits go to <out>/<step>.f32 as little-endian fp32 [wanted, vocab], entry by entry.
-Requests under `end` are over after the step and give their blocks back.  `done <step>` is printed when a step is complete.
+Requests under `end` are over after the step and give their blocks and state slots back.  `done <step>` is printed when a step is complete.
 Nothing is sampled; batches, blocks, kernels and CUDA graphs are those of generation (`LLMEngine.step_portions`).
 """
 from __future__ import annotations
@@ -20,6 +20,7 @@ import sys
 from typing import Dict, List, Optional
 
 BLOCK = 64          # tokens per KV block
+LIVE = 4            # requests that may hold recurrent state at a time, in models that keep any
 
 
 def main(argv: Optional[List[str]] = None) -> int:
@@ -37,7 +38,7 @@ def main(argv: Optional[List[str]] = None) -> int:
     from ..config import Options
     from ..runtime.engine import LLMEngine
     blocks = (a.max_tokens + BLOCK - 1) // BLOCK
-    engine = LLMEngine(Options(model=a.model, devices=a.device, dtype=a.dtype, block_size=BLOCK, num_kv_blocks=blocks + 1,
+    engine = LLMEngine(Options(model=a.model, devices=a.device, dtype=a.dtype, block_size=BLOCK, num_kv_blocks=blocks + 1, num_state_slots=LIVE,
                                max_tokens_per_batch=max(64, a.max_tokens), max_seqs_per_batch=64, enable_prefix_cache=False,
                                max_model_len=max(64, blocks * BLOCK), enable_numa_binding=False))
     os.makedirs(a.out, exist_ok=True)
