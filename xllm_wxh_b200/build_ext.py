@@ -116,6 +116,8 @@ def cuda_sources():
 MODEL_SOURCES = {
     "movolorn": ("attention_decode_tma", "attention_prefill_tc", "attention_simt", "gemm_bf16", "gemm_bf16_2cta", "gemm_simt",
                  "host_util", "moe", "sampling", "sandwich_norm"),
+    "falalix": ("attention_decode_tma", "attention_prefill_tc", "attention_simt", "gemm_bf16", "gemm_bf16_2cta", "gemm_simt",
+                "host_util", "recurrent", "sampling", "sandwich_norm"),
 }
 
 

@@ -13,8 +13,8 @@
 // bounds a decode kernel whose arithmetic intensity is a few FLOP per byte.
 //
 // Template parameters: DK / DV = query-key / value head dimension padded to 64 or 128 (the TMA loads fill the padding with
-// zeros), EXT = score extensions (per-head distance bias, per-head sink, chunk mask) and head dimensions below the padded
-// ones.
+// zeros), EXT = score extensions (per-head distance bias, per-head sink, chunk mask, first keys that stay visible behind a
+// window) and head dimensions below the padded ones.
 //
 // Role: the reference's FlashInfer `batch_decode_with_kv_cache` (xllm/core/kernels/cuda/batch_decode.cpp:26-85).
 #include "common.cuh"
@@ -65,6 +65,7 @@ struct DecParams {
   // score extensions (EXT): see xl_prefill_attention_ext
   int dk = 0, dv = 0;
   int chunk = 0;
+  int keep_first = 0;
   const float* slopes = nullptr;
   const float* sinks = nullptr;
 };
@@ -114,11 +115,14 @@ __global__ void __launch_bounds__(160) decode_attn_tma_kernel(const __grid_const
 
   int r_begin = 0;                                // first key that any row may see, rounded down to a tile
   if (EXT && p.chunk > 0) r_begin = (kv_len - q_len) / p.chunk * p.chunk / kTile * kTile;
-  const int per_split = ((kv_len - r_begin + p.num_splits - 1) / p.num_splits + kTile - 1) / kTile * kTile;
-  int s_begin = r_begin + split * per_split;
-  const int s_end = min(kv_len, s_begin + per_split);
-  if (p.window > 0) s_begin = max(s_begin, (max(0, kv_len - q_len - p.window + 1)) / kTile * kTile);
-  const int n_tiles = s_end > s_begin ? (s_end - s_begin + kTile - 1) / kTile : 0;
+  if (p.window > 0) r_begin = max(r_begin, max(0, kv_len - q_len - p.window + 1) / kTile * kTile);
+  const int n_keep = EXT ? (min(p.keep_first, r_begin) + kTile - 1) / kTile : 0;      // tiles of kept first keys ahead of it
+  const int all_tiles = n_keep + (kv_len - r_begin + kTile - 1) / kTile;
+  const int per_split = (all_tiles + p.num_splits - 1) / p.num_splits;
+  const int t_first = split * per_split;
+  const int n_tiles = max(0, min(all_tiles, t_first + per_split) - t_first);
+  // first key of this split's t-th tile
+  auto tile_kv = [&](int t) { return t_first + t < n_keep ? (t_first + t) * kTile : r_begin + (t_first + t - n_keep) * kTile; };
 
   if (threadIdx.x == 0) {
     for (int s = 0; s < kStages; ++s) {
@@ -161,8 +165,8 @@ __global__ void __launch_bounds__(160) decode_attn_tma_kernel(const __grid_const
           ok = false;
           break;
         }
-        const int base = s_begin + t * kTile;
-        const int n_tok = min(kTile, s_end - base);
+        const int base = tile_kv(t);
+        const int n_tok = min(kTile, kv_len - base);
         const int n_boxes = (n_tok + bt_tok - 1) / bt_tok;
         mbar_arrive_expect_tx(&bars->full[s], uint32_t(n_boxes) * bt_tok * 128 * (KH + VH));
         uint8_t* dK = ring + s * STAGE_BYTES;
@@ -218,8 +222,8 @@ __global__ void __launch_bounds__(160) decode_attn_tma_kernel(const __grid_const
         if (lane == 0) atomicExch(p.status, XL_ERR_WAIT_FULL);
         break;
       }
-      const int base = s_begin + t * kTile + warp * 16;
-      if (base < s_end) {
+      const int base = tile_kv(t) + warp * 16;
+      if (base < kv_len) {
         const uint8_t* tK = ring + s * STAGE_BYTES + warp * 2048;
         const uint8_t* tV = tK + K_BYTES;
         float sc[2][4];
@@ -240,8 +244,8 @@ __global__ void __launch_bounds__(160) decode_attn_tma_kernel(const __grid_const
           for (int e = 0; e < 4; ++e) {
             const int tok = base + i * 8 + (lane & 3) * 2 + (e & 1);
             const int lim = (e < 2) ? lim_a : lim_b;
-            bool ok = tok <= lim && tok < s_end;
-            if (p.window > 0) ok = ok && tok > lim - p.window;
+            bool ok = tok <= lim && tok < kv_len;
+            if (p.window > 0) ok = ok && (tok > lim - p.window || (EXT && tok < p.keep_first));
             float x = sc[i][e] * p.scale_log2;
             if (EXT) {
               ok = ok && tok >= ((e < 2) ? lo_a : lo_b);
@@ -550,10 +554,11 @@ __global__ void split_merge_ext_kernel(const float* __restrict__ part_o, const f
 XL_API int xl_decode_attention_ext(const void* q, const void* k_cache, const void* v_cache, void* out, const void* q_cu,
                                    const void* kv_lens, const void* block_tables, int seq_begin, int seq_end, int max_blocks,
                                    int block_size, int num_blocks_total, int n_q, int n_kv, int dk, int dv, int q_stride,
-                                   float scale, int window, int chunk, const void* slopes, const void* sinks, int num_splits,
-                                   void* part_o, void* part_lse, long max_rows, const void* dyn_end, void* stream) {
+                                   float scale, int window, int chunk, int keep_first, const void* slopes, const void* sinks,
+                                   int num_splits, void* part_o, void* part_lse, long max_rows, const void* dyn_end, void* stream) {
   using namespace xl_dec;
   if (seq_end <= seq_begin) return 0;
+  if (chunk > 0 && keep_first > 0) return -2;
   if (dk < 8 || dk > 128 || dk % 8 || dv < 8 || dv > 128 || dv % 8) return -3;
   if (block_size % 16 != 0 || (block_size > 64 && block_size % 64 != 0) || (block_size < 64 && 64 % block_size != 0)) return -3;
   if (n_q % n_kv || n_q / n_kv > 16) return -3;
@@ -583,7 +588,7 @@ XL_API int xl_decode_attention_ext(const void* q, const void* k_cache, const voi
   p.box_tokens = box_tokens;
   p.status = xl_host::status_word();
   p.dyn_end = static_cast<const int*>(dyn_end);
-  p.dk = dk; p.dv = dv; p.chunk = chunk;
+  p.dk = dk; p.dv = dv; p.chunk = chunk; p.keep_first = keep_first;
   p.slopes = static_cast<const float*>(slopes);
   p.sinks = static_cast<const float*>(sinks);
   if (p.num_splits > 1 && (!part_o || !part_lse)) return -2;

@@ -18,7 +18,8 @@
 //                   by the row sum), final O / l stored as bf16.
 // Template parameters: QS / VS = 64-column slabs of the query-key / value head dimension (a dimension that does not fill
 // its slabs is padded with zeros by the TMA loads), EXT = score extensions: per-head linear distance bias, per-head sink
-// (a score that joins the denominator and has no value), chunk mask (a query sees keys of its own position chunk only).
+// (a score that joins the denominator and has no value), chunk mask (a query sees keys of its own position chunk only),
+// first keys that stay visible behind a window (their tiles come ahead of the window's, the gap between is not read).
 // QK^T of tile j+1 is issued before P V of tile j, so the tensor pipe works while the softmax warps are busy.
 // Every wait is bounded; on expiry the kernel records a status code and leaves.
 #include <string.h>
@@ -62,6 +63,7 @@ struct Params {
   const float* slopes;         // EXT: [Hq] distance-bias slopes (null: none): score -= slope * (query pos - key pos)
   const float* sinks;          // EXT: [Hq] sink scores (null: none): denominator += exp(sink)
   int chunk;                   // EXT: positions per chunk (<= 0: no chunk mask)
+  int keep_first;              // EXT: first keys that stay visible behind the window
   const int* q_cu;
   const int* kv_lens;
   const int* block_tables;
@@ -164,7 +166,8 @@ prefill_attn_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_con
   int kv_begin = 0;
   if (p.window > 0) kv_begin = max(0, pos0 - p.window + 1) / BKV * BKV;
   if (EXT && p.chunk > 0) kv_begin = max(kv_begin, pos0 / p.chunk * p.chunk / BKV * BKV);
-  const int n_tiles_all = (kv_end - kv_begin + BKV - 1) / BKV;
+  const int n_keep = EXT ? (min(p.keep_first, kv_begin) + BKV - 1) / BKV : 0;   // tiles of kept first keys ahead of kv_begin
+  const int n_tiles_all = n_keep + (kv_end - kv_begin + BKV - 1) / BKV;
   // this CTA's share of the key tiles (all of them without a split); short key ranges are left whole
   int n_eff = 1;
   if (p.splits > 1 && tile_ord < p.ws_tiles) n_eff = max(1, min(p.splits, n_tiles_all / p.min_tiles));
@@ -173,7 +176,8 @@ prefill_attn_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_con
   const int chunk = (n_tiles_all + n_splits - 1) / n_splits;
   const int j_first = int(blockIdx.z) * chunk;
   const int n_tiles = max(0, min(n_tiles_all, j_first + chunk) - j_first);
-  kv_begin += j_first * BKV;
+  // first key of this CTA's j-th tile
+  auto tile_kv = [&](int j) { return j_first + j < n_keep ? (j_first + j) * BKV : kv_begin + (j_first + j - n_keep) * BKV; };
   const int* bt = p.block_tables + size_t(seq) * p.max_blocks;
   if (n_tiles > 0) {
 
@@ -231,7 +235,7 @@ prefill_attn_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_con
       // the block-table entry is fetched before the stage is waited for
       long slot = 0;
       if (lane < per_tile) {
-        const int tok = kv_begin + j * BKV + bx * p.box_tokens;
+        const int tok = tile_kv(j) + bx * p.box_tokens;
         int bi = tok / p.block_size;
         bi = bi < p.max_blocks ? bi : p.max_blocks - 1;
         slot = long(bt[bi]) * p.block_size + tok % p.block_size;
@@ -317,6 +321,8 @@ prefill_attn_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_con
     const int hi = min(pos, kv_len - 1);                     // last visible kv index of this row
     int lo = p.window > 0 ? max(0, pos - p.window + 1) : 0;
     if (EXT && p.chunk > 0) lo = max(lo, pos / p.chunk * p.chunk);
+    const int keep = EXT ? p.keep_first : 0;
+    const int lo_win = p.window > 0 ? pos0 + BQ - p.window : 0;                          // first key in every row's window
     const int lo_last = EXT && p.chunk > 0 ? (pos0 + BQ - 1) / p.chunk * p.chunk : 0;   // first key that every row's chunk may hold
     const float slope2 = EXT && p.slopes ? p.slopes[head0 + h] * 1.4426950408889634f : 0.f;
     // with the extensions v[] holds finished scores in the log2 domain, otherwise raw products that `sc` scales
@@ -338,8 +344,8 @@ prefill_attn_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_con
       tc_fence_before();
       __syncwarp();
       if (lane == 0) mbar_arrive(&bars->s_free[h][b]);
-      const int kv0 = kv_begin + j * BKV;
-      const bool need_mask = (kv0 + BKV - 1 > pos0) || (kv0 + BKV > kv_len) || (p.window > 0) || (EXT && kv0 < lo_last);
+      const int kv0 = tile_kv(j);
+      const bool need_mask = (kv0 + BKV - 1 > pos0) || (kv0 + BKV > kv_len) || (kv0 < lo_win && kv0 + BKV > keep) || (EXT && kv0 < lo_last);
       float v[64];
 #pragma unroll
       for (int c = 0; c < 32; ++c) {
@@ -355,7 +361,7 @@ prefill_attn_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_con
 #pragma unroll
         for (int c = 0; c < 64; ++c) {
           const int t = kv0 + c;
-          if (t > hi || t < lo) v[c] = -INFINITY;
+          if (t > hi || (t < lo && t >= keep)) v[c] = -INFINITY;
         }
       }
       // eight independent chains keep the dependent-issue latency off the critical path
@@ -634,16 +640,17 @@ XL_API int xl_prefill_attention_tc(const void* q, const void* k_cache, const voi
 }
 
 // The same with the score extensions and separate query-key / value head dimensions (multiples of 8, at most 128):
-//   score(i, j) = scale * q_i . k_j - slopes[h] * (i - j), visible when j <= i, within `window` (> 0) and in the same
-//   chunk of `chunk` positions (> 0); out = sum_j exp(score) v_j / (sum_j exp(score) + exp(sinks[h])).
+//   score(i, j) = scale * q_i . k_j - slopes[h] * (i - j), visible when j <= i, within `window` (> 0) or among the first
+//   `keep_first` keys, and in the same chunk of `chunk` positions (> 0); out = sum_j exp(score) v_j / (sum_j exp(score) + exp(sinks[h])).
 // `slopes` / `sinks` [n_q] fp32, null when absent.  Returns -3 when the shape is not covered.
 XL_API int xl_prefill_attention_ext(const void* q, const void* k_cache, const void* v_cache, void* out, const void* q_cu,
                                     const void* kv_lens, const void* block_tables, int seq_begin, int seq_end, int max_blocks,
                                     int block_size, int num_blocks_total, int n_q, int n_kv, int dk, int dv, int q_stride,
-                                    int total_q_rows, float scale, int window, int chunk, const void* slopes, const void* sinks,
-                                    int q_tiles_cap, const void* dyn_begin, const void* dyn_end, void* stream) {
+                                    int total_q_rows, float scale, int window, int chunk, int keep_first, const void* slopes,
+                                    const void* sinks, int q_tiles_cap, const void* dyn_begin, const void* dyn_end, void* stream) {
   using namespace xl_pf;
   if (dk < 8 || dk > 128 || dk % 8 || dv < 8 || dv > 128 || dv % 8) return -3;
+  if (chunk > 0 && keep_first > 0) return -2;
   if (block_size % 16 != 0 || (block_size > 64 && block_size % 64 != 0) || (block_size < 64 && 64 % block_size != 0)) return -3;
   if (n_q % n_kv) return -3;
   if ((q_stride % 8) || (reinterpret_cast<uintptr_t>(q) & 15) || (reinterpret_cast<uintptr_t>(out) & 15)) return -3;
@@ -666,6 +673,7 @@ XL_API int xl_prefill_attention_ext(const void* q, const void* k_cache, const vo
   p.slopes = static_cast<const float*>(slopes);
   p.sinks = static_cast<const float*>(sinks);
   p.chunk = chunk;
+  p.keep_first = keep_first;
   p.q_cu = static_cast<const int*>(q_cu);
   p.kv_lens = static_cast<const int*>(kv_lens);
   p.block_tables = static_cast<const int*>(block_tables);

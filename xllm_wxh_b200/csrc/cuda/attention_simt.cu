@@ -23,7 +23,7 @@ struct Params {
   int rows, n_seqs, max_blocks, block_size, n_q, n_kv, dk, dv;
   long q_stride, cache_slots;
   float scale;
-  int window, chunk;
+  int window, chunk, keep_first;
   const float* slopes;
   const float* sinks;
 };
@@ -52,8 +52,11 @@ __global__ void __launch_bounds__(128) attention_simt_kernel(const Params<T> p) 
   float acc[kMaxCols];
 #pragma unroll
   for (int c = 0; c < kMaxCols; ++c) acc[c] = 0.f;
-  for (int base = lo; base <= pos; base += 32) {
-    const int key = base + lane;
+  // visible keys in order: the kept first ones ahead of lo, then lo .. pos
+  const int kept = min(p.keep_first, lo), n_keys = kept + pos - lo + 1;
+  for (int base = 0; base < n_keys; base += 32) {
+    const int idx = base + lane;
+    const int key = idx < n_keys ? (idx < kept ? idx : lo + idx - kept) : pos + 1;
     float s = -INFINITY;
     long slot = 0;
     if (key <= pos) {
@@ -72,7 +75,7 @@ __global__ void __launch_bounds__(128) attention_simt_kernel(const Params<T> p) 
     m = m_new;
 #pragma unroll
     for (int c = 0; c < kMaxCols; ++c) acc[c] *= alpha;
-    const int n = min(32, pos - base + 1);
+    const int n = min(32, n_keys - base);
     for (int j = 0; j < n; ++j) {
       const float wj = __shfl_sync(0xffffffffu, w, j);
       const long sj = __shfl_sync(0xffffffffu, slot, j);
@@ -91,7 +94,7 @@ __global__ void __launch_bounds__(128) attention_simt_kernel(const Params<T> p) 
 template <typename T>
 static int launch(const void* q, const void* k_cache, const void* v_cache, void* out, const void* token_seq, const void* positions,
                   const void* block_tables, int rows, int n_seqs, int max_blocks, int block_size, long cache_slots, int n_q, int n_kv,
-                  int dk, int dv, long q_stride, float scale, int window, int chunk, const void* slopes, const void* sinks,
+                  int dk, int dv, long q_stride, float scale, int window, int chunk, int keep_first, const void* slopes, const void* sinks,
                   cudaStream_t st) {
   Params<T> p;
   p.q = static_cast<const T*>(q);
@@ -104,7 +107,7 @@ static int launch(const void* q, const void* k_cache, const void* v_cache, void*
   p.rows = rows; p.n_seqs = n_seqs; p.max_blocks = max_blocks; p.block_size = block_size;
   p.n_q = n_q; p.n_kv = n_kv; p.dk = dk; p.dv = dv;
   p.q_stride = q_stride; p.cache_slots = cache_slots;
-  p.scale = scale; p.window = window; p.chunk = chunk;
+  p.scale = scale; p.window = window; p.chunk = chunk; p.keep_first = keep_first;
   p.slopes = static_cast<const float*>(slopes);
   p.sinks = static_cast<const float*>(sinks);
   const long blocks = (long(rows) * n_q + 3) / 4;
@@ -114,17 +117,17 @@ static int launch(const void* q, const void* k_cache, const void* v_cache, void*
 
 }  // namespace xl_as
 
-// All rows of a step, prefill and decode.  `window` / `chunk` <= 0: none; `slopes` / `sinks` [n_q] fp32 or null.
+// All rows of a step, prefill and decode.  `window` / `chunk` <= 0: none; `keep_first`: so many first keys stay visible; `slopes` / `sinks` [n_q] fp32 or null.
 XL_API int xl_attention_simt(const void* q, const void* k_cache, const void* v_cache, void* out, const void* token_seq,
                              const void* positions, const void* block_tables, int rows, int n_seqs, int max_blocks, int block_size,
                              long cache_slots, int n_q, int n_kv, int dk, int dv, long q_stride, float scale, int window, int chunk,
-                             const void* slopes, const void* sinks, int f32, void* stream) {
+                             int keep_first, const void* slopes, const void* sinks, int f32, void* stream) {
   if (rows <= 0) return 0;
   if (n_kv <= 0 || n_q % n_kv || dk <= 0 || dk > 2048 || dv <= 0 || dv > 32 * xl_as::kMaxCols) return -2;
   cudaStream_t st = static_cast<cudaStream_t>(stream);
   if (f32)
     return xl_as::launch<float>(q, k_cache, v_cache, out, token_seq, positions, block_tables, rows, n_seqs, max_blocks, block_size,
-                                cache_slots, n_q, n_kv, dk, dv, q_stride, scale, window, chunk, slopes, sinks, st);
+                                cache_slots, n_q, n_kv, dk, dv, q_stride, scale, window, chunk, keep_first, slopes, sinks, st);
   return xl_as::launch<__nv_bfloat16>(q, k_cache, v_cache, out, token_seq, positions, block_tables, rows, n_seqs, max_blocks, block_size,
-                                      cache_slots, n_q, n_kv, dk, dv, q_stride, scale, window, chunk, slopes, sinks, st);
+                                      cache_slots, n_q, n_kv, dk, dv, q_stride, scale, window, chunk, keep_first, slopes, sinks, st);
 }

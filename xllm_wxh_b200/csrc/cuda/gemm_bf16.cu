@@ -33,8 +33,9 @@ struct GemmSmemBarriers {
   int abort_flag;
 };
 
-// EPI_GEGLU: as EPI_SWIGLU with the tanh form of gelu; EPI_F32: the accumulators are stored as fp32 (C is float).
-enum { EPI_NONE = 0, EPI_BIAS = 1, EPI_SWIGLU = 2, EPI_RS_PUSH = 3, EPI_GEGLU = 4, EPI_F32 = 5 };
+// EPI_GEGLU: as EPI_SWIGLU with the tanh form of gelu; EPI_F32: the accumulators are stored as fp32 (C is float);
+// EPI_RELU2 / EPI_TANH: squared relu / tanh of the accumulators.
+enum { EPI_NONE = 0, EPI_BIAS = 1, EPI_SWIGLU = 2, EPI_RS_PUSH = 3, EPI_GEGLU = 4, EPI_F32 = 5, EPI_RELU2 = 6, EPI_TANH = 7 };
 __host__ __device__ constexpr bool epi_gated(int epi) { return epi == EPI_SWIGLU || epi == EPI_GEGLU; }
 
 // EPI_RS_PUSH (tensor-parallel row-parallel linear): this rank's partial tile is not stored locally; each row is
@@ -248,7 +249,11 @@ gemm_bf16_kernel(const __grid_constant__ CUtensorMap tmA, const __grid_constant_
           if (row < row_lim && n < N) {
             float v[32];
 #pragma unroll
-            for (int j = 0; j < 32; ++j) v[j] = __uint_as_float(r[j]);
+            for (int j = 0; j < 32; ++j) {
+              v[j] = __uint_as_float(r[j]);
+              if (EPI == EPI_RELU2) v[j] = act_relu2(v[j]);
+              if (EPI == EPI_TANH) v[j] = act_tanh(v[j]);
+            }
             if (EPI == EPI_BIAS) {
 #pragma unroll
               for (int j = 0; j < 32; ++j)
@@ -364,7 +369,7 @@ static int launch(const void* A, const void* W, void* C, const void* bias, int M
   const CUtensorMap* tb = xl_host::tmap_2d(W, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 2, uint64_t(N) * num_experts, K, ldw, BN, kBK,
                                            CU_TENSOR_MAP_SWIZZLE_128B);
   if (!ta || !tb) return -4;
-  static bool attr_set[6] = {false, false, false, false, false, false};
+  static bool attr_set[8] = {false, false, false, false, false, false, false, false};
   RsPush rs;
   memset(&rs, 0, sizeof(rs));
   if (rs_in) rs = *rs_in;
@@ -409,6 +414,15 @@ XL_API int xl_gemm_bf16_gated(const void* A, const void* W, void* C, int M, int 
 // fp32 C[M,N] = A[M,K] W[N,K]^T: the fp32 accumulators leave unrounded (router logits).
 XL_API int xl_gemm_bf16_f32(const void* A, const void* W, void* C, int M, int N, int K, int lda, int ldw, int ldc, void* stream) {
   return xl::launch<xl::EPI_F32>(A, W, C, nullptr, M, N, K, lda, ldw, ldc, static_cast<cudaStream_t>(stream));
+}
+
+// C = act(A W^T) with an activation of the fp32 sums (ACT_RELU2 / ACT_TANH).
+XL_API int xl_gemm_bf16_act(const void* A, const void* W, void* C, int M, int N, int K, int lda, int ldw, int ldc, int act,
+                            void* stream) {
+  cudaStream_t st = static_cast<cudaStream_t>(stream);
+  if (act == xl::ACT_RELU2) return xl::launch<xl::EPI_RELU2>(A, W, C, nullptr, M, N, K, lda, ldw, ldc, st);
+  if (act == xl::ACT_TANH) return xl::launch<xl::EPI_TANH>(A, W, C, nullptr, M, N, K, lda, ldw, ldc, st);
+  return -2;
 }
 
 // Grouped GEMM over expert-sorted rows: C[r, :] = A[r, :] * W[expert(r)]^T for the rows listed in the tile table

@@ -37,7 +37,7 @@ constexpr int kMaxStages = 8;
 constexpr int kThreads = 192;
 constexpr int kOutStageBytes = 4 * 2 * 2048;   // 4 epilogue warps x 2 buffers x (32 rows x 64 bytes)
 
-enum { EPI_NONE = 0, EPI_BIAS = 1, EPI_SWIGLU = 2, EPI_RS_PUSH = 3, EPI_GEGLU = 4 };
+enum { EPI_NONE = 0, EPI_BIAS = 1, EPI_SWIGLU = 2, EPI_RS_PUSH = 3, EPI_GEGLU = 4, EPI_RELU2 = 6, EPI_TANH = 7 };   // as in gemm_bf16.cu
 __host__ __device__ constexpr bool epi_gated(int epi) { return epi == EPI_SWIGLU || epi == EPI_GEGLU; }
 
 struct Barriers {
@@ -141,6 +141,15 @@ __device__ __forceinline__ void tc_commit_pair(uint64_t* bar) {
                : "memory");
 }
 
+template <int EPI>
+__device__ __forceinline__ void act_chunk(float (&v)[32]) {
+#pragma unroll
+  for (int j = 0; j < 32; ++j) {
+    if (EPI == EPI_RELU2) v[j] = act_relu2(v[j]);
+    if (EPI == EPI_TANH) v[j] = act_tanh(v[j]);
+  }
+}
+
 // One 32-column chunk of an output row (fp32 in `v`) -> bias / SwiGLU / row push -> bf16 stores.
 template <int EPI>
 __device__ __forceinline__ void emit_chunk(float (&v)[32], int row, int n, int width, int M, int N, int ldc,
@@ -165,6 +174,7 @@ __device__ __forceinline__ void emit_chunk(float (&v)[32], int row, int n, int w
     for (int j = 0; j < 32; ++j)
       if (n + j < N) v[j] += __bfloat162float(__ldg(bias + n + j));
   }
+  act_chunk<EPI>(v);
   __nv_bfloat16* dst = C + size_t(row) * ldc + n;
   if (EPI == EPI_RS_PUSH && !rs.local) {
     const int owner = row / rs.shard;
@@ -219,6 +229,7 @@ __device__ __forceinline__ void store_chunk_tma(float (&v)[32], uint8_t* stage, 
       for (int j = 0; j < 32; ++j)
         if (n + j < N) v[j] += __bfloat162float(__ldg(bias + n + j));
     }
+    act_chunk<EPI>(v);
     const int sw = (lane >> 1) & 3;                     // 64-byte swizzle: piece ^= address bits 8:7
 #pragma unroll
     for (int j = 0; j < 4; ++j)
@@ -727,7 +738,7 @@ static int launch_pair(const void* A, const void* W, void* C, const void* bias, 
 }  // namespace xl2
 
 // Entry points used by gemm_bf16.cu's dispatch.  `epi`: 0 none, 1 bias, 2 SwiGLU (interleaved W), 3 row push (TP),
-// 4 gelu-gated (interleaved W).
+// 4 gelu-gated (interleaved W), 6 squared relu, 7 tanh.
 // `score` (may be null) receives the wave-fill score of the chosen tile width, comparable with the single-CTA one.
 extern "C" int xl_gemm_bf16_pair_launch(int epi, const void* A, const void* W, void* C, const void* bias, int M, int N, int K,
                                         int lda, int ldw, int ldc, void* stream, const void* rs) {
@@ -739,6 +750,8 @@ extern "C" int xl_gemm_bf16_pair_launch(int epi, const void* A, const void* W, v
     case 2: return xl2::launch_pair<xl2::EPI_SWIGLU>(A, W, C, bias, M, N, K, lda, ldw, ldc, st, nullptr);
     case 3: return xl2::launch_pair<xl2::EPI_RS_PUSH>(A, W, C, bias, M, N, K, lda, ldw, ldc, st, r);
     case 4: return xl2::launch_pair<xl2::EPI_GEGLU>(A, W, C, bias, M, N, K, lda, ldw, ldc, st, nullptr);
+    case 6: return xl2::launch_pair<xl2::EPI_RELU2>(A, W, C, bias, M, N, K, lda, ldw, ldc, st, nullptr);
+    case 7: return xl2::launch_pair<xl2::EPI_TANH>(A, W, C, bias, M, N, K, lda, ldw, ldc, st, nullptr);
   }
   return -2;
 }

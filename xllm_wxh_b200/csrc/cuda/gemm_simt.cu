@@ -19,10 +19,14 @@ struct Tiles {
   const int* row_src;          // null: A row = row; else A row = row_src[row] / row_div
   int row_div;
 };
+struct Epi {
+  const void* bias;            // [N] in the operands' type, or null
+  int act;                     // ACT_NONE / ACT_RELU2 / ACT_TANH, applied after the bias
+};
 
 template <typename T, typename TO>
 __global__ void __launch_bounds__(256) gemm_simt_kernel(const T* __restrict__ A, const T* __restrict__ W, TO* __restrict__ C, int M,
-                                                        int N, int K, long lda, long ldw, long ldc, const Tiles g) {
+                                                        int N, int K, long lda, long ldw, long ldc, const Tiles g, const Epi epi) {
   __shared__ float sA[BK][BM + 4], sW[BK][BN + 4];
   int m0 = blockIdx.x * BM, m_end = M;
   const int n0 = blockIdx.y * BN;
@@ -68,36 +72,39 @@ __global__ void __launch_bounds__(256) gemm_simt_kernel(const T* __restrict__ A,
 #pragma unroll
     for (int j = 0; j < 4; ++j) {
       const int n = n0 + tx * 4 + j;
-      if (n < N) from_f32(C + size_t(m) * ldc + n, acc[i][j]);
+      if (n >= N) continue;
+      const float b = epi.bias ? to_f32(static_cast<const T*>(epi.bias)[n]) : 0.f;
+      from_f32(C + size_t(m) * ldc + n, plain_act(acc[i][j] + b, epi.act));
     }
   }
 }
 
 template <typename T, typename TO>
-static int launch(const void* A, const void* W, void* C, int M, int N, int K, long lda, long ldw, long ldc, const Tiles& g, int m_blocks,
-                  cudaStream_t st) {
+static int launch(const void* A, const void* W, void* C, int M, int N, int K, long lda, long ldw, long ldc, const Tiles& g,
+                  const Epi& epi, int m_blocks, cudaStream_t st) {
   const dim3 grid(m_blocks, (N + BN - 1) / BN);
   if (grid.y > 65535) return -2;
   gemm_simt_kernel<T, TO><<<grid, 256, 0, st>>>(static_cast<const T*>(A), static_cast<const T*>(W), static_cast<TO*>(C), M, N, K, lda, ldw,
-                                                ldc, g);
+                                                ldc, g, epi);
   return cudaGetLastError() == cudaSuccess ? 0 : -1;
 }
 
 static int dispatch(const void* A, const void* W, void* C, int M, int N, int K, long lda, long ldw, long ldc, int in_f32, int out_f32,
-                    const Tiles& g, int m_blocks, cudaStream_t st) {
-  if (in_f32) return out_f32 ? launch<float, float>(A, W, C, M, N, K, lda, ldw, ldc, g, m_blocks, st) : -2;
-  if (out_f32) return launch<__nv_bfloat16, float>(A, W, C, M, N, K, lda, ldw, ldc, g, m_blocks, st);
-  return launch<__nv_bfloat16, __nv_bfloat16>(A, W, C, M, N, K, lda, ldw, ldc, g, m_blocks, st);
+                    const Tiles& g, const Epi& epi, int m_blocks, cudaStream_t st) {
+  if (in_f32) return out_f32 ? launch<float, float>(A, W, C, M, N, K, lda, ldw, ldc, g, epi, m_blocks, st) : -2;
+  if (out_f32) return launch<__nv_bfloat16, float>(A, W, C, M, N, K, lda, ldw, ldc, g, epi, m_blocks, st);
+  return launch<__nv_bfloat16, __nv_bfloat16>(A, W, C, M, N, K, lda, ldw, ldc, g, epi, m_blocks, st);
 }
 
 }  // namespace xl_simt
 
-// in_f32: A and W are fp32 (else bf16); out_f32: C is fp32 (else bf16).
-XL_API int xl_gemm_simt(const void* A, const void* W, void* C, int M, int N, int K, long lda, long ldw, long ldc, int in_f32, int out_f32,
-                        void* stream) {
+// in_f32: A and W are fp32 (else bf16); out_f32: C is fp32 (else bf16).  C = act(A W^T + bias), bias [N] or null.
+XL_API int xl_gemm_simt(const void* A, const void* W, void* C, const void* bias, int act, int M, int N, int K, long lda, long ldw,
+                        long ldc, int in_f32, int out_f32, void* stream) {
   if (M <= 0 || N <= 0) return 0;
   xl_simt::Tiles g = {};
-  return xl_simt::dispatch(A, W, C, M, N, K, lda, ldw, ldc, in_f32, out_f32, g, (M + xl_simt::BM - 1) / xl_simt::BM,
+  const xl_simt::Epi epi{bias, act};
+  return xl_simt::dispatch(A, W, C, M, N, K, lda, ldw, ldc, in_f32, out_f32, g, epi, (M + xl_simt::BM - 1) / xl_simt::BM,
                            static_cast<cudaStream_t>(stream));
 }
 
@@ -114,5 +121,5 @@ XL_API int xl_grouped_gemm_simt(const void* A, const void* W, void* C, int N, in
   g.num_m_tiles = static_cast<const int*>(num_m_tiles);
   g.row_src = static_cast<const int*>(row_src);
   g.row_div = row_div < 1 ? 1 : row_div;
-  return xl_simt::dispatch(A, W, C, 0, N, K, lda, K, ldc, f32, f32, g, 2 * max_m_tiles, static_cast<cudaStream_t>(stream));
+  return xl_simt::dispatch(A, W, C, 0, N, K, lda, K, ldc, f32, f32, g, xl_simt::Epi{nullptr, xl::ACT_NONE}, 2 * max_m_tiles, static_cast<cudaStream_t>(stream));
 }

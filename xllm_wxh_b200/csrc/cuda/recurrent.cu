@@ -1,0 +1,1075 @@
+// Layers with recurrent state, over ragged batches: every sequence of a step owns rows q_cu[i] .. q_cu[i + 1], the last ones
+// of its kv_lens[i] tokens, and record slots[i] of the layer's state tensors.  A sequence whose rows start at position 0
+// starts from zero, so a record needs no clearing when its slot changes hands.
+//
+//   token_shift     blends of every row with its predecessor (inputs of time mixing); keeps the last row
+//   conv_silu       causal convolution per channel + silu (ahead of the selective scan); keeps the last inputs
+//   time_mix        matrix state per head, decay per key channel, bonus for the current token; then RMS per head, weight and
+//                   silu gate.  Single rows: one CTA streams a head's matrix through registers.  Longer portions: a portion
+//                   is cut into segments; (A) every segment's own contribution to the state and its decay, (B) the states
+//                   that the segments start from, (C) the segments' outputs from those, all in fp32
+//   selective_scan  diagonal state space recurrence; its step sizes, decays, D x and silu(z) are part of the kernel
+//
+// All arithmetic is fp32 and states are fp32; other tensors are bf16, or fp32 when the model runs in 32-bit.
+#include <type_traits>
+
+#include "vec8.cuh"
+
+namespace xl_rc {
+using namespace xl;
+
+struct Seqs {
+  const int* q_cu;
+  const int* kv_lens;
+  const int* slots;
+  int n;               // sequences (a capacity in padded steps: the rest has no rows)
+  int n_slots;         // records in the state tensors
+  int* status;
+};
+
+// Record of sequence s, or -1 (recorded in the status word) if it lies outside the state tensors.
+__device__ __forceinline__ int record_of(const Seqs& q, int s) {
+  const int slot = q.slots[s];
+  if (slot < 0 || slot >= q.n_slots) {
+    if (threadIdx.x == 0) atomicExch(q.status, XL_ERR_BOUNDS);
+    return -1;
+  }
+  return slot;
+}
+
+__device__ __forceinline__ float ex2(float x) {
+  float y;
+  asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
+  return y;
+}
+__device__ __forceinline__ float softplus(float z) { return z > 20.f ? z : log1pf(__expf(z)); }
+// exp(x), x <= 0: the factor a state is multiplied by at every token, so its error adds up over the tokens that the state
+// remembers.  Models in 32-bit take the one that is exact to the last place near 1.
+template <typename T>
+__device__ __forceinline__ float decay_exp(float x) {
+  if constexpr (sizeof(T) == 4) return 1.f + expm1f(x);
+  else return __expf(x);
+}
+template <typename T>
+__device__ __forceinline__ float decay_of(float z) { return decay_exp<T>(-__expf(z)); }
+
+template <int V, typename T>
+__device__ __forceinline__ void load_n(const T* p, float (&f)[V]) {
+  if constexpr (V == 8) load8(p, f);
+  else f[0] = to_f32(*p);
+}
+template <int V, typename T>
+__device__ __forceinline__ void store_n(T* p, const float (&f)[V]) {
+  if constexpr (V == 8) store8(p, f);
+  else from_f32(p, f[0]);
+}
+
+// ============================================================================ token shift
+template <typename T, int V>
+__global__ void __launch_bounds__(256) token_shift_kernel(const T* __restrict__ h, const T* __restrict__ mu, T* __restrict__ last,
+                                                          T* __restrict__ out, const int* __restrict__ token_seq, const Seqs q, int rows,
+                                                          int W, int n_mix) {
+  const int t = blockIdx.x, seq = token_seq[t];
+  const size_t plane = size_t(rows) * W;
+  if (seq < 0 || seq >= q.n) {                     // padding row
+    const float zero[V] = {};
+    for (int c = threadIdx.x * V; c < W; c += blockDim.x * V)
+      for (int j = 0; j < n_mix; ++j) store_n<V>(out + j * plane + size_t(t) * W + c, zero);
+    return;
+  }
+  const int start = q.q_cu[seq], end = q.q_cu[seq + 1];
+  const int slot = record_of(q, seq);
+  if (slot < 0) return;
+  const bool first = t == start, cont = q.kv_lens[seq] > end - start;
+  for (int c = threadIdx.x * V; c < W; c += blockDim.x * V) {
+    float cur[V], prev[V] = {}, m[V], o[V];
+    load_n<V>(h + size_t(t) * W + c, cur);
+    if (!first) load_n<V>(h + size_t(t - 1) * W + c, prev);
+    else if (cont) load_n<V>(last + size_t(slot) * W + c, prev);
+    for (int j = 0; j < n_mix; ++j) {
+      load_n<V>(mu + size_t(j) * W + c, m);
+#pragma unroll
+      for (int e = 0; e < V; ++e) o[e] = fmaf(prev[e] - cur[e], m[e], cur[e]);
+      store_n<V>(out + j * plane + size_t(t) * W + c, o);
+    }
+    if (first) {                                   // only this thread reads this part of the record
+      load_n<V>(h + size_t(end - 1) * W + c, cur);
+      store_n<V>(last + size_t(slot) * W + c, cur);
+    }
+  }
+}
+
+// ============================================================================ causal convolution + silu
+// A thread owns V channels of a tile of consecutive rows and keeps the last TAPS - 1 inputs in registers (TAPS = 0: any
+// number of taps, inputs read again for every row).
+constexpr int kConvRows = 16;
+
+template <typename T, int V, int TAPS>
+__global__ void __launch_bounds__(128) conv_silu_kernel(const T* __restrict__ x, const T* __restrict__ w, const T* __restrict__ bias,
+                                                        T* __restrict__ state, T* __restrict__ out, const int* __restrict__ token_seq,
+                                                        const Seqs q, int rows, int C, int taps_rt, long ldx) {
+  constexpr int H = TAPS > 1 ? TAPS - 1 : 1;
+  const int taps = TAPS > 0 ? TAPS : taps_rt;
+  const int c = (blockIdx.y * blockDim.x + threadIdx.x) * V;
+  if (c >= C) return;
+  const int t0 = blockIdx.x * kConvRows, t1 = min(rows, t0 + kConvRows);
+  float b[V], wt[TAPS > 0 ? TAPS : 1][V], hist[H][V];
+  load_n<V>(bias + c, b);
+  if (TAPS > 0) {
+#pragma unroll
+    for (int i = 0; i < TAPS; ++i)
+#pragma unroll
+      for (int e = 0; e < V; ++e) wt[i][e] = to_f32(w[size_t(c + e) * TAPS + i]);
+  }
+  int cur_seq = -1, start = 0, end = 0, slot = 0;
+  bool cont = false;
+  for (int t = t0; t < t1; ++t) {
+    const int seq = token_seq[t];
+    if (seq < 0 || seq >= q.n) continue;
+    const bool fresh = seq != cur_seq;
+    if (fresh) {
+      cur_seq = seq;
+      start = q.q_cu[seq];
+      end = q.q_cu[seq + 1];
+      slot = record_of(q, seq);
+      cont = q.kv_lens[seq] > end - start;
+    }
+    if (slot < 0) continue;
+    // input `back` rows ahead of row t of this sequence
+    auto before = [&](int back, float (&f)[V]) {
+      const int j = t - start - back;
+#pragma unroll
+      for (int e = 0; e < V; ++e) f[e] = 0.f;
+      if (j >= 0) load_n<V>(x + size_t(t - back) * ldx + c, f);
+      else if (cont) load_n<V>(state + (size_t(slot) * (taps - 1) + (taps - 1 + j)) * C + c, f);
+    };
+    float y[V], cur[V];
+    load_n<V>(x + size_t(t) * ldx + c, cur);
+#pragma unroll
+    for (int e = 0; e < V; ++e) y[e] = b[e];
+    if (TAPS > 0) {
+      if (fresh) {
+#pragma unroll
+        for (int i = 0; i < TAPS - 1; ++i) before(TAPS - 1 - i, hist[i]);
+      }
+#pragma unroll
+      for (int i = 0; i < TAPS - 1; ++i)
+#pragma unroll
+        for (int e = 0; e < V; ++e) y[e] = fmaf(hist[i][e], wt[i][e], y[e]);
+#pragma unroll
+      for (int e = 0; e < V; ++e) y[e] = fmaf(cur[e], wt[TAPS > 0 ? TAPS - 1 : 0][e], y[e]);
+#pragma unroll
+      for (int i = 0; i + 1 < TAPS - 1; ++i)
+#pragma unroll
+        for (int e = 0; e < V; ++e) hist[i][e] = hist[i + 1][e];
+      if (TAPS > 1) {
+#pragma unroll
+        for (int e = 0; e < V; ++e) hist[H - 1][e] = cur[e];
+        if (end - start == 1) {                    // a single row: this thread alone reads and writes this part of the record
+#pragma unroll
+          for (int i = 0; i < TAPS - 1; ++i) store_n<V>(state + (size_t(slot) * (TAPS - 1) + i) * C + c, hist[i]);
+        }
+      }
+    } else {
+      for (int i = 0; i < taps; ++i) {
+        float f[V];
+        before(taps - 1 - i, f);
+#pragma unroll
+        for (int e = 0; e < V; ++e) y[e] = fmaf(f[e], to_f32(w[size_t(c + e) * taps + i]), y[e]);
+      }
+      if (end - start == 1) {
+        for (int i = 0; i < taps - 1; ++i) {
+          float f[V];
+          before(taps - 2 - i, f);                 // row i moves down by one, the last becomes the current input
+          store_n<V>(state + (size_t(slot) * (taps - 1) + i) * C + c, f);
+        }
+      }
+    }
+#pragma unroll
+    for (int e = 0; e < V; ++e) y[e] = act_silu(y[e]);
+    store_n<V>(out + size_t(t) * C + c, y);
+  }
+}
+
+// Records of the sequences with several rows, after the convolution has read the old ones.
+template <typename T, int V>
+__global__ void __launch_bounds__(128) conv_record_kernel(const T* __restrict__ x, T* __restrict__ state, const Seqs q, int C, int taps,
+                                                          long ldx) {
+  const int seq = blockIdx.x;
+  const int c = (blockIdx.y * blockDim.x + threadIdx.x) * V;
+  const int start = q.q_cu[seq], len = q.q_cu[seq + 1] - start;
+  if (len < 2 || c >= C) return;
+  const int slot = record_of(q, seq);
+  if (slot < 0) return;
+  const bool cont = q.kv_lens[seq] > len;
+  T* rec = state + size_t(slot) * (taps - 1) * C + c;
+  for (int i = 0; i < taps - 1; ++i) {             // ascending: row i comes from a later row of the record
+    const int j = len - (taps - 1) + i;
+    float f[V] = {};
+    if (j >= 0) load_n<V>(x + size_t(start + j) * ldx + c, f);
+    else if (cont) load_n<V>(rec + size_t(i + len) * C, f);
+    store_n<V>(rec + size_t(i) * C, f);
+  }
+}
+
+// ============================================================================ time mixing
+template <typename T>
+struct MixParams {
+  const T *r, *k, *v, *gate;       // [rows, H * d], row pitch ld
+  const float* z;                  // [rows, H * d] dense
+  const float *w0, *u;             // [H * d]
+  const T* norm_w;                 // [H * d]
+  float* state;                    // [records, H, d, d] (key, value)
+  T* out;                          // row pitch ldo
+  long ld, ldg, ldo;
+  int H, d;
+  float scale, eps;
+  Seqs q;
+  // segments of longer portions
+  int L;                           // rows per segment
+  float* ws_s;                     // [segments, H, d, d]: what a segment adds to the state, then the state it starts from
+  float* ws_p;                     // [segments, H, d]: product of its decays
+};
+
+// Portions of two and more rows are cut into segments of L rows, numbered through the batch.  Every warp finds segment
+// `target`: its sequence, its place there and how many the sequence has.
+__device__ __forceinline__ bool find_segment(const Seqs& q, int L, int target, int& seq, int& seg, int& n_seg) {
+  const int lane = threadIdx.x & 31;
+  int base = 0;
+  for (int b = 0; b < q.n; b += 32) {
+    const int s = b + lane;
+    const int len = s < q.n ? q.q_cu[s + 1] - q.q_cu[s] : 0;
+    const int cnt = len > 1 ? (len + L - 1) / L : 0;
+    int inc = cnt;
+#pragma unroll
+    for (int o = 1; o < 32; o <<= 1) {
+      const int v = __shfl_up_sync(0xffffffffu, inc, o);
+      if (lane >= o) inc += v;
+    }
+    const int total = __shfl_sync(0xffffffffu, inc, 31);
+    if (target < base + total) {
+      const int f = __ffs(__ballot_sync(0xffffffffu, base + inc > target)) - 1;
+      n_seg = __shfl_sync(0xffffffffu, cnt, f);
+      seg = target - (base + __shfl_sync(0xffffffffu, inc, f) - n_seg);
+      seq = b + f;
+      return true;
+    }
+    base += total;
+  }
+  return false;
+}
+
+// two fp32 lanes in one 64-bit register
+__device__ __forceinline__ uint64_t pack2(float a, float b) {
+  uint64_t r;
+  asm("mov.b64 %0, {%1, %2};" : "=l"(r) : "f"(a), "f"(b));
+  return r;
+}
+__device__ __forceinline__ float2 unpack2(uint64_t v) {
+  float2 r;
+  asm("mov.b64 {%0, %1}, %2;" : "=f"(r.x), "=f"(r.y) : "l"(v));
+  return r;
+}
+__device__ __forceinline__ uint64_t fma2(uint64_t a, uint64_t b, uint64_t c) {
+  uint64_t d;
+  asm("fma.rn.f32x2 %0, %1, %2, %3;" : "=l"(d) : "l"(a), "l"(b), "l"(c));
+  return d;
+}
+__device__ __forceinline__ uint64_t mul2(uint64_t a, uint64_t b) {
+  uint64_t d;
+  asm("mul.rn.f32x2 %0, %1, %2;" : "=l"(d) : "l"(a), "l"(b));
+  return d;
+}
+
+// One (segment, head) per CTA.  D: head dimension padded to 32, 64 or 128.  Thread (kg, vg) owns keys kg * KT ..., values
+// vg * 4 ... of the head's matrix, as pairs of neighbouring keys.
+template <int D> struct MixCfg {
+  static constexpr int KT = D == 32 ? 8 : 16;
+  static constexpr int KG = D / KT, VG = D / 4, kThreads = KG * VG;
+  static constexpr int SEG = KT + 4, ROW = KG * SEG;      // key groups 4 floats apart, so that their reads meet no bank twice
+};
+constexpr int kMixRows = 16;      // rows staged in shared memory at a time
+
+// v8: 8-element loads are aligned; s4: rows of the state are multiples of 16 bytes
+template <typename T, int D, bool OUT>
+__global__ void __launch_bounds__(MixCfg<D>::kThreads) time_mix_segment_kernel(const MixParams<T> p, int v8, int s4) {
+  using C = MixCfg<D>;
+  constexpr int KT = C::KT, KG = C::KG, SEG = C::SEG, ROW = C::ROW, NT = C::kThreads;
+  __shared__ __align__(16) float sK[kMixRows][ROW], sW[kMixRows][ROW], sV[kMixRows][D];
+  __shared__ __align__(16) float sR[OUT ? kMixRows : 1][ROW], sO[OUT ? kMixRows : 1][D];
+  __shared__ float sBonus[kMixRows];
+  int seq, seg, n_seg;
+  if (!find_segment(p.q, p.L, blockIdx.x, seq, seg, n_seg)) return;
+  if (!OUT && seg == n_seg - 1) return;                   // nothing starts behind the last segment
+  if (n_seg > 1 && !p.ws_s) {                             // a portion longer than the caller said
+    if (threadIdx.x == 0) atomicExch(p.q.status, XL_ERR_BOUNDS);
+    return;
+  }
+  const int slot = record_of(p.q, seq);
+  if (slot < 0) return;
+  const int h = blockIdx.y, d = p.d, tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
+  const int kg = tid % KG, vg = tid / KG;
+  const int start = p.q.q_cu[seq], len = p.q.q_cu[seq + 1] - start;
+  const int t0 = start + seg * p.L, n = min(p.L, len - seg * p.L);
+  const bool cont = p.q.kv_lens[seq] > len;
+  const size_t mat = size_t(d) * d;
+  float* rec = p.state + (size_t(slot) * p.H + h) * mat;
+  float* seg_s = p.ws_s ? p.ws_s + (size_t(blockIdx.x) * p.H + h) * mat : nullptr;
+
+  uint64_t S[KT / 2][4];
+#pragma unroll
+  for (int i = 0; i < KT / 2; ++i)
+#pragma unroll
+    for (int j = 0; j < 4; ++j) S[i][j] = 0;
+  if (OUT && (n_seg > 1 || cont)) {
+    const float* src = n_seg > 1 ? seg_s : rec;
+#pragma unroll
+    for (int i = 0; i < KT / 2; ++i) {
+      float a[2][4] = {};
+#pragma unroll
+      for (int e = 0; e < 2; ++e) {
+        const int key = kg * KT + 2 * i + e;
+        if (key < d) {
+          if (s4) {
+            if (vg * 4 < d) *reinterpret_cast<float4*>(a[e]) = *reinterpret_cast<const float4*>(src + size_t(key) * d + vg * 4);
+          } else {
+#pragma unroll
+            for (int j = 0; j < 4; ++j)
+              if (vg * 4 + j < d) a[e][j] = src[size_t(key) * d + vg * 4 + j];
+          }
+        }
+      }
+#pragma unroll
+      for (int j = 0; j < 4; ++j) S[i][j] = pack2(a[0][j], a[1][j]);
+    }
+  }
+  float prod = 1.f;                                       // !OUT: decay of key `tid` over the segment
+  float nw[D / 32];
+  if (OUT) {
+#pragma unroll
+    for (int i = 0; i < D / 32; ++i) nw[i] = lane + 32 * i < d ? to_f32(p.norm_w[h * d + lane + 32 * i]) * p.scale : 0.f;
+  }
+  for (int b = 0; b < n; b += kMixRows) {
+    const int m = min(kMixRows, n - b);
+    // stage m rows of this head
+    if (v8) {
+      for (int i = tid; i < kMixRows * (D / 8); i += NT) {
+        const int row = i / (D / 8), c = i % (D / 8) * 8;
+        float k[8] = {}, v[8] = {}, w[8] = {}, r[8] = {};
+        if (row < m && c < d) {
+          const size_t t = size_t(t0 + b + row), at = t * p.ld + size_t(h) * d + c;
+          load8(p.k + at, k);
+          load8(p.v + at, v);
+          if (OUT) load8(p.r + at, r);
+          float w0[8];
+          load8(p.z + t * (size_t(p.H) * d) + size_t(h) * d + c, w);
+          load8(p.w0 + h * d + c, w0);
+#pragma unroll
+          for (int e = 0; e < 8; ++e) w[e] = decay_of<T>(w[e] + w0[e]);
+        }
+        const int at = c / KT * SEG + c % KT;
+        store8(&sK[row][at], k);
+        store8(&sW[row][at], w);
+        store8(&sV[row][c], v);
+        if (OUT) store8(&sR[row][at], r);
+      }
+    } else {
+      for (int i = tid; i < kMixRows * D; i += NT) {
+        const int row = i / D, c = i % D;
+        const bool in = row < m && c < d;
+        const size_t t = size_t(t0 + b + row), at = t * p.ld + size_t(h) * d + c;
+        const int to = c / KT * SEG + c % KT;
+        sK[row][to] = in ? to_f32(p.k[at]) : 0.f;
+        sV[row][c] = in ? to_f32(p.v[at]) : 0.f;
+        sW[row][to] = in ? decay_of<T>(p.z[t * (size_t(p.H) * d) + size_t(h) * d + c] + p.w0[h * d + c]) : 0.f;
+        if (OUT) sR[row][to] = in ? to_f32(p.r[at]) : 0.f;
+      }
+    }
+    __syncthreads();
+    if (OUT) {
+      for (int row = warp; row < m; row += NT / 32) {
+        float s = 0.f;
+#pragma unroll
+        for (int i = 0; i < D / 32; ++i) {
+          const int c = lane + 32 * i, at = c / KT * SEG + c % KT;
+          if (c < d) s += sR[row][at] * p.u[h * d + c] * sK[row][at];
+        }
+        s = warp_sum(s);
+        if (lane == 0) sBonus[row] = s;
+      }
+      __syncthreads();
+    } else if (tid < D) {
+      for (int row = 0; row < m; ++row) prod *= sW[row][tid / KT * SEG + tid % KT];
+    }
+    for (int row = 0; row < m; ++row) {
+      const float4 v4 = *reinterpret_cast<const float4*>(&sV[row][vg * 4]);
+      const uint64_t v[4] = {pack2(v4.x, v4.x), pack2(v4.y, v4.y), pack2(v4.z, v4.z), pack2(v4.w, v4.w)};
+      uint64_t o[4] = {0, 0, 0, 0};
+#pragma unroll
+      for (int i = 0; i < KT / 4; ++i) {
+        const ulonglong2 k2 = *reinterpret_cast<const ulonglong2*>(&sK[row][kg * SEG + 4 * i]);
+        const ulonglong2 w2 = *reinterpret_cast<const ulonglong2*>(&sW[row][kg * SEG + 4 * i]);
+        if (OUT) {
+          const ulonglong2 r2 = *reinterpret_cast<const ulonglong2*>(&sR[row][kg * SEG + 4 * i]);
+#pragma unroll
+          for (int j = 0; j < 4; ++j) o[j] = fma2(r2.y, S[2 * i + 1][j], fma2(r2.x, S[2 * i][j], o[j]));
+        }
+#pragma unroll
+        for (int j = 0; j < 4; ++j) {
+          S[2 * i][j] = fma2(w2.x, S[2 * i][j], mul2(k2.x, v[j]));
+          S[2 * i + 1][j] = fma2(w2.y, S[2 * i + 1][j], mul2(k2.y, v[j]));
+        }
+      }
+      if (OUT) {
+        // sum over the key groups (neighbouring lanes); each of the first four ends with one of the four values
+        float y[4];
+#pragma unroll
+        for (int j = 0; j < 4; ++j) {
+          const float2 f = unpack2(o[j]);
+          y[j] = f.x + f.y;
+        }
+        const bool b0 = kg & 1, b1 = kg & 2;
+        float a0 = b0 ? y[2] : y[0], a1 = b0 ? y[3] : y[1];
+        a0 += __shfl_xor_sync(0xffffffffu, b0 ? y[0] : y[2], 1);
+        a1 += __shfl_xor_sync(0xffffffffu, b0 ? y[1] : y[3], 1);
+        float a = b1 ? a1 : a0;
+        a += __shfl_xor_sync(0xffffffffu, b1 ? a0 : a1, 2);
+        if (KG == 8) a += __shfl_xor_sync(0xffffffffu, a, 4);
+        const int j = (b0 ? 2 : 0) + (b1 ? 1 : 0);
+        if (KG == 4 || kg < 4) sO[row][vg * 4 + j] = a;
+      }
+    }
+    __syncthreads();
+    if (OUT) {
+      for (int row = warp; row < m; row += NT / 32) {
+        const size_t t = size_t(t0 + b + row);
+        float o[D / 32], ss = 0.f;
+#pragma unroll
+        for (int i = 0; i < D / 32; ++i) {
+          const int c = lane + 32 * i;
+          o[i] = fmaf(sBonus[row], sV[row][c], sO[row][c]);       // zero beyond d
+          ss += o[i] * o[i];
+        }
+        const float inv = rsqrtf(warp_sum(ss) / float(d) + p.eps);
+#pragma unroll
+        for (int i = 0; i < D / 32; ++i) {
+          const int c = lane + 32 * i;
+          if (c < d)
+            from_f32(p.out + t * p.ldo + size_t(h) * d + c,
+                     o[i] * inv * nw[i] * act_silu(to_f32(p.gate[t * p.ldg + size_t(h) * d + c])));
+        }
+      }
+      __syncthreads();
+    }
+  }
+  if (OUT && seg != n_seg - 1) return;
+  float* dst = OUT ? rec : seg_s;
+#pragma unroll
+  for (int i = 0; i < KT / 2; ++i) {
+    float a[2][4];
+#pragma unroll
+    for (int j = 0; j < 4; ++j) {
+      const float2 f = unpack2(S[i][j]);
+      a[0][j] = f.x;
+      a[1][j] = f.y;
+    }
+#pragma unroll
+    for (int e = 0; e < 2; ++e) {
+      const int key = kg * KT + 2 * i + e;
+      if (key >= d) continue;
+      if (s4) {
+        if (vg * 4 < d) *reinterpret_cast<float4*>(dst + size_t(key) * d + vg * 4) = *reinterpret_cast<const float4*>(a[e]);
+      } else {
+#pragma unroll
+        for (int j = 0; j < 4; ++j)
+          if (vg * 4 + j < d) dst[size_t(key) * d + vg * 4 + j] = a[e][j];
+      }
+    }
+  }
+  if (!OUT && tid < d) p.ws_p[(size_t(blockIdx.x) * p.H + h) * d + tid] = prod;
+}
+
+// (B): the state every segment starts from, in the place of what it adds.  One CTA per (sequence, head, part of the matrix).
+template <typename T>
+__global__ void __launch_bounds__(256) time_mix_chain_kernel(const MixParams<T> p) {
+  const int seq = blockIdx.x, h = blockIdx.y, d = p.d;
+  const int len = p.q.q_cu[seq + 1] - p.q.q_cu[seq];
+  const int n_seg = len > 1 ? (len + p.L - 1) / p.L : 0;
+  if (n_seg < 2) return;
+  const int slot = record_of(p.q, seq);
+  if (slot < 0) return;
+  int base = 0;                                           // segments of the sequences ahead of this one
+  {
+    const int lane = threadIdx.x & 31;
+    for (int s = lane; s < seq; s += 32) {
+      const int n = p.q.q_cu[s + 1] - p.q.q_cu[s];
+      base += n > 1 ? (n + p.L - 1) / p.L : 0;
+    }
+#pragma unroll
+    for (int o = 16; o > 0; o >>= 1) base += __shfl_xor_sync(0xffffffffu, base, o);
+  }
+  const bool cont = p.q.kv_lens[seq] > len;
+  const int mat = d * d;
+  const float* rec = p.state + (size_t(slot) * p.H + h) * mat;
+  const size_t step = size_t(p.H) * mat;
+  for (int e = blockIdx.z * blockDim.x + threadIdx.x; e < mat; e += gridDim.z * blockDim.x) {
+    float s = cont ? rec[e] : 0.f;
+    float* ws = p.ws_s + (size_t(base) * p.H + h) * mat + e;
+    const float* pr = p.ws_p + (size_t(base) * p.H + h) * d + e / d;
+#pragma unroll 4
+    for (int g = 0; g < n_seg - 1; ++g) {
+      const float add = *ws;
+      *ws = s;
+      s = fmaf(*pr, s, add);
+      ws += step;
+      pr += size_t(p.H) * d;
+    }
+    *ws = s;
+  }
+}
+
+// Single rows: the head's matrix (d a multiple of 4) passes through registers once.
+constexpr int kMixThreads = 128;
+template <typename T>
+__global__ void __launch_bounds__(kMixThreads) time_mix_single_kernel(const MixParams<T> p) {
+  extern __shared__ __align__(16) float sm[];
+  const int seq = blockIdx.x, h = blockIdx.y, d = p.d, tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
+  const int t = p.q.q_cu[seq], len = p.q.q_cu[seq + 1] - t;
+  if (len != 1) return;
+  const int slot = record_of(p.q, seq);
+  if (slot < 0) return;
+  const bool cont = p.q.kv_lens[seq] > 1;
+  const int quads = d / 4, groups = kMixThreads / quads;    // threads over value quads, then over keys
+  const int vq = tid % quads, kq = tid / quads;
+  float *sR = sm, *sK = sR + d, *sW = sK + d, *sV = sW + d, *sO = sV + d;      // sO [groups][d]
+  __shared__ float red[2][kMixThreads / 32];
+  float4* rec = reinterpret_cast<float4*>(p.state + (size_t(slot) * p.H + h) * size_t(d) * d);
+  constexpr int kAhead = 8;
+  float4 s[kAhead];
+  const bool mine = kq < groups;
+  if (mine && cont) {                                       // the first keys are on their way while the row is prepared
+#pragma unroll
+    for (int i = 0; i < kAhead; ++i)
+      if (kq + i * groups < d) s[i] = rec[size_t(kq + i * groups) * quads + vq];
+  }
+  float bonus = 0.f;
+  for (int c = tid; c < d; c += kMixThreads) {
+    const size_t at = size_t(t) * p.ld + size_t(h) * d + c;
+    const float r = to_f32(p.r[at]), k = to_f32(p.k[at]);
+    sR[c] = r;
+    sK[c] = k;
+    sV[c] = to_f32(p.v[at]);
+    sW[c] = decay_of<T>(p.z[size_t(t) * p.H * d + size_t(h) * d + c] + p.w0[h * d + c]);
+    bonus += r * p.u[h * d + c] * k;
+  }
+  bonus = warp_sum(bonus);
+  if (lane == 0) red[0][warp] = bonus;
+  __syncthreads();
+  bonus = 0.f;
+#pragma unroll
+  for (int i = 0; i < kMixThreads / 32; ++i) bonus += red[0][i];
+  if (mine) {
+    const float4 v = *reinterpret_cast<const float4*>(sV + vq * 4);
+    float4 o = make_float4(0.f, 0.f, 0.f, 0.f);
+    for (int k0 = kq; k0 < d; k0 += kAhead * groups) {
+#pragma unroll
+      for (int i = 0; i < kAhead; ++i) {
+        const int key = k0 + i * groups;
+        if (key < d) {
+          if (!cont) s[i] = make_float4(0.f, 0.f, 0.f, 0.f);
+          else if (k0 != kq) s[i] = rec[size_t(key) * quads + vq];
+        }
+      }
+#pragma unroll
+      for (int i = 0; i < kAhead; ++i) {
+        const int key = k0 + i * groups;
+        if (key < d) {
+          const float r = sR[key], k = sK[key], w = sW[key];
+          o.x = fmaf(r, s[i].x, o.x); o.y = fmaf(r, s[i].y, o.y); o.z = fmaf(r, s[i].z, o.z); o.w = fmaf(r, s[i].w, o.w);
+          rec[size_t(key) * quads + vq] = make_float4(fmaf(w, s[i].x, k * v.x), fmaf(w, s[i].y, k * v.y), fmaf(w, s[i].z, k * v.z),
+                                                      fmaf(w, s[i].w, k * v.w));
+        }
+      }
+    }
+    *reinterpret_cast<float4*>(sO + kq * d + vq * 4) = o;
+  }
+  __syncthreads();
+  float ss = 0.f;
+  for (int c = tid; c < d; c += kMixThreads) {
+    float o = bonus * sV[c];
+    for (int g = 0; g < groups; ++g) o += sO[g * d + c];
+    sO[c] = o;                                              // only this thread reads or writes column c from here on
+    ss += o * o;
+  }
+  ss = warp_sum(ss);
+  if (lane == 0) red[1][warp] = ss;
+  __syncthreads();
+  ss = 0.f;
+#pragma unroll
+  for (int i = 0; i < kMixThreads / 32; ++i) ss += red[1][i];
+  const float inv = rsqrtf(ss / float(d) + p.eps) * p.scale;
+  for (int c = tid; c < d; c += kMixThreads)
+    from_f32(p.out + size_t(t) * p.ldo + size_t(h) * d + c,
+             sO[c] * inv * to_f32(p.norm_w[h * d + c]) * act_silu(to_f32(p.gate[size_t(t) * p.ldg + size_t(h) * d + c])));
+}
+
+// Any head dimension, any number of rows: the state stays in memory, one thread per value column.
+template <typename T>
+__global__ void __launch_bounds__(256) time_mix_any_kernel(const MixParams<T> p, int min_len, int max_len) {
+  extern __shared__ __align__(16) float sm[];
+  const int seq = blockIdx.x, h = blockIdx.y, d = p.d, tid = threadIdx.x;
+  const int start = p.q.q_cu[seq], len = p.q.q_cu[seq + 1] - start;
+  if (len < min_len || len > max_len || len < 1) return;
+  const int slot = record_of(p.q, seq);
+  if (slot < 0) return;
+  bool fresh = p.q.kv_lens[seq] == len;
+  float *sR = sm, *sK = sR + d, *sW = sK + d, *sO = sW + d;
+  __shared__ float red[2][8];
+  float* rec = p.state + (size_t(slot) * p.H + h) * size_t(d) * d;
+  for (int t = start; t < start + len; ++t) {
+    float bonus = 0.f;
+    for (int c = tid; c < d; c += 256) {
+      const size_t at = size_t(t) * p.ld + size_t(h) * d + c;
+      const float r = to_f32(p.r[at]), k = to_f32(p.k[at]);
+      sR[c] = r;
+      sK[c] = k;
+      sW[c] = decay_of<T>(p.z[size_t(t) * p.H * d + size_t(h) * d + c] + p.w0[h * d + c]);
+      bonus += r * p.u[h * d + c] * k;
+    }
+    bonus = warp_sum(bonus);
+    if ((tid & 31) == 0) red[0][tid >> 5] = bonus;
+    __syncthreads();
+    bonus = 0.f;
+    for (int i = 0; i < 8; ++i) bonus += red[0][i];
+    float ss = 0.f;
+    for (int c = tid; c < d; c += 256) {
+      const float v = to_f32(p.v[size_t(t) * p.ld + size_t(h) * d + c]);
+      float o = bonus * v;
+      for (int k = 0; k < d; ++k) {
+        const float s = fresh ? 0.f : rec[size_t(k) * d + c];
+        o = fmaf(sR[k], s, o);
+        rec[size_t(k) * d + c] = fmaf(sW[k], s, sK[k] * v);
+      }
+      sO[c] = o;
+      ss += o * o;
+    }
+    ss = warp_sum(ss);
+    if ((tid & 31) == 0) red[1][tid >> 5] = ss;
+    __syncthreads();
+    ss = 0.f;
+    for (int i = 0; i < 8; ++i) ss += red[1][i];
+    const float inv = rsqrtf(ss / float(d) + p.eps) * p.scale;
+    for (int c = tid; c < d; c += 256)
+      from_f32(p.out + size_t(t) * p.ldo + size_t(h) * d + c,
+               sO[c] * inv * to_f32(p.norm_w[h * d + c]) * act_silu(to_f32(p.gate[size_t(t) * p.ldg + size_t(h) * d + c])));
+    fresh = false;
+  }
+}
+
+template <typename T>
+static int launch_time_mix(MixParams<T> p, int seg_cap, int has_long, int has_single, cudaStream_t st) {
+  const int d = p.d;
+  const bool v8 = d % 8 == 0 && p.ld % 8 == 0 &&
+                  !((reinterpret_cast<uintptr_t>(p.r) | reinterpret_cast<uintptr_t>(p.k) | reinterpret_cast<uintptr_t>(p.v) |
+                     reinterpret_cast<uintptr_t>(p.z) | reinterpret_cast<uintptr_t>(p.w0)) & 15);
+  const bool s4 = d % 4 == 0;
+  if (has_single) {
+    const dim3 grid(p.q.n, p.H);
+    if (s4 && d <= 4 * kMixThreads) {
+      const int groups = kMixThreads / (d / 4);
+      time_mix_single_kernel<T><<<grid, kMixThreads, size_t(4 + groups) * d * sizeof(float), st>>>(p);
+    } else {
+      time_mix_any_kernel<T><<<grid, 256, size_t(4) * d * sizeof(float), st>>>(p, 1, 1);
+    }
+  }
+  if (has_long) {
+    if (d <= 128) {
+      const dim3 grid(seg_cap, p.H);
+#define XL_MIX(D, OUT) time_mix_segment_kernel<T, D, OUT><<<grid, MixCfg<D>::kThreads, 0, st>>>(p, v8, s4)
+      if (p.ws_s) {
+        if (d <= 32) XL_MIX(32, false); else if (d <= 64) XL_MIX(64, false); else XL_MIX(128, false);
+        const int parts = (d * d + 1023) / 1024;
+        time_mix_chain_kernel<T><<<dim3(p.q.n, p.H, parts), 256, 0, st>>>(p);
+      }
+      if (d <= 32) XL_MIX(32, true); else if (d <= 64) XL_MIX(64, true); else XL_MIX(128, true);
+#undef XL_MIX
+    } else {
+      time_mix_any_kernel<T><<<dim3(p.q.n, p.H), 256, size_t(4) * d * sizeof(float), st>>>(p, 2, 1 << 30);
+    }
+  }
+  return cudaGetLastError() == cudaSuccess ? 0 : -1;
+}
+
+// ============================================================================ selective scan
+template <typename T>
+struct ScanParams {
+  const T* x;                  // [rows, C] dense
+  const float* dt;             // [rows, C] dense, ahead of bias and softplus
+  const float *dt_bias, *A, *D;   // [C], [C, N], [C]
+  const T *B, *Cm;             // [rows, N], row pitch ldb
+  const T* z;                  // [rows, C], row pitch ldz
+  float* state;                // [records, C, N]
+  T* out;                      // [rows, C] dense
+  long ldb, ldz;
+  int C, N;
+  Seqs q;
+};
+
+constexpr int kScanThreads = 128, kScanRows = 16;
+// exp(step * A) from step * (A * scan_unit): base 2 on the fast path
+template <typename T> __device__ __forceinline__ constexpr float scan_unit() { return sizeof(T) == 4 ? 1.f : 1.4426950408889634f; }
+template <typename T>
+__device__ __forceinline__ float scan_decay(float x) {
+  if constexpr (sizeof(T) == 4) return decay_exp<T>(x);
+  else return ex2(x);
+}
+
+// NPT states per thread, LPC neighbouring lanes per channel (NPT * LPC >= N); states beyond N stay zero.
+template <int NPT>
+__device__ __forceinline__ void load_states(const float* p, int n0, int N, float (&s)[NPT]) {
+  if (N % 4 == 0) {
+#pragma unroll
+    for (int i = 0; i < NPT; i += 4) {
+      float4 f = make_float4(0.f, 0.f, 0.f, 0.f);
+      if (n0 + i < N) f = *reinterpret_cast<const float4*>(p + n0 + i);
+      s[i] = f.x; s[i + 1] = f.y; s[i + 2] = f.z; s[i + 3] = f.w;
+    }
+  } else {
+#pragma unroll
+    for (int i = 0; i < NPT; ++i) s[i] = n0 + i < N ? p[n0 + i] : 0.f;
+  }
+}
+template <int NPT>
+__device__ __forceinline__ void store_states(float* p, int n0, int N, const float (&s)[NPT]) {
+  if (N % 4 == 0) {
+#pragma unroll
+    for (int i = 0; i < NPT; i += 4)
+      if (n0 + i < N) *reinterpret_cast<float4*>(p + n0 + i) = make_float4(s[i], s[i + 1], s[i + 2], s[i + 3]);
+  } else {
+#pragma unroll
+    for (int i = 0; i < NPT; ++i)
+      if (n0 + i < N) p[n0 + i] = s[i];
+  }
+}
+
+// Longer portions: a CTA walks one sequence for kScanThreads / LPC channels, kScanRows rows at a time; the next rows' inputs
+// are fetched into registers while the current ones are worked on.
+template <typename T, int NPT, int LPC>
+__global__ void __launch_bounds__(kScanThreads) scan_rows_kernel(const ScanParams<T> p) {
+  constexpr int CPB = kScanThreads / LPC, NP = NPT * LPC;
+  constexpr int NX = (kScanRows * CPB + kScanThreads - 1) / kScanThreads;       // per-channel inputs per thread
+  constexpr int NB = kScanRows * 2 * NP / kScanThreads;                         // B and C values per thread (a multiple)
+  constexpr bool kAheadB = NB <= 32 && NB > 0;
+  __shared__ __align__(16) float sBC[kScanRows][2 * NP];
+  __shared__ float sDt[kScanRows][CPB], sDx[kScanRows][CPB], sY[kScanRows][CPB];
+  const int seq = blockIdx.y, tid = threadIdx.x;
+  const int start = p.q.q_cu[seq], len = p.q.q_cu[seq + 1] - start;
+  if (len < 2) return;
+  const int slot = record_of(p.q, seq);
+  if (slot < 0) return;
+  const bool cont = p.q.kv_lens[seq] > len;
+  const int c0 = blockIdx.x * CPB, ch = tid / LPC, ln = tid % LPC, n0 = ln * NPT;
+  const int c = c0 + ch;
+  const bool live = c < p.C;
+  float S[NPT], A2[NPT];
+#pragma unroll
+  for (int i = 0; i < NPT; ++i) S[i] = A2[i] = 0.f;
+  float* rec = p.state + (size_t(slot) * p.C + c) * p.N;
+  if (live) {
+    load_states<NPT>(p.A + size_t(c) * p.N, n0, p.N, A2);
+    if (cont) load_states<NPT>(rec, n0, p.N, S);
+#pragma unroll
+    for (int i = 0; i < NPT; ++i) A2[i] *= scan_unit<T>();
+  }
+  // inputs of the channel part: element i * kScanThreads + tid of the [row][channel] tile
+  float rdt[NX], rx[NX], rz[NX], rb[kAheadB ? NB : 1];
+  auto fetch = [&](int b) {
+    const int m = min(kScanRows, len - b);
+#pragma unroll
+    for (int i = 0; i < NX; ++i) {
+      const int e = i * kScanThreads + tid, row = e / CPB, cc = c0 + e % CPB;
+      rdt[i] = rx[i] = rz[i] = 0.f;
+      if (row < m && cc < p.C) {
+        const size_t t = size_t(start + b + row);
+        rdt[i] = p.dt[t * p.C + cc];
+        rx[i] = to_f32(p.x[t * p.C + cc]);
+        rz[i] = to_f32(p.z[t * p.ldz + cc]);
+      }
+    }
+    if (kAheadB) {
+#pragma unroll
+      for (int i = 0; i < NB; ++i) {
+        const int e = i * kScanThreads + tid, row = e / (2 * NP), n = e % (2 * NP), nn = n < NP ? n : n - NP;
+        rb[kAheadB ? i : 0] = 0.f;
+        if (row < m && nn < p.N) rb[kAheadB ? i : 0] = to_f32((n < NP ? p.B : p.Cm)[size_t(start + b + row) * p.ldb + nn]);
+      }
+    }
+  };
+  fetch(0);
+  for (int b = 0; b < len; b += kScanRows) {
+    const int m = min(kScanRows, len - b);
+    float x[NX], z[NX];
+#pragma unroll
+    for (int i = 0; i < NX; ++i) {
+      const int e = i * kScanThreads + tid, row = e / CPB, cc = e % CPB;
+      x[i] = rx[i];
+      z[i] = rz[i];
+      if (row < kScanRows) {
+        const float dt = c0 + cc < p.C ? softplus(rdt[i] + p.dt_bias[c0 + cc]) : 0.f;
+        sDt[row][cc] = dt;
+        sDx[row][cc] = dt * x[i];
+      }
+    }
+    if (kAheadB) {
+#pragma unroll
+      for (int i = 0; i < NB; ++i) {
+        const int e = i * kScanThreads + tid;
+        (&sBC[0][0])[e] = rb[kAheadB ? i : 0];
+      }
+    } else {
+      for (int e = tid; e < kScanRows * 2 * NP; e += kScanThreads) {
+        const int row = e / (2 * NP), n = e % (2 * NP), nn = n < NP ? n : n - NP;
+        (&sBC[0][0])[e] = row < m && nn < p.N ? to_f32((n < NP ? p.B : p.Cm)[size_t(start + b + row) * p.ldb + nn]) : 0.f;
+      }
+    }
+    __syncthreads();
+    if (b + kScanRows < len) fetch(b + kScanRows);
+    // rows in groups of four, so that their exponentials overlap and the sums over a channel's lanes share their shuffles;
+    // rows beyond m hold dt = 0: they leave the state as it is
+#pragma unroll 1
+    for (int g = 0; g < kScanRows; g += 4) {
+      if (g >= m) break;
+      float y[4];
+#pragma unroll
+      for (int r = 0; r < 4; ++r) {
+        const bool in = g + r < m;
+        const float dt = in ? sDt[g + r][ch] : 0.f, dx = in ? sDx[g + r][ch] : 0.f;
+        float acc = 0.f;
+#pragma unroll
+        for (int i = 0; i < NPT; i += 4) {
+          const float4 bb = *reinterpret_cast<const float4*>(&sBC[g + r][n0 + i]);
+          const float4 cm = *reinterpret_cast<const float4*>(&sBC[g + r][NP + n0 + i]);
+          S[i] = fmaf(scan_decay<T>(dt * A2[i]), S[i], dx * bb.x);
+          S[i + 1] = fmaf(scan_decay<T>(dt * A2[i + 1]), S[i + 1], dx * bb.y);
+          S[i + 2] = fmaf(scan_decay<T>(dt * A2[i + 2]), S[i + 2], dx * bb.z);
+          S[i + 3] = fmaf(scan_decay<T>(dt * A2[i + 3]), S[i + 3], dx * bb.w);
+          acc = fmaf(S[i], cm.x, fmaf(S[i + 1], cm.y, fmaf(S[i + 2], cm.z, fmaf(S[i + 3], cm.w, acc))));
+        }
+        y[r] = acc;
+      }
+      if constexpr (LPC >= 4) {
+        const bool b0 = ln & 1, b1 = ln & 2;
+        float a0 = b0 ? y[2] : y[0], a1 = b0 ? y[3] : y[1];
+        a0 += __shfl_xor_sync(0xffffffffu, b0 ? y[0] : y[2], 1);
+        a1 += __shfl_xor_sync(0xffffffffu, b0 ? y[1] : y[3], 1);
+        float a = b1 ? a1 : a0;
+        a += __shfl_xor_sync(0xffffffffu, b1 ? a0 : a1, 2);
+#pragma unroll
+        for (int o = 4; o < LPC; o <<= 1) a += __shfl_xor_sync(0xffffffffu, a, o);
+        if (ln < 4) sY[g + (b0 ? 2 : 0) + (b1 ? 1 : 0)][ch] = a;
+      } else {
+#pragma unroll
+        for (int r = 0; r < 4; ++r) {
+          if (LPC == 2) y[r] += __shfl_xor_sync(0xffffffffu, y[r], 1);
+          if (ln == 0) sY[g + r][ch] = y[r];
+        }
+      }
+    }
+    __syncthreads();
+#pragma unroll
+    for (int i = 0; i < NX; ++i) {
+      const int e = i * kScanThreads + tid, row = e / CPB, cc = e % CPB;
+      if (row < m && c0 + cc < p.C)
+        from_f32(p.out + size_t(start + b + row) * p.C + c0 + cc, fmaf(p.D[c0 + cc], x[i], sY[row][cc]) * act_silu(z[i]));
+    }
+    __syncthreads();
+  }
+  if (live) store_states<NPT>(rec, n0, p.N, S);
+}
+
+// Single rows: kScanIter groups of channels per CTA, all their states requested before any is worked on.
+constexpr int kScanIter = 4;
+template <typename T, int NPT, int LPC>
+__global__ void __launch_bounds__(kScanThreads) scan_single_kernel(const ScanParams<T> p) {
+  constexpr int CPB = kScanThreads / LPC;
+  constexpr int IT = NPT > 4 ? 1 : kScanIter;
+  const int seq = blockIdx.y, tid = threadIdx.x;
+  const int t = p.q.q_cu[seq];
+  if (p.q.q_cu[seq + 1] - t != 1) return;
+  const int slot = record_of(p.q, seq);
+  if (slot < 0) return;
+  const bool cont = p.q.kv_lens[seq] > 1;
+  const int ch = tid / LPC, ln = tid % LPC, n0 = ln * NPT;
+  float S[IT][NPT], A[IT][NPT], dt[IT], x[IT], B[NPT], Cm[NPT];
+#pragma unroll
+  for (int k = 0; k < IT; ++k) {
+    const int c = (blockIdx.x * IT + k) * CPB + ch;
+    dt[k] = x[k] = 0.f;
+#pragma unroll
+    for (int i = 0; i < NPT; ++i) S[k][i] = A[k][i] = 0.f;
+    if (c < p.C) {
+      if (cont) load_states<NPT>(p.state + (size_t(slot) * p.C + c) * p.N, n0, p.N, S[k]);
+      load_states<NPT>(p.A + size_t(c) * p.N, n0, p.N, A[k]);
+      dt[k] = p.dt[size_t(t) * p.C + c] + p.dt_bias[c];
+      x[k] = to_f32(p.x[size_t(t) * p.C + c]);
+    }
+  }
+#pragma unroll
+  for (int i = 0; i < NPT; ++i) {
+    const bool in = n0 + i < p.N;
+    B[i] = in ? to_f32(p.B[size_t(t) * p.ldb + n0 + i]) : 0.f;
+    Cm[i] = in ? to_f32(p.Cm[size_t(t) * p.ldb + n0 + i]) : 0.f;
+  }
+#pragma unroll
+  for (int k = 0; k < IT; ++k) {
+    const int c = (blockIdx.x * IT + k) * CPB + ch;
+    const float step = softplus(dt[k]), dx = step * x[k];
+    float y = 0.f;
+#pragma unroll
+    for (int i = 0; i < NPT; ++i) {
+      S[k][i] = fmaf(scan_decay<T>(step * (A[k][i] * scan_unit<T>())), S[k][i], dx * B[i]);
+      y = fmaf(S[k][i], Cm[i], y);
+    }
+#pragma unroll
+    for (int o = 1; o < LPC; o <<= 1) y += __shfl_xor_sync(0xffffffffu, y, o);
+    if (c < p.C) {
+      store_states<NPT>(p.state + (size_t(slot) * p.C + c) * p.N, n0, p.N, S[k]);
+      if (ln == 0)
+        from_f32(p.out + size_t(t) * p.C + c, fmaf(p.D[c], x[k], y) * act_silu(to_f32(p.z[size_t(t) * p.ldz + c])));
+    }
+  }
+}
+
+template <typename T, int NPT, int LPC>
+static int launch_scan_as(const ScanParams<T>& p, int has_long, int has_single, cudaStream_t st) {
+  constexpr int CPB = kScanThreads / LPC;
+  constexpr int IT = NPT > 4 ? 1 : kScanIter;
+  if (has_single) scan_single_kernel<T, NPT, LPC><<<dim3((p.C + CPB * IT - 1) / (CPB * IT), p.q.n), kScanThreads, 0, st>>>(p);
+  if (has_long) scan_rows_kernel<T, NPT, LPC><<<dim3((p.C + CPB - 1) / CPB, p.q.n), kScanThreads, 0, st>>>(p);
+  return cudaGetLastError() == cudaSuccess ? 0 : -1;
+}
+template <typename T>
+static int launch_scan(const ScanParams<T>& p, int has_long, int has_single, cudaStream_t st) {
+  const int n = p.N;
+  if (n <= 4) return launch_scan_as<T, 4, 1>(p, has_long, has_single, st);
+  if (n <= 8) return launch_scan_as<T, 4, 2>(p, has_long, has_single, st);
+  if (n <= 16) return launch_scan_as<T, 4, 4>(p, has_long, has_single, st);
+  if (n <= 32) return launch_scan_as<T, 4, 8>(p, has_long, has_single, st);
+  if (n <= 64) return launch_scan_as<T, 4, 16>(p, has_long, has_single, st);
+  if (n <= 128) return launch_scan_as<T, 4, 32>(p, has_long, has_single, st);
+  if (n <= 256) return launch_scan_as<T, 8, 32>(p, has_long, has_single, st);
+  return -2;
+}
+
+template <typename F>
+static int by_type(int f32, F&& f) {
+  return f32 ? f(static_cast<float*>(nullptr)) : f(static_cast<__nv_bfloat16*>(nullptr));
+}
+static Seqs make_seqs(const void* q_cu, const void* kv_lens, const void* slots, int n, int n_slots) {
+  return Seqs{static_cast<const int*>(q_cu), static_cast<const int*>(kv_lens), static_cast<const int*>(slots), n, n_slots,
+              xl_host::status_word()};
+}
+static bool aligned16(const void* a, const void* b, const void* c, const void* d) {
+  return !((reinterpret_cast<uintptr_t>(a) | reinterpret_cast<uintptr_t>(b) | reinterpret_cast<uintptr_t>(c) |
+            reinterpret_cast<uintptr_t>(d)) & 15);
+}
+
+}  // namespace xl_rc
+
+using namespace xl_rc;
+
+// `f32` below: 1 when the model's tensors are fp32, 0 for bf16.  q_cu [n_seqs + 1], kv_lens and slots [n_seqs].
+// `has_long` / `has_single`: whether any sequence of the step may have several rows / a single one.
+
+// out [n_mix, rows, W] = h + (previous row of the sequence - h) * mu[j]; last [n_slots, W]
+XL_API int xl_token_shift(const void* h, const void* mu, void* last, void* out, const void* token_seq, const void* q_cu,
+                          const void* kv_lens, const void* slots, int n_seqs, int n_slots, int rows, int W, int n_mix, int f32,
+                          void* stream) {
+  if (rows <= 0) return 0;
+  cudaStream_t st = static_cast<cudaStream_t>(stream);
+  const Seqs q = make_seqs(q_cu, kv_lens, slots, n_seqs, n_slots);
+  return by_type(f32, [&](auto* tag) {
+    using T = std::remove_pointer_t<decltype(tag)>;
+    const T *hh = static_cast<const T*>(h), *m = static_cast<const T*>(mu);
+    T *l = static_cast<T*>(last), *o = static_cast<T*>(out);
+    const int* ts = static_cast<const int*>(token_seq);
+    if (W % 8 == 0 && aligned16(h, mu, last, out)) token_shift_kernel<T, 8><<<rows, 256, 0, st>>>(hh, m, l, o, ts, q, rows, W, n_mix);
+    else token_shift_kernel<T, 1><<<rows, 256, 0, st>>>(hh, m, l, o, ts, q, rows, W, n_mix);
+    return cudaGetLastError() == cudaSuccess ? 0 : -1;
+  });
+}
+
+// out [rows, C] = silu(bias + causal convolution of x (row pitch ldx) with w [C, taps]); state [n_slots, taps - 1, C]
+XL_API int xl_conv_silu(const void* x, const void* w, const void* bias, void* state, void* out, const void* token_seq, const void* q_cu,
+                        const void* kv_lens, const void* slots, int n_seqs, int n_slots, int rows, int C, int taps, long ldx,
+                        int has_long, int f32, void* stream) {
+  if (rows <= 0) return 0;
+  if (taps < 1) return -2;
+  cudaStream_t st = static_cast<cudaStream_t>(stream);
+  const Seqs q = make_seqs(q_cu, kv_lens, slots, n_seqs, n_slots);
+  return by_type(f32, [&](auto* tag) {
+    using T = std::remove_pointer_t<decltype(tag)>;
+    const T *xx = static_cast<const T*>(x), *ww = static_cast<const T*>(w), *b = static_cast<const T*>(bias);
+    T *s = static_cast<T*>(state), *o = static_cast<T*>(out);
+    const int* ts = static_cast<const int*>(token_seq);
+    const bool vec = C % 8 == 0 && ldx % 8 == 0 && aligned16(x, bias, state, out);
+    const int per = vec ? 8 : 1, cols = (C + per * 128 - 1) / (per * 128);
+    const dim3 grid((rows + kConvRows - 1) / kConvRows, cols);
+#define XL_CONV(V, TAPS) conv_silu_kernel<T, V, TAPS><<<grid, 128, 0, st>>>(xx, ww, b, s, o, ts, q, rows, C, taps, ldx)
+    if (vec) {
+      if (taps == 4) XL_CONV(8, 4); else if (taps == 3) XL_CONV(8, 3); else if (taps == 2) XL_CONV(8, 2); else XL_CONV(8, 0);
+    } else {
+      XL_CONV(1, 0);
+    }
+#undef XL_CONV
+    if (has_long && taps > 1) {
+      if (vec) conv_record_kernel<T, 8><<<dim3(n_seqs, cols), 128, 0, st>>>(xx, s, q, C, taps, ldx);
+      else conv_record_kernel<T, 1><<<dim3(n_seqs, cols), 128, 0, st>>>(xx, s, q, C, taps, ldx);
+    }
+    return cudaGetLastError() == cudaSuccess ? 0 : -1;
+  });
+}
+
+// r, k, v [rows, H * d] with row pitch ld, gate with ldg, z [rows, H * d] fp32 dense; state [n_slots, H, d, d] fp32; out with
+// row pitch ldo.  Longer portions in segments of L rows, at most seg_cap of them; ws_s / ws_p (null when no portion has more
+// than L rows) hold seg_cap * H * d * d and seg_cap * H * d floats.
+XL_API int xl_time_mix(const void* r, const void* k, const void* v, const void* z, const void* w0, const void* u, const void* gate,
+                       const void* norm_w, float scale, float eps, void* state, void* out, const void* q_cu, const void* kv_lens,
+                       const void* slots, int n_seqs, int n_slots, int H, int d, long ld, long ldg, long ldo, int L, int seg_cap,
+                       void* ws_s, void* ws_p, int has_long, int has_single, int f32, void* stream) {
+  if (n_seqs <= 0) return 0;
+  if (H < 1 || H > 65535 || d < 1 || d > 2048 || L < 2) return -2;
+  return by_type(f32, [&](auto* tag) {
+    using T = std::remove_pointer_t<decltype(tag)>;
+    MixParams<T> p;
+    p.r = static_cast<const T*>(r); p.k = static_cast<const T*>(k); p.v = static_cast<const T*>(v);
+    p.gate = static_cast<const T*>(gate);
+    p.z = static_cast<const float*>(z); p.w0 = static_cast<const float*>(w0); p.u = static_cast<const float*>(u);
+    p.norm_w = static_cast<const T*>(norm_w);
+    p.state = static_cast<float*>(state); p.out = static_cast<T*>(out);
+    p.ld = ld; p.ldg = ldg; p.ldo = ldo; p.H = H; p.d = d; p.scale = scale; p.eps = eps;
+    p.q = make_seqs(q_cu, kv_lens, slots, n_seqs, n_slots);
+    p.L = L; p.ws_s = static_cast<float*>(ws_s); p.ws_p = static_cast<float*>(ws_p);
+    return launch_time_mix<T>(p, seg_cap, has_long, has_single, static_cast<cudaStream_t>(stream));
+  });
+}
+
+// out [rows, C] = (scan + D x) silu(z); B, Cm with row pitch ldb, z with ldz; state [n_slots, C, N] fp32
+XL_API int xl_selective_scan(const void* x, const void* dt, const void* dt_bias, const void* A, const void* B, const void* Cm,
+                             const void* D, const void* z, void* state, void* out, const void* q_cu, const void* kv_lens,
+                             const void* slots, int n_seqs, int n_slots, int C, int N, long ldb, long ldz, int has_long, int has_single,
+                             int f32, void* stream) {
+  if (n_seqs <= 0) return 0;
+  if (C < 1 || N < 1 || n_seqs > 65535) return -2;
+  return by_type(f32, [&](auto* tag) {
+    using T = std::remove_pointer_t<decltype(tag)>;
+    ScanParams<T> p;
+    p.x = static_cast<const T*>(x); p.dt = static_cast<const float*>(dt); p.dt_bias = static_cast<const float*>(dt_bias);
+    p.A = static_cast<const float*>(A); p.D = static_cast<const float*>(D);
+    p.B = static_cast<const T*>(B); p.Cm = static_cast<const T*>(Cm); p.z = static_cast<const T*>(z);
+    p.state = static_cast<float*>(state); p.out = static_cast<T*>(out);
+    p.ldb = ldb; p.ldz = ldz; p.C = C; p.N = N;
+    p.q = make_seqs(q_cu, kv_lens, slots, n_seqs, n_slots);
+    return launch_scan<T>(p, has_long, has_single, static_cast<cudaStream_t>(stream));
+  });
+}

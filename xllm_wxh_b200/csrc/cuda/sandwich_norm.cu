@@ -1,4 +1,4 @@
-// Fused steps of a decoder whose sublayers are normed before and after and whose residual stream is fp32:
+// Fused steps around an fp32 residual stream, of decoders whose sublayers are normed before and after:
 //
 //   x += rms(y) * w_post;  h = rms(x) * w_next                      (one kernel between a sublayer and the next one)
 //
@@ -6,9 +6,14 @@
 //   SRC_ROWS   y is a tensor (the output of o_proj / down_proj);
 //   SRC_MOE    y is assembled here: weighted sum of the chosen experts' rows, identity experts (whose output is the
 //              sublayer's input itself, times the weight) and a shared expert, so that it never exists in memory;
-//   SRC_EMBED  there is no y: x = table[token] * scale starts the residual stream.
+//   SRC_EMBED  there is no y: x = table[token] * scale starts the residual stream;
+// and of decoders whose sublayers are normed before only:
+//   SRC_ADD    x += scale * y                                    (no norm behind the sublayer)
+//   SRC_SET    x = y + vec, y in fp32                            (the residual is replaced by a product of itself)
 // Also the kernel that follows the qkv projection where positions do not rotate anything: per-head q / k RMSNorm and the
-// write of k and v into the paged cache (q is normed in place); and the gated activation of an unfused feed-forward.
+// write of k and v into the paged cache (q is normed in place), with norms per head or over the whole projection; the gated
+// activation of an unfused feed-forward; a sigmoid gate on attention's output; and the rows [x, x0] of a product that takes
+// in the residual stream.
 //
 // All arithmetic is fp32; tensors are bf16, or fp32 when the model runs in 32-bit.
 #include <type_traits>
@@ -18,7 +23,7 @@
 namespace xl_sn {
 using namespace xl;
 
-enum { SRC_ROWS = 0, SRC_MOE = 1, SRC_EMBED = 2 };
+enum { SRC_ROWS = 0, SRC_MOE = 1, SRC_EMBED = 2, SRC_ADD = 3, SRC_SET = 4 };
 
 template <typename T>
 struct NormParams {
@@ -41,7 +46,10 @@ struct NormParams {
   const int* tokens;
   const T* table;            // [V, H]
   int V;
-  float scale;
+  float scale;               // also SRC_ADD
+  // SRC_SET
+  const float* y32;          // [rows, H]
+  const float* vec;          // [H]
 };
 
 // sum over the block of one value per thread; `red` holds one float per warp
@@ -75,6 +83,18 @@ __global__ void __launch_bounds__(256) sandwich_norm_kernel(const NormParams<T> 
     if (v < nvec) {
       if (SRC == SRC_ROWS) {
         load8(p.y + size_t(row) * H + v * 8, y[i]);
+      } else if (SRC == SRC_ADD) {
+        float x[8];
+        load8(p.y + size_t(row) * H + v * 8, y[i]);
+        load8(p.x + size_t(row) * H + v * 8, x);
+#pragma unroll
+        for (int e = 0; e < 8; ++e) y[i][e] = fmaf(p.scale, y[i][e], x[e]);
+      } else if (SRC == SRC_SET) {
+        float x[8];
+        load8(p.y32 + size_t(row) * H + v * 8, y[i]);
+        load8(p.vec + v * 8, x);
+#pragma unroll
+        for (int e = 0; e < 8; ++e) y[i][e] += x[e];
       } else if (SRC == SRC_EMBED) {
         load8(p.table + size_t(clamp_id(p.tokens[row], p.V)) * H + v * 8, y[i]);
 #pragma unroll
@@ -102,7 +122,7 @@ __global__ void __launch_bounds__(256) sandwich_norm_kernel(const NormParams<T> 
       for (int e = 0; e < 8; ++e) ss += y[i][e] * y[i][e];
     }
   }
-  if (SRC != SRC_EMBED) {
+  if (SRC == SRC_ROWS || SRC == SRC_MOE) {
     const float r_post = rsqrtf(block_sum(ss, red_a) / float(H) + p.eps);
     ss = 0.f;
 #pragma unroll
@@ -150,6 +170,10 @@ __global__ void __launch_bounds__(256) sandwich_norm_any_kernel(const NormParams
     float y = 0.f;
     if (SRC == SRC_ROWS) {
       y = to_f32(p.y[size_t(row) * H + i]);
+    } else if (SRC == SRC_ADD) {
+      y = fmaf(p.scale, to_f32(p.y[size_t(row) * H + i]), p.x[size_t(row) * H + i]);
+    } else if (SRC == SRC_SET) {
+      y = p.y32[size_t(row) * H + i] + p.vec[i];
     } else if (SRC == SRC_EMBED) {
       y = to_f32(p.table[size_t(clamp_id(p.tokens[row], p.V)) * H + i]) * p.scale;
     } else {
@@ -163,7 +187,7 @@ __global__ void __launch_bounds__(256) sandwich_norm_any_kernel(const NormParams
     row_cache[i] = y;
     ss += y * y;
   }
-  if (SRC != SRC_EMBED) {
+  if (SRC == SRC_ROWS || SRC == SRC_MOE) {
     const float r_post = rsqrtf(block_sum(ss, red_a) / float(H) + p.eps);
     ss = 0.f;
     for (int i = threadIdx.x; i < H; i += blockDim.x) {
@@ -318,6 +342,100 @@ static int launch_qknorm(void* qkv, const void* slots, const void* q_w, const vo
   return cudaGetLastError() == cudaSuccess ? 0 : -1;
 }
 
+// ---------------------------------------------------------------- q / k norm over the whole projection + cache write
+// One row per CTA; rows hold q, k and v (and possibly more behind them) with pitch ld.
+template <typename T, int V>
+__global__ void __launch_bounds__(256) qknorm_all_kernel(T* __restrict__ qkv, const int* __restrict__ slots, const T* __restrict__ q_w,
+                                                         const T* __restrict__ k_w, T* __restrict__ k_cache, T* __restrict__ v_cache,
+                                                         int nq, int nk, int nv, long ld, float eps, long cache_slots) {
+  __shared__ float red_q[8], red_k[8];
+  const int t = blockIdx.x;
+  T* row = qkv + size_t(t) * ld;
+  auto load = [](const T* p, float (&f)[V]) {
+    if constexpr (V == 8) load8(p, f); else f[0] = to_f32(*p);
+  };
+  auto store = [](T* p, const float (&f)[V]) {
+    if constexpr (V == 8) store8(p, f); else from_f32(p, f[0]);
+  };
+  float sq = 0.f, sk = 0.f, f[V], w[V];
+  for (int c = threadIdx.x * V; c < nq + nk; c += blockDim.x * V) {
+    load(row + c, f);
+    float s = 0.f;
+#pragma unroll
+    for (int e = 0; e < V; ++e) s += f[e] * f[e];
+    if (c < nq) sq += s; else sk += s;
+  }
+  const float rq = rsqrtf(block_sum(sq, red_q) / float(nq) + eps), rk = rsqrtf(block_sum(sk, red_k) / float(nk) + eps);
+  const int slot = slots[t];
+  const bool in = slot >= 0 && slot < cache_slots;
+  for (int c = threadIdx.x * V; c < nq + nk + nv; c += blockDim.x * V) {
+    load(row + c, f);
+    if (c < nq) {
+      load(q_w + c, w);
+#pragma unroll
+      for (int e = 0; e < V; ++e) f[e] = f[e] * rq * w[e];
+      store(row + c, f);
+    } else if (c < nq + nk) {
+      load(k_w + (c - nq), w);
+#pragma unroll
+      for (int e = 0; e < V; ++e) f[e] = f[e] * rk * w[e];
+      if (in) store(k_cache + size_t(slot) * nk + (c - nq), f);
+    } else if (in) {
+      store(v_cache + size_t(slot) * nv + (c - nq - nk), f);
+    }
+  }
+}
+template <typename T>
+static int launch_qknorm_all(void* qkv, const void* slots, const void* q_w, const void* k_w, void* k_cache, void* v_cache, int rows, int nq,
+                             int nk, int nv, long ld, float eps, long cache_slots, cudaStream_t st) {
+  T *x = static_cast<T*>(qkv), *kc = static_cast<T*>(k_cache), *vc = static_cast<T*>(v_cache);
+  const T *qw = static_cast<const T*>(q_w), *kw = static_cast<const T*>(k_w);
+  const int* s = static_cast<const int*>(slots);
+  if (nq % 8 == 0 && nk % 8 == 0 && nv % 8 == 0 && ld % 8 == 0 && al16(qkv, q_w, k_w, k_cache) && al16(v_cache))
+    qknorm_all_kernel<T, 8><<<rows, 256, 0, st>>>(x, s, qw, kw, kc, vc, nq, nk, nv, ld, eps, cache_slots);
+  else
+    qknorm_all_kernel<T, 1><<<rows, 256, 0, st>>>(x, s, qw, kw, kc, vc, nq, nk, nv, ld, eps, cache_slots);
+  return cudaGetLastError() == cudaSuccess ? 0 : -1;
+}
+
+// ---------------------------------------------------------------- out = o * sigmoid(gate) * scale, strided rows
+template <typename T, int V>
+__global__ void __launch_bounds__(256) sigmoid_gate_kernel(const T* __restrict__ o, const T* __restrict__ gate, T* __restrict__ out,
+                                                           long total, int n, long ldg, long ldo, float scale) {
+  const int per = n / V;
+  for (long idx = blockIdx.x * long(blockDim.x) + threadIdx.x; idx < total; idx += long(gridDim.x) * blockDim.x) {
+    const long t = idx / per;
+    const int c = int(idx % per) * V;
+    if constexpr (V == 8) {
+      float a[8], g[8];
+      load8(o + t * n + c, a);
+      load8(gate + t * ldg + c, g);
+#pragma unroll
+      for (int e = 0; e < 8; ++e) a[e] = a[e] * scale / (1.f + __expf(-g[e]));
+      store8(out + t * ldo + c, a);
+    } else {
+      from_f32(out + t * ldo + c, to_f32(o[t * n + c]) * scale / (1.f + __expf(-to_f32(gate[t * ldg + c]))));
+    }
+  }
+}
+
+// ---------------------------------------------------------------- rows [x, x0], x0 = table[token] * scale; in bf16 the fp32 x
+// as its rounded value and the rest
+template <typename T>
+__global__ void __launch_bounds__(256) split_rows_kernel(const float* __restrict__ x, const int* __restrict__ tokens,
+                                                         const T* __restrict__ table, float scale, T* __restrict__ out, int W, int V) {
+  const size_t t = blockIdx.x;
+  constexpr int parts = sizeof(T) == 2 ? 2 : 1;
+  T* dst = out + t * (parts + 1) * W;
+  const T* x0 = table + size_t(clamp_id(tokens[t], V)) * W;
+  for (int c = threadIdx.x; c < W; c += blockDim.x) {
+    const float v = x[t * W + c];
+    from_f32(dst + c, v);
+    if constexpr (parts == 2) from_f32(dst + W + c, v - to_f32(dst[c]));
+    from_f32(dst + parts * W + c, to_f32(x0[c]) * scale);
+  }
+}
+
 // ---------------------------------------------------------------- gated activation: out[t, i] = act(x[t, i]) * x[t, I + i]
 template <typename T>
 __global__ void gated_act_kernel(const T* __restrict__ x, T* __restrict__ out, long total, int I, int act) {
@@ -387,6 +505,79 @@ XL_API int xl_post_norm_add_norm(const void* y, void* x, const void* w_post, con
   auto p = base_params<__nv_bfloat16>(x, w_post, w_next, h, H, eps);
   p.y = static_cast<const __nv_bfloat16*>(y);
   return launch_norm<__nv_bfloat16, SRC_ROWS>(p, rows, al, st);
+}
+
+// x += mult * y;  h = rms(x) * w_next
+XL_API int xl_add_norm(const void* y, void* x, float mult, const void* w_next, void* h, int rows, int H, float eps, int f32, void* stream) {
+  cudaStream_t st = static_cast<cudaStream_t>(stream);
+  const bool al = al16(y, x, w_next, h);
+  if (f32) {
+    auto p = base_params<float>(x, nullptr, w_next, h, H, eps);
+    p.y = static_cast<const float*>(y); p.scale = mult;
+    return launch_norm<float, SRC_ADD>(p, rows, al, st);
+  }
+  auto p = base_params<__nv_bfloat16>(x, nullptr, w_next, h, H, eps);
+  p.y = static_cast<const __nv_bfloat16*>(y); p.scale = mult;
+  return launch_norm<__nv_bfloat16, SRC_ADD>(p, rows, al, st);
+}
+
+// x = y + vec (y [rows, H], vec [H] fp32);  h = rms(x) * w_next
+XL_API int xl_replace_norm(const void* y, const void* vec, void* x, const void* w_next, void* h, int rows, int H, float eps, int f32,
+                           void* stream) {
+  cudaStream_t st = static_cast<cudaStream_t>(stream);
+  const bool al = al16(y, x, w_next, h) && al16(vec);
+  if (f32) {
+    auto p = base_params<float>(x, nullptr, w_next, h, H, eps);
+    p.y32 = static_cast<const float*>(y); p.vec = static_cast<const float*>(vec);
+    return launch_norm<float, SRC_SET>(p, rows, al, st);
+  }
+  auto p = base_params<__nv_bfloat16>(x, nullptr, w_next, h, H, eps);
+  p.y32 = static_cast<const float*>(y); p.vec = static_cast<const float*>(vec);
+  return launch_norm<__nv_bfloat16, SRC_SET>(p, rows, al, st);
+}
+
+// out [rows, 2 W] = [x, x0] (fp32), or [rows, 3 W] = [bf16(x), bf16(x - bf16(x)), x0], x0 = table[token] * scale
+XL_API int xl_split_rows(const void* x, const void* tokens, const void* table, float scale, void* out, int rows, int W, int V, int f32,
+                         void* stream) {
+  if (rows <= 0) return 0;
+  cudaStream_t st = static_cast<cudaStream_t>(stream);
+  const float* xx = static_cast<const float*>(x);
+  const int* tk = static_cast<const int*>(tokens);
+  if (f32)
+    split_rows_kernel<float><<<rows, 256, 0, st>>>(xx, tk, static_cast<const float*>(table), scale, static_cast<float*>(out), W, V);
+  else
+    split_rows_kernel<__nv_bfloat16><<<rows, 256, 0, st>>>(xx, tk, static_cast<const __nv_bfloat16*>(table), scale,
+                                                          static_cast<__nv_bfloat16*>(out), W, V);
+  return cudaGetLastError() == cudaSuccess ? 0 : -1;
+}
+
+// RMSNorm over the nq query and over the nk key columns of rows with pitch ld (q in place); k and v to the cache slots
+// [cache_slots, nk | nv].
+XL_API int xl_qknorm_all_kvwrite(void* qkv, const void* slots, const void* q_w, const void* k_w, void* k_cache, void* v_cache, int rows,
+                                 int nq, int nk, int nv, long ld, float eps, long cache_slots, int f32, void* stream) {
+  if (rows <= 0) return 0;
+  cudaStream_t st = static_cast<cudaStream_t>(stream);
+  if (f32) return launch_qknorm_all<float>(qkv, slots, q_w, k_w, k_cache, v_cache, rows, nq, nk, nv, ld, eps, cache_slots, st);
+  return launch_qknorm_all<__nv_bfloat16>(qkv, slots, q_w, k_w, k_cache, v_cache, rows, nq, nk, nv, ld, eps, cache_slots, st);
+}
+
+// out [rows, n] (pitch ldo) = o (dense) * sigmoid(gate, pitch ldg) * scale
+XL_API int xl_sigmoid_gate(const void* o, const void* gate, void* out, int rows, int n, long ldg, long ldo, float scale, int f32,
+                           void* stream) {
+  if (rows <= 0) return 0;
+  cudaStream_t st = static_cast<cudaStream_t>(stream);
+  const bool vec = n % 8 == 0 && ldg % 8 == 0 && ldo % 8 == 0 && al16(o, gate, out);
+  const long total = long(rows) * (vec ? n / 8 : n);
+  long blocks = (total + 255) / 256;
+  if (blocks > 148 * 16) blocks = 148 * 16;
+  auto go = [&](auto* tag) {
+    using E = std::remove_pointer_t<decltype(tag)>;
+    const E *a = static_cast<const E*>(o), *g = static_cast<const E*>(gate);
+    if (vec) sigmoid_gate_kernel<E, 8><<<int(blocks), 256, 0, st>>>(a, g, static_cast<E*>(out), total, n, ldg, ldo, scale);
+    else sigmoid_gate_kernel<E, 1><<<int(blocks), 256, 0, st>>>(a, g, static_cast<E*>(out), total, n, ldg, ldo, scale);
+    return cudaGetLastError() == cudaSuccess ? 0 : -1;
+  };
+  return f32 ? go(static_cast<float*>(nullptr)) : go(static_cast<__nv_bfloat16*>(nullptr));
 }
 
 // y[t] = sum_j weights[t, j] * expert output (an expert's row of y_exp, or h_in[t] for ids >= first_identity) + shared[t];

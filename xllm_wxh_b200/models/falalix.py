@@ -270,11 +270,11 @@ class FalalixForCausalLM:
         a, eps, runs = self.args, self.args.rms_norm_eps, self.args.layer_runs
         passes = {r: t for t, r in enumerate(a.pass_starts)}
         x, h = ops.embed_rms_norm(inp.tokens, self.embed, a.embedding_scale, self.layers[runs[0]].norm1, eps)
-        x0 = ops.embedding(inp.tokens, self.embed) if passes else None
         for r, li in enumerate(runs):
             L, s = self.layers[li], a.layer_specs[li]
             if r in passes:
-                h = ops.replace_norm(ops.linear_f32(ops.split_rows(x, x0), self.loop_in), self.loop_step[passes[r]], x, L.norm1, eps)
+                both = ops.split_rows(x, inp.tokens, self.embed, a.embedding_scale)
+                h = ops.replace_norm(ops.linear_f32(both, self.loop_in), self.loop_step[passes[r]], x, L.norm1, eps)
             w_next = self.layers[runs[r + 1]].norm1 if r + 1 < len(runs) else self.final_norm
             if isinstance(s.mixer, SelectiveScanSpec):
                 y = self._scan(L.mix, s.mixer, h, inp, inp.states[r])

@@ -152,10 +152,11 @@ def replace_norm(y, vec, x, w_next, eps):
     return (_cuda() if y.is_cuda else ref).replace_norm(y, vec, x, w_next, eps)
 
 
-def split_rows(x, x0):
-    """Rows [x, x0] for a product with `split_columns` of its weight.  In a bf16 model the fp32 x enters as two bf16 parts
-    (its rounded value and the rest), so that a product of the residual stream does not round it to 8 bits."""
-    return (_cuda() if x.is_cuda else ref).split_rows(x, x0)
+def split_rows(x, ids, table, scale):
+    """Rows [x, x0] for a product with `split_columns` of its weight, x0 = table[ids] * scale.  In a bf16 model the fp32 x
+    enters as two bf16 parts (its rounded value and the rest), so that a product of the residual stream does not round it to
+    8 bits."""
+    return (_cuda() if x.is_cuda else ref).split_rows(x, ids, table, scale)
 
 
 def split_columns(w, width):

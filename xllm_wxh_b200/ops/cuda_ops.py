@@ -111,16 +111,17 @@ def _tc_gemm_ok(x: torch.Tensor, w: torch.Tensor, n_align: int = 8) -> bool:
             x.stride(0) % 8 == 0 and (x.data_ptr() | w.data_ptr()) % 16 == 0)
 
 
-def _gemm_simt(x2: torch.Tensor, w: torch.Tensor, out_dtype: torch.dtype) -> torch.Tensor:
-    """The fp32-pipe GEMM: fp32 operands, or bf16 ones of any shape."""
+def _gemm_simt(x2: torch.Tensor, w: torch.Tensor, out_dtype: torch.dtype, bias: Optional[torch.Tensor] = None, act: int = 0) -> torch.Tensor:
+    """The fp32-pipe GEMM: fp32 operands, or bf16 ones of any shape; act(x w^T + bias)."""
     global launch_count
     assert x2.dtype == w.dtype and x2.dtype in (torch.float32, torch.bfloat16) and w.stride(-1) == 1
+    assert bias is None or bias.dtype == w.dtype
     M, K = x2.shape
     N = w.shape[0]
     out = torch.empty((M, N), dtype=out_dtype, device=x2.device)
     if M > 0:
-        _check(lib().xl_gemm_simt(_ptr(x2), _ptr(w), _ptr(out), c_int(M), c_int(N), c_int(K), c_long(x2.stride(0)), c_long(w.stride(0)),
-                                  c_long(N), c_int(int(x2.dtype == torch.float32)), c_int(int(out_dtype == torch.float32)), _stream()),
+        _check(lib().xl_gemm_simt(_ptr(x2), _ptr(w), _ptr(out), _ptr(bias), c_int(act), c_int(M), c_int(N), c_int(K), c_long(x2.stride(0)),
+                                  c_long(w.stride(0)), c_long(N), c_int(int(x2.dtype == torch.float32)), c_int(int(out_dtype == torch.float32)), _stream()),
                "xl_gemm_simt")
         launch_count += 1
     return out
@@ -145,10 +146,10 @@ def linear_f32(x: torch.Tensor, w: torch.Tensor) -> torch.Tensor:
 
 def linear(x: torch.Tensor, w: torch.Tensor, bias: Optional[torch.Tensor] = None, out: Optional[torch.Tensor] = None) -> torch.Tensor:
     global launch_count
-    if x.dtype == torch.float32 or (bias is None and out is None and not _tc_gemm_ok(x.reshape(-1, x.shape[-1]), w)):
-        assert bias is None and out is None
+    if x.dtype == torch.float32 or (out is None and not _tc_gemm_ok(x.reshape(-1, x.shape[-1]), w)):
+        assert out is None
         x2 = x.reshape(-1, x.shape[-1])
-        return _gemm_simt(x2 if x2.stride(-1) == 1 else x2.contiguous(), w, x.dtype).reshape(x.shape[:-1] + (w.shape[0],))
+        return _gemm_simt(x2 if x2.stride(-1) == 1 else x2.contiguous(), w, x.dtype, bias).reshape(x.shape[:-1] + (w.shape[0],))
     assert x.dtype == torch.bfloat16 and w.dtype == torch.bfloat16, "GEMM kernel is bf16"
     x2 = x.reshape(-1, x.shape[-1])
     if x2.stride(-1) != 1:
@@ -164,6 +165,26 @@ def linear(x: torch.Tensor, w: torch.Tensor, bias: Optional[torch.Tensor] = None
         _check(rc, "xl_gemm_bf16")
         launch_count += 1
     return out.reshape(x.shape[:-1] + (N,))
+
+
+PLAIN_ACTS = {"relu2": 1, "tanh": 2}
+
+
+def act_linear(x: torch.Tensor, w: torch.Tensor, act: str) -> torch.Tensor:
+    """act(x w^T), applied to the fp32 sums in the GEMM epilogue."""
+    global launch_count
+    if x.stride(-1) != 1:
+        x = x.contiguous()
+    if not _tc_gemm_ok(x, w):
+        return _gemm_simt(x, w, x.dtype, None, PLAIN_ACTS[act])
+    M, K = x.shape
+    N = w.shape[0]
+    out = torch.empty((M, N), dtype=torch.bfloat16, device=x.device)
+    if M > 0:
+        _check(lib().xl_gemm_bf16_act(_ptr(x), _ptr(w), _ptr(out), c_int(M), c_int(N), c_int(K), c_int(x.stride(0)), c_int(w.stride(0)),
+                                      c_int(N), c_int(PLAIN_ACTS[act]), _stream()), "xl_gemm_bf16_act")
+        launch_count += 1
+    return out
 
 
 ACTS = {"silu": 0, "gelu_tanh": 1}
@@ -333,6 +354,151 @@ def qknorm_kvwrite(qkv, slots, q_w, k_w, eps, k_cache, v_cache, n_q, n_kv):
     return qkv[:, :n_q * dk]
 
 
+# ----------------------------------------------------------------------------- norms before a sublayer only, fp32 residual
+def add_norm(y: torch.Tensor, x: torch.Tensor, mult: float, w_next: torch.Tensor, eps: float) -> torch.Tensor:
+    """x += mult * y in place; returns rms(x) * w_next."""
+    global launch_count
+    T, H = y.shape
+    assert y.is_contiguous() and x.is_contiguous() and x.dtype == torch.float32
+    h = torch.empty_like(y)
+    _check(lib().xl_add_norm(_ptr(y), _ptr(x), c_float(mult), _ptr(w_next), _ptr(h), c_int(T), c_int(H), c_float(eps), _f32flag(y),
+                             _stream()), "xl_add_norm")
+    launch_count += 1
+    return h
+
+
+def replace_norm(y: torch.Tensor, vec: torch.Tensor, x: torch.Tensor, w_next: torch.Tensor, eps: float) -> torch.Tensor:
+    """x = y + vec (y, vec, x fp32); returns rms(x) * w_next."""
+    global launch_count
+    T, H = y.shape
+    assert y.is_contiguous() and x.is_contiguous() and y.dtype == x.dtype == vec.dtype == torch.float32
+    h = torch.empty((T, H), dtype=w_next.dtype, device=y.device)
+    _check(lib().xl_replace_norm(_ptr(y), _ptr(vec), _ptr(x), _ptr(w_next), _ptr(h), c_int(T), c_int(H), c_float(eps), _f32flag(h),
+                                 _stream()), "xl_replace_norm")
+    launch_count += 1
+    return h
+
+
+def split_rows(x: torch.Tensor, ids: torch.Tensor, table: torch.Tensor, scale: float) -> torch.Tensor:
+    global launch_count
+    T, W = x.shape
+    assert x.is_contiguous() and table.is_contiguous() and x.dtype == torch.float32
+    out = torch.empty((T, (2 if table.dtype == torch.float32 else 3) * W), dtype=table.dtype, device=x.device)
+    _check(lib().xl_split_rows(_ptr(x), _ptr(ids), _ptr(table), c_float(scale), _ptr(out), c_int(T), c_int(W), c_int(table.shape[0]),
+                               _f32flag(table), _stream()), "xl_split_rows")
+    launch_count += 1
+    return out
+
+
+def qknorm_all_kvwrite(qkv, slots, q_w, k_w, eps, k_cache, v_cache, n_q, n_kv):
+    """RMSNorm over all query and over all key columns (q in place), k and v into the paged caches; rows of qkv may hold more
+    behind v.  Returns q [T, n_q * dk] (a view of qkv)."""
+    global launch_count
+    T = qkv.shape[0]
+    dk, dv = k_cache.shape[-1], v_cache.shape[-1]
+    assert qkv.stride(1) == 1 and qkv.shape[1] >= (n_q + n_kv) * dk + n_kv * dv and k_cache.dtype == qkv.dtype
+    _check(lib().xl_qknorm_all_kvwrite(_ptr(qkv), _ptr(slots), _ptr(q_w), _ptr(k_w), _ptr(k_cache), _ptr(v_cache), c_int(T),
+                                       c_int(n_q * dk), c_int(n_kv * dk), c_int(n_kv * dv), c_long(qkv.stride(0)), c_float(eps),
+                                       c_long(k_cache.shape[0] * k_cache.shape[1]), _f32flag(qkv), _stream()), "xl_qknorm_all_kvwrite")
+    launch_count += 1
+    return qkv[:, :n_q * dk]
+
+
+def gate_into(o: torch.Tensor, gate: torch.Tensor, scale: float, out: torch.Tensor) -> None:
+    global launch_count
+    T, n = o.shape
+    assert o.is_contiguous() and gate.shape == out.shape == o.shape and gate.stride(1) == out.stride(1) == 1
+    _check(lib().xl_sigmoid_gate(_ptr(o), _ptr(gate), _ptr(out), c_int(T), c_int(n), c_long(gate.stride(0)), c_long(out.stride(0)),
+                                 c_float(scale), _f32flag(o), _stream()), "xl_sigmoid_gate")
+    launch_count += 1
+
+
+# ----------------------------------------------------------------------------- recurrent layers
+def _state_args(inp, state):
+    assert state.is_contiguous()
+    n = inp.B if inp.padded else inp.n_seqs
+    return n, (_ptr(inp.q_cu), _ptr(inp.kv_lens), _ptr(inp.state_slots), c_int(n), c_int(state.shape[0]))
+
+
+def _rows_out(inp, shape, like):
+    """Rows that belong to no sequence (padding) are written by no recurrent kernel: keep them finite."""
+    return (torch.zeros if inp.padded else torch.empty)(shape, dtype=like.dtype, device=like.device)
+
+
+def token_shift(h: torch.Tensor, mu: torch.Tensor, last: torch.Tensor, inp) -> torch.Tensor:
+    """[n, T, W]: h + (predecessor - h) * mu[i]; the record of every sequence in `last` [slots, W] becomes its last row."""
+    global launch_count
+    T, W = h.shape
+    assert h.is_contiguous() and mu.is_contiguous() and mu.dtype == last.dtype == h.dtype
+    n, seqs = _state_args(inp, last)
+    out = torch.empty((mu.shape[0], T, W), dtype=h.dtype, device=h.device)
+    _check(lib().xl_token_shift(_ptr(h), _ptr(mu), _ptr(last), _ptr(out), _ptr(inp.token_seq), *seqs, c_int(T), c_int(W),
+                                c_int(mu.shape[0]), _f32flag(h), _stream()), "xl_token_shift")
+    launch_count += 1
+    return out
+
+
+def conv_silu(x: torch.Tensor, w: torch.Tensor, b: torch.Tensor, state: torch.Tensor, inp) -> torch.Tensor:
+    """silu(b + causal convolution of x [T, C] (may be a strided view) with w [C, taps]); state [slots, taps - 1, C]."""
+    global launch_count
+    T, C = x.shape
+    assert x.stride(1) == 1 and w.is_contiguous() and w.dtype == b.dtype == state.dtype == x.dtype
+    n, seqs = _state_args(inp, state)
+    out = _rows_out(inp, (T, C), x)
+    _check(lib().xl_conv_silu(_ptr(x), _ptr(w), _ptr(b), _ptr(state), _ptr(out), _ptr(inp.token_seq), *seqs, c_int(T), c_int(C),
+                              c_int(w.shape[1]), c_long(x.stride(0)), c_int(int(inp.has_prefill)), _f32flag(x), _stream()), "xl_conv_silu")
+    launch_count += 2 if inp.has_prefill and w.shape[1] > 1 else 1
+    return out
+
+
+def mix_segment_rows(T: int, H: int, d: int) -> int:
+    """Rows per segment of the time mixing of longer portions: short enough that segments x heads fill the device a few times
+    over, long enough that the states between segments stay small beside the rows' own work."""
+    want = 8 * sm_count() * 64 // max(64, d)
+    L = max(1, T * H // want)
+    return min(512, max(64, 1 << (L.bit_length() - 1)))
+
+
+def time_mix(r, k, v, z, w0, u, gate, norm_w, scale, eps, state, inp, out) -> None:
+    global launch_count
+    H, d = u.shape
+    T = r.shape[0]
+    for t in (r, k, v):
+        assert t.stride(1) == 1 and t.stride(0) == r.stride(0) and t.dtype == out.dtype and t.shape == (T, H * d)
+    assert gate.stride(1) == out.stride(1) == 1 and z.is_contiguous() and z.dtype == w0.dtype == u.dtype == state.dtype == torch.float32
+    n, seqs = _state_args(inp, state)
+    has_long = bool(inp.has_prefill) and T > 1
+    if inp.padded:
+        out.zero_()
+    L, cap, ws, wp = 2, 0, None, None
+    if has_long:
+        L = mix_segment_rows(T, H, d)
+        cap = T // L + min(n, T // 2)                       # every portion of two and more rows ends with one partly filled segment
+        if (T if inp.padded else inp.max_q) > L and d <= 128:
+            ws = torch.empty((cap, H, d, d), dtype=torch.float32, device=r.device)
+            wp = torch.empty((cap, H, d), dtype=torch.float32, device=r.device)
+    _check(lib().xl_time_mix(_ptr(r), _ptr(k), _ptr(v), _ptr(z), _ptr(w0), _ptr(u), _ptr(gate), _ptr(norm_w), c_float(scale), c_float(eps),
+                             _ptr(state), _ptr(out), *seqs, c_int(H), c_int(d), c_long(r.stride(0)), c_long(gate.stride(0)),
+                             c_long(out.stride(0)), c_int(L), c_int(cap), _ptr(ws), _ptr(wp), c_int(int(has_long)), c_int(1), _f32flag(r),
+                             _stream()), "xl_time_mix")
+    launch_count += 1 + (0 if not has_long else 1 if ws is None else 3)
+
+
+def selective_scan(x, dt, dt_bias, A, B, C, D, z, state, inp) -> torch.Tensor:
+    global launch_count
+    T, ch = x.shape
+    N = A.shape[1]
+    assert x.is_contiguous() and dt.is_contiguous() and dt.dtype == dt_bias.dtype == A.dtype == D.dtype == state.dtype == torch.float32
+    assert B.stride(1) == C.stride(1) == z.stride(1) == 1 and B.stride(0) == C.stride(0) and B.dtype == z.dtype == x.dtype
+    n, seqs = _state_args(inp, state)
+    out = _rows_out(inp, (T, ch), x)
+    _check(lib().xl_selective_scan(_ptr(x), _ptr(dt), _ptr(dt_bias), _ptr(A), _ptr(B), _ptr(C), _ptr(D), _ptr(z), _ptr(state), _ptr(out),
+                                   *seqs, c_int(ch), c_int(N), c_long(B.stride(0)), c_long(z.stride(0)), c_int(int(inp.has_prefill)),
+                                   c_int(1), _f32flag(x), _stream()), "xl_selective_scan")
+    launch_count += 2 if inp.has_prefill else 1
+    return out
+
+
 # ----------------------------------------------------------------------------- attention
 decode_kernel = "tma"     # "tma" | "cp_async" (the fallback kernel; selectable for tests and comparisons)
 
@@ -417,11 +583,11 @@ def paged_attention(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tenso
 
 
 def paged_attention_ext(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tensor, inp, scale: float, window: int = -1, chunk: int = 0,
-                        slopes: Optional[torch.Tensor] = None, sinks: Optional[torch.Tensor] = None) -> torch.Tensor:
+                        slopes: Optional[torch.Tensor] = None, sinks: Optional[torch.Tensor] = None, keep_first: int = 0) -> torch.Tensor:
     """Paged attention with score extensions and a value dimension of its own: q [T, Hq, dk] (may be a view of the qkv
     buffer), caches [blocks, block, Hkv, dk | dv] -> [T, Hq * dv].  score = scale q.k - slopes[h] * distance; keys of the
-    query's own chunk of `chunk` positions only (0: all); exp(sinks[h]) joins the softmax denominator.  bf16 tensors with
-    head dimensions up to 128 (multiples of 8) run on the tensor-core kernels, anything else on the fp32-pipe kernel."""
+    query's own chunk of `chunk` positions only (0: all); `keep_first` first keys stay visible behind the window;
+    exp(sinks[h]) joins the softmax denominator.  bf16 tensors with head dimensions up to 128 (multiples of 8) run on the tensor-core kernels, anything else on the fp32-pipe kernel."""
     global launch_count
     from ..framework.step_input import H_NUM_DECODE, H_NUM_SEQS
     T, Hq, dk = q.shape
@@ -439,7 +605,7 @@ def paged_attention_ext(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.T
         _check(lib().xl_attention_simt(_ptr(q), _ptr(k_cache), _ptr(v_cache), _ptr(out), _ptr(inp.token_seq), _ptr(inp.positions),
                                        _ptr(inp.block_tables), c_int(T), c_int(n_all), c_int(L.MB_cap), c_int(block_size),
                                        c_long(k_cache.shape[0] * block_size), c_int(Hq), c_int(n_kv), c_int(dk), c_int(dv),
-                                       c_long(q_stride), c_float(scale), c_int(window), c_int(chunk), _ptr(slopes), _ptr(sinks),
+                                       c_long(q_stride), c_float(scale), c_int(window), c_int(chunk), c_int(keep_first), _ptr(slopes), _ptr(sinks),
                                        _f32flag(q), _stream()), "xl_attention_simt")
         return out
     if q.dtype == torch.float32 or dk % 8 or dv % 8 or dk > 128 or dv > 128 or q.stride(1) != dk or Hq // n_kv > 16:
@@ -452,14 +618,18 @@ def paged_attention_ext(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.T
     shape = (c_int(L.MB_cap), c_int(block_size), c_int(k_cache.shape[0]), c_int(Hq), c_int(n_kv), c_int(dk), c_int(dv), c_int(q_stride))
     if n_dec > 0:
         max_kv = (L.MB_cap * block_size) if padded else inp.max_kv
-        splits = decode_splits(n_dec, n_kv, min(max_kv, chunk) if chunk > 0 else max_kv)
+        if chunk > 0:
+            max_kv = min(max_kv, chunk)
+        if window > 0:
+            max_kv = min(max_kv, window + keep_first)
+        splits = decode_splits(n_dec, n_kv, max_kv)
         po = pl = None
         rows = max(T, n_dec)
         if splits > 1:
             po = torch.empty((rows, Hq, splits, dv), dtype=torch.float32, device=q.device)
             pl = torch.empty((rows, Hq, splits), dtype=torch.float32, device=q.device)
         rc = lib().xl_decode_attention_ext(*common, c_int(0), c_int(n_dec), *shape, c_float(scale), c_int(window), c_int(chunk),
-                                           _ptr(slopes), _ptr(sinks), c_int(splits), _ptr(po), _ptr(pl), c_long(rows), dyn_dec, _stream())
+                                           c_int(keep_first), _ptr(slopes), _ptr(sinks), c_int(splits), _ptr(po), _ptr(pl), c_long(rows), dyn_dec, _stream())
         if rc == -3:            # a block size outside the tensor-core kernels' limits
             launch_count += 1
             return simt()
@@ -468,7 +638,7 @@ def paged_attention_ext(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.T
     if has_prefill:
         tiles = (T + 127) // 128 + n_all if padded else (inp.n_prefill_tokens + 127) // 128 + (n_all - n_dec)
         rc = lib().xl_prefill_attention_ext(*common, c_int(0 if padded else n_dec), c_int(n_all), *shape, c_int(T), c_float(scale),
-                                            c_int(window), c_int(chunk), _ptr(slopes), _ptr(sinks), c_int(tiles), dyn_dec, dyn_all,
+                                            c_int(window), c_int(chunk), c_int(keep_first), _ptr(slopes), _ptr(sinks), c_int(tiles), dyn_dec, dyn_all,
                                             _stream())
         if rc == -3:
             launch_count += 1

@@ -406,8 +406,10 @@ def replace_norm(y: torch.Tensor, vec: torch.Tensor, x: torch.Tensor, w_next: to
     return _rms_f32(x, w_next, eps).to(w_next.dtype)
 
 
-def split_rows(x: torch.Tensor, x0: torch.Tensor) -> torch.Tensor:
-    """[x, x0] as the input of a product; an fp32 x in a bf16 model enters as its bf16 value and what that leaves."""
+def split_rows(x: torch.Tensor, ids: torch.Tensor, table: torch.Tensor, scale: float) -> torch.Tensor:
+    """[x, x0] as the input of a product, x0 = table[ids] * scale; an fp32 x in a bf16 model enters as its bf16 value and what
+    that leaves."""
+    x0 = (embedding(ids, table).float() * scale).to(table.dtype)
     if x0.dtype == torch.float32:
         return torch.cat([x, x0], -1)
     hi = x.to(x0.dtype)

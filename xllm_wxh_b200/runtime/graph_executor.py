@@ -65,8 +65,9 @@ class CudaGraphExecutor:
             # With collectives that cross the DP groups (expert parallelism under attention DP) every rank must run
             # each layer's exchange exactly once per step, whatever its own shape: the extra eager run that `_capture`
             # makes for lazy initialisation would leave this rank one exchange ahead of its peers.  The first step of
-            # each kind therefore runs eagerly as the step itself.
-            first_of_kind = self._cross_dp() and bool(inp.has_prefill) not in self.warmed
+            # each kind therefore runs eagerly as the step itself.  So does it with recurrent state, which a second run of
+            # the same step would move on twice (writing the same KV rows twice is harmless).
+            first_of_kind = (self._cross_dp() or len(inp.states) > 0) and bool(inp.has_prefill) not in self.warmed
             if (inp.has_prefill and seen < self.capture_after) or first_of_kind:
                 w = self.worker
                 self.num_eager_padded += 1
