@@ -855,6 +855,18 @@ class Scheduler {
     return true;
   }
 
+  // Whether sequences of other requests hold blocks or state slots.  Under schedule overlap that includes sequences which have
+  // left the queues but whose last step is still in flight: what they hold comes back, so a request must wait for it.
+  bool held_by_others(const Request* r, int rank) const {
+    int blocks = 0, slots = 0;
+    for (auto& s : r->seqs) {
+      blocks += static_cast<int>(s->blocks.size());
+      slots += s->state_slot != 0;
+    }
+    return pool_.at(rank).num_used_blocks() > blocks ||
+           (!slots_.empty() && slots_[rank].num_slots() - slots_[rank].num_free() > slots);
+  }
+
   void preempt(Request* r) {
     for (auto& s : r->seqs) {
       if (s->finished) continue;
@@ -962,7 +974,7 @@ class Scheduler {
       }
       if (!ok) {
         undo_match(s);
-        if (alone && !any && !pins_outstanding()) {
+        if (alone && !any && !pins_outstanding() && !held_by_others(r, rank)) {
           // nothing else holds memory: the request can never fit
           finish_sequence(s, FinishReason::RESOURCE_EXHAUSTED);
           emit(s);
@@ -1066,7 +1078,7 @@ class Scheduler {
           if (!in_current(r)) {
             if (running_.size() == 1 && !has_any_entry(bs)) {
               // alone: either it can never fit, or blocks held for copies in flight come back within two steps
-              if (!pins_outstanding()) {
+              if (!pins_outstanding() && !held_by_others(r, rank)) {
                 finish_sequence(s, FinishReason::RESOURCE_EXHAUSTED);
                 emit(s);
               }
@@ -1307,7 +1319,7 @@ class Scheduler {
           }
         }
         if (!ok) {
-          if (!any && !has_any_entry(bs) && !pins_outstanding()) {
+          if (!any && !has_any_entry(bs) && !pins_outstanding() && !held_by_others(r, rank)) {
             // nothing else holds memory: the request can never fit
             finish_sequence(s, FinishReason::RESOURCE_EXHAUSTED);
             emit(s);
