@@ -169,7 +169,7 @@ def test_conv(cuts, taps):
     x, w, b = [torch.randn(n, C, generator=g) for n in RAG], torch.randn(C, taps, generator=g), torch.randn(C, generator=g)
     state = torch.full((6, taps - 1, C), 1e3)
     for q, kv, sl, n, rows in Ragged().steps(RAG, cuts):
-        got = ops.ref.conv_silu(rag(x, rows), w, b, state, q, kv, sl, n)
+        got = ops.ref.conv_silu(rag(x, rows), w.t(), b, state, q, kv, sl, n)
         assert torch.allclose(got, rag([O.silu(O.causal_conv(s, w, b)) for s in x], rows), atol=1e-5)
 
 

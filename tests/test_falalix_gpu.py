@@ -129,7 +129,7 @@ def test_conv(C, taps, dtype, steps, pad):
     rg = ragged(steps, pad)
     state = torch.full((rg.n_slots, taps - 1, C), 1e4, dtype=dtype, device=DEV)
     for inp, rows in rg:
-        got = ops.conv_silu(rg.take(x, rows)[:, :C], w.to(DEV), b.to(DEV), state, inp)
+        got = ops.conv_silu(rg.take(x, rows)[:, :C], w.t().contiguous().to(DEV), b.to(DEV), state, inp)
         n = sum(q - p for _, p, q in rows)
         assert rel(got[:n], torch.cat([want[i][p:q] for i, p, q in rows])) < (4e-3 if dtype == torch.bfloat16 else 2e-6)
         assert got[n:].abs().sum() == 0

@@ -64,6 +64,33 @@ __device__ __forceinline__ void store_n(T* p, const float (&f)[V]) {
   else from_f32(p, f[0]);
 }
 
+// Eight elements as they come from memory, converted when they are used.
+template <typename T> struct Vec8;
+template <> struct Vec8<__nv_bfloat16> {
+  uint4 v;
+  __device__ __forceinline__ void load(const __nv_bfloat16* p) { v = *reinterpret_cast<const uint4*>(p); }
+  __device__ __forceinline__ void get(float (&f)[8]) const {
+    const uint32_t u[4] = {v.x, v.y, v.z, v.w};
+#pragma unroll
+    for (int j = 0; j < 4; ++j) {
+      const float2 t = unpack_bf16x2(u[j]);
+      f[2 * j] = t.x;
+      f[2 * j + 1] = t.y;
+    }
+  }
+};
+template <> struct Vec8<float> {
+  float4 a, b;
+  __device__ __forceinline__ void load(const float* p) {
+    a = reinterpret_cast<const float4*>(p)[0];
+    b = reinterpret_cast<const float4*>(p)[1];
+  }
+  __device__ __forceinline__ void get(float (&f)[8]) const {
+    f[0] = a.x; f[1] = a.y; f[2] = a.z; f[3] = a.w;
+    f[4] = b.x; f[5] = b.y; f[6] = b.z; f[7] = b.w;
+  }
+};
+
 // ============================================================================ token shift
 template <typename T, int V>
 __global__ void __launch_bounds__(256) token_shift_kernel(const T* __restrict__ h, const T* __restrict__ mu, T* __restrict__ last,
@@ -102,9 +129,9 @@ __global__ void __launch_bounds__(256) token_shift_kernel(const T* __restrict__ 
 // ============================================================================ causal convolution + silu
 // A thread owns V channels of a tile of consecutive rows and keeps the last TAPS - 1 inputs in registers (TAPS = 0: any
 // number of taps, inputs read again for every row).
-constexpr int kConvRows = 16;
+constexpr int kConvRows = 16, kConvRowsSingle = 2;
 
-template <typename T, int V, int TAPS>
+template <typename T, int V, int TAPS, int ROWS>
 __global__ void __launch_bounds__(128) conv_silu_kernel(const T* __restrict__ x, const T* __restrict__ w, const T* __restrict__ bias,
                                                         T* __restrict__ state, T* __restrict__ out, const int* __restrict__ token_seq,
                                                         const Seqs q, int rows, int C, int taps_rt, long ldx) {
@@ -112,19 +139,28 @@ __global__ void __launch_bounds__(128) conv_silu_kernel(const T* __restrict__ x,
   const int taps = TAPS > 0 ? TAPS : taps_rt;
   const int c = (blockIdx.y * blockDim.x + threadIdx.x) * V;
   if (c >= C) return;
-  const int t0 = blockIdx.x * kConvRows, t1 = min(rows, t0 + kConvRows);
+  const int t0 = blockIdx.x * ROWS, t1 = min(rows, t0 + ROWS);
   float b[V], wt[TAPS > 0 ? TAPS : 1][V], hist[H][V];
   load_n<V>(bias + c, b);
   if (TAPS > 0) {
 #pragma unroll
-    for (int i = 0; i < TAPS; ++i)
-#pragma unroll
-      for (int e = 0; e < V; ++e) wt[i][e] = to_f32(w[size_t(c + e) * TAPS + i]);
+    for (int i = 0; i < TAPS; ++i) load_n<V>(w + size_t(i) * C + c, wt[i]);
   }
   int cur_seq = -1, start = 0, end = 0, slot = 0;
   bool cont = false;
-  for (int t = t0; t < t1; ++t) {
-    const int seq = token_seq[t];
+  constexpr int AHEAD = ROWS < 4 ? ROWS : 4;             // rows requested together
+  float ahead[AHEAD][V];
+  int seqs[AHEAD];
+#pragma unroll 1
+  for (int tg = t0; tg < t1; tg += AHEAD) {
+#pragma unroll
+  for (int r = 0; r < AHEAD; ++r) {
+    seqs[r] = tg + r < t1 ? token_seq[tg + r] : -1;
+    if (tg + r < t1) load_n<V>(x + size_t(tg + r) * ldx + c, ahead[r]);
+  }
+#pragma unroll
+  for (int r = 0; r < AHEAD; ++r) {
+    const int t = tg + r, seq = seqs[r];
     if (seq < 0 || seq >= q.n) continue;
     const bool fresh = seq != cur_seq;
     if (fresh) {
@@ -143,8 +179,8 @@ __global__ void __launch_bounds__(128) conv_silu_kernel(const T* __restrict__ x,
       if (j >= 0) load_n<V>(x + size_t(t - back) * ldx + c, f);
       else if (cont) load_n<V>(state + (size_t(slot) * (taps - 1) + (taps - 1 + j)) * C + c, f);
     };
-    float y[V], cur[V];
-    load_n<V>(x + size_t(t) * ldx + c, cur);
+    float y[V];
+    const float(&cur)[V] = ahead[r];
 #pragma unroll
     for (int e = 0; e < V; ++e) y[e] = b[e];
     if (TAPS > 0) {
@@ -167,7 +203,7 @@ __global__ void __launch_bounds__(128) conv_silu_kernel(const T* __restrict__ x,
         for (int e = 0; e < V; ++e) hist[H - 1][e] = cur[e];
         if (end - start == 1) {                    // a single row: this thread alone reads and writes this part of the record
 #pragma unroll
-          for (int i = 0; i < TAPS - 1; ++i) store_n<V>(state + (size_t(slot) * (TAPS - 1) + i) * C + c, hist[i]);
+          for (int i = 0; i < TAPS - 1; ++i) store_n<V>(state + (size_t(slot) * H + i) * C + c, hist[i]);
         }
       }
     } else {
@@ -175,7 +211,7 @@ __global__ void __launch_bounds__(128) conv_silu_kernel(const T* __restrict__ x,
         float f[V];
         before(taps - 1 - i, f);
 #pragma unroll
-        for (int e = 0; e < V; ++e) y[e] = fmaf(f[e], to_f32(w[size_t(c + e) * taps + i]), y[e]);
+        for (int e = 0; e < V; ++e) y[e] = fmaf(f[e], to_f32(w[size_t(i) * C + c + e]), y[e]);
       }
       if (end - start == 1) {
         for (int i = 0; i < taps - 1; ++i) {
@@ -188,6 +224,7 @@ __global__ void __launch_bounds__(128) conv_silu_kernel(const T* __restrict__ x,
 #pragma unroll
     for (int e = 0; e < V; ++e) y[e] = act_silu(y[e]);
     store_n<V>(out + size_t(t) * C + c, y);
+  }
   }
 }
 
@@ -284,7 +321,7 @@ __device__ __forceinline__ uint64_t mul2(uint64_t a, uint64_t b) {
 // One (segment, head) per CTA.  D: head dimension padded to 32, 64 or 128.  Thread (kg, vg) owns keys kg * KT ..., values
 // vg * 4 ... of the head's matrix, as pairs of neighbouring keys.
 template <int D> struct MixCfg {
-  static constexpr int KT = D == 32 ? 8 : 16;
+  static constexpr int KT = D == 128 ? 16 : 8;
   static constexpr int KG = D / KT, VG = D / 4, kThreads = KG * VG;
   static constexpr int SEG = KT + 4, ROW = KG * SEG;      // key groups 4 floats apart, so that their reads meet no bank twice
 };
@@ -349,23 +386,44 @@ __global__ void __launch_bounds__(MixCfg<D>::kThreads) time_mix_segment_kernel(c
 #pragma unroll
     for (int i = 0; i < D / 32; ++i) nw[i] = lane + 32 * i < d ? to_f32(p.norm_w[h * d + lane + 32 * i]) * p.scale : 0.f;
   }
+  // rows of this head on their way: vector i * NT + tid of the [row][8 columns] tile (v8 only)
+  constexpr int NV = kMixRows * (D / 8) / NT;
+  Vec8<T> fk[NV], fv[NV], fr[OUT ? NV : 1];
+  Vec8<float> fz[NV];
+  auto fetch = [&](int b) {
+    const int m = min(kMixRows, n - b);
+#pragma unroll
+    for (int i = 0; i < NV; ++i) {
+      const int e = i * NT + tid, row = e / (D / 8), c = e % (D / 8) * 8;
+      if (row < m && c < d) {
+        const size_t t = size_t(t0 + b + row), at = t * p.ld + size_t(h) * d + c;
+        fk[i].load(p.k + at);
+        fv[i].load(p.v + at);
+        if (OUT) fr[OUT ? i : 0].load(p.r + at);
+        fz[i].load(p.z + t * (size_t(p.H) * d) + size_t(h) * d + c);
+      }
+    }
+  };
+  if (v8) fetch(0);
   for (int b = 0; b < n; b += kMixRows) {
     const int m = min(kMixRows, n - b);
-    // stage m rows of this head
+    // stage the rows; those beyond m leave the state as it is (decay 1, key 0)
     if (v8) {
-      for (int i = tid; i < kMixRows * (D / 8); i += NT) {
-        const int row = i / (D / 8), c = i % (D / 8) * 8;
-        float k[8] = {}, v[8] = {}, w[8] = {}, r[8] = {};
+#pragma unroll
+      for (int i = 0; i < NV; ++i) {
+        const int e = i * NT + tid, row = e / (D / 8), c = e % (D / 8) * 8;
+        float k[8] = {}, v[8] = {}, r[8] = {}, w[8];
+#pragma unroll
+        for (int j = 0; j < 8; ++j) w[j] = 1.f;
         if (row < m && c < d) {
-          const size_t t = size_t(t0 + b + row), at = t * p.ld + size_t(h) * d + c;
-          load8(p.k + at, k);
-          load8(p.v + at, v);
-          if (OUT) load8(p.r + at, r);
+          fk[i].get(k);
+          fv[i].get(v);
+          if (OUT) fr[OUT ? i : 0].get(r);
           float w0[8];
-          load8(p.z + t * (size_t(p.H) * d) + size_t(h) * d + c, w);
+          fz[i].get(w);
           load8(p.w0 + h * d + c, w0);
 #pragma unroll
-          for (int e = 0; e < 8; ++e) w[e] = decay_of<T>(w[e] + w0[e]);
+          for (int j = 0; j < 8; ++j) w[j] = decay_of<T>(w[j] + w0[j]);
         }
         const int at = c / KT * SEG + c % KT;
         store8(&sK[row][at], k);
@@ -381,11 +439,12 @@ __global__ void __launch_bounds__(MixCfg<D>::kThreads) time_mix_segment_kernel(c
         const int to = c / KT * SEG + c % KT;
         sK[row][to] = in ? to_f32(p.k[at]) : 0.f;
         sV[row][c] = in ? to_f32(p.v[at]) : 0.f;
-        sW[row][to] = in ? decay_of<T>(p.z[t * (size_t(p.H) * d) + size_t(h) * d + c] + p.w0[h * d + c]) : 0.f;
+        sW[row][to] = in ? decay_of<T>(p.z[t * (size_t(p.H) * d) + size_t(h) * d + c] + p.w0[h * d + c]) : 1.f;
         if (OUT) sR[row][to] = in ? to_f32(p.r[at]) : 0.f;
       }
     }
     __syncthreads();
+    if (v8 && b + kMixRows < n) fetch(b + kMixRows);
     if (OUT) {
       for (int row = warp; row < m; row += NT / 32) {
         float s = 0.f;
@@ -395,13 +454,13 @@ __global__ void __launch_bounds__(MixCfg<D>::kThreads) time_mix_segment_kernel(c
           if (c < d) s += sR[row][at] * p.u[h * d + c] * sK[row][at];
         }
         s = warp_sum(s);
-        if (lane == 0) sBonus[row] = s;
+        if (lane == 0) sBonus[row] = s;                    // read behind the next barrier
       }
-      __syncthreads();
     } else if (tid < D) {
       for (int row = 0; row < m; ++row) prod *= sW[row][tid / KT * SEG + tid % KT];
     }
-    for (int row = 0; row < m; ++row) {
+#pragma unroll 2
+    for (int row = 0; row < kMixRows; ++row) {
       const float4 v4 = *reinterpret_cast<const float4*>(&sV[row][vg * 4]);
       const uint64_t v[4] = {pack2(v4.x, v4.x), pack2(v4.y, v4.y), pack2(v4.z, v4.z), pack2(v4.w, v4.w)};
       uint64_t o[4] = {0, 0, 0, 0};
@@ -752,213 +811,287 @@ __device__ __forceinline__ void store_states(float* p, int n0, int N, const floa
   }
 }
 
-// Longer portions: a CTA walks one sequence for kScanThreads / LPC channels, kScanRows rows at a time; the next rows' inputs
-// are fetched into registers while the current ones are worked on.
+// Sums y[0 .. LPC) over the LPC lanes of a channel; lane l ends with the sum of y[l].  Halves the number of values with
+// every exchange.
+template <int LPC>
+__device__ __forceinline__ float sum_to_lanes(float (&y)[LPC], int ln) {
+#pragma unroll
+  for (int o = LPC / 2; o > 0; o >>= 1) {
+    const bool up = ln & o;
+#pragma unroll
+    for (int i = 0; i < o; ++i) {
+      const float send = up ? y[i] : y[i + o];
+      y[i] = (up ? y[i + o] : y[i]) + __shfl_xor_sync(0xffffffffu, send, o);
+    }
+  }
+  return y[0];
+}
+
+// Longer portions: a CTA walks one sequence for kScanThreads / LPC channels.  The lanes of a channel share its rows: lane l
+// fetches, prepares (step size, silu(z)) and finishes rows l, l + LPC, ...; step sizes and inputs reach the other lanes by
+// shuffles.  The inputs of the next kScanRows rows are under way while the current ones are worked on.
 template <typename T, int NPT, int LPC>
 __global__ void __launch_bounds__(kScanThreads) scan_rows_kernel(const ScanParams<T> p) {
   constexpr int CPB = kScanThreads / LPC, NP = NPT * LPC;
-  constexpr int NX = (kScanRows * CPB + kScanThreads - 1) / kScanThreads;       // per-channel inputs per thread
-  constexpr int NB = kScanRows * 2 * NP / kScanThreads;                         // B and C values per thread (a multiple)
-  constexpr bool kAheadB = NB <= 32 && NB > 0;
-  __shared__ __align__(16) float sBC[kScanRows][2 * NP];
-  __shared__ float sDt[kScanRows][CPB], sDx[kScanRows][CPB], sY[kScanRows][CPB];
+  constexpr int G = kScanRows / LPC;                                            // rows per lane and tile
+  constexpr int NB = kScanRows * 2 * NP / kScanThreads;                         // B and C values per thread and tile
+  constexpr bool kAheadB = NB >= 1 && NB <= 16;
+  constexpr int NBUF = NP > 128 ? 1 : 2;
+  __shared__ __align__(16) float sBC[NBUF][kScanRows][2 * NP];
   const int seq = blockIdx.y, tid = threadIdx.x;
   const int start = p.q.q_cu[seq], len = p.q.q_cu[seq + 1] - start;
   if (len < 2) return;
   const int slot = record_of(p.q, seq);
   if (slot < 0) return;
   const bool cont = p.q.kv_lens[seq] > len;
-  const int c0 = blockIdx.x * CPB, ch = tid / LPC, ln = tid % LPC, n0 = ln * NPT;
-  const int c = c0 + ch;
+  const int ch = tid / LPC, ln = tid % LPC, n0 = ln * NPT;
+  const int c = blockIdx.x * CPB + ch;
   const bool live = c < p.C;
-  float S[NPT], A2[NPT];
+  float S[NPT], A[NPT], bias = 0.f, D = 0.f;
 #pragma unroll
-  for (int i = 0; i < NPT; ++i) S[i] = A2[i] = 0.f;
+  for (int i = 0; i < NPT; ++i) S[i] = A[i] = 0.f;
   float* rec = p.state + (size_t(slot) * p.C + c) * p.N;
   if (live) {
-    load_states<NPT>(p.A + size_t(c) * p.N, n0, p.N, A2);
+    load_states<NPT>(p.A + size_t(c) * p.N, n0, p.N, A);
     if (cont) load_states<NPT>(rec, n0, p.N, S);
 #pragma unroll
-    for (int i = 0; i < NPT; ++i) A2[i] *= scan_unit<T>();
+    for (int i = 0; i < NPT; ++i) A[i] *= scan_unit<T>();
+    bias = p.dt_bias[c];
+    D = p.D[c];
   }
-  // inputs of the channel part: element i * kScanThreads + tid of the [row][channel] tile
-  float rdt[NX], rx[NX], rz[NX], rb[kAheadB ? NB : 1];
+  float rdt[G];
+  T rx[G], rz[G], rb[kAheadB ? NB : 1];
+  const T zero = T(0.f);
   auto fetch = [&](int b) {
     const int m = min(kScanRows, len - b);
 #pragma unroll
-    for (int i = 0; i < NX; ++i) {
-      const int e = i * kScanThreads + tid, row = e / CPB, cc = c0 + e % CPB;
-      rdt[i] = rx[i] = rz[i] = 0.f;
-      if (row < m && cc < p.C) {
+    for (int g = 0; g < G; ++g) {
+      const int row = g * LPC + ln;
+      rdt[g] = 0.f;
+      rx[g] = rz[g] = zero;
+      if (row < m && live) {
         const size_t t = size_t(start + b + row);
-        rdt[i] = p.dt[t * p.C + cc];
-        rx[i] = to_f32(p.x[t * p.C + cc]);
-        rz[i] = to_f32(p.z[t * p.ldz + cc]);
+        rdt[g] = p.dt[t * p.C + c];
+        rx[g] = p.x[t * p.C + c];
+        rz[g] = p.z[t * p.ldz + c];
       }
     }
     if (kAheadB) {
 #pragma unroll
       for (int i = 0; i < NB; ++i) {
         const int e = i * kScanThreads + tid, row = e / (2 * NP), n = e % (2 * NP), nn = n < NP ? n : n - NP;
-        rb[kAheadB ? i : 0] = 0.f;
-        if (row < m && nn < p.N) rb[kAheadB ? i : 0] = to_f32((n < NP ? p.B : p.Cm)[size_t(start + b + row) * p.ldb + nn]);
+        rb[kAheadB ? i : 0] = zero;
+        if (row < m && nn < p.N) rb[kAheadB ? i : 0] = (n < NP ? p.B : p.Cm)[size_t(start + b + row) * p.ldb + nn];
+      }
+    }
+  };
+  auto put = [&](int b, int buf) {
+    if (kAheadB) {
+#pragma unroll
+      for (int i = 0; i < NB; ++i) (&sBC[buf][0][0])[i * kScanThreads + tid] = to_f32(rb[kAheadB ? i : 0]);
+    } else {
+      const int m = min(kScanRows, len - b);
+      for (int e = tid; e < kScanRows * 2 * NP; e += kScanThreads) {
+        const int row = e / (2 * NP), n = e % (2 * NP), nn = n < NP ? n : n - NP;
+        (&sBC[buf][0][0])[e] = row < m && nn < p.N ? to_f32((n < NP ? p.B : p.Cm)[size_t(start + b + row) * p.ldb + nn]) : 0.f;
       }
     }
   };
   fetch(0);
-  for (int b = 0; b < len; b += kScanRows) {
+  put(0, 0);
+  int buf = 0;
+  for (int b = 0; b < len; b += kScanRows, buf ^= NBUF - 1) {
     const int m = min(kScanRows, len - b);
-    float x[NX], z[NX];
+    float dt[G], x[G], z[G];
 #pragma unroll
-    for (int i = 0; i < NX; ++i) {
-      const int e = i * kScanThreads + tid, row = e / CPB, cc = e % CPB;
-      x[i] = rx[i];
-      z[i] = rz[i];
-      if (row < kScanRows) {
-        const float dt = c0 + cc < p.C ? softplus(rdt[i] + p.dt_bias[c0 + cc]) : 0.f;
-        sDt[row][cc] = dt;
-        sDx[row][cc] = dt * x[i];
-      }
-    }
-    if (kAheadB) {
-#pragma unroll
-      for (int i = 0; i < NB; ++i) {
-        const int e = i * kScanThreads + tid;
-        (&sBC[0][0])[e] = rb[kAheadB ? i : 0];
-      }
-    } else {
-      for (int e = tid; e < kScanRows * 2 * NP; e += kScanThreads) {
-        const int row = e / (2 * NP), n = e % (2 * NP), nn = n < NP ? n : n - NP;
-        (&sBC[0][0])[e] = row < m && nn < p.N ? to_f32((n < NP ? p.B : p.Cm)[size_t(start + b + row) * p.ldb + nn]) : 0.f;
-      }
+    for (int g = 0; g < G; ++g) {                          // rows beyond m: a step of size 0 leaves the state as it is
+      dt[g] = g * LPC + ln < m ? softplus(rdt[g] + bias) : 0.f;
+      x[g] = to_f32(rx[g]);
+      z[g] = to_f32(rz[g]);
     }
     __syncthreads();
     if (b + kScanRows < len) fetch(b + kScanRows);
-    // rows in groups of four, so that their exponentials overlap and the sums over a channel's lanes share their shuffles;
-    // rows beyond m hold dt = 0: they leave the state as it is
-#pragma unroll 1
-    for (int g = 0; g < kScanRows; g += 4) {
-      if (g >= m) break;
-      float y[4];
 #pragma unroll
-      for (int r = 0; r < 4; ++r) {
-        const bool in = g + r < m;
-        const float dt = in ? sDt[g + r][ch] : 0.f, dx = in ? sDx[g + r][ch] : 0.f;
-        float acc = 0.f;
+    for (int g = 0; g < G; ++g) {
+      const float dx = dt[g] * x[g];
+      float y[LPC];
+#pragma unroll
+      for (int l = 0; l < LPC; ++l) {
+        const float dtl = LPC == 1 ? dt[g] : __shfl_sync(0xffffffffu, dt[g], l, LPC);
+        const float dxl = LPC == 1 ? dx : __shfl_sync(0xffffffffu, dx, l, LPC);
+        const float* bc = &sBC[buf][g * LPC + l][n0];
+        float acc[4] = {0.f, 0.f, 0.f, 0.f};
 #pragma unroll
         for (int i = 0; i < NPT; i += 4) {
-          const float4 bb = *reinterpret_cast<const float4*>(&sBC[g + r][n0 + i]);
-          const float4 cm = *reinterpret_cast<const float4*>(&sBC[g + r][NP + n0 + i]);
-          S[i] = fmaf(scan_decay<T>(dt * A2[i]), S[i], dx * bb.x);
-          S[i + 1] = fmaf(scan_decay<T>(dt * A2[i + 1]), S[i + 1], dx * bb.y);
-          S[i + 2] = fmaf(scan_decay<T>(dt * A2[i + 2]), S[i + 2], dx * bb.z);
-          S[i + 3] = fmaf(scan_decay<T>(dt * A2[i + 3]), S[i + 3], dx * bb.w);
-          acc = fmaf(S[i], cm.x, fmaf(S[i + 1], cm.y, fmaf(S[i + 2], cm.z, fmaf(S[i + 3], cm.w, acc))));
+          const float4 bb = *reinterpret_cast<const float4*>(bc + i);
+          const float4 cm = *reinterpret_cast<const float4*>(bc + NP + i);
+          S[i] = fmaf(scan_decay<T>(dtl * A[i]), S[i], dxl * bb.x);
+          S[i + 1] = fmaf(scan_decay<T>(dtl * A[i + 1]), S[i + 1], dxl * bb.y);
+          S[i + 2] = fmaf(scan_decay<T>(dtl * A[i + 2]), S[i + 2], dxl * bb.z);
+          S[i + 3] = fmaf(scan_decay<T>(dtl * A[i + 3]), S[i + 3], dxl * bb.w);
+          acc[0] = fmaf(S[i], cm.x, acc[0]);
+          acc[1] = fmaf(S[i + 1], cm.y, acc[1]);
+          acc[2] = fmaf(S[i + 2], cm.z, acc[2]);
+          acc[3] = fmaf(S[i + 3], cm.w, acc[3]);
         }
-        y[r] = acc;
+        y[l] = (acc[0] + acc[1]) + (acc[2] + acc[3]);
       }
-      if constexpr (LPC >= 4) {
-        const bool b0 = ln & 1, b1 = ln & 2;
-        float a0 = b0 ? y[2] : y[0], a1 = b0 ? y[3] : y[1];
-        a0 += __shfl_xor_sync(0xffffffffu, b0 ? y[0] : y[2], 1);
-        a1 += __shfl_xor_sync(0xffffffffu, b0 ? y[1] : y[3], 1);
-        float a = b1 ? a1 : a0;
-        a += __shfl_xor_sync(0xffffffffu, b1 ? a0 : a1, 2);
-#pragma unroll
-        for (int o = 4; o < LPC; o <<= 1) a += __shfl_xor_sync(0xffffffffu, a, o);
-        if (ln < 4) sY[g + (b0 ? 2 : 0) + (b1 ? 1 : 0)][ch] = a;
-      } else {
-#pragma unroll
-        for (int r = 0; r < 4; ++r) {
-          if (LPC == 2) y[r] += __shfl_xor_sync(0xffffffffu, y[r], 1);
-          if (ln == 0) sY[g + r][ch] = y[r];
-        }
-      }
+      const float sum = sum_to_lanes<LPC>(y, ln);
+      const int row = g * LPC + ln;
+      if (row < m && live) from_f32(p.out + size_t(start + b + row) * p.C + c, fmaf(D, x[g], sum) * act_silu(z[g]));
     }
-    __syncthreads();
-#pragma unroll
-    for (int i = 0; i < NX; ++i) {
-      const int e = i * kScanThreads + tid, row = e / CPB, cc = e % CPB;
-      if (row < m && c0 + cc < p.C)
-        from_f32(p.out + size_t(start + b + row) * p.C + c0 + cc, fmaf(p.D[c0 + cc], x[i], sY[row][cc]) * act_silu(z[i]));
-    }
-    __syncthreads();
+    if (NBUF == 1) __syncthreads();
+    if (b + kScanRows < len) put(b + kScanRows, buf ^ (NBUF - 1));
   }
   if (live) store_states<NPT>(rec, n0, p.N, S);
 }
 
-// Single rows: kScanIter groups of channels per CTA, all their states requested before any is worked on.
-constexpr int kScanIter = 4;
+// Single rows: LPC lanes per channel, NPT states each, and kScanSeqs sequences per thread, so that A is read once for them and
+// the states of all of them are under way before any is worked on.  bc4: B and C can be read four at a time.
+constexpr int kScanSeqs = 4;
+template <typename T>
+__device__ __forceinline__ void load_bc4(const T* p, float* f) {
+  if constexpr (sizeof(T) == 2) {
+    const uint2 u = *reinterpret_cast<const uint2*>(p);
+    const float2 a = unpack_bf16x2(u.x), b = unpack_bf16x2(u.y);
+    f[0] = a.x; f[1] = a.y; f[2] = b.x; f[3] = b.y;
+  } else {
+    *reinterpret_cast<float4*>(f) = *reinterpret_cast<const float4*>(p);
+  }
+}
 template <typename T, int NPT, int LPC>
-__global__ void __launch_bounds__(kScanThreads) scan_single_kernel(const ScanParams<T> p) {
+__global__ void __launch_bounds__(kScanThreads) scan_single_kernel(const ScanParams<T> p, int bc4) {
   constexpr int CPB = kScanThreads / LPC;
-  constexpr int IT = NPT > 4 ? 1 : kScanIter;
-  const int seq = blockIdx.y, tid = threadIdx.x;
-  const int t = p.q.q_cu[seq];
-  if (p.q.q_cu[seq + 1] - t != 1) return;
-  const int slot = record_of(p.q, seq);
-  if (slot < 0) return;
-  const bool cont = p.q.kv_lens[seq] > 1;
-  const int ch = tid / LPC, ln = tid % LPC, n0 = ln * NPT;
-  float S[IT][NPT], A[IT][NPT], dt[IT], x[IT], B[NPT], Cm[NPT];
+  constexpr int NS = NPT > 4 ? 1 : kScanSeqs;
+  const int tid = threadIdx.x, ch = tid / LPC, ln = tid % LPC, n0 = ln * NPT;
+  const int c = blockIdx.x * CPB + ch;
+  const bool live = c < p.C;
+  int t[NS], slot[NS];
+  bool cont[NS], any = false;
 #pragma unroll
-  for (int k = 0; k < IT; ++k) {
-    const int c = (blockIdx.x * IT + k) * CPB + ch;
+  for (int k = 0; k < NS; ++k) {
+    const int seq = blockIdx.y * NS + k;
+    t[k] = seq < p.q.n ? p.q.q_cu[seq] : 0;
+    slot[k] = -1;
+    cont[k] = false;
+    if (seq < p.q.n && p.q.q_cu[seq + 1] - t[k] == 1) {
+      slot[k] = record_of(p.q, seq);
+      cont[k] = p.q.kv_lens[seq] > 1;
+    }
+    any |= slot[k] >= 0;
+  }
+  if (!any) return;
+  float S[NS][NPT], A[NPT], dt[NS], x[NS], bias = 0.f, D = 0.f;
+#pragma unroll
+  for (int k = 0; k < NS; ++k) {
     dt[k] = x[k] = 0.f;
 #pragma unroll
-    for (int i = 0; i < NPT; ++i) S[k][i] = A[k][i] = 0.f;
-    if (c < p.C) {
-      if (cont) load_states<NPT>(p.state + (size_t(slot) * p.C + c) * p.N, n0, p.N, S[k]);
-      load_states<NPT>(p.A + size_t(c) * p.N, n0, p.N, A[k]);
-      dt[k] = p.dt[size_t(t) * p.C + c] + p.dt_bias[c];
-      x[k] = to_f32(p.x[size_t(t) * p.C + c]);
+    for (int i = 0; i < NPT; ++i) S[k][i] = 0.f;
+    if (live && slot[k] >= 0) {
+      if (cont[k]) load_states<NPT>(p.state + (size_t(slot[k]) * p.C + c) * p.N, n0, p.N, S[k]);
+      dt[k] = p.dt[size_t(t[k]) * p.C + c];
+      x[k] = to_f32(p.x[size_t(t[k]) * p.C + c]);
     }
   }
 #pragma unroll
-  for (int i = 0; i < NPT; ++i) {
-    const bool in = n0 + i < p.N;
-    B[i] = in ? to_f32(p.B[size_t(t) * p.ldb + n0 + i]) : 0.f;
-    Cm[i] = in ? to_f32(p.Cm[size_t(t) * p.ldb + n0 + i]) : 0.f;
+  for (int i = 0; i < NPT; ++i) A[i] = 0.f;
+  if (live) {
+    load_states<NPT>(p.A + size_t(c) * p.N, n0, p.N, A);
+    bias = p.dt_bias[c];
+    D = p.D[c];
   }
+  float y[NS];
 #pragma unroll
-  for (int k = 0; k < IT; ++k) {
-    const int c = (blockIdx.x * IT + k) * CPB + ch;
-    const float step = softplus(dt[k]), dx = step * x[k];
-    float y = 0.f;
+  for (int k = 0; k < NS; ++k) {
+    y[k] = 0.f;
+    if (slot[k] < 0) continue;                             // the same in every lane
+    float B[NPT], Cm[NPT];
+    const T *bp = p.B + size_t(t[k]) * p.ldb + n0, *cp = p.Cm + size_t(t[k]) * p.ldb + n0;
+#pragma unroll
+    for (int i = 0; i < NPT; i += 4) {
+      if (bc4) {
+#pragma unroll
+        for (int e = 0; e < 4; ++e) B[i + e] = Cm[i + e] = 0.f;
+        if (n0 + i < p.N) {
+          load_bc4(bp + i, B + i);
+          load_bc4(cp + i, Cm + i);
+        }
+      } else {
+#pragma unroll
+        for (int e = 0; e < 4; ++e) {
+          const bool in = n0 + i + e < p.N;
+          B[i + e] = in ? to_f32(bp[i + e]) : 0.f;
+          Cm[i + e] = in ? to_f32(cp[i + e]) : 0.f;
+        }
+      }
+    }
+    const float step = softplus(dt[k] + bias), dx = step * x[k];
 #pragma unroll
     for (int i = 0; i < NPT; ++i) {
-      S[k][i] = fmaf(scan_decay<T>(step * (A[k][i] * scan_unit<T>())), S[k][i], dx * B[i]);
-      y = fmaf(S[k][i], Cm[i], y);
+      S[k][i] = fmaf(scan_decay<T>(step * (A[i] * scan_unit<T>())), S[k][i], dx * B[i]);
+      y[k] = fmaf(S[k][i], Cm[i], y[k]);
     }
+    if (live) store_states<NPT>(p.state + (size_t(slot[k]) * p.C + c) * p.N, n0, p.N, S[k]);
+  }
+  if constexpr (NS == LPC) {                               // lane k finishes sequence k
+    const float xs[4] = {x[0], x[NS > 1 ? 1 : 0], x[NS > 2 ? 2 : 0], x[NS > 3 ? 3 : 0]};
+    const float sum = sum_to_lanes<NS>(y, ln);
+    int tk = t[0], sk = slot[0];
+    float xk = xs[0];
 #pragma unroll
-    for (int o = 1; o < LPC; o <<= 1) y += __shfl_xor_sync(0xffffffffu, y, o);
-    if (c < p.C) {
-      store_states<NPT>(p.state + (size_t(slot) * p.C + c) * p.N, n0, p.N, S[k]);
-      if (ln == 0)
-        from_f32(p.out + size_t(t) * p.C + c, fmaf(p.D[c], x[k], y) * act_silu(to_f32(p.z[size_t(t) * p.ldz + c])));
+    for (int k = 1; k < NS; ++k)
+      if (ln == k) { tk = t[k]; sk = slot[k]; xk = xs[k]; }
+    if (live && sk >= 0)
+      from_f32(p.out + size_t(tk) * p.C + c, fmaf(D, xk, sum) * act_silu(to_f32(p.z[size_t(tk) * p.ldz + c])));
+  } else {
+#pragma unroll
+    for (int k = 0; k < NS; ++k) {
+#pragma unroll
+      for (int o = 1; o < LPC; o <<= 1) y[k] += __shfl_xor_sync(0xffffffffu, y[k], o);
+      if (live && ln == 0 && slot[k] >= 0)
+        from_f32(p.out + size_t(t[k]) * p.C + c, fmaf(D, x[k], y[k]) * act_silu(to_f32(p.z[size_t(t[k]) * p.ldz + c])));
     }
   }
 }
 
 template <typename T, int NPT, int LPC>
-static int launch_scan_as(const ScanParams<T>& p, int has_long, int has_single, cudaStream_t st) {
+static int launch_rows(const ScanParams<T>& p, cudaStream_t st) {
   constexpr int CPB = kScanThreads / LPC;
-  constexpr int IT = NPT > 4 ? 1 : kScanIter;
-  if (has_single) scan_single_kernel<T, NPT, LPC><<<dim3((p.C + CPB * IT - 1) / (CPB * IT), p.q.n), kScanThreads, 0, st>>>(p);
-  if (has_long) scan_rows_kernel<T, NPT, LPC><<<dim3((p.C + CPB - 1) / CPB, p.q.n), kScanThreads, 0, st>>>(p);
+  scan_rows_kernel<T, NPT, LPC><<<dim3((p.C + CPB - 1) / CPB, p.q.n), kScanThreads, 0, st>>>(p);
+  return cudaGetLastError() == cudaSuccess ? 0 : -1;
+}
+template <typename T, int NPT, int LPC>
+static int launch_single(const ScanParams<T>& p, cudaStream_t st) {
+  constexpr int CPB = kScanThreads / LPC;
+  constexpr int NS = NPT > 4 ? 1 : kScanSeqs;
+  const int bytes = 4 * int(sizeof(T));
+  const bool bc4 = p.N % 4 == 0 && (p.ldb * sizeof(T)) % bytes == 0 && reinterpret_cast<uintptr_t>(p.B) % bytes == 0 &&
+                   reinterpret_cast<uintptr_t>(p.Cm) % bytes == 0;
+  scan_single_kernel<T, NPT, LPC><<<dim3((p.C + CPB - 1) / CPB, (p.q.n + NS - 1) / NS), kScanThreads, 0, st>>>(p, bc4);
   return cudaGetLastError() == cudaSuccess ? 0 : -1;
 }
 template <typename T>
 static int launch_scan(const ScanParams<T>& p, int has_long, int has_single, cudaStream_t st) {
   const int n = p.N;
-  if (n <= 4) return launch_scan_as<T, 4, 1>(p, has_long, has_single, st);
-  if (n <= 8) return launch_scan_as<T, 4, 2>(p, has_long, has_single, st);
-  if (n <= 16) return launch_scan_as<T, 4, 4>(p, has_long, has_single, st);
-  if (n <= 32) return launch_scan_as<T, 4, 8>(p, has_long, has_single, st);
-  if (n <= 64) return launch_scan_as<T, 4, 16>(p, has_long, has_single, st);
-  if (n <= 128) return launch_scan_as<T, 4, 32>(p, has_long, has_single, st);
-  if (n <= 256) return launch_scan_as<T, 8, 32>(p, has_long, has_single, st);
-  return -2;
+  if (n > 256) return -2;
+  int rc = 0;
+  if (has_single) {
+    if (n <= 4) rc = launch_single<T, 4, 1>(p, st);
+    else if (n <= 8) rc = launch_single<T, 4, 2>(p, st);
+    else if (n <= 16) rc = launch_single<T, 4, 4>(p, st);
+    else if (n <= 32) rc = launch_single<T, 4, 8>(p, st);
+    else if (n <= 64) rc = launch_single<T, 4, 16>(p, st);
+    else if (n <= 128) rc = launch_single<T, 4, 32>(p, st);
+    else rc = launch_single<T, 8, 32>(p, st);
+  }
+  if (rc || !has_long) return rc;
+  if (n <= 4) return launch_rows<T, 4, 1>(p, st);
+  if (n <= 8) return launch_rows<T, 8, 1>(p, st);
+  if (n <= 16) return launch_rows<T, 8, 2>(p, st);
+  if (n <= 32) return launch_rows<T, 8, 4>(p, st);
+  if (n <= 64) return launch_rows<T, 8, 8>(p, st);
+  if (n <= 128) return launch_rows<T, 16, 8>(p, st);
+  return launch_rows<T, 32, 8>(p, st);
 }
 
 template <typename F>
@@ -999,7 +1132,7 @@ XL_API int xl_token_shift(const void* h, const void* mu, void* last, void* out, 
   });
 }
 
-// out [rows, C] = silu(bias + causal convolution of x (row pitch ldx) with w [C, taps]); state [n_slots, taps - 1, C]
+// out [rows, C] = silu(bias + causal convolution of x (row pitch ldx) with w [taps, C]); state [n_slots, taps - 1, C]
 XL_API int xl_conv_silu(const void* x, const void* w, const void* bias, void* state, void* out, const void* token_seq, const void* q_cu,
                         const void* kv_lens, const void* slots, int n_seqs, int n_slots, int rows, int C, int taps, long ldx,
                         int has_long, int f32, void* stream) {
@@ -1012,12 +1145,15 @@ XL_API int xl_conv_silu(const void* x, const void* w, const void* bias, void* st
     const T *xx = static_cast<const T*>(x), *ww = static_cast<const T*>(w), *b = static_cast<const T*>(bias);
     T *s = static_cast<T*>(state), *o = static_cast<T*>(out);
     const int* ts = static_cast<const int*>(token_seq);
-    const bool vec = C % 8 == 0 && ldx % 8 == 0 && aligned16(x, bias, state, out);
+    const bool vec = C % 8 == 0 && ldx % 8 == 0 && aligned16(x, bias, state, out) && aligned16(w, w, w, w);
     const int per = vec ? 8 : 1, cols = (C + per * 128 - 1) / (per * 128);
-    const dim3 grid((rows + kConvRows - 1) / kConvRows, cols);
-#define XL_CONV(V, TAPS) conv_silu_kernel<T, V, TAPS><<<grid, 128, 0, st>>>(xx, ww, b, s, o, ts, q, rows, C, taps, ldx)
+    const int tile = has_long ? kConvRows : kConvRowsSingle;
+    const dim3 grid((rows + tile - 1) / tile, cols);
+#define XL_CONV(V, TAPS)                                                                                              \
+  if (has_long) conv_silu_kernel<T, V, TAPS, kConvRows><<<grid, 128, 0, st>>>(xx, ww, b, s, o, ts, q, rows, C, taps, ldx); \
+  else conv_silu_kernel<T, V, TAPS, kConvRowsSingle><<<grid, 128, 0, st>>>(xx, ww, b, s, o, ts, q, rows, C, taps, ldx)
     if (vec) {
-      if (taps == 4) XL_CONV(8, 4); else if (taps == 3) XL_CONV(8, 3); else if (taps == 2) XL_CONV(8, 2); else XL_CONV(8, 0);
+      if (taps == 4) { XL_CONV(8, 4); } else if (taps == 3) { XL_CONV(8, 3); } else if (taps == 2) { XL_CONV(8, 2); } else { XL_CONV(8, 0); }
     } else {
       XL_CONV(1, 0);
     }

@@ -42,7 +42,7 @@ class ParallelWeights:
 
 class ScanWeights:
     def __init__(self):
-        self.in_w = self.conv_w = self.conv_b = None
+        self.in_w = self.conv_w = self.conv_b = None     # conv_w: [taps, channels]
         self.x_w = self.dt_w = None             # bf16: rows / columns padded with zeros to multiples of 8
         self.dt_b = self.A = self.D = None      # fp32
         self.A_log = None                       # as stored
@@ -154,7 +154,7 @@ class FalalixForCausalLM:
                 L.norm2, L.mlp.up_w, L.mlp.down_w = dev(p + "norm2"), dev(p + "mlp.up"), dev(p + "mlp.down")
             p += "mix."
             if isinstance(m, SelectiveScanSpec):
-                W.in_w, W.conv_w, W.conv_b, W.o_w = dev(p + "in"), dev(p + "conv"), dev(p + "conv.b"), dev(p + "o")
+                W.in_w, W.conv_w, W.conv_b, W.o_w = dev(p + "in"), dev(p + "conv").t().contiguous(), dev(p + "conv.b"), dev(p + "o")
                 W.x_w = _pad(dev(p + "x"), pad8(m.dt_rank + 2 * m.state), m.inner)
                 W.dt_w = _pad(dev(p + "dt"), m.inner, pad8(m.dt_rank))
                 W.dt_b, W.D, W.A_log = f32(p + "dt.b"), f32(p + "D"), dev(p + "A_log")
@@ -224,7 +224,7 @@ class FalalixForCausalLM:
                 sd[p + "norm2"], sd[p + "mlp.up"], sd[p + "mlp.down"] = L.norm2, L.mlp.up_w, L.mlp.down_w
             p += "mix."
             if isinstance(m, SelectiveScanSpec):
-                sd.update({p + "in": W.in_w, p + "conv": W.conv_w, p + "conv.b": W.conv_b, p + "x": W.x_w[:m.dt_rank + 2 * m.state],
+                sd.update({p + "in": W.in_w, p + "conv": W.conv_w.t(), p + "conv.b": W.conv_b, p + "x": W.x_w[:m.dt_rank + 2 * m.state],
                            p + "dt": W.dt_w[:, :m.dt_rank], p + "dt.b": W.dt_b, p + "A_log": W.A_log, p + "D": W.D, p + "o": W.o_w})
                 continue
             a = m.left

@@ -202,7 +202,8 @@ def time_mix(r, k, v, z, w0, u, gate, norm_w, scale, eps, state, inp, out):
 
 
 def conv_silu(x, w, b, state, inp):
-    """silu of a causal convolution per channel over each sequence; x may be a strided view; state [slots, taps - 1, C]."""
+    """silu of a causal convolution per channel over each sequence; w [taps, C]; x may be a strided view; state
+    [slots, taps - 1, C]."""
     return _cuda().conv_silu(x, w, b, state, inp) if x.is_cuda else ref.conv_silu(x, w, b, state, *_seqs(inp))
 
 

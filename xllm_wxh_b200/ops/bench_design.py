@@ -1,4 +1,4 @@
-"""A model design beside the framework's closest other one at equal layer sizes (`bench.py --compare-design movolorn`):
+"""A model design beside the framework's closest other one at equal layer sizes (`bench.py --compare-design movolorn|falalix`):
 tokens per second of the decoder layers in prefill and decode, and the design's own kernels beside the like kernels with their
 distance from the roofline.  Random weights; kernel and layer times come from CUDA-graph replay between CUDA events, with
 weights, caches and activations rotated through (or larger than) more memory than L2 holds."""
@@ -14,14 +14,19 @@ import torch
 
 from ..framework.step_input import StepInput, make_layout
 from ..models.args import ModelArgs, preset
-from ..models.layer_spec import AttentionSpec
+from ..models.layer_spec import AttentionSpec, ParallelSpec
 from ..models.registry import get_model_class
 from . import cuda_ops as c
 from . import moe_cuda
 from .bench_kernels import time_graph
 
 DEV = "cuda:0"
-PAIRS = {"movolorn": [("movolorn-8b", "qwen3-8b"), ("movolorn-30b-a3b", "qwen3-30b-a3b")]}
+# (model, closest one, which of the model's kinds of layer)
+PAIRS = {"movolorn": [("movolorn-8b", "qwen3-8b", ""), ("movolorn-30b-a3b", "qwen3-30b-a3b", "")],
+         "falalix": [("falalix-8b", "qwen3-8b", "parallel"), ("falalix-8b", "qwen3-8b", "scan"), ("falalix-8b", "qwen3-8b", "")]}
+# Issue rates that bound recurrent kernels in fp32, per second over 148 SMs at 1.9 GHz: 128 multiply-adds and 16 exponentials
+# per SM and clock (nominal; there is no measured figure for them).
+FMA_RATE, EXP_RATE = 148 * 128 * 1.9e9, 148 * 16 * 1.9e9
 STEPS = [("prefill", 1, 8192, 8192), ("prefill", 8, 1024, 1024), ("decode", 256, 1, 1152), ("decode", 32, 1, 8192)]
 
 
@@ -49,6 +54,7 @@ def step_input(seqs: int, q_len: int, kv_len: int, block: int, vocab: int) -> St
     host[L.slots:L.slots + T] = (bt[seq, pos // block] * block + (pos % block)).int()
     host[L.q_cu:L.q_cu + seqs + 1] = (torch.arange(seqs + 1) * q_len).int()
     host[L.kv_lens:L.kv_lens + seqs] = kv_len
+    host[L.state_slots:L.state_slots + seqs] = torch.randperm(seqs).int() + 1
     host[L.block_tables:L.block_tables + seqs * nb] = bt.reshape(-1)
     hdr = np.zeros(32, dtype=np.int32)
     dec = q_len == 1
@@ -58,22 +64,28 @@ def step_input(seqs: int, q_len: int, kv_len: int, block: int, vocab: int) -> St
     return StepInput(host.to(DEV), L, hdr)
 
 
-def cut_to_layers(a: ModelArgs, n: int) -> ModelArgs:
+def cut_to_layers(a: ModelArgs, n: int, kind: str = "") -> ModelArgs:
+    """n layers, all of one kind where a model has several ("parallel", "scan") and one is named."""
     kw = dict(n_layers=n)
     if a.layer_specs:
-        kw.update(layer_specs=a.layer_specs[:n], layer_runs=a.layer_runs[:n])
+        specs = [s for s in a.layer_specs if not kind or (kind == "parallel") == isinstance(s.mixer, ParallelSpec)]
+        kw.update(layer_specs=specs[:n], layer_runs=list(range(n)), pass_starts=[])
     return dataclasses.replace(a, **kw)
 
 
 @torch.inference_mode()
-def layer_throughput(name: str, layers: int, block: int) -> List[Dict]:
-    args = cut_to_layers(preset(name), layers)
-    model = get_model_class(args.model_type)(args, device=DEV, dtype=torch.bfloat16).init_random(0).finalize_weights()
+def layer_throughput(name: str, layers: int, block: int, kind: str = "") -> List[Dict]:
+    args = cut_to_layers(preset(name), layers, kind)
+    model = get_model_class(args.model_type)(args, device=DEV, dtype=torch.bfloat16).init_random(0)
+    if hasattr(model, "finalize_weights"):
+        model.finalize_weights()
     rows = []
     for kind, seqs, q_len, kv_len in STEPS:
         inp = step_input(seqs, q_len, kv_len, block, args.vocab_size)
         blocks = seqs * (-(-kv_len // block)) + 1
         kv = [tuple(torch.randn(s, device=DEV, dtype=torch.bfloat16) for s in pair) for pair in model.kv_cache_shapes(blocks, block)]
+        if hasattr(model, "state_cache_shapes"):
+            inp.states = [tuple(torch.zeros(s, device=DEV, dtype=dt) for s, dt in run) for run in model.state_cache_shapes(seqs + 1)]
         us = time_graph([lambda: model.forward(inp, kv)] * 3)
         rows.append({"step": kind, "sequences": seqs, "tokens": seqs * q_len, "context": kv_len, "us_per_layer": round(us / layers, 1),
                      "tokens_per_s_per_layer": round(seqs * q_len / us * layers * 1e6)})
@@ -92,19 +104,32 @@ def _bf(*shape, std=1.0):
     return (torch.randn(*shape, device=DEV) * std).to(torch.bfloat16)
 
 
-@torch.inference_mode()
-def kernel_pairs() -> List[Dict]:
-    """Each kernel of the design beside the like one: microseconds, bytes or FLOPs of each, and the fraction of the roofline."""
-    pk = peaks()
-    rows = []
+class Rows:
+    """Kernels of a design beside the like ones: microseconds and fraction of the roofline of each."""
 
-    def add(what, ours, like, bytes_ours=0.0, bytes_like=0.0, flops=0.0):
+    def __init__(self):
+        self.pk = peaks()
+        self.rows = []
+
+    def add(self, what, ours, like, bytes_ours=0.0, bytes_like=0.0, flops=0.0):
         def frac(us, nbytes):
-            bound = max(nbytes / (pk["hbm_gbs"] * 1e3), flops / (pk["bf16_tflops"] * 1e6))
+            bound = max(nbytes / (self.pk["hbm_gbs"] * 1e3), flops / (self.pk["bf16_tflops"] * 1e6))
             return bound / us
         fo, fl = frac(ours, bytes_ours), frac(like, bytes_like)
-        rows.append({"what": what, "us": round(ours, 1), "like_us": round(like, 1), "roofline": round(fo, 3), "like_roofline": round(fl, 3),
-                     "farther_by": round(fl / fo, 2)})
+        self.rows.append({"what": what, "us": round(ours, 1), "like_us": round(like, 1), "roofline": round(fo, 3), "like_roofline": round(fl, 3),
+                          "farther_by": round(fl / fo, 2)})
+
+    def add_alone(self, what, us, nbytes, fma=0.0, exps=0.0):
+        """A kernel without a like one: its bound is the slowest of memory, fp32 multiply-adds and exponentials."""
+        bounds = {"memory": nbytes / (self.pk["hbm_gbs"] * 1e3), "fp32": fma / FMA_RATE * 1e6, "exp": exps / EXP_RATE * 1e6}
+        by = max(bounds, key=bounds.get)
+        self.rows.append({"what": what, "us": round(us, 1), "roofline": round(bounds[by] / us, 3), "bound_by": by})
+
+
+@torch.inference_mode()
+def movolorn_kernels() -> List[Dict]:
+    table_rows = Rows()
+    add, rows = table_rows.add, table_rows.rows
     # ---- attention
     for H, G, chunk in ((32, 8, 8192), (32, 4, 8192)):
         spec = AttentionSpec(heads=H, kv_heads=G, dim=128, vdim=128, scale=128 ** -0.5)
@@ -193,13 +218,94 @@ def kernel_pairs() -> List[Dict]:
     return rows
 
 
+@torch.inference_mode()
+def falalix_kernels() -> List[Dict]:
+    R = Rows()
+    add, alone = R.add, R.add_alone
+    H = 4096
+    # ---- attention with a window and kept first keys, beside the same window without
+    for kind, seqs, q_len, kv in STEPS:
+        heads, G, window, keep = 32, 8, 4096, 128
+        inp = step_input(seqs, q_len, kv, 16, 1000)
+        nb, row = seqs * (-(-kv // 16)) + 1, (heads + 2 * G) * 128
+        seen = min(kv, window + keep)
+        cache_bytes = 2.0 * seqs * (kv if kind == "prefill" else seen) * G * 128 * 2
+        sets = _rotated(lambda: (_bf(seqs * q_len, row), _bf(nb, 16, G, 128), _bf(nb, 16, G, 128)), cache_bytes + seqs * q_len * row * 2)[:8]
+        view = lambda q: q[:, :heads * 128].unflatten(1, (heads, 128))
+        o = time_graph([lambda s=s: c.paged_attention_ext(view(s[0]), s[1], s[2], inp, 128 ** -0.5, window, 0, None, None, keep) for s in sets])
+        k = time_graph([lambda s=s: c.paged_attention(view(s[0]), s[1], s[2], inp, 128 ** -0.5, window) for s in sets])
+        byts = cache_bytes + 2.0 * seqs * q_len * heads * 128 * 2
+        first = kv - q_len
+        pairs = sum(min(p + 1, window + keep) for p in range(first, kv)) * seqs
+        add(f"attention {kind} {seqs} x {q_len} of {kv}, window {window} + {keep}", o, k, byts, byts,
+            4.0 * heads * 128 * pairs if kind == "prefill" else 0.0)
+    # ---- norms, cache write, gates
+    cs = torch.randn(8192, 128, device=DEV)
+    for T in (8192, 256):
+        w, wa = _bf(H), (_bf(4096), _bf(1024))
+        sets = _rotated(lambda: (_bf(T, H), torch.randn(T, H, device=DEV), _bf(T, H)), T * H * 10.0)
+        o = time_graph([lambda s=s: c.add_norm(s[0], s[1], 0.3, w, 1e-6) for s in sets])
+        k = time_graph([lambda s=s: c.add_rms_norm(s[0], s[2], w, 1e-6) for s in sets])
+        add(f"residual + norm, {T} x {H}", o, k, T * H * 12.0, T * H * 8.0)
+        inp = step_input(1, T, T, 16, 1000)
+        sets = _rotated(lambda: (_bf(T, 10240), _bf(T // 16 + 1, 16, 8, 128), _bf(T // 16 + 1, 16, 8, 128), _bf(T, 6144)), T * 10240 * 2.0)[:24]
+        o = time_graph([lambda s=s: c.qknorm_all_kvwrite(s[0], inp.slots, wa[0], wa[1], 1e-6, s[1], s[2], 32, 8) for s in sets])
+        k = time_graph([lambda s=s: c.rope_qknorm_kvwrite(s[3], inp.positions, inp.slots, cs, w, w, 1e-6, s[1], s[2], 32, 8, 128) for s in sets])
+        add(f"q / k norm + cache write, {T} tokens", o, k, T * 96.0 * 256, T * 104.0 * 256 + T * 512.0)
+        sets = _rotated(lambda: (_bf(T, 4096), _bf(T, 10240), torch.empty(T, 8192, device=DEV, dtype=torch.bfloat16), _bf(T, 8192)), T * 4096 * 6.0)[:24]
+        o = time_graph([lambda s=s: c.gate_into(s[0], s[1][:, 6144:], 0.5, s[2][:, :4096]) for s in sets])
+        k = time_graph([lambda s=s: c.silu_and_mul(s[3]) for s in sets])
+        add(f"output gate, {T} x 4096", o, k, T * 4096 * 6.0, T * 4096 * 6.0)
+        # ---- products with an epilogue
+        sets = _rotated(lambda: (_bf(T, H), _bf(12288, H, std=0.02)), 12288 * 8192.0)[:4]
+        o = time_graph([lambda s=s: c.act_linear(s[0], s[1], "relu2") for s in sets])
+        k = time_graph([lambda s=s: c.linear(s[0], s[1]) for s in sets])
+        b = 12288 * 8192.0 + T * (8192.0 + 24576.0)
+        add(f"up product + squared relu, {T} x 12288 x 4096", o, k, b, b, 2.0 * T * 12288 * H)
+    # ---- recurrent kernels, which have no like one
+    C, N, taps, heads, d = 8192, 16, 4, 64, 64
+    for kind, seqs, q_len, kv in STEPS[:3]:
+        T = seqs * q_len
+        inp = step_input(seqs, q_len, kv, 16, 1000)
+        new = kv == q_len
+        sets = [(_bf(T, H), _bf(5, H), _bf(seqs + 1, H)) for _ in range(8)]
+        alone(f"token shift, {kind} {seqs} x {q_len}", time_graph([lambda s=s: c.token_shift(s[0], s[1], s[2], inp) for s in sets]), T * H * 12.0)
+        del sets
+        sets = [(_bf(T, 2 * C), _bf(taps, C), _bf(C), _bf(seqs + 1, taps - 1, C)) for _ in range(4 if kind == "prefill" else 16)]
+        alone(f"convolution, {kind} {seqs} x {q_len}", time_graph([lambda s=s: c.conv_silu(s[0][:, :C], s[1], s[2], s[3], inp) for s in sets]),
+              T * C * 4.0 + (0 if new else 2) * seqs * 3 * C * 2.0)
+        del sets
+        A = -torch.rand(C, N, device=DEV)
+        D, bias = torch.randn(C, device=DEV), torch.randn(C, device=DEV) - 3
+        sets = [(_bf(T, C), torch.randn(T, C, device=DEV), _bf(T, 288), _bf(T, 2 * C), torch.zeros(seqs + 1, C, N, device=DEV)) for _ in range(3)]
+        us = time_graph([lambda s=s: c.selective_scan(s[0], s[1], bias, A, s[2][:, 256:272], s[2][:, 272:], D, s[3][:, C:], s[4], inp) for s in sets])
+        alone(f"selective scan, {kind} {seqs} x {q_len}, {C} channels x {N}", us, T * C * 10.0 + (1 if new else 2) * seqs * C * N * 4.0,
+              3.0 * T * C * N, 1.0 * T * C * N)
+        del sets
+        n = heads * d
+        u, w0, nw = torch.randn(heads, d, device=DEV), torch.randn(n, device=DEV) - 3, _bf(n)
+        sets = [(_bf(T, n), _bf(T, n), _bf(T, n), torch.randn(T, n, device=DEV), _bf(T, n), torch.empty(T, 2 * n, device=DEV, dtype=torch.bfloat16),
+                 torch.zeros(seqs + 1, heads, d, d, device=DEV)) for _ in range(3)]
+        us = time_graph([lambda s=s: c.time_mix(s[0], s[1], s[2], s[3], w0, u, s[4], nw, 0.5, 1e-6, s[6], inp, s[5][:, n:]) for s in sets])
+        alone(f"time mixing, {kind} {seqs} x {q_len}, {heads} heads of {d}", us, T * n * 14.0 + (1 if new else 2) * seqs * n * d * 4.0, 3.0 * T * n * d,
+              2.0 * T * n)
+        del sets
+    return R.rows
+
+
+KERNELS = {"movolorn": movolorn_kernels, "falalix": falalix_kernels}
+
+
 def run(design: str, layers: int = 4, block: int = 16) -> Dict:
     out = {"design": design, "layers": layers, "block_size": block, "peaks": peaks(), "models": []}
-    for ours, like in PAIRS[design]:
-        a, b = layer_throughput(ours, layers, block), layer_throughput(like, layers, block)
-        out["models"].append({"model": ours, "closest": like,
+    seen: Dict[str, List[Dict]] = {}
+    for ours, like, kind in PAIRS[design]:
+        if like not in seen:
+            seen[like] = layer_throughput(like, layers, block)
+        a, b = layer_throughput(ours, layers, block, kind), seen[like]
+        out["models"].append({"model": ours + (f" ({kind} layers)" if kind else ""), "closest": like,
                               "steps": [dict(x, closest_us_per_layer=y["us_per_layer"], ratio=round(y["us_per_layer"] / x["us_per_layer"], 3))
                                         for x, y in zip(a, b)]})
-    out["kernels"] = kernel_pairs()
+    out["kernels"] = KERNELS[design]()
     out["device_status"] = c.read_status()
     return out

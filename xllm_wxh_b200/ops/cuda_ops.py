@@ -439,15 +439,15 @@ def token_shift(h: torch.Tensor, mu: torch.Tensor, last: torch.Tensor, inp) -> t
 
 
 def conv_silu(x: torch.Tensor, w: torch.Tensor, b: torch.Tensor, state: torch.Tensor, inp) -> torch.Tensor:
-    """silu(b + causal convolution of x [T, C] (may be a strided view) with w [C, taps]); state [slots, taps - 1, C]."""
+    """silu(b + causal convolution of x [T, C] (may be a strided view) with w [taps, C]); state [slots, taps - 1, C]."""
     global launch_count
     T, C = x.shape
     assert x.stride(1) == 1 and w.is_contiguous() and w.dtype == b.dtype == state.dtype == x.dtype
     n, seqs = _state_args(inp, state)
     out = _rows_out(inp, (T, C), x)
     _check(lib().xl_conv_silu(_ptr(x), _ptr(w), _ptr(b), _ptr(state), _ptr(out), _ptr(inp.token_seq), *seqs, c_int(T), c_int(C),
-                              c_int(w.shape[1]), c_long(x.stride(0)), c_int(int(inp.has_prefill)), _f32flag(x), _stream()), "xl_conv_silu")
-    launch_count += 2 if inp.has_prefill and w.shape[1] > 1 else 1
+                              c_int(w.shape[0]), c_long(x.stride(0)), c_int(int(inp.has_prefill)), _f32flag(x), _stream()), "xl_conv_silu")
+    launch_count += 2 if inp.has_prefill and w.shape[0] > 1 else 1
     return out
 
 

@@ -473,13 +473,13 @@ def time_mix(r, k, v, z, w0, u, gate, norm_w, scale, eps, state, q_cu, kv_lens, 
 
 
 def conv_silu(x, w, b, state, q_cu, kv_lens, slots, n_seqs):
-    """Causal convolution of every channel (w [C, taps], last column the current row) + b, then silu; state [slots, taps - 1, C]
+    """Causal convolution of every channel (w [taps, C], last row the current input's) + b, then silu; state [slots, taps - 1, C]
     keeps the last rows."""
-    taps = w.shape[1]
+    taps = w.shape[0]
     y = torch.zeros(x.shape, dtype=torch.float32)
     for lo, hi, cont, s in _spans(q_cu, kv_lens, slots, n_seqs):
         rows = torch.cat([state[s] if cont else torch.zeros_like(state[s]), x[lo:hi]])
-        y[lo:hi] = sum(rows[i:i + hi - lo].float() * w[:, i].float() for i in range(taps)) + b.float()
+        y[lo:hi] = sum(rows[i:i + hi - lo].float() * w[i].float() for i in range(taps)) + b.float()
         if taps > 1:
             state[s] = rows[1 - taps:]
     return torch.nn.functional.silu(y).to(x.dtype)
