@@ -64,6 +64,28 @@ __device__ __forceinline__ void store_n(T* p, const float (&f)[V]) {
   else from_f32(p, f[0]);
 }
 
+// two fp32 lanes in one 64-bit register
+__device__ __forceinline__ uint64_t pack2(float a, float b) {
+  uint64_t r;
+  asm("mov.b64 %0, {%1, %2};" : "=l"(r) : "f"(a), "f"(b));
+  return r;
+}
+__device__ __forceinline__ float2 unpack2(uint64_t v) {
+  float2 r;
+  asm("mov.b64 {%0, %1}, %2;" : "=f"(r.x), "=f"(r.y) : "l"(v));
+  return r;
+}
+__device__ __forceinline__ uint64_t fma2(uint64_t a, uint64_t b, uint64_t c) {
+  uint64_t d;
+  asm("fma.rn.f32x2 %0, %1, %2, %3;" : "=l"(d) : "l"(a), "l"(b), "l"(c));
+  return d;
+}
+__device__ __forceinline__ uint64_t mul2(uint64_t a, uint64_t b) {
+  uint64_t d;
+  asm("mul.rn.f32x2 %0, %1, %2;" : "=l"(d) : "l"(a), "l"(b));
+  return d;
+}
+
 // Eight elements as they come from memory, converted when they are used.
 template <typename T> struct Vec8;
 template <> struct Vec8<__nv_bfloat16> {
@@ -89,6 +111,13 @@ template <> struct Vec8<float> {
     f[0] = a.x; f[1] = a.y; f[2] = a.z; f[3] = a.w;
     f[4] = b.x; f[5] = b.y; f[6] = b.z; f[7] = b.w;
   }
+};
+
+template <typename T, int V> struct Raw : Vec8<T> {};
+template <typename T> struct Raw<T, 1> {
+  T v;
+  __device__ __forceinline__ void load(const T* p) { v = *p; }
+  __device__ __forceinline__ void get(float (&f)[1]) const { f[0] = to_f32(v); }
 };
 
 // ============================================================================ token shift
@@ -132,7 +161,7 @@ __global__ void __launch_bounds__(256) token_shift_kernel(const T* __restrict__ 
 constexpr int kConvRows = 16, kConvRowsSingle = 2;
 
 template <typename T, int V, int TAPS, int ROWS>
-__global__ void __launch_bounds__(128) conv_silu_kernel(const T* __restrict__ x, const T* __restrict__ w, const T* __restrict__ bias,
+__global__ void __launch_bounds__(128, sizeof(T) == 2 ? 6 : 1) conv_silu_kernel(const T* __restrict__ x, const T* __restrict__ w, const T* __restrict__ bias,
                                                         T* __restrict__ state, T* __restrict__ out, const int* __restrict__ token_seq,
                                                         const Seqs q, int rows, int C, int taps_rt, long ldx) {
   constexpr int H = TAPS > 1 ? TAPS - 1 : 1;
@@ -140,91 +169,93 @@ __global__ void __launch_bounds__(128) conv_silu_kernel(const T* __restrict__ x,
   const int c = (blockIdx.y * blockDim.x + threadIdx.x) * V;
   if (c >= C) return;
   const int t0 = blockIdx.x * ROWS, t1 = min(rows, t0 + ROWS);
-  float b[V], wt[TAPS > 0 ? TAPS : 1][V], hist[H][V];
+  float b[V], hist[H][V];
+  Raw<T, V> wt[TAPS > 0 ? TAPS : 1];
   load_n<V>(bias + c, b);
   if (TAPS > 0) {
 #pragma unroll
-    for (int i = 0; i < TAPS; ++i) load_n<V>(w + size_t(i) * C + c, wt[i]);
+    for (int i = 0; i < TAPS; ++i) wt[i].load(w + size_t(i) * C + c);
   }
   int cur_seq = -1, start = 0, end = 0, slot = 0;
   bool cont = false;
   constexpr int AHEAD = ROWS < 4 ? ROWS : 4;             // rows requested together
-  float ahead[AHEAD][V];
+  Raw<T, V> ahead[AHEAD];
   int seqs[AHEAD];
 #pragma unroll 1
   for (int tg = t0; tg < t1; tg += AHEAD) {
 #pragma unroll
-  for (int r = 0; r < AHEAD; ++r) {
-    seqs[r] = tg + r < t1 ? token_seq[tg + r] : -1;
-    if (tg + r < t1) load_n<V>(x + size_t(tg + r) * ldx + c, ahead[r]);
-  }
-#pragma unroll
-  for (int r = 0; r < AHEAD; ++r) {
-    const int t = tg + r, seq = seqs[r];
-    if (seq < 0 || seq >= q.n) continue;
-    const bool fresh = seq != cur_seq;
-    if (fresh) {
-      cur_seq = seq;
-      start = q.q_cu[seq];
-      end = q.q_cu[seq + 1];
-      slot = record_of(q, seq);
-      cont = q.kv_lens[seq] > end - start;
+    for (int r = 0; r < AHEAD; ++r) {
+      seqs[r] = tg + r < t1 ? token_seq[tg + r] : -1;
+      if (tg + r < t1) ahead[r].load(x + size_t(tg + r) * ldx + c);
     }
-    if (slot < 0) continue;
-    // input `back` rows ahead of row t of this sequence
-    auto before = [&](int back, float (&f)[V]) {
-      const int j = t - start - back;
 #pragma unroll
-      for (int e = 0; e < V; ++e) f[e] = 0.f;
-      if (j >= 0) load_n<V>(x + size_t(t - back) * ldx + c, f);
-      else if (cont) load_n<V>(state + (size_t(slot) * (taps - 1) + (taps - 1 + j)) * C + c, f);
-    };
-    float y[V];
-    const float(&cur)[V] = ahead[r];
-#pragma unroll
-    for (int e = 0; e < V; ++e) y[e] = b[e];
-    if (TAPS > 0) {
+    for (int r = 0; r < AHEAD; ++r) {
+      const int t = tg + r, seq = seqs[r];
+      if (seq < 0 || seq >= q.n) continue;
+      const bool fresh = seq != cur_seq;
       if (fresh) {
-#pragma unroll
-        for (int i = 0; i < TAPS - 1; ++i) before(TAPS - 1 - i, hist[i]);
+        cur_seq = seq;
+        start = q.q_cu[seq];
+        end = q.q_cu[seq + 1];
+        slot = record_of(q, seq);
+        cont = q.kv_lens[seq] > end - start;
       }
+      if (slot < 0) continue;
+      // input `back` rows ahead of row t of this sequence
+      auto before = [&](int back, float (&f)[V]) {
+        const int j = t - start - back;
 #pragma unroll
-      for (int i = 0; i < TAPS - 1; ++i)
+        for (int e = 0; e < V; ++e) f[e] = 0.f;
+        if (j >= 0) load_n<V>(x + size_t(t - back) * ldx + c, f);
+        else if (cont) load_n<V>(state + (size_t(slot) * (taps - 1) + (taps - 1 + j)) * C + c, f);
+      };
+      float y[V], cur[V], f[V];
+      ahead[r].get(cur);
 #pragma unroll
-        for (int e = 0; e < V; ++e) y[e] = fmaf(hist[i][e], wt[i][e], y[e]);
+      for (int e = 0; e < V; ++e) y[e] = b[e];
+      if (TAPS > 0) {
+        if (fresh) {
 #pragma unroll
-      for (int e = 0; e < V; ++e) y[e] = fmaf(cur[e], wt[TAPS > 0 ? TAPS - 1 : 0][e], y[e]);
+          for (int i = 0; i < TAPS - 1; ++i) before(TAPS - 1 - i, hist[i]);
+        }
 #pragma unroll
-      for (int i = 0; i + 1 < TAPS - 1; ++i)
+        for (int i = 0; i < TAPS - 1; ++i) {
+          wt[i].get(f);
 #pragma unroll
-        for (int e = 0; e < V; ++e) hist[i][e] = hist[i + 1][e];
-      if (TAPS > 1) {
+          for (int e = 0; e < V; ++e) y[e] = fmaf(hist[i][e], f[e], y[e]);
+        }
+        wt[TAPS > 0 ? TAPS - 1 : 0].get(f);
 #pragma unroll
-        for (int e = 0; e < V; ++e) hist[H - 1][e] = cur[e];
-        if (end - start == 1) {                    // a single row: this thread alone reads and writes this part of the record
+        for (int e = 0; e < V; ++e) y[e] = fmaf(cur[e], f[e], y[e]);
 #pragma unroll
-          for (int i = 0; i < TAPS - 1; ++i) store_n<V>(state + (size_t(slot) * H + i) * C + c, hist[i]);
+        for (int i = 0; i + 1 < TAPS - 1; ++i)
+#pragma unroll
+          for (int e = 0; e < V; ++e) hist[i][e] = hist[i + 1][e];
+        if (TAPS > 1) {
+#pragma unroll
+          for (int e = 0; e < V; ++e) hist[H - 1][e] = cur[e];
+          if (end - start == 1) {                    // a single row: this thread alone reads and writes this part of the record
+#pragma unroll
+            for (int i = 0; i < TAPS - 1; ++i) store_n<V>(state + (size_t(slot) * H + i) * C + c, hist[i]);
+          }
+        }
+      } else {
+        for (int i = 0; i < taps; ++i) {
+          before(taps - 1 - i, f);
+#pragma unroll
+          for (int e = 0; e < V; ++e) y[e] = fmaf(f[e], to_f32(w[size_t(i) * C + c + e]), y[e]);
+        }
+        if (end - start == 1) {
+          for (int i = 0; i < taps - 1; ++i) {
+            before(taps - 2 - i, f);                 // row i moves down by one, the last becomes the current input
+            store_n<V>(state + (size_t(slot) * (taps - 1) + i) * C + c, f);
+          }
         }
       }
-    } else {
-      for (int i = 0; i < taps; ++i) {
-        float f[V];
-        before(taps - 1 - i, f);
 #pragma unroll
-        for (int e = 0; e < V; ++e) y[e] = fmaf(f[e], to_f32(w[size_t(i) * C + c + e]), y[e]);
-      }
-      if (end - start == 1) {
-        for (int i = 0; i < taps - 1; ++i) {
-          float f[V];
-          before(taps - 2 - i, f);                 // row i moves down by one, the last becomes the current input
-          store_n<V>(state + (size_t(slot) * (taps - 1) + i) * C + c, f);
-        }
-      }
+      for (int e = 0; e < V; ++e) y[e] = act_silu(y[e]);
+      store_n<V>(out + size_t(t) * C + c, y);
     }
-#pragma unroll
-    for (int e = 0; e < V; ++e) y[e] = act_silu(y[e]);
-    store_n<V>(out + size_t(t) * C + c, y);
-  }
   }
 }
 
@@ -296,28 +327,6 @@ __device__ __forceinline__ bool find_segment(const Seqs& q, int L, int target, i
   return false;
 }
 
-// two fp32 lanes in one 64-bit register
-__device__ __forceinline__ uint64_t pack2(float a, float b) {
-  uint64_t r;
-  asm("mov.b64 %0, {%1, %2};" : "=l"(r) : "f"(a), "f"(b));
-  return r;
-}
-__device__ __forceinline__ float2 unpack2(uint64_t v) {
-  float2 r;
-  asm("mov.b64 {%0, %1}, %2;" : "=f"(r.x), "=f"(r.y) : "l"(v));
-  return r;
-}
-__device__ __forceinline__ uint64_t fma2(uint64_t a, uint64_t b, uint64_t c) {
-  uint64_t d;
-  asm("fma.rn.f32x2 %0, %1, %2, %3;" : "=l"(d) : "l"(a), "l"(b), "l"(c));
-  return d;
-}
-__device__ __forceinline__ uint64_t mul2(uint64_t a, uint64_t b) {
-  uint64_t d;
-  asm("mul.rn.f32x2 %0, %1, %2;" : "=l"(d) : "l"(a), "l"(b));
-  return d;
-}
-
 // One (segment, head) per CTA.  D: head dimension padded to 32, 64 or 128.  Thread (kg, vg) owns keys kg * KT ..., values
 // vg * 4 ... of the head's matrix, as pairs of neighbouring keys.
 template <int D> struct MixCfg {
@@ -329,7 +338,7 @@ constexpr int kMixRows = 16;      // rows staged in shared memory at a time
 
 // v8: 8-element loads are aligned; s4: rows of the state are multiples of 16 bytes
 template <typename T, int D, bool OUT>
-__global__ void __launch_bounds__(MixCfg<D>::kThreads) time_mix_segment_kernel(const MixParams<T> p, int v8, int s4) {
+__global__ void __launch_bounds__(MixCfg<D>::kThreads, sizeof(T) == 2 ? 512 / MixCfg<D>::kThreads : 1) time_mix_segment_kernel(const MixParams<T> p, int v8, int s4) {
   using C = MixCfg<D>;
   constexpr int KT = C::KT, KG = C::KG, SEG = C::SEG, ROW = C::ROW, NT = C::kThreads;
   __shared__ __align__(16) float sK[kMixRows][ROW], sW[kMixRows][ROW], sV[kMixRows][D];
@@ -381,10 +390,14 @@ __global__ void __launch_bounds__(MixCfg<D>::kThreads) time_mix_segment_kernel(c
     }
   }
   float prod = 1.f;                                       // !OUT: decay of key `tid` over the segment
-  float nw[D / 32];
+  float nw[D / 32], un[D / 32];
   if (OUT) {
 #pragma unroll
-    for (int i = 0; i < D / 32; ++i) nw[i] = lane + 32 * i < d ? to_f32(p.norm_w[h * d + lane + 32 * i]) * p.scale : 0.f;
+    for (int i = 0; i < D / 32; ++i) {
+      const int c = lane + 32 * i;
+      nw[i] = c < d ? to_f32(p.norm_w[h * d + c]) * p.scale : 0.f;
+      un[i] = c < d ? p.u[h * d + c] : 0.f;
+    }
   }
   // rows of this head on their way: vector i * NT + tid of the [row][8 columns] tile (v8 only)
   constexpr int NV = kMixRows * (D / 8) / NT;
@@ -445,13 +458,22 @@ __global__ void __launch_bounds__(MixCfg<D>::kThreads) time_mix_segment_kernel(c
     }
     __syncthreads();
     if (v8 && b + kMixRows < n) fetch(b + kMixRows);
+    constexpr int RW = kMixRows / (NT / 32);               // rows that a warp finishes: warp, warp + NT / 32, ...
+    T gate[OUT ? RW : 1][D / 32];
     if (OUT) {
+#pragma unroll
+      for (int i = 0; i < RW; ++i)
+#pragma unroll
+        for (int j = 0; j < D / 32; ++j) {
+          const int row = warp + i * (NT / 32), c = lane + 32 * j;
+          if (row < m && c < d) gate[OUT ? i : 0][j] = p.gate[size_t(t0 + b + row) * p.ldg + size_t(h) * d + c];
+        }
       for (int row = warp; row < m; row += NT / 32) {
         float s = 0.f;
 #pragma unroll
         for (int i = 0; i < D / 32; ++i) {
           const int c = lane + 32 * i, at = c / KT * SEG + c % KT;
-          if (c < d) s += sR[row][at] * p.u[h * d + c] * sK[row][at];
+          s += sR[row][at] * un[i] * sK[row][at];
         }
         s = warp_sum(s);
         if (lane == 0) sBonus[row] = s;                    // read behind the next barrier
@@ -500,7 +522,10 @@ __global__ void __launch_bounds__(MixCfg<D>::kThreads) time_mix_segment_kernel(c
     }
     __syncthreads();
     if (OUT) {
-      for (int row = warp; row < m; row += NT / 32) {
+#pragma unroll
+      for (int k = 0; k < RW; ++k) {
+        const int row = warp + k * (NT / 32);
+        if (row >= m) break;
         const size_t t = size_t(t0 + b + row);
         float o[D / 32], ss = 0.f;
 #pragma unroll
@@ -514,8 +539,7 @@ __global__ void __launch_bounds__(MixCfg<D>::kThreads) time_mix_segment_kernel(c
         for (int i = 0; i < D / 32; ++i) {
           const int c = lane + 32 * i;
           if (c < d)
-            from_f32(p.out + t * p.ldo + size_t(h) * d + c,
-                     o[i] * inv * nw[i] * act_silu(to_f32(p.gate[t * p.ldg + size_t(h) * d + c])));
+            from_f32(p.out + t * p.ldo + size_t(h) * d + c, o[i] * inv * nw[i] * act_silu(to_f32(gate[OUT ? k : 0][i])));
         }
       }
       __syncthreads();
@@ -575,15 +599,25 @@ __global__ void __launch_bounds__(256) time_mix_chain_kernel(const MixParams<T> 
     float s = cont ? rec[e] : 0.f;
     float* ws = p.ws_s + (size_t(base) * p.H + h) * mat + e;
     const float* pr = p.ws_p + (size_t(base) * p.H + h) * d + e / d;
-#pragma unroll 4
-    for (int g = 0; g < n_seg - 1; ++g) {
-      const float add = *ws;
-      *ws = s;
-      s = fmaf(*pr, s, add);
-      ws += step;
-      pr += size_t(p.H) * d;
+    constexpr int kGroup = 8;
+    const size_t pstep = size_t(p.H) * d;
+    for (int g = 0; g < n_seg; g += kGroup) {              // the last segment only takes its start
+      float add[kGroup], f[kGroup];
+#pragma unroll
+      for (int i = 0; i < kGroup; ++i)
+        if (g + i < n_seg - 1) {
+          add[i] = ws[i * step];
+          f[i] = pr[i * pstep];
+        }
+#pragma unroll
+      for (int i = 0; i < kGroup; ++i)
+        if (g + i < n_seg) {
+          ws[i * step] = s;
+          if (g + i < n_seg - 1) s = fmaf(f[i], s, add[i]);
+        }
+      ws += kGroup * step;
+      pr += kGroup * pstep;
     }
-    *ws = s;
   }
 }
 
@@ -747,7 +781,7 @@ static int launch_time_mix(MixParams<T> p, int seg_cap, int has_long, int has_si
 #define XL_MIX(D, OUT) time_mix_segment_kernel<T, D, OUT><<<grid, MixCfg<D>::kThreads, 0, st>>>(p, v8, s4)
       if (p.ws_s) {
         if (d <= 32) XL_MIX(32, false); else if (d <= 64) XL_MIX(64, false); else XL_MIX(128, false);
-        const int parts = (d * d + 1023) / 1024;
+        const int parts = (d * d + 255) / 256;
         time_mix_chain_kernel<T><<<dim3(p.q.n, p.H, parts), 256, 0, st>>>(p);
       }
       if (d <= 32) XL_MIX(32, true); else if (d <= 64) XL_MIX(64, true); else XL_MIX(128, true);
@@ -847,17 +881,21 @@ __global__ void __launch_bounds__(kScanThreads) scan_rows_kernel(const ScanParam
   const int ch = tid / LPC, ln = tid % LPC, n0 = ln * NPT;
   const int c = blockIdx.x * CPB + ch;
   const bool live = c < p.C;
-  float S[NPT], A[NPT], bias = 0.f, D = 0.f;
+  float s0[NPT], a0[NPT], bias = 0.f, D = 0.f;
 #pragma unroll
-  for (int i = 0; i < NPT; ++i) S[i] = A[i] = 0.f;
+  for (int i = 0; i < NPT; ++i) s0[i] = a0[i] = 0.f;
   float* rec = p.state + (size_t(slot) * p.C + c) * p.N;
   if (live) {
-    load_states<NPT>(p.A + size_t(c) * p.N, n0, p.N, A);
-    if (cont) load_states<NPT>(rec, n0, p.N, S);
-#pragma unroll
-    for (int i = 0; i < NPT; ++i) A[i] *= scan_unit<T>();
+    load_states<NPT>(p.A + size_t(c) * p.N, n0, p.N, a0);
+    if (cont) load_states<NPT>(rec, n0, p.N, s0);
     bias = p.dt_bias[c];
     D = p.D[c];
+  }
+  uint64_t S[NPT / 2], A[NPT / 2];                         // pairs of neighbouring states
+#pragma unroll
+  for (int i = 0; i < NPT / 2; ++i) {
+    S[i] = pack2(s0[2 * i], s0[2 * i + 1]);
+    A[i] = pack2(a0[2 * i] * scan_unit<T>(), a0[2 * i + 1] * scan_unit<T>());
   }
   float rdt[G];
   T rx[G], rz[G], rb[kAheadB ? NB : 1];
@@ -920,21 +958,20 @@ __global__ void __launch_bounds__(kScanThreads) scan_rows_kernel(const ScanParam
         const float dtl = LPC == 1 ? dt[g] : __shfl_sync(0xffffffffu, dt[g], l, LPC);
         const float dxl = LPC == 1 ? dx : __shfl_sync(0xffffffffu, dx, l, LPC);
         const float* bc = &sBC[buf][g * LPC + l][n0];
-        float acc[4] = {0.f, 0.f, 0.f, 0.f};
+        const uint64_t dt2 = pack2(dtl, dtl), dx2 = pack2(dxl, dxl);
+        uint64_t acc[2] = {0, 0};
 #pragma unroll
-        for (int i = 0; i < NPT; i += 4) {
-          const float4 bb = *reinterpret_cast<const float4*>(bc + i);
-          const float4 cm = *reinterpret_cast<const float4*>(bc + NP + i);
-          S[i] = fmaf(scan_decay<T>(dtl * A[i]), S[i], dxl * bb.x);
-          S[i + 1] = fmaf(scan_decay<T>(dtl * A[i + 1]), S[i + 1], dxl * bb.y);
-          S[i + 2] = fmaf(scan_decay<T>(dtl * A[i + 2]), S[i + 2], dxl * bb.z);
-          S[i + 3] = fmaf(scan_decay<T>(dtl * A[i + 3]), S[i + 3], dxl * bb.w);
-          acc[0] = fmaf(S[i], cm.x, acc[0]);
-          acc[1] = fmaf(S[i + 1], cm.y, acc[1]);
-          acc[2] = fmaf(S[i + 2], cm.z, acc[2]);
-          acc[3] = fmaf(S[i + 3], cm.w, acc[3]);
+        for (int i = 0; i < NPT / 2; i += 2) {
+          const ulonglong2 bb = *reinterpret_cast<const ulonglong2*>(bc + 2 * i);
+          const ulonglong2 cm = *reinterpret_cast<const ulonglong2*>(bc + NP + 2 * i);
+          const float2 e0 = unpack2(mul2(dt2, A[i])), e1 = unpack2(mul2(dt2, A[i + 1]));
+          S[i] = fma2(pack2(scan_decay<T>(e0.x), scan_decay<T>(e0.y)), S[i], mul2(dx2, bb.x));
+          S[i + 1] = fma2(pack2(scan_decay<T>(e1.x), scan_decay<T>(e1.y)), S[i + 1], mul2(dx2, bb.y));
+          acc[0] = fma2(S[i], cm.x, acc[0]);
+          acc[1] = fma2(S[i + 1], cm.y, acc[1]);
         }
-        y[l] = (acc[0] + acc[1]) + (acc[2] + acc[3]);
+        const float2 f0 = unpack2(acc[0]), f1 = unpack2(acc[1]);
+        y[l] = (f0.x + f0.y) + (f1.x + f1.y);
       }
       const float sum = sum_to_lanes<LPC>(y, ln);
       const int row = g * LPC + ln;
@@ -943,12 +980,21 @@ __global__ void __launch_bounds__(kScanThreads) scan_rows_kernel(const ScanParam
     if (NBUF == 1) __syncthreads();
     if (b + kScanRows < len) put(b + kScanRows, buf ^ (NBUF - 1));
   }
-  if (live) store_states<NPT>(rec, n0, p.N, S);
+  if (live) {
+#pragma unroll
+    for (int i = 0; i < NPT / 2; ++i) {
+      const float2 f = unpack2(S[i]);
+      s0[2 * i] = f.x;
+      s0[2 * i + 1] = f.y;
+    }
+    store_states<NPT>(rec, n0, p.N, s0);
+  }
 }
 
-// Single rows: LPC lanes per channel, NPT states each, and kScanSeqs sequences per thread, so that A is read once for them and
-// the states of all of them are under way before any is worked on.  bc4: B and C can be read four at a time.
-constexpr int kScanSeqs = 4;
+// Single rows: LPC lanes per channel, NPT states each, and several sequences per thread, so that A is read once for them and
+// the states of all of them are under way before any is worked on.  Lane k prepares and finishes sequence k.  bc4: B and C can
+// be read four at a time.
+template <int NPT, int LPC> struct SingleCfg { static constexpr int NS = NPT > 4 ? 1 : LPC < 8 ? LPC : 8; };
 template <typename T>
 __device__ __forceinline__ void load_bc4(const T* p, float* f) {
   if constexpr (sizeof(T) == 2) {
@@ -961,37 +1007,43 @@ __device__ __forceinline__ void load_bc4(const T* p, float* f) {
 }
 template <typename T, int NPT, int LPC>
 __global__ void __launch_bounds__(kScanThreads) scan_single_kernel(const ScanParams<T> p, int bc4) {
-  constexpr int CPB = kScanThreads / LPC;
-  constexpr int NS = NPT > 4 ? 1 : kScanSeqs;
+  constexpr int CPB = kScanThreads / LPC, NS = SingleCfg<NPT, LPC>::NS;
   const int tid = threadIdx.x, ch = tid / LPC, ln = tid % LPC, n0 = ln * NPT;
   const int c = blockIdx.x * CPB + ch;
   const bool live = c < p.C;
-  int t[NS], slot[NS];
-  bool cont[NS], any = false;
-#pragma unroll
-  for (int k = 0; k < NS; ++k) {
-    const int seq = blockIdx.y * NS + k;
-    t[k] = seq < p.q.n ? p.q.q_cu[seq] : 0;
-    slot[k] = -1;
-    cont[k] = false;
-    if (seq < p.q.n && p.q.q_cu[seq + 1] - t[k] == 1) {
-      slot[k] = record_of(p.q, seq);
-      cont[k] = p.q.kv_lens[seq] > 1;
+  // this lane's sequence
+  const int own = ln % NS, my_seq = blockIdx.y * NS + own;
+  int my_t = 0, my_slot = -1;
+  bool my_cont = false;
+  if (my_seq < p.q.n) {
+    my_t = p.q.q_cu[my_seq];
+    if (p.q.q_cu[my_seq + 1] - my_t == 1) {
+      my_slot = p.q.slots[my_seq];
+      my_cont = p.q.kv_lens[my_seq] > 1;
+      if (my_slot < 0 || my_slot >= p.q.n_slots) {
+        if (tid < NS) atomicExch(p.q.status, XL_ERR_BOUNDS);
+        my_slot = -1;
+      }
     }
-    any |= slot[k] >= 0;
   }
-  if (!any) return;
-  float S[NS][NPT], A[NPT], dt[NS], x[NS], bias = 0.f, D = 0.f;
+  if (!__any_sync(0xffffffffu, my_slot >= 0)) return;
+  const bool mine = live && my_slot >= 0;
+  float dt = 0.f, x = 0.f, z = 0.f, bias = 0.f, D = 0.f;
+  if (mine) {
+    dt = p.dt[size_t(my_t) * p.C + c];
+    x = to_f32(p.x[size_t(my_t) * p.C + c]);
+    z = to_f32(p.z[size_t(my_t) * p.ldz + c]);
+  }
+  float S[NS][NPT], A[NPT];
+  int t[NS], slot[NS];
 #pragma unroll
   for (int k = 0; k < NS; ++k) {
-    dt[k] = x[k] = 0.f;
+    t[k] = __shfl_sync(0xffffffffu, my_t, k, LPC);
+    slot[k] = __shfl_sync(0xffffffffu, my_slot, k, LPC);
+    const bool cont = __shfl_sync(0xffffffffu, int(my_cont), k, LPC);
 #pragma unroll
     for (int i = 0; i < NPT; ++i) S[k][i] = 0.f;
-    if (live && slot[k] >= 0) {
-      if (cont[k]) load_states<NPT>(p.state + (size_t(slot[k]) * p.C + c) * p.N, n0, p.N, S[k]);
-      dt[k] = p.dt[size_t(t[k]) * p.C + c];
-      x[k] = to_f32(p.x[size_t(t[k]) * p.C + c]);
-    }
+    if (live && slot[k] >= 0 && cont) load_states<NPT>(p.state + (size_t(slot[k]) * p.C + c) * p.N, n0, p.N, S[k]);
   }
 #pragma unroll
   for (int i = 0; i < NPT; ++i) A[i] = 0.f;
@@ -999,59 +1051,47 @@ __global__ void __launch_bounds__(kScanThreads) scan_single_kernel(const ScanPar
     load_states<NPT>(p.A + size_t(c) * p.N, n0, p.N, A);
     bias = p.dt_bias[c];
     D = p.D[c];
+#pragma unroll
+    for (int i = 0; i < NPT; ++i) A[i] *= scan_unit<T>();
   }
+  const float step = softplus(dt + bias), dx = step * x;
   float y[NS];
 #pragma unroll
   for (int k = 0; k < NS; ++k) {
     y[k] = 0.f;
+    const float step_k = __shfl_sync(0xffffffffu, step, k, LPC), dx_k = __shfl_sync(0xffffffffu, dx, k, LPC);
     if (slot[k] < 0) continue;                             // the same in every lane
     float B[NPT], Cm[NPT];
     const T *bp = p.B + size_t(t[k]) * p.ldb + n0, *cp = p.Cm + size_t(t[k]) * p.ldb + n0;
 #pragma unroll
     for (int i = 0; i < NPT; i += 4) {
-      if (bc4) {
 #pragma unroll
-        for (int e = 0; e < 4; ++e) B[i + e] = Cm[i + e] = 0.f;
+      for (int e = 0; e < 4; ++e) B[i + e] = Cm[i + e] = 0.f;
+      if (bc4) {
         if (n0 + i < p.N) {
           load_bc4(bp + i, B + i);
           load_bc4(cp + i, Cm + i);
         }
       } else {
 #pragma unroll
-        for (int e = 0; e < 4; ++e) {
-          const bool in = n0 + i + e < p.N;
-          B[i + e] = in ? to_f32(bp[i + e]) : 0.f;
-          Cm[i + e] = in ? to_f32(cp[i + e]) : 0.f;
-        }
+        for (int e = 0; e < 4; ++e)
+          if (n0 + i + e < p.N) {
+            B[i + e] = to_f32(bp[i + e]);
+            Cm[i + e] = to_f32(cp[i + e]);
+          }
       }
     }
-    const float step = softplus(dt[k] + bias), dx = step * x[k];
 #pragma unroll
     for (int i = 0; i < NPT; ++i) {
-      S[k][i] = fmaf(scan_decay<T>(step * (A[i] * scan_unit<T>())), S[k][i], dx * B[i]);
+      S[k][i] = fmaf(scan_decay<T>(step_k * A[i]), S[k][i], dx_k * B[i]);
       y[k] = fmaf(S[k][i], Cm[i], y[k]);
     }
     if (live) store_states<NPT>(p.state + (size_t(slot[k]) * p.C + c) * p.N, n0, p.N, S[k]);
   }
-  if constexpr (NS == LPC) {                               // lane k finishes sequence k
-    const float xs[4] = {x[0], x[NS > 1 ? 1 : 0], x[NS > 2 ? 2 : 0], x[NS > 3 ? 3 : 0]};
-    const float sum = sum_to_lanes<NS>(y, ln);
-    int tk = t[0], sk = slot[0];
-    float xk = xs[0];
+  float sum = sum_to_lanes<NS>(y, ln);
 #pragma unroll
-    for (int k = 1; k < NS; ++k)
-      if (ln == k) { tk = t[k]; sk = slot[k]; xk = xs[k]; }
-    if (live && sk >= 0)
-      from_f32(p.out + size_t(tk) * p.C + c, fmaf(D, xk, sum) * act_silu(to_f32(p.z[size_t(tk) * p.ldz + c])));
-  } else {
-#pragma unroll
-    for (int k = 0; k < NS; ++k) {
-#pragma unroll
-      for (int o = 1; o < LPC; o <<= 1) y[k] += __shfl_xor_sync(0xffffffffu, y[k], o);
-      if (live && ln == 0 && slot[k] >= 0)
-        from_f32(p.out + size_t(t[k]) * p.C + c, fmaf(D, x[k], y[k]) * act_silu(to_f32(p.z[size_t(t[k]) * p.ldz + c])));
-    }
-  }
+  for (int o = NS; o < LPC; o <<= 1) sum += __shfl_xor_sync(0xffffffffu, sum, o);
+  if (mine && ln < NS) from_f32(p.out + size_t(my_t) * p.C + c, fmaf(D, x, sum) * act_silu(z));
 }
 
 template <typename T, int NPT, int LPC>
@@ -1063,7 +1103,7 @@ static int launch_rows(const ScanParams<T>& p, cudaStream_t st) {
 template <typename T, int NPT, int LPC>
 static int launch_single(const ScanParams<T>& p, cudaStream_t st) {
   constexpr int CPB = kScanThreads / LPC;
-  constexpr int NS = NPT > 4 ? 1 : kScanSeqs;
+  constexpr int NS = SingleCfg<NPT, LPC>::NS;
   const int bytes = 4 * int(sizeof(T));
   const bool bc4 = p.N % 4 == 0 && (p.ldb * sizeof(T)) % bytes == 0 && reinterpret_cast<uintptr_t>(p.B) % bytes == 0 &&
                    reinterpret_cast<uintptr_t>(p.Cm) % bytes == 0;
@@ -1087,7 +1127,8 @@ static int launch_scan(const ScanParams<T>& p, int has_long, int has_single, cud
   if (rc || !has_long) return rc;
   if (n <= 4) return launch_rows<T, 4, 1>(p, st);
   if (n <= 8) return launch_rows<T, 8, 1>(p, st);
-  if (n <= 16) return launch_rows<T, 8, 2>(p, st);
+  // few channels x sequences: more lanes per channel, so that every scheduler has more than one warp
+  if (n <= 16) return long(p.C) * p.q.n <= 4096 * 3 ? launch_rows<T, 4, 4>(p, st) : launch_rows<T, 8, 2>(p, st);
   if (n <= 32) return launch_rows<T, 8, 4>(p, st);
   if (n <= 64) return launch_rows<T, 8, 8>(p, st);
   if (n <= 128) return launch_rows<T, 16, 8>(p, st);
