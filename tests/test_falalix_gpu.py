@@ -136,11 +136,14 @@ def test_conv(C, taps, dtype, steps, pad):
     assert status_ok()
 
 
+@pytest.mark.parametrize("rows", [0, 48])
 @pytest.mark.parametrize("pad", [0, 5])
 @pytest.mark.parametrize("steps", [0, 1, 2])
 @pytest.mark.parametrize("H,d", [(3, 64), (2, 32), (2, 128), (3, 48), (1, 8), (2, 96), (3, 21), (2, 9), (1, 160), (2, 132), (1, 139)])
 @pytest.mark.parametrize("dtype", DTYPES)
-def test_time_mix(H, d, dtype, steps, pad):
+def test_time_mix(H, d, dtype, steps, pad, rows, monkeypatch):
+    from xllm_wxh_b200.ops import cuda_ops
+    monkeypatch.setattr(cuda_ops, "mix_force_rows", rows)        # rows per segment of longer portions (0: chosen)
     g = torch.Generator().manual_seed(H * d)
     n_ = H * d
     r, k, v, gate = ([torch.randn(n, n_, generator=g).to(dtype) for n in LENS] for _ in range(4))
@@ -164,14 +167,14 @@ def test_time_mix(H, d, dtype, steps, pad):
     assert (state[0] == 1e4).all() and status_ok()
 
 
-def test_time_mix_of_long_and_many_portions():
+@pytest.mark.parametrize("rows", [0, 64, 16, 2, 130])
+def test_time_mix_of_long_and_many_portions(rows, monkeypatch):
     """Segments: several per sequence, sequences of all lengths around a segment's, more sequences than a warp has lanes."""
     H, d = 2, 64
     g = torch.Generator().manual_seed(0)
     from xllm_wxh_b200.ops import cuda_ops
+    monkeypatch.setattr(cuda_ops, "mix_force_rows", rows)
     lens = [900, 64, 65, 63, 128, 129, 2, 1, 3] + [2 + i % 5 for i in range(60)]
-    L = cuda_ops.mix_segment_rows(sum(lens), H, d)
-    assert 2 <= L < 300
     r, k, v, gate, z = ([torch.randn(n, H * d, generator=g) for n in lens] for _ in range(5))
     w0, u, nw = torch.rand(H * d, generator=g) * 5 - 6, torch.randn(H, d, generator=g), torch.ones(H * d)
     rg = Ragged(lens, [lens], n_slots=100)

@@ -42,7 +42,19 @@ __device__ __forceinline__ float ex2(float x) {
   asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
   return y;
 }
-__device__ __forceinline__ float softplus(float z) { return z > 20.f ? z : log1pf(__expf(z)); }
+// log(1 + e^z) = max(z, 0) + log(1 + t), t = e^-|z| in (0, 1]; log(1 + t) = 2 artanh(s), s = t / (2 + t) <= 1 / 3, by its power
+// series, which keeps the relative accuracy of small results (the next term is below 3e-9 of the sum).
+__device__ __forceinline__ float softplus(float z) {
+  const float t = __expf(-fabsf(z)), s = __fdividef(t, 2.f + t), q = s * s;
+  float p = 1.f / 15.f;
+  p = fmaf(p, q, 1.f / 13.f);
+  p = fmaf(p, q, 1.f / 11.f);
+  p = fmaf(p, q, 1.f / 9.f);
+  p = fmaf(p, q, 1.f / 7.f);
+  p = fmaf(p, q, 1.f / 5.f);
+  p = fmaf(p, q, 1.f / 3.f);
+  return fmaxf(z, 0.f) + 2.f * s * fmaf(p, q, 1.f);
+}
 // exp(x), x <= 0: the factor a state is multiplied by at every token, so its error adds up over the tokens that the state
 // remembers.  Models in 32-bit take the one that is exact to the last place near 1.
 template <typename T>
@@ -84,6 +96,22 @@ __device__ __forceinline__ uint64_t mul2(uint64_t a, uint64_t b) {
   uint64_t d;
   asm("mul.rn.f32x2 %0, %1, %2;" : "=l"(d) : "l"(a), "l"(b));
   return d;
+}
+
+// Sums y[0 .. LPC) over LPC neighbouring lanes (ln: place among them); lane l ends with the sum of y[l].  Halves the number of values with
+// every exchange.
+template <int LPC>
+__device__ __forceinline__ float sum_to_lanes(float (&y)[LPC], int ln) {
+#pragma unroll
+  for (int o = LPC / 2; o > 0; o >>= 1) {
+    const bool up = ln & o;
+#pragma unroll
+    for (int i = 0; i < o; ++i) {
+      const float send = up ? y[i] : y[i + o];
+      y[i] = (up ? y[i + o] : y[i]) + __shfl_xor_sync(0xffffffffu, send, o);
+    }
+  }
+  return y[0];
 }
 
 // Eight elements as they come from memory, converted when they are used.
@@ -161,7 +189,7 @@ __global__ void __launch_bounds__(256) token_shift_kernel(const T* __restrict__ 
 constexpr int kConvRows = 16, kConvRowsSingle = 2;
 
 template <typename T, int V, int TAPS, int ROWS>
-__global__ void __launch_bounds__(128, sizeof(T) == 2 ? 6 : 1) conv_silu_kernel(const T* __restrict__ x, const T* __restrict__ w, const T* __restrict__ bias,
+__global__ void __launch_bounds__(128, sizeof(T) == 2 ? 5 : 1) conv_silu_kernel(const T* __restrict__ x, const T* __restrict__ w, const T* __restrict__ bias,
                                                         T* __restrict__ state, T* __restrict__ out, const int* __restrict__ token_seq,
                                                         const Seqs q, int rows, int C, int taps_rt, long ldx) {
   constexpr int H = TAPS > 1 ? TAPS - 1 : 1;
@@ -328,21 +356,37 @@ __device__ __forceinline__ bool find_segment(const Seqs& q, int L, int target, i
 }
 
 // One (segment, head) per CTA.  D: head dimension padded to 32, 64 or 128.  Thread (kg, vg) owns keys kg * KT ..., values
-// vg * 4 ... of the head's matrix, as pairs of neighbouring keys.
+// vg * VT ... of the head's matrix, as pairs of neighbouring keys: the more of both, the fewer reads of shared memory per
+// element, which bound this kernel beside the multiply-adds.
 template <int D> struct MixCfg {
-  static constexpr int KT = D == 128 ? 16 : 8;
-  static constexpr int KG = D / KT, VG = D / 4, kThreads = KG * VG;
-  static constexpr int SEG = KT + 4, ROW = KG * SEG;      // key groups 4 floats apart, so that their reads meet no bank twice
+  static constexpr int KT = D == 32 ? 4 : 8, VT = 8;
+  static constexpr int KG = D / KT, VG = D / VT, kThreads = KG * VG;
+  static constexpr int kMinBlocks = D == 128 ? 1 : D == 64 ? 5 : 12;
+  // Place of key c in a row of shared memory.  Eight key groups are read at a time, four keys of each: with eight keys per
+  // group every other four groups have their halves swapped, so that the reads meet no bank twice.
+  __device__ static constexpr int key_at(int c) { return KT == 4 ? c : c ^ (((c >> 5) & 1) << 2); }
 };
+// Eight keys from c (a multiple of 8) on.
+template <int D>
+__device__ __forceinline__ void store_keys(float* row, int c, const float (&f)[8]) {
+  *reinterpret_cast<float4*>(row + MixCfg<D>::key_at(c)) = make_float4(f[0], f[1], f[2], f[3]);
+  *reinterpret_cast<float4*>(row + MixCfg<D>::key_at(c + 4)) = make_float4(f[4], f[5], f[6], f[7]);
+}
+template <int D>
+__device__ __forceinline__ void load_keys(const float* row, int c, float (&f)[8]) {
+  *reinterpret_cast<float4*>(f) = *reinterpret_cast<const float4*>(row + MixCfg<D>::key_at(c));
+  *reinterpret_cast<float4*>(f + 4) = *reinterpret_cast<const float4*>(row + MixCfg<D>::key_at(c + 4));
+}
 constexpr int kMixRows = 16;      // rows staged in shared memory at a time
 
-// v8: 8-element loads are aligned; s4: rows of the state are multiples of 16 bytes
+// v8, g8: 8-element accesses to the inputs / to gate and output are aligned; s4: rows of the state are multiples of 16 bytes
 template <typename T, int D, bool OUT>
-__global__ void __launch_bounds__(MixCfg<D>::kThreads, sizeof(T) == 2 ? 512 / MixCfg<D>::kThreads : 1) time_mix_segment_kernel(const MixParams<T> p, int v8, int s4) {
+__global__ void __launch_bounds__(MixCfg<D>::kThreads, sizeof(T) == 2 ? MixCfg<D>::kMinBlocks : 1) time_mix_segment_kernel(const MixParams<T> p, int v8, int g8, int s4) {
   using C = MixCfg<D>;
-  constexpr int KT = C::KT, KG = C::KG, SEG = C::SEG, ROW = C::ROW, NT = C::kThreads;
-  __shared__ __align__(16) float sK[kMixRows][ROW], sW[kMixRows][ROW], sV[kMixRows][D];
-  __shared__ __align__(16) float sR[OUT ? kMixRows : 1][ROW], sO[OUT ? kMixRows : 1][D];
+  constexpr int KT = C::KT, VT = C::VT, KG = C::KG, NT = C::kThreads;
+  __shared__ __align__(16) float sK[kMixRows][D], sW[kMixRows][D], sV[kMixRows][D];
+  __shared__ __align__(16) float sR[OUT ? kMixRows : 1][D], sO[OUT ? kMixRows : 1][D];
+  __shared__ __align__(16) float sNw[OUT ? D : 1], sU[OUT ? D : 1];
   __shared__ float sBonus[kMixRows];
   int seq, seg, n_seg;
   if (!find_segment(p.q, p.L, blockIdx.x, seq, seg, n_seg)) return;
@@ -362,41 +406,45 @@ __global__ void __launch_bounds__(MixCfg<D>::kThreads, sizeof(T) == 2 ? 512 / Mi
   float* rec = p.state + (size_t(slot) * p.H + h) * mat;
   float* seg_s = p.ws_s ? p.ws_s + (size_t(blockIdx.x) * p.H + h) * mat : nullptr;
 
-  uint64_t S[KT / 2][4];
+  uint64_t S[KT / 2][VT];
 #pragma unroll
   for (int i = 0; i < KT / 2; ++i)
 #pragma unroll
-    for (int j = 0; j < 4; ++j) S[i][j] = 0;
+    for (int j = 0; j < VT; ++j) S[i][j] = 0;
   if (OUT && (n_seg > 1 || cont)) {
     const float* src = n_seg > 1 ? seg_s : rec;
 #pragma unroll
     for (int i = 0; i < KT / 2; ++i) {
-      float a[2][4] = {};
+      float a[2][VT] = {};
 #pragma unroll
       for (int e = 0; e < 2; ++e) {
         const int key = kg * KT + 2 * i + e;
         if (key < d) {
-          if (s4) {
-            if (vg * 4 < d) *reinterpret_cast<float4*>(a[e]) = *reinterpret_cast<const float4*>(src + size_t(key) * d + vg * 4);
-          } else {
+          const float* row = src + size_t(key) * d + vg * VT;
 #pragma unroll
-            for (int j = 0; j < 4; ++j)
-              if (vg * 4 + j < d) a[e][j] = src[size_t(key) * d + vg * 4 + j];
+          for (int j = 0; j < VT; j += 4) {
+            if (s4) {
+              if (vg * VT + j < d) *reinterpret_cast<float4*>(a[e] + j) = *reinterpret_cast<const float4*>(row + j);
+            } else {
+#pragma unroll
+              for (int l = j; l < j + 4; ++l)
+                if (vg * VT + l < d) a[e][l] = row[l];
+            }
           }
         }
       }
 #pragma unroll
-      for (int j = 0; j < 4; ++j) S[i][j] = pack2(a[0][j], a[1][j]);
+      for (int j = 0; j < VT; ++j) S[i][j] = pack2(a[0][j], a[1][j]);
     }
   }
   float prod = 1.f;                                       // !OUT: decay of key `tid` over the segment
-  float nw[D / 32], un[D / 32];
-  if (OUT) {
-#pragma unroll
-    for (int i = 0; i < D / 32; ++i) {
-      const int c = lane + 32 * i;
-      nw[i] = c < d ? to_f32(p.norm_w[h * d + c]) * p.scale : 0.f;
-      un[i] = c < d ? p.u[h * d + c] : 0.f;
+  // Rows are finished (and their bonus is prepared) by vectors of 8 columns: LR lanes per row, RP rows per warp and pass.
+  constexpr int LR = D / 8, RP = 32 / LR, PASSES = kMixRows / (NT / 32 * RP);
+  const int fr_row = warp * RP + lane / LR, fr_c = lane % LR * 8;
+  if (OUT) {                                              // visible behind the first tile's barrier
+    for (int c = tid; c < D; c += NT) {
+      sNw[OUT ? c : 0] = c < d ? to_f32(p.norm_w[h * d + c]) * p.scale : 0.f;
+      sU[OUT ? c : 0] = c < d ? p.u[h * d + c] : 0.f;
     }
   }
   // rows of this head on their way: vector i * NT + tid of the [row][8 columns] tile (v8 only)
@@ -438,18 +486,17 @@ __global__ void __launch_bounds__(MixCfg<D>::kThreads, sizeof(T) == 2 ? 512 / Mi
 #pragma unroll
           for (int j = 0; j < 8; ++j) w[j] = decay_of<T>(w[j] + w0[j]);
         }
-        const int at = c / KT * SEG + c % KT;
-        store8(&sK[row][at], k);
-        store8(&sW[row][at], w);
+        store_keys<D>(sK[row], c, k);
+        store_keys<D>(sW[row], c, w);
         store8(&sV[row][c], v);
-        if (OUT) store8(&sR[row][at], r);
+        if (OUT) store_keys<D>(sR[row], c, r);
       }
     } else {
       for (int i = tid; i < kMixRows * D; i += NT) {
         const int row = i / D, c = i % D;
         const bool in = row < m && c < d;
         const size_t t = size_t(t0 + b + row), at = t * p.ld + size_t(h) * d + c;
-        const int to = c / KT * SEG + c % KT;
+        const int to = C::key_at(c);
         sK[row][to] = in ? to_f32(p.k[at]) : 0.f;
         sV[row][c] = in ? to_f32(p.v[at]) : 0.f;
         sW[row][to] = in ? decay_of<T>(p.z[t * (size_t(p.H) * d) + size_t(h) * d + c] + p.w0[h * d + c]) : 1.f;
@@ -458,88 +505,100 @@ __global__ void __launch_bounds__(MixCfg<D>::kThreads, sizeof(T) == 2 ? 512 / Mi
     }
     __syncthreads();
     if (v8 && b + kMixRows < n) fetch(b + kMixRows);
-    constexpr int RW = kMixRows / (NT / 32);               // rows that a warp finishes: warp, warp + NT / 32, ...
-    T gate[OUT ? RW : 1][D / 32];
+    Vec8<T> gate[OUT ? PASSES : 1];
     if (OUT) {
 #pragma unroll
-      for (int i = 0; i < RW; ++i)
-#pragma unroll
-        for (int j = 0; j < D / 32; ++j) {
-          const int row = warp + i * (NT / 32), c = lane + 32 * j;
-          if (row < m && c < d) gate[OUT ? i : 0][j] = p.gate[size_t(t0 + b + row) * p.ldg + size_t(h) * d + c];
-        }
-      for (int row = warp; row < m; row += NT / 32) {
+      for (int q = 0; q < PASSES; ++q) {
+        const int row = q * (NT / 32 * RP) + fr_row;
         float s = 0.f;
+        if (row < m) {
+          if (g8 && fr_c < d) gate[OUT ? q : 0].load(p.gate + size_t(t0 + b + row) * p.ldg + size_t(h) * d + fr_c);
+          float r[8], k[8], u[8];
+          load_keys<D>(sR[row], fr_c, r);
+          load_keys<D>(sK[row], fr_c, k);
+          load8(&sU[fr_c], u);
 #pragma unroll
-        for (int i = 0; i < D / 32; ++i) {
-          const int c = lane + 32 * i, at = c / KT * SEG + c % KT;
-          s += sR[row][at] * un[i] * sK[row][at];
+          for (int j = 0; j < 8; ++j) s = fmaf(r[j] * u[j], k[j], s);
         }
-        s = warp_sum(s);
-        if (lane == 0) sBonus[row] = s;                    // read behind the next barrier
+#pragma unroll
+        for (int o = LR / 2; o > 0; o >>= 1) s += __shfl_xor_sync(0xffffffffu, s, o);
+        if (lane % LR == 0 && row < m) sBonus[row] = s;    // read behind the next barrier
       }
     } else if (tid < D) {
-      for (int row = 0; row < m; ++row) prod *= sW[row][tid / KT * SEG + tid % KT];
+#pragma unroll
+      for (int row = 0; row < kMixRows; ++row) prod *= sW[row][C::key_at(tid)];
     }
-#pragma unroll 2
+#pragma unroll 1
     for (int row = 0; row < kMixRows; ++row) {
-      const float4 v4 = *reinterpret_cast<const float4*>(&sV[row][vg * 4]);
-      const uint64_t v[4] = {pack2(v4.x, v4.x), pack2(v4.y, v4.y), pack2(v4.z, v4.z), pack2(v4.w, v4.w)};
-      uint64_t o[4] = {0, 0, 0, 0};
+      float vf[8];
+      load8(&sV[row][vg * VT], vf);
+      uint64_t v[VT], o[VT];
+#pragma unroll
+      for (int j = 0; j < VT; ++j) {
+        v[j] = pack2(vf[j], vf[j]);
+        o[j] = 0;
+      }
 #pragma unroll
       for (int i = 0; i < KT / 4; ++i) {
-        const ulonglong2 k2 = *reinterpret_cast<const ulonglong2*>(&sK[row][kg * SEG + 4 * i]);
-        const ulonglong2 w2 = *reinterpret_cast<const ulonglong2*>(&sW[row][kg * SEG + 4 * i]);
+        const int at = C::key_at(kg * KT + 4 * i);
+        const ulonglong2 k2 = *reinterpret_cast<const ulonglong2*>(&sK[row][at]);
+        const ulonglong2 w2 = *reinterpret_cast<const ulonglong2*>(&sW[row][at]);
         if (OUT) {
-          const ulonglong2 r2 = *reinterpret_cast<const ulonglong2*>(&sR[row][kg * SEG + 4 * i]);
+          const ulonglong2 r2 = *reinterpret_cast<const ulonglong2*>(&sR[row][at]);
 #pragma unroll
-          for (int j = 0; j < 4; ++j) o[j] = fma2(r2.y, S[2 * i + 1][j], fma2(r2.x, S[2 * i][j], o[j]));
+          for (int j = 0; j < VT; ++j) o[j] = fma2(r2.y, S[2 * i + 1][j], fma2(r2.x, S[2 * i][j], o[j]));
         }
 #pragma unroll
-        for (int j = 0; j < 4; ++j) {
+        for (int j = 0; j < VT; ++j) {
           S[2 * i][j] = fma2(w2.x, S[2 * i][j], mul2(k2.x, v[j]));
           S[2 * i + 1][j] = fma2(w2.y, S[2 * i + 1][j], mul2(k2.y, v[j]));
         }
       }
       if (OUT) {
-        // sum over the key groups (neighbouring lanes); each of the first four ends with one of the four values
-        float y[4];
+        // sum over the key groups (neighbouring lanes); each of the first eight ends with one of the eight values
+        float y[VT];
 #pragma unroll
-        for (int j = 0; j < 4; ++j) {
+        for (int j = 0; j < VT; ++j) {
           const float2 f = unpack2(o[j]);
           y[j] = f.x + f.y;
         }
-        const bool b0 = kg & 1, b1 = kg & 2;
-        float a0 = b0 ? y[2] : y[0], a1 = b0 ? y[3] : y[1];
-        a0 += __shfl_xor_sync(0xffffffffu, b0 ? y[0] : y[2], 1);
-        a1 += __shfl_xor_sync(0xffffffffu, b0 ? y[1] : y[3], 1);
-        float a = b1 ? a1 : a0;
-        a += __shfl_xor_sync(0xffffffffu, b1 ? a0 : a1, 2);
-        if (KG == 8) a += __shfl_xor_sync(0xffffffffu, a, 4);
-        const int j = (b0 ? 2 : 0) + (b1 ? 1 : 0);
-        if (KG == 4 || kg < 4) sO[row][vg * 4 + j] = a;
+        float a = sum_to_lanes<VT>(y, kg);
+        if (KG == 16) a += __shfl_xor_sync(0xffffffffu, a, 8);
+        if (KG == 8 || kg < 8) sO[row][vg * VT + kg] = a;
       }
     }
     __syncthreads();
     if (OUT) {
 #pragma unroll
-      for (int k = 0; k < RW; ++k) {
-        const int row = warp + k * (NT / 32);
-        if (row >= m) break;
-        const size_t t = size_t(t0 + b + row);
-        float o[D / 32], ss = 0.f;
+      for (int q = 0; q < PASSES; ++q) {
+        const int row = q * (NT / 32 * RP) + fr_row;
+        const float bonus = row < m ? sBonus[row] : 0.f;
+        float o[8], ss = 0.f;
+        load8(&sO[row][fr_c], o);
 #pragma unroll
-        for (int i = 0; i < D / 32; ++i) {
-          const int c = lane + 32 * i;
-          o[i] = fmaf(sBonus[row], sV[row][c], sO[row][c]);       // zero beyond d
-          ss += o[i] * o[i];
+        for (int j = 0; j < 8; ++j) {
+          o[j] = fmaf(bonus, sV[row][fr_c + j], o[j]);            // zero beyond d
+          ss = fmaf(o[j], o[j], ss);
         }
-        const float inv = rsqrtf(warp_sum(ss) / float(d) + p.eps);
 #pragma unroll
-        for (int i = 0; i < D / 32; ++i) {
-          const int c = lane + 32 * i;
-          if (c < d)
-            from_f32(p.out + t * p.ldo + size_t(h) * d + c, o[i] * inv * nw[i] * act_silu(to_f32(gate[OUT ? k : 0][i])));
+        for (int w = LR / 2; w > 0; w >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, w);
+        const float inv = rsqrtf(ss / float(d) + p.eps);
+        if (row < m) {
+          const size_t t = size_t(t0 + b + row);
+          T* out = p.out + t * p.ldo + size_t(h) * d + fr_c;
+          float nw[8], g[8];
+          load8(&sNw[fr_c], nw);
+          if (g8) {
+            gate[OUT ? q : 0].get(g);
+#pragma unroll
+            for (int j = 0; j < 8; ++j) o[j] = o[j] * inv * nw[j] * act_silu(g[j]);
+            if (fr_c < d) store8(out, o);
+          } else {
+#pragma unroll
+            for (int j = 0; j < 8; ++j)
+              if (fr_c + j < d)
+                from_f32(out + j, o[j] * inv * nw[j] * act_silu(to_f32(p.gate[t * p.ldg + size_t(h) * d + fr_c + j])));
+          }
         }
       }
       __syncthreads();
@@ -549,9 +608,9 @@ __global__ void __launch_bounds__(MixCfg<D>::kThreads, sizeof(T) == 2 ? 512 / Mi
   float* dst = OUT ? rec : seg_s;
 #pragma unroll
   for (int i = 0; i < KT / 2; ++i) {
-    float a[2][4];
+    float a[2][VT];
 #pragma unroll
-    for (int j = 0; j < 4; ++j) {
+    for (int j = 0; j < VT; ++j) {
       const float2 f = unpack2(S[i][j]);
       a[0][j] = f.x;
       a[1][j] = f.y;
@@ -560,12 +619,16 @@ __global__ void __launch_bounds__(MixCfg<D>::kThreads, sizeof(T) == 2 ? 512 / Mi
     for (int e = 0; e < 2; ++e) {
       const int key = kg * KT + 2 * i + e;
       if (key >= d) continue;
-      if (s4) {
-        if (vg * 4 < d) *reinterpret_cast<float4*>(dst + size_t(key) * d + vg * 4) = *reinterpret_cast<const float4*>(a[e]);
-      } else {
+      float* row = dst + size_t(key) * d + vg * VT;
 #pragma unroll
-        for (int j = 0; j < 4; ++j)
-          if (vg * 4 + j < d) dst[size_t(key) * d + vg * 4 + j] = a[e][j];
+      for (int j = 0; j < VT; j += 4) {
+        if (s4) {
+          if (vg * VT + j < d) *reinterpret_cast<float4*>(row + j) = *reinterpret_cast<const float4*>(a[e] + j);
+        } else {
+#pragma unroll
+          for (int l = j; l < j + 4; ++l)
+            if (vg * VT + l < d) row[l] = a[e][l];
+        }
       }
     }
   }
@@ -765,6 +828,8 @@ static int launch_time_mix(MixParams<T> p, int seg_cap, int has_long, int has_si
   const bool v8 = d % 8 == 0 && p.ld % 8 == 0 &&
                   !((reinterpret_cast<uintptr_t>(p.r) | reinterpret_cast<uintptr_t>(p.k) | reinterpret_cast<uintptr_t>(p.v) |
                      reinterpret_cast<uintptr_t>(p.z) | reinterpret_cast<uintptr_t>(p.w0)) & 15);
+  const bool g8 = d % 8 == 0 && p.ldg % 8 == 0 && p.ldo % 8 == 0 &&
+                  !((reinterpret_cast<uintptr_t>(p.gate) | reinterpret_cast<uintptr_t>(p.out)) & 15);
   const bool s4 = d % 4 == 0;
   if (has_single) {
     const dim3 grid(p.q.n, p.H);
@@ -778,7 +843,7 @@ static int launch_time_mix(MixParams<T> p, int seg_cap, int has_long, int has_si
   if (has_long) {
     if (d <= 128) {
       const dim3 grid(seg_cap, p.H);
-#define XL_MIX(D, OUT) time_mix_segment_kernel<T, D, OUT><<<grid, MixCfg<D>::kThreads, 0, st>>>(p, v8, s4)
+#define XL_MIX(D, OUT) time_mix_segment_kernel<T, D, OUT><<<grid, MixCfg<D>::kThreads, 0, st>>>(p, v8, g8, s4)
       if (p.ws_s) {
         if (d <= 32) XL_MIX(32, false); else if (d <= 64) XL_MIX(64, false); else XL_MIX(128, false);
         const int parts = (d * d + 255) / 256;
@@ -845,33 +910,18 @@ __device__ __forceinline__ void store_states(float* p, int n0, int N, const floa
   }
 }
 
-// Sums y[0 .. LPC) over the LPC lanes of a channel; lane l ends with the sum of y[l].  Halves the number of values with
-// every exchange.
-template <int LPC>
-__device__ __forceinline__ float sum_to_lanes(float (&y)[LPC], int ln) {
-#pragma unroll
-  for (int o = LPC / 2; o > 0; o >>= 1) {
-    const bool up = ln & o;
-#pragma unroll
-    for (int i = 0; i < o; ++i) {
-      const float send = up ? y[i] : y[i + o];
-      y[i] = (up ? y[i + o] : y[i]) + __shfl_xor_sync(0xffffffffu, send, o);
-    }
-  }
-  return y[0];
-}
-
 // Longer portions: a CTA walks one sequence for kScanThreads / LPC channels.  The lanes of a channel share its rows: lane l
-// fetches, prepares (step size, silu(z)) and finishes rows l, l + LPC, ...; step sizes and inputs reach the other lanes by
-// shuffles.  The inputs of the next kScanRows rows are under way while the current ones are worked on.
+// fetches, prepares (step size, silu(z)) and finishes rows l, l + LPC, ...; step sizes and inputs reach the other lanes
+// through shared memory, the lanes' sums are put together behind the last row of a tile.  The inputs of the next kScanRows
+// rows are under way while the current ones are worked on.
 template <typename T, int NPT, int LPC>
 __global__ void __launch_bounds__(kScanThreads) scan_rows_kernel(const ScanParams<T> p) {
   constexpr int CPB = kScanThreads / LPC, NP = NPT * LPC;
   constexpr int G = kScanRows / LPC;                                            // rows per lane and tile
   constexpr int NB = kScanRows * 2 * NP / kScanThreads;                         // B and C values per thread and tile
   constexpr bool kAheadB = NB >= 1 && NB <= 16;
-  constexpr int NBUF = NP > 128 ? 1 : 2;
-  __shared__ __align__(16) float sBC[NBUF][kScanRows][2 * NP];
+  __shared__ __align__(16) float sBC[kScanRows][2 * NP];
+  __shared__ float2 sDt[kScanRows][CPB];                                       // (step size, step size * input)
   const int seq = blockIdx.y, tid = threadIdx.x;
   const int start = p.q.q_cu[seq], len = p.q.q_cu[seq + 1] - start;
   if (len < 2) return;
@@ -923,62 +973,77 @@ __global__ void __launch_bounds__(kScanThreads) scan_rows_kernel(const ScanParam
       }
     }
   };
-  auto put = [&](int b, int buf) {
+  auto put = [&](int b) {
     if (kAheadB) {
 #pragma unroll
-      for (int i = 0; i < NB; ++i) (&sBC[buf][0][0])[i * kScanThreads + tid] = to_f32(rb[kAheadB ? i : 0]);
+      for (int i = 0; i < NB; ++i) (&sBC[0][0])[i * kScanThreads + tid] = to_f32(rb[kAheadB ? i : 0]);
     } else {
       const int m = min(kScanRows, len - b);
       for (int e = tid; e < kScanRows * 2 * NP; e += kScanThreads) {
         const int row = e / (2 * NP), n = e % (2 * NP), nn = n < NP ? n : n - NP;
-        (&sBC[buf][0][0])[e] = row < m && nn < p.N ? to_f32((n < NP ? p.B : p.Cm)[size_t(start + b + row) * p.ldb + nn]) : 0.f;
+        (&sBC[0][0])[e] = row < m && nn < p.N ? to_f32((n < NP ? p.B : p.Cm)[size_t(start + b + row) * p.ldb + nn]) : 0.f;
       }
     }
   };
   fetch(0);
-  put(0, 0);
-  int buf = 0;
-  for (int b = 0; b < len; b += kScanRows, buf ^= NBUF - 1) {
+  put(0);
+  for (int b = 0; b < len; b += kScanRows) {
     const int m = min(kScanRows, len - b);
-    float dt[G], x[G], z[G];
+    float x[G], z[G];
 #pragma unroll
     for (int g = 0; g < G; ++g) {                          // rows beyond m: a step of size 0 leaves the state as it is
-      dt[g] = g * LPC + ln < m ? softplus(rdt[g] + bias) : 0.f;
+      const float dt = g * LPC + ln < m ? softplus(rdt[g] + bias) : 0.f;
       x[g] = to_f32(rx[g]);
       z[g] = to_f32(rz[g]);
+      sDt[g * LPC + ln][ch] = make_float2(dt, dt * x[g]);
     }
     __syncthreads();
     if (b + kScanRows < len) fetch(b + kScanRows);
+    float y[kScanRows];
+    constexpr int RG = NPT <= 4 ? 4 : NPT <= 8 ? 2 : 1;    // rows whose factors and inputs are prepared ahead of the recurrence
 #pragma unroll
-    for (int g = 0; g < G; ++g) {
-      const float dx = dt[g] * x[g];
-      float y[LPC];
+    for (int r0 = 0; r0 < kScanRows; r0 += RG) {
+      uint64_t e[RG][NPT / 2], u[RG][NPT / 2];
 #pragma unroll
-      for (int l = 0; l < LPC; ++l) {
-        const float dtl = LPC == 1 ? dt[g] : __shfl_sync(0xffffffffu, dt[g], l, LPC);
-        const float dxl = LPC == 1 ? dx : __shfl_sync(0xffffffffu, dx, l, LPC);
-        const float* bc = &sBC[buf][g * LPC + l][n0];
-        const uint64_t dt2 = pack2(dtl, dtl), dx2 = pack2(dxl, dxl);
+      for (int r = 0; r < RG; ++r) {
+        const float2 d = sDt[r0 + r][ch];
+        const uint64_t dt2 = pack2(d.x, d.x), dx2 = pack2(d.y, d.y);
+#pragma unroll
+        for (int i = 0; i < NPT / 2; i += 2) {
+          const ulonglong2 bb = *reinterpret_cast<const ulonglong2*>(&sBC[r0 + r][n0 + 2 * i]);
+          const float2 f0 = unpack2(mul2(dt2, A[i])), f1 = unpack2(mul2(dt2, A[i + 1]));
+          e[r][i] = pack2(scan_decay<T>(f0.x), scan_decay<T>(f0.y));
+          e[r][i + 1] = pack2(scan_decay<T>(f1.x), scan_decay<T>(f1.y));
+          u[r][i] = mul2(dx2, bb.x);
+          u[r][i + 1] = mul2(dx2, bb.y);
+        }
+      }
+#pragma unroll
+      for (int r = 0; r < RG; ++r) {
         uint64_t acc[2] = {0, 0};
 #pragma unroll
         for (int i = 0; i < NPT / 2; i += 2) {
-          const ulonglong2 bb = *reinterpret_cast<const ulonglong2*>(bc + 2 * i);
-          const ulonglong2 cm = *reinterpret_cast<const ulonglong2*>(bc + NP + 2 * i);
-          const float2 e0 = unpack2(mul2(dt2, A[i])), e1 = unpack2(mul2(dt2, A[i + 1]));
-          S[i] = fma2(pack2(scan_decay<T>(e0.x), scan_decay<T>(e0.y)), S[i], mul2(dx2, bb.x));
-          S[i + 1] = fma2(pack2(scan_decay<T>(e1.x), scan_decay<T>(e1.y)), S[i + 1], mul2(dx2, bb.y));
+          const ulonglong2 cm = *reinterpret_cast<const ulonglong2*>(&sBC[r0 + r][NP + n0 + 2 * i]);
+          S[i] = fma2(e[r][i], S[i], u[r][i]);
+          S[i + 1] = fma2(e[r][i + 1], S[i + 1], u[r][i + 1]);
           acc[0] = fma2(S[i], cm.x, acc[0]);
           acc[1] = fma2(S[i + 1], cm.y, acc[1]);
         }
         const float2 f0 = unpack2(acc[0]), f1 = unpack2(acc[1]);
-        y[l] = (f0.x + f0.y) + (f1.x + f1.y);
+        y[r0 + r] = (f0.x + f0.y) + (f1.x + f1.y);
       }
-      const float sum = sum_to_lanes<LPC>(y, ln);
+    }
+#pragma unroll
+    for (int g = 0; g < G; ++g) {
+      float part[LPC];
+#pragma unroll
+      for (int l = 0; l < LPC; ++l) part[l] = y[g * LPC + l];
+      const float sum = sum_to_lanes<LPC>(part, ln);
       const int row = g * LPC + ln;
       if (row < m && live) from_f32(p.out + size_t(start + b + row) * p.C + c, fmaf(D, x[g], sum) * act_silu(z[g]));
     }
-    if (NBUF == 1) __syncthreads();
-    if (b + kScanRows < len) put(b + kScanRows, buf ^ (NBUF - 1));
+    __syncthreads();                                       // the tile's rows are read: both arrays may be written again
+    if (b + kScanRows < len) put(b + kScanRows);
   }
   if (live) {
 #pragma unroll

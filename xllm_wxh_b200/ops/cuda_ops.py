@@ -451,9 +451,14 @@ def conv_silu(x: torch.Tensor, w: torch.Tensor, b: torch.Tensor, state: torch.Te
     return out
 
 
+mix_force_rows = 0        # > 0: that many rows per segment of time_mix (tests)
+
+
 def mix_segment_rows(T: int, H: int, d: int) -> int:
     """Rows per segment of the time mixing of longer portions: short enough that segments x heads fill the device a few times
     over, long enough that the states between segments stay small beside the rows' own work."""
+    if mix_force_rows > 0:
+        return mix_force_rows
     want = 8 * sm_count() * 64 // max(64, d)
     L = max(1, T * H // want)
     return min(512, max(64, 1 << (L.bit_length() - 1)))
