@@ -12,12 +12,14 @@
 // engine removes the per-chunk address arithmetic and block-table lookups from the compute warps, which is what
 // bounds a decode kernel whose arithmetic intensity is a few FLOP per byte.
 //
-// Template parameters: DK / DV = query-key / value head dimension padded to 64 or 128 (the TMA loads fill the padding with
+// Template parameters: DK / DV = query-key / value head dimension padded to 64, 128 or 256 (the TMA loads fill the padding with
 // zeros), EXT = score extensions (per-head distance bias, per-head sink, chunk mask, first keys that stay visible behind a
-// window) and head dimensions below the padded ones.
+// window, scores bounded by a tanh), head dimensions below the padded ones, and more than 16 query rows per kv head (a CTA per
+// block of 16).  Differential attention (maps = 2): a kv head's row holds the keys of both maps side by side and a query row is
+// zero in the other map's columns, so that one product serves both; the merge stores rms(first - factor * second) * mult.
 //
 // Role: the reference's FlashInfer `batch_decode_with_kv_cache` (xllm/core/kernels/cuda/batch_decode.cpp:26-85).
-#include "common.cuh"
+#include "softcap.cuh"
 
 namespace xl_dec {
 using namespace xl;
@@ -68,6 +70,11 @@ struct DecParams {
   int keep_first = 0;
   const float* slopes = nullptr;
   const float* sinks = nullptr;
+  int row_blocks = 1;             // blocks of 16 query rows per kv head (grid.y = n_kv * row_blocks)
+  int maps = 1;
+  float cap_in = 0.f, cap_out = 0.f;      // cap_out > 0: scores are cap_out * tanh(product * cap_in), in the log2 domain
+  const float* mix = nullptr;
+  float mix_mult = 0.f, mix_eps = 0.f;
 };
 
 constexpr int kStages = 3;
@@ -98,7 +105,8 @@ __global__ void __launch_bounds__(160) decode_attn_tma_kernel(const __grid_const
 
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const int seq = p.seq_begin + blockIdx.x;
-  const int kvh = blockIdx.y;
+  const int kvh = EXT ? blockIdx.y / p.row_blocks : blockIdx.y;
+  const int row0 = EXT ? blockIdx.y % p.row_blocks * 16 : 0;      // first query row (token x head) of this CTA
   const int split = blockIdx.z;
   const int group = p.n_q / p.n_kv;
   if (seq >= (p.dyn_end ? *p.dyn_end : p.seq_end)) return;
@@ -110,7 +118,8 @@ __global__ void __launch_bounds__(160) decode_attn_tma_kernel(const __grid_const
     if (threadIdx.x == 0) atomicExch(p.status, XL_ERR_BOUNDS);
     return;
   }
-  const int rows = min(16, q_len * group);
+  const int rows = min(16, q_len * group - row0);
+  if (rows <= 0) return;
   const int* bt = p.block_tables + size_t(seq) * p.max_blocks;
 
   int r_begin = 0;                                // first key that any row may see, rounded down to a tile
@@ -131,12 +140,14 @@ __global__ void __launch_bounds__(160) decode_attn_tma_kernel(const __grid_const
     }
     mbar_fence_init();
   }
-  // Q rows -> smem (zero beyond `rows`); row m = qtok * group + g
+  // Q rows -> smem (zero beyond `rows` and in the columns of another map); row m = qtok * group + g
+  const int dq = EXT ? dk / p.maps : dk;          // columns of a query head
   for (int i = threadIdx.x; i < 16 * CH; i += blockDim.x) {
     const int r = i / CH, c = i % CH;
-    const bool ok = r < rows && (!EXT || c * 8 < dk);
-    const int qt = ok ? r / group : 0, g = ok ? r % group : 0;
-    const __nv_bfloat16* src = p.q + size_t(q_start + qt) * p.q_stride + (kvh * group + g) * dk + (ok ? c * 8 : 0);
+    const int col = EXT ? c * 8 - (p.maps == 2 ? ((row0 + r) & 1) * dq : 0) : c * 8;      // column of this chunk in the query head
+    const bool ok = r < rows && (!EXT || (col >= 0 && col < dq));
+    const int qt = ok ? (row0 + r) / group : 0, g = ok ? (row0 + r) % group : 0;
+    const __nv_bfloat16* src = p.q + size_t(q_start + qt) * p.q_stride + (kvh * group + g) * dq + (ok ? col : 0);
     cp_async_16(sQ + uint32_t(r) * (DK * 2) + (uint32_t(c ^ (r & 7)) << 4), src, ok);
   }
   cp_async_commit();
@@ -190,17 +201,19 @@ __global__ void __launch_bounds__(160) decode_attn_tma_kernel(const __grid_const
     }
   } else {
     // ------------------------------------------------------------ consumers
-    uint32_t qf[DK / 16][4];
-    {
+    constexpr bool kKeepQ = DK <= 128;                     // wider query rows are read from shared memory at every tile
+    uint32_t qf[kKeepQ ? DK / 16 : 1][4];
+    auto load_q = [&](int ks, uint32_t (&f)[4]) {
       const int r = (lane & 7) + ((lane >> 3) & 1) * 8;
+      const int c = ks * 2 + (lane >> 4);
+      ldsm_x4(smem_u32(sQ + uint32_t(r) * (DK * 2) + (uint32_t(c ^ (r & 7)) << 4)), f[0], f[1], f[2], f[3]);
+    };
+    if (kKeepQ) {
 #pragma unroll
-      for (int ks = 0; ks < DK / 16; ++ks) {
-        const int c = ks * 2 + (lane >> 4);
-        ldsm_x4(smem_u32(sQ + uint32_t(r) * (DK * 2) + (uint32_t(c ^ (r & 7)) << 4)), qf[ks][0], qf[ks][1], qf[ks][2], qf[ks][3]);
-      }
+      for (int ks = 0; ks < (kKeepQ ? DK / 16 : 1); ++ks) load_q(ks, qf[ks]);
     }
-    const int lim_a = kv_len - q_len + (row_a < rows ? row_a / group : 0);
-    const int lim_b = kv_len - q_len + (row_b < rows ? row_b / group : 0);
+    const int lim_a = kv_len - q_len + (row_a < rows ? (row0 + row_a) / group : 0);
+    const int lim_b = kv_len - q_len + (row_b < rows ? (row0 + row_b) / group : 0);
     int lo_a = 0, lo_b = 0;                                // first visible key of the row's chunk
     float slope_a = 0.f, slope_b = 0.f;
     if (EXT) {
@@ -209,8 +222,8 @@ __global__ void __launch_bounds__(160) decode_attn_tma_kernel(const __grid_const
         lo_b = lim_b / p.chunk * p.chunk;
       }
       if (p.slopes) {
-        slope_a = p.slopes[kvh * group + (row_a < rows ? row_a % group : 0)] * kL2e;
-        slope_b = p.slopes[kvh * group + (row_b < rows ? row_b % group : 0)] * kL2e;
+        slope_a = p.slopes[kvh * group + (row_a < rows ? (row0 + row_a) % group : 0)] * kL2e;
+        slope_b = p.slopes[kvh * group + (row_b < rows ? (row0 + row_b) % group : 0)] * kL2e;
       }
     }
     const int rk = (lane & 7) + (lane >> 4) * 8;           // K fragment row (token) of this lane
@@ -234,8 +247,14 @@ __global__ void __launch_bounds__(160) decode_attn_tma_kernel(const __grid_const
           uint32_t b0, b1, b2, b3;
           const int c = (ks & 3) * 2 + ((lane >> 3) & 1);
           ldsm_x4(smem_u32(tK + (ks >> 2) * SLAB + rk * 128 + ((c ^ (rk & 7)) << 4)), b0, b1, b2, b3);
-          mma_bf16_16816(sc[0], qf[ks], b0, b1);
-          mma_bf16_16816(sc[1], qf[ks], b2, b3);
+          if (!kKeepQ) load_q(ks, qf[0]);
+          mma_bf16_16816(sc[0], qf[kKeepQ ? ks : 0], b0, b1);
+          mma_bf16_16816(sc[1], qf[kKeepQ ? ks : 0], b2, b3);
+        }
+        const bool capped = EXT && p.cap_out > 0.f;
+        if (capped) {
+          softcap_row(sc[0], p.cap_in, p.cap_out);
+          softcap_row(sc[1], p.cap_in, p.cap_out);
         }
         float mx[2] = {-INFINITY, -INFINITY};
 #pragma unroll
@@ -246,7 +265,7 @@ __global__ void __launch_bounds__(160) decode_attn_tma_kernel(const __grid_const
             const int lim = (e < 2) ? lim_a : lim_b;
             bool ok = tok <= lim && tok < kv_len;
             if (p.window > 0) ok = ok && (tok > lim - p.window || (EXT && tok < p.keep_first));
-            float x = sc[i][e] * p.scale_log2;
+            float x = capped ? sc[i][e] : sc[i][e] * p.scale_log2;
             if (EXT) {
               ok = ok && tok >= ((e < 2) ? lo_a : lo_b);
               x += ((e < 2) ? slope_a : slope_b) * float(tok - lim);
@@ -321,7 +340,44 @@ __global__ void __launch_bounds__(160) decode_attn_tma_kernel(const __grid_const
     }
   }
   __syncthreads();
-  if (warp < 4) {
+  if (EXT && p.maps == 2 && p.num_splits == 1) {
+    // rows 2 i and 2 i + 1 are the two maps of one output head
+    const float factor = *p.mix;
+    for (int i = warp; i < rows / 2 && warp < 4; i += 4) {
+      float w[2][4];
+#pragma unroll
+      for (int k = 0; k < 2; ++k) {
+        const int r = 2 * i + k;
+        const int hq = kvh * group + (row0 + r) % group;
+        const float m = fmaxf(fmaxf(sM[r], sM[16 + r]), fmaxf(sM[32 + r], sM[48 + r]));
+        float den = p.sinks && m != -INFINITY ? exp2f(p.sinks[hq] * kL2e - m) : 0.f;
+#pragma unroll
+        for (int j = 0; j < 4; ++j) {
+          w[k][j] = sM[16 * j + r] == -INFINITY ? 0.f : exp2f(sM[16 * j + r] - m);
+          den += w[k][j] * sL[16 * j + r];
+        }
+#pragma unroll
+        for (int j = 0; j < 4; ++j) w[k][j] *= den > 0.f ? 1.f / den : 0.f;
+      }
+      float d[DV / 32], ss = 0.f;
+#pragma unroll
+      for (int c = 0; c < DV / 32; ++c) {           // columns past dv hold zeros
+        float a[2] = {0.f, 0.f};
+#pragma unroll
+        for (int k = 0; k < 2; ++k)
+#pragma unroll
+          for (int j = 0; j < 4; ++j) a[k] += w[k][j] * sO[(16 * j + 2 * i + k) * DV + c * 32 + lane];
+        d[c] = fmaf(-factor, a[1], a[0]);
+        ss += d[c] * d[c];
+      }
+      const float s = rsqrtf(warp_sum(ss) / float(dv) + p.mix_eps) * p.mix_mult;
+      const int qt = (row0 + 2 * i) / group, head = (kvh * group + (row0 + 2 * i) % group) / 2;
+      __nv_bfloat16* dst = p.out + size_t(q_start + qt) * (size_t(p.n_q / 2) * dv) + head * dv;
+#pragma unroll
+      for (int c = 0; c < DV / 32; ++c)
+        if (c * 32 + lane < dv) dst[c * 32 + lane] = __float2bfloat16(d[c] * s);
+    }
+  } else if (warp < 4) {
     for (int r = warp; r < rows; r += 4) {
       const float m = fmaxf(fmaxf(sM[r], sM[16 + r]), fmaxf(sM[32 + r], sM[48 + r]));
       float w0 = (sM[r] == -INFINITY) ? 0.f : exp2f(sM[r] - m);
@@ -329,7 +385,7 @@ __global__ void __launch_bounds__(160) decode_attn_tma_kernel(const __grid_const
       float w2 = (sM[32 + r] == -INFINITY) ? 0.f : exp2f(sM[32 + r] - m);
       float w3 = (sM[48 + r] == -INFINITY) ? 0.f : exp2f(sM[48 + r] - m);
       const float l = w0 * sL[r] + w1 * sL[16 + r] + w2 * sL[32 + r] + w3 * sL[48 + r];
-      const int qt = r / group, g = r % group;
+      const int qt = (row0 + r) / group, g = (row0 + r) % group;
       const int hq = kvh * group + g;
       float den = l;                              // the sink joins once: here, or in the merge of the splits
       if (EXT && p.sinks && p.num_splits == 1 && m != -INFINITY) den += exp2f(p.sinks[hq] * kL2e - m);
@@ -547,21 +603,71 @@ __global__ void split_merge_ext_kernel(const float* __restrict__ part_o, const f
     out[tok * (size_t(n_q) * dv) + h * dv + c] = __float2bfloat16(acc * inv);
   }
 }
+
+// The same for differential attention: one warp per (token, output head) merges both maps and stores their normed difference.
+__global__ void split_merge_mix_kernel(const float* __restrict__ part_o, const float* __restrict__ part_lse,
+                                       __nv_bfloat16* __restrict__ out, const int* __restrict__ q_cu, int seq_begin, int seq_end,
+                                       int n_q, int dv, int splits, const float* __restrict__ sinks, const float* __restrict__ mix,
+                                       float mult, float eps, const int* dyn_end) {
+  const int lane = threadIdx.x & 31;
+  const long gw = (blockIdx.x * long(blockDim.x) + threadIdx.x) >> 5;
+  if (dyn_end) seq_end = *dyn_end;
+  if (seq_end <= seq_begin) return;
+  const int t0 = q_cu[seq_begin], t1 = q_cu[seq_end], heads = n_q / 2;
+  if (gw >= long(t1 - t0) * heads) return;
+  const size_t tok = size_t(t0) + size_t(gw / heads);
+  const int head = int(gw % heads);
+  constexpr int kCols = 8;                              // dv <= 256
+  float d[kCols];
+#pragma unroll
+  for (int c = 0; c < kCols; ++c) d[c] = 0.f;
+#pragma unroll
+  for (int k = 0; k < 2; ++k) {
+    const size_t row = tok * n_q + 2 * head + k;
+    const float* lse = part_lse + row * splits;
+    const float sink = sinks ? sinks[2 * head + k] * 1.4426950408889634f : -INFINITY;
+    float m = sink;
+    for (int s = 0; s < splits; ++s) m = fmaxf(m, lse[s]);
+    float den = sinks ? exp2f(sink - m) : 0.f;
+    for (int s = 0; s < splits; ++s) den += lse[s] == -INFINITY ? 0.f : exp2f(lse[s] - m);
+    const float f = (den > 0.f ? 1.f / den : 0.f) * (k == 0 ? 1.f : -*mix);
+    for (int s = 0; s < splits; ++s) {
+      const float w = lse[s] == -INFINITY ? 0.f : exp2f(lse[s] - m) * f;
+      if (w == 0.f) continue;
+      const float* po = part_o + (row * splits + s) * dv;
+#pragma unroll
+      for (int c = 0; c < kCols; ++c)
+        if (c * 32 + lane < dv) d[c] += w * po[c * 32 + lane];
+    }
+  }
+  float ss = 0.f;
+#pragma unroll
+  for (int c = 0; c < kCols; ++c) ss += d[c] * d[c];
+  const float s = rsqrtf(warp_sum(ss) / float(dv) + eps) * mult;
+#pragma unroll
+  for (int c = 0; c < kCols; ++c)
+    if (c * 32 + lane < dv) out[tok * (size_t(heads) * dv) + head * dv + c * 32 + lane] = __float2bfloat16(d[c] * s);
+}
 }  // namespace xl_dec
 
-// Decode attention with the score extensions of xl_prefill_attention_ext (head dimensions: multiples of 8, at most 128).
-// With num_splits > 1 the partials are merged by a second kernel; `max_rows` bounds the query tokens of the launch.
+// Decode attention with the score extensions of xl_prefill_attention_ext (head dimensions: multiples of 8, at most 256; with
+// maps = 2 the keys of both maps together).  With num_splits > 1 the partials are merged by a second kernel; `max_rows` bounds the
+// query tokens of the launch, `max_q` those of a sequence.
 XL_API int xl_decode_attention_ext(const void* q, const void* k_cache, const void* v_cache, void* out, const void* q_cu,
                                    const void* kv_lens, const void* block_tables, int seq_begin, int seq_end, int max_blocks,
                                    int block_size, int num_blocks_total, int n_q, int n_kv, int dk, int dv, int q_stride,
                                    float scale, int window, int chunk, int keep_first, const void* slopes, const void* sinks,
+                                   float softcap, long v_pitch, int maps, const void* mix, float mix_mult, float mix_eps, int max_q,
                                    int num_splits, void* part_o, void* part_lse, long max_rows, const void* dyn_end, void* stream) {
   using namespace xl_dec;
   if (seq_end <= seq_begin) return 0;
   if (chunk > 0 && keep_first > 0) return -2;
-  if (dk < 8 || dk > 128 || dk % 8 || dv < 8 || dv > 128 || dv % 8) return -3;
+  if (maps < 1 || maps > 2 || (maps == 2 && (!mix || (n_q / n_kv) % 2))) return -2;
+  if (dk < 8 || dk % 8) return -3;
+  dk *= maps;                                  // the keys of both maps lie side by side
+  if (dk > 256 || dv < 8 || dv > 256 || dv % 8 || v_pitch % 8) return -3;
   if (block_size % 16 != 0 || (block_size > 64 && block_size % 64 != 0) || (block_size < 64 && 64 % block_size != 0)) return -3;
-  if (n_q % n_kv || n_q / n_kv > 16) return -3;
+  if (n_q % n_kv) return -3;
   if ((q_stride % 8) || (reinterpret_cast<uintptr_t>(q) & 15)) return -3;
   if ((reinterpret_cast<uintptr_t>(k_cache) & 127) || (reinterpret_cast<uintptr_t>(v_cache) & 127)) return -3;
   const int box_tokens = block_size < 64 ? block_size : 64;
@@ -569,7 +675,7 @@ XL_API int xl_decode_attention_ext(const void* q, const void* k_cache, const voi
   const CUtensorMap* tk = xl_host::tmap_3d(k_cache, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 2, slots, n_kv, dk, box_tokens, 1, 64,
                                            CU_TENSOR_MAP_SWIZZLE_128B);
   const CUtensorMap* tv = xl_host::tmap_3d(v_cache, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 2, slots, n_kv, dv, box_tokens, 1, 64,
-                                           CU_TENSOR_MAP_SWIZZLE_128B);
+                                           CU_TENSOR_MAP_SWIZZLE_128B, v_pitch);
   if (!tk || !tv) return -3;
   DecParams p;
   p.q = static_cast<const __nv_bfloat16*>(q);
@@ -591,13 +697,28 @@ XL_API int xl_decode_attention_ext(const void* q, const void* k_cache, const voi
   p.dk = dk; p.dv = dv; p.chunk = chunk; p.keep_first = keep_first;
   p.slopes = static_cast<const float*>(slopes);
   p.sinks = static_cast<const float*>(sinks);
+  p.row_blocks = (n_q / n_kv * (max_q < 1 ? 1 : max_q) + 15) / 16;
+  p.maps = maps;
+  if (softcap > 0.f) {
+    p.cap_in = scale / softcap;
+    p.cap_out = softcap * 1.4426950408889634f;
+  }
+  p.mix = static_cast<const float*>(mix);
+  p.mix_mult = mix_mult; p.mix_eps = mix_eps;
   if (p.num_splits > 1 && (!part_o || !part_lse)) return -2;
   cudaStream_t st = static_cast<cudaStream_t>(stream);
-  const dim3 grid(seq_end - seq_begin, n_kv, p.num_splits);
+  const dim3 grid(seq_end - seq_begin, n_kv * p.row_blocks, p.num_splits);
   int rc;
-  if (dk > 64) rc = dv > 64 ? launch_ext<128, 128>(tk, tv, p, grid, st) : launch_ext<128, 64>(tk, tv, p, grid, st);
+  if (dv > 128) rc = launch_ext<256, 256>(tk, tv, p, grid, st);
+  else if (dk > 128) rc = launch_ext<256, 128>(tk, tv, p, grid, st);
+  else if (dk > 64) rc = dv > 64 ? launch_ext<128, 128>(tk, tv, p, grid, st) : launch_ext<128, 64>(tk, tv, p, grid, st);
   else rc = dv > 64 ? launch_ext<64, 128>(tk, tv, p, grid, st) : launch_ext<64, 64>(tk, tv, p, grid, st);
   if (rc != 0 || p.num_splits == 1) return rc;
+  if (maps == 2) {
+    split_merge_mix_kernel<<<int((max_rows * (n_q / 2) + 3) / 4), 128, 0, st>>>(p.part_o, p.part_lse, p.out, p.q_cu, seq_begin, seq_end, n_q, dv,
+                                                                                p.num_splits, p.sinks, p.mix, mix_mult, mix_eps, p.dyn_end);
+    return cudaGetLastError() == cudaSuccess ? 0 : -1;
+  }
   split_merge_ext_kernel<<<int((max_rows * n_q + 3) / 4), 128, 0, st>>>(p.part_o, p.part_lse, p.out, p.q_cu, seq_begin, seq_end, n_q, dv,
                                                                         p.num_splits, p.sinks, p.dyn_end);
   return cudaGetLastError() == cudaSuccess ? 0 : -1;

@@ -19,12 +19,15 @@
 // Template parameters: QS / VS = 64-column slabs of the query-key / value head dimension (a dimension that does not fill
 // its slabs is padded with zeros by the TMA loads), EXT = score extensions: per-head linear distance bias, per-head sink
 // (a score that joins the denominator and has no value), chunk mask (a query sees keys of its own position chunk only),
-// first keys that stay visible behind a window (their tiles come ahead of the window's, the gap between is not read).
+// first keys that stay visible behind a window (their tiles come ahead of the window's, the gap between is not read), scores
+// bounded by a tanh.  MAPS = 2: differential attention.  The CTA's two heads are the two maps of one output head: each has its own
+// keys (slabs of their own in a stage), both read the same values, and the epilogue hands the second map's output to the first
+// map's warps through the idle ring, which store rms(first - factor * second) * mult.
 // QK^T of tile j+1 is issued before P V of tile j, so the tensor pipe works while the softmax warps are busy.
 // Every wait is bounded; on expiry the kernel records a status code and leaves.
 #include <string.h>
 
-#include "common.cuh"
+#include "softcap.cuh"
 
 namespace xl_pf {
 using namespace xl;
@@ -34,14 +37,16 @@ constexpr int BKV = 64;          // kv tokens per tile
 constexpr int Q_SLAB = BQ * 128;               // 16 KB: [128 rows][64 columns]
 constexpr int KV_SLAB = BKV * 128;             // 8 KB: [64 tokens][64 columns]
 constexpr int P_BYTES = BQ * BKV * 2;          // 16 KB: [128][64] K-major
-template <int NH, int QS, int VS> struct Cfg {
-  static constexpr int kStages = NH == 2 ? 4 : 5;
+template <int NH, int QS, int VS, int MAPS = 1> struct Cfg {
   static constexpr int kThreads = 64 + 128 * NH;
-  static constexpr uint32_t kTmemCols = NH == 2 ? 512 : 256;   // per head: S0, S1 (64 columns each) and O (up to 128)
+  static constexpr uint32_t kTmemCols = NH == 2 || VS > 2 ? 512 : 256;   // per head: S0, S1 (64 columns each) and O
   static constexpr int DK = 64 * QS, DV = 64 * VS;             // padded head dimensions
   static constexpr int Q_BYTES = QS * Q_SLAB;
-  static constexpr int K_BYTES = QS * KV_SLAB, V_BYTES = VS * KV_SLAB;
-  static constexpr int STAGE_BYTES = K_BYTES + V_BYTES;        // K then V
+  static constexpr int K_BYTES = MAPS * QS * KV_SLAB, V_BYTES = VS * KV_SLAB;
+  static constexpr int STAGE_BYTES = K_BYTES + V_BYTES;        // K (of every map) then V
+  static constexpr int kFit = (226 * 1024 - NH * (Q_BYTES + P_BYTES)) / STAGE_BYTES, kMost = NH == 2 ? 4 : 5;
+  static constexpr int kStages = kFit < kMost ? kFit : kMost;
+  static_assert(kStages >= 2 && (NH == 1 || VS <= 2) && (MAPS == 1 || (NH == 2 && kStages * STAGE_BYTES >= DV * BQ * 4)), "tile sizes");
 };
 constexpr int kMaxStages = 5;
 
@@ -64,6 +69,9 @@ struct Params {
   const float* sinks;          // EXT: [Hq] sink scores (null: none): denominator += exp(sink)
   int chunk;                   // EXT: positions per chunk (<= 0: no chunk mask)
   int keep_first;              // EXT: first keys that stay visible behind the window
+  float cap_in, cap_out;       // EXT: bounded scores, cap_out * tanh(product * cap_in) in the log2 domain (cap_out 0: not bounded)
+  const float* mix;            // MAPS = 2: factor of the second map
+  float mix_mult, mix_eps;
   const int* q_cu;
   const int* kv_lens;
   const int* block_tables;
@@ -115,11 +123,29 @@ __device__ __forceinline__ float fast_exp2(float x) {
   return y;
 }
 
-template <int NH, int QS, int VS, bool EXT>
-__global__ void __launch_bounds__(Cfg<NH, QS, VS>::kThreads, 1)
+__device__ __forceinline__ void softmax_warps_sync() { asm volatile("bar.sync 1, 256;" ::: "memory"); }
+
+// MAPS = 2, first map's thread of row r: ex[c * BQ + r] holds first - factor * second (columns past dv are zero), `ss` its squares.
+template <int DV>
+__device__ __forceinline__ void store_difference(const Params& p, const float* ex, float ss, int r, size_t row, int head) {
+  const float s = rsqrtf(ss / float(p.dv) + p.mix_eps) * p.mix_mult;
+  __nv_bfloat16* dst = p.out + row * (size_t(p.n_q / 2) * p.dv) + head * p.dv;
+#pragma unroll 4
+  for (int c = 0; c < DV; c += 8) {
+    float f[8];
+#pragma unroll
+    for (int e = 0; e < 8; ++e) f[e] = ex[(c + e) * BQ + r] * s;
+    if (c < p.dv)
+      *reinterpret_cast<uint4*>(dst + c) =
+          make_uint4(pack_bf16x2(f[0], f[1]), pack_bf16x2(f[2], f[3]), pack_bf16x2(f[4], f[5]), pack_bf16x2(f[6], f[7]));
+  }
+}
+
+template <int NH, int QS, int VS, bool EXT, int MAPS>
+__global__ void __launch_bounds__(Cfg<NH, QS, VS, MAPS>::kThreads, 1)
 prefill_attn_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__ CUtensorMap tmK,
                        const __grid_constant__ CUtensorMap tmV, const Params p) {
-  using C = Cfg<NH, QS, VS>;
+  using C = Cfg<NH, QS, VS, MAPS>;
   constexpr int kStages = C::kStages;
   constexpr uint32_t kTmemCols = C::kTmemCols;
   constexpr int DK = C::DK, DV = C::DV, Q_BYTES = C::Q_BYTES, K_BYTES = C::K_BYTES, STAGE_BYTES = C::STAGE_BYTES;
@@ -223,10 +249,13 @@ prefill_attn_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_con
       }
     }
     const int boxes = BKV / p.box_tokens;            // boxes per 64-token slab (1, 2 or 4)
-    const int per_tile = boxes * (QS + VS);          // x slabs of K, then of V
+    constexpr int KS = MAPS * QS;                    // K slabs, map by map
+    const int per_tile = boxes * (KS + VS);          // x slabs of K, then of V (at most 4 x 8)
     const int sl_all = lane / boxes;
-    const int which = sl_all >= QS ? 1 : 0;          // 0 = K, 1 = V
-    const int slab = which ? sl_all - QS : sl_all;
+    const int which = sl_all >= KS ? 1 : 0;          // 0 = K, 1 = V
+    const int slab = which ? sl_all - KS : sl_all;
+    const int column = which ? slab * 64 : slab % QS * 64;
+    const int cache_head = which || MAPS == 1 ? kvh : kvh * MAPS + slab / QS;
     const int bx = lane % boxes;
     bool ok = true;
     for (int j = 0; j < n_tiles && ok; ++j) {
@@ -253,7 +282,7 @@ prefill_attn_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_con
       if (!ok) break;
       if (lane < per_tile) {
         uint8_t* dst = sKV + st * STAGE_BYTES + which * K_BYTES + slab * KV_SLAB + bx * p.box_tokens * 128;
-        tma_load_3d(dst, which ? &tmV : &tmK, &bars->kv_full[st], slab * 64, kvh, int(slot));
+        tma_load_3d(dst, which ? &tmV : &tmK, &bars->kv_full[st], column, cache_head, int(slot));
       }
       __syncwarp();
     }
@@ -302,7 +331,7 @@ prefill_attn_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_con
 #pragma unroll
           for (int k = 0; k < DK / 16; ++k)
             tc_mma_f16(tmem_base + h * 256 + b * 64, umma_desc_sw128(q_addr + h * Q_BYTES + (k >> 2) * Q_SLAB, (k & 3) * 32),
-                       umma_desc_sw128(k_addr + (k >> 2) * KV_SLAB, (k & 3) * 32), idesc_s, k != 0);
+                       umma_desc_sw128(k_addr + ((MAPS == 2 ? h * QS : 0) + (k >> 2)) * KV_SLAB, (k & 3) * 32), idesc_s, k != 0);
           tc_commit(&bars->s_full[h][b]);
         }
         if (ok && j > 0) ok = issue_pv(j - 1);
@@ -354,8 +383,16 @@ prefill_attn_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_con
       }
       if (EXT) {
         const float b0 = slope2 * float(kv0 - pos);
+        if (p.cap_out > 0.f) {
+          softcap_row(v, p.cap_in, p.cap_out);
+          if (slope2 != 0.f) {
 #pragma unroll
-        for (int c = 0; c < 64; ++c) v[c] = fmaf(v[c], p.scale_log2, fmaf(slope2, float(c), b0));
+            for (int c = 0; c < 64; ++c) v[c] += fmaf(slope2, float(c), b0);
+          }
+        } else {
+#pragma unroll
+          for (int c = 0; c < 64; ++c) v[c] = fmaf(v[c], p.scale_log2, fmaf(slope2, float(c), b0));
+        }
       }
       if (need_mask) {
 #pragma unroll
@@ -439,6 +476,41 @@ prefill_attn_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_con
       }
       p.ws_ml[(unit * p.splits + blockIdx.z) * BQ + r] = make_float2(m_ref == -INFINITY ? -INFINITY : m_ref * sc, l_run);
       __threadfence();
+    } else if (MAPS == 2 && n_splits == 1) {
+      float* ex = reinterpret_cast<float*>(sKV);             // every product has read its tiles: the ring is free
+      float inv = 0.f, ss = 0.f;
+      if (ok) {
+        tc_fence_after();
+        if (p.sinks && m_ref != -INFINITY) l_run += fast_exp2(p.sinks[head0 + h] * 1.4426950408889634f - m_ref);
+        inv = l_run > 0.f ? 1.f / l_run : 0.f;
+      }
+      if (ok && h == 1) {
+#pragma unroll 1
+        for (int c = 0; c < DV; c += 32) {
+          uint32_t o[32];
+          tmem_ld_32x32(t_o + c, o);
+          tc_wait_ld();
+#pragma unroll
+          for (int i = 0; i < 32; ++i) ex[(c + i) * BQ + r] = __uint_as_float(o[i]) * inv;
+        }
+      }
+      softmax_warps_sync();                                  // reached by both groups whatever their waits did
+      if (ok && h == 0) {
+        const float factor = *p.mix;
+#pragma unroll 1
+        for (int c = 0; c < DV; c += 32) {
+          uint32_t o[32];
+          tmem_ld_32x32(t_o + c, o);
+          tc_wait_ld();
+#pragma unroll
+          for (int i = 0; i < 32; ++i) {
+            const float d = fmaf(-factor, ex[(c + i) * BQ + r], __uint_as_float(o[i]) * inv);
+            ss += d * d;
+            ex[(c + i) * BQ + r] = d;
+          }
+        }
+        if (r < rows) store_difference<DV>(p, ex, ss, r, size_t(q_start + q0 + r), blockIdx.y);
+      }
     } else if (ok) {
       tc_fence_after();
       if (EXT && p.sinks && m_ref != -INFINITY) l_run += fast_exp2(p.sinks[head0 + h] * 1.4426950408889634f - m_ref);
@@ -507,7 +579,44 @@ prefill_attn_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_con
     }
     if (EXT && p.sinks && m_all != -INFINITY) l_all += fast_exp2(p.sinks[head0 + h] * 1.4426950408889634f - m_all);
     const float inv = l_all > 0.f ? 1.f / l_all : 0.f;
-    if (r < rows) {
+    if (MAPS == 2) {
+      float* ex = reinterpret_cast<float*>(sKV);
+      const float4* wo = reinterpret_cast<const float4*>(p.ws_o) + unit * p.splits * (DV / 4) * BQ + r;
+      const float factor = *p.mix;
+      float ss = 0.f;
+      auto merged = [&](int c4) {
+        float4 a = make_float4(0.f, 0.f, 0.f, 0.f);
+#pragma unroll
+        for (int z = 0; z < 8; ++z) {
+          if (z < n_valid && w[z] != 0.f) {
+            const float4 x = __ldcg(wo + (size_t(z) * (DV / 4) + c4) * BQ);
+            a.x += w[z] * x.x; a.y += w[z] * x.y; a.z += w[z] * x.z; a.w += w[z] * x.w;
+          }
+        }
+        return make_float4(a.x * inv, a.y * inv, a.z * inv, a.w * inv);
+      };
+      if (h == 1) {
+        for (int c4 = 0; c4 < DV / 4; ++c4) {
+          const float4 a = merged(c4);
+          ex[(4 * c4) * BQ + r] = a.x; ex[(4 * c4 + 1) * BQ + r] = a.y; ex[(4 * c4 + 2) * BQ + r] = a.z; ex[(4 * c4 + 3) * BQ + r] = a.w;
+        }
+      }
+      softmax_warps_sync();
+      if (h == 0) {
+        for (int c4 = 0; c4 < DV / 4; ++c4) {
+          const float4 a = merged(c4);
+          const float v4[4] = {a.x, a.y, a.z, a.w};
+#pragma unroll
+          for (int e = 0; e < 4; ++e) {
+            float* x = ex + (4 * c4 + e) * BQ + r;
+            const float d = fmaf(-factor, *x, v4[e]);
+            ss += d * d;
+            *x = d;
+          }
+        }
+        if (r < rows) store_difference<DV>(p, ex, ss, r, size_t(q_start + q0 + r), blockIdx.y);
+      }
+    } else if (r < rows) {
       const int dv = EXT ? p.dv : DV;
       const float4* wo = reinterpret_cast<const float4*>(p.ws_o) + unit * p.splits * (DV / 4) * BQ + r;
       __nv_bfloat16* dst = p.out + size_t(q_start + q0 + r) * (size_t(p.n_q) * dv) + (head0 + h) * dv;
@@ -548,14 +657,14 @@ static uint8_t* split_workspace(cudaStream_t stream) {
   return ws[dev];
 }
 
-template <int NH, int QS, int VS, bool EXT>
+template <int NH, int QS, int VS, bool EXT, int MAPS = 1>
 static int launch_prefill(const CUtensorMap* tq, const CUtensorMap* tk, const CUtensorMap* tv, const Params& p_in, int q_tiles_cap,
                           int total_q_rows, cudaStream_t stream) {
-  using C = Cfg<NH, QS, VS>;
+  using C = Cfg<NH, QS, VS, MAPS>;
   const size_t smem = size_t(NH) * (C::Q_BYTES + P_BYTES) + C::kStages * C::STAGE_BYTES + sizeof(Barriers);
   static bool set = false;
   if (!set) {
-    cudaFuncSetAttribute(prefill_attn_tc_kernel<NH, QS, VS, EXT>, cudaFuncAttributeMaxDynamicSharedMemorySize, int(smem));
+    cudaFuncSetAttribute(prefill_attn_tc_kernel<NH, QS, VS, EXT, MAPS>, cudaFuncAttributeMaxDynamicSharedMemorySize, int(smem));
     set = true;
   }
   Params p = p_in;
@@ -586,7 +695,7 @@ static int launch_prefill(const CUtensorMap* tq, const CUtensorMap* tk, const CU
     }
   }
   dim3 grid(q_tiles_cap, p.n_q / NH, p.splits);
-  prefill_attn_tc_kernel<NH, QS, VS, EXT><<<grid, C::kThreads, smem, stream>>>(*tq, *tk, *tv, p);
+  prefill_attn_tc_kernel<NH, QS, VS, EXT, MAPS><<<grid, C::kThreads, smem, stream>>>(*tq, *tk, *tv, p);
   return cudaGetLastError() == cudaSuccess ? 0 : -1;
 }
 
@@ -639,17 +748,24 @@ XL_API int xl_prefill_attention_tc(const void* q, const void* k_cache, const voi
   return launch_prefill<1, 2, 2, false>(tq, tk, tv, p, q_tiles_cap, total_q_rows, st);
 }
 
-// The same with the score extensions and separate query-key / value head dimensions (multiples of 8, at most 128):
+// The same with the score extensions and separate query-key / value head dimensions (multiples of 8, at most 256; 128 with maps = 2):
 //   score(i, j) = scale * q_i . k_j - slopes[h] * (i - j), visible when j <= i, within `window` (> 0) or among the first
 //   `keep_first` keys, and in the same chunk of `chunk` positions (> 0); out = sum_j exp(score) v_j / (sum_j exp(score) + exp(sinks[h])).
-// `slopes` / `sinks` [n_q] fp32, null when absent.  Returns -3 when the shape is not covered.
+// `slopes` / `sinks` [n_q] fp32, null when absent; `softcap` > 0: scale * q . k becomes softcap * tanh(scale * q . k / softcap).
+// `v_pitch`: elements from one cache slot's values to the next one's (0: n_kv * dv), so that values may be a part of the keys.
+// maps = 2: n_q counts the maps' heads (pairs of neighbours), k_cache has 2 n_kv heads, out [T, n_q / 2 * dv] =
+// rms(first - mix[0] * second, mix_eps) * mix_mult.  Returns -3 when the shape is not covered.
 XL_API int xl_prefill_attention_ext(const void* q, const void* k_cache, const void* v_cache, void* out, const void* q_cu,
                                     const void* kv_lens, const void* block_tables, int seq_begin, int seq_end, int max_blocks,
                                     int block_size, int num_blocks_total, int n_q, int n_kv, int dk, int dv, int q_stride,
                                     int total_q_rows, float scale, int window, int chunk, int keep_first, const void* slopes,
-                                    const void* sinks, int q_tiles_cap, const void* dyn_begin, const void* dyn_end, void* stream) {
+                                    const void* sinks, float softcap, long v_pitch, int maps, const void* mix, float mix_mult, float mix_eps,
+                                    int q_tiles_cap, const void* dyn_begin, const void* dyn_end, void* stream) {
   using namespace xl_pf;
-  if (dk < 8 || dk > 128 || dk % 8 || dv < 8 || dv > 128 || dv % 8) return -3;
+  if (maps < 1 || maps > 2 || (maps == 2 && (!mix || (n_q / n_kv) % 2))) return -2;
+  const int d_max = maps == 2 ? 128 : 256;
+  if (dk < 8 || dk > d_max || dk % 8 || dv < 8 || dv > d_max || dv % 8) return -3;
+  if (v_pitch % 8) return -3;
   if (chunk > 0 && keep_first > 0) return -2;
   if (block_size % 16 != 0 || (block_size > 64 && block_size % 64 != 0) || (block_size < 64 && 64 % block_size != 0)) return -3;
   if (n_q % n_kv) return -3;
@@ -661,10 +777,10 @@ XL_API int xl_prefill_attention_ext(const void* q, const void* k_cache, const vo
   // boxes of 64 columns: columns past the head dimension come back as zeros and add nothing to the products
   const CUtensorMap* tq = xl_host::tmap_3d(q, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 2, total_q_rows, n_q, dk, BQ, 1, 64,
                                            CU_TENSOR_MAP_SWIZZLE_128B, q_stride);
-  const CUtensorMap* tk = xl_host::tmap_3d(k_cache, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 2, slots, n_kv, dk, box_tokens, 1, 64,
+  const CUtensorMap* tk = xl_host::tmap_3d(k_cache, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 2, slots, n_kv * maps, dk, box_tokens, 1, 64,
                                            CU_TENSOR_MAP_SWIZZLE_128B);
   const CUtensorMap* tv = xl_host::tmap_3d(v_cache, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 2, slots, n_kv, dv, box_tokens, 1, 64,
-                                           CU_TENSOR_MAP_SWIZZLE_128B);
+                                           CU_TENSOR_MAP_SWIZZLE_128B, v_pitch);
   if (!tq || !tk || !tv) return -3;
   Params p;
   memset(&p, 0, sizeof(p));
@@ -674,6 +790,12 @@ XL_API int xl_prefill_attention_ext(const void* q, const void* k_cache, const vo
   p.sinks = static_cast<const float*>(sinks);
   p.chunk = chunk;
   p.keep_first = keep_first;
+  if (softcap > 0.f) {
+    p.cap_in = scale / softcap;
+    p.cap_out = softcap * 1.4426950408889634f;
+  }
+  p.mix = static_cast<const float*>(mix);
+  p.mix_mult = mix_mult; p.mix_eps = mix_eps;
   p.q_cu = static_cast<const int*>(q_cu);
   p.kv_lens = static_cast<const int*>(kv_lens);
   p.block_tables = static_cast<const int*>(block_tables);
@@ -688,7 +810,14 @@ XL_API int xl_prefill_attention_ext(const void* q, const void* k_cache, const vo
   cudaStream_t st = static_cast<cudaStream_t>(stream);
   const bool pair = (n_q / n_kv) % 2 == 0, k2 = dk > 64, v2 = dv > 64;
 #define XL_PF_EXT(NH, QS, VS) launch_prefill<NH, QS, VS, true>(tq, tk, tv, p, q_tiles_cap, total_q_rows, st)
+#define XL_PF_MAPS(QS, VS) launch_prefill<2, QS, VS, true, 2>(tq, tk, tv, p, q_tiles_cap, total_q_rows, st)
+  if (maps == 2) return k2 ? (v2 ? XL_PF_MAPS(2, 2) : XL_PF_MAPS(2, 1)) : (v2 ? XL_PF_MAPS(1, 2) : XL_PF_MAPS(1, 1));
+  if (dk > 128 || dv > 128) {
+    if (dv > 128) return XL_PF_EXT(1, 4, 4);
+    return dk > 192 ? XL_PF_EXT(1, 4, 2) : XL_PF_EXT(1, 3, 2);
+  }
   if (pair) return k2 ? (v2 ? XL_PF_EXT(2, 2, 2) : XL_PF_EXT(2, 2, 1)) : (v2 ? XL_PF_EXT(2, 1, 2) : XL_PF_EXT(2, 1, 1));
   return k2 ? (v2 ? XL_PF_EXT(1, 2, 2) : XL_PF_EXT(1, 2, 1)) : (v2 ? XL_PF_EXT(1, 1, 2) : XL_PF_EXT(1, 1, 1));
 #undef XL_PF_EXT
+#undef XL_PF_MAPS
 }

@@ -3,7 +3,8 @@
 // per lane for the scores, then one slice of the value columns per lane for the weighted sum, with an online softmax.
 //
 // Serves prefill rows and decode rows alike, because every row finds its sequence and position in the step's own arrays.
-// Score extensions (distance bias, sink, chunk mask) as in xl_prefill_attention_ext.
+// Score extensions (distance bias, sink, chunk mask, bounded scores) and differential attention (MAPS = 2: the warp walks the keys
+// once per map and keeps the first map's output) as in xl_prefill_attention_ext.
 #include "vec8.cuh"
 
 namespace xl_as {
@@ -26,21 +27,31 @@ struct Params {
   int window, chunk, keep_first;
   const float* slopes;
   const float* sinks;
+  float softcap;                  // > 0: bounded scores
+  long v_pitch;                   // elements from one slot's values to the next one's
+  const float* mix;               // MAPS = 2
+  float mix_mult, mix_eps;
 };
 
-template <typename T>
+template <typename T, int MAPS>
 __global__ void __launch_bounds__(128) attention_simt_kernel(const Params<T> p) {
   extern __shared__ float s_q[];                 // one query vector per warp
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const long item = blockIdx.x * long(blockDim.x >> 5) + warp;
-  if (item >= long(p.rows) * p.n_q) return;
-  const int t = int(item / p.n_q), h = int(item % p.n_q);
+  const int n_out = p.n_q / MAPS;                // output heads
+  if (item >= long(p.rows) * n_out) return;
+  const int t = int(item / n_out), h_out = int(item % n_out);
   const int seq = p.token_seq[t];
   if (seq < 0 || seq >= p.n_seqs) return;
   const int pos = p.positions[t];
-  const int kvh = h / (p.n_q / p.n_kv);
+  const int kvh = h_out / (n_out / p.n_kv);
   const int* bt = p.block_tables + size_t(seq) * p.max_blocks;
   float* q = s_q + warp * p.dk;
+  float first[kMaxCols];                         // MAPS = 2: the first map's output
+#pragma unroll
+  for (int map = 0; map < MAPS; ++map) {
+  const int h = h_out * MAPS + map, kh = kvh * MAPS + map;
+  __syncwarp();
   for (int i = lane; i < p.dk; i += 32) q[i] = to_f32(p.q[size_t(t) * p.q_stride + size_t(h) * p.dk + i]) * p.scale;
   __syncwarp();
   int lo = 0;
@@ -63,9 +74,10 @@ __global__ void __launch_bounds__(128) attention_simt_kernel(const Params<T> p) 
       const int b = min(key / p.block_size, p.max_blocks - 1);
       slot = long(bt[b]) * p.block_size + key % p.block_size;
       if (slot < 0 || slot >= p.cache_slots) slot = 0;
-      const T* k = p.k_cache + (size_t(slot) * p.n_kv + kvh) * p.dk;
+      const T* k = p.k_cache + (size_t(slot) * (p.n_kv * MAPS) + kh) * p.dk;
       float d = 0.f;
       for (int i = 0; i < p.dk; ++i) d = fmaf(q[i], to_f32(k[i]), d);
+      if (p.softcap > 0.f) d = act_softcap(d, p.softcap);
       s = d - slope * float(pos - key);
     }
     const float m_new = fmaxf(m, warp_max(s));
@@ -79,23 +91,40 @@ __global__ void __launch_bounds__(128) attention_simt_kernel(const Params<T> p) 
     for (int j = 0; j < n; ++j) {
       const float wj = __shfl_sync(0xffffffffu, w, j);
       const long sj = __shfl_sync(0xffffffffu, slot, j);
-      const T* v = p.v_cache + (size_t(sj) * p.n_kv + kvh) * p.dv;
+      const T* v = p.v_cache + size_t(sj) * p.v_pitch + size_t(kvh) * p.dv;
 #pragma unroll
       for (int c = 0; c < kMaxCols; ++c)
         if (c * 32 + lane < p.dv) acc[c] = fmaf(wj, to_f32(v[c * 32 + lane]), acc[c]);
     }
   }
   const float inv = 1.f / l;
+  if (MAPS == 2 && map == 0) {
+#pragma unroll
+    for (int c = 0; c < kMaxCols; ++c) first[c] = acc[c] * inv;
+    continue;
+  }
+  float s = inv;
+  if (MAPS == 2) {
+    const float f = *p.mix * inv;
+    float ss = 0.f;
+#pragma unroll
+    for (int c = 0; c < kMaxCols; ++c) {           // columns past dv hold zeros
+      acc[c] = first[c] - f * acc[c];
+      ss += acc[c] * acc[c];
+    }
+    s = rsqrtf(warp_sum(ss) / float(p.dv) + p.mix_eps) * p.mix_mult;
+  }
 #pragma unroll
   for (int c = 0; c < kMaxCols; ++c)
-    if (c * 32 + lane < p.dv) from_f32(p.out + (size_t(t) * p.n_q + h) * p.dv + c * 32 + lane, acc[c] * inv);
+    if (c * 32 + lane < p.dv) from_f32(p.out + (size_t(t) * n_out + h_out) * p.dv + c * 32 + lane, acc[c] * s);
+  }
 }
 
 template <typename T>
 static int launch(const void* q, const void* k_cache, const void* v_cache, void* out, const void* token_seq, const void* positions,
                   const void* block_tables, int rows, int n_seqs, int max_blocks, int block_size, long cache_slots, int n_q, int n_kv,
                   int dk, int dv, long q_stride, float scale, int window, int chunk, int keep_first, const void* slopes, const void* sinks,
-                  cudaStream_t st) {
+                  float softcap, long v_pitch, int maps, const void* mix, float mix_mult, float mix_eps, cudaStream_t st) {
   Params<T> p;
   p.q = static_cast<const T*>(q);
   p.k_cache = static_cast<const T*>(k_cache);
@@ -110,24 +139,32 @@ static int launch(const void* q, const void* k_cache, const void* v_cache, void*
   p.scale = scale; p.window = window; p.chunk = chunk; p.keep_first = keep_first;
   p.slopes = static_cast<const float*>(slopes);
   p.sinks = static_cast<const float*>(sinks);
-  const long blocks = (long(rows) * n_q + 3) / 4;
-  attention_simt_kernel<T><<<int(blocks), 128, 4 * dk * sizeof(float), st>>>(p);
+  p.softcap = softcap;
+  p.v_pitch = v_pitch > 0 ? v_pitch : long(n_kv) * dv;
+  p.mix = static_cast<const float*>(mix);
+  p.mix_mult = mix_mult; p.mix_eps = mix_eps;
+  const long blocks = (long(rows) * (n_q / maps) + 3) / 4;
+  if (maps == 2) attention_simt_kernel<T, 2><<<int(blocks), 128, 4 * dk * sizeof(float), st>>>(p);
+  else attention_simt_kernel<T, 1><<<int(blocks), 128, 4 * dk * sizeof(float), st>>>(p);
   return cudaGetLastError() == cudaSuccess ? 0 : -1;
 }
 
 }  // namespace xl_as
 
-// All rows of a step, prefill and decode.  `window` / `chunk` <= 0: none; `keep_first`: so many first keys stay visible; `slopes` / `sinks` [n_q] fp32 or null.
+// All rows of a step, prefill and decode.  `window` / `chunk` <= 0: none; `keep_first`: so many first keys stay visible; `slopes` /
+// `sinks` [n_q] fp32 or null; the rest as in xl_prefill_attention_ext.
 XL_API int xl_attention_simt(const void* q, const void* k_cache, const void* v_cache, void* out, const void* token_seq,
                              const void* positions, const void* block_tables, int rows, int n_seqs, int max_blocks, int block_size,
                              long cache_slots, int n_q, int n_kv, int dk, int dv, long q_stride, float scale, int window, int chunk,
-                             int keep_first, const void* slopes, const void* sinks, int f32, void* stream) {
+                             int keep_first, const void* slopes, const void* sinks, float softcap, long v_pitch, int maps, const void* mix,
+                             float mix_mult, float mix_eps, int f32, void* stream) {
   if (rows <= 0) return 0;
+  if (maps < 1 || maps > 2 || (maps == 2 && (!mix || (n_q / n_kv) % 2))) return -2;
   if (n_kv <= 0 || n_q % n_kv || dk <= 0 || dk > 2048 || dv <= 0 || dv > 32 * xl_as::kMaxCols) return -2;
   cudaStream_t st = static_cast<cudaStream_t>(stream);
   if (f32)
     return xl_as::launch<float>(q, k_cache, v_cache, out, token_seq, positions, block_tables, rows, n_seqs, max_blocks, block_size,
-                                cache_slots, n_q, n_kv, dk, dv, q_stride, scale, window, chunk, keep_first, slopes, sinks, st);
+                                cache_slots, n_q, n_kv, dk, dv, q_stride, scale, window, chunk, keep_first, slopes, sinks, softcap, v_pitch, maps, mix, mix_mult, mix_eps, st);
   return xl_as::launch<__nv_bfloat16>(q, k_cache, v_cache, out, token_seq, positions, block_tables, rows, n_seqs, max_blocks, block_size,
-                                      cache_slots, n_q, n_kv, dk, dv, q_stride, scale, window, chunk, keep_first, slopes, sinks, st);
+                                      cache_slots, n_q, n_kv, dk, dv, q_stride, scale, window, chunk, keep_first, slopes, sinks, softcap, v_pitch, maps, mix, mix_mult, mix_eps, st);
 }

@@ -211,23 +211,35 @@ __device__ __forceinline__ float warp_max(float v) {
   return v;
 }
 // Gate activations of a gated feed-forward: z * sigmoid(z), and the tanh form of gelu written with the identity
-// (1 + tanh(u)) / 2 = 1 / (1 + exp(-2u)), u = sqrt(2 / pi) (z + 0.044715 z^3).
-enum : int { ACT_SILU = 0, ACT_GELU_TANH = 1 };
-// Activations of a product without a gate.
-enum : int { ACT_NONE = 0, ACT_RELU2 = 1, ACT_TANH = 2 };
+// (1 + tanh(u)) / 2 = 1 / (1 + exp(-2u)), u = sqrt(2 / pi) (z + 0.044715 z^3).  ACT_CLAMPED: g sigmoid(1.702 g) (u + 1), the gate
+// at most `limit`, the other factor within +- limit.
+enum : int { ACT_SILU = 0, ACT_GELU_TANH = 1, ACT_CLAMPED = 2 };
+// Activations of a product without a gate.  ACT_SOFTCAP: cap * tanh(z / cap).
+enum : int { ACT_NONE = 0, ACT_RELU2 = 1, ACT_TANH = 2, ACT_SOFTCAP = 3 };
 __device__ __forceinline__ float act_relu2(float z) { const float r = fmaxf(z, 0.f); return r * r; }
 // (1 - e^(-2|z|)) / (1 + e^(-2|z|)) with the sign of z, through expm1 so that small arguments keep their relative accuracy
 __device__ __forceinline__ float act_tanh(float z) {
   const float e = expm1f(-2.f * fabsf(z));
   return copysignf(-e / (2.f + e), z);
 }
-__device__ __forceinline__ float plain_act(float z, int act) { return act == ACT_RELU2 ? act_relu2(z) : act == ACT_TANH ? act_tanh(z) : z; }
+__device__ __forceinline__ float act_softcap(float z, float cap) { return cap * act_tanh(z / cap); }
+__device__ __forceinline__ float plain_act(float z, int act, float cap) {
+  return act == ACT_RELU2 ? act_relu2(z) : act == ACT_TANH ? act_tanh(z) : act == ACT_SOFTCAP ? act_softcap(z, cap) : z;
+}
 __device__ __forceinline__ float act_silu(float z) { return z / (1.f + __expf(-z)); }
 __device__ __forceinline__ float act_gelu_tanh(float z) {
   const float u2 = -1.5957691216057308f * (z + 0.044715f * z * z * z);
   return z / (1.f + __expf(u2));
 }
+__device__ __forceinline__ float gate_clamped(float g, float u, float limit) {
+  g = fminf(g, limit);
+  u = fminf(fmaxf(u, -limit), limit);
+  return g / (1.f + __expf(-1.702f * g)) * (u + 1.f);
+}
 __device__ __forceinline__ float gate_act(float z, int act) { return act == ACT_GELU_TANH ? act_gelu_tanh(z) : act_silu(z); }
+__device__ __forceinline__ float gated(float g, float u, int act, float limit) {
+  return act == ACT_CLAMPED ? gate_clamped(g, u, limit) : gate_act(g, act) * u;
+}
 __device__ __forceinline__ uint32_t pack_bf16x2(float lo, float hi) {
   __nv_bfloat162 v = __floats2bfloat162_rn(lo, hi);
   return *reinterpret_cast<uint32_t*>(&v);

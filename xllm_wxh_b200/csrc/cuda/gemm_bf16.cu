@@ -34,9 +34,11 @@ struct GemmSmemBarriers {
 };
 
 // EPI_GEGLU: as EPI_SWIGLU with the tanh form of gelu; EPI_F32: the accumulators are stored as fp32 (C is float);
-// EPI_RELU2 / EPI_TANH: squared relu / tanh of the accumulators.
-enum { EPI_NONE = 0, EPI_BIAS = 1, EPI_SWIGLU = 2, EPI_RS_PUSH = 3, EPI_GEGLU = 4, EPI_F32 = 5, EPI_RELU2 = 6, EPI_TANH = 7 };
-__host__ __device__ constexpr bool epi_gated(int epi) { return epi == EPI_SWIGLU || epi == EPI_GEGLU; }
+// EPI_RELU2 / EPI_TANH: squared relu / tanh of the accumulators; EPI_CLAMPED: the clamped gate with limit `earg`, as
+// EPI_SWIGLU; EPI_SOFTCAP: earg * tanh(accumulator / earg).
+enum { EPI_NONE = 0, EPI_BIAS = 1, EPI_SWIGLU = 2, EPI_RS_PUSH = 3, EPI_GEGLU = 4, EPI_F32 = 5, EPI_RELU2 = 6, EPI_TANH = 7, EPI_CLAMPED = 8,
+       EPI_SOFTCAP = 9 };
+__host__ __device__ constexpr bool epi_gated(int epi) { return epi == EPI_SWIGLU || epi == EPI_GEGLU || epi == EPI_CLAMPED; }
 
 // EPI_RS_PUSH (tensor-parallel row-parallel linear): this rank's partial tile is not stored locally; each row is
 // pushed over NVLink straight from the epilogue registers into the receive buffer of the rank that owns the row
@@ -63,7 +65,30 @@ struct Grouped {
   // (both 0 for the plain "sorted rows in, sorted rows out" case)
   int c_rows_per_expert;
   int c_col_stride;
+  // Batched mode (batch_rows > 0, no table): the groups are `batch` matrices of batch_rows rows each, group e reads A at row
+  // e * a_row_stride and column e * a_col_stride and writes C at row e * c_row_stride and column e * c_col_stride.  Columns that a
+  // k-block reads past the group's own K meet zeros of W.
+  int batch, batch_rows;
+  int a_row_stride, a_col_stride, c_row_stride;
 };
+
+// Where output row block `mt` of a grouped or batched problem lies.
+struct GroupTile {
+  int expert, row0, row_end, a_row, a_col, c_row, c_col;    // rows of the group's own matrix [row0, row_end); offsets into A and C
+};
+__device__ __forceinline__ GroupTile group_tile(const Grouped& g, int mt, int M) {
+  if (g.batch_rows > 0) {
+    const int per = (g.batch_rows + 127) / 128, e = mt / per;
+    return {e, mt % per * 128, g.batch_rows, e * g.a_row_stride, e * g.a_col_stride, e * g.c_row_stride, e * g.c_col_stride};
+  }
+  if (!g.enabled) return {0, mt * 128, M, 0, 0, 0, 0};
+  const int e = g.tile_expert[mt];
+  return {e, g.tile_row0[mt], g.tile_row_end[mt], 0, 0, -e * g.c_rows_per_expert, e * g.c_col_stride};
+}
+__device__ __forceinline__ int group_m_tiles(const Grouped& g, int M) {
+  if (g.batch_rows > 0) return g.batch * ((g.batch_rows + 127) / 128);
+  return g.enabled ? *g.num_m_tiles : (M + 127) / 128;
+}
 
 // EPI_SWIGLU: W rows are interleaved in groups of 16 (16 gate rows, then the 16 matching up rows), so
 // every 32-column accumulator chunk holds both halves; the output has N/2 columns.
@@ -72,7 +97,7 @@ __global__ void __launch_bounds__(kGemmThreads, 1)
 gemm_bf16_kernel(const __grid_constant__ CUtensorMap tmA, const __grid_constant__ CUtensorMap tmB,
                  __nv_bfloat16* __restrict__ C, const __nv_bfloat16* __restrict__ bias, int M, int N, int K, int ldc,
                  int BN, int stages, int* __restrict__ status, const __grid_constant__ RsPush rs,
-                 const __grid_constant__ Grouped grp) {
+                 const __grid_constant__ Grouped grp, float earg) {
   extern __shared__ __align__(1024) uint8_t smem_raw[];
   uint8_t* smem = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(smem_raw) + 1023) & ~uintptr_t(1023));
   const int a_stage_bytes = kBM * kBK * 2;
@@ -83,7 +108,7 @@ gemm_bf16_kernel(const __grid_constant__ CUtensorMap tmA, const __grid_constant_
 
   const int warp = threadIdx.x >> 5;
   const int lane = threadIdx.x & 31;
-  const int m_tiles = grp.enabled ? *grp.num_m_tiles : (M + kBM - 1) / kBM;
+  const int m_tiles = group_m_tiles(grp, M);
   const int n_tiles = (N + BN - 1) / BN;
   const int num_tiles = m_tiles * n_tiles;
   const int k_blocks = (K + kBK - 1) / kBK;
@@ -119,10 +144,9 @@ gemm_bf16_kernel(const __grid_constant__ CUtensorMap tmA, const __grid_constant_
       uint32_t it = 0;
       bool ok = true;
       for (int tile = blockIdx.x; tile < num_tiles && ok; tile += gridDim.x) {
-        const int mt = tile % m_tiles;
-        const int m0 = grp.enabled ? grp.tile_row0[mt] : mt * kBM;
+        const GroupTile gt = group_tile(grp, tile % m_tiles, M);
         const int n0 = (tile / m_tiles) * BN;
-        const int w_row = n0 + (grp.enabled ? grp.tile_expert[mt] * N : 0);
+        const int w_row = n0 + gt.expert * N;
         for (int kb = 0; kb < k_blocks; ++kb, ++it) {
           const int s = it % stages;
           const uint32_t ph = (it / stages) & 1;
@@ -132,7 +156,7 @@ gemm_bf16_kernel(const __grid_constant__ CUtensorMap tmA, const __grid_constant_
             break;
           }
           mbar_arrive_expect_tx(&bars->full[s], a_stage_bytes + b_stage_bytes);
-          tma_load_2d(smem_a + s * a_stage_bytes, &tmA, &bars->full[s], kb * kBK, m0);
+          tma_load_2d(smem_a + s * a_stage_bytes, &tmA, &bars->full[s], gt.a_col + kb * kBK, gt.a_row + gt.row0);
           tma_load_2d(smem_b + s * b_stage_bytes, &tmB, &bars->full[s], kb * kBK, w_row);
         }
       }
@@ -185,12 +209,9 @@ gemm_bf16_kernel(const __grid_constant__ CUtensorMap tmA, const __grid_constant_
     uint32_t local_tile = 0;
     bool ok = true;
     for (int tile = blockIdx.x; tile < num_tiles && ok; tile += gridDim.x, ++local_tile) {
-      const int mt = tile % m_tiles;
-      const int m0 = grp.enabled ? grp.tile_row0[mt] : mt * kBM;
-      const int row_lim = grp.enabled ? grp.tile_row_end[mt] : M;
+      const GroupTile gt = group_tile(grp, tile % m_tiles, M);
+      const int m0 = gt.row0, row_lim = gt.row_end, c_row_off = gt.c_row, c_col_off = gt.c_col;
       const int n0 = (tile / m_tiles) * BN;
-      const int c_row_off = grp.enabled ? grp.tile_expert[mt] * grp.c_rows_per_expert : 0;
-      const int c_col_off = grp.enabled ? grp.tile_expert[mt] * grp.c_col_stride : 0;
       const uint32_t acc = local_tile & 1;
       const uint32_t acc_ph = (local_tile >> 1) & 1;
       if (!mbar_wait(&bars->tmem_full[acc], acc_ph)) {
@@ -222,17 +243,21 @@ gemm_bf16_kernel(const __grid_constant__ CUtensorMap tmA, const __grid_constant_
             for (int j = 0; j < 8; ++j) {
               float g0 = __uint_as_float(r[2 * j]), g1 = __uint_as_float(r[2 * j + 1]);
               float u0 = __uint_as_float(r[16 + 2 * j]), u1 = __uint_as_float(r[16 + 2 * j + 1]);
-              float a0 = (EPI == EPI_GEGLU ? act_gelu_tanh(g0) : act_silu(g0)) * u0;
-              float a1 = (EPI == EPI_GEGLU ? act_gelu_tanh(g1) : act_silu(g1)) * u1;
-              o[j] = pack_bf16x2(a0, a1);
+              if (EPI == EPI_CLAMPED) {
+                o[j] = pack_bf16x2(gate_clamped(g0, u0, earg), gate_clamped(g1, u1, earg));
+              } else {
+                float a0 = (EPI == EPI_GEGLU ? act_gelu_tanh(g0) : act_silu(g0)) * u0;
+                float a1 = (EPI == EPI_GEGLU ? act_gelu_tanh(g1) : act_silu(g1)) * u1;
+                o[j] = pack_bf16x2(a0, a1);
+              }
             }
-            uint4* dst = reinterpret_cast<uint4*>(C + size_t(row - c_row_off) * ldc + c_col_off + (n >> 1));
+            uint4* dst = reinterpret_cast<uint4*>(C + size_t(row + c_row_off) * ldc + c_col_off + (n >> 1));
             dst[0] = make_uint4(o[0], o[1], o[2], o[3]);
             dst[1] = make_uint4(o[4], o[5], o[6], o[7]);
           }
         } else if (EPI == EPI_F32) {
           if (row < row_lim && n < N) {
-            float* dst = reinterpret_cast<float*>(C) + size_t(row - c_row_off) * ldc + c_col_off + n;
+            float* dst = reinterpret_cast<float*>(C) + size_t(row + c_row_off) * ldc + c_col_off + n;
             if (n + width <= N && (ldc & 3) == 0) {
 #pragma unroll
               for (int j = 0; j < 8; ++j)
@@ -253,13 +278,14 @@ gemm_bf16_kernel(const __grid_constant__ CUtensorMap tmA, const __grid_constant_
               v[j] = __uint_as_float(r[j]);
               if (EPI == EPI_RELU2) v[j] = act_relu2(v[j]);
               if (EPI == EPI_TANH) v[j] = act_tanh(v[j]);
+              if (EPI == EPI_SOFTCAP) v[j] = act_softcap(v[j], earg);
             }
             if (EPI == EPI_BIAS) {
 #pragma unroll
               for (int j = 0; j < 32; ++j)
                 if (n + j < N) v[j] += __bfloat162float(__ldg(bias + n + j));
             }
-            __nv_bfloat16* dst = C + size_t(row - c_row_off) * ldc + c_col_off + n;
+            __nv_bfloat16* dst = C + size_t(row + c_row_off) * ldc + c_col_off + n;
             if (EPI == EPI_RS_PUSH && !rs.local) {
               const int owner = row / rs.shard;
               dst = rs.recv[owner] + (size_t(rs.rank) * rs.shard_cap + (row - owner * rs.shard)) * size_t(ldc) + n;
@@ -307,7 +333,7 @@ static int g_mode = 0;      // 0: choose per problem, 1: single-CTA tiles only, 
 }  // namespace xl
 // CTA-pair kernel (gemm_bf16_2cta.cu)
 extern "C" int xl_gemm_bf16_pair_launch(int epi, const void* A, const void* W, void* C, const void* bias, int M, int N, int K,
-                                        int lda, int ldw, int ldc, void* stream, const void* rs);
+                                        int lda, int ldw, int ldc, void* stream, const void* rs, float earg);
 extern "C" double xl_gemm_bf16_pair_score(int epi, int M, int N, int K, int may_split);
 namespace xl {
 
@@ -340,7 +366,7 @@ static int pick_bn(int M, int N, int sms, int epi) {
 template <int EPI>
 static int launch(const void* A, const void* W, void* C, const void* bias, int M, int N, int K, int lda, int ldw, int ldc,
                   cudaStream_t stream, const RsPush* rs_in = nullptr, const Grouped* grp_in = nullptr, int num_experts = 1,
-                  int max_m_tiles = 0) {
+                  int max_m_tiles = 0, float earg = 0.f) {
   if (M <= 0 || N <= 0 || K <= 0) return 0;
   if ((lda % 8) || (ldw % 8) || (EPI != EPI_F32 && (ldc % 8)) || (reinterpret_cast<uintptr_t>(A) & 15) || (reinterpret_cast<uintptr_t>(W) & 15) ||
       ((EPI != EPI_RS_PUSH || (rs_in && rs_in->local)) && (reinterpret_cast<uintptr_t>(C) & 15)))
@@ -357,7 +383,7 @@ static int launch(const void* A, const void* W, void* C, const void* bias, int M
       RsPush rs_copy;
       memset(&rs_copy, 0, sizeof(rs_copy));
       if (rs_in) rs_copy = *rs_in;
-      return xl_gemm_bf16_pair_launch(EPI, A, W, C, bias, M, N, K, lda, ldw, ldc, stream, rs_in ? &rs_copy : nullptr);
+      return xl_gemm_bf16_pair_launch(EPI, A, W, C, bias, M, N, K, lda, ldw, ldc, stream, rs_in ? &rs_copy : nullptr, earg);
     }
   }
   const int stage_bytes = kBM * kBK * 2 + BN * kBK * 2;
@@ -369,22 +395,46 @@ static int launch(const void* A, const void* W, void* C, const void* bias, int M
   const CUtensorMap* tb = xl_host::tmap_2d(W, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 2, uint64_t(N) * num_experts, K, ldw, BN, kBK,
                                            CU_TENSOR_MAP_SWIZZLE_128B);
   if (!ta || !tb) return -4;
-  static bool attr_set[8] = {false, false, false, false, false, false, false, false};
+  static bool attr_set = false;
   RsPush rs;
   memset(&rs, 0, sizeof(rs));
   if (rs_in) rs = *rs_in;
   Grouped grp;
   memset(&grp, 0, sizeof(grp));
   if (grp_in) grp = *grp_in;
-  if (!attr_set[EPI]) {
+  if (!attr_set) {
     cudaFuncSetAttribute(gemm_bf16_kernel<EPI>, cudaFuncAttributeMaxDynamicSharedMemorySize, 227 * 1024);
-    attr_set[EPI] = true;
+    attr_set = true;
   }
   const int m_tiles = grp_in ? max_m_tiles : (M + kBM - 1) / kBM, n_tiles = (N + BN - 1) / BN;
   const int grid = max(1, min(m_tiles * n_tiles, sms));
   gemm_bf16_kernel<EPI><<<grid, kGemmThreads, smem, stream>>>(*ta, *tb, reinterpret_cast<__nv_bfloat16*>(C),
                                                             reinterpret_cast<const __nv_bfloat16*>(bias), M, N, K, ldc, BN,
-                                                            stages, xl_host::status_word(), rs, grp);
+                                                            stages, xl_host::status_word(), rs, grp, earg);
+  return cudaGetLastError() == cudaSuccess ? 0 : -1;
+}
+
+static int launch_heads(const void* A, const void* W, void* C, int rows, int cols, int N, int K, int lda, int ldc, const Grouped& g,
+                        cudaStream_t stream) {
+  if ((lda % 8) || (ldc % 8) || ((reinterpret_cast<uintptr_t>(A) | reinterpret_cast<uintptr_t>(W) | reinterpret_cast<uintptr_t>(C)) & 15)) return -2;
+  const int sms = xl_host::sm_count(), m_tiles = g.batch * ((g.batch_rows + kBM - 1) / kBM);
+  const int BN = pick_bn(m_tiles * kBM, N, sms, EPI_NONE);
+  const int stage_bytes = kBM * kBK * 2 + BN * kBK * 2;
+  const int stages = min(kMaxStages, (200 * 1024) / stage_bytes);
+  const size_t smem = size_t(stages) * stage_bytes + sizeof(GemmSmemBarriers) + 1024;
+  const CUtensorMap* ta = xl_host::tmap_2d(A, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 2, rows, cols, lda, kBM, kBK, CU_TENSOR_MAP_SWIZZLE_128B);
+  const CUtensorMap* tb = xl_host::tmap_2d(W, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 2, uint64_t(N) * g.batch, K, K, BN, kBK, CU_TENSOR_MAP_SWIZZLE_128B);
+  if (!ta || !tb) return -4;
+  static bool attr_set = false;
+  if (!attr_set) {
+    cudaFuncSetAttribute(gemm_bf16_kernel<EPI_NONE>, cudaFuncAttributeMaxDynamicSharedMemorySize, 227 * 1024);
+    attr_set = true;
+  }
+  RsPush rs;
+  memset(&rs, 0, sizeof(rs));
+  const int grid = max(1, min(m_tiles * ((N + BN - 1) / BN), sms));
+  gemm_bf16_kernel<EPI_NONE><<<grid, kGemmThreads, smem, stream>>>(*ta, *tb, reinterpret_cast<__nv_bfloat16*>(C), nullptr, g.batch_rows, N, K, ldc, BN,
+                                                                  stages, xl_host::status_word(), rs, g, 0.f);
   return cudaGetLastError() == cudaSuccess ? 0 : -1;
 }
 
@@ -403,9 +453,12 @@ XL_API int xl_gemm_bf16_swiglu(const void* A, const void* W, void* C, int M, int
   return xl::launch<xl::EPI_SWIGLU>(A, W, C, nullptr, M, N, K, lda, ldw, ldc, static_cast<cudaStream_t>(stream));
 }
 
-// Same with a chosen gate activation (ACT_SILU / ACT_GELU_TANH).
+// Same with a chosen gate activation (ACT_SILU / ACT_GELU_TANH / ACT_CLAMPED with its limit).
 XL_API int xl_gemm_bf16_gated(const void* A, const void* W, void* C, int M, int N, int K, int lda, int ldw, int ldc, int act,
-                              void* stream) {
+                              float limit, void* stream) {
+  if (act == xl::ACT_CLAMPED)
+    return xl::launch<xl::EPI_CLAMPED>(A, W, C, nullptr, M, N, K, lda, ldw, ldc, static_cast<cudaStream_t>(stream), nullptr, nullptr, 1, 0,
+                                       limit);
   if (act == xl::ACT_GELU_TANH)
     return xl::launch<xl::EPI_GEGLU>(A, W, C, nullptr, M, N, K, lda, ldw, ldc, static_cast<cudaStream_t>(stream));
   return xl::launch<xl::EPI_SWIGLU>(A, W, C, nullptr, M, N, K, lda, ldw, ldc, static_cast<cudaStream_t>(stream));
@@ -416,9 +469,12 @@ XL_API int xl_gemm_bf16_f32(const void* A, const void* W, void* C, int M, int N,
   return xl::launch<xl::EPI_F32>(A, W, C, nullptr, M, N, K, lda, ldw, ldc, static_cast<cudaStream_t>(stream));
 }
 
-// C = act(A W^T) with an activation of the fp32 sums (ACT_RELU2 / ACT_TANH).
-XL_API int xl_gemm_bf16_act(const void* A, const void* W, void* C, int M, int N, int K, int lda, int ldw, int ldc, int act,
+// C = act(A W^T) with an activation of the fp32 sums (ACT_RELU2 / ACT_TANH / ACT_SOFTCAP with its cap).
+XL_API int xl_gemm_bf16_act(const void* A, const void* W, void* C, int M, int N, int K, int lda, int ldw, int ldc, int act, float cap,
                             void* stream) {
+  if (act == xl::ACT_SOFTCAP)
+    return xl::launch<xl::EPI_SOFTCAP>(A, W, C, nullptr, M, N, K, lda, ldw, ldc, static_cast<cudaStream_t>(stream), nullptr, nullptr, 1, 0,
+                                       cap);
   cudaStream_t st = static_cast<cudaStream_t>(stream);
   if (act == xl::ACT_RELU2) return xl::launch<xl::EPI_RELU2>(A, W, C, nullptr, M, N, K, lda, ldw, ldc, st);
   if (act == xl::ACT_TANH) return xl::launch<xl::EPI_TANH>(A, W, C, nullptr, M, N, K, lda, ldw, ldc, st);
@@ -427,12 +483,13 @@ XL_API int xl_gemm_bf16_act(const void* A, const void* W, void* C, int M, int N,
 
 // Grouped GEMM over expert-sorted rows: C[r, :] = A[r, :] * W[expert(r)]^T for the rows listed in the tile table
 // (`tile_*` arrays and `num_m_tiles` live on the device; `max_m_tiles` bounds them for the launch).
-// swiglu != 0: W holds interleaved gate/up rows and C has N/2 columns (1: silu gate, 2: tanh-gelu gate).
+// swiglu != 0: W holds interleaved gate/up rows and C has N/2 columns (1: silu gate, 2: tanh-gelu gate, 3: clamped gate).
 XL_API int xl_grouped_gemm_bf16(const void* A, const void* W, void* C, int M_cap, int N, int K, int lda, int ldc, int num_experts,
                                 const void* tile_expert, const void* tile_row0, const void* tile_row_end,
                                 const void* num_m_tiles, int max_m_tiles, int swiglu, int c_rows_per_expert, int c_col_stride,
-                                void* stream) {
+                                float limit, void* stream) {
   xl::Grouped g;
+  memset(&g, 0, sizeof(g));
   g.c_rows_per_expert = c_rows_per_expert;
   g.c_col_stride = c_col_stride;
   g.tile_expert = static_cast<const int*>(tile_expert);
@@ -441,6 +498,9 @@ XL_API int xl_grouped_gemm_bf16(const void* A, const void* W, void* C, int M_cap
   g.num_m_tiles = static_cast<const int*>(num_m_tiles);
   g.enabled = 1;
   if (max_m_tiles <= 0) return 0;
+  if (swiglu == 3)
+    return xl::launch<xl::EPI_CLAMPED>(A, W, C, nullptr, M_cap, N, K, lda, K, ldc, static_cast<cudaStream_t>(stream), nullptr, &g,
+                                       num_experts, max_m_tiles, limit);
   if (swiglu == 2)
     return xl::launch<xl::EPI_GEGLU>(A, W, C, nullptr, M_cap, N, K, lda, K, ldc, static_cast<cudaStream_t>(stream), nullptr, &g,
                                      num_experts, max_m_tiles);
@@ -449,6 +509,22 @@ XL_API int xl_grouped_gemm_bf16(const void* A, const void* W, void* C, int M_cap
                                       num_experts, max_m_tiles);
   return xl::launch<xl::EPI_NONE>(A, W, C, nullptr, M_cap, N, K, lda, K, ldc, static_cast<cudaStream_t>(stream), nullptr, &g,
                                   num_experts, max_m_tiles);
+}
+
+// Products of `heads` matrices of T rows with a weight each (W [heads, N, K]): head h reads A [T, K] at row h * a_rows, column
+// h * a_cols and writes C [T, N] at row h * c_rows, column h * c_cols, so that both may be head-major (rows = T, cols = 0) or
+// lie side by side in token-major rows (rows = 0).  All offsets and pitches are multiples of 8 columns.
+XL_API int xl_gemm_bf16_heads(const void* A, const void* W, void* C, int T, int N, int K, int lda, int ldc, int heads, int a_rows,
+                              int a_cols, int c_rows, int c_cols, void* stream) {
+  if (T <= 0 || heads <= 0) return 0;
+  if ((a_cols % 8) || (c_cols % 8) || (K % 8) || (N % 8)) return -2;
+  xl::Grouped g;
+  memset(&g, 0, sizeof(g));
+  g.batch = heads;
+  g.batch_rows = T;
+  g.a_row_stride = a_rows; g.a_col_stride = a_cols; g.c_row_stride = c_rows; g.c_col_stride = c_cols;
+  const int rows = a_rows * (heads - 1) + T, cols = a_cols * (heads - 1) + K;
+  return xl::launch_heads(A, W, C, rows, cols, N, K, lda, ldc, g, static_cast<cudaStream_t>(stream));
 }
 
 // Row-parallel GEMM whose output rows are pushed to their owner ranks (see RsPush).  `recv` / `flags` hold `tp`

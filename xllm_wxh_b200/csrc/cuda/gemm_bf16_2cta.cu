@@ -37,8 +37,9 @@ constexpr int kMaxStages = 8;
 constexpr int kThreads = 192;
 constexpr int kOutStageBytes = 4 * 2 * 2048;   // 4 epilogue warps x 2 buffers x (32 rows x 64 bytes)
 
-enum { EPI_NONE = 0, EPI_BIAS = 1, EPI_SWIGLU = 2, EPI_RS_PUSH = 3, EPI_GEGLU = 4, EPI_RELU2 = 6, EPI_TANH = 7 };   // as in gemm_bf16.cu
-__host__ __device__ constexpr bool epi_gated(int epi) { return epi == EPI_SWIGLU || epi == EPI_GEGLU; }
+enum { EPI_NONE = 0, EPI_BIAS = 1, EPI_SWIGLU = 2, EPI_RS_PUSH = 3, EPI_GEGLU = 4, EPI_RELU2 = 6, EPI_TANH = 7, EPI_CLAMPED = 8,
+       EPI_SOFTCAP = 9 };   // as in gemm_bf16.cu
+__host__ __device__ constexpr bool epi_gated(int epi) { return epi == EPI_SWIGLU || epi == EPI_GEGLU || epi == EPI_CLAMPED; }
 
 struct Barriers {
   uint64_t full[kMaxStages];
@@ -142,11 +143,12 @@ __device__ __forceinline__ void tc_commit_pair(uint64_t* bar) {
 }
 
 template <int EPI>
-__device__ __forceinline__ void act_chunk(float (&v)[32]) {
+__device__ __forceinline__ void act_chunk(float (&v)[32], float earg) {
 #pragma unroll
   for (int j = 0; j < 32; ++j) {
     if (EPI == EPI_RELU2) v[j] = act_relu2(v[j]);
     if (EPI == EPI_TANH) v[j] = act_tanh(v[j]);
+    if (EPI == EPI_SOFTCAP) v[j] = act_softcap(v[j], earg);
   }
 }
 
@@ -154,14 +156,15 @@ __device__ __forceinline__ void act_chunk(float (&v)[32]) {
 template <int EPI>
 __device__ __forceinline__ void emit_chunk(float (&v)[32], int row, int n, int width, int M, int N, int ldc,
                                            __nv_bfloat16* __restrict__ C, const __nv_bfloat16* __restrict__ bias,
-                                           const RsPush& rs) {
+                                           const RsPush& rs, float earg) {
   if (row >= M || n >= N) return;
   if (epi_gated(EPI)) {
     uint32_t o[8];
 #pragma unroll
     for (int j = 0; j < 8; ++j) {
       const float g0 = v[2 * j], g1 = v[2 * j + 1], u0 = v[16 + 2 * j], u1 = v[16 + 2 * j + 1];
-      if (EPI == EPI_GEGLU) o[j] = pack_bf16x2(act_gelu_tanh(g0) * u0, act_gelu_tanh(g1) * u1);
+      if (EPI == EPI_CLAMPED) o[j] = pack_bf16x2(gate_clamped(g0, u0, earg), gate_clamped(g1, u1, earg));
+      else if (EPI == EPI_GEGLU) o[j] = pack_bf16x2(act_gelu_tanh(g0) * u0, act_gelu_tanh(g1) * u1);
       else o[j] = pack_bf16x2(act_silu(g0) * u0, act_silu(g1) * u1);
     }
     uint4* dst = reinterpret_cast<uint4*>(C + size_t(row) * ldc + (n >> 1));
@@ -174,7 +177,7 @@ __device__ __forceinline__ void emit_chunk(float (&v)[32], int row, int n, int w
     for (int j = 0; j < 32; ++j)
       if (n + j < N) v[j] += __bfloat162float(__ldg(bias + n + j));
   }
-  act_chunk<EPI>(v);
+  act_chunk<EPI>(v, earg);
   __nv_bfloat16* dst = C + size_t(row) * ldc + n;
   if (EPI == EPI_RS_PUSH && !rs.local) {
     const int owner = row / rs.shard;
@@ -207,7 +210,7 @@ __device__ __forceinline__ void scale_chunk(float (&v)[32], int row, int n, int 
 // tensor map's swizzle (16-byte pieces XOR-ed with row bits, which also keeps the lanes' writes on distinct banks).
 template <int EPI>
 __device__ __forceinline__ void store_chunk_tma(float (&v)[32], uint8_t* stage, int lane, int row0, int n, int M, int N,
-                                                const CUtensorMap* tmC, const __nv_bfloat16* __restrict__ bias) {
+                                                const CUtensorMap* tmC, const __nv_bfloat16* __restrict__ bias, float earg) {
   if (row0 >= M || n >= N) return;                      // warp-uniform
   // the store issued two chunks ago read this buffer: it must be done with it
   if (lane == 0) tma_store_wait_read<1>();
@@ -217,7 +220,8 @@ __device__ __forceinline__ void store_chunk_tma(float (&v)[32], uint8_t* stage, 
 #pragma unroll
     for (int j = 0; j < 8; ++j) {
       const float g0 = v[2 * j], g1 = v[2 * j + 1], u0 = v[16 + 2 * j], u1 = v[16 + 2 * j + 1];
-      if (EPI == EPI_GEGLU) o[j] = pack_bf16x2(act_gelu_tanh(g0) * u0, act_gelu_tanh(g1) * u1);
+      if (EPI == EPI_CLAMPED) o[j] = pack_bf16x2(gate_clamped(g0, u0, earg), gate_clamped(g1, u1, earg));
+      else if (EPI == EPI_GEGLU) o[j] = pack_bf16x2(act_gelu_tanh(g0) * u0, act_gelu_tanh(g1) * u1);
       else o[j] = pack_bf16x2(act_silu(g0) * u0, act_silu(g1) * u1);
     }
     const int sw = (lane >> 2) & 1;                     // 32-byte swizzle: piece ^= address bit 7
@@ -229,7 +233,7 @@ __device__ __forceinline__ void store_chunk_tma(float (&v)[32], uint8_t* stage, 
       for (int j = 0; j < 32; ++j)
         if (n + j < N) v[j] += __bfloat162float(__ldg(bias + n + j));
     }
-    act_chunk<EPI>(v);
+    act_chunk<EPI>(v, earg);
     const int sw = (lane >> 1) & 3;                     // 64-byte swizzle: piece ^= address bits 8:7
 #pragma unroll
     for (int j = 0; j < 4; ++j)
@@ -251,7 +255,7 @@ gemm_bf16_pair_kernel(const __grid_constant__ CUtensorMap tmA, const __grid_cons
                       const __grid_constant__ CUtensorMap tmC, int tma_out,
                       __nv_bfloat16* __restrict__ C, const __nv_bfloat16* __restrict__ bias, int M, int N, int K, int ldc,
                       int BN, int stages, int* __restrict__ status, const __grid_constant__ RsPush rs,
-                      const __grid_constant__ SplitK sk, const __grid_constant__ Scales sc) {
+                      const __grid_constant__ SplitK sk, const __grid_constant__ Scales sc, float earg) {
   constexpr int kBKe = 128 / ESIZE;                 // elements per K block
   extern __shared__ __align__(1024) uint8_t smem_raw[];
   uint8_t* smem = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(smem_raw) + 1023) & ~uintptr_t(1023));
@@ -452,10 +456,10 @@ gemm_bf16_pair_kernel(const __grid_constant__ CUtensorMap tmA, const __grid_cons
         for (int j = 0; j < 32; ++j) v[j] = (width == 32 || j < 16) ? __uint_as_float(r[j]) : 0.f;
         if (ESIZE == 1) scale_chunk(v, row, n, M, N, sc);
         if (tma_out && width == 32) {
-          store_chunk_tma<EPI>(v, smem_out + q * 4096 + (store_seq & 1) * 2048, lane, m0 + q * 32, n, M, N, &tmC, bias);
+          store_chunk_tma<EPI>(v, smem_out + q * 4096 + (store_seq & 1) * 2048, lane, m0 + q * 32, n, M, N, &tmC, bias, earg);
           ++store_seq;
         } else {
-          emit_chunk<EPI>(v, row, n, width, M, N, ldc, C, bias, rs);
+          emit_chunk<EPI>(v, row, n, width, M, N, ldc, C, bias, rs, earg);
         }
       };
       {
@@ -523,7 +527,7 @@ gemm_bf16_pair_kernel(const __grid_constant__ CUtensorMap tmA, const __grid_cons
             }
           }
           if (ESIZE == 1) scale_chunk(v, row, n0 + c, M, N, sc);
-          emit_chunk<EPI>(v, row, n0 + c, width, M, N, ldc, C, bias, rs);
+          emit_chunk<EPI>(v, row, n0 + c, width, M, N, ldc, C, bias, rs, earg);
         }
         if (!epi_rendezvous()) { ok = false; break; }          // this split is done reading the slabs
         if (epi_tid == 0) {
@@ -633,7 +637,7 @@ static uint8_t* splitk_workspace(cudaStream_t stream) {
 
 template <int EPI, int ESIZE = 2>
 static int launch_pair(const void* A, const void* W, void* C, const void* bias, int M, int N, int K, int lda, int ldw, int ldc,
-                       cudaStream_t stream, const RsPush* rs_in, const Scales* sc_in = nullptr) {
+                       cudaStream_t stream, const RsPush* rs_in, const Scales* sc_in = nullptr, float earg = 0.f) {
   constexpr int kBKe = 128 / ESIZE;
   const int sms = xl_host::sm_count();
   const int pairs = sms / 2;
@@ -731,17 +735,17 @@ static int launch_pair(const void* A, const void* W, void* C, const void* bias, 
   cudaError_t e = cudaLaunchKernelEx(&cfg, gemm_bf16_pair_kernel<EPI, ESIZE>, *ta, *tb, tc ? *tc : *ta, tc ? 1 : 0,
                                      reinterpret_cast<__nv_bfloat16*>(C),
                                      reinterpret_cast<const __nv_bfloat16*>(bias), M, N, K, ldc, BN, stages,
-                                     xl_host::status_word(), rs, sk, sc);
+                                     xl_host::status_word(), rs, sk, sc, earg);
   return e == cudaSuccess ? 0 : -1;
 }
 
 }  // namespace xl2
 
 // Entry points used by gemm_bf16.cu's dispatch.  `epi`: 0 none, 1 bias, 2 SwiGLU (interleaved W), 3 row push (TP),
-// 4 gelu-gated (interleaved W), 6 squared relu, 7 tanh.
+// 4 gelu-gated (interleaved W), 6 squared relu, 7 tanh, 8 clamped gate (interleaved W) with limit `earg`, 9 soft cap `earg`.
 // `score` (may be null) receives the wave-fill score of the chosen tile width, comparable with the single-CTA one.
 extern "C" int xl_gemm_bf16_pair_launch(int epi, const void* A, const void* W, void* C, const void* bias, int M, int N, int K,
-                                        int lda, int ldw, int ldc, void* stream, const void* rs) {
+                                        int lda, int ldw, int ldc, void* stream, const void* rs, float earg) {
   cudaStream_t st = static_cast<cudaStream_t>(stream);
   const xl2::RsPush* r = static_cast<const xl2::RsPush*>(rs);
   switch (epi) {
@@ -752,6 +756,8 @@ extern "C" int xl_gemm_bf16_pair_launch(int epi, const void* A, const void* W, v
     case 4: return xl2::launch_pair<xl2::EPI_GEGLU>(A, W, C, bias, M, N, K, lda, ldw, ldc, st, nullptr);
     case 6: return xl2::launch_pair<xl2::EPI_RELU2>(A, W, C, bias, M, N, K, lda, ldw, ldc, st, nullptr);
     case 7: return xl2::launch_pair<xl2::EPI_TANH>(A, W, C, bias, M, N, K, lda, ldw, ldc, st, nullptr);
+    case 8: return xl2::launch_pair<xl2::EPI_CLAMPED>(A, W, C, bias, M, N, K, lda, ldw, ldc, st, nullptr, nullptr, earg);
+    case 9: return xl2::launch_pair<xl2::EPI_SOFTCAP>(A, W, C, bias, M, N, K, lda, ldw, ldc, st, nullptr, nullptr, earg);
   }
   return -2;
 }

@@ -21,7 +21,9 @@ struct Tiles {
 };
 struct Epi {
   const void* bias;            // [N] in the operands' type, or null
-  int act;                     // ACT_NONE / ACT_RELU2 / ACT_TANH, applied after the bias
+  int act;                     // ACT_NONE / ACT_RELU2 / ACT_TANH / ACT_SOFTCAP, applied after the bias
+  float cap;                   // ACT_SOFTCAP
+  long a_step, w_step, c_step; // batched (blockIdx.z): element offsets from one matrix to the next
 };
 
 template <typename T, typename TO>
@@ -29,6 +31,9 @@ __global__ void __launch_bounds__(256) gemm_simt_kernel(const T* __restrict__ A,
                                                         int N, int K, long lda, long ldw, long ldc, const Tiles g, const Epi epi) {
   __shared__ float sA[BK][BM + 4], sW[BK][BN + 4];
   int m0 = blockIdx.x * BM, m_end = M;
+  A += blockIdx.z * epi.a_step;
+  W += blockIdx.z * epi.w_step;
+  C += blockIdx.z * epi.c_step;
   const int n0 = blockIdx.y * BN;
   if (g.num_m_tiles) {                           // 128-row tiles of one expert each, two blocks per tile
     const int tile = blockIdx.x >> 1;
@@ -74,38 +79,48 @@ __global__ void __launch_bounds__(256) gemm_simt_kernel(const T* __restrict__ A,
       const int n = n0 + tx * 4 + j;
       if (n >= N) continue;
       const float b = epi.bias ? to_f32(static_cast<const T*>(epi.bias)[n]) : 0.f;
-      from_f32(C + size_t(m) * ldc + n, plain_act(acc[i][j] + b, epi.act));
+      from_f32(C + size_t(m) * ldc + n, plain_act(acc[i][j] + b, epi.act, epi.cap));
     }
   }
 }
 
 template <typename T, typename TO>
 static int launch(const void* A, const void* W, void* C, int M, int N, int K, long lda, long ldw, long ldc, const Tiles& g,
-                  const Epi& epi, int m_blocks, cudaStream_t st) {
-  const dim3 grid(m_blocks, (N + BN - 1) / BN);
-  if (grid.y > 65535) return -2;
+                  const Epi& epi, int m_blocks, cudaStream_t st, int batch = 1) {
+  const dim3 grid(m_blocks, (N + BN - 1) / BN, batch);
+  if (grid.y > 65535 || batch > 65535) return -2;
   gemm_simt_kernel<T, TO><<<grid, 256, 0, st>>>(static_cast<const T*>(A), static_cast<const T*>(W), static_cast<TO*>(C), M, N, K, lda, ldw,
                                                 ldc, g, epi);
   return cudaGetLastError() == cudaSuccess ? 0 : -1;
 }
 
 static int dispatch(const void* A, const void* W, void* C, int M, int N, int K, long lda, long ldw, long ldc, int in_f32, int out_f32,
-                    const Tiles& g, const Epi& epi, int m_blocks, cudaStream_t st) {
-  if (in_f32) return out_f32 ? launch<float, float>(A, W, C, M, N, K, lda, ldw, ldc, g, epi, m_blocks, st) : -2;
-  if (out_f32) return launch<__nv_bfloat16, float>(A, W, C, M, N, K, lda, ldw, ldc, g, epi, m_blocks, st);
-  return launch<__nv_bfloat16, __nv_bfloat16>(A, W, C, M, N, K, lda, ldw, ldc, g, epi, m_blocks, st);
+                    const Tiles& g, const Epi& epi, int m_blocks, cudaStream_t st, int batch = 1) {
+  if (in_f32) return out_f32 ? launch<float, float>(A, W, C, M, N, K, lda, ldw, ldc, g, epi, m_blocks, st, batch) : -2;
+  if (out_f32) return launch<__nv_bfloat16, float>(A, W, C, M, N, K, lda, ldw, ldc, g, epi, m_blocks, st, batch);
+  return launch<__nv_bfloat16, __nv_bfloat16>(A, W, C, M, N, K, lda, ldw, ldc, g, epi, m_blocks, st, batch);
 }
 
 }  // namespace xl_simt
 
 // in_f32: A and W are fp32 (else bf16); out_f32: C is fp32 (else bf16).  C = act(A W^T + bias), bias [N] or null.
-XL_API int xl_gemm_simt(const void* A, const void* W, void* C, const void* bias, int act, int M, int N, int K, long lda, long ldw,
+XL_API int xl_gemm_simt(const void* A, const void* W, void* C, const void* bias, int act, float cap, int M, int N, int K, long lda, long ldw,
                         long ldc, int in_f32, int out_f32, void* stream) {
   if (M <= 0 || N <= 0) return 0;
   xl_simt::Tiles g = {};
-  const xl_simt::Epi epi{bias, act};
+  const xl_simt::Epi epi{bias, act, cap, 0, 0, 0};
   return xl_simt::dispatch(A, W, C, M, N, K, lda, ldw, ldc, in_f32, out_f32, g, epi, (M + xl_simt::BM - 1) / xl_simt::BM,
                            static_cast<cudaStream_t>(stream));
+}
+
+// `batch` products of the same shape, whose A, W and C lie a_step, w_step and c_step elements apart.
+XL_API int xl_gemm_simt_batched(const void* A, const void* W, void* C, int batch, int M, int N, int K, long lda, long ldw, long ldc,
+                                long a_step, long w_step, long c_step, int f32, void* stream) {
+  if (M <= 0 || N <= 0 || batch <= 0) return 0;
+  xl_simt::Tiles g = {};
+  const xl_simt::Epi epi{nullptr, xl::ACT_NONE, 0.f, a_step, w_step, c_step};
+  return xl_simt::dispatch(A, W, C, M, N, K, lda, ldw, ldc, f32, f32, g, epi, (M + xl_simt::BM - 1) / xl_simt::BM,
+                           static_cast<cudaStream_t>(stream), batch);
 }
 
 // Grouped form: W [E, N, K] dense, the tile table of `xl_moe_sort`; `row_src` (may be null) maps a sorted row to
@@ -121,5 +136,5 @@ XL_API int xl_grouped_gemm_simt(const void* A, const void* W, void* C, int N, in
   g.num_m_tiles = static_cast<const int*>(num_m_tiles);
   g.row_src = static_cast<const int*>(row_src);
   g.row_div = row_div < 1 ? 1 : row_div;
-  return xl_simt::dispatch(A, W, C, 0, N, K, lda, K, ldc, f32, f32, g, xl_simt::Epi{nullptr, xl::ACT_NONE}, 2 * max_m_tiles, static_cast<cudaStream_t>(stream));
+  return xl_simt::dispatch(A, W, C, 0, N, K, lda, K, ldc, f32, f32, g, xl_simt::Epi{nullptr, xl::ACT_NONE, 0.f, 0, 0, 0}, 2 * max_m_tiles, static_cast<cudaStream_t>(stream));
 }

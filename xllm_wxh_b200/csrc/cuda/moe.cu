@@ -13,7 +13,7 @@ namespace xl {
 template <typename T>
 __global__ void moe_router_kernel(const T* __restrict__ logits, const float* __restrict__ bias, float* __restrict__ out_w,
                                   int* __restrict__ out_id, long long* __restrict__ load_hist, int T_tokens, int E, int top_k,
-                                  int sigmoid, int renorm, int n_group, int topk_group, int group_top2, float route_scale) {
+                                  int scoring, int renorm, int n_group, int topk_group, int group_top2, float route_scale) {
   constexpr int MAXV = 16;   // values per lane -> E <= 512
   const int lane = threadIdx.x & 31;
   const long t = (blockIdx.x * long(blockDim.x) + threadIdx.x) >> 5;
@@ -26,11 +26,13 @@ __global__ void moe_router_kernel(const T* __restrict__ logits, const float* __r
   for (int j = 0; j < MAXV; ++j) {
     const int e = j * 32 + lane;
     float v = -INFINITY;
-    if (j < per && e < E) v = float(logits[t * E + e]);
+    if (j < per && e < E) v = float(logits[t * E + e]) + (scoring == 2 && bias ? bias[e] : 0.f);
     score[j] = v;
     mx = fmaxf(mx, v);
   }
-  if (sigmoid) {
+  if (scoring == 2) {
+    // the logits themselves are ranked; the chosen ones become weights below
+  } else if (scoring == 1) {
 #pragma unroll
     for (int j = 0; j < MAXV; ++j) score[j] = (score[j] == -INFINITY) ? -INFINITY : 1.f / (1.f + __expf(-score[j]));
   } else {
@@ -52,7 +54,7 @@ __global__ void moe_router_kernel(const T* __restrict__ logits, const float* __r
 #pragma unroll
   for (int j = 0; j < MAXV; ++j) {
     const int e = j * 32 + lane;
-    sel[j] = (j < per && e < E) ? score[j] + (bias ? bias[e] : 0.f) : -INFINITY;
+    sel[j] = (j < per && e < E) ? score[j] + (bias && scoring != 2 ? bias[e] : 0.f) : -INFINITY;
   }
   // ---- group-limited selection: keep the topk_group groups with the largest score
   if (n_group > 1) {
@@ -126,12 +128,16 @@ __global__ void moe_router_kernel(const T* __restrict__ logits, const float* __r
         if (jj == j) { w = score[jj]; sel[jj] = -INFINITY; }
     }
     w = __shfl_sync(0xffffffffu, w, idx & 31);
+    if (scoring == 2) {                          // softmax over the chosen logits; the first one is the largest
+      if (k == 0) mx = w;
+      w = expf(w - mx);
+    }
     wsum += w;
     if (lane == k) { my_w = w; my_id = idx; }
   }
   if (lane < top_k) {
     float w = my_w;
-    if (renorm) w = w / fmaxf(wsum, 1e-20f);
+    if (renorm || scoring == 2) w = w / fmaxf(wsum, 1e-20f);
     out_w[t * top_k + lane] = w * route_scale;
     out_id[t * top_k + lane] = my_id;
     if (load_hist) atomicAdd(reinterpret_cast<unsigned long long*>(load_hist + my_id), 1ull);
@@ -239,10 +245,11 @@ __global__ void moe_combine_kernel(const __nv_bfloat16* __restrict__ y, const in
 
 using namespace xl;
 
-// dtype: 0 fp32 logits, 1 bf16 logits.  group_top2: a group's score is the sum of its two best selection scores instead of
+// dtype: 0 fp32 logits, 1 bf16 logits.  scoring: 0 softmax, 1 sigmoid, 2 softmax over the chosen logits only (`bias` is then part of
+// the logits).  group_top2: a group's score is the sum of its two best selection scores instead of
 // the best one.
 XL_API int xl_moe_router(const void* logits, int dtype, const void* bias, void* out_w, void* out_id, void* load_hist, int T,
-                         int E, int top_k, int sigmoid, int renorm, int n_group, int topk_group, int group_top2,
+                         int E, int top_k, int scoring, int renorm, int n_group, int topk_group, int group_top2,
                          float route_scale, void* stream) {
   if (T <= 0) return 0;
   if (E > 512 || top_k > 32 || top_k < 1 || n_group > 32 || (n_group > 1 && E % n_group)) return -2;
@@ -251,12 +258,12 @@ XL_API int xl_moe_router(const void* logits, int dtype, const void* bias, void* 
   if (dtype == 0)
     moe_router_kernel<float><<<blocks, 256, 0, st>>>(static_cast<const float*>(logits), static_cast<const float*>(bias),
                                                      static_cast<float*>(out_w), static_cast<int*>(out_id),
-                                                     static_cast<long long*>(load_hist), T, E, top_k, sigmoid, renorm, n_group,
+                                                     static_cast<long long*>(load_hist), T, E, top_k, scoring, renorm, n_group,
                                                      topk_group, group_top2, route_scale);
   else
     moe_router_kernel<__nv_bfloat16><<<blocks, 256, 0, st>>>(
         static_cast<const __nv_bfloat16*>(logits), static_cast<const float*>(bias), static_cast<float*>(out_w),
-        static_cast<int*>(out_id), static_cast<long long*>(load_hist), T, E, top_k, sigmoid, renorm, n_group, topk_group,
+        static_cast<int*>(out_id), static_cast<long long*>(load_hist), T, E, top_k, scoring, renorm, n_group, topk_group,
         group_top2, route_scale);
   return cudaGetLastError() == cudaSuccess ? 0 : -1;
 }

@@ -10,8 +10,12 @@
 // and of decoders whose sublayers are normed before only:
 //   SRC_ADD    x += scale * y                                    (no norm behind the sublayer)
 //   SRC_SET    x = y + vec, y in fp32                            (the residual is replaced by a product of itself)
+//   SRC_MOE with `add_only`  as SRC_ADD, y assembled as in SRC_MOE
+// SRC_ADD and SRC_MOE may scale y by a vector (layer scale) and add embedding rows to x (`lead`, at the head of a pass through a
+// loop); embedding rows may have a position vector; the norm's weight may be stored as its distance from `w_off`.
 // Also the kernel that follows the qkv projection where positions do not rotate anything: per-head q / k RMSNorm and the
-// write of k and v into the paged cache (q is normed in place), with norms per head or over the whole projection; the gated
+// write of k and v into the paged cache (q is normed in place), with norms per head (and a rotation behind them) or over the whole
+// projection; the norms, rotation and cache write of latent attention's down projection, and the rotation of its queries; the gated
 // activation of an unfused feed-forward; a sigmoid gate on attention's output; and the rows [x, x0] of a product that takes
 // in the residual stream.
 //
@@ -50,6 +54,16 @@ struct NormParams {
   // SRC_SET
   const float* y32;          // [rows, H]
   const float* vec;          // [H]
+  float w_off;               // joins w_next
+  const T* ls;               // SRC_ADD, SRC_MOE with add_only: [H] factor of y (null: `scale`)
+  int add_only;              // SRC_MOE: no norm behind the sublayer
+  // rows of an embedding: SRC_EMBED (tokens, table, V, scale above), and `lead` of the others
+  const int* positions;
+  const T* pos_table;        // [pos_rows, H] or null
+  int pos_rows;
+  int lead;                  // add table[token] * lead_scale + pos_table[position] to x
+  float lead_scale;
+  int keep_x;                // SRC_EMBED: x is added to instead of written
 };
 
 // sum over the block of one value per thread; `red` holds one float per warp
@@ -64,6 +78,25 @@ __device__ __forceinline__ float block_sum(float v, float* red) {
 }
 
 __device__ __forceinline__ int clamp_id(int id, int V) { return id < 0 ? 0 : (id >= V ? V - 1 : id); }
+
+// Embedding row (8 elements from column c), times s, plus its position vector.
+template <typename T>
+__device__ __forceinline__ void embed8(const NormParams<T>& p, int row, int c, float s, float (&y)[8]) {
+  load8(p.table + size_t(clamp_id(p.tokens[row], p.V)) * p.H + c, y);
+#pragma unroll
+  for (int e = 0; e < 8; ++e) y[e] *= s;
+  if (p.pos_table) {
+    float f[8];
+    load8(p.pos_table + size_t(clamp_id(p.positions[row], p.pos_rows)) * p.H + c, f);
+#pragma unroll
+    for (int e = 0; e < 8; ++e) y[e] += f[e];
+  }
+}
+template <typename T>
+__device__ __forceinline__ float embed1(const NormParams<T>& p, int row, int c, float s) {
+  const float y = to_f32(p.table[size_t(clamp_id(p.tokens[row], p.V)) * p.H + c]) * s;
+  return p.pos_table ? y + to_f32(p.pos_table[size_t(clamp_id(p.positions[row], p.pos_rows)) * p.H + c]) : y;
+}
 
 // Register-resident rows: thread i owns the 8-element vectors i, i + blockDim, ... (VPT of them).
 template <typename T, int VPT, int SRC>
@@ -84,11 +117,22 @@ __global__ void __launch_bounds__(256) sandwich_norm_kernel(const NormParams<T> 
       if (SRC == SRC_ROWS) {
         load8(p.y + size_t(row) * H + v * 8, y[i]);
       } else if (SRC == SRC_ADD) {
-        float x[8];
+        float x[8], s[8];
         load8(p.y + size_t(row) * H + v * 8, y[i]);
         load8(p.x + size_t(row) * H + v * 8, x);
+        if (p.ls) {
+          load8(p.ls + v * 8, s);
+        } else {
 #pragma unroll
-        for (int e = 0; e < 8; ++e) y[i][e] = fmaf(p.scale, y[i][e], x[e]);
+          for (int e = 0; e < 8; ++e) s[e] = p.scale;
+        }
+#pragma unroll
+        for (int e = 0; e < 8; ++e) y[i][e] = fmaf(s[e], y[i][e], x[e]);
+        if (p.lead) {
+          embed8(p, row, v * 8, p.lead_scale, x);
+#pragma unroll
+          for (int e = 0; e < 8; ++e) y[i][e] += x[e];
+        }
       } else if (SRC == SRC_SET) {
         float x[8];
         load8(p.y32 + size_t(row) * H + v * 8, y[i]);
@@ -96,9 +140,13 @@ __global__ void __launch_bounds__(256) sandwich_norm_kernel(const NormParams<T> 
 #pragma unroll
         for (int e = 0; e < 8; ++e) y[i][e] += x[e];
       } else if (SRC == SRC_EMBED) {
-        load8(p.table + size_t(clamp_id(p.tokens[row], p.V)) * H + v * 8, y[i]);
+        embed8(p, row, v * 8, p.scale, y[i]);
+        if (p.keep_x) {
+          float x[8];
+          load8(p.x + size_t(row) * H + v * 8, x);
 #pragma unroll
-        for (int e = 0; e < 8; ++e) y[i][e] *= p.scale;
+          for (int e = 0; e < 8; ++e) y[i][e] += x[e];
+        }
       } else {
         float f[8];
 #pragma unroll
@@ -117,12 +165,24 @@ __global__ void __launch_bounds__(256) sandwich_norm_kernel(const NormParams<T> 
 #pragma unroll
           for (int e = 0; e < 8; ++e) y[i][e] += wj * f[e];
         }
+        if (p.add_only) {
+          float x[8];
+          load8(p.x + size_t(row) * H + v * 8, x);
+          load8(p.ls + v * 8, f);
+#pragma unroll
+          for (int e = 0; e < 8; ++e) y[i][e] = fmaf(f[e], y[i][e], x[e]);
+          if (p.lead) {
+            embed8(p, row, v * 8, p.lead_scale, x);
+#pragma unroll
+            for (int e = 0; e < 8; ++e) y[i][e] += x[e];
+          }
+        }
       }
 #pragma unroll
       for (int e = 0; e < 8; ++e) ss += y[i][e] * y[i][e];
     }
   }
-  if (SRC == SRC_ROWS || SRC == SRC_MOE) {
+  if (SRC == SRC_ROWS || (SRC == SRC_MOE && !p.add_only)) {
     const float r_post = rsqrtf(block_sum(ss, red_a) / float(H) + p.eps);
     ss = 0.f;
 #pragma unroll
@@ -149,7 +209,7 @@ __global__ void __launch_bounds__(256) sandwich_norm_kernel(const NormParams<T> 
       load8(p.w_next + v * 8, w);
       store8(p.x + size_t(row) * H + v * 8, y[i]);
 #pragma unroll
-      for (int e = 0; e < 8; ++e) w[e] = y[i][e] * r_next * w[e];
+      for (int e = 0; e < 8; ++e) w[e] = y[i][e] * r_next * (w[e] + p.w_off);
       store8(p.h + size_t(row) * H + v * 8, w);
     }
   }
@@ -171,11 +231,13 @@ __global__ void __launch_bounds__(256) sandwich_norm_any_kernel(const NormParams
     if (SRC == SRC_ROWS) {
       y = to_f32(p.y[size_t(row) * H + i]);
     } else if (SRC == SRC_ADD) {
-      y = fmaf(p.scale, to_f32(p.y[size_t(row) * H + i]), p.x[size_t(row) * H + i]);
+      y = fmaf(p.ls ? to_f32(p.ls[i]) : p.scale, to_f32(p.y[size_t(row) * H + i]), p.x[size_t(row) * H + i]);
+      if (p.lead) y += embed1(p, row, i, p.lead_scale);
     } else if (SRC == SRC_SET) {
       y = p.y32[size_t(row) * H + i] + p.vec[i];
     } else if (SRC == SRC_EMBED) {
-      y = to_f32(p.table[size_t(clamp_id(p.tokens[row], p.V)) * H + i]) * p.scale;
+      y = embed1(p, row, i, p.scale);
+      if (p.keep_x) y += p.x[size_t(row) * H + i];
     } else {
       if (p.shared) y = to_f32(p.shared[size_t(row) * H + i]);
       if (w_id != 0.f) y += w_id * to_f32(p.h_in[size_t(row) * H + i]);
@@ -183,11 +245,15 @@ __global__ void __launch_bounds__(256) sandwich_norm_any_kernel(const NormParams
         const int r = p.dst_of[row * p.k + j];
         if (r >= 0) y += p.weights[row * p.k + j] * to_f32(p.y_exp[size_t(r) * H + i]);
       }
+      if (p.add_only) {
+        y = fmaf(to_f32(p.ls[i]), y, p.x[size_t(row) * H + i]);
+        if (p.lead) y += embed1(p, row, i, p.lead_scale);
+      }
     }
     row_cache[i] = y;
     ss += y * y;
   }
-  if (SRC == SRC_ROWS || SRC == SRC_MOE) {
+  if (SRC == SRC_ROWS || (SRC == SRC_MOE && !p.add_only)) {
     const float r_post = rsqrtf(block_sum(ss, red_a) / float(H) + p.eps);
     ss = 0.f;
     for (int i = threadIdx.x; i < H; i += blockDim.x) {
@@ -199,7 +265,7 @@ __global__ void __launch_bounds__(256) sandwich_norm_any_kernel(const NormParams
   const float r_next = rsqrtf(block_sum(ss, red_b) / float(H) + p.eps);
   for (int i = threadIdx.x; i < H; i += blockDim.x) {
     p.x[size_t(row) * H + i] = row_cache[i];
-    from_f32(p.h + size_t(row) * H + i, row_cache[i] * r_next * to_f32(p.w_next[i]));
+    from_f32(p.h + size_t(row) * H + i, row_cache[i] * r_next * (to_f32(p.w_next[i]) + p.w_off));
   }
 }
 
@@ -245,23 +311,40 @@ static NormParams<T> base_params(void* x, const void* w_post, const void* w_next
 
 // ---------------------------------------------------------------- q / k norm + cache write
 // LPH lanes per (token, head), 8 elements per lane; heads as laid out by the fused qkv projection:
-// n_q query heads of dk, n_kv key heads of dk, n_kv value heads of dv.
+// n_q query heads of dk, n_k key heads of dk, n_v value heads of dv.
+struct Rotation {
+  const float* table;        // [rows, dims] cosines of the dims / 2 pairs, then their sines (null: no rotation)
+  const int* positions;
+  int dims, rows, interleaved;
+};
+// Element i of a rotated head (v: its value, `other`: its pair's other one).
+__device__ __forceinline__ int rot_pair(const Rotation& r, int i) {
+  const int half = r.dims / 2;
+  return r.interleaved ? i ^ 1 : (i < half ? i + half : i - half);
+}
+__device__ __forceinline__ float rot_one(const Rotation& r, const float* cs, int i, float v, float other) {
+  const int half = r.dims / 2, j = r.interleaved ? i >> 1 : (i < half ? i : i - half);
+  const bool first = r.interleaved ? !(i & 1) : i < half;
+  return first ? v * cs[j] - other * cs[half + j] : v * cs[j] + other * cs[half + j];
+}
+
 template <typename T>
 __global__ void __launch_bounds__(256) qknorm_kvwrite_vec_kernel(T* __restrict__ qkv, const int* __restrict__ slots,
                                                                  const T* __restrict__ q_w, const T* __restrict__ k_w,
                                                                  T* __restrict__ k_cache, T* __restrict__ v_cache, int T_rows,
-                                                                 int n_q, int n_kv, int dk, int dv, int lph, float eps,
-                                                                 long cache_slots) {
-  const int heads = n_q + 2 * n_kv;
+                                                                 int n_q, int n_k, int n_v, int dk, int dv, int lph, float eps,
+                                                                 long cache_slots, const Rotation rot) {
+  __shared__ __align__(16) float s_rot[256 * 8];
+  const int heads = n_q + n_k + n_v;
   const long gt = blockIdx.x * long(blockDim.x) + threadIdx.x;
   const long item = gt / lph;
   const int sub = int(gt % lph);
   const bool active = item < long(T_rows) * heads;
   const int t = active ? int(item / heads) : 0, h = active ? int(item % heads) : 0;
-  const size_t row = size_t(t) * (size_t(n_q + n_kv) * dk + size_t(n_kv) * dv);
-  const bool is_v = h >= n_q + n_kv;
+  const size_t row = size_t(t) * (size_t(n_q + n_k) * dk + size_t(n_v) * dv);
+  const bool is_v = h >= n_q + n_k;
   const int dim = is_v ? dv : dk;
-  T* src = qkv + row + (is_v ? size_t(n_q + n_kv) * dk + size_t(h - n_q - n_kv) * dv : size_t(h) * dk);
+  T* src = qkv + row + (is_v ? size_t(n_q + n_k) * dk + size_t(h - n_q - n_k) * dv : size_t(h) * dk);
   const bool mine = active && sub * 8 < dim;
   float f[8] = {0, 0, 0, 0, 0, 0, 0, 0};
   if (mine) load8(src + sub * 8, f);
@@ -269,8 +352,7 @@ __global__ void __launch_bounds__(256) qknorm_kvwrite_vec_kernel(T* __restrict__
 #pragma unroll
   for (int e = 0; e < 8; ++e) ss += f[e] * f[e];
   for (int o = lph / 2; o > 0; o >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, o);
-  if (!mine) return;
-  if (!is_v) {
+  if (mine && !is_v) {
     const T* w = h >= n_q ? k_w : q_w;
     if (w) {
       const float r = rsqrtf(ss / float(dk) + eps);
@@ -280,13 +362,39 @@ __global__ void __launch_bounds__(256) qknorm_kvwrite_vec_kernel(T* __restrict__
       for (int e = 0; e < 8; ++e) f[e] = f[e] * r * wf[e];
     }
   }
+  if (rot.table) {                                // the pair's other element may lie with another lane of the head
+    float* mem = s_rot + (threadIdx.x - sub) * 8;
+    store8(mem + sub * 8, f);
+    __syncwarp();
+    if (mine && !is_v && sub * 8 < rot.dims) {
+      const float* cs = rot.table + size_t(clamp_id(rot.positions[t], rot.rows)) * rot.dims;
+      const int half = rot.dims / 2;
+      if (!rot.interleaved && half % 8 == 0) {
+        float o[8], c[8], s[8];
+        const bool first = sub * 8 < half;
+        const int j = first ? sub * 8 : sub * 8 - half;
+        load8(mem + (first ? j + half : j), o);
+        load8(cs + j, c);
+        load8(cs + half + j, s);
+#pragma unroll
+        for (int e = 0; e < 8; ++e) f[e] = first ? f[e] * c[e] - o[e] * s[e] : f[e] * c[e] + o[e] * s[e];
+      } else {
+#pragma unroll
+        for (int e = 0; e < 8; ++e) {
+          const int i = sub * 8 + e;
+          if (i < rot.dims) f[e] = rot_one(rot, cs, i, f[e], mem[rot_pair(rot, i)]);
+        }
+      }
+    }
+  }
+  if (!mine) return;
   if (h < n_q) {
     store8(src + sub * 8, f);
     return;
   }
   const int slot = slots[t];
   if (slot < 0 || slot >= cache_slots) return;
-  T* dst = is_v ? v_cache + (size_t(slot) * n_kv + (h - n_q - n_kv)) * dv : k_cache + (size_t(slot) * n_kv + (h - n_q)) * dk;
+  T* dst = is_v ? v_cache + (size_t(slot) * n_v + (h - n_q - n_k)) * dv : k_cache + (size_t(slot) * n_k + (h - n_q)) * dk;
   store8(dst + sub * 8, f);
 }
 
@@ -295,15 +403,16 @@ template <typename T>
 __global__ void __launch_bounds__(256) qknorm_kvwrite_any_kernel(T* __restrict__ qkv, const int* __restrict__ slots,
                                                                  const T* __restrict__ q_w, const T* __restrict__ k_w,
                                                                  T* __restrict__ k_cache, T* __restrict__ v_cache, int T_rows,
-                                                                 int n_q, int n_kv, int dk, int dv, float eps, long cache_slots) {
-  const int heads = n_q + 2 * n_kv, lane = threadIdx.x & 31;
+                                                                 int n_q, int n_k, int n_v, int dk, int dv, float eps, long cache_slots,
+                                                                 const Rotation rot) {
+  const int heads = n_q + n_k + n_v, lane = threadIdx.x & 31;
   const long item = (blockIdx.x * long(blockDim.x) + threadIdx.x) >> 5;
   if (item >= long(T_rows) * heads) return;
   const int t = int(item / heads), h = int(item % heads);
-  const size_t row = size_t(t) * (size_t(n_q + n_kv) * dk + size_t(n_kv) * dv);
-  const bool is_v = h >= n_q + n_kv;
+  const size_t row = size_t(t) * (size_t(n_q + n_k) * dk + size_t(n_v) * dv);
+  const bool is_v = h >= n_q + n_k;
   const int dim = is_v ? dv : dk;
-  T* src = qkv + row + (is_v ? size_t(n_q + n_kv) * dk + size_t(h - n_q - n_kv) * dv : size_t(h) * dk);
+  T* src = qkv + row + (is_v ? size_t(n_q + n_k) * dk + size_t(h - n_q - n_k) * dv : size_t(h) * dk);
   const T* w = is_v ? nullptr : (h >= n_q ? k_w : q_w);
   float r = 1.f;
   if (w) {
@@ -315,29 +424,38 @@ __global__ void __launch_bounds__(256) qknorm_kvwrite_any_kernel(T* __restrict__
   T* dst = src;
   if (h >= n_q) {
     if (slot < 0 || slot >= cache_slots) return;
-    dst = is_v ? v_cache + (size_t(slot) * n_kv + (h - n_q - n_kv)) * dv : k_cache + (size_t(slot) * n_kv + (h - n_q)) * dk;
+    dst = is_v ? v_cache + (size_t(slot) * n_v + (h - n_q - n_k)) * dv : k_cache + (size_t(slot) * n_k + (h - n_q)) * dk;
   }
-  for (int i = lane; i < dim; i += 32) {
-    const float v = to_f32(src[i]);
-    from_f32(dst + i, w ? v * r * to_f32(w[i]) : v);
+  auto value = [&](int i) { return w ? to_f32(src[i]) * r * to_f32(w[i]) : to_f32(src[i]); };
+  const int turned = rot.table && !is_v ? rot.dims : 0;
+  if (turned) {                                   // one lane per pair, so that q may be turned in place
+    const float* cs = rot.table + size_t(clamp_id(rot.positions[t], rot.rows)) * rot.dims;
+    const int half = turned / 2;
+    for (int j = lane; j < half; j += 32) {
+      const int a = rot.interleaved ? 2 * j : j, b = rot_pair(rot, a);
+      const float u = value(a), v = value(b);
+      from_f32(dst + a, rot_one(rot, cs, a, u, v));
+      from_f32(dst + b, rot_one(rot, cs, b, v, u));
+    }
   }
+  for (int i = turned + lane; i < dim; i += 32) from_f32(dst + i, value(i));
 }
 
 template <typename T>
 static int launch_qknorm(void* qkv, const void* slots, const void* q_w, const void* k_w, void* k_cache, void* v_cache, int rows, int n_q,
-                         int n_kv, int dk, int dv, float eps, long cache_slots, cudaStream_t st) {
-  const long items = long(rows) * (n_q + 2 * n_kv);
+                         int n_k, int n_v, int dk, int dv, float eps, long cache_slots, const Rotation& rot, cudaStream_t st) {
+  const long items = long(rows) * (n_q + n_k + n_v);
   const int dmax = dk > dv ? dk : dv;
-  if (dk % 8 == 0 && dv % 8 == 0 && dmax <= 256 && al16(qkv, k_cache, v_cache, q_w) && al16(k_w)) {
+  if (dk % 8 == 0 && dv % 8 == 0 && dmax <= 256 && al16(qkv, k_cache, v_cache, q_w) && al16(k_w) && (!rot.table || rot.dims % 8 == 0)) {
     int lph = 1;
     while (lph * 8 < dmax) lph *= 2;
     qknorm_kvwrite_vec_kernel<T><<<int((items * lph + 255) / 256), 256, 0, st>>>(
         static_cast<T*>(qkv), static_cast<const int*>(slots), static_cast<const T*>(q_w), static_cast<const T*>(k_w),
-        static_cast<T*>(k_cache), static_cast<T*>(v_cache), rows, n_q, n_kv, dk, dv, lph, eps, cache_slots);
+        static_cast<T*>(k_cache), static_cast<T*>(v_cache), rows, n_q, n_k, n_v, dk, dv, lph, eps, cache_slots, rot);
   } else {
     qknorm_kvwrite_any_kernel<T><<<int((items + 7) / 8), 256, 0, st>>>(
         static_cast<T*>(qkv), static_cast<const int*>(slots), static_cast<const T*>(q_w), static_cast<const T*>(k_w),
-        static_cast<T*>(k_cache), static_cast<T*>(v_cache), rows, n_q, n_kv, dk, dv, eps, cache_slots);
+        static_cast<T*>(k_cache), static_cast<T*>(v_cache), rows, n_q, n_k, n_v, dk, dv, eps, cache_slots, rot);
   }
   return cudaGetLastError() == cudaSuccess ? 0 : -1;
 }
@@ -398,6 +516,64 @@ static int launch_qknorm_all(void* qkv, const void* slots, const void* q_w, cons
   return cudaGetLastError() == cudaSuccess ? 0 : -1;
 }
 
+// ---------------------------------------------------------------- latent attention: norms, rotation and cache write of one row per CTA
+template <typename T, int V>
+__global__ void __launch_bounds__(256) latent_down_kernel(const T* __restrict__ low, const T* __restrict__ q_w, const T* __restrict__ kv_w,
+                                                          T* __restrict__ c_q, T* __restrict__ cache, const int* __restrict__ slots, int nq,
+                                                          int nc, long ld, float eps, long cache_slots, const Rotation rot) {
+  __shared__ float red_q[8], red_k[8];
+  const int t = blockIdx.x;
+  const T* row = low + size_t(t) * ld;
+  auto load = [](const T* p, float (&f)[V]) {
+    if constexpr (V == 8) load8(p, f); else f[0] = to_f32(*p);
+  };
+  auto store = [](T* p, const float (&f)[V]) {
+    if constexpr (V == 8) store8(p, f); else from_f32(p, f[0]);
+  };
+  float sq = 0.f, sk = 0.f, f[V], w[V];
+  for (int c = threadIdx.x * V; c < nq + nc; c += blockDim.x * V) {
+    load(row + c, f);
+    float s = 0.f;
+#pragma unroll
+    for (int e = 0; e < V; ++e) s += f[e] * f[e];
+    if (c < nq) sq += s; else sk += s;
+  }
+  const float rq = rsqrtf(block_sum(sq, red_q) / float(nq) + eps), rk = rsqrtf(block_sum(sk, red_k) / float(nc) + eps);
+  const int slot = slots[t];
+  const bool in = slot >= 0 && slot < cache_slots;
+  T* dst = cache + (in ? size_t(slot) : 0) * (nc + rot.dims);
+  for (int c = threadIdx.x * V; c < nq + nc; c += blockDim.x * V) {
+    load(row + c, f);
+    load(c < nq ? q_w + c : kv_w + (c - nq), w);
+#pragma unroll
+    for (int e = 0; e < V; ++e) f[e] = f[e] * (c < nq ? rq : rk) * w[e];
+    if (c < nq) store(c_q + size_t(t) * nq + c, f);
+    else if (in) store(dst + (c - nq), f);
+  }
+  const float* cs = rot.table + size_t(clamp_id(rot.positions[t], rot.rows)) * rot.dims;
+  const T* key = row + nq + nc;
+  if (in)
+    for (int i = threadIdx.x; i < rot.dims; i += blockDim.x)
+      from_f32(dst + nc + i, rot_one(rot, cs, i, to_f32(key[i]), to_f32(key[rot_pair(rot, i)])));
+}
+
+// One pair per thread; x and out may be one and the same.
+template <typename T>
+__global__ void __launch_bounds__(256) rotate_kernel(const T* __restrict__ x, T* __restrict__ out, long total, int heads, long x_row,
+                                                     long x_head, long out_row, long out_head, const Rotation rot) {
+  const int half = rot.dims / 2;
+  for (long idx = blockIdx.x * long(blockDim.x) + threadIdx.x; idx < total; idx += long(gridDim.x) * blockDim.x) {
+    const long item = idx / half, t = item / heads, h = item % heads;
+    const int j = int(idx % half), a = rot.interleaved ? 2 * j : j, b = rot_pair(rot, a);
+    const T* src = x + t * x_row + h * x_head;
+    T* dst = out + t * out_row + h * out_head;
+    const float* cs = rot.table + size_t(clamp_id(rot.positions[t], rot.rows)) * rot.dims;
+    const float u = to_f32(src[a]), v = to_f32(src[b]);
+    from_f32(dst + a, rot_one(rot, cs, a, u, v));
+    from_f32(dst + b, rot_one(rot, cs, b, v, u));
+  }
+}
+
 // ---------------------------------------------------------------- out = o * sigmoid(gate) * scale, strided rows
 template <typename T, int V>
 __global__ void __launch_bounds__(256) sigmoid_gate_kernel(const T* __restrict__ o, const T* __restrict__ gate, T* __restrict__ out,
@@ -438,16 +614,16 @@ __global__ void __launch_bounds__(256) split_rows_kernel(const float* __restrict
 
 // ---------------------------------------------------------------- gated activation: out[t, i] = act(x[t, i]) * x[t, I + i]
 template <typename T>
-__global__ void gated_act_kernel(const T* __restrict__ x, T* __restrict__ out, long total, int I, int act) {
+__global__ void gated_act_kernel(const T* __restrict__ x, T* __restrict__ out, long total, int I, int act, float limit) {
   for (long idx = blockIdx.x * long(blockDim.x) + threadIdx.x; idx < total; idx += long(gridDim.x) * blockDim.x) {
     const long t = idx / I;
     const int i = int(idx % I);
     const T* row = x + t * 2 * I;
-    from_f32(out + idx, gate_act(to_f32(row[i]), act) * to_f32(row[I + i]));
+    from_f32(out + idx, gated(to_f32(row[i]), to_f32(row[I + i]), act, limit));
   }
 }
 template <typename T>
-__global__ void gated_act_vec_kernel(const T* __restrict__ x, T* __restrict__ out, long total, int nvec, int act) {
+__global__ void gated_act_vec_kernel(const T* __restrict__ x, T* __restrict__ out, long total, int nvec, int act, float limit) {
   for (long idx = blockIdx.x * long(blockDim.x) + threadIdx.x; idx < total; idx += long(gridDim.x) * blockDim.x) {
     const long t = idx / nvec;
     const int v = int(idx % nvec);
@@ -456,18 +632,18 @@ __global__ void gated_act_vec_kernel(const T* __restrict__ x, T* __restrict__ ou
     load8(row + v * 8, g);
     load8(row + (nvec + v) * 8, u);
 #pragma unroll
-    for (int e = 0; e < 8; ++e) g[e] = gate_act(g[e], act) * u[e];
+    for (int e = 0; e < 8; ++e) g[e] = gated(g[e], u[e], act, limit);
     store8(out + idx * 8, g);
   }
 }
 template <typename T>
-static int launch_gated_act(const void* x, void* out, int rows, int I, int act, cudaStream_t st) {
+static int launch_gated_act(const void* x, void* out, int rows, int I, int act, float limit, cudaStream_t st) {
   const bool vec = I % 8 == 0 && al16(x, out);
   const long total = long(rows) * (vec ? I / 8 : I);
   long blocks = (total + 255) / 256;
   if (blocks > 148 * 16) blocks = 148 * 16;
-  if (vec) gated_act_vec_kernel<T><<<int(blocks), 256, 0, st>>>(static_cast<const T*>(x), static_cast<T*>(out), total, I / 8, act);
-  else gated_act_kernel<T><<<int(blocks), 256, 0, st>>>(static_cast<const T*>(x), static_cast<T*>(out), total, I, act);
+  if (vec) gated_act_vec_kernel<T><<<int(blocks), 256, 0, st>>>(static_cast<const T*>(x), static_cast<T*>(out), total, I / 8, act, limit);
+  else gated_act_kernel<T><<<int(blocks), 256, 0, st>>>(static_cast<const T*>(x), static_cast<T*>(out), total, I, act, limit);
   return cudaGetLastError() == cudaSuccess ? 0 : -1;
 }
 
@@ -477,19 +653,39 @@ using namespace xl_sn;
 
 // `f32` in the entry points below: 1 when the model's tensors are fp32, 0 for bf16 (the residual x is fp32 either way).
 
-// x[t] = table[tokens[t]] * scale;  h = rms(x) * w_next
-XL_API int xl_embed_rms_norm(const void* tokens, const void* table, float scale, void* x, const void* w_next, void* h, int rows, int H,
-                             int V, float eps, int f32, void* stream) {
+// Rows of an embedding: table[tokens[t]] * scale + pos_table[positions[t]] (pos_table null: none).
+struct LeadRows {
+  const void *tokens, *table, *positions, *pos_table;
+  int V, pos_rows;
+  float scale;
+};
+template <typename T>
+static void set_lead(NormParams<T>& p, const LeadRows& l) {
+  p.tokens = static_cast<const int*>(l.tokens);
+  p.table = static_cast<const T*>(l.table);
+  p.positions = static_cast<const int*>(l.positions);
+  p.pos_table = static_cast<const T*>(l.pos_table);
+  p.V = l.V;
+  p.pos_rows = l.pos_rows;
+  p.scale = p.lead_scale = l.scale;
+}
+
+// x[t] = table[tokens[t]] * scale (+ pos_table[positions[t]]), or with keep_x: x[t] += it;  h = rms(x) * (w_next + w_off)
+XL_API int xl_embed_rms_norm(const void* tokens, const void* table, float scale, const void* positions, const void* pos_table, int pos_rows,
+                             int keep_x, void* x, const void* w_next, float w_off, void* h, int rows, int H, int V, float eps, int f32,
+                             void* stream) {
   cudaStream_t st = static_cast<cudaStream_t>(stream);
-  const bool al = al16(table, x, w_next, h);
-  if (f32) {
-    auto p = base_params<float>(x, nullptr, w_next, h, H, eps);
-    p.tokens = static_cast<const int*>(tokens); p.table = static_cast<const float*>(table); p.V = V; p.scale = scale;
-    return launch_norm<float, SRC_EMBED>(p, rows, al, st);
-  }
-  auto p = base_params<__nv_bfloat16>(x, nullptr, w_next, h, H, eps);
-  p.tokens = static_cast<const int*>(tokens); p.table = static_cast<const __nv_bfloat16*>(table); p.V = V; p.scale = scale;
-  return launch_norm<__nv_bfloat16, SRC_EMBED>(p, rows, al, st);
+  const bool al = al16(table, x, w_next, h) && al16(pos_table);
+  const LeadRows l{tokens, table, positions, pos_table, V, pos_rows, scale};
+  auto go = [&](auto* tag) {
+    using E = std::remove_pointer_t<decltype(tag)>;
+    auto p = base_params<E>(x, nullptr, w_next, h, H, eps);
+    set_lead(p, l);
+    p.w_off = w_off;
+    p.keep_x = keep_x;
+    return launch_norm<E, SRC_EMBED>(p, rows, al, st);
+  };
+  return f32 ? go(static_cast<float*>(nullptr)) : go(static_cast<__nv_bfloat16*>(nullptr));
 }
 
 // x += rms(y) * w_post;  h = rms(x) * w_next
@@ -507,18 +703,51 @@ XL_API int xl_post_norm_add_norm(const void* y, void* x, const void* w_post, con
   return launch_norm<__nv_bfloat16, SRC_ROWS>(p, rows, al, st);
 }
 
-// x += mult * y;  h = rms(x) * w_next
-XL_API int xl_add_norm(const void* y, void* x, float mult, const void* w_next, void* h, int rows, int H, float eps, int f32, void* stream) {
+// x += mult * y, or ls * y element by element (ls [H], null: mult);  with `table`: x += table[tokens[t]] * lead_scale
+// (+ pos_table[positions[t]]);  h = rms(x) * (w_next + w_off)
+XL_API int xl_add_norm(const void* y, void* x, float mult, const void* ls, const void* w_next, float w_off, void* h, int rows, int H, float eps,
+                       const void* tokens, const void* table, int V, float lead_scale, const void* positions, const void* pos_table,
+                       int pos_rows, int f32, void* stream) {
   cudaStream_t st = static_cast<cudaStream_t>(stream);
-  const bool al = al16(y, x, w_next, h);
-  if (f32) {
-    auto p = base_params<float>(x, nullptr, w_next, h, H, eps);
-    p.y = static_cast<const float*>(y); p.scale = mult;
-    return launch_norm<float, SRC_ADD>(p, rows, al, st);
-  }
-  auto p = base_params<__nv_bfloat16>(x, nullptr, w_next, h, H, eps);
-  p.y = static_cast<const __nv_bfloat16*>(y); p.scale = mult;
-  return launch_norm<__nv_bfloat16, SRC_ADD>(p, rows, al, st);
+  const bool al = al16(y, x, w_next, h) && al16(ls, table, pos_table);
+  auto go = [&](auto* tag) {
+    using E = std::remove_pointer_t<decltype(tag)>;
+    auto p = base_params<E>(x, nullptr, w_next, h, H, eps);
+    if (table) set_lead(p, LeadRows{tokens, table, positions, pos_table, V, pos_rows, lead_scale});
+    p.lead = table != nullptr;
+    p.y = static_cast<const E*>(y);
+    p.scale = mult;
+    p.ls = static_cast<const E*>(ls);
+    p.w_off = w_off;
+    return launch_norm<E, SRC_ADD>(p, rows, al, st);
+  };
+  return f32 ? go(static_cast<float*>(nullptr)) : go(static_cast<__nv_bfloat16*>(nullptr));
+}
+
+// The same with y[t] = sum_j weights[t, j] * y_exp[dst_of[t, j]] (k choices, dst_of < 0: none); ls is required.
+XL_API int xl_moe_combine_add_norm(const void* y_exp, const void* dst_of, const void* weights, int k, void* x, const void* ls,
+                                   const void* w_next, float w_off, void* h, int rows, int H, float eps, const void* tokens, const void* table,
+                                   int V, float lead_scale, const void* positions, const void* pos_table, int pos_rows, int f32, void* stream) {
+  if (!ls) return -2;
+  cudaStream_t st = static_cast<cudaStream_t>(stream);
+  const bool al = al16(y_exp, x, w_next, h) && al16(ls, table, pos_table);
+  auto go = [&](auto* tag) {
+    using E = std::remove_pointer_t<decltype(tag)>;
+    auto p = base_params<E>(x, nullptr, w_next, h, H, eps);
+    if (table) set_lead(p, LeadRows{tokens, table, positions, pos_table, V, pos_rows, lead_scale});
+    p.lead = table != nullptr;
+    p.y_exp = static_cast<const E*>(y_exp);
+    p.dst_of = static_cast<const int*>(dst_of);
+    p.ids = p.dst_of;                        // any array of k entries: nothing reaches first_identity
+    p.first_identity = 0x7fffffff;
+    p.weights = static_cast<const float*>(weights);
+    p.k = k;
+    p.ls = static_cast<const E*>(ls);
+    p.w_off = w_off;
+    p.add_only = 1;
+    return launch_norm<E, SRC_MOE>(p, rows, al, st);
+  };
+  return f32 ? go(static_cast<float*>(nullptr)) : go(static_cast<__nv_bfloat16*>(nullptr));
 }
 
 // x = y + vec (y [rows, H], vec [H] fp32);  h = rms(x) * w_next
@@ -609,18 +838,62 @@ XL_API int xl_moe_combine_post_norm_add_norm(const void* y_exp, const void* dst_
   return launch_norm<__nv_bfloat16, SRC_MOE>(p, rows, al, st);
 }
 
-// Per-head RMSNorm of q (in place) and k (null weight: none), k and v to the cache slots [cache_slots, n_kv, dk | dv].
+// Per-head RMSNorm of q (in place) and k (null weight: none), then their first `rot_dims` dimensions turned by the angles of
+// rot_table [rot_rows, rot_dims] (null: not) at `positions`; k and v to the cache slots [cache_slots, n_k, dk] and [.., n_v, dv].
 XL_API int xl_qknorm_kvwrite(void* qkv, const void* slots, const void* q_w, const void* k_w, void* k_cache, void* v_cache, int rows,
-                             int n_q, int n_kv, int dk, int dv, float eps, long cache_slots, int f32, void* stream) {
+                             int n_q, int n_k, int n_v, int dk, int dv, float eps, long cache_slots, const void* rot_table,
+                             const void* positions, int rot_dims, int rot_rows, int interleaved, int f32, void* stream) {
   if (rows <= 0) return 0;
+  if (rot_table && (rot_dims > dk || rot_dims % 2 || rot_rows < 1)) return -2;
   cudaStream_t st = static_cast<cudaStream_t>(stream);
-  if (f32) return launch_qknorm<float>(qkv, slots, q_w, k_w, k_cache, v_cache, rows, n_q, n_kv, dk, dv, eps, cache_slots, st);
-  return launch_qknorm<__nv_bfloat16>(qkv, slots, q_w, k_w, k_cache, v_cache, rows, n_q, n_kv, dk, dv, eps, cache_slots, st);
+  const Rotation rot{static_cast<const float*>(rot_table), static_cast<const int*>(positions), rot_dims, rot_rows, interleaved};
+  if (f32) return launch_qknorm<float>(qkv, slots, q_w, k_w, k_cache, v_cache, rows, n_q, n_k, n_v, dk, dv, eps, cache_slots, rot, st);
+  return launch_qknorm<__nv_bfloat16>(qkv, slots, q_w, k_w, k_cache, v_cache, rows, n_q, n_k, n_v, dk, dv, eps, cache_slots, rot, st);
 }
 
-// x [rows, 2 I] = [gate | up] -> act(gate) * up; act: 0 silu, 1 tanh-gelu
-XL_API int xl_gated_act(const void* x, void* out, int rows, int I, int act, int f32, void* stream) {
+// Latent attention behind its down projection: rows (pitch ld) of nq query-latent, nc key/value-latent and rot.dims key columns.
+// Both latents are normed; the query latent goes to c_q [rows, nq], [latent | turned key part] to the cache.
+XL_API int xl_latent_down(const void* low, const void* q_w, const void* kv_w, void* c_q, void* cache, const void* slots, int rows, int nq,
+                          int nc, long ld, float eps, long cache_slots, const void* rot_table, const void* positions, int rot_dims,
+                          int rot_rows, int interleaved, int f32, void* stream) {
+  if (rows <= 0) return 0;
+  if (!rot_table || rot_dims < 2 || rot_dims % 2 || rot_rows < 1) return -2;
+  cudaStream_t st = static_cast<cudaStream_t>(stream);
+  const Rotation rot{static_cast<const float*>(rot_table), static_cast<const int*>(positions), rot_dims, rot_rows, interleaved};
+  const bool vec = nq % 8 == 0 && nc % 8 == 0 && rot_dims % 8 == 0 && ld % 8 == 0 && al16(low, q_w, kv_w, c_q) && al16(cache);
+  auto go = [&](auto* tag) {
+    using E = std::remove_pointer_t<decltype(tag)>;
+    const E *x = static_cast<const E*>(low), *qw = static_cast<const E*>(q_w), *kw = static_cast<const E*>(kv_w);
+    const int* s = static_cast<const int*>(slots);
+    const int threads = (nq + nc) / 8 > 128 ? 256 : 128;
+    if (vec) latent_down_kernel<E, 8><<<rows, threads, 0, st>>>(x, qw, kw, static_cast<E*>(c_q), static_cast<E*>(cache), s, nq, nc, ld, eps, cache_slots, rot);
+    else latent_down_kernel<E, 1><<<rows, 256, 0, st>>>(x, qw, kw, static_cast<E*>(c_q), static_cast<E*>(cache), s, nq, nc, ld, eps, cache_slots, rot);
+    return cudaGetLastError() == cudaSuccess ? 0 : -1;
+  };
+  return f32 ? go(static_cast<float*>(nullptr)) : go(static_cast<__nv_bfloat16*>(nullptr));
+}
+
+// out[t, h] = x[t, h] turned (rot_dims columns each; element strides of rows and heads given).
+XL_API int xl_rotate(const void* x, void* out, int rows, int heads, long x_row, long x_head, long out_row, long out_head,
+                     const void* rot_table, const void* positions, int rot_dims, int rot_rows, int interleaved, int f32, void* stream) {
+  if (rows <= 0 || heads <= 0) return 0;
+  if (!rot_table || rot_dims < 2 || rot_dims % 2 || rot_rows < 1) return -2;
+  const Rotation rot{static_cast<const float*>(rot_table), static_cast<const int*>(positions), rot_dims, rot_rows, interleaved};
+  const long total = long(rows) * heads * (rot_dims / 2);
+  long blocks = (total + 255) / 256;
+  if (blocks > 148 * 32) blocks = 148 * 32;
+  auto go = [&](auto* tag) {
+    using E = std::remove_pointer_t<decltype(tag)>;
+    rotate_kernel<E><<<int(blocks), 256, 0, static_cast<cudaStream_t>(stream)>>>(static_cast<const E*>(x), static_cast<E*>(out), total, heads,
+                                                                                x_row, x_head, out_row, out_head, rot);
+    return cudaGetLastError() == cudaSuccess ? 0 : -1;
+  };
+  return f32 ? go(static_cast<float*>(nullptr)) : go(static_cast<__nv_bfloat16*>(nullptr));
+}
+
+// x [rows, 2 I] = [gate | up] -> act(gate) * up; act: 0 silu, 1 tanh-gelu, 2 clamped gate with `limit`
+XL_API int xl_gated_act(const void* x, void* out, int rows, int I, int act, float limit, int f32, void* stream) {
   if (rows <= 0) return 0;
   cudaStream_t st = static_cast<cudaStream_t>(stream);
-  return f32 ? launch_gated_act<float>(x, out, rows, I, act, st) : launch_gated_act<__nv_bfloat16>(x, out, rows, I, act, st);
+  return f32 ? launch_gated_act<float>(x, out, rows, I, act, limit, st) : launch_gated_act<__nv_bfloat16>(x, out, rows, I, act, limit, st);
 }

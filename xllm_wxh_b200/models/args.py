@@ -13,8 +13,8 @@ import json
 import os
 from typing import Any, Dict, List, Optional
 
-from .layer_spec import (AttentionSpec, FeedForwardSpec, LayerSpec, ParallelSpec, SelectiveScanSpec, TimeMixSpec, attention_of,
-                         pass_starts, run_order)
+from .layer_spec import (AttentionSpec, FeedForwardSpec, LatentAttentionSpec, LayerSpec, ParallelSpec, RotarySpec, SelectiveScanSpec,
+                         TimeMixSpec, attention_of, pass_starts, run_order)
 
 @dataclasses.dataclass
 class QuantArgs:
@@ -90,13 +90,15 @@ class ModelArgs:
     # MTP
     num_nextn_predict_layers: int = 0
     quant: QuantArgs = dataclasses.field(default_factory=QuantArgs)
-    # designs that list their layers one by one (models/movolorn.py, models/falalix.py); the flat sizes above then hold maxima
-    # over the layers
+    # designs that list their layers one by one (models/movolorn.py, falalix.py, babadra.py); the flat sizes above then hold
+    # maxima over the layers
     layer_specs: List[LayerSpec] = dataclasses.field(default_factory=list)
     layer_runs: List[int] = dataclasses.field(default_factory=list)      # layer of every run, in order (layers may repeat)
     pass_starts: List[int] = dataclasses.field(default_factory=list)     # run that opens pass t of a looped range
     embedding_scale: float = 1.0
     residual_mult: float = 1.0          # factor of every sublayer's output on its way into the residual
+    position_rows: int = 0              # rows of a learned position table that joins the embedding (0: none)
+    logit_softcap: float = 0.0          # logits become softcap * tanh(logits / softcap) (0: they do not)
 
     # ------------------------------------------------------------------ derived
     @property
@@ -164,7 +166,9 @@ def _movolorn_layer(i: int, cfg: Dict[str, Any]) -> LayerSpec:
 
 def args_from_layer_list(specs: List[LayerSpec], runs: List[int], **kw) -> ModelArgs:
     """ModelArgs of a design given layer by layer; the flat sizes that the engine plans with are maxima over the layers."""
-    mix = [a for a in (attention_of(s.mixer) for s in specs) if a is not None] or [AttentionSpec(1, 1, 1, 1, 1.0)]
+    mix = [a for a in (attention_of(s.mixer) for s in specs) if a is not None]
+    mix += [AttentionSpec(s.mixer.heads, 1, s.mixer.row, s.mixer.vdim, 1.0) for s in specs if isinstance(s.mixer, LatentAttentionSpec)]
+    mix = mix or [AttentionSpec(1, 1, 1, 1, 1.0)]
     ffs = [s.mlp for s in specs if s.mlp is not None]
     inner = [f.shared_ff + f.ff * (f.top_k if f.is_moe else 1) for f in ffs]
     return ModelArgs(layer_specs=specs, layer_runs=runs, n_layers=len(runs), n_heads=max(m.heads for m in mix),
@@ -224,8 +228,64 @@ def _falalix_args(cfg: Dict[str, Any]) -> ModelArgs:
         eos_token_id=int(_first(cfg, "eos_token_id", default=-1)))
 
 
+def _rotary(cfg: Optional[Dict[str, Any]], interleaved: bool) -> Optional[RotarySpec]:
+    if not cfg or int(cfg.get("dims") or 0) == 0:
+        return None
+    s = cfg.get("scaling")
+    kw = dict(factor=float(s["factor"]), original=float(s["original"]), fast=float(s["fast"]), slow=float(s["slow"])) if s else {}
+    return RotarySpec(int(cfg["dims"]), float(cfg["base"]), interleaved, **kw)
+
+
+def _babadra_layer(i: int, cfg: Dict[str, Any]) -> LayerSpec:
+    kind, m = cfg.get("type"), cfg["mixer"]
+    if kind == "latent_attention":
+        rot = _rotary(m["rot"], True)
+        mixer = LatentAttentionSpec(heads=int(m["heads"]), dim=int(m["dim"]), rot_dim=int(m["rot_dim"]), vdim=int(m["vdim"]),
+                                    kv_rank=int(m["kv_rank"]), q_rank=int(m["q_rank"]), scale=float(m["scale"]), rot=rot)
+        if min(mixer.heads, mixer.dim, mixer.vdim, mixer.kv_rank, mixer.q_rank) < 1:
+            raise ValueError(f"layer {i}: sizes of latent attention must be positive")
+        if rot is None or rot.dims != mixer.rot_dim or rot.dims % 2:
+            raise ValueError(f"layer {i}: the rotated part has {mixer.rot_dim} dimensions, the rotation {rot.dims if rot else 0}")
+    elif kind == "attention":
+        H, G, dim, rot = int(m["heads"]), int(m["kv_heads"]), int(m["dim"]), _rotary(m.get("rot"), False)
+        if H < 1 or G < 1 or H % G:
+            raise ValueError(f"layer {i}: {H} heads do not divide over {G} key/value heads")
+        if rot is not None and (rot.dims > dim or rot.dims % 2):
+            raise ValueError(f"layer {i}: {rot.dims} rotated dimensions of {dim}")
+        mixer = AttentionSpec(heads=H, kv_heads=G, dim=dim, vdim=int(m["vdim"]), scale=float(m["scale"]), qk_norm=True, rot=rot,
+                              softcap=float(m.get("softcap") or 0.0), maps=2, diff=float(m["diff"]))
+    else:
+        raise ValueError(f"layer {i}: mixer '{kind}' is not supported")
+    f = cfg.get("mlp")
+    if not f:
+        return LayerSpec(mixer, None)
+    if f["kind"] == "dense":
+        return LayerSpec(mixer, FeedForwardSpec(ff=int(f["ff"]), act="clamped", limit=float(f["limit"])))
+    if f["kind"] != "moe":
+        raise ValueError(f"layer {i}: feed-forward '{f['kind']}' is not supported")
+    e, r = f["expert"], f["router"]
+    mlp = FeedForwardSpec(ff=int(e["ff"]), act="clamped", limit=float(e["limit"]), experts=int(r["experts"]), top_k=int(r["top"]),
+                          scoring="softmax_chosen")
+    if not 1 <= mlp.top_k <= mlp.experts:
+        raise ValueError(f"layer {i}: top {mlp.top_k} of {mlp.experts} experts")
+    return LayerSpec(mixer, mlp)
+
+
+def _babadra_args(cfg: Dict[str, Any]) -> ModelArgs:
+    specs = [_babadra_layer(i, c) for i, c in enumerate(cfg["layers"])]
+    loop = cfg.get("loop") or {}
+    span = (int(loop.get("start", 0)), int(loop.get("stop", 0)), int(loop.get("times", 1)))
+    dt = str(_first(cfg, "torch_dtype", "dtype", default="bfloat16"))
+    return args_from_layer_list(
+        specs, run_order(len(specs), *span), model_type="babadra", dtype=dt if dt in _DTYPES else "bfloat16",
+        pass_starts=pass_starts(len(specs), *span), vocab_size=int(cfg["vocab"]), hidden_size=int(cfg["width"]),
+        rms_norm_eps=float(cfg["norm"]["eps"]), embedding_scale=float((cfg.get("embedding") or {}).get("scale", 1.0)),
+        position_rows=int(cfg["max_positions"]), max_position_embeddings=int(cfg["max_positions"]),
+        logit_softcap=float(cfg.get("logit_softcap") or 0.0), eos_token_id=int(_first(cfg, "eos_token_id", default=-1)))
+
+
 _DTYPES = ("float32", "bfloat16")
-_LAYER_LISTS = {"movolorn": _movolorn_args, "falalix": _falalix_args}     # designs that are named by "architecture"
+_LAYER_LISTS = {"movolorn": _movolorn_args, "falalix": _falalix_args, "babadra": _babadra_args}     # designs that are named by "architecture"
 
 
 def args_from_hf_config(cfg: Dict[str, Any]) -> ModelArgs:
@@ -410,4 +470,18 @@ def preset(name: str) -> ModelArgs:
         spec = [par, scan] * 18
         return args_from_layer_list(spec, run_order(36), model_type="falalix", vocab_size=151936, hidden_size=4096,
                                     max_position_embeddings=40960)
+    if name in ("babadra-8b", "babadra_8b", "babadra-30b-a3b", "babadra_30b_a3b"):
+        # layer sizes of qwen3-8b / qwen3-30b-a3b: differential attention with as many query, key and value columns as theirs, and
+        # latent attention with the latent of deepseek-v3 and as many heads as theirs, turn about
+        moe = "30b" in name
+        width, kv_heads, n = (2048, 4, 48) if moe else (4096, 8, 36)
+        mlp = FeedForwardSpec(ff=768, act="clamped", limit=7.0, experts=128, top_k=8, scoring="softmax_chosen") if moe else \
+            FeedForwardSpec(ff=12288, act="clamped", limit=7.0)
+        two = AttentionSpec(heads=32, kv_heads=kv_heads, dim=64, vdim=128, scale=64 ** -0.5, qk_norm=True, rot=RotarySpec(64, 1e6),
+                            softcap=50.0, maps=2, diff=0.6)
+        lat = LatentAttentionSpec(heads=32, dim=128, rot_dim=64, vdim=128, kv_rank=512, q_rank=1536, scale=192 ** -0.5,
+                                  rot=RotarySpec(64, 1e4, True, 4.0, 8192.0))
+        return args_from_layer_list([LayerSpec(lat, mlp), LayerSpec(two, mlp)] * (n // 2), run_order(n), model_type="babadra",
+                                    vocab_size=151936, hidden_size=width, position_rows=32768, max_position_embeddings=32768,
+                                    logit_softcap=30.0)
     raise KeyError(name)

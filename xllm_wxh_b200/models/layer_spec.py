@@ -3,7 +3,32 @@ for designs whose configuration lists the layers one by one instead of giving on
 from __future__ import annotations
 
 import dataclasses
-from typing import List, Optional, Union
+import math
+from typing import List, Optional, Tuple, Union
+
+
+@dataclasses.dataclass(frozen=True)
+class RotarySpec:
+    """Rotary positions on the first `dims` dimensions of a head, optionally with YaRN scaling."""
+    dims: int
+    base: float
+    interleaved: bool = False     # pairs (2i, 2i + 1); else (i, i + dims / 2)
+    factor: float = 0.0           # YaRN: context extension (0: no scaling) ...
+    original: float = 0.0         # ... of a model of so many positions ...
+    fast: float = 32.0            # ... whose dimensions of at least so many turns over them keep their frequency
+    slow: float = 1.0             # ... and of at most so many turns are slowed by the factor
+
+    def frequencies(self) -> Tuple[List[float], float]:
+        """(angle per position of every pair, factor of cos and sin)."""
+        f = [self.base ** (-2.0 * i / self.dims) for i in range(self.dims // 2)]
+        if self.factor <= 0:
+            return f, 1.0
+
+        def dim_of(turns):        # dimension that turns so often over the original positions
+            return self.dims * math.log(self.original / (2 * math.pi * turns)) / (2 * math.log(self.base))
+        lo, hi = max(math.floor(dim_of(self.fast)), 0), min(math.ceil(dim_of(self.slow)), self.dims - 1)
+        ramp = [min(max((i - lo) / max(hi - lo, 0.001), 0.0), 1.0) for i in range(self.dims // 2)]
+        return [x / self.factor * r + x * (1 - r) for x, r in zip(f, ramp)], 0.1 * math.log(self.factor) + 1
 
 
 @dataclasses.dataclass
@@ -22,10 +47,33 @@ class AttentionSpec:
     qk_norm_all: bool = False     # RMS norm over the whole query and the whole key projection, ahead of the split into heads
     qkv_bias: bool = False        # biases on the query, key and value projections
     output_gate: bool = False     # the heads' outputs times sigmoid of a projection of the layer's input
+    rot: Optional[RotarySpec] = None
+    softcap: float = 0.0          # scores become softcap * tanh(score / softcap) (0: they do not)
+    maps: int = 1                 # 2: differential attention, two maps of query / key size `dim` per head over the same values
+    diff: float = 0.0             # constant part of the second map's factor; the normed difference is multiplied by 1 - diff
 
     def head_slopes(self) -> List[float]:
         """Geometric slopes 2^(-8 (h + 1) / H), h = 0 .. H - 1."""
         return [2.0 ** (-8.0 * (h + 1) / self.heads) for h in range(self.heads)]
+
+
+@dataclasses.dataclass
+class LatentAttentionSpec:
+    """Attention whose keys and values are projections of one latent per token, beside one rotated key part that all heads
+    share; only those two are cached."""
+    heads: int
+    dim: int                      # unrotated query / key size of a head
+    rot_dim: int                  # rotated one
+    vdim: int                     # value size of a head
+    kv_rank: int                  # size of the latent
+    q_rank: int                   # size of the queries' own latent
+    scale: float                  # factor of the whole score
+    rot: RotarySpec
+
+    @property
+    def row(self) -> int:
+        """Cached elements per token."""
+        return self.kv_rank + self.rot_dim
 
 
 @dataclasses.dataclass
@@ -56,11 +104,11 @@ class ParallelSpec:
     right_scale: float = 1.0
 
 
-Mixer = Union[AttentionSpec, SelectiveScanSpec, ParallelSpec]
+Mixer = Union[AttentionSpec, LatentAttentionSpec, SelectiveScanSpec, ParallelSpec]
 
 
 def attention_of(mixer: Mixer) -> Optional[AttentionSpec]:
-    """The attention part of a mixer: what its layer keeps in the paged cache (None: nothing)."""
+    """The attention part of a mixer: what its layer keeps in the paged cache as keys and values of heads (None: nothing)."""
     if isinstance(mixer, ParallelSpec):
         return mixer.left
     return mixer if isinstance(mixer, AttentionSpec) else None
@@ -69,14 +117,15 @@ def attention_of(mixer: Mixer) -> Optional[AttentionSpec]:
 @dataclasses.dataclass
 class FeedForwardSpec:
     ff: int                       # inner size (of one expert in a mixture)
-    act: str                      # gate activation "silu" | "gelu_tanh", or "relu2": squared relu without a gate
+    act: str                      # gate activation "silu" | "gelu_tanh" | "clamped", or "relu2": squared relu without a gate
+    limit: float = 0.0            # "clamped": bound of the gate (from above) and of the other factor (both sides)
     experts: int = 0              # experts with weights (0: a dense feed-forward)
     identity_experts: int = 0     # router outputs behind them whose expert is the identity
     top_k: int = 0
     n_group: int = 1              # equal groups of neighbouring router outputs ...
     topk_group: int = 1           # ... of which only the best ones may be chosen from
     group_score: str = "max"      # rank of a group: "max" | "top2" (sum of its two best choice scores)
-    scoring: str = "softmax"      # "softmax" | "sigmoid"
+    scoring: str = "softmax"      # "softmax" | "sigmoid" | "softmax_chosen": over the chosen logits only
     renormalize: bool = False     # chosen weights scaled to sum 1
     shared_ff: int = 0            # inner size of an expert that every token uses (0: none)
 

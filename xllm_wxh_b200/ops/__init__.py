@@ -45,14 +45,17 @@ def paged_attention(q, k_cache, v_cache, inp, scale, sliding_window=-1):
                                sliding_window)
 
 
-def paged_attention_ext(q, k_cache, v_cache, inp, scale, window=-1, chunk=0, slopes=None, sinks=None, keep_first=0):
+def paged_attention_ext(q, k_cache, v_cache, inp, scale, window=-1, chunk=0, slopes=None, sinks=None, keep_first=0, softcap=0.0, mix=None):
     """Paged attention with a per-head linear distance bias (`slopes` [Hq] fp32), a per-head sink score in the softmax
     denominator (`sinks` [Hq] fp32), keys limited to the query's chunk of `chunk` positions, first positions that stay
-    visible behind the window (`keep_first`), and a value head dimension of its own.  q [T, Hq, dk] -> [T, Hq * dv]."""
+    visible behind the window (`keep_first`), scores bounded by `softcap` * tanh(score / softcap), and a value head dimension of
+    its own.  q [T, Hq, dk] -> [T, Hq * dv].
+    `mix` = (factor fp32 [1], mult, eps): differential attention.  Query and key heads are pairs of two maps, every pair of query
+    heads has one value head's values, and its output is rms(first - factor * second) * mult: [T, Hq / 2 * dv]."""
     if q.is_cuda:
-        return _cuda().paged_attention_ext(q, k_cache, v_cache, inp, scale, window, chunk, slopes, sinks, keep_first)
+        return _cuda().paged_attention_ext(q, k_cache, v_cache, inp, scale, window, chunk, slopes, sinks, keep_first, softcap, mix)
     return ref.paged_attention(q, k_cache, v_cache, inp.q_cu, inp.kv_lens, inp.block_tables, inp.n_seqs, scale, window, chunk,
-                               slopes, sinks, keep_first)
+                               slopes, sinks, keep_first, softcap, mix)
 
 
 def sample(logits, inp):
@@ -78,7 +81,8 @@ def topk_candidates(logits, inp, id_offset: int, width: int):
 
 
 def moe_router(logits, top_k, scoring="softmax", renorm=True, bias=None, n_group=1, topk_group=1, route_scale=1.0, group_score=None):
-    """`group_score`: how a group of experts is ranked, "max" or "top2" (sum of its two best); None: top2 with a bias, else max."""
+    """`group_score`: how a group of experts is ranked, "max" or "top2" (sum of its two best); None: top2 with a bias, else max.
+    scoring "softmax_chosen": the bias is part of the logits, the weights are the softmax over the chosen ones."""
     f = _cuda().moe_router if logits.is_cuda else ref.moe_router
     extra = {} if group_score is None else {"group_score": group_score}
     return f(logits, top_k, scoring, renorm, bias, n_group, topk_group, route_scale, **extra)
@@ -101,9 +105,9 @@ def gate_up_swiglu(x, w, interleaved=False):
 
 
 # ----------------------------------------------------------------------------- sublayers normed before and after, fp32 residual
-def embed_rms_norm(ids, table, scale, w_next, eps):
-    """(fp32 residual x = table[ids] * scale, rms(x) * w_next in the table's dtype)."""
-    return (_cuda() if table.is_cuda else ref).embed_rms_norm(ids, table, scale, w_next, eps)
+def embed_rms_norm(ids, table, scale, w_next, eps, positions=None, pos_table=None, w_offset=0.0):
+    """(fp32 residual x = table[ids] * scale (+ pos_table[positions]), rms(x) * (w_next + w_offset) in the table's dtype)."""
+    return (_cuda() if table.is_cuda else ref).embed_rms_norm(ids, table, scale, w_next, eps, positions, pos_table, w_offset)
 
 
 def post_norm_add_norm(y, x, w_post, w_next, eps):
@@ -111,9 +115,10 @@ def post_norm_add_norm(y, x, w_post, w_next, eps):
     return (_cuda() if y.is_cuda else ref).post_norm_add_norm(y, x, w_post, w_next, eps)
 
 
-def qknorm_kvwrite(qkv, slots, q_w, k_w, eps, k_cache, v_cache, n_q, n_kv):
-    """Per-head RMSNorm of q and k without any rotation; k and v into the paged caches.  Returns q [T, n_q * dk]."""
-    return (_cuda() if qkv.is_cuda else ref).qknorm_kvwrite(qkv, slots, q_w, k_w, eps, k_cache, v_cache, n_q, n_kv)
+def qknorm_kvwrite(qkv, slots, q_w, k_w, eps, k_cache, v_cache, n_q, n_kv, rot=None):
+    """Per-head RMSNorm of q and k, then the rotation `rot` = (table of `ref.rotary_table`, positions, interleaved) if there is one;
+    k and v into the paged caches (n_kv key heads, as many value heads as v_cache has).  Returns q [T, n_q * dk]."""
+    return (_cuda() if qkv.is_cuda else ref).qknorm_kvwrite(qkv, slots, q_w, k_w, eps, k_cache, v_cache, n_q, n_kv, rot)
 
 
 def linear_f32(x, w):
@@ -121,12 +126,17 @@ def linear_f32(x, w):
     return (_cuda() if x.is_cuda else ref).linear_f32(x, w)
 
 
-def gated_linear(x, w, act="silu", interleaved=False):
+def gated_linear(x, w, act="silu", interleaved=False, limit=0.0):
     """act(x Wg^T) * (x Wu^T) with W = [gate rows; up rows], or the interleaved layout on CUDA (applied in the GEMM epilogue).
-    act: "silu" | "gelu_tanh"."""
+    act: "silu" | "gelu_tanh" | "clamped" (g sigmoid(1.702 g) (u + 1), g at most `limit`, u within +- limit)."""
     if not x.is_cuda:
-        return ref.gated_act(linear(x, w), act)
-    return _cuda().linear_gated(x, w, act) if interleaved else _cuda().gated_act(linear(x, w), act)
+        return ref.gated_act(linear(x, w), act, limit)
+    return _cuda().linear_gated(x, w, act, limit) if interleaved else _cuda().gated_act(linear(x, w), act, limit)
+
+
+def linear_softcap(x, w, cap):
+    """cap * tanh(x w^T / cap), applied to the fp32 sums (logits)."""
+    return (_cuda() if x.is_cuda else ref).linear_softcap(x, w, cap)
 
 
 def moe_post_norm_add_norm(h_in, w13, w2, weights, ids, shared, first_identity, x, w_post, w_next, eps, act="silu", interleaved=False):
@@ -142,9 +152,26 @@ def moe_post_norm_add_norm(h_in, w13, w2, weights, ids, shared, first_identity, 
 
 
 # ----------------------------------------------------------------------------- sublayers normed before only, fp32 residual
-def add_norm(y, x, mult, w_next, eps):
-    """x += mult * y (x fp32, in place); returns rms(x) * w_next."""
-    return (_cuda() if y.is_cuda else ref).add_norm(y, x, mult, w_next, eps)
+def add_norm(y, x, mult, w_next, eps, vec=None, w_offset=0.0, lead=None):
+    """x += mult * y, or vec * y element by element (x fp32, in place); returns rms(x) * (w_next + w_offset).
+    `lead` = (ids, table, scale, positions, pos_table): rows of the embedding that are added to x before the norm."""
+    return (_cuda() if y.is_cuda else ref).add_norm(y, x, mult, w_next, eps, vec, w_offset, lead)
+
+
+def lead_norm(lead, x, w_next, eps, w_offset=0.0):
+    """x += embedding rows (`lead` as in `add_norm`); returns rms(x) * (w_next + w_offset)."""
+    return (_cuda() if x.is_cuda else ref).lead_norm(lead, x, w_next, eps, w_offset)
+
+
+def moe_add_norm(h_in, w13, w2, weights, ids, vec, x, w_next, eps, act="silu", interleaved=False, limit=0.0, w_offset=0.0, lead=None):
+    """Mixture sublayer from its routing to the next sublayer's input: x += vec * sum_j weights_j expert_j(h_in) (x fp32, in
+    place), then as `add_norm`."""
+    if h_in.is_cuda:
+        from . import moe_cuda
+        y, dst_of = moe_cuda.expert_rows(h_in, w13, w2, ids, act, interleaved, limit)
+        return moe_cuda.combine_add_norm(y, dst_of, weights, vec, x, w_next, eps, w_offset, lead)
+    y = ref.moe_mixture(h_in, w13, w2, weights, ids, None, w13.shape[0], act, limit)
+    return ref.add_norm(y, x, 1.0, w_next, eps, vec, w_offset, lead)
 
 
 def replace_norm(y, vec, x, w_next, eps):
@@ -212,6 +239,42 @@ def selective_scan(x, dt, dt_bias, A, B, C, D, z, state, inp):
     if x.is_cuda:
         return _cuda().selective_scan(x, dt, dt_bias, A, B, C, D, z, state, inp)
     return ref.selective_scan(x, dt, dt_bias, A, B, C, D, z, state, *_seqs(inp))
+
+
+# ----------------------------------------------------------------------------- latent attention of any size
+def latent_down(low, q_rank, kv_rank, q_w, kv_w, eps, rot, slots, cache):
+    """Rows [query latent | key/value latent | key part]: both latents normed, the key part rotated (`rot` as in
+    `qknorm_kvwrite`); [latent | key part] into the cache [blocks, block, kv_rank + rot_dim].  Returns the query latent."""
+    return (_cuda() if low.is_cuda else ref).latent_down(low, q_rank, kv_rank, q_w, kv_w, eps, rot, slots, cache)
+
+
+def latent_attention(q, w_uk, w_uv, cache, inp, rot, scale, dim):
+    """Attention over cached latents in absorbed form.  q [T, H, dim + rot_dim] (unrotated part first), w_uk [H, kv_rank, dim],
+    w_uv [H, vdim, kv_rank], cache of `latent_down`.  Returns [T, H * vdim]."""
+    import torch
+    T, H, _ = q.shape
+    C, row = w_uk.shape[1], cache.shape[-1]
+    if q.is_cuda and _cuda().mla_serves(H, C, row - C, q.dtype):
+        return _cuda().latent_attention_mla(q, w_uk, w_uv, cache, inp, rot, scale, dim)
+    lat = torch.empty((T, H, row), dtype=q.dtype, device=q.device)
+    heads_linear(q[..., :dim].transpose(0, 1), w_uk, lat[..., :C].transpose(0, 1))
+    rotate_into(q[..., dim:], rot, lat[..., C:])
+    # one key / value head whose values are the first columns of its keys
+    keys = cache.unsqueeze(2)
+    o = paged_attention_ext(lat, keys, keys[..., :C], inp, scale)
+    out = torch.empty((T, H, w_uv.shape[1]), dtype=q.dtype, device=q.device)
+    heads_linear(o.view(T, H, C).transpose(0, 1), w_uv, out.transpose(0, 1))
+    return out.flatten(1)
+
+
+def heads_linear(x, w, out):
+    """out[h] = x[h] w[h]^T for every head: x [H, T, K], w [H, N, K], out [H, T, N]; x and out may be views of token-major tensors."""
+    return (_cuda() if x.is_cuda else ref).heads_linear(x, w, out)
+
+
+def rotate_into(x, rot, out):
+    """out = x rotated (x, out [T, H, d], may be strided views)."""
+    (_cuda() if x.is_cuda else ref).rotate_into(x, rot, out)
 
 
 # ----------------------------------------------------------------------------- MLA (DeepSeek)

@@ -111,7 +111,8 @@ def _tc_gemm_ok(x: torch.Tensor, w: torch.Tensor, n_align: int = 8) -> bool:
             x.stride(0) % 8 == 0 and (x.data_ptr() | w.data_ptr()) % 16 == 0)
 
 
-def _gemm_simt(x2: torch.Tensor, w: torch.Tensor, out_dtype: torch.dtype, bias: Optional[torch.Tensor] = None, act: int = 0) -> torch.Tensor:
+def _gemm_simt(x2: torch.Tensor, w: torch.Tensor, out_dtype: torch.dtype, bias: Optional[torch.Tensor] = None, act: int = 0,
+               cap: float = 0.0) -> torch.Tensor:
     """The fp32-pipe GEMM: fp32 operands, or bf16 ones of any shape; act(x w^T + bias)."""
     global launch_count
     assert x2.dtype == w.dtype and x2.dtype in (torch.float32, torch.bfloat16) and w.stride(-1) == 1
@@ -120,7 +121,7 @@ def _gemm_simt(x2: torch.Tensor, w: torch.Tensor, out_dtype: torch.dtype, bias: 
     N = w.shape[0]
     out = torch.empty((M, N), dtype=out_dtype, device=x2.device)
     if M > 0:
-        _check(lib().xl_gemm_simt(_ptr(x2), _ptr(w), _ptr(out), _ptr(bias), c_int(act), c_int(M), c_int(N), c_int(K), c_long(x2.stride(0)),
+        _check(lib().xl_gemm_simt(_ptr(x2), _ptr(w), _ptr(out), _ptr(bias), c_int(act), c_float(cap), c_int(M), c_int(N), c_int(K), c_long(x2.stride(0)),
                                   c_long(w.stride(0)), c_long(N), c_int(int(x2.dtype == torch.float32)), c_int(int(out_dtype == torch.float32)), _stream()),
                "xl_gemm_simt")
         launch_count += 1
@@ -167,30 +168,34 @@ def linear(x: torch.Tensor, w: torch.Tensor, bias: Optional[torch.Tensor] = None
     return out.reshape(x.shape[:-1] + (N,))
 
 
-PLAIN_ACTS = {"relu2": 1, "tanh": 2}
+PLAIN_ACTS = {"relu2": 1, "tanh": 2, "softcap": 3}
 
 
-def act_linear(x: torch.Tensor, w: torch.Tensor, act: str) -> torch.Tensor:
+def act_linear(x: torch.Tensor, w: torch.Tensor, act: str, cap: float = 0.0) -> torch.Tensor:
     """act(x w^T), applied to the fp32 sums in the GEMM epilogue."""
     global launch_count
     if x.stride(-1) != 1:
         x = x.contiguous()
     if not _tc_gemm_ok(x, w):
-        return _gemm_simt(x, w, x.dtype, None, PLAIN_ACTS[act])
+        return _gemm_simt(x, w, x.dtype, None, PLAIN_ACTS[act], cap)
     M, K = x.shape
     N = w.shape[0]
     out = torch.empty((M, N), dtype=torch.bfloat16, device=x.device)
     if M > 0:
         _check(lib().xl_gemm_bf16_act(_ptr(x), _ptr(w), _ptr(out), c_int(M), c_int(N), c_int(K), c_int(x.stride(0)), c_int(w.stride(0)),
-                                      c_int(N), c_int(PLAIN_ACTS[act]), _stream()), "xl_gemm_bf16_act")
+                                      c_int(N), c_int(PLAIN_ACTS[act]), c_float(cap), _stream()), "xl_gemm_bf16_act")
         launch_count += 1
     return out
 
 
-ACTS = {"silu": 0, "gelu_tanh": 1}
+def linear_softcap(x: torch.Tensor, w: torch.Tensor, cap: float) -> torch.Tensor:
+    return act_linear(x, w, "softcap", cap)
 
 
-def linear_gated(x: torch.Tensor, w_interleaved: torch.Tensor, act: str) -> torch.Tensor:
+ACTS = {"silu": 0, "gelu_tanh": 1, "clamped": 2}
+
+
+def linear_gated(x: torch.Tensor, w_interleaved: torch.Tensor, act: str, limit: float = 0.0) -> torch.Tensor:
     """gate_up GEMM whose epilogue applies act(gate) * up; `w_interleaved` from `interleave_gate_up`."""
     global launch_count
     if x.stride(-1) != 1:
@@ -200,20 +205,20 @@ def linear_gated(x: torch.Tensor, w_interleaved: torch.Tensor, act: str) -> torc
     out = torch.empty((M, N // 2), dtype=torch.bfloat16, device=x.device)
     if M > 0:
         _check(lib().xl_gemm_bf16_gated(_ptr(x), _ptr(w_interleaved), _ptr(out), c_int(M), c_int(N), c_int(K), c_int(x.stride(0)),
-                                        c_int(w_interleaved.stride(0)), c_int(out.stride(0)), c_int(ACTS[act]), _stream()),
-               "xl_gemm_bf16_gated")
+                                        c_int(w_interleaved.stride(0)), c_int(out.stride(0)), c_int(ACTS[act]), c_float(limit),
+                                        _stream()), "xl_gemm_bf16_gated")
         launch_count += 1
     return out
 
 
-def gated_act(x: torch.Tensor, act: str) -> torch.Tensor:
+def gated_act(x: torch.Tensor, act: str, limit: float = 0.0) -> torch.Tensor:
     """[T, 2I] = [gate | up] -> act(gate) * up (bf16 or fp32, any I)."""
     global launch_count
     T, I2 = x.shape
     assert x.is_contiguous()
     out = torch.empty((T, I2 // 2), dtype=x.dtype, device=x.device)
-    _check(lib().xl_gated_act(_ptr(x), _ptr(out), c_int(T), c_int(I2 // 2), c_int(ACTS[act]), c_int(int(x.dtype == torch.float32)),
-                              _stream()), "xl_gated_act")
+    _check(lib().xl_gated_act(_ptr(x), _ptr(out), c_int(T), c_int(I2 // 2), c_int(ACTS[act]), c_float(limit),
+                              c_int(int(x.dtype == torch.float32)), _stream()), "xl_gated_act")
     launch_count += 1
     return out
 
@@ -316,17 +321,39 @@ def _f32flag(t: torch.Tensor):
     return c_int(int(t.dtype == torch.float32))
 
 
-def embed_rms_norm(ids: torch.Tensor, table: torch.Tensor, scale: float, w_next: torch.Tensor, eps: float):
-    """(fp32 residual x = table[ids] * scale, rms(x) * w_next)."""
+def _embed_norm(ids, table, scale, positions, pos_table, x, keep_x, w_next, eps, w_offset) -> torch.Tensor:
     global launch_count
-    T = ids.numel()
-    V, H = table.shape
-    x = torch.empty((T, H), dtype=torch.float32, device=table.device)
+    T, H = x.shape
+    assert x.is_contiguous() and x.dtype == torch.float32 and ids.numel() == T and table.shape[1] == H and w_next.dtype == table.dtype
+    assert pos_table is None or (pos_table.dtype == table.dtype and pos_table.is_contiguous() and pos_table.shape[1] == H)
     h = torch.empty((T, H), dtype=table.dtype, device=table.device)
-    _check(lib().xl_embed_rms_norm(_ptr(ids), _ptr(table), c_float(scale), _ptr(x), _ptr(w_next), _ptr(h), c_int(T), c_int(H), c_int(V),
-                                   c_float(eps), _f32flag(table), _stream()), "xl_embed_rms_norm")
+    _check(lib().xl_embed_rms_norm(_ptr(ids), _ptr(table), c_float(scale), _ptr(positions), _ptr(pos_table),
+                                   c_int(0 if pos_table is None else pos_table.shape[0]), c_int(int(keep_x)), _ptr(x), _ptr(w_next),
+                                   c_float(w_offset), _ptr(h), c_int(T), c_int(H), c_int(table.shape[0]), c_float(eps), _f32flag(table),
+                                   _stream()), "xl_embed_rms_norm")
     launch_count += 1
-    return x, h
+    return h
+
+
+def embed_rms_norm(ids: torch.Tensor, table: torch.Tensor, scale: float, w_next: torch.Tensor, eps: float, positions=None, pos_table=None,
+                   w_offset: float = 0.0):
+    """(fp32 residual x = table[ids] * scale (+ pos_table[positions]), rms(x) * (w_next + w_offset))."""
+    x = torch.empty((ids.numel(), table.shape[1]), dtype=torch.float32, device=table.device)
+    return x, _embed_norm(ids, table, scale, positions, pos_table, x, False, w_next, eps, w_offset)
+
+
+def lead_norm(lead, x: torch.Tensor, w_next: torch.Tensor, eps: float, w_offset: float = 0.0) -> torch.Tensor:
+    """x += embedding rows; returns rms(x) * (w_next + w_offset)."""
+    return _embed_norm(*lead, x, True, w_next, eps, w_offset)
+
+
+def _lead_args(lead, H: int, dtype: torch.dtype):
+    if lead is None:
+        return c_void_p(0), c_void_p(0), c_int(0), c_float(0.0), c_void_p(0), c_void_p(0), c_int(0)
+    ids, table, scale, positions, pos = lead
+    for t in (table, pos):
+        assert t is None or (t.dtype == dtype and t.is_contiguous() and t.shape[1] == H)
+    return (_ptr(ids), _ptr(table), c_int(table.shape[0]), c_float(scale), _ptr(positions), _ptr(pos), c_int(0 if pos is None else pos.shape[0]))
 
 
 def post_norm_add_norm(y: torch.Tensor, x: torch.Tensor, w_post: torch.Tensor, w_next: torch.Tensor, eps: float) -> torch.Tensor:
@@ -341,28 +368,39 @@ def post_norm_add_norm(y: torch.Tensor, x: torch.Tensor, w_post: torch.Tensor, w
     return h
 
 
-def qknorm_kvwrite(qkv, slots, q_w, k_w, eps, k_cache, v_cache, n_q, n_kv):
-    """Per-head RMSNorm of q (in place) and k, k and v into the paged caches; returns q [T, n_q * dk] (a view of qkv)."""
+def _rot_args(rot):
+    """(table, positions, dims, rows, interleaved) of a rotation (table of `reference.rotary_table`, positions, interleaved)."""
+    if rot is None:
+        return c_void_p(0), c_void_p(0), c_int(0), c_int(0), c_int(0)
+    table, positions, interleaved = rot
+    assert table.dtype == torch.float32 and table.is_contiguous()
+    return _ptr(table), _ptr(positions), c_int(table.shape[1]), c_int(table.shape[0]), c_int(int(interleaved))
+
+
+def qknorm_kvwrite(qkv, slots, q_w, k_w, eps, k_cache, v_cache, n_q, n_kv, rot=None):
+    """Per-head RMSNorm of q (in place) and k, the rotation `rot` behind it, k and v into the paged caches; returns q
+    [T, n_q * dk] (a view of qkv)."""
     global launch_count
     T = qkv.shape[0]
-    dk, dv = k_cache.shape[-1], v_cache.shape[-1]
-    assert qkv.is_contiguous() and qkv.shape[1] == (n_q + n_kv) * dk + n_kv * dv and k_cache.dtype == qkv.dtype
+    dk, n_v, dv = k_cache.shape[-1], v_cache.shape[-2], v_cache.shape[-1]
+    assert qkv.is_contiguous() and qkv.shape[1] == (n_q + n_kv) * dk + n_v * dv and k_cache.dtype == qkv.dtype
     _check(lib().xl_qknorm_kvwrite(_ptr(qkv), _ptr(slots), _ptr(q_w), _ptr(k_w), _ptr(k_cache), _ptr(v_cache), c_int(T), c_int(n_q),
-                                   c_int(n_kv), c_int(dk), c_int(dv), c_float(eps), c_long(k_cache.shape[0] * k_cache.shape[1]),
-                                   _f32flag(qkv), _stream()), "xl_qknorm_kvwrite")
+                                   c_int(n_kv), c_int(n_v), c_int(dk), c_int(dv), c_float(eps), c_long(k_cache.shape[0] * k_cache.shape[1]),
+                                   *_rot_args(rot), _f32flag(qkv), _stream()), "xl_qknorm_kvwrite")
     launch_count += 1
     return qkv[:, :n_q * dk]
 
 
 # ----------------------------------------------------------------------------- norms before a sublayer only, fp32 residual
-def add_norm(y: torch.Tensor, x: torch.Tensor, mult: float, w_next: torch.Tensor, eps: float) -> torch.Tensor:
-    """x += mult * y in place; returns rms(x) * w_next."""
+def add_norm(y: torch.Tensor, x: torch.Tensor, mult: float, w_next: torch.Tensor, eps: float, vec: Optional[torch.Tensor] = None,
+             w_offset: float = 0.0, lead=None) -> torch.Tensor:
+    """x += mult * y, or vec * y, + the embedding rows of `lead`, in place; returns rms(x) * (w_next + w_offset)."""
     global launch_count
     T, H = y.shape
-    assert y.is_contiguous() and x.is_contiguous() and x.dtype == torch.float32
+    assert y.is_contiguous() and x.is_contiguous() and x.dtype == torch.float32 and (vec is None or vec.dtype == y.dtype)
     h = torch.empty_like(y)
-    _check(lib().xl_add_norm(_ptr(y), _ptr(x), c_float(mult), _ptr(w_next), _ptr(h), c_int(T), c_int(H), c_float(eps), _f32flag(y),
-                             _stream()), "xl_add_norm")
+    _check(lib().xl_add_norm(_ptr(y), _ptr(x), c_float(mult), _ptr(vec), _ptr(w_next), c_float(w_offset), _ptr(h), c_int(T), c_int(H),
+                             c_float(eps), *_lead_args(lead, H, y.dtype), _f32flag(y), _stream()), "xl_add_norm")
     launch_count += 1
     return h
 
@@ -411,6 +449,80 @@ def gate_into(o: torch.Tensor, gate: torch.Tensor, scale: float, out: torch.Tens
     _check(lib().xl_sigmoid_gate(_ptr(o), _ptr(gate), _ptr(out), c_int(T), c_int(n), c_long(gate.stride(0)), c_long(out.stride(0)),
                                  c_float(scale), _f32flag(o), _stream()), "xl_sigmoid_gate")
     launch_count += 1
+
+
+# ----------------------------------------------------------------------------- latent attention of any size
+def latent_down(low, q_rank, kv_rank, q_w, kv_w, eps, rot, slots, cache):
+    global launch_count
+    T = low.shape[0]
+    assert low.stride(1) == 1 and low.shape[1] == q_rank + cache.shape[-1] and cache.dtype == low.dtype
+    assert cache.shape[-1] == kv_rank + rot[0].shape[1]
+    c_q = torch.empty((T, q_rank), dtype=low.dtype, device=low.device)
+    _check(lib().xl_latent_down(_ptr(low), _ptr(q_w), _ptr(kv_w), _ptr(c_q), _ptr(cache), _ptr(slots), c_int(T), c_int(q_rank), c_int(kv_rank),
+                                c_long(low.stride(0)), c_float(eps), c_long(cache.shape[0] * cache.shape[1]), *_rot_args(rot), _f32flag(low),
+                                _stream()), "xl_latent_down")
+    launch_count += 1
+    return c_q
+
+
+def rotate_into(x, rot, out) -> None:
+    global launch_count
+    T, H, d = x.shape
+    assert out.shape == x.shape and d == rot[0].shape[1] and x.stride(2) == out.stride(2) == 1 and x.dtype == out.dtype
+    _check(lib().xl_rotate(_ptr(x), _ptr(out), c_int(T), c_int(H), c_long(x.stride(0)), c_long(x.stride(1)), c_long(out.stride(0)),
+                           c_long(out.stride(1)), *_rot_args(rot), _f32flag(x), _stream()), "xl_rotate")
+    launch_count += 1
+
+
+def _head_layout(t: torch.Tensor):
+    """(pitch, rows from one head to the next, columns from one head to the next) of a view [H, T, n], or None."""
+    H, T, n = t.shape
+    if t.stride(2) != 1:
+        return None
+    if t.stride(0) == T * t.stride(1) and t.stride(1) >= n:
+        return t.stride(1), T, 0                      # head-major
+    return (t.stride(1), 0, t.stride(0)) if t.stride(1) >= (H - 1) * t.stride(0) + n else None
+
+
+def heads_linear(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor) -> torch.Tensor:
+    """out[h] = x[h] w[h]^T: x [H, T, K], w [H, N, K], out [H, T, N]; x and out may be views of token-major tensors."""
+    global launch_count
+    H, T, K = x.shape
+    N = w.shape[1]
+    assert w.shape == (H, N, K) and w.is_contiguous() and out.shape == (H, T, N) and x.dtype == w.dtype == out.dtype
+    assert x.stride(2) == out.stride(2) == 1
+    if T == 0:
+        return out
+    a, c = _head_layout(x), _head_layout(out)
+    if (x.dtype == torch.bfloat16 and a and c and K % 8 == 0 and N % 8 == 0 and a[0] % 8 == 0 and a[2] % 8 == 0 and c[0] % 8 == 0 and
+            c[2] % 8 == 0 and (x.data_ptr() | w.data_ptr() | out.data_ptr()) % 16 == 0):
+        _check(lib().xl_gemm_bf16_heads(_ptr(x), _ptr(w), _ptr(out), c_int(T), c_int(N), c_int(K), c_int(a[0]), c_int(c[0]), c_int(H),
+                                        c_int(a[1]), c_int(a[2]), c_int(c[1]), c_int(c[2]), _stream()), "xl_gemm_bf16_heads")
+    else:
+        _check(lib().xl_gemm_simt_batched(_ptr(x), _ptr(w), _ptr(out), c_int(H), c_int(T), c_int(N), c_int(K), c_long(x.stride(1)), c_long(K),
+                                          c_long(out.stride(1)), c_long(x.stride(0)), c_long(N * K), c_long(out.stride(0)), _f32flag(x),
+                                          _stream()), "xl_gemm_simt_batched")
+    launch_count += 1
+    return out
+
+
+def mla_serves(heads: int, kv_rank: int, rot_dim: int, dtype: torch.dtype) -> bool:
+    """Whether the kernels of `mla_attention` serve a latent attention of these sizes."""
+    return dtype == torch.bfloat16 and kv_rank == 512 and rot_dim == 64 and ((heads <= 128 and 128 % heads == 0) or heads % 16 == 0)
+
+
+def latent_attention_mla(q, w_uk, w_uv, cache, inp, rot, scale, dim):
+    """`ops.latent_attention` through the head-major kernels of `mla_attention`."""
+    T, H, _ = q.shape
+    C = w_uk.shape[1]
+    lat = torch.empty((H, T, C), dtype=q.dtype, device=q.device)
+    heads_linear(q[..., :dim].transpose(0, 1), w_uk, lat)
+    q_rot = torch.empty((H, T, q.shape[2] - dim), dtype=q.dtype, device=q.device)
+    rotate_into(q[..., dim:], rot, q_rot.transpose(0, 1))
+    o = mla_attention(lat, q_rot, cache, inp, scale, C)
+    out = torch.empty((T, H, w_uv.shape[1]), dtype=q.dtype, device=q.device)
+    heads_linear(o, w_uv, out.transpose(0, 1))
+    return out.flatten(1)
 
 
 # ----------------------------------------------------------------------------- recurrent layers
@@ -588,19 +700,27 @@ def paged_attention(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tenso
 
 
 def paged_attention_ext(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tensor, inp, scale: float, window: int = -1, chunk: int = 0,
-                        slopes: Optional[torch.Tensor] = None, sinks: Optional[torch.Tensor] = None, keep_first: int = 0) -> torch.Tensor:
+                        slopes: Optional[torch.Tensor] = None, sinks: Optional[torch.Tensor] = None, keep_first: int = 0,
+                        softcap: float = 0.0, mix=None) -> torch.Tensor:
     """Paged attention with score extensions and a value dimension of its own: q [T, Hq, dk] (may be a view of the qkv
-    buffer), caches [blocks, block, Hkv, dk | dv] -> [T, Hq * dv].  score = scale q.k - slopes[h] * distance; keys of the
-    query's own chunk of `chunk` positions only (0: all); `keep_first` first keys stay visible behind the window;
-    exp(sinks[h]) joins the softmax denominator.  bf16 tensors with head dimensions up to 128 (multiples of 8) run on the tensor-core kernels, anything else on the fp32-pipe kernel."""
+    buffer), caches [blocks, block, Hkv, dk | dv] -> [T, Hq * dv].  score = scale q.k (bounded by softcap tanh(. / softcap)) -
+    slopes[h] * distance; keys of the query's own chunk of `chunk` positions only (0: all); `keep_first` first keys stay visible
+    behind the window; exp(sinks[h]) joins the softmax denominator; `mix`: differential attention (see `ops`).  The values may be
+    a view of the keys.  bf16 tensors with head dimensions up to 256 (128 with `mix`; multiples of 8) run on the tensor-core
+    kernels, anything else on the fp32-pipe kernel."""
     global launch_count
     from ..framework.step_input import H_NUM_DECODE, H_NUM_SEQS
     T, Hq, dk = q.shape
-    block_size, n_kv, dv = k_cache.shape[1], k_cache.shape[2], v_cache.shape[3]
+    block_size, n_kv, dv = k_cache.shape[1], v_cache.shape[2], v_cache.shape[3]
+    maps = 1 if mix is None else 2
+    assert k_cache.is_contiguous() and k_cache.shape[2] == n_kv * maps and v_cache.stride(3) == 1 and v_cache.stride(0) == block_size * v_cache.stride(1)
+    assert v_cache.stride(2) == dv or n_kv == 1
     L, padded = inp.layout, inp.padded
     for t in (slopes, sinks):
         assert t is None or (t.dtype == torch.float32 and t.numel() == Hq and t.is_contiguous())
-    out = (torch.zeros if padded else torch.empty)((T, Hq * dv), dtype=q.dtype, device=q.device)
+    out = (torch.zeros if padded else torch.empty)((T, Hq // maps * dv), dtype=q.dtype, device=q.device)
+    factor, mult, eps = mix if mix is not None else (None, 0.0, 0.0)
+    ext = (c_float(softcap), c_long(v_cache.stride(1)), c_int(maps), _ptr(factor), c_float(mult), c_float(eps))
     n_dec = inp.B if padded else inp.n_decode
     n_all = inp.B if padded else inp.n_seqs
     has_prefill = inp.has_prefill if padded else n_all > n_dec
@@ -611,9 +731,10 @@ def paged_attention_ext(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.T
                                        _ptr(inp.block_tables), c_int(T), c_int(n_all), c_int(L.MB_cap), c_int(block_size),
                                        c_long(k_cache.shape[0] * block_size), c_int(Hq), c_int(n_kv), c_int(dk), c_int(dv),
                                        c_long(q_stride), c_float(scale), c_int(window), c_int(chunk), c_int(keep_first), _ptr(slopes), _ptr(sinks),
-                                       _f32flag(q), _stream()), "xl_attention_simt")
+                                       *ext, _f32flag(q), _stream()), "xl_attention_simt")
         return out
-    if q.dtype == torch.float32 or dk % 8 or dv % 8 or dk > 128 or dv > 128 or q.stride(1) != dk or Hq // n_kv > 16:
+    most = 256 if mix is None else 128
+    if q.dtype == torch.float32 or dk % 8 or dv % 8 or dk > most or dv > most or q.stride(1) != dk:
         launch_count += 1
         return simt()
     hdr = getattr(inp, "header_dev", None)
@@ -627,14 +748,16 @@ def paged_attention_ext(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.T
             max_kv = min(max_kv, chunk)
         if window > 0:
             max_kv = min(max_kv, window + keep_first)
-        splits = decode_splits(n_dec, n_kv, max_kv)
+        max_q = max(1, inp.max_q) if inp.n_spec > 0 else 1
+        splits = decode_splits(n_dec, n_kv * -(-Hq // n_kv * max_q // 16), max_kv)
         po = pl = None
         rows = max(T, n_dec)
         if splits > 1:
             po = torch.empty((rows, Hq, splits, dv), dtype=torch.float32, device=q.device)
             pl = torch.empty((rows, Hq, splits), dtype=torch.float32, device=q.device)
         rc = lib().xl_decode_attention_ext(*common, c_int(0), c_int(n_dec), *shape, c_float(scale), c_int(window), c_int(chunk),
-                                           c_int(keep_first), _ptr(slopes), _ptr(sinks), c_int(splits), _ptr(po), _ptr(pl), c_long(rows), dyn_dec, _stream())
+                                           c_int(keep_first), _ptr(slopes), _ptr(sinks), *ext, c_int(max_q), c_int(splits), _ptr(po), _ptr(pl),
+                                           c_long(rows), dyn_dec, _stream())
         if rc == -3:            # a block size outside the tensor-core kernels' limits
             launch_count += 1
             return simt()
@@ -643,8 +766,8 @@ def paged_attention_ext(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.T
     if has_prefill:
         tiles = (T + 127) // 128 + n_all if padded else (inp.n_prefill_tokens + 127) // 128 + (n_all - n_dec)
         rc = lib().xl_prefill_attention_ext(*common, c_int(0 if padded else n_dec), c_int(n_all), *shape, c_int(T), c_float(scale),
-                                            c_int(window), c_int(chunk), c_int(keep_first), _ptr(slopes), _ptr(sinks), c_int(tiles), dyn_dec, dyn_all,
-                                            _stream())
+                                            c_int(window), c_int(chunk), c_int(keep_first), _ptr(slopes), _ptr(sinks), *ext, c_int(tiles), dyn_dec,
+                                            dyn_all, _stream())
         if rc == -3:
             launch_count += 1
             return simt()

@@ -32,7 +32,7 @@ def moe_router(logits: torch.Tensor, top_k: int, scoring: str = "softmax", renor
     if bias is not None and bias.dtype != torch.float32:
         bias = bias.float()
     _check(lib().xl_moe_router(_ptr(logits), c_int(0 if logits.dtype == torch.float32 else 1), _ptr(bias), _ptr(w), _ptr(ids),
-                               _ptr(load_hist), c_int(T), c_int(E), c_int(top_k), c_int(int(scoring == "sigmoid")),
+                               _ptr(load_hist), c_int(T), c_int(E), c_int(top_k), c_int({"softmax": 0, "sigmoid": 1, "softmax_chosen": 2}[scoring]),
                                c_int(int(renorm)), c_int(n_group), c_int(topk_group), c_int(int(top2)), c_float(route_scale), _stream()),
            "xl_moe_router")
     cuda_ops.launch_count += 1
@@ -77,9 +77,9 @@ def moe_sort(ids: torch.Tensor, expert_offset: int, E_local: int, max_rows: Opti
 
 
 def grouped_gemm(a: torch.Tensor, w: torch.Tensor, r, swiglu: int = 0, out: Optional[torch.Tensor] = None,
-                 c_rows_per_expert: int = 0, c_col_stride: int = 0) -> torch.Tensor:
+                 c_rows_per_expert: int = 0, c_col_stride: int = 0, limit: float = 0.0) -> torch.Tensor:
     """a [R_cap, K] rows sorted by expert; w [E_local, N, K]; returns [R_cap, N] (or [R_cap, N/2] with a gated epilogue:
-    `swiglu` 1 = silu gate, 2 = tanh-gelu gate).
+    `swiglu` 1 = silu gate, 2 = tanh-gelu gate, 3 = clamped gate with `limit`).
     `r` provides the device-side tile table (`tile_expert`, `tile_row0`, `tile_row_end`, `num_m_tiles`, `max_tiles`).
     With `out` given, row `row - expert * c_rows_per_expert` / column offset `expert * c_col_stride` place each tile."""
     R_cap, K = a.shape
@@ -90,7 +90,7 @@ def grouped_gemm(a: torch.Tensor, w: torch.Tensor, r, swiglu: int = 0, out: Opti
     _check(lib().xl_grouped_gemm_bf16(_ptr(a), _ptr(w), _ptr(out), c_int(R_cap), c_int(N), c_int(K), c_int(a.stride(0)),
                                       c_int(out.stride(0)), c_int(E), _ptr(r.tile_expert), _ptr(r.tile_row0), _ptr(r.tile_row_end),
                                       _ptr(r.num_m_tiles), c_int(r.max_tiles), c_int(int(swiglu)), c_int(c_rows_per_expert),
-                                      c_int(c_col_stride), _stream()),
+                                      c_int(c_col_stride), c_float(limit), _stream()),
            "xl_grouped_gemm_bf16")
     cuda_ops.launch_count += 1
     return out
@@ -154,17 +154,18 @@ def grouped_gemm_simt(a: torch.Tensor, w: torch.Tensor, r: SortedRouting, gather
     return out
 
 
-def expert_rows(x: torch.Tensor, w13: torch.Tensor, w2: torch.Tensor, ids: torch.Tensor, act: str = "silu", interleaved: bool = False):
+def expert_rows(x: torch.Tensor, w13: torch.Tensor, w2: torch.Tensor, ids: torch.Tensor, act: str = "silu", interleaved: bool = False,
+                limit: float = 0.0):
     """Outputs of the chosen experts before their weighted sum: (rows [*, H], dst_of [T * k] with -1 for ids outside the
     experts of w13)."""
     k = ids.shape[1]
     r = moe_sort(ids, 0, w13.shape[0])
     if interleaved:
-        y = grouped_gemm(grouped_gemm(gather_rows(x, r, k), w13, r, swiglu=1 + cuda_ops.ACTS[act]), w2, r)
+        y = grouped_gemm(grouped_gemm(gather_rows(x, r, k), w13, r, swiglu=1 + cuda_ops.ACTS[act], limit=limit), w2, r)
     elif cuda_ops._tc_gemm_ok(x, w13) and cuda_ops._tc_gemm_ok(x, w2) and x.shape[1] % 8 == 0:
-        y = grouped_gemm(cuda_ops.gated_act(grouped_gemm(gather_rows(x, r, k), w13, r), act), w2, r)
+        y = grouped_gemm(cuda_ops.gated_act(grouped_gemm(gather_rows(x, r, k), w13, r), act, limit), w2, r)
     else:
-        y = grouped_gemm_simt(cuda_ops.gated_act(grouped_gemm_simt(x, w13, r, k), act), w2, r)
+        y = grouped_gemm_simt(cuda_ops.gated_act(grouped_gemm_simt(x, w13, r, k), act, limit), w2, r)
     return y, r.dst_of
 
 
@@ -179,5 +180,18 @@ def combine_post_norm_add_norm(y_exp, dst_of, ids, weights, h_in, shared, first_
                                                    c_int(ids.shape[1]), c_int(first_identity), _ptr(x), _ptr(w_post), _ptr(w_next), _ptr(h),
                                                    c_int(T), c_int(H), c_float(eps), c_int(int(h_in.dtype == torch.float32)), _stream()),
            "xl_moe_combine_post_norm_add_norm")
+    cuda_ops.launch_count += 1
+    return h
+
+
+def combine_add_norm(y_exp, dst_of, weights, vec, x, w_next, eps, w_offset=0.0, lead=None) -> torch.Tensor:
+    """x += vec * sum of the chosen experts' rows times their weights, + the embedding rows of `lead`, in place; returns
+    rms(x) * (w_next + w_offset).  One kernel; the sum is not stored."""
+    T, H = x.shape
+    assert x.is_contiguous() and x.dtype == torch.float32 and y_exp.shape[1] == H and vec.dtype == y_exp.dtype == w_next.dtype
+    h = torch.empty((T, H), dtype=y_exp.dtype, device=x.device)
+    _check(lib().xl_moe_combine_add_norm(_ptr(y_exp), _ptr(dst_of), _ptr(weights), c_int(weights.shape[1]), _ptr(x), _ptr(vec), _ptr(w_next),
+                                         c_float(w_offset), _ptr(h), c_int(T), c_int(H), c_float(eps), *cuda_ops._lead_args(lead, H, y_exp.dtype),
+                                         c_int(int(y_exp.dtype == torch.float32)), _stream()), "xl_moe_combine_add_norm")
     cuda_ops.launch_count += 1
     return h

@@ -116,6 +116,22 @@ def apply_rope_interleaved(x: torch.Tensor, cos: torch.Tensor, sin: torch.Tensor
     return out.to(x.dtype)
 
 
+def rotary_table(spec, max_pos: int, device="cpu") -> torch.Tensor:
+    """fp32 [max_pos, dims] of a `RotarySpec`: cosines, then sines, of every pair's angle (computed in double)."""
+    f, m = spec.frequencies()
+    ang = torch.outer(torch.arange(max_pos, dtype=torch.float64), torch.tensor(f, dtype=torch.float64))
+    return torch.cat([ang.cos() * m, ang.sin() * m], -1).float().contiguous().to(device)
+
+
+def apply_rotary(x: torch.Tensor, rot) -> torch.Tensor:
+    """x [T, H, d] fp32; rot = (table of `rotary_table`, positions [T], interleaved); columns past the table's stay."""
+    table, positions, interleaved = rot
+    n = table.shape[1]
+    cs = table.index_select(0, positions.long().clamp(0, table.shape[0] - 1))
+    y = (apply_rope_interleaved if interleaved else apply_rope_neox)(x[..., :n], cs[:, :n // 2], cs[:, n // 2:])
+    return torch.cat([y, x[..., n:]], -1)
+
+
 def rope_qknorm_kvwrite(qkv: torch.Tensor, positions: torch.Tensor, slots: torch.Tensor, cos_sin: torch.Tensor,
                         q_w: Optional[torch.Tensor], k_w: Optional[torch.Tensor], eps: float,
                         k_cache: torch.Tensor, v_cache: torch.Tensor, n_q: int, n_kv: int, head_dim: int) -> torch.Tensor:
@@ -144,17 +160,21 @@ def rope_qknorm_kvwrite(qkv: torch.Tensor, positions: torch.Tensor, slots: torch
 def paged_attention(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tensor, q_cu: torch.Tensor,
                     kv_lens: torch.Tensor, block_tables: torch.Tensor, n_seqs: int, scale: float,
                     sliding_window: int = -1, chunk: int = 0, slopes: Optional[torch.Tensor] = None,
-                    sinks: Optional[torch.Tensor] = None, keep_first: int = 0) -> torch.Tensor:
+                    sinks: Optional[torch.Tensor] = None, keep_first: int = 0, softcap: float = 0.0, mix=None) -> torch.Tensor:
     """Causal attention of ragged query rows over paged KV.
     q [T, Hq, D]; caches [n_blocks, block, Hkv, D]; sequence i owns q rows q_cu[i]:q_cu[i+1], which are the
     last rows of its kv_lens[i] tokens.  `chunk` > 0: a query sees keys of its own chunk of positions only; `slopes` [Hq]:
     slopes[h] * (query position - key position) is taken off the scores; `sinks` [Hq]: exp(sinks[h]) joins the denominator;
-    `keep_first`: so many first positions stay visible behind the window."""
+    `keep_first`: so many first positions stay visible behind the window; `softcap` > 0: scores become softcap * tanh(score /
+    softcap); `mix` (factor [1], mult, eps): query and key heads come in pairs of two maps over one value head, and a pair's
+    output is rms(first - factor * second) * mult."""
     T, Hq, D = q.shape
     block = k_cache.shape[1]
     Hkv = k_cache.shape[2]
     Dv = v_cache.shape[-1]
-    group = Hq // Hkv
+    group = Hq // v_cache.shape[2]                  # query heads per value head
+    heads = torch.arange(Hq, device=q.device)
+    key_of = heads // group if mix is None else heads // group * 2 + heads % 2
     out = torch.zeros(T, Hq, Dv, dtype=q.dtype, device=q.device)
     q_cu_h = q_cu.tolist()
     kv_h = kv_lens.tolist()
@@ -166,12 +186,14 @@ def paged_attention(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tenso
         nb = (L + block - 1) // block
         blocks = block_tables[i, :nb].long()
         k = k_cache.index_select(0, blocks).reshape(nb * block, Hkv, D)[:L].float()
-        v = v_cache.index_select(0, blocks).reshape(nb * block, Hkv, Dv)[:L].float()
+        v = v_cache.index_select(0, blocks).reshape(nb * block, -1, Dv)[:L].float()
         qi = q[qs:qe].float()                       # [n, Hq, D]
         n = qe - qs
-        k = k.repeat_interleave(group, dim=1)       # [L, Hq, D]
+        k = k[:, key_of]                            # [L, Hq, D]
         v = v.repeat_interleave(group, dim=1)
         s = torch.einsum("nhd,lhd->hnl", qi, k) * scale
+        if softcap > 0:
+            s = softcap * torch.tanh(s / softcap)
         qpos = torch.arange(L - n, L, device=q.device)[:, None]
         kpos = torch.arange(L, device=q.device)[None, :]
         mask = kpos <= qpos
@@ -187,8 +209,13 @@ def paged_attention(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tenso
             p = torch.softmax(s, dim=-1)[..., :-1]
         else:
             p = torch.softmax(s, dim=-1)
-        out[qs:qe] = torch.einsum("hnl,lhd->nhd", p, v).to(q.dtype)
-    return out.reshape(T, Hq * Dv)
+        o = torch.einsum("hnl,lhd->nhd", p, v)
+        if mix is not None:
+            factor, mult, eps = mix
+            o = o[:, 0::2] - factor.float() * o[:, 1::2]
+            o = o * torch.rsqrt(o.pow(2).mean(-1, keepdim=True) + eps) * mult
+        out[qs:qe, :o.shape[1]] = o.to(q.dtype)
+    return out.reshape(T, Hq * Dv) if mix is None else out[:, :Hq // 2].reshape(T, Hq // 2 * Dv)
 
 
 # ----------------------------------------------------------------------------- sampling
@@ -304,6 +331,9 @@ def moe_router(logits: torch.Tensor, top_k: int, scoring: str = "softmax", renor
     group-limited rule of the MLU `moe_active_topk` op, param.h:402-442).
     Returns (weights fp32 [T, k], expert ids int32 [T, k])."""
     lf = logits.float()
+    if scoring == "softmax_chosen":             # the bias belongs to the logits, the softmax to the chosen ones
+        top = (lf if bias is None else lf + bias.float()).topk(top_k, dim=-1)
+        return torch.softmax(top.values, -1) * route_scale, top.indices.int()
     scores = torch.softmax(lf, dim=-1) if scoring == "softmax" else torch.sigmoid(lf)
     sel = scores + bias.float()[None, :] if bias is not None else scores
     T, E = scores.shape
@@ -345,37 +375,48 @@ def linear_f32(x: torch.Tensor, w: torch.Tensor) -> torch.Tensor:
     return torch.nn.functional.linear(x.float(), w.float())
 
 
-def gated_act(x: torch.Tensor, act: str) -> torch.Tensor:
-    """[T, 2I] = [gate | up] -> act(gate) * up, act "silu" or "gelu_tanh"."""
+def gated_act(x: torch.Tensor, act: str, limit: float = 0.0) -> torch.Tensor:
+    """[T, 2I] = [gate | up] -> act(gate) * up, act "silu" or "gelu_tanh"; "clamped": g sigmoid(1.702 g) (u + 1) with the gate at
+    most `limit` and u within +- limit."""
     d = x.shape[-1] // 2
     g, u = x[..., :d].float(), x[..., d:].float()
+    if act == "clamped":
+        g = g.clamp(max=limit)
+        return (g * torch.sigmoid(1.702 * g) * (u.clamp(-limit, limit) + 1)).to(x.dtype)
     g = torch.nn.functional.silu(g) if act == "silu" else torch.nn.functional.gelu(g, approximate="tanh")
     return (g * u).to(x.dtype)
 
 
 def moe_mixture(h: torch.Tensor, w13: torch.Tensor, w2: torch.Tensor, weights: torch.Tensor, ids: torch.Tensor,
-                shared: Optional[torch.Tensor], first_identity: int, act: str) -> torch.Tensor:
+                shared: Optional[torch.Tensor], first_identity: int, act: str, limit: float = 0.0) -> torch.Tensor:
     """fp32 sum of the chosen experts' outputs times their weights, identity choices (ids >= first_identity) and `shared`."""
     out = torch.zeros(h.shape, dtype=torch.float32, device=h.device)
     for e in range(w13.shape[0]):
         hit = ids == e
         tok = hit.any(-1).nonzero().squeeze(-1)
         if tok.numel():
-            y = linear(gated_act(linear(h[tok], w13[e]), act), w2[e])
+            y = linear(gated_act(linear(h[tok], w13[e]), act, limit), w2[e])
             out.index_add_(0, tok, y.float() * (weights * hit).sum(-1)[tok][:, None])
     out += (weights * (ids >= first_identity)).sum(-1, keepdim=True) * h.float()
     return out if shared is None else out + shared.float()
 
 
 # norms before and after a sublayer around an fp32 residual stream
-def _rms_f32(x: torch.Tensor, w: torch.Tensor, eps: float) -> torch.Tensor:
+def _rms_f32(x: torch.Tensor, w: torch.Tensor, eps: float, w_offset: float = 0.0) -> torch.Tensor:
     xf = x.float()
-    return xf * torch.rsqrt(xf.pow(2).mean(-1, keepdim=True) + eps) * w.float()
+    return xf * torch.rsqrt(xf.pow(2).mean(-1, keepdim=True) + eps) * (w.float() + w_offset)
 
 
-def embed_rms_norm(ids: torch.Tensor, table: torch.Tensor, scale: float, w_next: torch.Tensor, eps: float):
+def embed_rows(ids: torch.Tensor, table: torch.Tensor, scale: float, positions=None, pos_table=None) -> torch.Tensor:
     x = embedding(ids, table).float() * scale
-    return x, _rms_f32(x, w_next, eps).to(table.dtype)
+    if pos_table is not None:
+        x = x + pos_table.index_select(0, positions.long().clamp(0, pos_table.shape[0] - 1)).float()
+    return x
+
+
+def embed_rms_norm(ids, table, scale: float, w_next, eps: float, positions=None, pos_table=None, w_offset: float = 0.0):
+    x = embed_rows(ids, table, scale, positions, pos_table)
+    return x, _rms_f32(x, w_next, eps, w_offset).to(table.dtype)
 
 
 def post_norm_add_norm(y: torch.Tensor, x: torch.Tensor, w_post: torch.Tensor, w_next: torch.Tensor, eps: float) -> torch.Tensor:
@@ -383,22 +424,56 @@ def post_norm_add_norm(y: torch.Tensor, x: torch.Tensor, w_post: torch.Tensor, w
     return _rms_f32(x, w_next, eps).to(w_next.dtype)
 
 
-def qknorm_kvwrite(qkv, slots, q_w, k_w, eps, k_cache, v_cache, n_q, n_kv):
+def qknorm_kvwrite(qkv, slots, q_w, k_w, eps, k_cache, v_cache, n_q, n_kv, rot=None):
     T = qkv.shape[0]
-    dk, dv = k_cache.shape[-1], v_cache.shape[-1]
-    q, k, v = qkv.split([n_q * dk, n_kv * dk, n_kv * dv], dim=-1)
-    q, k = q.reshape(T, n_q, dk), k.reshape(T, n_kv, dk)
+    dk, n_v, dv = k_cache.shape[-1], v_cache.shape[-2], v_cache.shape[-1]
+    q, k, v = qkv.split([n_q * dk, n_kv * dk, n_v * dv], dim=-1)
+    q, k = q.reshape(T, n_q, dk).float(), k.reshape(T, n_kv, dk).float()
     if q_w is not None:
-        q, k = _rms_f32(q, q_w, eps).to(qkv.dtype), _rms_f32(k, k_w, eps).to(qkv.dtype)
+        q, k = _rms_f32(q, q_w, eps), _rms_f32(k, k_w, eps)
+    if rot is not None:
+        q, k = apply_rotary(q, rot), apply_rotary(k, rot)
+    q, k = q.to(qkv.dtype), k.to(qkv.dtype)
     k_cache.view(-1, n_kv, dk).index_copy_(0, slots.long(), k.to(k_cache.dtype))
-    v_cache.view(-1, n_kv, dv).index_copy_(0, slots.long(), v.reshape(T, n_kv, dv).to(v_cache.dtype))
+    v_cache.view(-1, n_v, dv).index_copy_(0, slots.long(), v.reshape(T, n_v, dv).to(v_cache.dtype))
     return q.reshape(T, n_q * dk)
 
 
 # norms ahead of a sublayer only, around an fp32 residual stream
-def add_norm(y: torch.Tensor, x: torch.Tensor, mult: float, w_next: torch.Tensor, eps: float) -> torch.Tensor:
-    x += mult * y.float()
-    return _rms_f32(x, w_next, eps).to(w_next.dtype)
+def add_norm(y, x, mult: float, w_next, eps: float, vec=None, w_offset: float = 0.0, lead=None) -> torch.Tensor:
+    x += (mult if vec is None else vec.float()) * y.float()
+    if lead is not None:
+        x += embed_rows(*lead)
+    return _rms_f32(x, w_next, eps, w_offset).to(w_next.dtype)
+
+
+def lead_norm(lead, x, w_next, eps: float, w_offset: float = 0.0) -> torch.Tensor:
+    x += embed_rows(*lead)
+    return _rms_f32(x, w_next, eps, w_offset).to(w_next.dtype)
+
+
+# latent attention
+def latent_down(low, q_rank, kv_rank, q_w, kv_w, eps, rot, slots, cache):
+    row = cache.shape[-1]
+    cq = _rms_f32(low[:, :q_rank], q_w, eps).to(low.dtype)
+    c = _rms_f32(low[:, q_rank:q_rank + kv_rank], kv_w, eps)
+    k = apply_rotary(low[:, None, q_rank + kv_rank:].float(), rot)[:, 0]
+    cache.view(-1, row).index_copy_(0, slots.long(), torch.cat([c, k], -1).to(cache.dtype))
+    return cq
+
+
+def rotate_into(x, rot, out) -> None:
+    out.copy_(apply_rotary(x.float(), rot))
+
+
+def heads_linear(x, w, out) -> torch.Tensor:
+    out.copy_(torch.einsum("htk,hnk->htn", x.float(), w.float()))
+    return out
+
+
+def linear_softcap(x, w, cap: float) -> torch.Tensor:
+    y = linear(x, w).float()
+    return (cap * torch.tanh(y / cap)).to(x.dtype)
 
 
 def replace_norm(y: torch.Tensor, vec: torch.Tensor, x: torch.Tensor, w_next: torch.Tensor, eps: float) -> torch.Tensor:
