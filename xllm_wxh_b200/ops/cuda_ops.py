@@ -898,7 +898,9 @@ def mla_attention(q_lat_hm, q_pe_hm, cache, inp, scale, kv_lora):
     global launch_count
     Hh, T, C = q_lat_hm.shape
     rope = q_pe_hm.shape[-1]
-    out = torch.empty_like(q_lat_hm)
+    # padded rows belong to no sequence and are written by no kernel: keep them finite, since the next layer writes their latents
+    # into the padding block, which tiles past a sequence's end may read
+    out = (torch.zeros_like if inp.padded else torch.empty_like)(q_lat_hm)
     L = inp.layout
     n_all = inp.B if inp.padded else inp.n_seqs
     common = (_ptr(inp.q_cu), _ptr(inp.kv_lens), _ptr(inp.block_tables), c_int(0), c_int(n_all), c_int(L.MB_cap),
