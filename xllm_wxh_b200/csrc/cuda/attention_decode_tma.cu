@@ -85,7 +85,7 @@ struct DecBarriers {
   uint64_t empty[kStages];
 };
 
-template <int DK, int DV, bool EXT>
+template <int DK, int DV, bool EXT, bool CAP = false>
 __global__ void __launch_bounds__(160) decode_attn_tma_kernel(const __grid_constant__ CUtensorMap tmK,
                                                               const __grid_constant__ CUtensorMap tmV, DecParams p) {
   constexpr int KH = DK / 64, VH = DV / 64;       // 128-byte column slabs per row
@@ -105,8 +105,11 @@ __global__ void __launch_bounds__(160) decode_attn_tma_kernel(const __grid_const
 
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const int seq = p.seq_begin + blockIdx.x;
-  const int kvh = EXT ? blockIdx.y / p.row_blocks : blockIdx.y;
-  const int row0 = EXT ? blockIdx.y % p.row_blocks * 16 : 0;      // first query row (token x head) of this CTA
+  int kvh = blockIdx.y, row0 = 0;                 // row0: first query row (token x head) of this CTA
+  if (EXT && p.row_blocks > 1) {
+    kvh = blockIdx.y / p.row_blocks;
+    row0 = blockIdx.y % p.row_blocks * 16;
+  }
   const int split = blockIdx.z;
   const int group = p.n_q / p.n_kv;
   if (seq >= (p.dyn_end ? *p.dyn_end : p.seq_end)) return;
@@ -251,10 +254,9 @@ __global__ void __launch_bounds__(160) decode_attn_tma_kernel(const __grid_const
           mma_bf16_16816(sc[0], qf[kKeepQ ? ks : 0], b0, b1);
           mma_bf16_16816(sc[1], qf[kKeepQ ? ks : 0], b2, b3);
         }
-        const bool capped = EXT && p.cap_out > 0.f;
-        if (capped) {
-          softcap_row(sc[0], p.cap_in, p.cap_out);
-          softcap_row(sc[1], p.cap_in, p.cap_out);
+        if (CAP) {
+          softcap_row<false>(sc[0], p.cap_in, p.cap_out);
+          softcap_row<false>(sc[1], p.cap_in, p.cap_out);
         }
         float mx[2] = {-INFINITY, -INFINITY};
 #pragma unroll
@@ -265,7 +267,7 @@ __global__ void __launch_bounds__(160) decode_attn_tma_kernel(const __grid_const
             const int lim = (e < 2) ? lim_a : lim_b;
             bool ok = tok <= lim && tok < kv_len;
             if (p.window > 0) ok = ok && (tok > lim - p.window || (EXT && tok < p.keep_first));
-            float x = capped ? sc[i][e] : sc[i][e] * p.scale_log2;
+            float x = CAP ? sc[i][e] : sc[i][e] * p.scale_log2;
             if (EXT) {
               ok = ok && tok >= ((e < 2) ? lo_a : lo_b);
               x += ((e < 2) ? slope_a : slope_b) * float(tok - lim);
@@ -560,18 +562,23 @@ XL_API int xl_decode_split_merge(const void* part_o, const void* part_lse, void*
 
 // ============================================================================ score extensions
 namespace xl_dec {
-template <int DK, int DV>
-static int launch_ext(const CUtensorMap* tk, const CUtensorMap* tv, const DecParams& p, dim3 grid, cudaStream_t st) {
+template <int DK, int DV, bool CAP>
+static int launch_ext_as(const CUtensorMap* tk, const CUtensorMap* tv, const DecParams& p, dim3 grid, cudaStream_t st) {
   const size_t ring = size_t(kStages) * (DK / 64 + DV / 64) * kTile * 128;
   const size_t merge = 4 * 16 * DV * 4 + 128 * 4;
   const size_t smem = (ring > merge ? ring : merge) + 16 * DK * 2 + sizeof(DecBarriers) + 1024;
   static bool set = false;
   if (!set) {
-    cudaFuncSetAttribute(decode_attn_tma_kernel<DK, DV, true>, cudaFuncAttributeMaxDynamicSharedMemorySize, int(smem));
+    cudaFuncSetAttribute(decode_attn_tma_kernel<DK, DV, true, CAP>, cudaFuncAttributeMaxDynamicSharedMemorySize, int(smem));
     set = true;
   }
-  decode_attn_tma_kernel<DK, DV, true><<<grid, 160, smem, st>>>(*tk, *tv, p);
+  decode_attn_tma_kernel<DK, DV, true, CAP><<<grid, 160, smem, st>>>(*tk, *tv, p);
   return cudaGetLastError() == cudaSuccess ? 0 : -1;
+}
+
+template <int DK, int DV>
+static int launch_ext(const CUtensorMap* tk, const CUtensorMap* tv, const DecParams& p, dim3 grid, cudaStream_t st) {
+  return p.cap_out > 0.f ? launch_ext_as<DK, DV, true>(tk, tv, p, grid, st) : launch_ext_as<DK, DV, false>(tk, tv, p, grid, st);
 }
 
 // merge of split-KV partials for any value head dimension, with the sink's share of the denominator: one warp per

@@ -20,7 +20,7 @@
 // its slabs is padded with zeros by the TMA loads), EXT = score extensions: per-head linear distance bias, per-head sink
 // (a score that joins the denominator and has no value), chunk mask (a query sees keys of its own position chunk only),
 // first keys that stay visible behind a window (their tiles come ahead of the window's, the gap between is not read), scores
-// bounded by a tanh.  MAPS = 2: differential attention.  The CTA's two heads are the two maps of one output head: each has its own
+// bounded by a tanh; SCORE = which of them change the scores (instances of their own keep the softmax loop short).  MAPS = 2: differential attention.  The CTA's two heads are the two maps of one output head: each has its own
 // keys (slabs of their own in a stage), both read the same values, and the epilogue hands the second map's output to the first
 // map's warps through the idle ring, which store rms(first - factor * second) * mult.
 // QK^T of tile j+1 is issued before P V of tile j, so the tensor pipe works while the softmax warps are busy.
@@ -141,7 +141,9 @@ __device__ __forceinline__ void store_difference(const Params& p, const float* e
   }
 }
 
-template <int NH, int QS, int VS, bool EXT, int MAPS>
+enum { SCORE_RAW = 0, SCORE_BIAS = 1, SCORE_CAP = 2 };   // products as they are; less a distance bias; bounded (if cap_out > 0)
+
+template <int NH, int QS, int VS, bool EXT, int SCORE, int MAPS>
 __global__ void __launch_bounds__(Cfg<NH, QS, VS, MAPS>::kThreads, 1)
 prefill_attn_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__ CUtensorMap tmK,
                        const __grid_constant__ CUtensorMap tmV, const Params p) {
@@ -353,9 +355,11 @@ prefill_attn_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_con
     const int keep = EXT ? p.keep_first : 0;
     const int lo_win = p.window > 0 ? pos0 + BQ - p.window : 0;                          // first key in every row's window
     const int lo_last = EXT && p.chunk > 0 ? (pos0 + BQ - 1) / p.chunk * p.chunk : 0;   // first key that every row's chunk may hold
-    const float slope2 = EXT && p.slopes ? p.slopes[head0 + h] * 1.4426950408889634f : 0.f;
-    // with the extensions v[] holds finished scores in the log2 domain, otherwise raw products that `sc` scales
-    const float sc = EXT ? 1.f : p.scale_log2;
+    const float slope2 = SCORE == SCORE_BIAS ? p.slopes[head0 + h] * 1.4426950408889634f : 0.f;
+    // with a distance bias v[] holds finished scores in the log2 domain, otherwise (bounded) raw products that `sc` scales
+    const bool capped = SCORE == SCORE_CAP && p.cap_out > 0.f;
+    const float sc = SCORE == SCORE_BIAS ? 1.f : capped ? p.cap_in * p.cap_out : p.scale_log2;
+    const float cap_top = capped ? 1.f / p.cap_in : 0.f;
     float m_ref = -INFINITY, l_run = 0.f;                    // m_ref: reference maximum of the raw scores
     bool ok = true;
     for (int j = 0; j < n_tiles && ok; ++j) {
@@ -381,18 +385,11 @@ prefill_attn_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_con
         v[c] = __uint_as_float(s0[c]);
         v[32 + c] = __uint_as_float(s1[c]);
       }
-      if (EXT) {
+      if (capped) softcap_row<true>(v, p.cap_in, cap_top);
+      if (SCORE == SCORE_BIAS) {
         const float b0 = slope2 * float(kv0 - pos);
-        if (p.cap_out > 0.f) {
-          softcap_row(v, p.cap_in, p.cap_out);
-          if (slope2 != 0.f) {
 #pragma unroll
-            for (int c = 0; c < 64; ++c) v[c] += fmaf(slope2, float(c), b0);
-          }
-        } else {
-#pragma unroll
-          for (int c = 0; c < 64; ++c) v[c] = fmaf(v[c], p.scale_log2, fmaf(slope2, float(c), b0));
-        }
+        for (int c = 0; c < 64; ++c) v[c] = fmaf(v[c], p.scale_log2, fmaf(slope2, float(c), b0));
       }
       if (need_mask) {
 #pragma unroll
@@ -481,7 +478,7 @@ prefill_attn_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_con
       float inv = 0.f, ss = 0.f;
       if (ok) {
         tc_fence_after();
-        if (p.sinks && m_ref != -INFINITY) l_run += fast_exp2(p.sinks[head0 + h] * 1.4426950408889634f - m_ref);
+        if (p.sinks && m_ref != -INFINITY) l_run += fast_exp2(p.sinks[head0 + h] * 1.4426950408889634f - m_ref * sc);
         inv = l_run > 0.f ? 1.f / l_run : 0.f;
       }
       if (ok && h == 1) {
@@ -513,7 +510,7 @@ prefill_attn_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_con
       }
     } else if (ok) {
       tc_fence_after();
-      if (EXT && p.sinks && m_ref != -INFINITY) l_run += fast_exp2(p.sinks[head0 + h] * 1.4426950408889634f - m_ref);
+      if (EXT && p.sinks && m_ref != -INFINITY) l_run += fast_exp2(p.sinks[head0 + h] * 1.4426950408889634f - m_ref * sc);
       const float inv = l_run > 0.f ? 1.f / l_run : 0.f;
       const int dv = EXT ? p.dv : DV;
       __nv_bfloat16* dst = p.out + size_t(q_start + q0 + r) * (size_t(p.n_q) * dv) + (head0 + h) * dv;
@@ -657,14 +654,14 @@ static uint8_t* split_workspace(cudaStream_t stream) {
   return ws[dev];
 }
 
-template <int NH, int QS, int VS, bool EXT, int MAPS = 1>
+template <int NH, int QS, int VS, bool EXT, int SCORE = SCORE_RAW, int MAPS = 1>
 static int launch_prefill(const CUtensorMap* tq, const CUtensorMap* tk, const CUtensorMap* tv, const Params& p_in, int q_tiles_cap,
                           int total_q_rows, cudaStream_t stream) {
   using C = Cfg<NH, QS, VS, MAPS>;
   const size_t smem = size_t(NH) * (C::Q_BYTES + P_BYTES) + C::kStages * C::STAGE_BYTES + sizeof(Barriers);
   static bool set = false;
   if (!set) {
-    cudaFuncSetAttribute(prefill_attn_tc_kernel<NH, QS, VS, EXT, MAPS>, cudaFuncAttributeMaxDynamicSharedMemorySize, int(smem));
+    cudaFuncSetAttribute(prefill_attn_tc_kernel<NH, QS, VS, EXT, SCORE, MAPS>, cudaFuncAttributeMaxDynamicSharedMemorySize, int(smem));
     set = true;
   }
   Params p = p_in;
@@ -695,7 +692,7 @@ static int launch_prefill(const CUtensorMap* tq, const CUtensorMap* tk, const CU
     }
   }
   dim3 grid(q_tiles_cap, p.n_q / NH, p.splits);
-  prefill_attn_tc_kernel<NH, QS, VS, EXT, MAPS><<<grid, C::kThreads, smem, stream>>>(*tq, *tk, *tv, p);
+  prefill_attn_tc_kernel<NH, QS, VS, EXT, SCORE, MAPS><<<grid, C::kThreads, smem, stream>>>(*tq, *tk, *tv, p);
   return cudaGetLastError() == cudaSuccess ? 0 : -1;
 }
 
@@ -754,7 +751,8 @@ XL_API int xl_prefill_attention_tc(const void* q, const void* k_cache, const voi
 // `slopes` / `sinks` [n_q] fp32, null when absent; `softcap` > 0: scale * q . k becomes softcap * tanh(scale * q . k / softcap).
 // `v_pitch`: elements from one cache slot's values to the next one's (0: n_kv * dv), so that values may be a part of the keys.
 // maps = 2: n_q counts the maps' heads (pairs of neighbours), k_cache has 2 n_kv heads, out [T, n_q / 2 * dv] =
-// rms(first - mix[0] * second, mix_eps) * mix_mult.  Returns -3 when the shape is not covered.
+// rms(first - mix[0] * second, mix_eps) * mix_mult.  Returns -3 when the shape, or a distance bias beside bounded scores or two
+// maps, is not covered.
 XL_API int xl_prefill_attention_ext(const void* q, const void* k_cache, const void* v_cache, void* out, const void* q_cu,
                                     const void* kv_lens, const void* block_tables, int seq_begin, int seq_end, int max_blocks,
                                     int block_size, int num_blocks_total, int n_q, int n_kv, int dk, int dv, int q_stride,
@@ -765,7 +763,7 @@ XL_API int xl_prefill_attention_ext(const void* q, const void* k_cache, const vo
   if (maps < 1 || maps > 2 || (maps == 2 && (!mix || (n_q / n_kv) % 2))) return -2;
   const int d_max = maps == 2 ? 128 : 256;
   if (dk < 8 || dk > d_max || dk % 8 || dv < 8 || dv > d_max || dv % 8) return -3;
-  if (v_pitch % 8) return -3;
+  if (v_pitch % 8 || (slopes && (softcap > 0.f || maps == 2))) return -3;
   if (chunk > 0 && keep_first > 0) return -2;
   if (block_size % 16 != 0 || (block_size > 64 && block_size % 64 != 0) || (block_size < 64 && 64 % block_size != 0)) return -3;
   if (n_q % n_kv) return -3;
@@ -808,16 +806,23 @@ XL_API int xl_prefill_attention_ext(const void* q, const void* k_cache, const vo
   p.window = window;
   p.status = xl_host::status_word();
   cudaStream_t st = static_cast<cudaStream_t>(stream);
-  const bool pair = (n_q / n_kv) % 2 == 0, k2 = dk > 64, v2 = dv > 64;
-#define XL_PF_EXT(NH, QS, VS) launch_prefill<NH, QS, VS, true>(tq, tk, tv, p, q_tiles_cap, total_q_rows, st)
-#define XL_PF_MAPS(QS, VS) launch_prefill<2, QS, VS, true, 2>(tq, tk, tv, p, q_tiles_cap, total_q_rows, st)
-  if (maps == 2) return k2 ? (v2 ? XL_PF_MAPS(2, 2) : XL_PF_MAPS(2, 1)) : (v2 ? XL_PF_MAPS(1, 2) : XL_PF_MAPS(1, 1));
-  if (dk > 128 || dv > 128) {
-    if (dv > 128) return XL_PF_EXT(1, 4, 4);
-    return dk > 192 ? XL_PF_EXT(1, 4, 2) : XL_PF_EXT(1, 3, 2);
+  const bool pair = (n_q / n_kv) % 2 == 0, k2 = dk > 64, v2 = dv > 64, wide = dk > 128 || dv > 128;
+#define XL_PF_EXT(...) launch_prefill<__VA_ARGS__>(tq, tk, tv, p, q_tiles_cap, total_q_rows, st)
+  if (maps == 2) {
+    if (k2) return v2 ? XL_PF_EXT(2, 2, 2, true, SCORE_CAP, 2) : XL_PF_EXT(2, 2, 1, true, SCORE_CAP, 2);
+    return v2 ? XL_PF_EXT(2, 1, 2, true, SCORE_CAP, 2) : XL_PF_EXT(2, 1, 1, true, SCORE_CAP, 2);
   }
-  if (pair) return k2 ? (v2 ? XL_PF_EXT(2, 2, 2) : XL_PF_EXT(2, 2, 1)) : (v2 ? XL_PF_EXT(2, 1, 2) : XL_PF_EXT(2, 1, 1));
-  return k2 ? (v2 ? XL_PF_EXT(1, 2, 2) : XL_PF_EXT(1, 2, 1)) : (v2 ? XL_PF_EXT(1, 1, 2) : XL_PF_EXT(1, 1, 1));
+  if (softcap > 0.f)           // columns past a head's own are zeros
+    return wide ? XL_PF_EXT(1, 4, 4, true, SCORE_CAP) : pair ? XL_PF_EXT(2, 2, 2, true, SCORE_CAP) : XL_PF_EXT(1, 2, 2, true, SCORE_CAP);
+  if (slopes) {
+    if (wide) return XL_PF_EXT(1, 4, 4, true, SCORE_BIAS);
+    if (pair) return k2 ? (v2 ? XL_PF_EXT(2, 2, 2, true, SCORE_BIAS) : XL_PF_EXT(2, 2, 1, true, SCORE_BIAS))
+                        : (v2 ? XL_PF_EXT(2, 1, 2, true, SCORE_BIAS) : XL_PF_EXT(2, 1, 1, true, SCORE_BIAS));
+    return k2 ? (v2 ? XL_PF_EXT(1, 2, 2, true, SCORE_BIAS) : XL_PF_EXT(1, 2, 1, true, SCORE_BIAS))
+              : (v2 ? XL_PF_EXT(1, 1, 2, true, SCORE_BIAS) : XL_PF_EXT(1, 1, 1, true, SCORE_BIAS));
+  }
+  if (wide) return dv > 128 ? XL_PF_EXT(1, 4, 4, true) : dk > 192 ? XL_PF_EXT(1, 4, 2, true) : XL_PF_EXT(1, 3, 2, true);
+  if (pair) return k2 ? (v2 ? XL_PF_EXT(2, 2, 2, true) : XL_PF_EXT(2, 2, 1, true)) : (v2 ? XL_PF_EXT(2, 1, 2, true) : XL_PF_EXT(2, 1, 1, true));
+  return k2 ? (v2 ? XL_PF_EXT(1, 2, 2, true) : XL_PF_EXT(1, 2, 1, true)) : (v2 ? XL_PF_EXT(1, 1, 2, true) : XL_PF_EXT(1, 1, 1, true));
 #undef XL_PF_EXT
-#undef XL_PF_MAPS
 }

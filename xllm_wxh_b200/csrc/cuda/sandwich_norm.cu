@@ -328,74 +328,114 @@ __device__ __forceinline__ float rot_one(const Rotation& r, const float* cs, int
   return first ? v * cs[j] - other * cs[half + j] : v * cs[j] + other * cs[half + j];
 }
 
+// Eight elements as they lie in memory.
+template <typename T> struct Raw8 { uint4 v[sizeof(T) / 2]; };
 template <typename T>
-__global__ void __launch_bounds__(256) qknorm_kvwrite_vec_kernel(T* __restrict__ qkv, const int* __restrict__ slots,
-                                                                 const T* __restrict__ q_w, const T* __restrict__ k_w,
-                                                                 T* __restrict__ k_cache, T* __restrict__ v_cache, int T_rows,
-                                                                 int n_q, int n_k, int n_v, int dk, int dv, int lph, float eps,
-                                                                 long cache_slots, const Rotation rot) {
-  __shared__ __align__(16) float s_rot[256 * 8];
-  const int heads = n_q + n_k + n_v;
-  const long gt = blockIdx.x * long(blockDim.x) + threadIdx.x;
-  const long item = gt / lph;
-  const int sub = int(gt % lph);
-  const bool active = item < long(T_rows) * heads;
-  const int t = active ? int(item / heads) : 0, h = active ? int(item % heads) : 0;
-  const size_t row = size_t(t) * (size_t(n_q + n_k) * dk + size_t(n_v) * dv);
-  const bool is_v = h >= n_q + n_k;
-  const int dim = is_v ? dv : dk;
-  T* src = qkv + row + (is_v ? size_t(n_q + n_k) * dk + size_t(h - n_q - n_k) * dv : size_t(h) * dk);
-  const bool mine = active && sub * 8 < dim;
-  float f[8] = {0, 0, 0, 0, 0, 0, 0, 0};
-  if (mine) load8(src + sub * 8, f);
-  float ss = 0.f;
+__device__ __forceinline__ Raw8<T> load_raw8(const T* p) {
+  Raw8<T> r;
 #pragma unroll
-  for (int e = 0; e < 8; ++e) ss += f[e] * f[e];
-  for (int o = lph / 2; o > 0; o >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, o);
-  if (mine && !is_v) {
+  for (int i = 0; i < int(sizeof(T) / 2); ++i) r.v[i] = reinterpret_cast<const uint4*>(p)[i];
+  return r;
+}
+
+// One token per CTA.  A q or k head takes 2^lph lanes of 8 elements each; a thread keeps its place in the head over all the heads it
+// serves, and with it the angles, and fetches several heads ahead.  Values are copied as one run of nv elements.
+template <typename T>
+__global__ void __launch_bounds__(256, sizeof(T) == 2 ? 4 : 2) qknorm_kvwrite_vec_kernel(T* __restrict__ qkv, const int* __restrict__ slots,
+                                                                 const T* __restrict__ q_w, const T* __restrict__ k_w,
+                                                                 T* __restrict__ k_cache, T* __restrict__ v_cache, int n_q, int n_k, int nv,
+                                                                 int dk, int lph, float eps, long cache_slots, const Rotation rot) {
+  __shared__ __align__(16) float s_rot[256 * 8];
+  const int t = blockIdx.x, heads = n_q + n_k, step = blockDim.x >> lph;
+  const int sub = threadIdx.x & ((1 << lph) - 1), c0 = sub * 8;
+  T* row = qkv + size_t(t) * (size_t(heads) * dk + nv);
+  const int slot = slots[t];
+  const bool in = slot >= 0 && slot < cache_slots, mine = c0 < dk;
+  // 0: no rotation here, 1: both elements of every pair in this lane, 2: the others' lane is half / 8 away, 3: through shared memory
+  const int half = rot.dims / 2;
+  const int turn = !rot.table ? 0 : rot.interleaved ? 1 : half % 8 == 0 ? 2 : 3;
+  const bool first = c0 < half;
+  constexpr int kAhead = 4;
+  const int h_own = threadIdx.x >> lph;
+  Raw8<T> raw[kAhead];
+  auto fetch = [&](int h0) {
+#pragma unroll
+    for (int u = 0; u < kAhead; ++u) {
+      const int h = h0 + u * step + h_own;
+      if (mine && h < heads) raw[u] = load_raw8(row + size_t(h) * dk + c0);
+    }
+  };
+  fetch(0);
+  float cs[8], sn[8];
+#pragma unroll
+  for (int e = 0; e < 8; ++e) cs[e] = 1.f, sn[e] = 0.f;
+  if (turn && mine && c0 < rot.dims) {
+    const float* tab = rot.table + size_t(clamp_id(rot.positions[t], rot.rows)) * rot.dims;
+    if (turn == 2) {
+      load8(tab + (first ? c0 : c0 - half), cs);
+      load8(tab + half + (first ? c0 : c0 - half), sn);
+    } else {
+#pragma unroll
+      for (int e = 0; e < 8; ++e) {
+        const int i = c0 + e, j = rot.interleaved ? i >> 1 : (i < half ? i : i - half);
+        if (i < rot.dims) cs[e] = tab[j], sn[e] = tab[half + j];
+      }
+    }
+#pragma unroll
+    for (int e = 0; e < 8; ++e)                   // the element of a pair that comes first takes the other's sine off
+      if (rot.interleaved ? !(e & 1) : c0 + e < half) sn[e] = -sn[e];
+  }
+  for (int c = threadIdx.x * 8; c < nv; c += blockDim.x * 8) {
+    float f[8];
+    load8(row + size_t(heads) * dk + c, f);
+    if (in) store8(v_cache + size_t(slot) * nv + c, f);
+  }
+  for (int h0 = 0; h0 < heads; h0 += kAhead * step) {
+    if (h0 > 0) fetch(h0);
+#pragma unroll
+    for (int u = 0; u < kAhead; ++u) {
+    if (h0 + u * step >= heads) break;            // whole warps stay in step
+    const int h = h0 + u * step + h_own;
+    const bool active = mine && h < heads;
+    float f[8] = {0, 0, 0, 0, 0, 0, 0, 0};
+    if (active) load8(reinterpret_cast<const T*>(&raw[u]), f);
+    float ss = 0.f;
+#pragma unroll
+    for (int e = 0; e < 8; ++e) ss += f[e] * f[e];
+    for (int o = 1 << lph >> 1; o > 0; o >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, o);
     const T* w = h >= n_q ? k_w : q_w;
-    if (w) {
+    if (w && active) {
       const float r = rsqrtf(ss / float(dk) + eps);
       float wf[8];
-      load8(w + sub * 8, wf);
+      load8(w + c0, wf);
 #pragma unroll
       for (int e = 0; e < 8; ++e) f[e] = f[e] * r * wf[e];
     }
-  }
-  if (rot.table) {                                // the pair's other element may lie with another lane of the head
-    float* mem = s_rot + (threadIdx.x - sub) * 8;
-    store8(mem + sub * 8, f);
-    __syncwarp();
-    if (mine && !is_v && sub * 8 < rot.dims) {
-      const float* cs = rot.table + size_t(clamp_id(rot.positions[t], rot.rows)) * rot.dims;
-      const int half = rot.dims / 2;
-      if (!rot.interleaved && half % 8 == 0) {
-        float o[8], c[8], s[8];
-        const bool first = sub * 8 < half;
-        const int j = first ? sub * 8 : sub * 8 - half;
-        load8(mem + (first ? j + half : j), o);
-        load8(cs + j, c);
-        load8(cs + half + j, s);
+    if (turn) {
+      float o[8];
+      if (turn == 1) {
 #pragma unroll
-        for (int e = 0; e < 8; ++e) f[e] = first ? f[e] * c[e] - o[e] * s[e] : f[e] * c[e] + o[e] * s[e];
+        for (int e = 0; e < 8; ++e) o[e] = f[e ^ 1];
+      } else if (turn == 2) {
+        const int lane = threadIdx.x & 31, other = c0 >= rot.dims ? lane : first ? lane + half / 8 : lane - half / 8;
+#pragma unroll
+        for (int e = 0; e < 8; ++e) o[e] = __shfl_sync(0xffffffffu, f[e], other);
       } else {
+        float* mem = s_rot + (threadIdx.x - sub) * 8;
+        __syncwarp();
+        store8(mem + c0, f);
+        __syncwarp();
 #pragma unroll
-        for (int e = 0; e < 8; ++e) {
-          const int i = sub * 8 + e;
-          if (i < rot.dims) f[e] = rot_one(rot, cs, i, f[e], mem[rot_pair(rot, i)]);
-        }
+        for (int e = 0; e < 8; ++e) o[e] = c0 + e < rot.dims ? mem[rot_pair(rot, c0 + e)] : 0.f;
       }
+#pragma unroll
+      for (int e = 0; e < 8; ++e) f[e] = fmaf(o[e], sn[e], f[e] * cs[e]);
+    }
+    if (!active) continue;
+    if (h < n_q) store8(row + size_t(h) * dk + c0, f);
+    else if (in) store8(k_cache + (size_t(slot) * n_k + (h - n_q)) * dk + c0, f);
     }
   }
-  if (!mine) return;
-  if (h < n_q) {
-    store8(src + sub * 8, f);
-    return;
-  }
-  const int slot = slots[t];
-  if (slot < 0 || slot >= cache_slots) return;
-  T* dst = is_v ? v_cache + (size_t(slot) * n_v + (h - n_q - n_k)) * dv : k_cache + (size_t(slot) * n_k + (h - n_q)) * dk;
-  store8(dst + sub * 8, f);
 }
 
 // Any head dimension: one warp per (token, head).
@@ -445,13 +485,13 @@ template <typename T>
 static int launch_qknorm(void* qkv, const void* slots, const void* q_w, const void* k_w, void* k_cache, void* v_cache, int rows, int n_q,
                          int n_k, int n_v, int dk, int dv, float eps, long cache_slots, const Rotation& rot, cudaStream_t st) {
   const long items = long(rows) * (n_q + n_k + n_v);
-  const int dmax = dk > dv ? dk : dv;
-  if (dk % 8 == 0 && dv % 8 == 0 && dmax <= 256 && al16(qkv, k_cache, v_cache, q_w) && al16(k_w) && (!rot.table || rot.dims % 8 == 0)) {
-    int lph = 1;
-    while (lph * 8 < dmax) lph *= 2;
-    qknorm_kvwrite_vec_kernel<T><<<int((items * lph + 255) / 256), 256, 0, st>>>(
+  if (dk % 8 == 0 && dv % 8 == 0 && dk <= 256 && al16(qkv, k_cache, v_cache, q_w) && al16(k_w) && (!rot.table || rot.dims % 8 == 0)) {
+    int lph = 0;
+    while (8 << lph < dk) ++lph;
+    const int lanes = (n_q + n_k) << lph;
+    qknorm_kvwrite_vec_kernel<T><<<rows, lanes > 128 ? 256 : 128, 0, st>>>(
         static_cast<T*>(qkv), static_cast<const int*>(slots), static_cast<const T*>(q_w), static_cast<const T*>(k_w),
-        static_cast<T*>(k_cache), static_cast<T*>(v_cache), rows, n_q, n_k, n_v, dk, dv, lph, eps, cache_slots, rot);
+        static_cast<T*>(k_cache), static_cast<T*>(v_cache), n_q, n_k, n_v * dv, dk, lph, eps, cache_slots, rot);
   } else {
     qknorm_kvwrite_any_kernel<T><<<int((items + 7) / 8), 256, 0, st>>>(
         static_cast<T*>(qkv), static_cast<const int*>(slots), static_cast<const T*>(q_w), static_cast<const T*>(k_w),

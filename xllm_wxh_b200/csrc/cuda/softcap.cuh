@@ -34,8 +34,8 @@ __device__ __forceinline__ uint64_t mul_f32x2(uint64_t a, uint64_t b) {
   return d;
 }
 
-// v[i] = top * tanh(v[i] * in), two values per instruction while all of them are small.
-template <int N>
+// v[i] = top * tanh(v[i] * in), two values per instruction while all of them are small.  UNIT: top is 1 / in.
+template <bool UNIT, int N>
 __device__ __forceinline__ void softcap_row(float (&v)[N], float in, float top) {
   float big[4] = {0.f, 0.f, 0.f, 0.f};
 #pragma unroll
@@ -49,7 +49,7 @@ __device__ __forceinline__ void softcap_row(float (&v)[N], float in, float top) 
       const uint64_t x = pack_f32x2(v[c], v[c + 1]);
       const uint64_t y = mul_f32x2(x, in2), z = mul_f32x2(y, y);
       const uint64_t p = fma_f32x2(fma_f32x2(fma_f32x2(fma_f32x2(c4, z, c3), z, c2), z, c1), z, c0);
-      unpack_f32x2(mul_f32x2(mul_f32x2(x, top2), p), v[c], v[c + 1]);
+      unpack_f32x2(mul_f32x2(UNIT ? x : mul_f32x2(x, top2), p), v[c], v[c + 1]);
     }
   } else {
 #pragma unroll

@@ -1,4 +1,4 @@
-"""A model design beside the framework's closest other one at equal layer sizes (`bench.py --compare-design movolorn|falalix`):
+"""A model design beside the framework's closest other one at equal layer sizes (`bench.py --compare-design movolorn|falalix|babadra`):
 tokens per second of the decoder layers in prefill and decode, and the design's own kernels beside the like kernels with their
 distance from the roofline.  Random weights; kernel and layer times come from CUDA-graph replay between CUDA events, with
 weights, caches and activations rotated through (or larger than) more memory than L2 holds."""
@@ -13,8 +13,8 @@ import numpy as np
 import torch
 
 from ..framework.step_input import StepInput, make_layout
-from ..models.args import ModelArgs, preset
-from ..models.layer_spec import AttentionSpec, ParallelSpec
+from ..models.args import ModelArgs, QuantArgs, preset
+from ..models.layer_spec import AttentionSpec, LatentAttentionSpec, ParallelSpec, RotarySpec, SelectiveScanSpec
 from ..models.registry import get_model_class
 from . import cuda_ops as c
 from . import moe_cuda
@@ -23,7 +23,21 @@ from .bench_kernels import time_graph
 DEV = "cuda:0"
 # (model, closest one, which of the model's kinds of layer)
 PAIRS = {"movolorn": [("movolorn-8b", "qwen3-8b", ""), ("movolorn-30b-a3b", "qwen3-30b-a3b", "")],
-         "falalix": [("falalix-8b", "qwen3-8b", "parallel"), ("falalix-8b", "qwen3-8b", "scan"), ("falalix-8b", "qwen3-8b", "")]}
+         "falalix": [("falalix-8b", "qwen3-8b", "parallel"), ("falalix-8b", "qwen3-8b", "scan"), ("falalix-8b", "qwen3-8b", "")],
+         "babadra": [("babadra-8b", "deepseek-8b", "latent"), ("babadra-8b", "qwen3-8b", "two-map"),
+                     ("babadra-30b-a3b", "qwen3-30b-a3b", "two-map")]}
+KINDS = {"parallel": lambda m: isinstance(m, ParallelSpec), "scan": lambda m: isinstance(m, SelectiveScanSpec),
+         "latent": lambda m: isinstance(m, LatentAttentionSpec), "two-map": lambda m: getattr(m, "maps", 1) == 2}
+
+
+def args_of(name: str) -> ModelArgs:
+    if name == "deepseek-8b":            # the attention of deepseek-v3 with the width, heads and feed-forward of qwen3-8b, in bf16
+        return dataclasses.replace(preset("deepseek-v3"), hidden_size=4096, n_heads=32, n_kv_heads=32, intermediate_size=12288, vocab_size=151936,
+                                   n_routed_experts=0, quant=QuantArgs(), rope_scaling_factor=4.0, rope_original_max_position=8192,
+                                   max_position_embeddings=32768)
+    return preset(name)
+
+
 # Issue rates that bound recurrent kernels in fp32, per second over 148 SMs at 1.9 GHz: 128 multiply-adds and 16 exponentials
 # per SM and clock (nominal; there is no measured figure for them).
 FMA_RATE, EXP_RATE = 148 * 128 * 1.9e9, 148 * 16 * 1.9e9
@@ -65,17 +79,17 @@ def step_input(seqs: int, q_len: int, kv_len: int, block: int, vocab: int) -> St
 
 
 def cut_to_layers(a: ModelArgs, n: int, kind: str = "") -> ModelArgs:
-    """n layers, all of one kind where a model has several ("parallel", "scan") and one is named."""
+    """n layers, all of one kind (a key of KINDS) where a model has several and one is named."""
     kw = dict(n_layers=n)
     if a.layer_specs:
-        specs = [s for s in a.layer_specs if not kind or (kind == "parallel") == isinstance(s.mixer, ParallelSpec)]
+        specs = [s for s in a.layer_specs if not kind or KINDS[kind](s.mixer)]
         kw.update(layer_specs=specs[:n], layer_runs=list(range(n)), pass_starts=[])
     return dataclasses.replace(a, **kw)
 
 
 @torch.inference_mode()
 def layer_throughput(name: str, layers: int, block: int, kind: str = "") -> List[Dict]:
-    args = cut_to_layers(preset(name), layers, kind)
+    args = cut_to_layers(args_of(name), layers, kind)
     model = get_model_class(args.model_type)(args, device=DEV, dtype=torch.bfloat16).init_random(0)
     if hasattr(model, "finalize_weights"):
         model.finalize_weights()
@@ -111,11 +125,11 @@ class Rows:
         self.pk = peaks()
         self.rows = []
 
-    def add(self, what, ours, like, bytes_ours=0.0, bytes_like=0.0, flops=0.0):
-        def frac(us, nbytes):
-            bound = max(nbytes / (self.pk["hbm_gbs"] * 1e3), flops / (self.pk["bf16_tflops"] * 1e6))
+    def add(self, what, ours, like, bytes_ours=0.0, bytes_like=0.0, flops=0.0, flops_like=None):
+        def frac(us, nbytes, ops):
+            bound = max(nbytes / (self.pk["hbm_gbs"] * 1e3), ops / (self.pk["bf16_tflops"] * 1e6))
             return bound / us
-        fo, fl = frac(ours, bytes_ours), frac(like, bytes_like)
+        fo, fl = frac(ours, bytes_ours, flops), frac(like, bytes_like, flops if flops_like is None else flops_like)
         self.rows.append({"what": what, "us": round(ours, 1), "like_us": round(like, 1), "roofline": round(fo, 3), "like_roofline": round(fl, 3),
                           "farther_by": round(fl / fo, 2)})
 
@@ -293,7 +307,122 @@ def falalix_kernels() -> List[Dict]:
     return R.rows
 
 
-KERNELS = {"movolorn": movolorn_kernels, "falalix": falalix_kernels}
+@torch.inference_mode()
+def babadra_kernels() -> List[Dict]:
+    R = Rows()
+    add = R.add
+    H, heads = 4096, 32
+    # ---- differential attention beside attention with as many query, key and value columns
+    factor = torch.tensor([0.7], device=DEV)
+    for G in (8, 4):
+        for kind, seqs, q_len, kv in STEPS:
+            inp = step_input(seqs, q_len, kv, 16, 1000)
+            nb, row, T = seqs * (-(-kv // 16)) + 1, (heads + 2 * G) * 128, seqs * q_len
+            cache_bytes = 2.0 * seqs * kv * G * 128 * 2
+            sets = _rotated(lambda: (_bf(T, row), _bf(nb, 16, G, 128), _bf(nb, 16, G, 128)), cache_bytes + T * row * 2)[:8]
+            o = time_graph([lambda s=s: c.paged_attention_ext(s[0][:, :heads * 128].unflatten(1, (2 * heads, 64)), s[1].view(nb, 16, 2 * G, 64), s[2], inp,
+                                                              64 ** -0.5, softcap=50.0, mix=(factor, 0.4, 1e-6)) for s in sets])
+            k = time_graph([lambda s=s: c.paged_attention(s[0][:, :heads * 128].unflatten(1, (heads, 128)), s[1], s[2], inp, 128 ** -0.5) for s in sets])
+            byts = cache_bytes + 2.0 * T * heads * 128 * 2
+            pairs = seqs * (q_len * (kv - q_len) + q_len * (q_len + 1) / 2)
+            # products: both maps' scores, and both maps' sums of the values
+            fo, fk = (2.0 * 2 * 64 + 2.0 * 2 * 128) * heads * pairs, 4.0 * 128 * heads * pairs
+            if kind == "prefill":
+                add(f"two-map attention {kind} {seqs} x {q_len} of {kv}, {heads}/{G} heads", o, k, byts, byts, fo, fk)
+            else:
+                add(f"two-map attention {kind} {seqs} x {q_len} of {kv}, {heads}/{G} heads", o, k, byts, byts)
+            del sets
+    # ---- latent attention: from the projected queries to the heads' outputs
+    dim, rd, C, nq, dv = 128, 64, 512, 1536, 128
+    uk, uv = _bf(heads, C, dim, std=0.05), _bf(heads, dv, C, std=0.05)
+    table = torch.randn(8192, rd, device=DEV)
+    kc = uk.transpose(1, 2).contiguous()
+    w_q, w_c, w_down = _bf(nq), _bf(C), _bf(nq + C + rd, H, std=0.02)
+    w_qa, w_kva = w_down[:nq].contiguous(), w_down[nq:].contiguous()
+    for kind, seqs, q_len, kv in STEPS:
+        inp = step_input(seqs, q_len, kv, 16, 1000)
+        nb, T = seqs * (-(-kv // 16)) + 1, seqs * q_len
+        rot = (table, inp.positions, True)
+        sets = _rotated(lambda: (_bf(T, heads * (dim + rd)), _bf(nb, 16, C + rd), _bf(T, C + rd), _bf(T, H)), seqs * kv * 1152.0)[:8]
+        o = time_graph([lambda s=s: c.latent_attention_mla(s[0].view(T, heads, dim + rd), uk, uv, s[1], inp, rot, 0.07, dim) for s in sets])
+
+        def like(s):
+            a, b = c.mla_prepare(s[0].view(T, heads, dim + rd), s[2], inp.positions, inp.slots, table, w_c, 1e-6, s[1], kc, dim, rd, C)
+            return c.mla_v_up(c.mla_attention(a, b, s[1], inp, 0.07, C), uv)
+        k = time_graph([lambda s=s: like(s) for s in sets])
+        pairs = seqs * (q_len * (kv - q_len) + q_len * (q_len + 1) / 2)
+        fl = 2.0 * heads * ((2 * C + rd) * pairs + T * C * (dim + dv))
+        byts = seqs * kv * (C + rd) * 2.0 + T * heads * (dim + rd + dv) * 2.0
+        add(f"latent attention {kind} {seqs} x {q_len} of {kv}, {heads} heads", o, k, byts, byts, fl)
+        if (seqs, q_len) not in ((1, 8192), (256, 1)):
+            continue
+        # ---- what lies ahead of it: down products, norms, rotation, cache write
+        o = time_graph([lambda s=s: c.latent_down(c.linear(s[3], w_down), nq, C, w_q, w_c, 1e-6, rot, inp.slots, s[1]) for s in sets])
+        k = time_graph([lambda s=s: (c.rms_norm(c.linear(s[3], w_qa), w_q, 1e-6), c.linear(s[3], w_kva)) for s in sets])
+        n = nq + C + rd
+        add(f"down products + norms, {T} tokens", o, k, T * (H * 2.0 + n * 2) + n * H * 2.0, T * (H * 4.0 + n * 2) + n * H * 2.0, 2.0 * T * n * H)
+        low = [_bf(T, n) for _ in range(8 if T > 1000 else 32)]
+        o = time_graph([lambda x=x: c.latent_down(x, nq, C, w_q, w_c, 1e-6, rot, inp.slots, sets[0][1]) for x in low])
+        k = time_graph([lambda x=x: (c.rms_norm(x[:, :nq], w_q, 1e-6), c.rms_norm(x[:, nq:nq + C], w_c, 1e-6)) for x in low])
+        add(f"norms + rotation + cache write of {T} latents", o, k, T * n * 4.0, T * (nq + C) * 4.0)
+    # ---- norms, embedding, q / k norm with rotation
+    cs = torch.randn(8192, 128, device=DEV)
+    t64 = torch.randn(8192, 64, device=DEV)
+    pos = _bf(8192, H)
+    for T in (8192, 256):
+        w, w64, w128 = _bf(H), _bf(64), _bf(128)
+        sets = _rotated(lambda: (_bf(T, H), torch.randn(T, H, device=DEV), _bf(T, H)), T * H * 10.0)
+        k = time_graph([lambda s=s: c.add_rms_norm(s[0], s[2], w, 1e-6) for s in sets])
+        o = time_graph([lambda s=s: c.add_norm(s[0], s[1], 1.0, w, 1e-6, w, 1.0) for s in sets])
+        add(f"layer scale + residual + norm, {T} x {H}", o, k, T * H * 12.0, T * H * 8.0)
+        ids, at = torch.randint(0, 30000, (T,), device=DEV).int(), torch.arange(T, device=DEV).int()
+        emb = _bf(30000, H)
+        o = time_graph([lambda s=s: c.add_norm(s[0], s[1], 1.0, w, 1e-6, w, 1.0, (ids, emb, 2.0, at, pos)) for s in sets])
+        add(f"the same at the head of a pass, {T} x {H}", o, k, T * H * 16.0, T * H * 8.0)
+        o = time_graph([lambda: c.embed_rms_norm(ids, emb, 2.0, w, 1e-6, at, pos, 1.0)] * 8)
+        k = time_graph([lambda: c.rms_norm(c.embedding(ids, emb), w, 1e-6)] * 8)
+        add(f"embedding + positions + first norm, {T} x {H}", o, k, T * H * 10.0, T * H * 8.0)
+        inp, row = step_input(1, T, T, 16, 1000), 48 * 128
+        sets = _rotated(lambda: (_bf(T, row), _bf(T // 16 + 1, 16, 8, 128), _bf(T // 16 + 1, 16, 8, 128)), T * row * 2.0)[:24]
+        o = time_graph([lambda s=s: c.qknorm_kvwrite(s[0], inp.slots, w64, w64, 1e-6, s[1].view(-1, 16, 16, 64), s[2], 64, 16, (t64, inp.positions, False))
+                        for s in sets])
+        k = time_graph([lambda s=s: c.rope_qknorm_kvwrite(s[0], inp.positions, inp.slots, cs, w128, w128, 1e-6, s[1], s[2], 32, 8, 128) for s in sets])
+        add(f"q / k norm + rotation + cache write, {T} tokens", o, k, T * 104.0 * 256 + T * 256.0, T * 104.0 * 256 + T * 512.0)
+        # ---- products with an epilogue
+        sets = _rotated(lambda: (_bf(T, H), _bf(24576, H, std=0.02)), 24576 * 8192.0)[:3]
+        o = time_graph([lambda s=s: c.linear_gated(s[0], s[1], "clamped", 7.0) for s in sets])
+        k = time_graph([lambda s=s: c.linear_swiglu(s[0], s[1]) for s in sets])
+        b = 24576 * 8192.0 + T * (8192.0 + 24576.0)
+        add(f"gate / up product + clamped gate, {T} x 24576 x {H}", o, k, b, b, 2.0 * T * 24576 * H)
+        del sets
+    x, head = _bf(256, H), _bf(151936, H, std=0.02)
+    o, k = time_graph([lambda: c.linear_softcap(x, head, 30.0)] * 3), time_graph([lambda: c.linear(x, head)] * 3)
+    add("bounded logits, 256 x 151936", o, k, 151936 * (H * 2.0 + 512.0), 151936 * (H * 2.0 + 512.0), 2.0 * 256 * 151936 * H)
+    del x, head
+    # ---- router and mixture
+    E, W, I, top = 128, 2048, 768, 8
+    wr, br = _bf(E, W, std=0.02), torch.randn(E, device=DEV) * 0.01
+    w13, w2, ls, w = _bf(E, 2 * I, W, std=0.02), _bf(E, W, I, std=0.02), _bf(W), _bf(W)
+    moe_cuda.interleave_w13(w13)
+    for T in (8192, 256):
+        sets = _rotated(lambda: (_bf(T, W), torch.randn(T, W, device=DEV), _bf(T, W)), T * W * 10.0)[:16]
+        o = time_graph([lambda s=s: c.moe_router(c.linear_f32(s[0], wr), top, "softmax_chosen", bias=br) for s in sets])
+        k = time_graph([lambda s=s: c.moe_router(c.linear(s[0], wr), top, "softmax", True) for s in sets])
+        b = T * W * 2.0 + E * W * 2.0 + T * 64.0
+        add(f"router product + choice, {T} x {E}", o, k, b, b, 2.0 * T * E * W)
+        wts, idx = c.moe_router(c.linear(sets[0][0], wr), top, "softmax", True)
+
+        def ours_mix(s):
+            y, dst = moe_cuda.expert_rows(s[0], w13, w2, idx, "clamped", True, 7.0)
+            return moe_cuda.combine_add_norm(y, dst, wts, ls, s[1], w, 1e-6, 1.0)
+        o = time_graph([lambda s=s: ours_mix(s) for s in sets])
+        k = time_graph([lambda s=s: c.add_rms_norm(moe_cuda.moe_experts(s[0], w13, w2, wts, idx, 0, True), s[2], w, 1e-6) for s in sets])
+        b = 3.0 * E * I * W * 2
+        add(f"mixture to the next sublayer's input, {T} tokens", o, k, b + T * W * 12.0, b + T * W * 8.0, 6.0 * T * top * I * W)
+    return R.rows
+
+
+KERNELS = {"movolorn": movolorn_kernels, "falalix": falalix_kernels, "babadra": babadra_kernels}
 
 
 def run(design: str, layers: int = 4, block: int = 16) -> Dict:
