@@ -89,8 +89,11 @@ def test_bounded_scores_keep_their_accuracy():
         def edit(q, k, v):
             q *= size
         step, q, seqs = two_map_step([(0, 150), (150, 1)], 4, 2, 64, 64, 64, 3, edit, DEV, torch.bfloat16)
-        got = ops.paged_attention_ext(q, *step.caches, step.inp, 0.3, softcap=4.0, mix=(torch.tensor([0.2], device=DEV), 1.0, 1e-6))
-        assert rel(got, two_map_want(step, seqs, 0.3, 4.0, 0.2, 0.0, 1e-6)) < 1.2e-2
+        want = two_map_want(step, seqs, 0.3, 4.0, 0.2, 0.0, 1e-6)
+        largest = max(float(torch.einsum("nhid,mhid->hinm", x, y.repeat_interleave(2, 1)).abs().max()) for x, y, _ in seqs)
+        for bound in (0.0, largest):
+            got = ops.paged_attention_ext(q, *step.caches, step.inp, 0.3, softcap=4.0, mix=(torch.tensor([0.2], device=DEV), 1.0, 1e-6), bound=bound)
+            assert rel(got, want) < 1.2e-2
 
 
 # ----------------------------------------------------------------------------- latent attention

@@ -73,6 +73,7 @@ struct DecParams {
   int row_blocks = 1;             // blocks of 16 query rows per kv head (grid.y = n_kv * row_blocks)
   int maps = 1;
   float cap_in = 0.f, cap_out = 0.f;      // cap_out > 0: scores are cap_out * tanh(product * cap_in), in the log2 domain
+  int cap_level = CAP_CHECK;
   const float* mix = nullptr;
   float mix_mult = 0.f, mix_eps = 0.f;
 };
@@ -255,8 +256,8 @@ __global__ void __launch_bounds__(160) decode_attn_tma_kernel(const __grid_const
           mma_bf16_16816(sc[1], qf[kKeepQ ? ks : 0], b2, b3);
         }
         if (CAP) {
-          softcap_row<false>(sc[0], p.cap_in, p.cap_out);
-          softcap_row<false>(sc[1], p.cap_in, p.cap_out);
+          softcap_row(sc[0], p.cap_in, p.cap_level);
+          softcap_row(sc[1], p.cap_in, p.cap_level);
         }
         float mx[2] = {-INFINITY, -INFINITY};
 #pragma unroll
@@ -267,7 +268,7 @@ __global__ void __launch_bounds__(160) decode_attn_tma_kernel(const __grid_const
             const int lim = (e < 2) ? lim_a : lim_b;
             bool ok = tok <= lim && tok < kv_len;
             if (p.window > 0) ok = ok && (tok > lim - p.window || (EXT && tok < p.keep_first));
-            float x = CAP ? sc[i][e] : sc[i][e] * p.scale_log2;
+            float x = sc[i][e] * (CAP ? p.cap_in * p.cap_out : p.scale_log2);
             if (EXT) {
               ok = ok && tok >= ((e < 2) ? lo_a : lo_b);
               x += ((e < 2) ? slope_a : slope_b) * float(tok - lim);
@@ -664,7 +665,7 @@ XL_API int xl_decode_attention_ext(const void* q, const void* k_cache, const voi
                                    const void* kv_lens, const void* block_tables, int seq_begin, int seq_end, int max_blocks,
                                    int block_size, int num_blocks_total, int n_q, int n_kv, int dk, int dv, int q_stride,
                                    float scale, int window, int chunk, int keep_first, const void* slopes, const void* sinks,
-                                   float softcap, long v_pitch, int maps, const void* mix, float mix_mult, float mix_eps, int max_q,
+                                   float softcap, float bound, long v_pitch, int maps, const void* mix, float mix_mult, float mix_eps, int max_q,
                                    int num_splits, void* part_o, void* part_lse, long max_rows, const void* dyn_end, void* stream) {
   using namespace xl_dec;
   if (seq_end <= seq_begin) return 0;
@@ -709,6 +710,7 @@ XL_API int xl_decode_attention_ext(const void* q, const void* k_cache, const voi
   if (softcap > 0.f) {
     p.cap_in = scale / softcap;
     p.cap_out = softcap * 1.4426950408889634f;
+    p.cap_level = cap_level(p.cap_in, bound) == CAP_SMALL ? CAP_SMALL : CAP_CHECK;    // a check finds most rows small
   }
   p.mix = static_cast<const float*>(mix);
   p.mix_mult = mix_mult; p.mix_eps = mix_eps;

@@ -70,6 +70,7 @@ struct Params {
   int chunk;                   // EXT: positions per chunk (<= 0: no chunk mask)
   int keep_first;              // EXT: first keys that stay visible behind the window
   float cap_in, cap_out;       // EXT: bounded scores, cap_out * tanh(product * cap_in) in the log2 domain (cap_out 0: not bounded)
+  int cap_level;
   const float* mix;            // MAPS = 2: factor of the second map
   float mix_mult, mix_eps;
   const int* q_cu;
@@ -359,7 +360,6 @@ prefill_attn_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_con
     // with a distance bias v[] holds finished scores in the log2 domain, otherwise (bounded) raw products that `sc` scales
     const bool capped = SCORE == SCORE_CAP && p.cap_out > 0.f;
     const float sc = SCORE == SCORE_BIAS ? 1.f : capped ? p.cap_in * p.cap_out : p.scale_log2;
-    const float cap_top = capped ? 1.f / p.cap_in : 0.f;
     float m_ref = -INFINITY, l_run = 0.f;                    // m_ref: reference maximum of the raw scores
     bool ok = true;
     for (int j = 0; j < n_tiles && ok; ++j) {
@@ -385,7 +385,7 @@ prefill_attn_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_con
         v[c] = __uint_as_float(s0[c]);
         v[32 + c] = __uint_as_float(s1[c]);
       }
-      if (capped) softcap_row<true>(v, p.cap_in, cap_top);
+      if (capped) softcap_row(v, p.cap_in, p.cap_level);
       if (SCORE == SCORE_BIAS) {
         const float b0 = slope2 * float(kv0 - pos);
 #pragma unroll
@@ -748,7 +748,8 @@ XL_API int xl_prefill_attention_tc(const void* q, const void* k_cache, const voi
 // The same with the score extensions and separate query-key / value head dimensions (multiples of 8, at most 256; 128 with maps = 2):
 //   score(i, j) = scale * q_i . k_j - slopes[h] * (i - j), visible when j <= i, within `window` (> 0) or among the first
 //   `keep_first` keys, and in the same chunk of `chunk` positions (> 0); out = sum_j exp(score) v_j / (sum_j exp(score) + exp(sinks[h])).
-// `slopes` / `sinks` [n_q] fp32, null when absent; `softcap` > 0: scale * q . k becomes softcap * tanh(scale * q . k / softcap).
+// `slopes` / `sinks` [n_q] fp32, null when absent; `softcap` > 0: scale * q . k becomes softcap * tanh(scale * q . k / softcap), and
+// `bound` > 0 promises |q . k| <= bound.
 // `v_pitch`: elements from one cache slot's values to the next one's (0: n_kv * dv), so that values may be a part of the keys.
 // maps = 2: n_q counts the maps' heads (pairs of neighbours), k_cache has 2 n_kv heads, out [T, n_q / 2 * dv] =
 // rms(first - mix[0] * second, mix_eps) * mix_mult.  Returns -3 when the shape, or a distance bias beside bounded scores or two
@@ -757,8 +758,8 @@ XL_API int xl_prefill_attention_ext(const void* q, const void* k_cache, const vo
                                     const void* kv_lens, const void* block_tables, int seq_begin, int seq_end, int max_blocks,
                                     int block_size, int num_blocks_total, int n_q, int n_kv, int dk, int dv, int q_stride,
                                     int total_q_rows, float scale, int window, int chunk, int keep_first, const void* slopes,
-                                    const void* sinks, float softcap, long v_pitch, int maps, const void* mix, float mix_mult, float mix_eps,
-                                    int q_tiles_cap, const void* dyn_begin, const void* dyn_end, void* stream) {
+                                    const void* sinks, float softcap, float bound, long v_pitch, int maps, const void* mix, float mix_mult,
+                                    float mix_eps, int q_tiles_cap, const void* dyn_begin, const void* dyn_end, void* stream) {
   using namespace xl_pf;
   if (maps < 1 || maps > 2 || (maps == 2 && (!mix || (n_q / n_kv) % 2))) return -2;
   const int d_max = maps == 2 ? 128 : 256;
@@ -791,6 +792,7 @@ XL_API int xl_prefill_attention_ext(const void* q, const void* k_cache, const vo
   if (softcap > 0.f) {
     p.cap_in = scale / softcap;
     p.cap_out = softcap * 1.4426950408889634f;
+    p.cap_level = cap_level(p.cap_in, bound) == CAP_SMALL ? CAP_SMALL : CAP_CHECK;    // a check finds most rows small
   }
   p.mix = static_cast<const float*>(mix);
   p.mix_mult = mix_mult; p.mix_eps = mix_eps;

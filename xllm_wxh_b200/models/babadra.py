@@ -42,6 +42,7 @@ class TwoMapWeights:
         self.qkv_w = self.q_norm = self.k_norm = None
         self.lam = None                         # fp32 [4, dim]: lq1, lk1, lq2, lk2
         self.factor = None                      # fp32 [1], of the second map
+        self.bound = 0.0                        # of |q . k|, from the norms' weights
         self.o_w = None
 
 
@@ -136,6 +137,9 @@ class BabadraForCausalLM:
             else:
                 W.qkv_w = torch.cat([dev(q + n) for n in "qkv"], 0)
                 W.q_norm, W.k_norm = dev(q + "q.norm"), dev(q + "k.norm")
+                turn = m.rot.frequencies()[1] if m.rot is not None else 1.0
+                # a normed row is no longer than sqrt(dim); 2 % for the rounding of q and k
+                W.bound = 1.02 * m.dim * float(W.q_norm.abs().max()) * float(W.k_norm.abs().max()) * max(1.0, turn * turn)
                 W.lam = torch.stack([f32(q + n) for n in ("lq1", "lk1", "lq2", "lk2")])
                 W.factor = (torch.exp((W.lam[0] * W.lam[1]).sum()) - torch.exp((W.lam[2] * W.lam[3]).sum()) + m.diff).reshape(1)
             W.o_w = dev(q + "o")
@@ -241,7 +245,7 @@ class BabadraForCausalLM:
         q = ops.qknorm_kvwrite(ops.linear(h, W.qkv_w), inp.slots, W.q_norm, W.k_norm, eps, kv[0], kv[1], n_q, m.kv_heads * m.maps,
                                self._rotation(m.rot, inp))
         return ops.paged_attention_ext(q.unflatten(1, (n_q, m.dim)), kv[0], kv[1], inp, m.scale, softcap=m.softcap,
-                                       mix=(W.factor, 1.0 - m.diff, eps))
+                                       mix=(W.factor, 1.0 - m.diff, eps), bound=W.bound)
 
     def _feed_forward(self, L: BlockWeights, f: FeedForwardSpec, h: torch.Tensor, x: torch.Tensor, w_next: torch.Tensor, lead) -> torch.Tensor:
         """The second sublayer from its normed input h; adds to x and returns the next sublayer's input."""

@@ -45,15 +45,17 @@ def paged_attention(q, k_cache, v_cache, inp, scale, sliding_window=-1):
                                sliding_window)
 
 
-def paged_attention_ext(q, k_cache, v_cache, inp, scale, window=-1, chunk=0, slopes=None, sinks=None, keep_first=0, softcap=0.0, mix=None):
+def paged_attention_ext(q, k_cache, v_cache, inp, scale, window=-1, chunk=0, slopes=None, sinks=None, keep_first=0, softcap=0.0, mix=None,
+                        bound=0.0):
     """Paged attention with a per-head linear distance bias (`slopes` [Hq] fp32), a per-head sink score in the softmax
     denominator (`sinks` [Hq] fp32), keys limited to the query's chunk of `chunk` positions, first positions that stay
     visible behind the window (`keep_first`), scores bounded by `softcap` * tanh(score / softcap), and a value head dimension of
     its own.  q [T, Hq, dk] -> [T, Hq * dv].
     `mix` = (factor fp32 [1], mult, eps): differential attention.  Query and key heads are pairs of two maps, every pair of query
-    heads has one value head's values, and its output is rms(first - factor * second) * mult: [T, Hq / 2 * dv]."""
+    heads has one value head's values, and its output is rms(first - factor * second) * mult: [T, Hq / 2 * dv].
+    `bound` > 0 promises |q . k| <= bound (normed queries and keys), which saves the kernels a check of bounded scores."""
     if q.is_cuda:
-        return _cuda().paged_attention_ext(q, k_cache, v_cache, inp, scale, window, chunk, slopes, sinks, keep_first, softcap, mix)
+        return _cuda().paged_attention_ext(q, k_cache, v_cache, inp, scale, window, chunk, slopes, sinks, keep_first, softcap, mix, bound)
     return ref.paged_attention(q, k_cache, v_cache, inp.q_cu, inp.kv_lens, inp.block_tables, inp.n_seqs, scale, window, chunk,
                                slopes, sinks, keep_first, softcap, mix)
 

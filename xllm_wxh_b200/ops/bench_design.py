@@ -313,7 +313,7 @@ def babadra_kernels() -> List[Dict]:
     add = R.add
     H, heads = 4096, 32
     # ---- differential attention beside attention with as many query, key and value columns
-    factor = torch.tensor([0.7], device=DEV)
+    factor, bound = torch.tensor([0.7], device=DEV), 1.02 * 64         # norm weights of one
     for G in (8, 4):
         for kind, seqs, q_len, kv in STEPS:
             inp = step_input(seqs, q_len, kv, 16, 1000)
@@ -321,7 +321,7 @@ def babadra_kernels() -> List[Dict]:
             cache_bytes = 2.0 * seqs * kv * G * 128 * 2
             sets = _rotated(lambda: (_bf(T, row), _bf(nb, 16, G, 128), _bf(nb, 16, G, 128)), cache_bytes + T * row * 2)[:8]
             o = time_graph([lambda s=s: c.paged_attention_ext(s[0][:, :heads * 128].unflatten(1, (2 * heads, 64)), s[1].view(nb, 16, 2 * G, 64), s[2], inp,
-                                                              64 ** -0.5, softcap=50.0, mix=(factor, 0.4, 1e-6)) for s in sets])
+                                                              64 ** -0.5, softcap=50.0, mix=(factor, 0.4, 1e-6), bound=bound) for s in sets])
             k = time_graph([lambda s=s: c.paged_attention(s[0][:, :heads * 128].unflatten(1, (heads, 128)), s[1], s[2], inp, 128 ** -0.5) for s in sets])
             byts = cache_bytes + 2.0 * T * heads * 128 * 2
             pairs = seqs * (q_len * (kv - q_len) + q_len * (q_len + 1) / 2)

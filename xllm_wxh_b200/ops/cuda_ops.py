@@ -701,7 +701,7 @@ def paged_attention(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tenso
 
 def paged_attention_ext(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tensor, inp, scale: float, window: int = -1, chunk: int = 0,
                         slopes: Optional[torch.Tensor] = None, sinks: Optional[torch.Tensor] = None, keep_first: int = 0,
-                        softcap: float = 0.0, mix=None) -> torch.Tensor:
+                        softcap: float = 0.0, mix=None, bound: float = 0.0) -> torch.Tensor:
     """Paged attention with score extensions and a value dimension of its own: q [T, Hq, dk] (may be a view of the qkv
     buffer), caches [blocks, block, Hkv, dk | dv] -> [T, Hq * dv].  score = scale q.k (bounded by softcap tanh(. / softcap)) -
     slopes[h] * distance; keys of the query's own chunk of `chunk` positions only (0: all); `keep_first` first keys stay visible
@@ -720,7 +720,8 @@ def paged_attention_ext(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.T
         assert t is None or (t.dtype == torch.float32 and t.numel() == Hq and t.is_contiguous())
     out = (torch.zeros if padded else torch.empty)((T, Hq // maps * dv), dtype=q.dtype, device=q.device)
     factor, mult, eps = mix if mix is not None else (None, 0.0, 0.0)
-    ext = (c_float(softcap), c_long(v_cache.stride(1)), c_int(maps), _ptr(factor), c_float(mult), c_float(eps))
+    last = (c_long(v_cache.stride(1)), c_int(maps), _ptr(factor), c_float(mult), c_float(eps))
+    ext = (c_float(softcap), c_float(bound)) + last
     n_dec = inp.B if padded else inp.n_decode
     n_all = inp.B if padded else inp.n_seqs
     has_prefill = inp.has_prefill if padded else n_all > n_dec
@@ -731,7 +732,7 @@ def paged_attention_ext(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.T
                                        _ptr(inp.block_tables), c_int(T), c_int(n_all), c_int(L.MB_cap), c_int(block_size),
                                        c_long(k_cache.shape[0] * block_size), c_int(Hq), c_int(n_kv), c_int(dk), c_int(dv),
                                        c_long(q_stride), c_float(scale), c_int(window), c_int(chunk), c_int(keep_first), _ptr(slopes), _ptr(sinks),
-                                       *ext, _f32flag(q), _stream()), "xl_attention_simt")
+                                       c_float(softcap), *last, _f32flag(q), _stream()), "xl_attention_simt")
         return out
     most = 256 if mix is None else 128
     if q.dtype == torch.float32 or dk % 8 or dv % 8 or dk > most or dv > most or q.stride(1) != dk:
