@@ -120,6 +120,8 @@ MODEL_SOURCES = {
                 "host_util", "recurrent", "sampling", "sandwich_norm"),
     "babadra": ("attention_decode_tma", "attention_prefill_tc", "attention_simt", "gemm_bf16", "gemm_bf16_2cta", "gemm_simt",
                 "host_util", "mla", "mla_attention_tc", "moe", "sampling", "sandwich_norm"),
+    "govuvik": ("attention_decode_tma", "attention_prefill_tc", "attention_simt", "gemm_bf16", "gemm_bf16_2cta", "gemm_simt",
+                "host_util", "moe", "recurrent", "sampling", "sandwich_norm"),
 }
 
 

@@ -13,8 +13,8 @@ import json
 import os
 from typing import Any, Dict, List, Optional
 
-from .layer_spec import (AttentionSpec, FeedForwardSpec, LatentAttentionSpec, LayerSpec, ParallelSpec, RotarySpec, SelectiveScanSpec,
-                         TimeMixSpec, attention_of, pass_starts, run_order)
+from .layer_spec import (AttentionSpec, FeedForwardSpec, GatedLinearSpec, LatentAttentionSpec, LayerSpec, MatrixMemorySpec, ParallelSpec,
+                         RotarySpec, SelectiveScanSpec, TimeMixSpec, attention_of, pass_starts, run_order)
 
 @dataclasses.dataclass
 class QuantArgs:
@@ -90,7 +90,7 @@ class ModelArgs:
     # MTP
     num_nextn_predict_layers: int = 0
     quant: QuantArgs = dataclasses.field(default_factory=QuantArgs)
-    # designs that list their layers one by one (models/movolorn.py, falalix.py, babadra.py); the flat sizes above then hold
+    # designs that list their layers one by one (models/movolorn.py, falalix.py, babadra.py, govuvik.py); the flat sizes above then hold
     # maxima over the layers
     layer_specs: List[LayerSpec] = dataclasses.field(default_factory=list)
     layer_runs: List[int] = dataclasses.field(default_factory=list)      # layer of every run, in order (layers may repeat)
@@ -98,6 +98,7 @@ class ModelArgs:
     embedding_scale: float = 1.0
     residual_mult: float = 1.0          # factor of every sublayer's output on its way into the residual
     position_rows: int = 0              # rows of a learned position table that joins the embedding (0: none)
+    input_conv: int = 0                 # taps of a causal convolution that is added to every mixer's input (0: none)
     logit_softcap: float = 0.0          # logits become softcap * tanh(logits / softcap) (0: they do not)
 
     # ------------------------------------------------------------------ derived
@@ -232,7 +233,11 @@ def _rotary(cfg: Optional[Dict[str, Any]], interleaved: bool) -> Optional[Rotary
     if not cfg or int(cfg.get("dims") or 0) == 0:
         return None
     s = cfg.get("scaling")
-    kw = dict(factor=float(s["factor"]), original=float(s["original"]), fast=float(s["fast"]), slow=float(s["slow"])) if s else {}
+    kw = dict(factor=float(s["factor"]), original=float(s["original"])) if s else {}
+    if s and "high" in s:
+        kw.update(fast=float(s["high"]), slow=float(s["low"]), by_turns=True)
+    elif s:
+        kw.update(fast=float(s["fast"]), slow=float(s["slow"]))
     return RotarySpec(int(cfg["dims"]), float(cfg["base"]), interleaved, **kw)
 
 
@@ -284,8 +289,56 @@ def _babadra_args(cfg: Dict[str, Any]) -> ModelArgs:
         logit_softcap=float(cfg.get("logit_softcap") or 0.0), eos_token_id=int(_first(cfg, "eos_token_id", default=-1)))
 
 
+def _govuvik_layer(i: int, cfg: Dict[str, Any]) -> LayerSpec:
+    kind, m = cfg.get("type"), cfg["mixer"]
+    if kind == "mlstm":
+        mixer = MatrixMemorySpec(heads=int(m["heads"]), dim=int(m["dim"]), vdim=int(m["vdim"]), gate_cap=float(m["gate_cap"]))
+        if min(mixer.heads, mixer.dim, mixer.vdim) < 1 or mixer.gate_cap <= 0:
+            raise ValueError(f"layer {i}: sizes of a matrix memory and the bound of its gates must be positive")
+    elif kind == "parallel":
+        a, t = m["left"], m["right"]
+        H, G, dim, rot = int(a["heads"]), int(a["kv_heads"]), int(a["dim"]), _rotary(a.get("rot"), False)
+        if H < 1 or G < 1 or H % G:
+            raise ValueError(f"layer {i}: {H} heads do not divide over {G} key/value heads")
+        if rot is not None and (rot.dims > dim or rot.dims % 2):
+            raise ValueError(f"layer {i}: {rot.dims} rotated dimensions of {dim}")
+        left = AttentionSpec(heads=H, kv_heads=G, dim=dim, vdim=int(a["vdim"]), scale=float(a["scale"]),
+                             window=int((a.get("mask") or {}).get("size") or 0), conv=int(a["conv"]), mixed_scores=True, learned_sink=True,
+                             qk_norm_all=True, rot=rot)
+        right = GatedLinearSpec(heads=int(t["heads"]), dim=int(t["dim"]), vdim=int(t["vdim"]), tau=float(t["tau"]))
+        if min(left.conv, right.heads, right.dim, right.vdim) < 1 or right.tau <= 0:
+            raise ValueError(f"layer {i}: sizes of a parallel mixer and the root of its decay must be positive")
+        mixer = ParallelSpec(left, right, 0.5, 0.5, branch_norm=True)
+    else:
+        raise ValueError(f"layer {i}: mixer '{kind}' is not supported")
+    f = cfg.get("mlp")
+    if not f:
+        return LayerSpec(mixer, None)
+    if f["kind"] != "moe":
+        raise ValueError(f"layer {i}: feed-forward '{f['kind']}' is not supported")
+    mlp = FeedForwardSpec(ff=int(f["expert"]["ff"]), act="relu2", experts=int(f["router"]["experts"]), top_k=int(f["router"]["top"]),
+                          scoring="softmax_chosen")
+    if not 1 <= mlp.top_k <= mlp.experts:
+        raise ValueError(f"layer {i}: top {mlp.top_k} of {mlp.experts} experts")
+    return LayerSpec(mixer, mlp)
+
+
+def _govuvik_args(cfg: Dict[str, Any]) -> ModelArgs:
+    specs = [_govuvik_layer(i, c) for i, c in enumerate(cfg["layers"])]
+    taps = int((cfg.get("canon") or {}).get("taps", 0))
+    if taps < 1:
+        raise ValueError(f"the input convolution has {taps} taps")
+    dt = str(_first(cfg, "torch_dtype", "dtype", default="bfloat16"))
+    return args_from_layer_list(
+        specs, run_order(len(specs)), model_type="govuvik", dtype=dt if dt in _DTYPES else "bfloat16", vocab_size=int(cfg["vocab"]),
+        hidden_size=int(cfg["width"]), rms_norm_eps=float(cfg["norm"]["eps"]), input_conv=taps,
+        max_position_embeddings=int(_first(cfg, "max_position_embeddings", default=131072)),
+        logit_softcap=float(cfg.get("logit_softcap") or 0.0), eos_token_id=int(_first(cfg, "eos_token_id", default=-1)))
+
+
 _DTYPES = ("float32", "bfloat16")
-_LAYER_LISTS = {"movolorn": _movolorn_args, "falalix": _falalix_args, "babadra": _babadra_args}     # designs that are named by "architecture"
+# designs that are named by "architecture"
+_LAYER_LISTS = {"movolorn": _movolorn_args, "falalix": _falalix_args, "babadra": _babadra_args, "govuvik": _govuvik_args}
 
 
 def args_from_hf_config(cfg: Dict[str, Any]) -> ModelArgs:

@@ -9,7 +9,7 @@ from typing import List, Optional, Tuple, Union
 
 @dataclasses.dataclass(frozen=True)
 class RotarySpec:
-    """Rotary positions on the first `dims` dimensions of a head, optionally with YaRN scaling."""
+    """Rotary positions on the first `dims` dimensions of a head, optionally with YaRN scaling or slowed long wavelengths."""
     dims: int
     base: float
     interleaved: bool = False     # pairs (2i, 2i + 1); else (i, i + dims / 2)
@@ -17,12 +17,18 @@ class RotarySpec:
     original: float = 0.0         # ... of a model of so many positions ...
     fast: float = 32.0            # ... whose dimensions of at least so many turns over them keep their frequency
     slow: float = 1.0             # ... and of at most so many turns are slowed by the factor
+    by_turns: bool = False        # the ramp between the two runs over turns per original context, not over dimensions, and cos and
+                                  # sin keep their size (the scaling of Llama 3.1)
 
     def frequencies(self) -> Tuple[List[float], float]:
         """(angle per position of every pair, factor of cos and sin)."""
         f = [self.base ** (-2.0 * i / self.dims) for i in range(self.dims // 2)]
         if self.factor <= 0:
             return f, 1.0
+        if self.by_turns:
+            turns = [self.original * x / (2 * math.pi) for x in f]
+            keep = [min(max((t - self.slow) / max(self.fast - self.slow, 1e-12), 0.0), 1.0) for t in turns]
+            return [x * s + x / self.factor * (1 - s) for x, s in zip(f, keep)], 1.0
 
         def dim_of(turns):        # dimension that turns so often over the original positions
             return self.dims * math.log(self.original / (2 * math.pi * turns)) / (2 * math.log(self.base))
@@ -41,6 +47,9 @@ class AttentionSpec:
     chunk: int = 0                # positions per chunk that a query may look at (0: all earlier ones)
     window: int = 0               # sliding window in positions (0: none)
     keep_first: int = 0           # first positions of the sequence that stay visible behind the window
+    conv: int = 0                 # taps of a causal convolution on q, k and v ahead of norm and rotation (0: none)
+    mixed_scores: bool = False    # a factor per head, then every head's scores become a weighted sum over all heads' scores
+    learned_sink: bool = False    # a sink score of every head's own, part of the checkpoint
     distance_bias: bool = False   # take slope_h * (i - j) off the scores, slopes from `head_slopes`
     sink: Optional[float] = None  # score of a key without a value that joins the softmax denominator (None: no sink)
     qk_norm: bool = False         # RMS norm over every query and key head
@@ -86,6 +95,26 @@ class TimeMixSpec:
 
 
 @dataclasses.dataclass
+class GatedLinearSpec:
+    """Linear attention with a matrix state per head that decays per key channel, by a power of a gate, ahead of every token."""
+    heads: int
+    dim: int                      # key size of a head
+    vdim: int                     # value size of a head
+    tau: float                    # decay = sigmoid(z)^(1 / tau)
+    decay_rank: int = 0           # inner size of the gate's low-rank projection (0: the checkpoint's tensors tell)
+
+
+@dataclasses.dataclass
+class MatrixMemorySpec:
+    """Matrix memory with exponential input gates and one forget gate per head, kept relative to a running maximum, and a
+    normaliser (xLSTM's mLSTM)."""
+    heads: int
+    dim: int                      # query / key size of a head
+    vdim: int                     # value size of a head
+    gate_cap: float               # bound of both gates ahead of their exponential
+
+
+@dataclasses.dataclass
 class SelectiveScanSpec:
     """Diagonal state space layer with data-dependent step sizes, input and output vectors, behind a short causal
     convolution."""
@@ -99,12 +128,13 @@ class SelectiveScanSpec:
 class ParallelSpec:
     """Two mixers side by side on the same input; their outputs are added with a factor each."""
     left: AttentionSpec
-    right: TimeMixSpec
+    right: Union[TimeMixSpec, GatedLinearSpec]
     left_scale: float = 1.0
     right_scale: float = 1.0
+    branch_norm: bool = False     # every branch's output is normed over the model width ahead of its factor
 
 
-Mixer = Union[AttentionSpec, LatentAttentionSpec, SelectiveScanSpec, ParallelSpec]
+Mixer = Union[AttentionSpec, LatentAttentionSpec, SelectiveScanSpec, MatrixMemorySpec, ParallelSpec]
 
 
 def attention_of(mixer: Mixer) -> Optional[AttentionSpec]:

@@ -24,7 +24,7 @@ def get_model_class(model_type: str):
 
 def _populate():
     import importlib
-    for mod in ("qwen", "deepseek_impl", "movolorn", "falalix", "babadra"):
+    for mod in ("qwen", "deepseek_impl", "movolorn", "falalix", "babadra", "govuvik"):
         importlib.import_module(f"{__package__}.{mod}")
 
 

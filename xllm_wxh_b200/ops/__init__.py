@@ -53,7 +53,8 @@ def paged_attention_ext(q, k_cache, v_cache, inp, scale, window=-1, chunk=0, slo
     its own.  q [T, Hq, dk] -> [T, Hq * dv].
     `mix` = (factor fp32 [1], mult, eps): differential attention.  Query and key heads are pairs of two maps, every pair of query
     heads has one value head's values, and its output is rms(first - factor * second) * mult: [T, Hq / 2 * dv].
-    `bound` > 0 promises |q . k| <= bound (normed queries and keys), which saves the kernels a check of bounded scores."""
+    `bound` > 0 promises |q . k| <= bound (normed queries and keys), which saves the kernels a check of bounded scores.
+    k_cache may have one key head beside several value heads: all query heads then share it (queries of `mix_query_heads`)."""
     if q.is_cuda:
         return _cuda().paged_attention_ext(q, k_cache, v_cache, inp, scale, window, chunk, slopes, sinks, keep_first, softcap, mix, bound)
     return ref.paged_attention(q, k_cache, v_cache, inp.q_cu, inp.kv_lens, inp.block_tables, inp.n_seqs, scale, window, chunk,
@@ -107,14 +108,20 @@ def gate_up_swiglu(x, w, interleaved=False):
 
 
 # ----------------------------------------------------------------------------- sublayers normed before and after, fp32 residual
-def embed_rms_norm(ids, table, scale, w_next, eps, positions=None, pos_table=None, w_offset=0.0):
-    """(fp32 residual x = table[ids] * scale (+ pos_table[positions]), rms(x) * (w_next + w_offset) in the table's dtype)."""
-    return (_cuda() if table.is_cuda else ref).embed_rms_norm(ids, table, scale, w_next, eps, positions, pos_table, w_offset)
+def embed_rms_norm(ids, table, scale, w_next, eps, positions=None, pos_table=None, w_offset=0.0, w_rows=None):
+    """(fp32 residual x = table[ids] * scale (+ pos_table[positions]), rms(x) * (w_next + w_offset) in the table's dtype).
+    With `w_rows` the embedding is normed itself: x = rms(row) * w_rows."""
+    return (_cuda() if table.is_cuda else ref).embed_rms_norm(ids, table, scale, w_next, eps, positions, pos_table, w_offset, w_rows)
 
 
 def post_norm_add_norm(y, x, w_post, w_next, eps):
     """x += rms(y) * w_post (x fp32, in place); returns rms(x) * w_next."""
     return (_cuda() if y.is_cuda else ref).post_norm_add_norm(y, x, w_post, w_next, eps)
+
+
+def branches_post_norm_add_norm(ya, yb, w_a, w_b, scale, x, w_post, w_next, eps):
+    """y = scale * (rms(ya) * w_a + rms(yb) * w_b); x += rms(y) * w_post (x fp32, in place); returns rms(x) * w_next."""
+    return (_cuda() if ya.is_cuda else ref).branches_post_norm_add_norm(ya, yb, w_a, w_b, scale, x, w_post, w_next, eps)
 
 
 def qknorm_kvwrite(qkv, slots, q_w, k_w, eps, k_cache, v_cache, n_q, n_kv, rot=None):
@@ -144,7 +151,7 @@ def linear_softcap(x, w, cap):
 def moe_post_norm_add_norm(h_in, w13, w2, weights, ids, shared, first_identity, x, w_post, w_next, eps, act="silu", interleaved=False):
     """Mixture sublayer from its routing to the next sublayer's input: y = sum_j weights_j expert_j(h_in) (ids from
     `first_identity` on are identity experts: weight times h_in) + shared (or None); x += rms(y) * w_post (fp32, in place);
-    returns rms(x) * w_next."""
+    returns rms(x) * w_next.  act "relu2": experts without a gate, w13 [experts, ff, H]."""
     if h_in.is_cuda:
         from . import moe_cuda
         y, dst_of = moe_cuda.expert_rows(h_in, w13, w2, ids, act, interleaved)
@@ -199,10 +206,12 @@ def act_linear(x, w, act):
     return (_cuda() if x.is_cuda else ref).act_linear(x, w, act)
 
 
-def qknorm_all_kvwrite(qkv, slots, q_w, k_w, eps, k_cache, v_cache, n_q, n_kv):
-    """RMSNorm over the whole query and the whole key projection; k and v into the paged caches.  Rows of qkv may be longer
-    than q, k and v.  Returns q [T, n_q * dk]."""
-    return (_cuda() if qkv.is_cuda else ref).qknorm_all_kvwrite(qkv, slots, q_w, k_w, eps, k_cache, v_cache, n_q, n_kv)
+def qknorm_all_kvwrite(qkv, slots, q_w, k_w, eps, k_cache, v_cache, n_q, n_kv, rot=None, mix=None):
+    """RMSNorm over the whole query and the whole key projection, then the rotation `rot` (as in `qknorm_kvwrite`) if there is one;
+    k and v into the paged caches.  Rows of qkv may be longer than q, k and v.  Returns q [T, n_q * dk], or with `mix` (fp32
+    [n_q, n_q]) the queries [T, n_q * n_kv * dk] of attention whose scores are mixed over the heads: the product of row h and a
+    token's keys of all key heads side by side is sum_g mix[h, g] q_g . k_(g's key head)."""
+    return (_cuda() if qkv.is_cuda else ref).qknorm_all_kvwrite(qkv, slots, q_w, k_w, eps, k_cache, v_cache, n_q, n_kv, rot, mix)
 
 
 def gate_into(o, gate, scale, out):
@@ -233,7 +242,33 @@ def time_mix(r, k, v, z, w0, u, gate, norm_w, scale, eps, state, inp, out):
 def conv_silu(x, w, b, state, inp):
     """silu of a causal convolution per channel over each sequence; w [taps, C]; x may be a strided view; state
     [slots, taps - 1, C]."""
-    return _cuda().conv_silu(x, w, b, state, inp) if x.is_cuda else ref.conv_silu(x, w, b, state, *_seqs(inp))
+    return causal_conv(x, w, b, state, inp, act="silu")
+
+
+def causal_conv(x, w, b, state, inp, act="none", residual=False):
+    """act(b + causal convolution per channel over each sequence) (+ x with `residual`); layouts as `conv_silu`; b may be None."""
+    if x.is_cuda:
+        return _cuda().causal_conv(x, w, b, state, inp, act, residual)
+    return ref.causal_conv(x, w, b, state, *_seqs(inp), act, residual)
+
+
+def gated_memory(q, k, v, z, bias, inv_tau, gate, norm_w, eps, state, inp):
+    """Matrix-state recurrence S = diag(sigmoid(z + bias)^inv_tau) S + k v^T per head, o = S^T q / sqrt(dim); RMS per head with the
+    weight norm_w [vdim], silu gate.  q, k [T, heads * dim], v, gate [T, heads * vdim] may be strided views, z fp32; state
+    [slots, heads, dim, vdim] fp32.  Returns [T, heads * vdim]."""
+    if q.is_cuda:
+        return _cuda().gated_memory(q, k, v, z, bias, inv_tau, gate, norm_w, eps, state, inp)
+    return ref.gated_memory(q, k, v, z, bias, inv_tau, gate, norm_w, eps, state, *_seqs(inp))
+
+
+def matrix_memory(q, k, v, gates, bias, cap, gate, norm_w, eps, state, top, inp):
+    """Matrix memory with exponential gates: per head i = cap tanh((gates_i + bias_i) / cap), f = log sigmoid of the same of gates_f,
+    S = e^f S + e^i k v^T and n = e^f n + e^i k, both relative to e^m of a running maximum m; o = S^T q / max(|n q|, e^-m) with q
+    over sqrt(dim); RMS per head, weight norm_w [heads * vdim], sigmoid gate.  gates fp32 [T, 2 heads] (i, then f), bias fp32
+    [2 heads]; state [slots, heads, dim * vdim + dim] fp32 (S, then n), top [slots, heads] fp32 (m).  Returns [T, heads * vdim]."""
+    if q.is_cuda:
+        return _cuda().matrix_memory(q, k, v, gates, bias, cap, gate, norm_w, eps, state, top, inp)
+    return ref.matrix_memory(q, k, v, gates, bias, cap, gate, norm_w, eps, state, top, *_seqs(inp))
 
 
 def selective_scan(x, dt, dt_bias, A, B, C, D, z, state, inp):

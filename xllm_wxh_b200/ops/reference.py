@@ -175,6 +175,8 @@ def paged_attention(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tenso
     group = Hq // v_cache.shape[2]                  # query heads per value head
     heads = torch.arange(Hq, device=q.device)
     key_of = heads // group if mix is None else heads // group * 2 + heads % 2
+    if mix is None and Hkv == 1:
+        key_of = heads * 0                          # one key head that all query heads share
     out = torch.zeros(T, Hq, Dv, dtype=q.dtype, device=q.device)
     q_cu_h = q_cu.tolist()
     kv_h = kv_lens.tolist()
@@ -395,7 +397,8 @@ def moe_mixture(h: torch.Tensor, w13: torch.Tensor, w2: torch.Tensor, weights: t
         hit = ids == e
         tok = hit.any(-1).nonzero().squeeze(-1)
         if tok.numel():
-            y = linear(gated_act(linear(h[tok], w13[e]), act, limit), w2[e])
+            up = act_linear(h[tok], w13[e], act) if act == "relu2" else gated_act(linear(h[tok], w13[e]), act, limit)
+            y = linear(up, w2[e])
             out.index_add_(0, tok, y.float() * (weights * hit).sum(-1)[tok][:, None])
     out += (weights * (ids >= first_identity)).sum(-1, keepdim=True) * h.float()
     return out if shared is None else out + shared.float()
@@ -414,14 +417,20 @@ def embed_rows(ids: torch.Tensor, table: torch.Tensor, scale: float, positions=N
     return x
 
 
-def embed_rms_norm(ids, table, scale: float, w_next, eps: float, positions=None, pos_table=None, w_offset: float = 0.0):
+def embed_rms_norm(ids, table, scale: float, w_next, eps: float, positions=None, pos_table=None, w_offset: float = 0.0, w_rows=None):
     x = embed_rows(ids, table, scale, positions, pos_table)
+    if w_rows is not None:
+        x = _rms_f32(x, w_rows, eps)
     return x, _rms_f32(x, w_next, eps, w_offset).to(table.dtype)
 
 
 def post_norm_add_norm(y: torch.Tensor, x: torch.Tensor, w_post: torch.Tensor, w_next: torch.Tensor, eps: float) -> torch.Tensor:
     x += _rms_f32(y, w_post, eps)
     return _rms_f32(x, w_next, eps).to(w_next.dtype)
+
+
+def branches_post_norm_add_norm(ya, yb, w_a, w_b, scale, x, w_post, w_next, eps):
+    return post_norm_add_norm(scale * (_rms_f32(ya, w_a, eps) + _rms_f32(yb, w_b, eps)), x, w_post, w_next, eps)
 
 
 def qknorm_kvwrite(qkv, slots, q_w, k_w, eps, k_cache, v_cache, n_q, n_kv, rot=None):
@@ -496,12 +505,18 @@ def act_linear(x: torch.Tensor, w: torch.Tensor, act: str) -> torch.Tensor:
     return (torch.relu(y) ** 2 if act == "relu2" else torch.tanh(y)).to(x.dtype)
 
 
-def qknorm_all_kvwrite(qkv, slots, q_w, k_w, eps, k_cache, v_cache, n_q, n_kv):
-    dk, dv = k_cache.shape[-1], v_cache.shape[-1]
+def qknorm_all_kvwrite(qkv, slots, q_w, k_w, eps, k_cache, v_cache, n_q, n_kv, rot=None, mix=None):
+    T, dk, dv = qkv.shape[0], k_cache.shape[-1], v_cache.shape[-1]
     q, k, v = qkv[:, :(n_q + n_kv) * dk + n_kv * dv].split([n_q * dk, n_kv * dk, n_kv * dv], dim=-1)
-    k_cache.view(-1, n_kv * dk).index_copy_(0, slots.long(), _rms_f32(k, k_w, eps).to(k_cache.dtype))
+    q, k = _rms_f32(q, q_w, eps).view(T, n_q, dk), _rms_f32(k, k_w, eps).view(T, n_kv, dk)
+    if rot is not None:
+        q, k = apply_rotary(q, rot), apply_rotary(k, rot)
+    k_cache.view(-1, n_kv * dk).index_copy_(0, slots.long(), k.reshape(T, -1).to(k_cache.dtype))
     v_cache.view(-1, n_kv * dv).index_copy_(0, slots.long(), v.to(v_cache.dtype))
-    return _rms_f32(q, q_w, eps).to(qkv.dtype)
+    if mix is None:
+        return q.reshape(T, -1).to(qkv.dtype)
+    by_key = torch.einsum("hjg,tjgd->thjd", mix.float().view(n_q, n_kv, -1), q.view(T, n_kv, -1, dk))
+    return by_key.reshape(T, -1).to(qkv.dtype)
 
 
 def gate_into(o: torch.Tensor, gate: torch.Tensor, scale: float, out: torch.Tensor) -> None:
@@ -547,17 +562,68 @@ def time_mix(r, k, v, z, w0, u, gate, norm_w, scale, eps, state, q_cu, kv_lens, 
     out.copy_(o.view(T, H * d) * norm_w.float() * torch.nn.functional.silu(gate.float()) * scale)
 
 
-def conv_silu(x, w, b, state, q_cu, kv_lens, slots, n_seqs):
-    """Causal convolution of every channel (w [taps, C], last row the current input's) + b, then silu; state [slots, taps - 1, C]
-    keeps the last rows."""
+def causal_conv(x, w, b, state, q_cu, kv_lens, slots, n_seqs, act="silu", residual=False):
+    """Causal convolution of every channel (w [taps, C], last row the current input's) + b, then silu (act "silu"); with `residual`
+    x is added; state [slots, taps - 1, C] keeps the last rows."""
     taps = w.shape[0]
     y = torch.zeros(x.shape, dtype=torch.float32)
     for lo, hi, cont, s in _spans(q_cu, kv_lens, slots, n_seqs):
         rows = torch.cat([state[s] if cont else torch.zeros_like(state[s]), x[lo:hi]])
-        y[lo:hi] = sum(rows[i:i + hi - lo].float() * w[i].float() for i in range(taps)) + b.float()
+        y[lo:hi] = sum(rows[i:i + hi - lo].float() * w[i].float() for i in range(taps))
         if taps > 1:
             state[s] = rows[1 - taps:]
-    return torch.nn.functional.silu(y).to(x.dtype)
+    if b is not None:
+        y += b.float()
+    if act == "silu":
+        y = torch.nn.functional.silu(y)
+    return (y + x.float() if residual else y).to(x.dtype)
+
+
+def conv_silu(x, w, b, state, q_cu, kv_lens, slots, n_seqs):
+    return causal_conv(x, w, b, state, q_cu, kv_lens, slots, n_seqs)
+
+
+def gated_memory(q, k, v, z, bias, inv_tau, gate, norm_w, eps, state, q_cu, kv_lens, slots, n_seqs):
+    _, H, dk, dv = state.shape
+    T = q.shape[0]
+    Q, K, V = q.float().reshape(T, H, dk) * dk ** -0.5, k.float().reshape(T, H, dk), v.float().reshape(T, H, dv)
+    W = torch.exp(torch.nn.functional.logsigmoid(z + bias) * inv_tau).view(T, H, dk)
+    o = torch.zeros(T, H, dv)
+    for lo, hi, cont, s in _spans(q_cu, kv_lens, slots, n_seqs):
+        S = state[s].clone() if cont else torch.zeros_like(state[s])
+        for t in range(lo, hi):
+            S = W[t][:, :, None] * S + K[t][:, :, None] * V[t][:, None, :]
+            o[t] = torch.einsum("hk,hkv->hv", Q[t], S)
+        state[s] = S
+    o = _rms_f32(o, norm_w, eps).view(T, H * dv)
+    return (o * torch.nn.functional.silu(gate.float())).to(q.dtype)
+
+
+def matrix_memory(q, k, v, gates, bias, cap, gate, norm_w, eps, state, top, q_cu, kv_lens, slots, n_seqs):
+    T, H = q.shape[0], top.shape[1]
+    dk = q.shape[1] // H
+    dv = v.shape[1] // H
+    Q, K, V = q.float().reshape(T, H, dk) * dk ** -0.5, k.float().reshape(T, H, dk), v.float().reshape(T, H, dv)
+    log_i, f = (cap * torch.tanh((gates + bias) / cap)).split(H, -1)
+    log_f = torch.nn.functional.logsigmoid(f)
+    o = torch.zeros(T, H, dv)
+    for lo, hi, cont, s in _spans(q_cu, kv_lens, slots, n_seqs):
+        S = (state[s] if cont else torch.zeros_like(state[s]))[:, :dk * dv].reshape(H, dk, dv).clone()
+        n = (state[s] if cont else torch.zeros_like(state[s]))[:, dk * dv:].clone()
+        m = top[s].clone() if cont else torch.zeros_like(top[s])
+        for t in range(lo, hi):
+            m_new = torch.maximum(log_f[t] + m, log_i[t])
+            fd, ia = torch.exp(log_f[t] + m - m_new), torch.exp(log_i[t] - m_new)
+            m = m_new
+            ki = ia[:, None] * K[t]
+            S = fd[:, None, None] * S + ki[:, :, None] * V[t][:, None, :]
+            n = fd[:, None] * n + ki
+            den = torch.maximum((n * Q[t]).sum(-1).abs(), torch.exp(-m)) + 1e-6
+            o[t] = torch.einsum("hk,hkv->hv", Q[t], S) / den[:, None]
+        state[s] = torch.cat([S.reshape(H, -1), n], -1)
+        top[s] = m
+    o = o * torch.rsqrt(o.pow(2).mean(-1, keepdim=True) + eps)
+    return (o.view(T, H * dv) * norm_w.float() * torch.sigmoid(gate.float())).to(q.dtype)
 
 
 def selective_scan(x, dt, dt_bias, A, B, C, D, z, state, q_cu, kv_lens, slots, n_seqs):
