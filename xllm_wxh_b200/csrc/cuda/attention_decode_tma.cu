@@ -71,6 +71,7 @@ struct DecParams {
   const float* slopes = nullptr;
   const float* sinks = nullptr;
   int row_blocks = 1;             // blocks of 16 query rows per kv head (grid.y = n_kv * row_blocks)
+  int shared_keys = 0;            // one key head for all value heads
   int maps = 1;
   float cap_in = 0.f, cap_out = 0.f;      // cap_out > 0: scores are cap_out * tanh(product * cap_in), in the log2 domain
   int cap_level = CAP_CHECK;
@@ -193,7 +194,7 @@ __global__ void __launch_bounds__(160) decode_attn_tma_kernel(const __grid_const
           const int z = blk * p.block_size + tok % p.block_size;
 #pragma unroll
           for (int h = 0; h < (KH > VH ? KH : VH); ++h) {
-            if (h < KH) tma_load_3d(dK + h * SLAB + b * bt_tok * 128, &tmK, &bars->full[s], h * 64, kvh, z);
+            if (h < KH) tma_load_3d(dK + h * SLAB + b * bt_tok * 128, &tmK, &bars->full[s], h * 64, EXT && p.shared_keys ? 0 : kvh, z);
             if (h < VH) tma_load_3d(dV + h * SLAB + b * bt_tok * 128, &tmV, &bars->full[s], h * 64, kvh, z);
           }
         }
@@ -665,12 +666,13 @@ XL_API int xl_decode_attention_ext(const void* q, const void* k_cache, const voi
                                    const void* kv_lens, const void* block_tables, int seq_begin, int seq_end, int max_blocks,
                                    int block_size, int num_blocks_total, int n_q, int n_kv, int dk, int dv, int q_stride,
                                    float scale, int window, int chunk, int keep_first, const void* slopes, const void* sinks,
-                                   float softcap, float bound, long v_pitch, int maps, const void* mix, float mix_mult, float mix_eps, int max_q,
+                                   float softcap, float bound, long v_pitch, int shared_keys, int maps, const void* mix, float mix_mult,
+                                   float mix_eps, int max_q,
                                    int num_splits, void* part_o, void* part_lse, long max_rows, const void* dyn_end, void* stream) {
   using namespace xl_dec;
   if (seq_end <= seq_begin) return 0;
   if (chunk > 0 && keep_first > 0) return -2;
-  if (maps < 1 || maps > 2 || (maps == 2 && (!mix || (n_q / n_kv) % 2))) return -2;
+  if (maps < 1 || maps > 2 || (maps == 2 && (!mix || shared_keys || (n_q / n_kv) % 2))) return -2;
   if (dk < 8 || dk % 8) return -3;
   dk *= maps;                                  // the keys of both maps lie side by side
   if (dk > 256 || dv < 8 || dv > 256 || dv % 8 || v_pitch % 8) return -3;
@@ -680,7 +682,7 @@ XL_API int xl_decode_attention_ext(const void* q, const void* k_cache, const voi
   if ((reinterpret_cast<uintptr_t>(k_cache) & 127) || (reinterpret_cast<uintptr_t>(v_cache) & 127)) return -3;
   const int box_tokens = block_size < 64 ? block_size : 64;
   const uint64_t slots = uint64_t(num_blocks_total) * block_size;
-  const CUtensorMap* tk = xl_host::tmap_3d(k_cache, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 2, slots, n_kv, dk, box_tokens, 1, 64,
+  const CUtensorMap* tk = xl_host::tmap_3d(k_cache, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 2, slots, shared_keys ? 1 : n_kv, dk, box_tokens, 1, 64,
                                            CU_TENSOR_MAP_SWIZZLE_128B);
   const CUtensorMap* tv = xl_host::tmap_3d(v_cache, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 2, slots, n_kv, dv, box_tokens, 1, 64,
                                            CU_TENSOR_MAP_SWIZZLE_128B, v_pitch);
@@ -707,6 +709,7 @@ XL_API int xl_decode_attention_ext(const void* q, const void* k_cache, const voi
   p.sinks = static_cast<const float*>(sinks);
   p.row_blocks = (n_q / n_kv * (max_q < 1 ? 1 : max_q) + 15) / 16;
   p.maps = maps;
+  p.shared_keys = shared_keys;
   if (softcap > 0.f) {
     p.cap_in = scale / softcap;
     p.cap_out = softcap * 1.4426950408889634f;

@@ -71,6 +71,7 @@ struct Params {
   int keep_first;              // EXT: first keys that stay visible behind the window
   float cap_in, cap_out;       // EXT: bounded scores, cap_out * tanh(product * cap_in) in the log2 domain (cap_out 0: not bounded)
   int cap_level;
+  int shared_keys;             // EXT: one key head for all value heads
   const float* mix;            // MAPS = 2: factor of the second map
   float mix_mult, mix_eps;
   const int* q_cu;
@@ -258,7 +259,7 @@ prefill_attn_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_con
     const int which = sl_all >= KS ? 1 : 0;          // 0 = K, 1 = V
     const int slab = which ? sl_all - KS : sl_all;
     const int column = which ? slab * 64 : slab % QS * 64;
-    const int cache_head = which || MAPS == 1 ? kvh : kvh * MAPS + slab / QS;
+    const int cache_head = !which && EXT && p.shared_keys ? 0 : which || MAPS == 1 ? kvh : kvh * MAPS + slab / QS;
     const int bx = lane % boxes;
     bool ok = true;
     for (int j = 0; j < n_tiles && ok; ++j) {
@@ -751,6 +752,7 @@ XL_API int xl_prefill_attention_tc(const void* q, const void* k_cache, const voi
 // `slopes` / `sinks` [n_q] fp32, null when absent; `softcap` > 0: scale * q . k becomes softcap * tanh(scale * q . k / softcap), and
 // `bound` > 0 promises |q . k| <= bound.
 // `v_pitch`: elements from one cache slot's values to the next one's (0: n_kv * dv), so that values may be a part of the keys.
+// `shared_keys`: k_cache has one key head, which all query heads share, beside n_kv value heads.
 // maps = 2: n_q counts the maps' heads (pairs of neighbours), k_cache has 2 n_kv heads, out [T, n_q / 2 * dv] =
 // rms(first - mix[0] * second, mix_eps) * mix_mult.  Returns -3 when the shape, or a distance bias beside bounded scores or two
 // maps, is not covered.
@@ -758,10 +760,10 @@ XL_API int xl_prefill_attention_ext(const void* q, const void* k_cache, const vo
                                     const void* kv_lens, const void* block_tables, int seq_begin, int seq_end, int max_blocks,
                                     int block_size, int num_blocks_total, int n_q, int n_kv, int dk, int dv, int q_stride,
                                     int total_q_rows, float scale, int window, int chunk, int keep_first, const void* slopes,
-                                    const void* sinks, float softcap, float bound, long v_pitch, int maps, const void* mix, float mix_mult,
-                                    float mix_eps, int q_tiles_cap, const void* dyn_begin, const void* dyn_end, void* stream) {
+                                    const void* sinks, float softcap, float bound, long v_pitch, int shared_keys, int maps, const void* mix,
+                                    float mix_mult, float mix_eps, int q_tiles_cap, const void* dyn_begin, const void* dyn_end, void* stream) {
   using namespace xl_pf;
-  if (maps < 1 || maps > 2 || (maps == 2 && (!mix || (n_q / n_kv) % 2))) return -2;
+  if (maps < 1 || maps > 2 || (maps == 2 && (!mix || shared_keys || (n_q / n_kv) % 2))) return -2;
   const int d_max = maps == 2 ? 128 : 256;
   if (dk < 8 || dk > d_max || dk % 8 || dv < 8 || dv > d_max || dv % 8) return -3;
   if (v_pitch % 8 || (slopes && (softcap > 0.f || maps == 2))) return -3;
@@ -776,7 +778,7 @@ XL_API int xl_prefill_attention_ext(const void* q, const void* k_cache, const vo
   // boxes of 64 columns: columns past the head dimension come back as zeros and add nothing to the products
   const CUtensorMap* tq = xl_host::tmap_3d(q, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 2, total_q_rows, n_q, dk, BQ, 1, 64,
                                            CU_TENSOR_MAP_SWIZZLE_128B, q_stride);
-  const CUtensorMap* tk = xl_host::tmap_3d(k_cache, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 2, slots, n_kv * maps, dk, box_tokens, 1, 64,
+  const CUtensorMap* tk = xl_host::tmap_3d(k_cache, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 2, slots, shared_keys ? 1 : n_kv * maps, dk, box_tokens, 1, 64,
                                            CU_TENSOR_MAP_SWIZZLE_128B);
   const CUtensorMap* tv = xl_host::tmap_3d(v_cache, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 2, slots, n_kv, dv, box_tokens, 1, 64,
                                            CU_TENSOR_MAP_SWIZZLE_128B, v_pitch);
@@ -789,6 +791,7 @@ XL_API int xl_prefill_attention_ext(const void* q, const void* k_cache, const vo
   p.sinks = static_cast<const float*>(sinks);
   p.chunk = chunk;
   p.keep_first = keep_first;
+  p.shared_keys = shared_keys;
   if (softcap > 0.f) {
     p.cap_in = scale / softcap;
     p.cap_out = softcap * 1.4426950408889634f;

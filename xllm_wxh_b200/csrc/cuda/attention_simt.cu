@@ -29,6 +29,7 @@ struct Params {
   const float* sinks;
   float softcap;                  // > 0: bounded scores
   long v_pitch;                   // elements from one slot's values to the next one's
+  int shared_keys;                // one key head for all value heads
   const float* mix;               // MAPS = 2
   float mix_mult, mix_eps;
 };
@@ -50,7 +51,7 @@ __global__ void __launch_bounds__(128) attention_simt_kernel(const Params<T> p) 
   float first[kMaxCols];                         // MAPS = 2: the first map's output
 #pragma unroll
   for (int map = 0; map < MAPS; ++map) {
-  const int h = h_out * MAPS + map, kh = kvh * MAPS + map;
+  const int h = h_out * MAPS + map, kh = p.shared_keys ? 0 : kvh * MAPS + map, n_kh = p.shared_keys ? 1 : p.n_kv * MAPS;
   __syncwarp();
   for (int i = lane; i < p.dk; i += 32) q[i] = to_f32(p.q[size_t(t) * p.q_stride + size_t(h) * p.dk + i]) * p.scale;
   __syncwarp();
@@ -74,7 +75,7 @@ __global__ void __launch_bounds__(128) attention_simt_kernel(const Params<T> p) 
       const int b = min(key / p.block_size, p.max_blocks - 1);
       slot = long(bt[b]) * p.block_size + key % p.block_size;
       if (slot < 0 || slot >= p.cache_slots) slot = 0;
-      const T* k = p.k_cache + (size_t(slot) * (p.n_kv * MAPS) + kh) * p.dk;
+      const T* k = p.k_cache + (size_t(slot) * n_kh + kh) * p.dk;
       float d = 0.f;
       for (int i = 0; i < p.dk; ++i) d = fmaf(q[i], to_f32(k[i]), d);
       if (p.softcap > 0.f) d = act_softcap(d, p.softcap);
@@ -124,7 +125,7 @@ template <typename T>
 static int launch(const void* q, const void* k_cache, const void* v_cache, void* out, const void* token_seq, const void* positions,
                   const void* block_tables, int rows, int n_seqs, int max_blocks, int block_size, long cache_slots, int n_q, int n_kv,
                   int dk, int dv, long q_stride, float scale, int window, int chunk, int keep_first, const void* slopes, const void* sinks,
-                  float softcap, long v_pitch, int maps, const void* mix, float mix_mult, float mix_eps, cudaStream_t st) {
+                  float softcap, long v_pitch, int shared_keys, int maps, const void* mix, float mix_mult, float mix_eps, cudaStream_t st) {
   Params<T> p;
   p.q = static_cast<const T*>(q);
   p.k_cache = static_cast<const T*>(k_cache);
@@ -141,11 +142,14 @@ static int launch(const void* q, const void* k_cache, const void* v_cache, void*
   p.sinks = static_cast<const float*>(sinks);
   p.softcap = softcap;
   p.v_pitch = v_pitch > 0 ? v_pitch : long(n_kv) * dv;
+  p.shared_keys = shared_keys;
   p.mix = static_cast<const float*>(mix);
   p.mix_mult = mix_mult; p.mix_eps = mix_eps;
   const long blocks = (long(rows) * (n_q / maps) + 3) / 4;
-  if (maps == 2) attention_simt_kernel<T, 2><<<int(blocks), 128, 4 * dk * sizeof(float), st>>>(p);
-  else attention_simt_kernel<T, 1><<<int(blocks), 128, 4 * dk * sizeof(float), st>>>(p);
+  const size_t smem = size_t(4) * dk * sizeof(float);
+  auto kernel = maps == 2 ? attention_simt_kernel<T, 2> : attention_simt_kernel<T, 1>;
+  if (smem > 48 * 1024) cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, int(smem));
+  kernel<<<int(blocks), 128, smem, st>>>(p);
   return cudaGetLastError() == cudaSuccess ? 0 : -1;
 }
 
@@ -156,15 +160,17 @@ static int launch(const void* q, const void* k_cache, const void* v_cache, void*
 XL_API int xl_attention_simt(const void* q, const void* k_cache, const void* v_cache, void* out, const void* token_seq,
                              const void* positions, const void* block_tables, int rows, int n_seqs, int max_blocks, int block_size,
                              long cache_slots, int n_q, int n_kv, int dk, int dv, long q_stride, float scale, int window, int chunk,
-                             int keep_first, const void* slopes, const void* sinks, float softcap, long v_pitch, int maps, const void* mix,
-                             float mix_mult, float mix_eps, int f32, void* stream) {
+                             int keep_first, const void* slopes, const void* sinks, float softcap, long v_pitch, int shared_keys, int maps,
+                             const void* mix, float mix_mult, float mix_eps, int f32, void* stream) {
   if (rows <= 0) return 0;
-  if (maps < 1 || maps > 2 || (maps == 2 && (!mix || (n_q / n_kv) % 2))) return -2;
-  if (n_kv <= 0 || n_q % n_kv || dk <= 0 || dk > 2048 || dv <= 0 || dv > 32 * xl_as::kMaxCols) return -2;
+  if (maps < 1 || maps > 2 || (maps == 2 && (!mix || shared_keys || (n_q / n_kv) % 2))) return -2;
+  if (n_kv <= 0 || n_q % n_kv || dk <= 0 || dk > 12288 || dv <= 0 || dv > 32 * xl_as::kMaxCols) return -2;
   cudaStream_t st = static_cast<cudaStream_t>(stream);
   if (f32)
     return xl_as::launch<float>(q, k_cache, v_cache, out, token_seq, positions, block_tables, rows, n_seqs, max_blocks, block_size,
-                                cache_slots, n_q, n_kv, dk, dv, q_stride, scale, window, chunk, keep_first, slopes, sinks, softcap, v_pitch, maps, mix, mix_mult, mix_eps, st);
+                                cache_slots, n_q, n_kv, dk, dv, q_stride, scale, window, chunk, keep_first, slopes, sinks, softcap, v_pitch, shared_keys, maps, mix,
+                                mix_mult, mix_eps, st);
   return xl_as::launch<__nv_bfloat16>(q, k_cache, v_cache, out, token_seq, positions, block_tables, rows, n_seqs, max_blocks, block_size,
-                                      cache_slots, n_q, n_kv, dk, dv, q_stride, scale, window, chunk, keep_first, slopes, sinks, softcap, v_pitch, maps, mix, mix_mult, mix_eps, st);
+                                      cache_slots, n_q, n_kv, dk, dv, q_stride, scale, window, chunk, keep_first, slopes, sinks, softcap, v_pitch, shared_keys, maps, mix,
+                                mix_mult, mix_eps, st);
 }

@@ -483,7 +483,8 @@ XL_API int xl_gemm_bf16_act(const void* A, const void* W, void* C, int M, int N,
 
 // Grouped GEMM over expert-sorted rows: C[r, :] = A[r, :] * W[expert(r)]^T for the rows listed in the tile table
 // (`tile_*` arrays and `num_m_tiles` live on the device; `max_m_tiles` bounds them for the launch).
-// swiglu != 0: W holds interleaved gate/up rows and C has N/2 columns (1: silu gate, 2: tanh-gelu gate, 3: clamped gate).
+// swiglu != 0: W holds interleaved gate/up rows and C has N/2 columns (1: silu gate, 2: tanh-gelu gate, 3: clamped gate);
+// 4: N columns without a gate, squared relu of the accumulators.
 XL_API int xl_grouped_gemm_bf16(const void* A, const void* W, void* C, int M_cap, int N, int K, int lda, int ldc, int num_experts,
                                 const void* tile_expert, const void* tile_row0, const void* tile_row_end,
                                 const void* num_m_tiles, int max_m_tiles, int swiglu, int c_rows_per_expert, int c_col_stride,
@@ -498,6 +499,9 @@ XL_API int xl_grouped_gemm_bf16(const void* A, const void* W, void* C, int M_cap
   g.num_m_tiles = static_cast<const int*>(num_m_tiles);
   g.enabled = 1;
   if (max_m_tiles <= 0) return 0;
+  if (swiglu == 4)
+    return xl::launch<xl::EPI_RELU2>(A, W, C, nullptr, M_cap, N, K, lda, K, ldc, static_cast<cudaStream_t>(stream), nullptr, &g,
+                                     num_experts, max_m_tiles);
   if (swiglu == 3)
     return xl::launch<xl::EPI_CLAMPED>(A, W, C, nullptr, M_cap, N, K, lda, K, ldc, static_cast<cudaStream_t>(stream), nullptr, &g,
                                        num_experts, max_m_tiles, limit);

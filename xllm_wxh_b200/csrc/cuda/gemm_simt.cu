@@ -124,10 +124,10 @@ XL_API int xl_gemm_simt_batched(const void* A, const void* W, void* C, int batch
 }
 
 // Grouped form: W [E, N, K] dense, the tile table of `xl_moe_sort`; `row_src` (may be null) maps a sorted row to
-// row_src[row] / row_div of A.
+// row_src[row] / row_div of A.  `act` as in xl_gemm_simt.
 XL_API int xl_grouped_gemm_simt(const void* A, const void* W, void* C, int N, int K, long lda, long ldc, const void* tile_expert,
                                 const void* tile_row0, const void* tile_row_end, const void* num_m_tiles, int max_m_tiles,
-                                const void* row_src, int row_div, int f32, void* stream) {
+                                const void* row_src, int row_div, int act, int f32, void* stream) {
   if (max_m_tiles <= 0 || N <= 0) return 0;
   xl_simt::Tiles g;
   g.tile_expert = static_cast<const int*>(tile_expert);
@@ -136,5 +136,6 @@ XL_API int xl_grouped_gemm_simt(const void* A, const void* W, void* C, int N, in
   g.num_m_tiles = static_cast<const int*>(num_m_tiles);
   g.row_src = static_cast<const int*>(row_src);
   g.row_div = row_div < 1 ? 1 : row_div;
-  return xl_simt::dispatch(A, W, C, 0, N, K, lda, K, ldc, f32, f32, g, xl_simt::Epi{nullptr, xl::ACT_NONE, 0.f, 0, 0, 0}, 2 * max_m_tiles, static_cast<cudaStream_t>(stream));
+  return xl_simt::dispatch(A, W, C, 0, N, K, lda, K, ldc, f32, f32, g, xl_simt::Epi{nullptr, act, 0.f, 0, 0, 0}, 2 * max_m_tiles,
+                           static_cast<cudaStream_t>(stream));
 }

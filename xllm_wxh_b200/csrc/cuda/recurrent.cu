@@ -3,9 +3,9 @@
 // starts from zero, so a record needs no clearing when its slot changes hands.
 //
 //   token_shift     blends of every row with its predecessor (inputs of time mixing); keeps the last row
-//   conv_silu       causal convolution per channel + silu (ahead of the selective scan); keeps the last inputs
-//   time_mix        matrix state per head, decay per key channel, bonus for the current token; then RMS per head, weight and
-//                   silu gate.  Single rows: one CTA streams a head's matrix through registers.  Longer portions: a portion
+//   causal_conv     causal convolution per channel (+ silu, ahead of the selective scan); keeps the last inputs
+//   matrix_*        matrix state per head (time mixing, gated linear attention, matrix memory); then RMS per head, weight and
+//                   gate.  Single rows: one CTA streams a head's matrix through registers.  Longer portions: a portion
 //                   is cut into segments; (A) every segment's own contribution to the state and its decay, (B) the states
 //                   that the segments start from, (C) the segments' outputs from those, all in fp32
 //   selective_scan  diagonal state space recurrence; its step sizes, decays, D x and silu(z) are part of the kernel
@@ -59,12 +59,9 @@ __device__ __forceinline__ float softplus(float z) {
 // remembers.  Models in 32-bit take the one that is exact to the last place near 1.
 template <typename T>
 __device__ __forceinline__ float decay_exp(float x) {
-  if constexpr (sizeof(T) == 4) return 1.f + expm1f(x);
+  if constexpr (sizeof(T) == 4) return x > -0.5f ? 1.f + expm1f(x) : __expf(x);
   else return __expf(x);
 }
-template <typename T>
-__device__ __forceinline__ float decay_of(float z) { return decay_exp<T>(-__expf(z)); }
-
 template <int V, typename T>
 __device__ __forceinline__ void load_n(const T* p, float (&f)[V]) {
   if constexpr (V == 8) load8(p, f);
@@ -183,15 +180,16 @@ __global__ void __launch_bounds__(256) token_shift_kernel(const T* __restrict__ 
   }
 }
 
-// ============================================================================ causal convolution + silu
+// ============================================================================ causal convolution (+ silu, + its input)
+struct ConvOut { int silu, residual; };          // out = act(convolution) (+ x)
 // A thread owns V channels of a tile of consecutive rows and keeps the last TAPS - 1 inputs in registers (TAPS = 0: any
 // number of taps, inputs read again for every row).
 constexpr int kConvRows = 16, kConvRowsSingle = 2;
 
 template <typename T, int V, int TAPS, int ROWS>
-__global__ void __launch_bounds__(128, sizeof(T) == 2 ? 5 : 1) conv_silu_kernel(const T* __restrict__ x, const T* __restrict__ w, const T* __restrict__ bias,
+__global__ void __launch_bounds__(128, sizeof(T) == 2 ? 5 : 1) causal_conv_kernel(const T* __restrict__ x, const T* __restrict__ w, const T* __restrict__ bias,
                                                         T* __restrict__ state, T* __restrict__ out, const int* __restrict__ token_seq,
-                                                        const Seqs q, int rows, int C, int taps_rt, long ldx) {
+                                                        const Seqs q, int rows, int C, int taps_rt, long ldx, const ConvOut act) {
   constexpr int H = TAPS > 1 ? TAPS - 1 : 1;
   const int taps = TAPS > 0 ? TAPS : taps_rt;
   const int c = (blockIdx.y * blockDim.x + threadIdx.x) * V;
@@ -199,7 +197,9 @@ __global__ void __launch_bounds__(128, sizeof(T) == 2 ? 5 : 1) conv_silu_kernel(
   const int t0 = blockIdx.x * ROWS, t1 = min(rows, t0 + ROWS);
   float b[V], hist[H][V];
   Raw<T, V> wt[TAPS > 0 ? TAPS : 1];
-  load_n<V>(bias + c, b);
+#pragma unroll
+  for (int e = 0; e < V; ++e) b[e] = 0.f;
+  if (bias) load_n<V>(bias + c, b);
   if (TAPS > 0) {
 #pragma unroll
     for (int i = 0; i < TAPS; ++i) wt[i].load(w + size_t(i) * C + c);
@@ -281,7 +281,10 @@ __global__ void __launch_bounds__(128, sizeof(T) == 2 ? 5 : 1) conv_silu_kernel(
         }
       }
 #pragma unroll
-      for (int e = 0; e < V; ++e) y[e] = act_silu(y[e]);
+      for (int e = 0; e < V; ++e) {
+        if (act.silu) y[e] = act_silu(y[e]);
+        if (act.residual) y[e] += cur[e];
+      }
       store_n<V>(out + size_t(t) * C + c, y);
     }
   }
@@ -308,24 +311,110 @@ __global__ void __launch_bounds__(128) conv_record_kernel(const T* __restrict__ 
   }
 }
 
-// ============================================================================ time mixing
+// ============================================================================ matrix state per head
+// S [dk, dv] per head, updated by every token's k v^T behind a decay:
+//   MIX_BONUS   time mixing: decay exp(-exp(z + w0)) per key channel; o = S^T r ahead of the update, plus the current token times u
+//   MIX_GATED   gated linear attention: decay sigmoid(z + w0)^inv_tau per key channel; o = S^T q behind the update
+//   MIX_MEMORY  matrix memory: decay e^f and input factor e^i per head relative to a running maximum m, a normaliser n that is updated
+//               like a column of S with value 1; o = S^T q / (max(|n q|, e^-m) + 1e-6) behind the update
+// then RMS per head, weight and gate (silu, MIX_MEMORY: sigmoid).
+enum { MIX_BONUS = 0, MIX_GATED = 1, MIX_MEMORY = 2 };
+constexpr float kMemoryEps = 1e-6f;
+
 template <typename T>
 struct MixParams {
-  const T *r, *k, *v, *gate;       // [rows, H * d], row pitch ld
-  const float* z;                  // [rows, H * d] dense
-  const float *w0, *u;             // [H * d]
-  const T* norm_w;                 // [H * d]
-  float* state;                    // [records, H, d, d] (key, value)
+  const T *r, *k, *v, *gate;       // [rows, H * dk] (queries, keys), [rows, H * dv], row pitch ld (gate: ldg)
+  const float* z;                  // [rows, H * dk] dense; MIX_MEMORY: [rows, 2 H], input gates, then forget gates
+  const float *w0, *u;             // [H * dk] (MIX_MEMORY: biases [2 H]); MIX_BONUS
+  const T* norm_w;                 // weight of head h at h * norm_step
+  float* state;                    // [records, H, dk, dv] (key, value), MIX_MEMORY: n [dk] behind every head's matrix
   T* out;                          // row pitch ldo
   long ld, ldg, ldo;
-  int H, d;
+  int H, dk, dv, norm_step;
   float scale, eps;
+  float q_scale, inv_tau, cap;     // MIX_GATED, MIX_MEMORY: factor of q; MIX_GATED; MIX_MEMORY: bound of the gates
+  float* top;                      // MIX_MEMORY: [records, H] running maxima
+  float* fi;                       // MIX_MEMORY: decays, input factors and e^-m of longer portions, [3, H, rows]
+  int rows;
   Seqs q;
   // segments of longer portions
   int L;                           // rows per segment
-  float* ws_s;                     // [segments, H, d, d]: what a segment adds to the state, then the state it starts from
-  float* ws_p;                     // [segments, H, d]: product of its decays
+  float* ws_s;                     // [segments, H, record]: what a segment adds to the state, then the state it starts from
+  float* ws_p;                     // [segments, H, dk]: product of its decays
 };
+template <int KIND, typename T>
+__device__ __forceinline__ size_t record_size(const MixParams<T>& p) {
+  return size_t(p.dk) * p.dv + (KIND == MIX_MEMORY ? p.dk : 0);
+}
+template <int KIND, typename T>
+__device__ __forceinline__ float decay_of(const MixParams<T>& p, float z) {
+  if constexpr (KIND == MIX_BONUS) return decay_exp<T>(-__expf(z));
+  else return decay_exp<T>(-softplus(-z) * p.inv_tau);
+}
+template <int KIND>
+__device__ __forceinline__ float out_gate(float g) {
+  if constexpr (KIND == MIX_MEMORY) return 1.f / (1.f + __expf(-g));
+  else return act_silu(g);
+}
+// log input and log forget gate of a head
+template <typename T>
+__device__ __forceinline__ float2 log_gates(const MixParams<T>& p, size_t t, int h) {
+  const float* z = p.z + t * (2 * p.H);
+  return make_float2(act_softcap(z[h] + p.w0[h], p.cap), -softplus(-act_softcap(z[p.H + h] + p.w0[p.H + h], p.cap)));
+}
+
+// MIX_MEMORY, portions of min_len and more rows: m <- max(log f + m, log i) over a sequence, one warp per (sequence, head).  A lane
+// composes the steps of kGateRows neighbouring tokens, the lanes' compositions are scanned.
+constexpr int kGateRows = 8;
+template <typename T>
+__global__ void __launch_bounds__(128) memory_gates_kernel(const MixParams<T> p, int min_len) {
+  const int seq = blockIdx.x, h = blockIdx.y * 4 + (threadIdx.x >> 5), lane = threadIdx.x & 31;
+  const int start = p.q.q_cu[seq], len = p.q.q_cu[seq + 1] - start;
+  if (len < min_len || len < 1 || h >= p.H) return;
+  const int slot = p.q.slots[seq];
+  if (slot < 0 || slot >= p.q.n_slots) return;             // recorded by the kernels that follow
+  float carry = p.q.kv_lens[seq] > len ? p.top[size_t(slot) * p.H + h] : 0.f;
+  const size_t plane = size_t(p.H) * p.rows;
+  for (int b = 0; b < len; b += 32 * kGateRows) {
+    float li[kGateRows], lf[kGateRows], F = 0.f, I = -INFINITY;
+#pragma unroll
+    for (int e = 0; e < kGateRows; ++e) {
+      const int t = b + lane * kGateRows + e;
+      const float2 g = t < len ? log_gates(p, size_t(start + t), h) : make_float2(-INFINITY, 0.f);
+      li[e] = g.x;
+      lf[e] = g.y;
+      I = fmaxf(g.y + I, g.x);
+      F += g.y;
+    }
+#pragma unroll
+    for (int o = 1; o < 32; o <<= 1) {
+      const float pf = __shfl_up_sync(0xffffffffu, F, o), pi = __shfl_up_sync(0xffffffffu, I, o);
+      if (lane >= o) {
+        I = fmaxf(F + pi, I);
+        F += pf;
+      }
+    }
+    float before = __shfl_up_sync(0xffffffffu, fmaxf(F + carry, I), 1);
+    if (lane == 0) before = carry;
+    float m[kGateRows];
+#pragma unroll
+    for (int e = 0; e < kGateRows; ++e) m[e] = fmaxf(lf[e] + (e > 0 ? m[e > 0 ? e - 1 : 0] : before), li[e]);
+    before = __shfl_up_sync(0xffffffffu, m[kGateRows - 1], 1);        // what the lane ahead of this one arrived at
+    if (lane == 0) before = carry;
+#pragma unroll
+    for (int e = 0; e < kGateRows; ++e) {
+      const int t = b + lane * kGateRows + e;
+      if (t < len) {
+        float* dst = p.fi + size_t(h) * p.rows + start + t;
+        dst[0] = decay_exp<T>(fminf(lf[e] + (e > 0 ? m[e > 0 ? e - 1 : 0] : before) - m[e], 0.f));
+        dst[plane] = __expf(li[e] - m[e]);
+        dst[2 * plane] = __expf(-m[e]);
+      }
+    }
+    carry = __shfl_sync(0xffffffffu, m[kGateRows - 1], 31);
+  }
+  if (lane == 0) p.top[size_t(slot) * p.H + h] = carry;
+}
 
 // Portions of two and more rows are cut into segments of L rows, numbered through the batch.  Every warp finds segment
 // `target`: its sequence, its place there and how many the sequence has.
@@ -355,39 +444,42 @@ __device__ __forceinline__ bool find_segment(const Seqs& q, int L, int target, i
   return false;
 }
 
-// One (segment, head) per CTA.  D: head dimension padded to 32, 64 or 128.  Thread (kg, vg) owns keys kg * KT ..., values
-// vg * VT ... of the head's matrix, as pairs of neighbouring keys: the more of both, the fewer reads of shared memory per
+// One (segment, head) per CTA.  DK, DV: key and value size of a head padded to 32, 64 or 128.  Thread (kg, vg) owns keys kg * KT ...,
+// values vg * VT ... of the head's matrix, as pairs of neighbouring keys: the more of both, the fewer reads of shared memory per
 // element, which bound this kernel beside the multiply-adds.
-template <int D> struct MixCfg {
-  static constexpr int KT = D == 32 ? 4 : 8, VT = 8;
-  static constexpr int KG = D / KT, VG = D / VT, kThreads = KG * VG;
-  static constexpr int kMinBlocks = D == 128 ? 1 : D == 64 ? 5 : 12;
+template <int DK, int DV> struct MixCfg {
+  static constexpr int KT = DK == 32 ? 4 : 8, VT = 8;
+  static constexpr int KG = DK / KT, VG = DV / VT, kThreads = KG * VG;
+  static constexpr int kMinBlocks = kThreads > 128 ? 1 : kThreads > 64 ? 2 : kThreads > 32 ? 5 : DK == 32 ? 12 : 8;
   // Place of key c in a row of shared memory.  Eight key groups are read at a time, four keys of each: with eight keys per
   // group every other four groups have their halves swapped, so that the reads meet no bank twice.
   __device__ static constexpr int key_at(int c) { return KT == 4 ? c : c ^ (((c >> 5) & 1) << 2); }
 };
 // Eight keys from c (a multiple of 8) on.
-template <int D>
+template <int DK>
 __device__ __forceinline__ void store_keys(float* row, int c, const float (&f)[8]) {
-  *reinterpret_cast<float4*>(row + MixCfg<D>::key_at(c)) = make_float4(f[0], f[1], f[2], f[3]);
-  *reinterpret_cast<float4*>(row + MixCfg<D>::key_at(c + 4)) = make_float4(f[4], f[5], f[6], f[7]);
+  *reinterpret_cast<float4*>(row + MixCfg<DK, 32>::key_at(c)) = make_float4(f[0], f[1], f[2], f[3]);
+  *reinterpret_cast<float4*>(row + MixCfg<DK, 32>::key_at(c + 4)) = make_float4(f[4], f[5], f[6], f[7]);
 }
-template <int D>
+template <int DK>
 __device__ __forceinline__ void load_keys(const float* row, int c, float (&f)[8]) {
-  *reinterpret_cast<float4*>(f) = *reinterpret_cast<const float4*>(row + MixCfg<D>::key_at(c));
-  *reinterpret_cast<float4*>(f + 4) = *reinterpret_cast<const float4*>(row + MixCfg<D>::key_at(c + 4));
+  *reinterpret_cast<float4*>(f) = *reinterpret_cast<const float4*>(row + MixCfg<DK, 32>::key_at(c));
+  *reinterpret_cast<float4*>(f + 4) = *reinterpret_cast<const float4*>(row + MixCfg<DK, 32>::key_at(c + 4));
 }
 constexpr int kMixRows = 16;      // rows staged in shared memory at a time
 
 // v8, g8: 8-element accesses to the inputs / to gate and output are aligned; s4: rows of the state are multiples of 16 bytes
-template <typename T, int D, bool OUT>
-__global__ void __launch_bounds__(MixCfg<D>::kThreads, sizeof(T) == 2 ? MixCfg<D>::kMinBlocks : 1) time_mix_segment_kernel(const MixParams<T> p, int v8, int g8, int s4) {
-  using C = MixCfg<D>;
+template <typename T, int DK, int DV, int KIND, bool OUT>
+__global__ void __launch_bounds__(MixCfg<DK, DV>::kThreads, sizeof(T) == 2 ? MixCfg<DK, DV>::kMinBlocks : 1)
+matrix_segment_kernel(const MixParams<T> p, int v8, int g8, int s4) {
+  using C = MixCfg<DK, DV>;
   constexpr int KT = C::KT, VT = C::VT, KG = C::KG, NT = C::kThreads;
-  __shared__ __align__(16) float sK[kMixRows][D], sW[kMixRows][D], sV[kMixRows][D];
-  __shared__ __align__(16) float sR[OUT ? kMixRows : 1][D], sO[OUT ? kMixRows : 1][D];
-  __shared__ __align__(16) float sNw[OUT ? D : 1], sU[OUT ? D : 1];
-  __shared__ float sBonus[kMixRows];
+  constexpr bool BONUS = KIND == MIX_BONUS, MEMORY = KIND == MIX_MEMORY;
+  __shared__ __align__(16) float sK[kMixRows][DK], sW[kMixRows][DK], sV[kMixRows][DV];
+  __shared__ __align__(16) float sR[OUT ? kMixRows : 1][DK], sO[OUT ? kMixRows : 1][DV];
+  __shared__ __align__(16) float sNw[OUT ? DV : 1], sU[OUT && BONUS ? DK : 1];
+  __shared__ float sRow[kMixRows];                        // MIX_BONUS: product with the current token; MIX_MEMORY: n q
+  __shared__ float sLeast[MEMORY ? kMixRows : 1];         // e^-m
   int seq, seg, n_seg;
   if (!find_segment(p.q, p.L, blockIdx.x, seq, seg, n_seg)) return;
   if (!OUT && seg == n_seg - 1) return;                   // nothing starts behind the last segment
@@ -397,110 +489,164 @@ __global__ void __launch_bounds__(MixCfg<D>::kThreads, sizeof(T) == 2 ? MixCfg<D
   }
   const int slot = record_of(p.q, seq);
   if (slot < 0) return;
-  const int h = blockIdx.y, d = p.d, tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
+  const int h = blockIdx.y, dk = p.dk, dv = p.dv, tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
   const int kg = tid % KG, vg = tid / KG;
   const int start = p.q.q_cu[seq], len = p.q.q_cu[seq + 1] - start;
   const int t0 = start + seg * p.L, n = min(p.L, len - seg * p.L);
   const bool cont = p.q.kv_lens[seq] > len;
-  const size_t mat = size_t(d) * d;
+  const size_t mat = record_size<KIND>(p);
   float* rec = p.state + (size_t(slot) * p.H + h) * mat;
   float* seg_s = p.ws_s ? p.ws_s + (size_t(blockIdx.x) * p.H + h) * mat : nullptr;
 
-  uint64_t S[KT / 2][VT];
+  uint64_t S[KT / 2][VT], N[MEMORY ? KT / 2 : 1];
 #pragma unroll
   for (int i = 0; i < KT / 2; ++i)
 #pragma unroll
     for (int j = 0; j < VT; ++j) S[i][j] = 0;
+#pragma unroll
+  for (int i = 0; i < (MEMORY ? KT / 2 : 1); ++i) N[i] = 0;
   if (OUT && (n_seg > 1 || cont)) {
     const float* src = n_seg > 1 ? seg_s : rec;
 #pragma unroll
     for (int i = 0; i < KT / 2; ++i) {
       float a[2][VT] = {};
+      float nn[2] = {};
 #pragma unroll
       for (int e = 0; e < 2; ++e) {
         const int key = kg * KT + 2 * i + e;
-        if (key < d) {
-          const float* row = src + size_t(key) * d + vg * VT;
+        if (key < dk) {
+          if (MEMORY) nn[e] = src[size_t(dk) * dv + key];
+          const float* row = src + size_t(key) * dv + vg * VT;
 #pragma unroll
           for (int j = 0; j < VT; j += 4) {
             if (s4) {
-              if (vg * VT + j < d) *reinterpret_cast<float4*>(a[e] + j) = *reinterpret_cast<const float4*>(row + j);
+              if (vg * VT + j < dv) *reinterpret_cast<float4*>(a[e] + j) = *reinterpret_cast<const float4*>(row + j);
             } else {
 #pragma unroll
               for (int l = j; l < j + 4; ++l)
-                if (vg * VT + l < d) a[e][l] = row[l];
+                if (vg * VT + l < dv) a[e][l] = row[l];
             }
           }
         }
       }
+      if (MEMORY) N[MEMORY ? i : 0] = pack2(nn[0], nn[1]);
 #pragma unroll
       for (int j = 0; j < VT; ++j) S[i][j] = pack2(a[0][j], a[1][j]);
     }
   }
-  float prod = 1.f;                                       // !OUT: decay of key `tid` over the segment
-  // Rows are finished (and their bonus is prepared) by vectors of 8 columns: LR lanes per row, RP rows per warp and pass.
-  constexpr int LR = D / 8, RP = 32 / LR, PASSES = kMixRows / (NT / 32 * RP);
+  constexpr int PR = (DK + NT - 1) / NT;
+  float prod[PR];                                         // !OUT: decay of keys `tid`, `tid` + NT ... over the segment
+#pragma unroll
+  for (int i = 0; i < PR; ++i) prod[i] = 1.f;
+  // Rows are finished by vectors of 8 columns: LR lanes per row, RP rows per warp and pass; LK lanes per row for its keys.
+  constexpr int LR = DV / 8, RP = 32 / LR, PASSES = kMixRows / (NT / 32 * RP);
+  constexpr int LK = DK / 8, RK = 32 / LK;
+  static_assert(PASSES >= 1, "rows per pass");
   const int fr_row = warp * RP + lane / LR, fr_c = lane % LR * 8;
   if (OUT) {                                              // visible behind the first tile's barrier
-    for (int c = tid; c < D; c += NT) {
-      sNw[OUT ? c : 0] = c < d ? to_f32(p.norm_w[h * d + c]) * p.scale : 0.f;
-      sU[OUT ? c : 0] = c < d ? p.u[h * d + c] : 0.f;
-    }
+    for (int c = tid; c < DV; c += NT) sNw[OUT ? c : 0] = c < dv ? to_f32(p.norm_w[h * p.norm_step + c]) * p.scale : 0.f;
+    if (BONUS)
+      for (int c = tid; c < DK; c += NT) sU[OUT && BONUS ? c : 0] = c < dk ? p.u[h * dk + c] : 0.f;
   }
-  // rows of this head on their way: vector i * NT + tid of the [row][8 columns] tile (v8 only)
-  constexpr int NV = kMixRows * (D / 8) / NT;
-  Vec8<T> fk[NV], fv[NV], fr[OUT ? NV : 1];
-  Vec8<float> fz[NV];
+  // rows of this head on their way: vector i * NT + tid of the [row][8 columns] tiles (v8 only)
+  constexpr int EK = kMixRows * (DK / 8), EV = kMixRows * (DV / 8);
+  constexpr int NK = (EK + NT - 1) / NT, NV = (EV + NT - 1) / NT;
+  Vec8<T> fk[NK], fv[NV], fr[OUT ? NK : 1];
+  Vec8<float> fz[MEMORY ? 1 : NK];
+  float2 ffi[MEMORY ? NK : 1];
+  const size_t plane = size_t(p.H) * p.rows;
   auto fetch = [&](int b) {
     const int m = min(kMixRows, n - b);
 #pragma unroll
-    for (int i = 0; i < NV; ++i) {
-      const int e = i * NT + tid, row = e / (D / 8), c = e % (D / 8) * 8;
-      if (row < m && c < d) {
-        const size_t t = size_t(t0 + b + row), at = t * p.ld + size_t(h) * d + c;
+    for (int i = 0; i < NK; ++i) {
+      const int e = i * NT + tid, row = e / (DK / 8), c = e % (DK / 8) * 8;
+      if (row < m && c < dk) {
+        const size_t t = size_t(t0 + b + row), at = t * p.ld + size_t(h) * dk + c;
         fk[i].load(p.k + at);
-        fv[i].load(p.v + at);
         if (OUT) fr[OUT ? i : 0].load(p.r + at);
-        fz[i].load(p.z + t * (size_t(p.H) * d) + size_t(h) * d + c);
+        if constexpr (MEMORY) {
+          const float* g = p.fi + size_t(h) * p.rows + t;
+          ffi[i] = make_float2(g[0], g[plane]);
+        } else {
+          fz[i].load(p.z + t * (size_t(p.H) * dk) + size_t(h) * dk + c);
+        }
       }
+    }
+#pragma unroll
+    for (int i = 0; i < NV; ++i) {
+      const int e = i * NT + tid, row = e / (DV / 8), c = e % (DV / 8) * 8;
+      if (row < m && c < dv) fv[i].load(p.v + size_t(t0 + b + row) * p.ld + size_t(h) * dv + c);
     }
   };
   if (v8) fetch(0);
   for (int b = 0; b < n; b += kMixRows) {
     const int m = min(kMixRows, n - b);
     // stage the rows; those beyond m leave the state as it is (decay 1, key 0)
+    if (MEMORY && OUT && tid < kMixRows) sLeast[MEMORY ? tid : 0] = tid < m ? p.fi[2 * plane + size_t(h) * p.rows + t0 + b + tid] : 1.f;
     if (v8) {
 #pragma unroll
-      for (int i = 0; i < NV; ++i) {
-        const int e = i * NT + tid, row = e / (D / 8), c = e % (D / 8) * 8;
-        float k[8] = {}, v[8] = {}, r[8] = {}, w[8];
+      for (int i = 0; i < NK; ++i) {
+        const int e = i * NT + tid, row = e / (DK / 8), c = e % (DK / 8) * 8;
+        if (EK % NT && e >= EK) break;
+        float k[8] = {}, r[8] = {}, w[8];
 #pragma unroll
         for (int j = 0; j < 8; ++j) w[j] = 1.f;
-        if (row < m && c < d) {
+        if (row < m && c < dk) {
           fk[i].get(k);
-          fv[i].get(v);
           if (OUT) fr[OUT ? i : 0].get(r);
-          float w0[8];
-          fz[i].get(w);
-          load8(p.w0 + h * d + c, w0);
+          if constexpr (MEMORY) {
 #pragma unroll
-          for (int j = 0; j < 8; ++j) w[j] = decay_of<T>(w[j] + w0[j]);
+            for (int j = 0; j < 8; ++j) {
+              w[j] = ffi[i].x;
+              k[j] *= ffi[i].y;
+            }
+          } else {
+            float w0[8];
+            fz[i].get(w);
+            load8(p.w0 + h * dk + c, w0);
+#pragma unroll
+            for (int j = 0; j < 8; ++j) w[j] = decay_of<KIND>(p, w[j] + w0[j]);
+          }
+          if (!BONUS) {
+#pragma unroll
+            for (int j = 0; j < 8; ++j) r[j] *= p.q_scale;
+          }
         }
-        store_keys<D>(sK[row], c, k);
-        store_keys<D>(sW[row], c, w);
+        store_keys<DK>(sK[row], c, k);
+        store_keys<DK>(sW[row], c, w);
+        if (OUT) store_keys<DK>(sR[row], c, r);
+      }
+#pragma unroll
+      for (int i = 0; i < NV; ++i) {
+        const int e = i * NT + tid, row = e / (DV / 8), c = e % (DV / 8) * 8;
+        if (EV % NT && e >= EV) break;
+        float v[8] = {};
+        if (row < m && c < dv) fv[i].get(v);
         store8(&sV[row][c], v);
-        if (OUT) store_keys<D>(sR[row], c, r);
       }
     } else {
-      for (int i = tid; i < kMixRows * D; i += NT) {
-        const int row = i / D, c = i % D;
-        const bool in = row < m && c < d;
-        const size_t t = size_t(t0 + b + row), at = t * p.ld + size_t(h) * d + c;
+      for (int i = tid; i < kMixRows * DK; i += NT) {
+        const int row = i / DK, c = i % DK;
+        const bool in = row < m && c < dk;
+        const size_t t = size_t(t0 + b + row), at = t * p.ld + size_t(h) * dk + c;
         const int to = C::key_at(c);
-        sK[row][to] = in ? to_f32(p.k[at]) : 0.f;
-        sV[row][c] = in ? to_f32(p.v[at]) : 0.f;
-        sW[row][to] = in ? decay_of<T>(p.z[t * (size_t(p.H) * d) + size_t(h) * d + c] + p.w0[h * d + c]) : 1.f;
-        if (OUT) sR[row][to] = in ? to_f32(p.r[at]) : 0.f;
+        float k = in ? to_f32(p.k[at]) : 0.f, w = 1.f;
+        if (in) {
+          if constexpr (MEMORY) {
+            const float* g = p.fi + size_t(h) * p.rows + t;
+            w = g[0];
+            k *= g[plane];
+          } else {
+            w = decay_of<KIND>(p, p.z[t * (size_t(p.H) * dk) + size_t(h) * dk + c] + p.w0[h * dk + c]);
+          }
+        }
+        sK[row][to] = k;
+        sW[row][to] = w;
+        if (OUT) sR[row][to] = in ? to_f32(p.r[at]) * (BONUS ? 1.f : p.q_scale) : 0.f;
+      }
+      for (int i = tid; i < kMixRows * DV; i += NT) {
+        const int row = i / DV, c = i % DV;
+        sV[row][c] = row < m && c < dv ? to_f32(p.v[size_t(t0 + b + row) * p.ld + size_t(h) * dv + c]) : 0.f;
       }
     }
     __syncthreads();
@@ -510,29 +656,41 @@ __global__ void __launch_bounds__(MixCfg<D>::kThreads, sizeof(T) == 2 ? MixCfg<D
 #pragma unroll
       for (int q = 0; q < PASSES; ++q) {
         const int row = q * (NT / 32 * RP) + fr_row;
-        float s = 0.f;
-        if (row < m) {
-          if (g8 && fr_c < d) gate[OUT ? q : 0].load(p.gate + size_t(t0 + b + row) * p.ldg + size_t(h) * d + fr_c);
-          float r[8], k[8], u[8];
-          load_keys<D>(sR[row], fr_c, r);
-          load_keys<D>(sK[row], fr_c, k);
-          load8(&sU[fr_c], u);
-#pragma unroll
-          for (int j = 0; j < 8; ++j) s = fmaf(r[j] * u[j], k[j], s);
-        }
-#pragma unroll
-        for (int o = LR / 2; o > 0; o >>= 1) s += __shfl_xor_sync(0xffffffffu, s, o);
-        if (lane % LR == 0 && row < m) sBonus[row] = s;    // read behind the next barrier
+        if (row < m && g8 && fr_c < dv) gate[OUT ? q : 0].load(p.gate + size_t(t0 + b + row) * p.ldg + size_t(h) * dv + fr_c);
       }
-    } else if (tid < D) {
+      if (BONUS) {
 #pragma unroll
-      for (int row = 0; row < kMixRows; ++row) prod *= sW[row][C::key_at(tid)];
+        for (int q = 0; q < kMixRows; q += NT / 32 * RK) {
+          const int row = q + warp * RK + lane / LK, c = lane % LK * 8;
+          float s = 0.f;
+          if (row < m) {
+            float r[8], k[8], u[8];
+            load_keys<DK>(sR[row], c, r);
+            load_keys<DK>(sK[row], c, k);
+            load8(&sU[c], u);
+#pragma unroll
+            for (int j = 0; j < 8; ++j) s = fmaf(r[j] * u[j], k[j], s);
+          }
+#pragma unroll
+          for (int o = LK / 2; o > 0; o >>= 1) s += __shfl_xor_sync(0xffffffffu, s, o);
+          if (lane % LK == 0 && row < m) sRow[row] = s;    // read behind the next barrier
+        }
+      }
+    } else {
+#pragma unroll
+      for (int i = 0; i < PR; ++i) {
+        const int c = i * NT + tid;
+        if (DK % NT == 0 || c < DK) {
+#pragma unroll
+          for (int row = 0; row < kMixRows; ++row) prod[i] *= sW[row][C::key_at(c)];
+        }
+      }
     }
 #pragma unroll 1
     for (int row = 0; row < kMixRows; ++row) {
       float vf[8];
       load8(&sV[row][vg * VT], vf);
-      uint64_t v[VT], o[VT];
+      uint64_t v[VT], o[VT], den = 0;
 #pragma unroll
       for (int j = 0; j < VT; ++j) {
         v[j] = pack2(vf[j], vf[j]);
@@ -543,8 +701,9 @@ __global__ void __launch_bounds__(MixCfg<D>::kThreads, sizeof(T) == 2 ? MixCfg<D
         const int at = C::key_at(kg * KT + 4 * i);
         const ulonglong2 k2 = *reinterpret_cast<const ulonglong2*>(&sK[row][at]);
         const ulonglong2 w2 = *reinterpret_cast<const ulonglong2*>(&sW[row][at]);
-        if (OUT) {
-          const ulonglong2 r2 = *reinterpret_cast<const ulonglong2*>(&sR[row][at]);
+        ulonglong2 r2 = {0, 0};
+        if (OUT) r2 = *reinterpret_cast<const ulonglong2*>(&sR[row][at]);
+        if (OUT && BONUS) {
 #pragma unroll
           for (int j = 0; j < VT; ++j) o[j] = fma2(r2.y, S[2 * i + 1][j], fma2(r2.x, S[2 * i][j], o[j]));
         }
@@ -552,6 +711,15 @@ __global__ void __launch_bounds__(MixCfg<D>::kThreads, sizeof(T) == 2 ? MixCfg<D
         for (int j = 0; j < VT; ++j) {
           S[2 * i][j] = fma2(w2.x, S[2 * i][j], mul2(k2.x, v[j]));
           S[2 * i + 1][j] = fma2(w2.y, S[2 * i + 1][j], mul2(k2.y, v[j]));
+        }
+        if (MEMORY) {
+          N[MEMORY ? 2 * i : 0] = fma2(w2.x, N[MEMORY ? 2 * i : 0], k2.x);
+          N[MEMORY ? 2 * i + 1 : 0] = fma2(w2.y, N[MEMORY ? 2 * i + 1 : 0], k2.y);
+          if (OUT) den = fma2(r2.y, N[MEMORY ? 2 * i + 1 : 0], fma2(r2.x, N[MEMORY ? 2 * i : 0], den));
+        }
+        if (OUT && !BONUS) {
+#pragma unroll
+          for (int j = 0; j < VT; ++j) o[j] = fma2(r2.y, S[2 * i + 1][j], fma2(r2.x, S[2 * i][j], o[j]));
         }
       }
       if (OUT) {
@@ -565,6 +733,13 @@ __global__ void __launch_bounds__(MixCfg<D>::kThreads, sizeof(T) == 2 ? MixCfg<D
         float a = sum_to_lanes<VT>(y, kg);
         if (KG == 16) a += __shfl_xor_sync(0xffffffffu, a, 8);
         if (KG == 8 || kg < 8) sO[row][vg * VT + kg] = a;
+        if (MEMORY) {
+          const float2 f = unpack2(den);
+          float d = f.x + f.y;
+#pragma unroll
+          for (int w = KG / 2; w > 0; w >>= 1) d += __shfl_xor_sync(0xffffffffu, d, w);
+          if (tid == 0) sRow[row] = d;
+        }
       }
     }
     __syncthreads();
@@ -572,32 +747,34 @@ __global__ void __launch_bounds__(MixCfg<D>::kThreads, sizeof(T) == 2 ? MixCfg<D
 #pragma unroll
       for (int q = 0; q < PASSES; ++q) {
         const int row = q * (NT / 32 * RP) + fr_row;
-        const float bonus = row < m ? sBonus[row] : 0.f;
-        float o[8], ss = 0.f;
+        float o[8], ss = 0.f, f = 0.f;                     // f: factor of the current token, or of the whole row
+        if (BONUS && row < m) f = sRow[row];
+        if (MEMORY && row < m) f = 1.f / (fmaxf(fabsf(sRow[row]), sLeast[MEMORY ? row : 0]) + kMemoryEps);
         load8(&sO[row][fr_c], o);
 #pragma unroll
         for (int j = 0; j < 8; ++j) {
-          o[j] = fmaf(bonus, sV[row][fr_c + j], o[j]);            // zero beyond d
+          if (BONUS) o[j] = fmaf(f, sV[row][fr_c + j], o[j]);     // zero beyond dv
+          if (MEMORY) o[j] *= f;
           ss = fmaf(o[j], o[j], ss);
         }
 #pragma unroll
         for (int w = LR / 2; w > 0; w >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, w);
-        const float inv = rsqrtf(ss / float(d) + p.eps);
+        const float inv = rsqrtf(ss / float(dv) + p.eps);
         if (row < m) {
           const size_t t = size_t(t0 + b + row);
-          T* out = p.out + t * p.ldo + size_t(h) * d + fr_c;
+          T* out = p.out + t * p.ldo + size_t(h) * dv + fr_c;
           float nw[8], g[8];
           load8(&sNw[fr_c], nw);
           if (g8) {
             gate[OUT ? q : 0].get(g);
 #pragma unroll
-            for (int j = 0; j < 8; ++j) o[j] = o[j] * inv * nw[j] * act_silu(g[j]);
-            if (fr_c < d) store8(out, o);
+            for (int j = 0; j < 8; ++j) o[j] = o[j] * inv * nw[j] * out_gate<KIND>(g[j]);
+            if (fr_c < dv) store8(out, o);
           } else {
 #pragma unroll
             for (int j = 0; j < 8; ++j)
-              if (fr_c + j < d)
-                from_f32(out + j, o[j] * inv * nw[j] * act_silu(to_f32(p.gate[t * p.ldg + size_t(h) * d + fr_c + j])));
+              if (fr_c + j < dv)
+                from_f32(out + j, o[j] * inv * nw[j] * out_gate<KIND>(to_f32(p.gate[t * p.ldg + size_t(h) * dv + fr_c + j])));
           }
         }
       }
@@ -615,30 +792,38 @@ __global__ void __launch_bounds__(MixCfg<D>::kThreads, sizeof(T) == 2 ? MixCfg<D
       a[0][j] = f.x;
       a[1][j] = f.y;
     }
+    const float2 nn = unpack2(N[MEMORY ? i : 0]);
 #pragma unroll
     for (int e = 0; e < 2; ++e) {
       const int key = kg * KT + 2 * i + e;
-      if (key >= d) continue;
-      float* row = dst + size_t(key) * d + vg * VT;
+      if (key >= dk) continue;
+      if (MEMORY && vg == 0) dst[size_t(dk) * dv + key] = e ? nn.y : nn.x;
+      float* row = dst + size_t(key) * dv + vg * VT;
 #pragma unroll
       for (int j = 0; j < VT; j += 4) {
         if (s4) {
-          if (vg * VT + j < d) *reinterpret_cast<float4*>(row + j) = *reinterpret_cast<const float4*>(a[e] + j);
+          if (vg * VT + j < dv) *reinterpret_cast<float4*>(row + j) = *reinterpret_cast<const float4*>(a[e] + j);
         } else {
 #pragma unroll
           for (int l = j; l < j + 4; ++l)
-            if (vg * VT + l < d) row[l] = a[e][l];
+            if (vg * VT + l < dv) row[l] = a[e][l];
         }
       }
     }
   }
-  if (!OUT && tid < d) p.ws_p[(size_t(blockIdx.x) * p.H + h) * d + tid] = prod;
+  if (!OUT) {
+#pragma unroll
+    for (int i = 0; i < PR; ++i) {
+      const int c = i * NT + tid;
+      if (c < dk) p.ws_p[(size_t(blockIdx.x) * p.H + h) * dk + c] = prod[i];
+    }
+  }
 }
 
-// (B): the state every segment starts from, in the place of what it adds.  One CTA per (sequence, head, part of the matrix).
-template <typename T>
-__global__ void __launch_bounds__(256) time_mix_chain_kernel(const MixParams<T> p) {
-  const int seq = blockIdx.x, h = blockIdx.y, d = p.d;
+// (B): the state every segment starts from, in the place of what it adds.  One CTA per (sequence, head, part of the record).
+template <typename T, int KIND>
+__global__ void __launch_bounds__(256) matrix_chain_kernel(const MixParams<T> p) {
+  const int seq = blockIdx.x, h = blockIdx.y, dk = p.dk;
   const int len = p.q.q_cu[seq + 1] - p.q.q_cu[seq];
   const int n_seg = len > 1 ? (len + p.L - 1) / p.L : 0;
   if (n_seg < 2) return;
@@ -655,15 +840,15 @@ __global__ void __launch_bounds__(256) time_mix_chain_kernel(const MixParams<T> 
     for (int o = 16; o > 0; o >>= 1) base += __shfl_xor_sync(0xffffffffu, base, o);
   }
   const bool cont = p.q.kv_lens[seq] > len;
-  const int mat = d * d;
+  const int mat = int(record_size<KIND>(p)), cells = dk * p.dv;
   const float* rec = p.state + (size_t(slot) * p.H + h) * mat;
   const size_t step = size_t(p.H) * mat;
   for (int e = blockIdx.z * blockDim.x + threadIdx.x; e < mat; e += gridDim.z * blockDim.x) {
     float s = cont ? rec[e] : 0.f;
     float* ws = p.ws_s + (size_t(base) * p.H + h) * mat + e;
-    const float* pr = p.ws_p + (size_t(base) * p.H + h) * d + e / d;
+    const float* pr = p.ws_p + (size_t(base) * p.H + h) * dk + (KIND == MIX_MEMORY && e >= cells ? e - cells : e / p.dv);
     constexpr int kGroup = 8;
-    const size_t pstep = size_t(p.H) * d;
+    const size_t pstep = size_t(p.H) * dk;
     for (int g = 0; g < n_seg; g += kGroup) {              // the last segment only takes its start
       float add[kGroup], f[kGroup];
 #pragma unroll
@@ -684,54 +869,79 @@ __global__ void __launch_bounds__(256) time_mix_chain_kernel(const MixParams<T> 
   }
 }
 
-// Single rows: the head's matrix (d a multiple of 4) passes through registers once.
-constexpr int kMixThreads = 128;
+// Factors of one token of a matrix memory whose state comes from the records.
+struct TokenGates { float f, i, least, m; };
 template <typename T>
-__global__ void __launch_bounds__(kMixThreads) time_mix_single_kernel(const MixParams<T> p) {
+__device__ __forceinline__ TokenGates token_gates(const MixParams<T>& p, size_t t, int h, float m) {
+  const float2 g = log_gates(p, t, h);
+  const float m_new = fmaxf(g.y + m, g.x);
+  return {decay_exp<T>(g.y + m - m_new), __expf(g.x - m_new), __expf(-m_new), m_new};
+}
+
+// Single rows: the head's matrix (dv a multiple of 4) passes through registers once.
+constexpr int kMixThreads = 128;
+template <typename T, int KIND>
+__global__ void __launch_bounds__(kMixThreads) matrix_single_kernel(const MixParams<T> p) {
+  constexpr bool BONUS = KIND == MIX_BONUS, MEMORY = KIND == MIX_MEMORY;
   extern __shared__ __align__(16) float sm[];
-  const int seq = blockIdx.x, h = blockIdx.y, d = p.d, tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
+  const int seq = blockIdx.x, h = blockIdx.y, dk = p.dk, dv = p.dv, tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
   const int t = p.q.q_cu[seq], len = p.q.q_cu[seq + 1] - t;
   if (len != 1) return;
   const int slot = record_of(p.q, seq);
   if (slot < 0) return;
   const bool cont = p.q.kv_lens[seq] > 1;
-  const int quads = d / 4, groups = kMixThreads / quads;    // threads over value quads, then over keys
+  const int quads = dv / 4, groups = kMixThreads / quads;   // threads over value quads, then over keys
   const int vq = tid % quads, kq = tid / quads;
-  float *sR = sm, *sK = sR + d, *sW = sK + d, *sV = sW + d, *sO = sV + d;      // sO [groups][d]
+  float *sV = sm, *sO = sV + dv, *sR = sO + groups * dv, *sK = sR + dk, *sW = sK + dk;      // sO [groups][dv]
   __shared__ float red[2][kMixThreads / 32];
-  float4* rec = reinterpret_cast<float4*>(p.state + (size_t(slot) * p.H + h) * size_t(d) * d);
+  const size_t mat = record_size<KIND>(p);
+  float* rec0 = p.state + (size_t(slot) * p.H + h) * mat;
+  float4* rec = reinterpret_cast<float4*>(rec0);
   constexpr int kAhead = 8;
   float4 s[kAhead];
   const bool mine = kq < groups;
   if (mine && cont) {                                       // the first keys are on their way while the row is prepared
 #pragma unroll
     for (int i = 0; i < kAhead; ++i)
-      if (kq + i * groups < d) s[i] = rec[size_t(kq + i * groups) * quads + vq];
+      if (kq + i * groups < dk) s[i] = rec[size_t(kq + i * groups) * quads + vq];
   }
-  float bonus = 0.f;
-  for (int c = tid; c < d; c += kMixThreads) {
-    const size_t at = size_t(t) * p.ld + size_t(h) * d + c;
-    const float r = to_f32(p.r[at]), k = to_f32(p.k[at]);
+  TokenGates g = {};
+  if (MEMORY) g = token_gates(p, t, h, cont ? p.top[size_t(slot) * p.H + h] : 0.f);
+  float dot = 0.f;                                          // MIX_BONUS: product with the current token; MIX_MEMORY: n q
+  for (int c = tid; c < dk; c += kMixThreads) {
+    const size_t at = size_t(t) * p.ld + size_t(h) * dk + c;
+    float r = to_f32(p.r[at]), k = to_f32(p.k[at]);
+    if (MEMORY) {
+      k *= g.i;
+      r *= p.q_scale;
+      const float nn = fmaf(g.f, cont ? rec0[size_t(dk) * dv + c] : 0.f, k);
+      rec0[size_t(dk) * dv + c] = nn;
+      dot = fmaf(nn, r, dot);
+      sW[c] = g.f;
+    } else {
+      sW[c] = decay_of<KIND>(p, p.z[size_t(t) * p.H * dk + size_t(h) * dk + c] + p.w0[h * dk + c]);
+      if (BONUS) dot += r * p.u[h * dk + c] * k;
+      else r *= p.q_scale;
+    }
     sR[c] = r;
     sK[c] = k;
-    sV[c] = to_f32(p.v[at]);
-    sW[c] = decay_of<T>(p.z[size_t(t) * p.H * d + size_t(h) * d + c] + p.w0[h * d + c]);
-    bonus += r * p.u[h * d + c] * k;
   }
-  bonus = warp_sum(bonus);
-  if (lane == 0) red[0][warp] = bonus;
+  for (int c = tid; c < dv; c += kMixThreads) sV[c] = to_f32(p.v[size_t(t) * p.ld + size_t(h) * dv + c]);
+  dot = warp_sum(dot);
+  if (lane == 0) red[0][warp] = dot;
   __syncthreads();
-  bonus = 0.f;
+  dot = 0.f;
 #pragma unroll
-  for (int i = 0; i < kMixThreads / 32; ++i) bonus += red[0][i];
+  for (int i = 0; i < kMixThreads / 32; ++i) dot += red[0][i];
+  if (MEMORY && tid == 0) p.top[size_t(slot) * p.H + h] = g.m;      // every thread has read the old one
   if (mine) {
     const float4 v = *reinterpret_cast<const float4*>(sV + vq * 4);
     float4 o = make_float4(0.f, 0.f, 0.f, 0.f);
-    for (int k0 = kq; k0 < d; k0 += kAhead * groups) {
+    for (int k0 = kq; k0 < dk; k0 += kAhead * groups) {
 #pragma unroll
       for (int i = 0; i < kAhead; ++i) {
         const int key = k0 + i * groups;
-        if (key < d) {
+        if (key < dk) {
           if (!cont) s[i] = make_float4(0.f, 0.f, 0.f, 0.f);
           else if (k0 != kq) s[i] = rec[size_t(key) * quads + vq];
         }
@@ -739,21 +949,24 @@ __global__ void __launch_bounds__(kMixThreads) time_mix_single_kernel(const MixP
 #pragma unroll
       for (int i = 0; i < kAhead; ++i) {
         const int key = k0 + i * groups;
-        if (key < d) {
+        if (key < dk) {
           const float r = sR[key], k = sK[key], w = sW[key];
-          o.x = fmaf(r, s[i].x, o.x); o.y = fmaf(r, s[i].y, o.y); o.z = fmaf(r, s[i].z, o.z); o.w = fmaf(r, s[i].w, o.w);
-          rec[size_t(key) * quads + vq] = make_float4(fmaf(w, s[i].x, k * v.x), fmaf(w, s[i].y, k * v.y), fmaf(w, s[i].z, k * v.z),
-                                                      fmaf(w, s[i].w, k * v.w));
+          const float4 a = make_float4(fmaf(w, s[i].x, k * v.x), fmaf(w, s[i].y, k * v.y), fmaf(w, s[i].z, k * v.z), fmaf(w, s[i].w, k * v.w));
+          const float4 c = BONUS ? s[i] : a;
+          o.x = fmaf(r, c.x, o.x); o.y = fmaf(r, c.y, o.y); o.z = fmaf(r, c.z, o.z); o.w = fmaf(r, c.w, o.w);
+          rec[size_t(key) * quads + vq] = a;
         }
       }
     }
-    *reinterpret_cast<float4*>(sO + kq * d + vq * 4) = o;
+    *reinterpret_cast<float4*>(sO + kq * dv + vq * 4) = o;
   }
   __syncthreads();
+  const float whole = MEMORY ? 1.f / (fmaxf(fabsf(dot), g.least) + kMemoryEps) : 1.f;
   float ss = 0.f;
-  for (int c = tid; c < d; c += kMixThreads) {
-    float o = bonus * sV[c];
-    for (int g = 0; g < groups; ++g) o += sO[g * d + c];
+  for (int c = tid; c < dv; c += kMixThreads) {
+    float o = BONUS ? dot * sV[c] : 0.f;
+    for (int i = 0; i < groups; ++i) o += sO[i * dv + c];
+    if (MEMORY) o *= whole;
     sO[c] = o;                                              // only this thread reads or writes column c from here on
     ss += o * o;
   }
@@ -763,49 +976,64 @@ __global__ void __launch_bounds__(kMixThreads) time_mix_single_kernel(const MixP
   ss = 0.f;
 #pragma unroll
   for (int i = 0; i < kMixThreads / 32; ++i) ss += red[1][i];
-  const float inv = rsqrtf(ss / float(d) + p.eps) * p.scale;
-  for (int c = tid; c < d; c += kMixThreads)
-    from_f32(p.out + size_t(t) * p.ldo + size_t(h) * d + c,
-             sO[c] * inv * to_f32(p.norm_w[h * d + c]) * act_silu(to_f32(p.gate[size_t(t) * p.ldg + size_t(h) * d + c])));
+  const float inv = rsqrtf(ss / float(dv) + p.eps) * p.scale;
+  for (int c = tid; c < dv; c += kMixThreads)
+    from_f32(p.out + size_t(t) * p.ldo + size_t(h) * dv + c,
+             sO[c] * inv * to_f32(p.norm_w[h * p.norm_step + c]) * out_gate<KIND>(to_f32(p.gate[size_t(t) * p.ldg + size_t(h) * dv + c])));
 }
 
-// Any head dimension, any number of rows: the state stays in memory, one thread per value column.
-template <typename T>
-__global__ void __launch_bounds__(256) time_mix_any_kernel(const MixParams<T> p, int min_len, int max_len) {
+// Any head sizes, any number of rows: the state stays in memory, one thread per value column.
+template <typename T, int KIND>
+__global__ void __launch_bounds__(256) matrix_any_kernel(const MixParams<T> p, int min_len, int max_len) {
+  constexpr bool BONUS = KIND == MIX_BONUS, MEMORY = KIND == MIX_MEMORY;
   extern __shared__ __align__(16) float sm[];
-  const int seq = blockIdx.x, h = blockIdx.y, d = p.d, tid = threadIdx.x;
+  const int seq = blockIdx.x, h = blockIdx.y, dk = p.dk, dv = p.dv, tid = threadIdx.x;
   const int start = p.q.q_cu[seq], len = p.q.q_cu[seq + 1] - start;
   if (len < min_len || len > max_len || len < 1) return;
   const int slot = record_of(p.q, seq);
   if (slot < 0) return;
   bool fresh = p.q.kv_lens[seq] == len;
-  float *sR = sm, *sK = sR + d, *sW = sK + d, *sO = sW + d;
+  float *sR = sm, *sK = sR + dk, *sW = sK + dk, *sO = sW + dk;
   __shared__ float red[2][8];
-  float* rec = p.state + (size_t(slot) * p.H + h) * size_t(d) * d;
+  float* rec = p.state + (size_t(slot) * p.H + h) * record_size<KIND>(p);
+  const size_t plane = size_t(p.H) * p.rows;
   for (int t = start; t < start + len; ++t) {
-    float bonus = 0.f;
-    for (int c = tid; c < d; c += 256) {
-      const size_t at = size_t(t) * p.ld + size_t(h) * d + c;
-      const float r = to_f32(p.r[at]), k = to_f32(p.k[at]);
+    const float* fi = MEMORY ? p.fi + size_t(h) * p.rows + t : nullptr;
+    float dot = 0.f;
+    for (int c = tid; c < dk; c += 256) {
+      const size_t at = size_t(t) * p.ld + size_t(h) * dk + c;
+      float r = to_f32(p.r[at]), k = to_f32(p.k[at]);
+      if (MEMORY) {
+        k *= fi[plane];
+        r *= p.q_scale;
+        float* nn = rec + size_t(dk) * dv + c;
+        *nn = fmaf(fi[0], fresh ? 0.f : *nn, k);
+        dot = fmaf(*nn, r, dot);
+        sW[c] = fi[0];
+      } else {
+        sW[c] = decay_of<KIND>(p, p.z[size_t(t) * p.H * dk + size_t(h) * dk + c] + p.w0[h * dk + c]);
+        if (BONUS) dot += r * p.u[h * dk + c] * k;
+        else r *= p.q_scale;
+      }
       sR[c] = r;
       sK[c] = k;
-      sW[c] = decay_of<T>(p.z[size_t(t) * p.H * d + size_t(h) * d + c] + p.w0[h * d + c]);
-      bonus += r * p.u[h * d + c] * k;
     }
-    bonus = warp_sum(bonus);
-    if ((tid & 31) == 0) red[0][tid >> 5] = bonus;
+    dot = warp_sum(dot);
+    if ((tid & 31) == 0) red[0][tid >> 5] = dot;
     __syncthreads();
-    bonus = 0.f;
-    for (int i = 0; i < 8; ++i) bonus += red[0][i];
+    dot = 0.f;
+    for (int i = 0; i < 8; ++i) dot += red[0][i];
+    const float whole = MEMORY ? 1.f / (fmaxf(fabsf(dot), fi[2 * plane]) + kMemoryEps) : 1.f;
     float ss = 0.f;
-    for (int c = tid; c < d; c += 256) {
-      const float v = to_f32(p.v[size_t(t) * p.ld + size_t(h) * d + c]);
-      float o = bonus * v;
-      for (int k = 0; k < d; ++k) {
-        const float s = fresh ? 0.f : rec[size_t(k) * d + c];
-        o = fmaf(sR[k], s, o);
-        rec[size_t(k) * d + c] = fmaf(sW[k], s, sK[k] * v);
+    for (int c = tid; c < dv; c += 256) {
+      const float v = to_f32(p.v[size_t(t) * p.ld + size_t(h) * dv + c]);
+      float o = BONUS ? dot * v : 0.f;
+      for (int k = 0; k < dk; ++k) {
+        const float s = fresh ? 0.f : rec[size_t(k) * dv + c], a = fmaf(sW[k], s, sK[k] * v);
+        o = fmaf(sR[k], BONUS ? s : a, o);
+        rec[size_t(k) * dv + c] = a;
       }
+      if (MEMORY) o *= whole;
       sO[c] = o;
       ss += o * o;
     }
@@ -814,45 +1042,63 @@ __global__ void __launch_bounds__(256) time_mix_any_kernel(const MixParams<T> p,
     __syncthreads();
     ss = 0.f;
     for (int i = 0; i < 8; ++i) ss += red[1][i];
-    const float inv = rsqrtf(ss / float(d) + p.eps) * p.scale;
-    for (int c = tid; c < d; c += 256)
-      from_f32(p.out + size_t(t) * p.ldo + size_t(h) * d + c,
-               sO[c] * inv * to_f32(p.norm_w[h * d + c]) * act_silu(to_f32(p.gate[size_t(t) * p.ldg + size_t(h) * d + c])));
+    const float inv = rsqrtf(ss / float(dv) + p.eps) * p.scale;
+    for (int c = tid; c < dv; c += 256)
+      from_f32(p.out + size_t(t) * p.ldo + size_t(h) * dv + c,
+               sO[c] * inv * to_f32(p.norm_w[h * p.norm_step + c]) * out_gate<KIND>(to_f32(p.gate[size_t(t) * p.ldg + size_t(h) * dv + c])));
     fresh = false;
   }
 }
 
-template <typename T>
-static int launch_time_mix(MixParams<T> p, int seg_cap, int has_long, int has_single, cudaStream_t st) {
-  const int d = p.d;
-  const bool v8 = d % 8 == 0 && p.ld % 8 == 0 &&
+template <typename T, int KIND, int DK, int DV>
+static int launch_segments(const MixParams<T>& p, int seg_cap, int v8, int g8, int s4, cudaStream_t st) {
+  using C = MixCfg<DK, DV>;
+  const dim3 grid(seg_cap, p.H);
+  if (p.ws_s) {
+    matrix_segment_kernel<T, DK, DV, KIND, false><<<grid, C::kThreads, 0, st>>>(p, v8, g8, s4);
+    const int parts = (p.dk * p.dv + 255) / 256;
+    matrix_chain_kernel<T, KIND><<<dim3(p.q.n, p.H, parts), 256, 0, st>>>(p);
+  }
+  matrix_segment_kernel<T, DK, DV, KIND, true><<<grid, C::kThreads, 0, st>>>(p, v8, g8, s4);
+  return cudaGetLastError() == cudaSuccess ? 0 : -1;
+}
+
+template <typename T, int KIND>
+static int launch_matrix(MixParams<T> p, int seg_cap, int has_long, int has_single, cudaStream_t st) {
+  const int dk = p.dk, dv = p.dv;
+  const bool v8 = dk % 8 == 0 && dv % 8 == 0 && p.ld % 8 == 0 &&
                   !((reinterpret_cast<uintptr_t>(p.r) | reinterpret_cast<uintptr_t>(p.k) | reinterpret_cast<uintptr_t>(p.v) |
                      reinterpret_cast<uintptr_t>(p.z) | reinterpret_cast<uintptr_t>(p.w0)) & 15);
-  const bool g8 = d % 8 == 0 && p.ldg % 8 == 0 && p.ldo % 8 == 0 &&
+  const bool g8 = dv % 8 == 0 && p.ldg % 8 == 0 && p.ldo % 8 == 0 &&
                   !((reinterpret_cast<uintptr_t>(p.gate) | reinterpret_cast<uintptr_t>(p.out)) & 15);
-  const bool s4 = d % 4 == 0;
+  const bool s4 = dv % 4 == 0 && (KIND != MIX_MEMORY || dk % 4 == 0);
+  const bool regs = dv % 4 == 0 && dv <= 4 * kMixThreads && s4;       // single rows through registers
+  const bool tiles = dk <= 128 && dv <= 128;                          // longer portions in segments
+  if (KIND == MIX_MEMORY && (has_long || !regs))
+    memory_gates_kernel<T><<<dim3(p.q.n, (p.H + 3) / 4), 128, 0, st>>>(p, regs ? 2 : 1);
+  const size_t any_smem = (size_t(3) * dk + dv) * sizeof(float);
+  const dim3 by_seq(p.q.n, p.H);
   if (has_single) {
-    const dim3 grid(p.q.n, p.H);
-    if (s4 && d <= 4 * kMixThreads) {
-      const int groups = kMixThreads / (d / 4);
-      time_mix_single_kernel<T><<<grid, kMixThreads, size_t(4 + groups) * d * sizeof(float), st>>>(p);
-    } else {
-      time_mix_any_kernel<T><<<grid, 256, size_t(4) * d * sizeof(float), st>>>(p, 1, 1);
-    }
+    const int groups = regs ? kMixThreads / (dv / 4) : 0;
+    if (regs) matrix_single_kernel<T, KIND><<<by_seq, kMixThreads, (size_t(3) * dk + size_t(1 + groups) * dv) * sizeof(float), st>>>(p);
+    else matrix_any_kernel<T, KIND><<<by_seq, 256, any_smem, st>>>(p, 1, 1);
   }
   if (has_long) {
-    if (d <= 128) {
-      const dim3 grid(seg_cap, p.H);
-#define XL_MIX(D, OUT) time_mix_segment_kernel<T, D, OUT><<<grid, MixCfg<D>::kThreads, 0, st>>>(p, v8, g8, s4)
-      if (p.ws_s) {
-        if (d <= 32) XL_MIX(32, false); else if (d <= 64) XL_MIX(64, false); else XL_MIX(128, false);
-        const int parts = (d * d + 255) / 256;
-        time_mix_chain_kernel<T><<<dim3(p.q.n, p.H, parts), 256, 0, st>>>(p);
-      }
-      if (d <= 32) XL_MIX(32, true); else if (d <= 64) XL_MIX(64, true); else XL_MIX(128, true);
-#undef XL_MIX
+    if (!tiles) {
+      matrix_any_kernel<T, KIND><<<by_seq, 256, any_smem, st>>>(p, 2, 1 << 30);
     } else {
-      time_mix_any_kernel<T><<<dim3(p.q.n, p.H), 256, size_t(4) * d * sizeof(float), st>>>(p, 2, 1 << 30);
+#define XL_MIX(DK, DV) return launch_segments<T, KIND, DK, DV>(p, seg_cap, v8, g8, s4, st)
+      if (KIND == MIX_BONUS) {                                         // keys and values of one size
+        if (dk <= 32) XL_MIX(32, 32);
+        if (dk <= 64) XL_MIX(64, 64);
+        XL_MIX(128, 128);
+      }
+      if (dk <= 32) { if (dv <= 32) XL_MIX(32, 32); if (dv <= 64) XL_MIX(32, 64); XL_MIX(32, 128); }
+      if (dk <= 64) { if (dv <= 32) XL_MIX(64, 32); if (dv <= 64) XL_MIX(64, 64); XL_MIX(64, 128); }
+      if (dv <= 32) XL_MIX(128, 32);
+      if (dv <= 64) XL_MIX(128, 64);
+      XL_MIX(128, 128);
+#undef XL_MIX
     }
   }
   return cudaGetLastError() == cudaSuccess ? 0 : -1;
@@ -1238,14 +1484,16 @@ XL_API int xl_token_shift(const void* h, const void* mu, void* last, void* out, 
   });
 }
 
-// out [rows, C] = silu(bias + causal convolution of x (row pitch ldx) with w [taps, C]); state [n_slots, taps - 1, C]
-XL_API int xl_conv_silu(const void* x, const void* w, const void* bias, void* state, void* out, const void* token_seq, const void* q_cu,
-                        const void* kv_lens, const void* slots, int n_seqs, int n_slots, int rows, int C, int taps, long ldx,
-                        int has_long, int f32, void* stream) {
+// out [rows, C] = act(bias + causal convolution of x (row pitch ldx) with w [taps, C]) (+ x); bias may be null; act: silu or none;
+// state [n_slots, taps - 1, C]
+XL_API int xl_causal_conv(const void* x, const void* w, const void* bias, void* state, void* out, const void* token_seq, const void* q_cu,
+                          const void* kv_lens, const void* slots, int n_seqs, int n_slots, int rows, int C, int taps, long ldx,
+                          int has_long, int silu, int residual, int f32, void* stream) {
   if (rows <= 0) return 0;
   if (taps < 1) return -2;
   cudaStream_t st = static_cast<cudaStream_t>(stream);
   const Seqs q = make_seqs(q_cu, kv_lens, slots, n_seqs, n_slots);
+  const ConvOut act{silu, residual};
   return by_type(f32, [&](auto* tag) {
     using T = std::remove_pointer_t<decltype(tag)>;
     const T *xx = static_cast<const T*>(x), *ww = static_cast<const T*>(w), *b = static_cast<const T*>(bias);
@@ -1256,8 +1504,8 @@ XL_API int xl_conv_silu(const void* x, const void* w, const void* bias, void* st
     const int tile = has_long ? kConvRows : kConvRowsSingle;
     const dim3 grid((rows + tile - 1) / tile, cols);
 #define XL_CONV(V, TAPS)                                                                                              \
-  if (has_long) conv_silu_kernel<T, V, TAPS, kConvRows><<<grid, 128, 0, st>>>(xx, ww, b, s, o, ts, q, rows, C, taps, ldx); \
-  else conv_silu_kernel<T, V, TAPS, kConvRowsSingle><<<grid, 128, 0, st>>>(xx, ww, b, s, o, ts, q, rows, C, taps, ldx)
+  if (has_long) causal_conv_kernel<T, V, TAPS, kConvRows><<<grid, 128, 0, st>>>(xx, ww, b, s, o, ts, q, rows, C, taps, ldx, act); \
+  else causal_conv_kernel<T, V, TAPS, kConvRowsSingle><<<grid, 128, 0, st>>>(xx, ww, b, s, o, ts, q, rows, C, taps, ldx, act)
     if (vec) {
       if (taps == 4) { XL_CONV(8, 4); } else if (taps == 3) { XL_CONV(8, 3); } else if (taps == 2) { XL_CONV(8, 2); } else { XL_CONV(8, 0); }
     } else {
@@ -1272,28 +1520,75 @@ XL_API int xl_conv_silu(const void* x, const void* w, const void* bias, void* st
   });
 }
 
-// r, k, v [rows, H * d] with row pitch ld, gate with ldg, z [rows, H * d] fp32 dense; state [n_slots, H, d, d] fp32; out with
+// What the matrix-state entry points share: r (queries) and k [rows, H * dk], v [rows, H * dv] with row pitch ld, gate with ldg; out with
 // row pitch ldo.  Longer portions in segments of L rows, at most seg_cap of them; ws_s / ws_p (null when no portion has more
-// than L rows) hold seg_cap * H * d * d and seg_cap * H * d floats.
+// than L rows) hold seg_cap * H records and seg_cap * H * dk floats.
+struct MatrixArgs {
+  const void *r, *k, *v, *z, *w0, *u, *gate, *norm_w;
+  float scale, eps;
+  void *state, *out;
+  const void *q_cu, *kv_lens, *slots;
+  int n_seqs, n_slots, H, dk, dv, norm_step;
+  long ld, ldg, ldo;
+  int L, seg_cap;
+  void *ws_s, *ws_p;
+  int has_long, has_single, f32;
+  void* stream;
+  float inv_tau, cap;
+  void *top, *fi;
+  int rows;
+};
+template <int KIND>
+static int run_matrix(const MatrixArgs& a) {
+  if (a.n_seqs <= 0) return 0;
+  if (a.H < 1 || a.H > 65535 || a.dk < 1 || a.dk > 2048 || a.dv < 1 || a.dv > 2048 || a.L < 2) return -2;
+  return by_type(a.f32, [&](auto* tag) {
+    using T = std::remove_pointer_t<decltype(tag)>;
+    MixParams<T> p = {};
+    p.r = static_cast<const T*>(a.r); p.k = static_cast<const T*>(a.k); p.v = static_cast<const T*>(a.v);
+    p.gate = static_cast<const T*>(a.gate);
+    p.z = static_cast<const float*>(a.z); p.w0 = static_cast<const float*>(a.w0); p.u = static_cast<const float*>(a.u);
+    p.norm_w = static_cast<const T*>(a.norm_w); p.norm_step = a.norm_step;
+    p.state = static_cast<float*>(a.state); p.out = static_cast<T*>(a.out);
+    p.ld = a.ld; p.ldg = a.ldg; p.ldo = a.ldo; p.H = a.H; p.dk = a.dk; p.dv = a.dv; p.scale = a.scale; p.eps = a.eps;
+    p.q_scale = 1.f / sqrtf(float(a.dk)); p.inv_tau = a.inv_tau; p.cap = a.cap;
+    p.top = static_cast<float*>(a.top); p.fi = static_cast<float*>(a.fi); p.rows = a.rows;
+    p.q = make_seqs(a.q_cu, a.kv_lens, a.slots, a.n_seqs, a.n_slots);
+    p.L = a.L; p.ws_s = static_cast<float*>(a.ws_s); p.ws_p = static_cast<float*>(a.ws_p);
+    return launch_matrix<T, KIND>(p, a.seg_cap, a.has_long, a.has_single, static_cast<cudaStream_t>(a.stream));
+  });
+}
+
+// Time mixing: z [rows, H * d] fp32 dense; state [n_slots, H, d, d] fp32.
 XL_API int xl_time_mix(const void* r, const void* k, const void* v, const void* z, const void* w0, const void* u, const void* gate,
                        const void* norm_w, float scale, float eps, void* state, void* out, const void* q_cu, const void* kv_lens,
                        const void* slots, int n_seqs, int n_slots, int H, int d, long ld, long ldg, long ldo, int L, int seg_cap,
                        void* ws_s, void* ws_p, int has_long, int has_single, int f32, void* stream) {
-  if (n_seqs <= 0) return 0;
-  if (H < 1 || H > 65535 || d < 1 || d > 2048 || L < 2) return -2;
-  return by_type(f32, [&](auto* tag) {
-    using T = std::remove_pointer_t<decltype(tag)>;
-    MixParams<T> p;
-    p.r = static_cast<const T*>(r); p.k = static_cast<const T*>(k); p.v = static_cast<const T*>(v);
-    p.gate = static_cast<const T*>(gate);
-    p.z = static_cast<const float*>(z); p.w0 = static_cast<const float*>(w0); p.u = static_cast<const float*>(u);
-    p.norm_w = static_cast<const T*>(norm_w);
-    p.state = static_cast<float*>(state); p.out = static_cast<T*>(out);
-    p.ld = ld; p.ldg = ldg; p.ldo = ldo; p.H = H; p.d = d; p.scale = scale; p.eps = eps;
-    p.q = make_seqs(q_cu, kv_lens, slots, n_seqs, n_slots);
-    p.L = L; p.ws_s = static_cast<float*>(ws_s); p.ws_p = static_cast<float*>(ws_p);
-    return launch_time_mix<T>(p, seg_cap, has_long, has_single, static_cast<cudaStream_t>(stream));
-  });
+  return run_matrix<MIX_BONUS>(MatrixArgs{r, k, v, z, w0, u, gate, norm_w, scale, eps, state, out, q_cu, kv_lens, slots, n_seqs, n_slots, H, d,
+                                          d, d, ld, ldg, ldo, L, seg_cap, ws_s, ws_p, has_long, has_single, f32, stream, 0.f, 0.f, nullptr,
+                                          nullptr, 0});
+}
+
+// Gated linear attention: z [rows, H * dk] fp32 dense, decay sigmoid(z + bias)^inv_tau; state [n_slots, H, dk, dv] fp32; norm_w [dv].
+XL_API int xl_gated_memory(const void* q, const void* k, const void* v, const void* z, const void* bias, float inv_tau, const void* gate,
+                           const void* norm_w, float eps, void* state, void* out, const void* q_cu, const void* kv_lens, const void* slots,
+                           int n_seqs, int n_slots, int H, int dk, int dv, long ld, long ldg, long ldo, int L, int seg_cap, void* ws_s,
+                           void* ws_p, int has_long, int has_single, int f32, void* stream) {
+  return run_matrix<MIX_GATED>(MatrixArgs{q, k, v, z, bias, nullptr, gate, norm_w, 1.f, eps, state, out, q_cu, kv_lens, slots, n_seqs, n_slots,
+                                          H, dk, dv, 0, ld, ldg, ldo, L, seg_cap, ws_s, ws_p, has_long, has_single, f32, stream, inv_tau,
+                                          0.f, nullptr, nullptr, 0});
+}
+
+// Matrix memory: gates [rows, 2 H] fp32 dense ahead of bias [2 H] and the bound `cap`; state [n_slots, H, dk * dv + dk] fp32, top
+// [n_slots, H] fp32; norm_w [H * dv]; fi: 3 * H * rows floats of workspace.
+XL_API int xl_matrix_memory(const void* q, const void* k, const void* v, const void* gates, const void* bias, float cap, const void* gate,
+                            const void* norm_w, float eps, void* state, void* top, void* out, const void* q_cu, const void* kv_lens,
+                            const void* slots, int n_seqs, int n_slots, int H, int dk, int dv, long ld, long ldg, long ldo, int L, int seg_cap,
+                            void* ws_s, void* ws_p, void* fi, int rows, int has_long, int has_single, int f32, void* stream) {
+  if (!fi || cap <= 0.f) return -2;
+  return run_matrix<MIX_MEMORY>(MatrixArgs{q, k, v, gates, bias, nullptr, gate, norm_w, 1.f, eps, state, out, q_cu, kv_lens, slots, n_seqs,
+                                           n_slots, H, dk, dv, dv, ld, ldg, ldo, L, seg_cap, ws_s, ws_p, has_long, has_single, f32, stream, 0.f,
+                                           cap, top, fi, rows});
 }
 
 // out [rows, C] = (scan + D x) silu(z); B, Cm with row pitch ldb, z with ldz; state [n_slots, C, N] fp32

@@ -6,7 +6,8 @@
 //   SRC_ROWS   y is a tensor (the output of o_proj / down_proj);
 //   SRC_MOE    y is assembled here: weighted sum of the chosen experts' rows, identity experts (whose output is the
 //              sublayer's input itself, times the weight) and a shared expert, so that it never exists in memory;
-//   SRC_EMBED  there is no y: x = table[token] * scale starts the residual stream;
+//   SRC_PAIR   y is put together here from two branches, each normed with a weight of its own;
+//   SRC_EMBED  there is no y: x = table[token] * scale (normed itself if w_post is given) starts the residual stream;
 // and of decoders whose sublayers are normed before only:
 //   SRC_ADD    x += scale * y                                    (no norm behind the sublayer)
 //   SRC_SET    x = y + vec, y in fp32                            (the residual is replaced by a product of itself)
@@ -27,7 +28,7 @@
 namespace xl_sn {
 using namespace xl;
 
-enum { SRC_ROWS = 0, SRC_MOE = 1, SRC_EMBED = 2, SRC_ADD = 3, SRC_SET = 4 };
+enum { SRC_ROWS = 0, SRC_MOE = 1, SRC_EMBED = 2, SRC_ADD = 3, SRC_SET = 4, SRC_PAIR = 5 };
 
 template <typename T>
 struct NormParams {
@@ -37,7 +38,8 @@ struct NormParams {
   T* h;                      // [rows, H] its output
   int H;
   float eps;
-  const T* y;                // SRC_ROWS: [rows, H]
+  const T* y;                // SRC_ROWS, SRC_PAIR: [rows, H]
+  const T *y2, *w_y, *w_y2;  // SRC_PAIR: y = scale * (rms(y) w_y + rms(y2) w_y2)
   // SRC_MOE
   const T* y_exp;            // [*, H] expert outputs, row dst_of[t * k + j] belongs to choice j of token t (-1: none)
   const int* dst_of;
@@ -50,7 +52,7 @@ struct NormParams {
   const int* tokens;
   const T* table;            // [V, H]
   int V;
-  float scale;               // also SRC_ADD
+  float scale;               // also SRC_ADD, SRC_PAIR
   // SRC_SET
   const float* y32;          // [rows, H]
   const float* vec;          // [H]
@@ -74,6 +76,24 @@ __device__ __forceinline__ float block_sum(float v, float* red) {
   float t = 0.f;
   const int warps = (blockDim.x + 31) >> 5;
   for (int i = 0; i < warps; ++i) t += red[i];
+  return t;
+}
+
+// the same for two values; `red` holds two floats per warp
+__device__ __forceinline__ float2 block_sum2(float a, float b, float* red) {
+  a = warp_sum(a);
+  b = warp_sum(b);
+  if ((threadIdx.x & 31) == 0) {
+    red[threadIdx.x >> 5] = a;
+    red[8 + (threadIdx.x >> 5)] = b;
+  }
+  __syncthreads();
+  float2 t = make_float2(0.f, 0.f);
+  const int warps = (blockDim.x + 31) >> 5;
+  for (int i = 0; i < warps; ++i) {
+    t.x += red[i];
+    t.y += red[8 + i];
+  }
   return t;
 }
 
@@ -101,7 +121,7 @@ __device__ __forceinline__ float embed1(const NormParams<T>& p, int row, int c, 
 // Register-resident rows: thread i owns the 8-element vectors i, i + blockDim, ... (VPT of them).
 template <typename T, int VPT, int SRC>
 __global__ void __launch_bounds__(256) sandwich_norm_kernel(const NormParams<T> p) {
-  __shared__ float red_a[8], red_b[8];
+  __shared__ float red_a[8], red_b[8], red_c[SRC == SRC_PAIR ? 16 : 1];
   const int row = blockIdx.x, H = p.H, nvec = H / 8;
   float y[VPT][8];
   float ss = 0.f;
@@ -110,11 +130,41 @@ __global__ void __launch_bounds__(256) sandwich_norm_kernel(const NormParams<T> 
     for (int j = 0; j < p.k; ++j)
       if (p.ids[row * p.k + j] >= p.first_identity) w_id += p.weights[row * p.k + j];
   }
+  if constexpr (SRC == SRC_PAIR) {
+    float b[VPT][8], sa = 0.f, sb = 0.f;
+#pragma unroll
+    for (int i = 0; i < VPT; ++i) {
+      const int v = threadIdx.x + i * blockDim.x;
+      if (v < nvec) {
+        load8(p.y + size_t(row) * H + v * 8, y[i]);
+        load8(p.y2 + size_t(row) * H + v * 8, b[i]);
+#pragma unroll
+        for (int e = 0; e < 8; ++e) {
+          sa += y[i][e] * y[i][e];
+          sb += b[i][e] * b[i][e];
+        }
+      }
+    }
+    const float2 s = block_sum2(sa, sb, red_c);
+    const float ra = rsqrtf(s.x / float(H) + p.eps) * p.scale, rb = rsqrtf(s.y / float(H) + p.eps) * p.scale;
+#pragma unroll
+    for (int i = 0; i < VPT; ++i) {
+      const int v = threadIdx.x + i * blockDim.x;
+      if (v < nvec) {
+        float wa[8], wb[8];
+        load8(p.w_y + v * 8, wa);
+        load8(p.w_y2 + v * 8, wb);
+#pragma unroll
+        for (int e = 0; e < 8; ++e) y[i][e] = fmaf(y[i][e] * ra, wa[e], b[i][e] * rb * wb[e]);
+      }
+    }
+  }
 #pragma unroll
   for (int i = 0; i < VPT; ++i) {
     const int v = threadIdx.x + i * blockDim.x;
     if (v < nvec) {
-      if (SRC == SRC_ROWS) {
+      if (SRC == SRC_PAIR) {                               // put together above
+      } else if (SRC == SRC_ROWS) {
         load8(p.y + size_t(row) * H + v * 8, y[i]);
       } else if (SRC == SRC_ADD) {
         float x[8], s[8];
@@ -182,16 +232,17 @@ __global__ void __launch_bounds__(256) sandwich_norm_kernel(const NormParams<T> 
       for (int e = 0; e < 8; ++e) ss += y[i][e] * y[i][e];
     }
   }
-  if (SRC == SRC_ROWS || (SRC == SRC_MOE && !p.add_only)) {
+  const bool post = SRC == SRC_ROWS || SRC == SRC_PAIR || (SRC == SRC_MOE && !p.add_only) || (SRC == SRC_EMBED && p.w_post);
+  if (post) {
     const float r_post = rsqrtf(block_sum(ss, red_a) / float(H) + p.eps);
     ss = 0.f;
 #pragma unroll
     for (int i = 0; i < VPT; ++i) {
       const int v = threadIdx.x + i * blockDim.x;
       if (v < nvec) {
-        float w[8], x[8];
+        float w[8], x[8] = {};
         load8(p.w_post + v * 8, w);
-        load8(p.x + size_t(row) * H + v * 8, x);
+        if (SRC != SRC_EMBED) load8(p.x + size_t(row) * H + v * 8, x);
 #pragma unroll
         for (int e = 0; e < 8; ++e) {
           y[i][e] = x[e] + y[i][e] * r_post * w[e];
@@ -219,16 +270,29 @@ __global__ void __launch_bounds__(256) sandwich_norm_kernel(const NormParams<T> 
 template <typename T, int SRC>
 __global__ void __launch_bounds__(256) sandwich_norm_any_kernel(const NormParams<T> p) {
   extern __shared__ float row_cache[];
-  __shared__ float red_a[8], red_b[8];
+  __shared__ float red_a[8], red_b[8], red_c[SRC == SRC_PAIR ? 16 : 1];
   const int row = blockIdx.x, H = p.H;
-  float ss = 0.f, w_id = 0.f;
+  float ss = 0.f, w_id = 0.f, ra = 0.f, rb = 0.f;
+  if constexpr (SRC == SRC_PAIR) {
+    for (int i = threadIdx.x; i < H; i += blockDim.x) {
+      const float a = to_f32(p.y[size_t(row) * H + i]), b = to_f32(p.y2[size_t(row) * H + i]);
+      ra += a * a;
+      rb += b * b;
+    }
+    const float2 s = block_sum2(ra, rb, red_c);
+    ra = rsqrtf(s.x / float(H) + p.eps) * p.scale;
+    rb = rsqrtf(s.y / float(H) + p.eps) * p.scale;
+  }
   if (SRC == SRC_MOE) {
     for (int j = 0; j < p.k; ++j)
       if (p.ids[row * p.k + j] >= p.first_identity) w_id += p.weights[row * p.k + j];
   }
   for (int i = threadIdx.x; i < H; i += blockDim.x) {
     float y = 0.f;
-    if (SRC == SRC_ROWS) {
+    if (SRC == SRC_PAIR) {
+      const size_t at = size_t(row) * H + i;
+      y = fmaf(to_f32(p.y[at]) * ra, to_f32(p.w_y[i]), to_f32(p.y2[at]) * rb * to_f32(p.w_y2[i]));
+    } else if (SRC == SRC_ROWS) {
       y = to_f32(p.y[size_t(row) * H + i]);
     } else if (SRC == SRC_ADD) {
       y = fmaf(p.ls ? to_f32(p.ls[i]) : p.scale, to_f32(p.y[size_t(row) * H + i]), p.x[size_t(row) * H + i]);
@@ -253,11 +317,11 @@ __global__ void __launch_bounds__(256) sandwich_norm_any_kernel(const NormParams
     row_cache[i] = y;
     ss += y * y;
   }
-  if (SRC == SRC_ROWS || (SRC == SRC_MOE && !p.add_only)) {
+  if (SRC == SRC_ROWS || SRC == SRC_PAIR || (SRC == SRC_MOE && !p.add_only) || (SRC == SRC_EMBED && p.w_post)) {
     const float r_post = rsqrtf(block_sum(ss, red_a) / float(H) + p.eps);
     ss = 0.f;
     for (int i = threadIdx.x; i < H; i += blockDim.x) {
-      const float x = p.x[size_t(row) * H + i] + row_cache[i] * r_post * to_f32(p.w_post[i]);
+      const float x = (SRC == SRC_EMBED ? 0.f : p.x[size_t(row) * H + i]) + row_cache[i] * r_post * to_f32(p.w_post[i]);
       row_cache[i] = x;
       ss += x * x;
     }
@@ -501,14 +565,66 @@ static int launch_qknorm(void* qkv, const void* slots, const void* q_w, const vo
 }
 
 // ---------------------------------------------------------------- q / k norm over the whole projection + cache write
-// One row per CTA; rows hold q, k and v (and possibly more behind them) with pitch ld.
-template <typename T, int V>
+// One row per CTA; rows hold q, k and v (and possibly more behind them) with pitch ld.  With a rotation the first rot.dims columns of
+// every head of dk are turned.  With `mix` [n_q, n_q] q leaves as n_q rows of n_k * dk columns: row h, key head j holds
+// sum over the query heads g of j of mix[h, g] q_g.
+struct AllNorm {
+  int n_q, n_k, dk, nv;
+  long ld;
+  float eps;
+  long cache_slots;
+  const float* mix;
+};
+
+// q of one token in shared memory (fp32) -> its rows for every query head; a thread keeps V columns of the query heads of one key head
+// in registers (GROUP of them; 0: any number, read again for every row).
+template <typename T, int V, int GROUP>
+__device__ __forceinline__ void mix_rows(const float* q, const float* mix, T* __restrict__ out, int n_q, int n_k, int dk) {
+  const int width = n_k * dk, group = GROUP > 0 ? GROUP : n_q / n_k;
+  for (int c = threadIdx.x * V; c < width; c += blockDim.x * V) {
+    const int j = c / dk, d = c % dk;
+    const float* src = q + size_t(j) * group * dk + d;
+    float qv[GROUP > 0 ? GROUP : 1][V];
+    if (GROUP > 0) {
+#pragma unroll
+      for (int g = 0; g < GROUP; ++g)
+#pragma unroll
+        for (int e = 0; e < V; ++e) qv[g][e] = src[g * dk + e];
+    }
+#pragma unroll 2
+    for (int h = 0; h < n_q; ++h) {
+      const float* m = mix + size_t(h) * n_q + j * group;
+      float a[V] = {};
+      if (GROUP > 0) {
+#pragma unroll
+        for (int g = 0; g < GROUP; ++g)
+#pragma unroll
+          for (int e = 0; e < V; ++e) a[e] = fmaf(m[g], qv[GROUP > 0 ? g : 0][e], a[e]);
+      } else {
+        for (int g = 0; g < group; ++g)
+#pragma unroll
+          for (int e = 0; e < V; ++e) a[e] = fmaf(m[g], src[g * dk + e], a[e]);
+      }
+      T* dst = out + size_t(h) * width + c;
+      if constexpr (V == 4 && sizeof(T) == 2) {
+        *reinterpret_cast<uint2*>(dst) = make_uint2(pack_bf16x2(a[0], a[1]), pack_bf16x2(a[2], a[3]));
+      } else if constexpr (V == 4) {
+        *reinterpret_cast<float4*>(dst) = make_float4(a[0], a[1], a[2], a[3]);
+      } else {
+        from_f32(dst, a[0]);
+      }
+    }
+  }
+}
+
+template <typename T, int V, bool MIX>
 __global__ void __launch_bounds__(256) qknorm_all_kernel(T* __restrict__ qkv, const int* __restrict__ slots, const T* __restrict__ q_w,
                                                          const T* __restrict__ k_w, T* __restrict__ k_cache, T* __restrict__ v_cache,
-                                                         int nq, int nk, int nv, long ld, float eps, long cache_slots) {
+                                                         T* __restrict__ wide, const AllNorm a, const Rotation rot, int mix_smem) {
+  extern __shared__ __align__(16) float s_row[];       // MIX or rotation: normed q and k of the row; MIX: then the mixing matrix
   __shared__ float red_q[8], red_k[8];
-  const int t = blockIdx.x;
-  T* row = qkv + size_t(t) * ld;
+  const int t = blockIdx.x, nq = a.n_q * a.dk, nk = a.n_k * a.dk, nv = a.nv;
+  T* row = qkv + size_t(t) * a.ld;
   auto load = [](const T* p, float (&f)[V]) {
     if constexpr (V == 8) load8(p, f); else f[0] = to_f32(*p);
   };
@@ -523,36 +639,88 @@ __global__ void __launch_bounds__(256) qknorm_all_kernel(T* __restrict__ qkv, co
     for (int e = 0; e < V; ++e) s += f[e] * f[e];
     if (c < nq) sq += s; else sk += s;
   }
-  const float rq = rsqrtf(block_sum(sq, red_q) / float(nq) + eps), rk = rsqrtf(block_sum(sk, red_k) / float(nk) + eps);
+  const float rq = rsqrtf(block_sum(sq, red_q) / float(nq) + a.eps), rk = rsqrtf(block_sum(sk, red_k) / float(nk) + a.eps);
   const int slot = slots[t];
-  const bool in = slot >= 0 && slot < cache_slots;
+  const bool in = slot >= 0 && slot < a.cache_slots;
+  const bool turned = rot.table != nullptr;
   for (int c = threadIdx.x * V; c < nq + nk + nv; c += blockDim.x * V) {
     load(row + c, f);
-    if (c < nq) {
-      load(q_w + c, w);
+    if (c < nq + nk) {
+      const float r = c < nq ? rq : rk;
+      load(c < nq ? q_w + c : k_w + (c - nq), w);
 #pragma unroll
-      for (int e = 0; e < V; ++e) f[e] = f[e] * rq * w[e];
-      store(row + c, f);
-    } else if (c < nq + nk) {
-      load(k_w + (c - nq), w);
+      for (int e = 0; e < V; ++e) f[e] = f[e] * r * w[e];
+      if (turned || (MIX && c < nq)) {
 #pragma unroll
-      for (int e = 0; e < V; ++e) f[e] = f[e] * rk * w[e];
-      if (in) store(k_cache + size_t(slot) * nk + (c - nq), f);
+        for (int e = 0; e < V; ++e) s_row[c + e] = f[e];
+      } else if (c < nq) {
+        store(row + c, f);
+      } else if (in) {
+        store(k_cache + size_t(slot) * nk + (c - nq), f);
+      }
     } else if (in) {
       store(v_cache + size_t(slot) * nv + (c - nq - nk), f);
     }
   }
+  if (!turned && !MIX) return;
+  float* s_mix = s_row + (nq + nk + 3) / 4 * 4;
+  if (MIX && mix_smem)
+    for (int i = threadIdx.x; i < a.n_q * a.n_q; i += blockDim.x) s_mix[i] = a.mix[i];
+  __syncthreads();
+  if (turned) {
+    const float* cs = rot.table + size_t(clamp_id(rot.positions[t], rot.rows)) * rot.dims;
+    const int half = rot.dims / 2;
+    for (int i = threadIdx.x; i < (a.n_q + a.n_k) * half; i += blockDim.x) {
+      const int j = i % half, x = rot.interleaved ? 2 * j : j, y = rot_pair(rot, x);
+      float* head = s_row + i / half * a.dk;
+      const float u = head[x], v = head[y];
+      head[x] = rot_one(rot, cs, x, u, v);
+      head[y] = rot_one(rot, cs, y, v, u);
+    }
+    __syncthreads();
+    for (int c = (MIX ? nq : 0) + threadIdx.x * V; c < nq + nk; c += blockDim.x * V) {
+#pragma unroll
+      for (int e = 0; e < V; ++e) f[e] = s_row[c + e];
+      if (c < nq) store(row + c, f);
+      else if (in) store(k_cache + size_t(slot) * nk + (c - nq), f);
+    }
+  }
+  if constexpr (MIX) {
+    T* out = wide + size_t(t) * a.n_q * nk;
+    const float* m = mix_smem ? s_mix : a.mix;
+    constexpr int W = V == 8 ? 4 : 1;
+    switch (a.n_q / a.n_k) {
+      case 1: mix_rows<T, W, 1>(s_row, m, out, a.n_q, a.n_k, a.dk); break;
+      case 2: mix_rows<T, W, 2>(s_row, m, out, a.n_q, a.n_k, a.dk); break;
+      case 4: mix_rows<T, W, 4>(s_row, m, out, a.n_q, a.n_k, a.dk); break;
+      case 8: mix_rows<T, W, 8>(s_row, m, out, a.n_q, a.n_k, a.dk); break;
+      default: mix_rows<T, W, 0>(s_row, m, out, a.n_q, a.n_k, a.dk); break;
+    }
+  }
 }
 template <typename T>
-static int launch_qknorm_all(void* qkv, const void* slots, const void* q_w, const void* k_w, void* k_cache, void* v_cache, int rows, int nq,
-                             int nk, int nv, long ld, float eps, long cache_slots, cudaStream_t st) {
-  T *x = static_cast<T*>(qkv), *kc = static_cast<T*>(k_cache), *vc = static_cast<T*>(v_cache);
+static int launch_qknorm_all(void* qkv, const void* slots, const void* q_w, const void* k_w, void* k_cache, void* v_cache, void* wide, int rows,
+                             const AllNorm& a, const Rotation& rot, cudaStream_t st) {
+  T *x = static_cast<T*>(qkv), *kc = static_cast<T*>(k_cache), *vc = static_cast<T*>(v_cache), *o = static_cast<T*>(wide);
   const T *qw = static_cast<const T*>(q_w), *kw = static_cast<const T*>(k_w);
   const int* s = static_cast<const int*>(slots);
-  if (nq % 8 == 0 && nk % 8 == 0 && nv % 8 == 0 && ld % 8 == 0 && al16(qkv, q_w, k_w, k_cache) && al16(v_cache))
-    qknorm_all_kernel<T, 8><<<rows, 256, 0, st>>>(x, s, qw, kw, kc, vc, nq, nk, nv, ld, eps, cache_slots);
-  else
-    qknorm_all_kernel<T, 1><<<rows, 256, 0, st>>>(x, s, qw, kw, kc, vc, nq, nk, nv, ld, eps, cache_slots);
+  const int nq = a.n_q * a.dk, nk = a.n_k * a.dk;
+  const bool vec = nq % 8 == 0 && nk % 8 == 0 && a.nv % 8 == 0 && a.ld % 8 == 0 && al16(qkv, q_w, k_w, k_cache) && al16(v_cache) &&
+                   (!a.mix || (a.dk % 8 == 0 && al16(wide)));
+  constexpr size_t kMost = 160 * 1024;
+  size_t smem = a.mix || rot.table ? size_t(nq + nk + 3) / 4 * 16 : 0;
+  const int mix_smem = a.mix && smem + size_t(a.n_q) * a.n_q * 4 <= kMost;
+  if (mix_smem) smem += size_t(a.n_q) * a.n_q * 4;
+  if (smem > kMost) return -2;
+#define XL_ALL(V, MIX)                                                                                                                 \
+  do {                                                                                                                                 \
+    static bool set = false;                                                                                                           \
+    if (!set) { cudaFuncSetAttribute(qknorm_all_kernel<T, V, MIX>, cudaFuncAttributeMaxDynamicSharedMemorySize, int(kMost)); set = true; } \
+    qknorm_all_kernel<T, V, MIX><<<rows, 256, smem, st>>>(x, s, qw, kw, kc, vc, o, a, rot, mix_smem);                                  \
+  } while (0)
+  if (a.mix) { if (vec) XL_ALL(8, true); else XL_ALL(1, true); }
+  else { if (vec) XL_ALL(8, false); else XL_ALL(1, false); }
+#undef XL_ALL
   return cudaGetLastError() == cudaSuccess ? 0 : -1;
 }
 
@@ -710,16 +878,18 @@ static void set_lead(NormParams<T>& p, const LeadRows& l) {
   p.scale = p.lead_scale = l.scale;
 }
 
-// x[t] = table[tokens[t]] * scale (+ pos_table[positions[t]]), or with keep_x: x[t] += it;  h = rms(x) * (w_next + w_off)
+// x[t] = table[tokens[t]] * scale (+ pos_table[positions[t]]), with w_rows its rms times w_rows, or with keep_x: x[t] += it;
+// h = rms(x) * (w_next + w_off)
 XL_API int xl_embed_rms_norm(const void* tokens, const void* table, float scale, const void* positions, const void* pos_table, int pos_rows,
-                             int keep_x, void* x, const void* w_next, float w_off, void* h, int rows, int H, int V, float eps, int f32,
+                             const void* w_rows, int keep_x, void* x, const void* w_next, float w_off, void* h, int rows, int H, int V, float eps, int f32,
                              void* stream) {
+  if (w_rows && keep_x) return -2;
   cudaStream_t st = static_cast<cudaStream_t>(stream);
-  const bool al = al16(table, x, w_next, h) && al16(pos_table);
+  const bool al = al16(table, x, w_next, h) && al16(pos_table, w_rows);
   const LeadRows l{tokens, table, positions, pos_table, V, pos_rows, scale};
   auto go = [&](auto* tag) {
     using E = std::remove_pointer_t<decltype(tag)>;
-    auto p = base_params<E>(x, nullptr, w_next, h, H, eps);
+    auto p = base_params<E>(x, w_rows, w_next, h, H, eps);
     set_lead(p, l);
     p.w_off = w_off;
     p.keep_x = keep_x;
@@ -741,6 +911,24 @@ XL_API int xl_post_norm_add_norm(const void* y, void* x, const void* w_post, con
   auto p = base_params<__nv_bfloat16>(x, w_post, w_next, h, H, eps);
   p.y = static_cast<const __nv_bfloat16*>(y);
   return launch_norm<__nv_bfloat16, SRC_ROWS>(p, rows, al, st);
+}
+
+// y = scale * (rms(ya) * w_a + rms(yb) * w_b);  x += rms(y) * w_post;  h = rms(x) * w_next
+XL_API int xl_branches_post_norm_add_norm(const void* ya, const void* yb, const void* w_a, const void* w_b, float scale, void* x,
+                                          const void* w_post, const void* w_next, void* h, int rows, int H, float eps, int f32, void* stream) {
+  cudaStream_t st = static_cast<cudaStream_t>(stream);
+  const bool al = al16(ya, yb, w_a, w_b) && al16(x, w_post, w_next, h);
+  auto go = [&](auto* tag) {
+    using E = std::remove_pointer_t<decltype(tag)>;
+    auto p = base_params<E>(x, w_post, w_next, h, H, eps);
+    p.y = static_cast<const E*>(ya);
+    p.y2 = static_cast<const E*>(yb);
+    p.w_y = static_cast<const E*>(w_a);
+    p.w_y2 = static_cast<const E*>(w_b);
+    p.scale = scale;
+    return launch_norm<E, SRC_PAIR>(p, rows, al, st);
+  };
+  return f32 ? go(static_cast<float*>(nullptr)) : go(static_cast<__nv_bfloat16*>(nullptr));
 }
 
 // x += mult * y, or ls * y element by element (ls [H], null: mult);  with `table`: x += table[tokens[t]] * lead_scale
@@ -820,14 +1008,20 @@ XL_API int xl_split_rows(const void* x, const void* tokens, const void* table, f
   return cudaGetLastError() == cudaSuccess ? 0 : -1;
 }
 
-// RMSNorm over the nq query and over the nk key columns of rows with pitch ld (q in place); k and v to the cache slots
-// [cache_slots, nk | nv].
+// RMSNorm over the n_q * dk query and over the n_k * dk key columns of rows with pitch ld, then the rotation (null table: none); q in
+// place, or with `mix` to wide [rows, n_q, n_k * dk] (see qknorm_all_kernel); k and v to the cache slots [cache_slots, nk | nv].
 XL_API int xl_qknorm_all_kvwrite(void* qkv, const void* slots, const void* q_w, const void* k_w, void* k_cache, void* v_cache, int rows,
-                                 int nq, int nk, int nv, long ld, float eps, long cache_slots, int f32, void* stream) {
+                                 int n_q, int n_k, int dk, int nv, long ld, float eps, long cache_slots, const void* rot_table,
+                                 const void* positions, int rot_dims, int rot_rows, int interleaved, const void* mix, void* wide, int f32,
+                                 void* stream) {
   if (rows <= 0) return 0;
+  if (rot_table && (rot_dims > dk || rot_dims % 2 || rot_rows < 1)) return -2;
+  if (mix && (!wide || n_q % n_k)) return -2;
   cudaStream_t st = static_cast<cudaStream_t>(stream);
-  if (f32) return launch_qknorm_all<float>(qkv, slots, q_w, k_w, k_cache, v_cache, rows, nq, nk, nv, ld, eps, cache_slots, st);
-  return launch_qknorm_all<__nv_bfloat16>(qkv, slots, q_w, k_w, k_cache, v_cache, rows, nq, nk, nv, ld, eps, cache_slots, st);
+  const Rotation rot{static_cast<const float*>(rot_table), static_cast<const int*>(positions), rot_dims, rot_rows, interleaved};
+  const AllNorm a{n_q, n_k, dk, nv, ld, eps, cache_slots, static_cast<const float*>(mix)};
+  if (f32) return launch_qknorm_all<float>(qkv, slots, q_w, k_w, k_cache, v_cache, wide, rows, a, rot, st);
+  return launch_qknorm_all<__nv_bfloat16>(qkv, slots, q_w, k_w, k_cache, v_cache, wide, rows, a, rot, st);
 }
 
 // out [rows, n] (pitch ldo) = o (dense) * sigmoid(gate, pitch ldg) * scale

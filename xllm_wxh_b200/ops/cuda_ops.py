@@ -321,14 +321,14 @@ def _f32flag(t: torch.Tensor):
     return c_int(int(t.dtype == torch.float32))
 
 
-def _embed_norm(ids, table, scale, positions, pos_table, x, keep_x, w_next, eps, w_offset) -> torch.Tensor:
+def _embed_norm(ids, table, scale, positions, pos_table, x, keep_x, w_next, eps, w_offset, w_rows=None) -> torch.Tensor:
     global launch_count
     T, H = x.shape
     assert x.is_contiguous() and x.dtype == torch.float32 and ids.numel() == T and table.shape[1] == H and w_next.dtype == table.dtype
     assert pos_table is None or (pos_table.dtype == table.dtype and pos_table.is_contiguous() and pos_table.shape[1] == H)
     h = torch.empty((T, H), dtype=table.dtype, device=table.device)
     _check(lib().xl_embed_rms_norm(_ptr(ids), _ptr(table), c_float(scale), _ptr(positions), _ptr(pos_table),
-                                   c_int(0 if pos_table is None else pos_table.shape[0]), c_int(int(keep_x)), _ptr(x), _ptr(w_next),
+                                   c_int(0 if pos_table is None else pos_table.shape[0]), _ptr(w_rows), c_int(int(keep_x)), _ptr(x), _ptr(w_next),
                                    c_float(w_offset), _ptr(h), c_int(T), c_int(H), c_int(table.shape[0]), c_float(eps), _f32flag(table),
                                    _stream()), "xl_embed_rms_norm")
     launch_count += 1
@@ -336,10 +336,11 @@ def _embed_norm(ids, table, scale, positions, pos_table, x, keep_x, w_next, eps,
 
 
 def embed_rms_norm(ids: torch.Tensor, table: torch.Tensor, scale: float, w_next: torch.Tensor, eps: float, positions=None, pos_table=None,
-                   w_offset: float = 0.0):
-    """(fp32 residual x = table[ids] * scale (+ pos_table[positions]), rms(x) * (w_next + w_offset))."""
+                   w_offset: float = 0.0, w_rows: Optional[torch.Tensor] = None):
+    """(fp32 residual x = table[ids] * scale (+ pos_table[positions]), or rms of that times w_rows, rms(x) * (w_next + w_offset))."""
+    assert w_rows is None or (w_rows.dtype == table.dtype and w_rows.numel() == table.shape[1])
     x = torch.empty((ids.numel(), table.shape[1]), dtype=torch.float32, device=table.device)
-    return x, _embed_norm(ids, table, scale, positions, pos_table, x, False, w_next, eps, w_offset)
+    return x, _embed_norm(ids, table, scale, positions, pos_table, x, False, w_next, eps, w_offset, w_rows)
 
 
 def lead_norm(lead, x: torch.Tensor, w_next: torch.Tensor, eps: float, w_offset: float = 0.0) -> torch.Tensor:
@@ -364,6 +365,19 @@ def post_norm_add_norm(y: torch.Tensor, x: torch.Tensor, w_post: torch.Tensor, w
     h = torch.empty_like(y)
     _check(lib().xl_post_norm_add_norm(_ptr(y), _ptr(x), _ptr(w_post), _ptr(w_next), _ptr(h), c_int(T), c_int(H), c_float(eps),
                                        _f32flag(y), _stream()), "xl_post_norm_add_norm")
+    launch_count += 1
+    return h
+
+
+def branches_post_norm_add_norm(ya, yb, w_a, w_b, scale, x, w_post, w_next, eps) -> torch.Tensor:
+    """y = scale * (rms(ya) * w_a + rms(yb) * w_b); x += rms(y) * w_post in place; returns rms(x) * w_next."""
+    global launch_count
+    T, H = ya.shape
+    assert ya.is_contiguous() and yb.is_contiguous() and ya.shape == yb.shape == x.shape and x.is_contiguous() and x.dtype == torch.float32
+    h = torch.empty_like(ya)
+    _check(lib().xl_branches_post_norm_add_norm(_ptr(ya), _ptr(yb), _ptr(w_a), _ptr(w_b), c_float(scale), _ptr(x), _ptr(w_post), _ptr(w_next),
+                                                _ptr(h), c_int(T), c_int(H), c_float(eps), _f32flag(ya), _stream()),
+           "xl_branches_post_norm_add_norm")
     launch_count += 1
     return h
 
@@ -428,18 +442,23 @@ def split_rows(x: torch.Tensor, ids: torch.Tensor, table: torch.Tensor, scale: f
     return out
 
 
-def qknorm_all_kvwrite(qkv, slots, q_w, k_w, eps, k_cache, v_cache, n_q, n_kv):
-    """RMSNorm over all query and over all key columns (q in place), k and v into the paged caches; rows of qkv may hold more
-    behind v.  Returns q [T, n_q * dk] (a view of qkv)."""
+def qknorm_all_kvwrite(qkv, slots, q_w, k_w, eps, k_cache, v_cache, n_q, n_kv, rot=None, mix=None):
+    """RMSNorm over all query and over all key columns, the rotation `rot` behind it, k and v into the paged caches; rows of qkv may
+    hold more behind v.  Returns q [T, n_q * dk] (a view of qkv), or with `mix` the queries [T, n_q * n_kv * dk] of mixed scores."""
     global launch_count
     T = qkv.shape[0]
     dk, dv = k_cache.shape[-1], v_cache.shape[-1]
     assert qkv.stride(1) == 1 and qkv.shape[1] >= (n_q + n_kv) * dk + n_kv * dv and k_cache.dtype == qkv.dtype
-    _check(lib().xl_qknorm_all_kvwrite(_ptr(qkv), _ptr(slots), _ptr(q_w), _ptr(k_w), _ptr(k_cache), _ptr(v_cache), c_int(T),
-                                       c_int(n_q * dk), c_int(n_kv * dk), c_int(n_kv * dv), c_long(qkv.stride(0)), c_float(eps),
-                                       c_long(k_cache.shape[0] * k_cache.shape[1]), _f32flag(qkv), _stream()), "xl_qknorm_all_kvwrite")
+    wide = None
+    if mix is not None:
+        assert mix.dtype == torch.float32 and mix.is_contiguous() and mix.shape == (n_q, n_q)
+        wide = torch.empty((T, n_q * n_kv * dk), dtype=qkv.dtype, device=qkv.device)
+    _check(lib().xl_qknorm_all_kvwrite(_ptr(qkv), _ptr(slots), _ptr(q_w), _ptr(k_w), _ptr(k_cache), _ptr(v_cache), c_int(T), c_int(n_q),
+                                       c_int(n_kv), c_int(dk), c_int(n_kv * dv), c_long(qkv.stride(0)), c_float(eps),
+                                       c_long(k_cache.shape[0] * k_cache.shape[1]), *_rot_args(rot), _ptr(mix), _ptr(wide), _f32flag(qkv),
+                                       _stream()), "xl_qknorm_all_kvwrite")
     launch_count += 1
-    return qkv[:, :n_q * dk]
+    return qkv[:, :n_q * dk] if wide is None else wide
 
 
 def gate_into(o: torch.Tensor, gate: torch.Tensor, scale: float, out: torch.Tensor) -> None:
@@ -550,15 +569,18 @@ def token_shift(h: torch.Tensor, mu: torch.Tensor, last: torch.Tensor, inp) -> t
     return out
 
 
-def conv_silu(x: torch.Tensor, w: torch.Tensor, b: torch.Tensor, state: torch.Tensor, inp) -> torch.Tensor:
-    """silu(b + causal convolution of x [T, C] (may be a strided view) with w [taps, C]); state [slots, taps - 1, C]."""
+def causal_conv(x: torch.Tensor, w: torch.Tensor, b: Optional[torch.Tensor], state: torch.Tensor, inp, act: str = "none",
+                residual: bool = False) -> torch.Tensor:
+    """act(b + causal convolution of x [T, C] (may be a strided view) with w [taps, C]) (+ x); act "silu" or "none"; state
+    [slots, taps - 1, C]."""
     global launch_count
     T, C = x.shape
-    assert x.stride(1) == 1 and w.is_contiguous() and w.dtype == b.dtype == state.dtype == x.dtype
+    assert x.stride(1) == 1 and w.is_contiguous() and w.dtype == state.dtype == x.dtype and (b is None or b.dtype == x.dtype)
     n, seqs = _state_args(inp, state)
     out = _rows_out(inp, (T, C), x)
-    _check(lib().xl_conv_silu(_ptr(x), _ptr(w), _ptr(b), _ptr(state), _ptr(out), _ptr(inp.token_seq), *seqs, c_int(T), c_int(C),
-                              c_int(w.shape[0]), c_long(x.stride(0)), c_int(int(inp.has_prefill)), _f32flag(x), _stream()), "xl_conv_silu")
+    _check(lib().xl_causal_conv(_ptr(x), _ptr(w), _ptr(b), _ptr(state), _ptr(out), _ptr(inp.token_seq), *seqs, c_int(T), c_int(C),
+                                c_int(w.shape[0]), c_long(x.stride(0)), c_int(int(inp.has_prefill)), c_int(int(act == "silu")),
+                                c_int(int(residual)), _f32flag(x), _stream()), "xl_causal_conv")
     launch_count += 2 if inp.has_prefill and w.shape[0] > 1 else 1
     return out
 
@@ -576,29 +598,78 @@ def mix_segment_rows(T: int, H: int, d: int) -> int:
     return min(512, max(64, 1 << (L.bit_length() - 1)))
 
 
+def _segments(inp, T: int, n: int, H: int, dk: int, dv: int, record: int, device):
+    """(segment arguments of a matrix-state kernel, whether longer portions may occur, launches): rows per segment, how many there
+    can be and the workspace of the states between them."""
+    has_long = bool(inp.has_prefill) and T > 1
+    if not has_long:
+        return (c_int(2), c_int(0), c_void_p(0), c_void_p(0)), (), False, 1
+    L = mix_segment_rows(T, H, max(dk, dv))
+    cap = T // L + min(n, T // 2)                           # every portion of two and more rows ends with one partly filled segment
+    ws = wp = None
+    if (T if inp.padded else inp.max_q) > L and max(dk, dv) <= 128:
+        ws = torch.empty((cap, H, record), dtype=torch.float32, device=device)
+        wp = torch.empty((cap, H, dk), dtype=torch.float32, device=device)
+    return (c_int(L), c_int(cap), _ptr(ws), _ptr(wp)), (ws, wp), True, 2 if ws is None else 4
+
+
+def _check_rows(r, k, v, gate, out, T, dk, dv):
+    for t, width in ((r, dk), (k, dk), (v, dv)):
+        assert t.stride(1) == 1 and t.stride(0) == r.stride(0) and t.dtype == out.dtype and t.shape == (T, width)
+    assert gate.stride(1) == out.stride(1) == 1 and gate.shape == (T, dv)
+
+
 def time_mix(r, k, v, z, w0, u, gate, norm_w, scale, eps, state, inp, out) -> None:
     global launch_count
     H, d = u.shape
     T = r.shape[0]
-    for t in (r, k, v):
-        assert t.stride(1) == 1 and t.stride(0) == r.stride(0) and t.dtype == out.dtype and t.shape == (T, H * d)
-    assert gate.stride(1) == out.stride(1) == 1 and z.is_contiguous() and z.dtype == w0.dtype == u.dtype == state.dtype == torch.float32
+    _check_rows(r, k, v, gate, out, T, H * d, H * d)
+    assert z.is_contiguous() and z.dtype == w0.dtype == u.dtype == state.dtype == torch.float32
     n, seqs = _state_args(inp, state)
-    has_long = bool(inp.has_prefill) and T > 1
     if inp.padded:
         out.zero_()
-    L, cap, ws, wp = 2, 0, None, None
-    if has_long:
-        L = mix_segment_rows(T, H, d)
-        cap = T // L + min(n, T // 2)                       # every portion of two and more rows ends with one partly filled segment
-        if (T if inp.padded else inp.max_q) > L and d <= 128:
-            ws = torch.empty((cap, H, d, d), dtype=torch.float32, device=r.device)
-            wp = torch.empty((cap, H, d), dtype=torch.float32, device=r.device)
+    seg, keep, has_long, launches = _segments(inp, T, n, H, d, d, d * d, r.device)
     _check(lib().xl_time_mix(_ptr(r), _ptr(k), _ptr(v), _ptr(z), _ptr(w0), _ptr(u), _ptr(gate), _ptr(norm_w), c_float(scale), c_float(eps),
                              _ptr(state), _ptr(out), *seqs, c_int(H), c_int(d), c_long(r.stride(0)), c_long(gate.stride(0)),
-                             c_long(out.stride(0)), c_int(L), c_int(cap), _ptr(ws), _ptr(wp), c_int(int(has_long)), c_int(1), _f32flag(r),
-                             _stream()), "xl_time_mix")
-    launch_count += 1 + (0 if not has_long else 1 if ws is None else 3)
+                             c_long(out.stride(0)), *seg, c_int(int(has_long)), c_int(1), _f32flag(r), _stream()), "xl_time_mix")
+    launch_count += launches
+
+
+def gated_memory(q, k, v, z, bias, inv_tau, gate, norm_w, eps, state, inp) -> torch.Tensor:
+    global launch_count
+    _, H, dk, dv = state.shape
+    T = q.shape[0]
+    n, seqs = _state_args(inp, state)
+    out = _rows_out(inp, (T, H * dv), q)
+    _check_rows(q, k, v, gate, out, T, H * dk, H * dv)
+    assert z.is_contiguous() and z.shape == (T, H * dk) and bias.numel() == H * dk and norm_w.numel() == dv
+    assert z.dtype == bias.dtype == state.dtype == torch.float32 and norm_w.dtype == q.dtype
+    seg, keep, has_long, launches = _segments(inp, T, n, H, dk, dv, dk * dv, q.device)
+    _check(lib().xl_gated_memory(_ptr(q), _ptr(k), _ptr(v), _ptr(z), _ptr(bias), c_float(inv_tau), _ptr(gate), _ptr(norm_w), c_float(eps),
+                                 _ptr(state), _ptr(out), *seqs, c_int(H), c_int(dk), c_int(dv), c_long(q.stride(0)), c_long(gate.stride(0)),
+                                 c_long(out.stride(0)), *seg, c_int(int(has_long)), c_int(1), _f32flag(q), _stream()), "xl_gated_memory")
+    launch_count += launches
+    return out
+
+
+def matrix_memory(q, k, v, gates, bias, cap, gate, norm_w, eps, state, top, inp) -> torch.Tensor:
+    global launch_count
+    H = top.shape[1]
+    T, dk, dv = q.shape[0], q.shape[1] // H, v.shape[1] // H
+    n, seqs = _state_args(inp, state)
+    out = _rows_out(inp, (T, H * dv), q)
+    _check_rows(q, k, v, gate, out, T, H * dk, H * dv)
+    assert gates.is_contiguous() and gates.shape == (T, 2 * H) and bias.numel() == 2 * H and norm_w.numel() == H * dv
+    assert state.shape == (state.shape[0], H, dk * dv + dk) and top.shape[0] == state.shape[0] and top.is_contiguous()
+    assert gates.dtype == bias.dtype == state.dtype == top.dtype == torch.float32 and norm_w.dtype == q.dtype
+    seg, keep, has_long, launches = _segments(inp, T, n, H, dk, dv, dk * dv + dk, q.device)
+    fi = torch.empty((3, H, T), dtype=torch.float32, device=q.device)
+    _check(lib().xl_matrix_memory(_ptr(q), _ptr(k), _ptr(v), _ptr(gates), _ptr(bias), c_float(cap), _ptr(gate), _ptr(norm_w), c_float(eps),
+                                  _ptr(state), _ptr(top), _ptr(out), *seqs, c_int(H), c_int(dk), c_int(dv), c_long(q.stride(0)),
+                                  c_long(gate.stride(0)), c_long(out.stride(0)), *seg, _ptr(fi), c_int(T), c_int(int(has_long)), c_int(1),
+                                  _f32flag(q), _stream()), "xl_matrix_memory")
+    launch_count += launches + int(has_long)
+    return out
 
 
 def selective_scan(x, dt, dt_bias, A, B, C, D, z, state, inp) -> torch.Tensor:
@@ -706,21 +777,22 @@ def paged_attention_ext(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.T
     buffer), caches [blocks, block, Hkv, dk | dv] -> [T, Hq * dv].  score = scale q.k (bounded by softcap tanh(. / softcap)) -
     slopes[h] * distance; keys of the query's own chunk of `chunk` positions only (0: all); `keep_first` first keys stay visible
     behind the window; exp(sinks[h]) joins the softmax denominator; `mix`: differential attention (see `ops`).  The values may be
-    a view of the keys.  bf16 tensors with head dimensions up to 256 (128 with `mix`; multiples of 8) run on the tensor-core
+    a view of the keys; one key head may serve several value heads.  bf16 tensors with head dimensions up to 256 (128 with `mix`; multiples of 8) run on the tensor-core
     kernels, anything else on the fp32-pipe kernel."""
     global launch_count
     from ..framework.step_input import H_NUM_DECODE, H_NUM_SEQS
     T, Hq, dk = q.shape
     block_size, n_kv, dv = k_cache.shape[1], v_cache.shape[2], v_cache.shape[3]
     maps = 1 if mix is None else 2
-    assert k_cache.is_contiguous() and k_cache.shape[2] == n_kv * maps and v_cache.stride(3) == 1 and v_cache.stride(0) == block_size * v_cache.stride(1)
+    shared_keys = maps == 1 and n_kv > 1 and k_cache.shape[2] == 1
+    assert k_cache.is_contiguous() and k_cache.shape[2] == (1 if shared_keys else n_kv * maps) and v_cache.stride(3) == 1 and v_cache.stride(0) == block_size * v_cache.stride(1)
     assert v_cache.stride(2) == dv or n_kv == 1
     L, padded = inp.layout, inp.padded
     for t in (slopes, sinks):
         assert t is None or (t.dtype == torch.float32 and t.numel() == Hq and t.is_contiguous())
     out = (torch.zeros if padded else torch.empty)((T, Hq // maps * dv), dtype=q.dtype, device=q.device)
     factor, mult, eps = mix if mix is not None else (None, 0.0, 0.0)
-    last = (c_long(v_cache.stride(1)), c_int(maps), _ptr(factor), c_float(mult), c_float(eps))
+    last = (c_long(v_cache.stride(1)), c_int(int(shared_keys)), c_int(maps), _ptr(factor), c_float(mult), c_float(eps))
     ext = (c_float(softcap), c_float(bound)) + last
     n_dec = inp.B if padded else inp.n_decode
     n_all = inp.B if padded else inp.n_seqs

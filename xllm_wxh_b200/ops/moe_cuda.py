@@ -76,17 +76,20 @@ def moe_sort(ids: torch.Tensor, expert_offset: int, E_local: int, max_rows: Opti
     return SortedRouting(work, sorted_src, dst_of, E_local, max_tiles, rows)
 
 
+RELU2 = 4        # grouped_gemm's epilogue without a gate
+
+
 def grouped_gemm(a: torch.Tensor, w: torch.Tensor, r, swiglu: int = 0, out: Optional[torch.Tensor] = None,
                  c_rows_per_expert: int = 0, c_col_stride: int = 0, limit: float = 0.0) -> torch.Tensor:
     """a [R_cap, K] rows sorted by expert; w [E_local, N, K]; returns [R_cap, N] (or [R_cap, N/2] with a gated epilogue:
-    `swiglu` 1 = silu gate, 2 = tanh-gelu gate, 3 = clamped gate with `limit`).
+    `swiglu` 1 = silu gate, 2 = tanh-gelu gate, 3 = clamped gate with `limit`; 4 = squared relu of all N columns).
     `r` provides the device-side tile table (`tile_expert`, `tile_row0`, `tile_row_end`, `num_m_tiles`, `max_tiles`).
     With `out` given, row `row - expert * c_rows_per_expert` / column offset `expert * c_col_stride` place each tile."""
     R_cap, K = a.shape
     E, N, K2 = w.shape
     assert K == K2 and w.is_contiguous() and a.stride(-1) == 1
     if out is None:
-        out = torch.empty((R_cap, N // 2 if swiglu else N), dtype=torch.bfloat16, device=a.device)
+        out = torch.empty((R_cap, N // 2 if swiglu and swiglu != RELU2 else N), dtype=torch.bfloat16, device=a.device)
     _check(lib().xl_grouped_gemm_bf16(_ptr(a), _ptr(w), _ptr(out), c_int(R_cap), c_int(N), c_int(K), c_int(a.stride(0)),
                                       c_int(out.stride(0)), c_int(E), _ptr(r.tile_expert), _ptr(r.tile_row0), _ptr(r.tile_row_end),
                                       _ptr(r.num_m_tiles), c_int(r.max_tiles), c_int(int(swiglu)), c_int(c_rows_per_expert),
@@ -140,16 +143,16 @@ def moe_experts(x: torch.Tensor, w13: torch.Tensor, w2: torch.Tensor, weights: t
     return combine(y, r, weights, T, add)
 
 
-def grouped_gemm_simt(a: torch.Tensor, w: torch.Tensor, r: SortedRouting, gather_k: int = 0) -> torch.Tensor:
+def grouped_gemm_simt(a: torch.Tensor, w: torch.Tensor, r: SortedRouting, gather_k: int = 0, act: int = 0) -> torch.Tensor:
     """The fp32-pipe grouped GEMM (fp32 operands, or bf16 ones of any shape).  `gather_k` > 0: `a` holds the unsorted token
-    rows and sorted row i reads row sorted_src[i] // gather_k of it."""
+    rows and sorted row i reads row sorted_src[i] // gather_k of it.  `act`: one of `cuda_ops.PLAIN_ACTS`."""
     E, N, K = w.shape
     assert a.shape[1] == K and w.is_contiguous() and a.stride(-1) == 1 and a.dtype == w.dtype
     out = torch.empty((max(r.n, 1), N), dtype=a.dtype, device=a.device)
     _check(lib().xl_grouped_gemm_simt(_ptr(a), _ptr(w), _ptr(out), c_int(N), c_int(K), ctypes.c_long(a.stride(0)), ctypes.c_long(N),
                                       _ptr(r.tile_expert), _ptr(r.tile_row0), _ptr(r.tile_row_end), _ptr(r.num_m_tiles), c_int(r.max_tiles),
                                       _ptr(r.sorted_src) if gather_k else c_void_p(0), c_int(max(gather_k, 1)),
-                                      c_int(int(a.dtype == torch.float32)), _stream()), "xl_grouped_gemm_simt")
+                                      c_int(act), c_int(int(a.dtype == torch.float32)), _stream()), "xl_grouped_gemm_simt")
     cuda_ops.launch_count += 1
     return out
 
@@ -157,9 +160,13 @@ def grouped_gemm_simt(a: torch.Tensor, w: torch.Tensor, r: SortedRouting, gather
 def expert_rows(x: torch.Tensor, w13: torch.Tensor, w2: torch.Tensor, ids: torch.Tensor, act: str = "silu", interleaved: bool = False,
                 limit: float = 0.0):
     """Outputs of the chosen experts before their weighted sum: (rows [*, H], dst_of [T * k] with -1 for ids outside the
-    experts of w13)."""
+    experts of w13).  act "relu2": w13 [E, ff, H] without a gate."""
     k = ids.shape[1]
     r = moe_sort(ids, 0, w13.shape[0])
+    if act == "relu2":
+        if cuda_ops._tc_gemm_ok(x, w13) and cuda_ops._tc_gemm_ok(x, w2) and x.shape[1] % 8 == 0:
+            return grouped_gemm(grouped_gemm(gather_rows(x, r, k), w13, r, swiglu=RELU2), w2, r), r.dst_of
+        return grouped_gemm_simt(grouped_gemm_simt(x, w13, r, k, cuda_ops.PLAIN_ACTS[act]), w2, r), r.dst_of
     if interleaved:
         y = grouped_gemm(grouped_gemm(gather_rows(x, r, k), w13, r, swiglu=1 + cuda_ops.ACTS[act], limit=limit), w2, r)
     elif cuda_ops._tc_gemm_ok(x, w13) and cuda_ops._tc_gemm_ok(x, w2) and x.shape[1] % 8 == 0:
