@@ -412,6 +412,287 @@ __global__ void __launch_bounds__(160) decode_attn_tma_kernel(const __grid_const
   }
 }
 
+// ---------------------------------------------------------------- one wide key head for all query heads
+// One CTA handles one (sequence, block of 16 query rows, KV split); a row is (token, query head), so the rows of a block may belong to
+// several value heads.  Keys and values pass through a ring of [64 tokens][64 columns] slabs: the slabs of a tile's keys, whose
+// products add up to S, then those of the value heads that the block's rows need; P is zero in the rows of other value heads, so all of
+// them accumulate into one O.
+constexpr int kWideSlabs = 10;
+struct WideDecBarriers {
+  uint64_t full[kWideSlabs];
+  uint64_t empty[kWideSlabs];
+};
+
+template <int DV>
+__global__ void __launch_bounds__(160) decode_attn_wide_kernel(const __grid_constant__ CUtensorMap tmK, const __grid_constant__ CUtensorMap tmV,
+                                                               const DecParams p, const int KS) {
+  constexpr int VH = DV / 64;
+  constexpr int SLAB = kTile * 128;
+  constexpr float kL2e = 1.4426950408889634f;
+  extern __shared__ uint8_t smem_raw[];
+  uint8_t* ring = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(smem_raw) + 1023) & ~uintptr_t(1023));
+  uint8_t* sQ = ring + kWideSlabs * SLAB;                        // 16 x 64 KS bf16, 16-byte-chunk XOR swizzle
+  WideDecBarriers* bars = reinterpret_cast<WideDecBarriers*>(sQ + 16 * KS * 128);
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  const int seq = p.seq_begin + blockIdx.x, row0 = blockIdx.y * 16, split = blockIdx.z;
+  const int group = p.n_q / p.n_kv, dk = p.dk, dv = p.dv;
+  if (seq >= (p.dyn_end ? *p.dyn_end : p.seq_end)) return;
+  const int q_start = p.q_cu[seq];
+  const int q_len = p.q_cu[seq + 1] - q_start;
+  const int kv_len = p.kv_lens[seq];
+  if (q_len <= 0) return;
+  const int rows = min(16, q_len * p.n_q - row0);
+  if (rows <= 0) return;
+  // value heads of the rows: consecutive ones, all of them when the block reaches into the next token
+  const int h_first = row0 % p.n_q, h_last = h_first + rows - 1;
+  const int v_first = h_last >= p.n_q ? 0 : h_first / group, v_last = h_last >= p.n_q ? p.n_kv - 1 : h_last / group;
+  const int* bt = p.block_tables + size_t(seq) * p.max_blocks;
+  const int r_begin = p.window > 0 ? max(0, kv_len - q_len - p.window + 1) / kTile * kTile : 0;
+  const int all_tiles = (kv_len - r_begin + kTile - 1) / kTile;
+  const int per_split = (all_tiles + p.num_splits - 1) / p.num_splits;
+  const int t_first = split * per_split;
+  const int n_tiles = max(0, min(all_tiles, t_first + per_split) - t_first);
+
+  if (threadIdx.x == 0) {
+    for (int s = 0; s < kWideSlabs; ++s) {
+      mbar_init(&bars->full[s], 1);
+      mbar_init(&bars->empty[s], 4);
+    }
+    mbar_fence_init();
+  }
+  for (int i = threadIdx.x; i < 16 * KS * 8; i += blockDim.x) {
+    const int r = i / (KS * 8), c = i % (KS * 8);
+    const bool ok = r < rows && c * 8 < dk;
+    const int m = ok ? row0 + r : 0;
+    const __nv_bfloat16* src = p.q + size_t(q_start + m / p.n_q) * p.q_stride + size_t(m % p.n_q) * dk + (ok ? c * 8 : 0);
+    cp_async_16(sQ + uint32_t(r) * (KS * 128) + (uint32_t(c ^ (r & 7)) << 4), src, ok);
+  }
+  cp_async_commit();
+  cp_async_wait_all();
+  __syncthreads();
+
+  float o[DV / 8][4];
+#pragma unroll
+  for (int i = 0; i < DV / 8; ++i) o[i][0] = o[i][1] = o[i][2] = o[i][3] = 0.f;
+  float m_run[2] = {-INFINITY, -INFINITY}, l_run[2] = {0.f, 0.f};
+  const int row_a = lane >> 2, row_b = row_a + 8;
+
+  if (warp == 4) {
+    // ------------------------------------------------------------ producer: lanes share a slab's boxes
+    const int bt_tok = p.box_tokens;
+    if (lane == 0) {
+      prefetch_tmap(&tmK);
+      prefetch_tmap(&tmV);
+    }
+    const int per_tile = KS + (v_last - v_first + 1) * VH;
+    int c = 0;
+    bool ok = true;
+    for (int t = 0; t < n_tiles && ok; ++t) {
+      const int base = r_begin + (t_first + t) * kTile;
+      const int n_boxes = (min(kTile, kv_len - base) + bt_tok - 1) / bt_tok;
+      int z = 0;
+      if (lane < n_boxes) {
+        const int tok = base + lane * bt_tok;
+        int blk = bt[tok / p.block_size];
+        if (blk < 0 || blk >= p.num_blocks_total) blk = 0;
+        z = blk * p.block_size + tok % p.block_size;
+      }
+      for (int i = 0; i < per_tile && ok; ++i, ++c) {
+        const int s = c % kWideSlabs;
+        if (lane == 0) {
+          if (!mbar_wait(&bars->empty[s], ((c / kWideSlabs) & 1) ^ 1)) {
+            atomicExch(p.status, XL_ERR_WAIT_EMPTY);
+            ok = false;
+          } else {
+            mbar_arrive_expect_tx(&bars->full[s], uint32_t(n_boxes) * bt_tok * 128);
+          }
+        }
+        ok = __shfl_sync(0xffffffffu, ok, 0);
+        if (ok && lane < n_boxes) {
+          uint8_t* dst = ring + s * SLAB + lane * bt_tok * 128;
+          if (i < KS) tma_load_3d(dst, &tmK, &bars->full[s], i * 64, 0, z);
+          else tma_load_3d(dst, &tmV, &bars->full[s], (i - KS) % VH * 64, v_first + (i - KS) / VH, z);
+        }
+        __syncwarp();
+      }
+    }
+    if (!ok && lane == 0)    // let the copies already issued land (bounded) before the CTA retires
+      for (int j = max(0, c - kWideSlabs); j < c - 1; ++j) mbar_wait(&bars->full[j % kWideSlabs], (j / kWideSlabs) & 1);
+  } else {
+    // ------------------------------------------------------------ consumers
+    const int m_a = row0 + (row_a < rows ? row_a : 0), m_b = row0 + (row_b < rows ? row_b : 0);
+    const int lim_a = kv_len - q_len + m_a / p.n_q, lim_b = kv_len - q_len + m_b / p.n_q;
+    const int vh_a = m_a % p.n_q / group, vh_b = m_b % p.n_q / group;
+    const int rk = (lane & 7) + (lane >> 4) * 8;           // K fragment row (token) of this lane
+    const int rv = (lane & 7) + ((lane >> 3) & 1) * 8;     // V fragment row (token) of this lane
+    const int rq = (lane & 7) + ((lane >> 3) & 1) * 8;     // Q fragment row
+    const uint32_t q_row = smem_u32(sQ + uint32_t(rq) * (KS * 128)), ring_u = smem_u32(ring);
+    int c = 0;
+    bool ok = true;
+    auto take = [&]() -> bool {
+      if (mbar_wait(&bars->full[c % kWideSlabs], (c / kWideSlabs) & 1)) return true;
+      if (lane == 0) atomicExch(p.status, XL_ERR_WAIT_FULL);
+      return false;
+    };
+    auto give = [&]() {
+      __syncwarp();
+      if (lane == 0) mbar_arrive(&bars->empty[c % kWideSlabs]);
+      ++c;
+    };
+    for (int t = 0; t < n_tiles && ok; ++t) {
+      const int base = r_begin + (t_first + t) * kTile + warp * 16;
+      const bool mine = base < kv_len;
+      float sc[2][4];
+#pragma unroll
+      for (int i = 0; i < 2; ++i) sc[i][0] = sc[i][1] = sc[i][2] = sc[i][3] = 0.f;
+      for (int ks = 0; ks < KS; ++ks) {
+        if (!(ok = take())) break;
+        if (mine) {
+          const uint32_t tK = ring_u + (c % kWideSlabs) * SLAB + warp * 2048 + rk * 128;
+#pragma unroll
+          for (int i = 0; i < 4; ++i) {
+            uint32_t b0, b1, b2, b3, a[4];
+            ldsm_x4(tK + (((i * 2 + ((lane >> 3) & 1)) ^ (rk & 7)) << 4), b0, b1, b2, b3);
+            ldsm_x4(q_row + (uint32_t((ks * 8 + i * 2 + (lane >> 4)) ^ (rq & 7)) << 4), a[0], a[1], a[2], a[3]);
+            mma_bf16_16816(sc[0], a, b0, b1);
+            mma_bf16_16816(sc[1], a, b2, b3);
+          }
+        }
+        give();
+      }
+      if (!ok) break;
+      uint32_t pa[4] = {0, 0, 0, 0};
+      if (mine) {
+        float mx[2] = {-INFINITY, -INFINITY};
+#pragma unroll
+        for (int i = 0; i < 2; ++i) {
+#pragma unroll
+          for (int e = 0; e < 4; ++e) {
+            const int tok = base + i * 8 + (lane & 3) * 2 + (e & 1);
+            const int lim = (e < 2) ? lim_a : lim_b;
+            const bool see = tok <= lim && tok < kv_len && (p.window <= 0 || tok > lim - p.window);
+            sc[i][e] = see ? sc[i][e] * p.scale_log2 : -INFINITY;
+            mx[e >> 1] = fmaxf(mx[e >> 1], sc[i][e]);
+          }
+        }
+        float alpha[2];
+#pragma unroll
+        for (int h = 0; h < 2; ++h) {
+          mx[h] = fmaxf(mx[h], __shfl_xor_sync(0xffffffffu, mx[h], 1));
+          mx[h] = fmaxf(mx[h], __shfl_xor_sync(0xffffffffu, mx[h], 2));
+          const float m_new = fmaxf(m_run[h], mx[h]);
+          alpha[h] = (m_new == -INFINITY) ? 1.f : exp2f(m_run[h] - m_new);
+          m_run[h] = m_new;
+        }
+        float rs[2] = {0.f, 0.f};
+#pragma unroll
+        for (int i = 0; i < 2; ++i) {
+#pragma unroll
+          for (int e = 0; e < 4; ++e) {
+            const float m = m_run[e >> 1];
+            sc[i][e] = (m == -INFINITY) ? 0.f : exp2f(sc[i][e] - m);
+            rs[e >> 1] += sc[i][e];
+          }
+        }
+        l_run[0] = l_run[0] * alpha[0] + rs[0];
+        l_run[1] = l_run[1] * alpha[1] + rs[1];
+        pa[0] = pack_bf16x2(sc[0][0], sc[0][1]);
+        pa[1] = pack_bf16x2(sc[0][2], sc[0][3]);
+        pa[2] = pack_bf16x2(sc[1][0], sc[1][1]);
+        pa[3] = pack_bf16x2(sc[1][2], sc[1][3]);
+        if (alpha[0] != 1.f || alpha[1] != 1.f) {
+#pragma unroll
+          for (int i = 0; i < DV / 8; ++i) {
+            o[i][0] *= alpha[0]; o[i][1] *= alpha[0]; o[i][2] *= alpha[1]; o[i][3] *= alpha[1];
+          }
+        }
+      }
+      for (int v = v_first; v <= v_last && ok; ++v) {
+        const bool ua = vh_a == v, ub = vh_b == v;
+        const uint32_t pv[4] = {ua ? pa[0] : 0u, ub ? pa[1] : 0u, ua ? pa[2] : 0u, ub ? pa[3] : 0u};
+#pragma unroll
+        for (int vs = 0; vs < VH; ++vs) {
+          if (!(ok = take())) break;
+          if (mine) {
+            const uint32_t tV = ring_u + (c % kWideSlabs) * SLAB + warp * 2048 + rv * 128;
+#pragma unroll
+            for (int d = 0; d < 4; ++d) {
+              uint32_t b0, b1, b2, b3;
+              ldsm_x4_t(tV + (((d * 2 + (lane >> 4)) ^ (rv & 7)) << 4), b0, b1, b2, b3);
+              mma_bf16_16816(o[vs * 8 + 2 * d], pv, b0, b1);
+              mma_bf16_16816(o[vs * 8 + 2 * d + 1], pv, b2, b3);
+            }
+          }
+          give();
+        }
+      }
+    }
+#pragma unroll
+    for (int h = 0; h < 2; ++h) {
+      l_run[h] += __shfl_xor_sync(0xffffffffu, l_run[h], 1);
+      l_run[h] += __shfl_xor_sync(0xffffffffu, l_run[h], 2);
+    }
+  }
+  __syncthreads();   // ring no longer needed: reuse it for the merge
+
+  float* sO = reinterpret_cast<float*>(ring);     // [4][16][DV]
+  float* sM = sO + 4 * 16 * DV;                   // [4][16]
+  float* sL = sM + 64;
+  if (warp < 4) {
+#pragma unroll
+    for (int i = 0; i < DV / 8; ++i) {
+      const int col = i * 8 + (lane & 3) * 2;
+      *reinterpret_cast<float2*>(sO + (warp * 16 + row_a) * DV + col) = make_float2(o[i][0], o[i][1]);
+      *reinterpret_cast<float2*>(sO + (warp * 16 + row_b) * DV + col) = make_float2(o[i][2], o[i][3]);
+    }
+    if ((lane & 3) == 0) {
+      sM[warp * 16 + row_a] = m_run[0]; sL[warp * 16 + row_a] = l_run[0];
+      sM[warp * 16 + row_b] = m_run[1]; sL[warp * 16 + row_b] = l_run[1];
+    }
+  }
+  __syncthreads();
+  if (warp == 4) return;
+  for (int r = warp; r < rows; r += 4) {
+    const float m = fmaxf(fmaxf(sM[r], sM[16 + r]), fmaxf(sM[32 + r], sM[48 + r]));
+    float w[4], l = 0.f;
+#pragma unroll
+    for (int j = 0; j < 4; ++j) {
+      w[j] = sM[16 * j + r] == -INFINITY ? 0.f : exp2f(sM[16 * j + r] - m);
+      l += w[j] * sL[16 * j + r];
+    }
+    const int hq = (row0 + r) % p.n_q;
+    float den = l;                                // the sink joins once: here, or in the merge of the splits
+    if (p.sinks && p.num_splits == 1 && m != -INFINITY) den += exp2f(p.sinks[hq] * kL2e - m);
+    const float inv = den > 0.f ? 1.f / den : 0.f;
+    const size_t tok = size_t(q_start + (row0 + r) / p.n_q);
+    for (int col = lane * 2; col < dv; col += 64) {
+      float a = 0.f, b = 0.f;
+#pragma unroll
+      for (int j = 0; j < 4; ++j) {
+        a += w[j] * sO[(16 * j + r) * DV + col];
+        b += w[j] * sO[(16 * j + r) * DV + col + 1];
+      }
+      if (p.num_splits == 1)
+        *reinterpret_cast<uint32_t*>(p.out + tok * (size_t(p.n_q) * dv) + hq * dv + col) = pack_bf16x2(a * inv, b * inv);
+      else
+        *reinterpret_cast<float2*>(p.part_o + ((tok * p.n_q + hq) * p.num_splits + split) * dv + col) = make_float2(a * inv, b * inv);
+    }
+    if (p.num_splits > 1 && lane == 0)
+      p.part_lse[(tok * p.n_q + hq) * p.num_splits + split] = (l > 0.f) ? m + log2f(l) : -INFINITY;
+  }
+}
+
+template <int DV>
+static int launch_wide(const CUtensorMap* tk, const CUtensorMap* tv, const DecParams& p, int max_q, cudaStream_t st) {
+  const int KS = (p.dk + 63) / 64;
+  const size_t smem = size_t(kWideSlabs) * kTile * 128 + size_t(16) * KS * 128 + sizeof(WideDecBarriers) + 1024;
+  if (smem > 227 * 1024) return -3;
+  cudaFuncSetAttribute(decode_attn_wide_kernel<DV>, cudaFuncAttributeMaxDynamicSharedMemorySize, int(smem));
+  const dim3 grid(p.seq_end - p.seq_begin, (p.n_q * max_q + 15) / 16, p.num_splits);
+  decode_attn_wide_kernel<DV><<<grid, 160, smem, st>>>(*tk, *tv, p, KS);
+  return cudaGetLastError() == cudaSuccess ? 0 : -1;
+}
+
 }  // namespace xl_dec
 
 using namespace xl_dec;
@@ -675,7 +956,9 @@ XL_API int xl_decode_attention_ext(const void* q, const void* k_cache, const voi
   if (maps < 1 || maps > 2 || (maps == 2 && (!mix || shared_keys || (n_q / n_kv) % 2))) return -2;
   if (dk < 8 || dk % 8) return -3;
   dk *= maps;                                  // the keys of both maps lie side by side
-  if (dk > 256 || dv < 8 || dv > 256 || dv % 8 || v_pitch % 8) return -3;
+  // keys that all heads share may be wider, without the other score extensions
+  const bool wide_keys = shared_keys && dk > 128 && dv <= 128 && !slopes && softcap <= 0.f && chunk <= 0 && keep_first <= 0;
+  if ((dk > 256 && !wide_keys) || dv < 8 || dv > 256 || dv % 8 || v_pitch % 8) return -3;
   if (block_size % 16 != 0 || (block_size > 64 && block_size % 64 != 0) || (block_size < 64 && 64 % block_size != 0)) return -3;
   if (n_q % n_kv) return -3;
   if ((q_stride % 8) || (reinterpret_cast<uintptr_t>(q) & 15)) return -3;
@@ -721,7 +1004,8 @@ XL_API int xl_decode_attention_ext(const void* q, const void* k_cache, const voi
   cudaStream_t st = static_cast<cudaStream_t>(stream);
   const dim3 grid(seq_end - seq_begin, n_kv * p.row_blocks, p.num_splits);
   int rc;
-  if (dv > 128) rc = launch_ext<256, 256>(tk, tv, p, grid, st);
+  if (wide_keys) rc = dv > 64 ? launch_wide<128>(tk, tv, p, max_q < 1 ? 1 : max_q, st) : launch_wide<64>(tk, tv, p, max_q < 1 ? 1 : max_q, st);
+  else if (dv > 128) rc = launch_ext<256, 256>(tk, tv, p, grid, st);
   else if (dk > 128) rc = launch_ext<256, 128>(tk, tv, p, grid, st);
   else if (dk > 64) rc = dv > 64 ? launch_ext<128, 128>(tk, tv, p, grid, st) : launch_ext<128, 64>(tk, tv, p, grid, st);
   else rc = dv > 64 ? launch_ext<64, 128>(tk, tv, p, grid, st) : launch_ext<64, 64>(tk, tv, p, grid, st);

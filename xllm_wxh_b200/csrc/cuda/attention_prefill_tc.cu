@@ -635,6 +635,415 @@ prefill_attn_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_con
   }
 }
 
+// ---------------------------------------------------------------- one wide key head for all query heads
+// Query rows of up to hundreds of columns against one key head (scores that are mixed over the heads: the keys of all key heads lie
+// side by side), values of n_kv heads.  One CTA = (sequence, 128 query rows, query head); key tiles of 128, so that a product is
+// 128 x 128 x 16 (its issue, not its arithmetic, is what a product of this size costs).  The first QR slabs of the query rows stay in
+// shared memory, any further ones pass through the ring beside their key slabs.  The ring's units are [128 tokens or rows][64
+// columns]; they come in the order of use: K(j + 1), V(j).  Roles, softmax and waits as in the kernel above, with one softmax group.
+constexpr int WKV = 128;                       // kv tokens per tile
+constexpr int W_UNIT = 128 * 128;              // 16 KB
+template <int QR> struct WideCfg {
+  static constexpr int kUnits = QR == 8 ? 4 : 8;                      // even: a pair of V units never wraps
+  static constexpr int kSmem = (QR + 2 + kUnits) * W_UNIT;            // query slabs, P, ring
+  static constexpr int kThreads = 192;
+};
+struct WideBarriers {
+  uint64_t q_full;
+  uint64_t full[8];
+  uint64_t empty[8];
+  uint64_t s_full[2];
+  uint64_t s_free[2];
+  uint64_t p_full;
+  uint64_t pv_done;
+  uint32_t tmem_base;
+  int last_split;
+};
+
+template <int QR>
+__global__ void __launch_bounds__(192, 1)
+prefill_attn_wide_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__ CUtensorMap tmK, const __grid_constant__ CUtensorMap tmV,
+                         const Params p, const int KS) {
+  constexpr int U = WideCfg<QR>::kUnits;
+  constexpr int DV = 128;
+  extern __shared__ __align__(1024) uint8_t smem[];
+  if (smem_u32(smem) & 1023u) {
+    if (threadIdx.x == 0) atomicExch(p.status, XL_ERR_BOUNDS);
+    return;
+  }
+  uint8_t* sQ = smem;
+  uint8_t* sP = sQ + QR * W_UNIT;
+  uint8_t* ring = sP + 2 * W_UNIT;
+  WideBarriers* bars = reinterpret_cast<WideBarriers*>(ring + U * W_UNIT);
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  const int head = blockIdx.y, vh = head / (p.n_q / p.n_kv);
+
+  int tile = int(gridDim.x) - 1 - int(blockIdx.x), seq = -1, q_start = 0, q_len = 0, tile_ord = 0;
+  {
+    const int sb = p.dyn_begin ? *p.dyn_begin : p.seq_begin;
+    const int se = p.dyn_end ? *p.dyn_end : p.seq_end;
+    int total = 0;
+    for (int s = sb; s < se; ++s) total += (p.q_cu[s + 1] - p.q_cu[s] + BQ - 1) / BQ;
+    tile -= int(gridDim.x) - total;
+    if (tile < 0) return;
+    tile_ord = tile;
+    for (int s = sb; s < se; ++s) {
+      const int a = p.q_cu[s], b = p.q_cu[s + 1];
+      const int nt = (b - a + BQ - 1) / BQ;
+      if (tile < nt) { seq = s; q_start = a; q_len = b - a; break; }
+      tile -= nt;
+    }
+  }
+  if (seq < 0) return;
+  const int kv_len = p.kv_lens[seq];
+  const int q0 = tile * BQ;
+  const int rows = min(BQ, q_len - q0);
+  const int pos0 = kv_len - q_len + q0;
+  const int kv_end = min(kv_len, pos0 + rows);
+  const int kv_begin = p.window > 0 ? max(0, pos0 - p.window + 1) / WKV * WKV : 0;
+  const int n_all = (kv_end - kv_begin + WKV - 1) / WKV;
+  int n_splits = 1;
+  if (p.splits > 1 && tile_ord < p.ws_tiles) n_splits = max(1, min(p.splits, n_all / p.min_tiles));
+  if (int(blockIdx.z) >= n_splits) return;
+  const int share = (n_all + n_splits - 1) / n_splits;
+  const int j_first = int(blockIdx.z) * share;
+  const int n_tiles = max(0, min(n_all, j_first + share) - j_first);
+  const int* bt = p.block_tables + size_t(seq) * p.max_blocks;
+  if (n_tiles > 0) {
+
+  if (threadIdx.x == 0) {
+    mbar_init(&bars->q_full, 1);
+    for (int u = 0; u < U; ++u) {
+      mbar_init(&bars->full[u], 1);
+      mbar_init(&bars->empty[u], 1);
+    }
+    for (int b = 0; b < 2; ++b) {
+      mbar_init(&bars->s_full[b], 1);
+      mbar_init(&bars->s_free[b], 4);
+    }
+    mbar_init(&bars->p_full, 4);
+    mbar_init(&bars->pv_done, 1);
+    mbar_fence_init();
+  }
+  if (warp == 1) {
+    tmem_alloc(&bars->tmem_base, 512);
+    tmem_relinquish();
+  }
+  tc_fence_before();
+  __syncthreads();
+  tc_fence_after();
+  const uint32_t tmem_base = bars->tmem_base;             // S buffers at 0 and 128, O at 256
+
+  if (warp == 0) {
+    // ------------------------------------------------------------ TMA producer (whole warp: lanes share a unit's boxes)
+    const int boxes = WKV / p.box_tokens;                 // per unit: 2, 4 or 8
+    if (lane == 0) {
+      prefetch_tmap(&tmQ);
+      prefetch_tmap(&tmK);
+      prefetch_tmap(&tmV);
+      const int kept = min(QR, KS);
+      mbar_arrive_expect_tx(&bars->q_full, kept * W_UNIT);
+      for (int sl = 0; sl < kept; ++sl) tma_load_3d(sQ + sl * W_UNIT, &tmQ, &bars->q_full, sl * 64, head, q_start + q0);
+    }
+    auto slot_of = [&](int j) {                           // cache slot of this lane's box of tile j
+      if (lane >= boxes) return 0;
+      const int tok = kv_begin + (j_first + j) * WKV + lane * p.box_tokens;
+      const int bi = min(tok / p.block_size, p.max_blocks - 1);
+      const long slot = long(bt[bi]) * p.block_size + tok % p.block_size;
+      return slot < 0 || slot + p.box_tokens > p.num_slots ? 0 : int(slot);
+    };
+    int c = 0;
+    bool ok = true;
+    // one unit: map 0 = query rows, 1 = keys, 2 = values
+    auto put = [&](int map, int slab, int slot) {
+      const int u = c % U;
+      if (lane == 0) {
+        if (!mbar_wait(&bars->empty[u], ((c / U) & 1) ^ 1)) {
+          atomicExch(p.status, XL_ERR_WAIT_EMPTY);
+          ok = false;
+        } else {
+          mbar_arrive_expect_tx(&bars->full[u], W_UNIT);
+        }
+      }
+      ok = __shfl_sync(0xffffffffu, ok, 0);
+      if (!ok) return false;
+      uint8_t* dst = ring + u * W_UNIT;
+      if (map == 0) {
+        if (lane == 0) tma_load_3d(dst, &tmQ, &bars->full[u], slab * 64, head, q_start + q0);
+      } else if (lane < boxes) {
+        tma_load_3d(dst + lane * p.box_tokens * 128, map == 1 ? &tmK : &tmV, &bars->full[u], slab * 64, map == 1 ? 0 : vh, slot);
+      }
+      __syncwarp();
+      ++c;
+      return true;
+    };
+    int slot = slot_of(0), slot_v = 0;
+    for (int j = 0; j <= n_tiles && ok; ++j) {
+      const int next = j + 1 < n_tiles ? slot_of(j + 1) : 0;
+      if (j < n_tiles)
+        for (int s = 0; s < KS && ok; ++s) {
+          if (s >= QR && !put(0, s, 0)) break;
+          put(1, s, slot);
+        }
+      if (j > 0 && ok && put(2, 0, slot_v)) put(2, 1, slot_v);
+      slot_v = slot;
+      slot = next;
+    }
+  } else if (warp == 1) {
+    // ------------------------------------------------------------ MMA issuer
+    if (elect_one_sync()) {
+      const uint32_t idesc_s = umma_idesc_f16(BQ, WKV, 1);
+      const uint32_t idesc_o = umma_idesc_f16(BQ, DV, 1) | (1u << 16);      // B operand (V) is MN-major
+      const uint32_t q_addr = smem_u32(sQ), p_addr = smem_u32(sP), r_addr = smem_u32(ring);
+      int c = 0;
+      bool ok = mbar_wait(&bars->q_full, 0);
+      if (!ok) atomicExch(p.status, XL_ERR_WAIT_FULL);
+      auto take = [&](int i) -> bool {                    // unit i has arrived
+        if (mbar_wait(&bars->full[i % U], (i / U) & 1)) return true;
+        atomicExch(p.status, XL_ERR_WAIT_FULL);
+        return false;
+      };
+      for (int j = 0; j <= n_tiles && ok; ++j) {
+        if (j < n_tiles) {
+          const int b = j & 1;
+          if (!mbar_wait(&bars->s_free[b], ((j >> 1) & 1) ^ 1)) {
+            atomicExch(p.status, XL_ERR_WAIT_TMEM_EMPTY);
+            ok = false;
+            break;
+          }
+          tc_fence_after();
+          for (int s = 0; s < KS && ok; ++s) {
+            uint32_t a = q_addr + s * W_UNIT;
+            int cq = -1;
+            if (s >= QR) {
+              cq = c++;
+              if (!(ok = take(cq))) break;
+              a = r_addr + (cq % U) * W_UNIT;
+            }
+            if (!(ok = take(c))) break;
+            const uint32_t k = r_addr + (c % U) * W_UNIT;
+            tc_fence_after();
+#pragma unroll
+            for (int i = 0; i < 4; ++i)
+              tc_mma_f16(tmem_base + b * 128, umma_desc_sw128(a, i * 32), umma_desc_sw128(k, i * 32), idesc_s, (s | i) != 0);
+            if (cq >= 0) tc_commit(&bars->empty[cq % U]);
+            tc_commit(&bars->empty[c % U]);
+            ++c;
+          }
+          if (!ok) break;
+          tc_commit(&bars->s_full[b]);
+        }
+        if (j > 0) {
+          if (!mbar_wait(&bars->p_full, (j - 1) & 1)) {
+            atomicExch(p.status, XL_ERR_WAIT_TMEM_FULL);
+            ok = false;
+            break;
+          }
+          if (!(ok = take(c) && take(c + 1))) break;
+          tc_fence_after();
+          const uint32_t v = r_addr + (c % U) * W_UNIT;   // two units side by side
+#pragma unroll
+          for (int i = 0; i < WKV / 16; ++i)
+            tc_mma_f16(tmem_base + 256, umma_desc_sw128(p_addr + (i >> 2) * W_UNIT, (i & 3) * 32), umma_desc_sw128_mn(v + i * 2048, W_UNIT, 1024),
+                       idesc_o, ((j - 1) | i) != 0);
+          tc_commit(&bars->pv_done);
+          tc_commit(&bars->empty[c % U]);
+          tc_commit(&bars->empty[(c + 1) % U]);
+          c += 2;
+        }
+      }
+    }
+  } else {
+    // ------------------------------------------------------------ softmax / correction / epilogue: one row per thread
+    const int q = warp & 3;
+    const int r = q * 32 + lane;
+    const uint32_t t_s = tmem_base + (uint32_t(q * 32) << 16);
+    const uint32_t t_o = t_s + 256;
+    const int pos = pos0 + r;
+    const int hi = min(pos, kv_len - 1);
+    const int lo = p.window > 0 ? max(0, pos - p.window + 1) : 0;
+    const int lo_win = p.window > 0 ? pos0 + BQ - p.window : 0;              // first key in every row's window
+    const float sc = p.scale_log2;
+    float m_ref = -INFINITY, l_run = 0.f;
+    bool ok = true;
+    for (int j = 0; j < n_tiles && ok; ++j) {
+      const int b = j & 1;
+      if (!__all_sync(0xffffffffu, mbar_wait(&bars->s_full[b], (j >> 1) & 1))) {
+        if (lane == 0) atomicExch(p.status, XL_ERR_WAIT_TMEM_FULL);
+        ok = false;
+        break;
+      }
+      tc_fence_after();
+      uint32_t raw[4][32];
+#pragma unroll
+      for (int i = 0; i < 4; ++i) tmem_ld_32x32(t_s + b * 128 + i * 32, raw[i]);
+      tc_wait_ld();
+      tc_fence_before();
+      __syncwarp();
+      if (lane == 0) mbar_arrive(&bars->s_free[b]);
+      float (&v)[128] = *reinterpret_cast<float (*)[128]>(raw);
+      const int kv0 = kv_begin + (j_first + j) * WKV;
+      if (kv0 + WKV - 1 > pos0 || kv0 + WKV > kv_len || kv0 < lo_win) {
+#pragma unroll
+        for (int c = 0; c < 128; ++c)
+          if (kv0 + c > hi || kv0 + c < lo) v[c] = -INFINITY;
+      }
+      float mx8[8];
+#pragma unroll
+      for (int i = 0; i < 8; ++i) mx8[i] = v[i];
+#pragma unroll
+      for (int c = 8; c < 128; ++c) mx8[c & 7] = fmaxf(mx8[c & 7], v[c]);
+      const float mx = fmaxf(fmaxf(fmaxf(mx8[0], mx8[1]), fmaxf(mx8[2], mx8[3])), fmaxf(fmaxf(mx8[4], mx8[5]), fmaxf(mx8[6], mx8[7])));
+      const bool had = m_ref != -INFINITY;
+      const bool grow = (mx - m_ref) * sc > 8.f || (!had && mx != -INFINITY);
+      const float m_new = grow ? mx : m_ref;
+      const bool rescale = grow && had;
+      const float alpha = rescale ? fast_exp2((m_ref - m_new) * sc) : 1.f;
+      m_ref = m_new;
+      const float mneg = (m_ref == -INFINITY) ? 0.f : -m_ref * sc;
+      float sum4[4] = {0.f, 0.f, 0.f, 0.f};
+      uint32_t pk[64];
+#pragma unroll
+      for (int c = 0; c < 128; c += 2) {
+        const float e0 = fast_exp2(fmaf(v[c], sc, mneg)), e1 = fast_exp2(fmaf(v[c + 1], sc, mneg));
+        sum4[(c >> 1) & 3] += e0 + e1;
+        pk[c >> 1] = pack_bf16x2(e0, e1);
+      }
+      l_run = l_run * alpha + ((sum4[0] + sum4[1]) + (sum4[2] + sum4[3]));
+      // P and O are touched only after P V of the previous tile has finished
+      if (j > 0 && !__all_sync(0xffffffffu, mbar_wait(&bars->pv_done, (j - 1) & 1))) {
+        if (lane == 0) atomicExch(p.status, XL_ERR_WAIT_TMEM_EMPTY);
+        ok = false;
+        break;
+      }
+      tc_fence_after();
+      if (j > 0 && __any_sync(0xffffffffu, rescale)) {
+#pragma unroll
+        for (int c = 0; c < DV; c += 32) {
+          uint32_t o[32];
+          tmem_ld_32x32(t_o + c, o);
+          tc_wait_ld();
+#pragma unroll
+          for (int i = 0; i < 32; ++i) o[i] = __float_as_uint(__uint_as_float(o[i]) * alpha);
+          tmem_st_32x32(t_o + c, o);
+        }
+        tc_wait_st();
+      }
+#pragma unroll
+      for (int g = 0; g < 2; ++g) {
+        uint8_t* prow = sP + g * W_UNIT + r * 128;
+#pragma unroll
+        for (int c = 0; c < 8; ++c)
+          *reinterpret_cast<uint4*>(prow + ((c ^ (r & 7)) << 4)) =
+              make_uint4(pk[g * 32 + 4 * c], pk[g * 32 + 4 * c + 1], pk[g * 32 + 4 * c + 2], pk[g * 32 + 4 * c + 3]);
+      }
+      fence_proxy_async_smem();
+      tc_fence_before();
+      __syncwarp();
+      if (lane == 0) mbar_arrive(&bars->p_full);
+    }
+    if (ok && !__all_sync(0xffffffffu, mbar_wait(&bars->pv_done, (n_tiles - 1) & 1))) {
+      if (lane == 0) atomicExch(p.status, XL_ERR_WAIT_TMEM_EMPTY);
+      ok = false;
+    }
+    if (ok && n_splits > 1) {
+      tc_fence_after();
+      const size_t unit = size_t(tile_ord) * gridDim.y + blockIdx.y;
+      float4* wo = reinterpret_cast<float4*>(p.ws_o) + (unit * p.splits + blockIdx.z) * (DV / 4) * BQ;
+#pragma unroll
+      for (int c = 0; c < DV; c += 32) {
+        uint32_t o[32];
+        tmem_ld_32x32(t_o + c, o);
+        tc_wait_ld();
+#pragma unroll
+        for (int i = 0; i < 8; ++i)
+          wo[size_t(c / 4 + i) * BQ + r] = make_float4(__uint_as_float(o[4 * i]), __uint_as_float(o[4 * i + 1]),
+                                                       __uint_as_float(o[4 * i + 2]), __uint_as_float(o[4 * i + 3]));
+      }
+      p.ws_ml[(unit * p.splits + blockIdx.z) * BQ + r] = make_float2(m_ref == -INFINITY ? -INFINITY : m_ref * sc, l_run);
+      __threadfence();
+    } else if (ok) {
+      tc_fence_after();
+      if (p.sinks && m_ref != -INFINITY) l_run += fast_exp2(p.sinks[head] * 1.4426950408889634f - m_ref * sc);
+      const float inv = l_run > 0.f ? 1.f / l_run : 0.f;
+      __nv_bfloat16* dst = p.out + size_t(q_start + q0 + r) * (size_t(p.n_q) * p.dv) + size_t(head) * p.dv;
+#pragma unroll
+      for (int c = 0; c < DV; c += 32) {
+        uint32_t o[32];
+        tmem_ld_32x32(t_o + c, o);
+        tc_wait_ld();
+        if (r < rows) {
+#pragma unroll
+          for (int i = 0; i < 4; ++i) {
+            uint32_t w[4];
+#pragma unroll
+            for (int e = 0; e < 4; ++e)
+              w[e] = pack_bf16x2(__uint_as_float(o[8 * i + 2 * e]) * inv, __uint_as_float(o[8 * i + 2 * e + 1]) * inv);
+            if (c + 8 * i < p.dv) *reinterpret_cast<uint4*>(dst + c + 8 * i) = make_uint4(w[0], w[1], w[2], w[3]);
+          }
+        }
+      }
+    }
+  }
+  tc_fence_before();
+  __syncthreads();
+  if (warp == 1) tmem_dealloc(tmem_base, 512);
+  }  // n_tiles > 0
+  if (n_splits == 1) return;
+
+  // ---------------------------------------------------------------- merge of the key splits by the last arrival
+  if (threadIdx.x == 0) {
+    __threadfence();
+    int* cnt = p.ws_cnt + size_t(tile_ord) * gridDim.y + blockIdx.y;
+    const int prev = atomicAdd(cnt, 1);
+    bars->last_split = prev == n_splits - 1;
+    if (prev == n_splits - 1) *cnt = 0;
+  }
+  __syncthreads();
+  if (!bars->last_split || warp < 2) return;
+  __threadfence();
+  const int r = (warp & 3) * 32 + lane;
+  const int n_valid = (n_all + share - 1) / share;          // splits that had keys to look at
+  const size_t unit = size_t(tile_ord) * gridDim.y + blockIdx.y;
+  const float2* ml = p.ws_ml + unit * p.splits * BQ + r;
+  float w[8], m_all = -INFINITY, l_all = 0.f;
+#pragma unroll
+  for (int z = 0; z < 8; ++z) {
+    w[z] = 0.f;
+    if (z < n_valid) {
+      const float2 x = __ldcg(ml + size_t(z) * BQ);
+      if (x.y > 0.f) m_all = fmaxf(m_all, x.x);
+    }
+  }
+#pragma unroll
+  for (int z = 0; z < 8; ++z) {
+    if (z < n_valid) {
+      const float2 x = __ldcg(ml + size_t(z) * BQ);
+      w[z] = x.y > 0.f ? fast_exp2(x.x - m_all) : 0.f;
+      l_all += w[z] * x.y;
+    }
+  }
+  if (p.sinks && m_all != -INFINITY) l_all += fast_exp2(p.sinks[head] * 1.4426950408889634f - m_all);
+  const float inv = l_all > 0.f ? 1.f / l_all : 0.f;
+  if (r >= rows) return;
+  const float4* wo = reinterpret_cast<const float4*>(p.ws_o) + unit * p.splits * (DV / 4) * BQ + r;
+  __nv_bfloat16* dst = p.out + size_t(q_start + q0 + r) * (size_t(p.n_q) * p.dv) + size_t(head) * p.dv;
+  for (int c4 = 0; c4 < p.dv / 4; c4 += 2) {
+    float a[8] = {};
+#pragma unroll
+    for (int z = 0; z < 8; ++z) {
+      if (z < n_valid && w[z] != 0.f) {
+        const float4 x = __ldcg(wo + (size_t(z) * (DV / 4) + c4) * BQ), y = __ldcg(wo + (size_t(z) * (DV / 4) + c4 + 1) * BQ);
+        const float f[8] = {x.x, x.y, x.z, x.w, y.x, y.y, y.z, y.w};
+#pragma unroll
+        for (int e = 0; e < 8; ++e) a[e] += w[z] * f[e];
+      }
+    }
+    *reinterpret_cast<uint4*>(dst + c4 * 4) = make_uint4(pack_bf16x2(a[0] * inv, a[1] * inv), pack_bf16x2(a[2] * inv, a[3] * inv),
+                                                        pack_bf16x2(a[4] * inv, a[5] * inv), pack_bf16x2(a[6] * inv, a[7] * inv));
+  }
+}
+
 // Workspace of the KV split: one allocation per device, made at the first use outside a stream capture.
 constexpr size_t kSplitWsBytes = size_t(64) << 20;
 constexpr size_t kSplitCntBytes = size_t(1) << 16;
@@ -655,6 +1064,36 @@ static uint8_t* split_workspace(cudaStream_t stream) {
   return ws[dev];
 }
 
+// Key splits of a launch with heads_per_cta heads per CTA, key tiles and value columns of the given sizes.
+static void plan_splits(Params& p, int heads_per_cta, int dv_cols, int min_tiles, int q_tiles_cap, int total_q_rows, cudaStream_t stream) {
+  // Few query tiles x heads (short prompts against a long context, or a tensor-parallel shard with a handful of heads)
+  // leave most SMs idle while the busiest CTA walks its whole key range alone: cut key ranges into up to 8 splits.  The
+  // grid only offers the splits; every tile takes as many as its own key range is worth (`min_tiles` key tiles each).
+  const int tiles_est = (total_q_rows + BQ - 1) / BQ;                 // q_tiles_cap also counts one spare tile per sequence
+  const int ctas = (tiles_est > 0 ? tiles_est : 1) * (p.n_q / heads_per_cta);
+  int splits = 1;
+  if (g_kv_split > 1) splits = g_kv_split;
+  else if (g_kv_split == 1 && ctas * 2 <= xl_host::sm_count()) splits = xl_host::sm_count() / ctas;
+  if (splits > 8) splits = 8;
+  p.splits = 1;
+  p.min_tiles = g_kv_split > 1 ? 1 : min_tiles;
+  p.ws_tiles = 0;
+  if (splits > 1) {
+    uint8_t* w = split_workspace(stream);
+    const size_t per_tile = size_t(p.n_q) * splits * (size_t(BQ) * dv_cols * 4 + size_t(BQ) * 8);
+    size_t tiles = kSplitWsBytes / per_tile;
+    const size_t cnt_cap = kSplitCntBytes / 4 / size_t(p.n_q / heads_per_cta);
+    if (tiles > cnt_cap) tiles = cnt_cap;
+    if (w && tiles > 0) {
+      p.splits = splits;
+      p.ws_tiles = int(tiles < size_t(q_tiles_cap) ? tiles : size_t(q_tiles_cap));
+      p.ws_o = reinterpret_cast<float*>(w);
+      p.ws_ml = reinterpret_cast<float2*>(w + size_t(p.ws_tiles) * p.n_q * splits * size_t(BQ) * dv_cols * 4);
+      p.ws_cnt = reinterpret_cast<int*>(w + kSplitWsBytes);
+    }
+  }
+}
+
 template <int NH, int QS, int VS, bool EXT, int SCORE = SCORE_RAW, int MAPS = 1>
 static int launch_prefill(const CUtensorMap* tq, const CUtensorMap* tk, const CUtensorMap* tv, const Params& p_in, int q_tiles_cap,
                           int total_q_rows, cudaStream_t stream) {
@@ -666,34 +1105,24 @@ static int launch_prefill(const CUtensorMap* tq, const CUtensorMap* tk, const CU
     set = true;
   }
   Params p = p_in;
-  // Few query tiles x heads (short prompts against a long context, or a tensor-parallel shard with a handful of heads)
-  // leave most SMs idle while the busiest CTA walks its whole key range alone: cut key ranges into up to 8 splits.  The
-  // grid only offers the splits; every tile takes as many as its own key range is worth (`min_tiles` key tiles each).
-  const int tiles_est = (total_q_rows + BQ - 1) / BQ;                 // q_tiles_cap also counts one spare tile per sequence
-  const int ctas = (tiles_est > 0 ? tiles_est : 1) * (p.n_q / NH);
-  int splits = 1;
-  if (g_kv_split > 1) splits = g_kv_split;
-  else if (g_kv_split == 1 && ctas * 2 <= xl_host::sm_count()) splits = xl_host::sm_count() / ctas;
-  if (splits > 8) splits = 8;
-  p.splits = 1;
-  p.min_tiles = g_kv_split > 1 ? 1 : 12;
-  p.ws_tiles = 0;
-  if (splits > 1) {
-    uint8_t* w = split_workspace(stream);
-    const size_t per_tile = size_t(p.n_q) * splits * (size_t(BQ) * C::DV * 4 + size_t(BQ) * 8);
-    size_t tiles = kSplitWsBytes / per_tile;
-    const size_t cnt_cap = kSplitCntBytes / 4 / size_t(p.n_q / NH);
-    if (tiles > cnt_cap) tiles = cnt_cap;
-    if (w && tiles > 0) {
-      p.splits = splits;
-      p.ws_tiles = int(tiles < size_t(q_tiles_cap) ? tiles : size_t(q_tiles_cap));
-      p.ws_o = reinterpret_cast<float*>(w);
-      p.ws_ml = reinterpret_cast<float2*>(w + size_t(p.ws_tiles) * p.n_q * splits * size_t(BQ) * C::DV * 4);
-      p.ws_cnt = reinterpret_cast<int*>(w + kSplitWsBytes);
-    }
-  }
+  plan_splits(p, NH, C::DV, 12, q_tiles_cap, total_q_rows, stream);
   dim3 grid(q_tiles_cap, p.n_q / NH, p.splits);
   prefill_attn_tc_kernel<NH, QS, VS, EXT, SCORE, MAPS><<<grid, C::kThreads, smem, stream>>>(*tq, *tk, *tv, p);
+  return cudaGetLastError() == cudaSuccess ? 0 : -1;
+}
+
+template <int QR>
+static int launch_wide(const CUtensorMap* tq, const CUtensorMap* tk, const CUtensorMap* tv, const Params& p_in, int dk, int q_tiles_cap,
+                       int total_q_rows, cudaStream_t stream) {
+  const size_t smem = WideCfg<QR>::kSmem + sizeof(WideBarriers);
+  static bool set = false;
+  if (!set) {
+    cudaFuncSetAttribute(prefill_attn_wide_kernel<QR>, cudaFuncAttributeMaxDynamicSharedMemorySize, int(smem));
+    set = true;
+  }
+  Params p = p_in;
+  plan_splits(p, 1, 128, 6, q_tiles_cap, total_q_rows, stream);
+  prefill_attn_wide_kernel<QR><<<dim3(q_tiles_cap, p.n_q, p.splits), WideCfg<QR>::kThreads, smem, stream>>>(*tq, *tk, *tv, p, (dk + 127) / 128 * 2);
   return cudaGetLastError() == cudaSuccess ? 0 : -1;
 }
 
@@ -752,7 +1181,8 @@ XL_API int xl_prefill_attention_tc(const void* q, const void* k_cache, const voi
 // `slopes` / `sinks` [n_q] fp32, null when absent; `softcap` > 0: scale * q . k becomes softcap * tanh(scale * q . k / softcap), and
 // `bound` > 0 promises |q . k| <= bound.
 // `v_pitch`: elements from one cache slot's values to the next one's (0: n_kv * dv), so that values may be a part of the keys.
-// `shared_keys`: k_cache has one key head, which all query heads share, beside n_kv value heads.
+// `shared_keys`: k_cache has one key head, which all query heads share, beside n_kv value heads; it may be wider than 256 where dv <= 128
+// and the score has no other extension than window and sinks.
 // maps = 2: n_q counts the maps' heads (pairs of neighbours), k_cache has 2 n_kv heads, out [T, n_q / 2 * dv] =
 // rms(first - mix[0] * second, mix_eps) * mix_mult.  Returns -3 when the shape, or a distance bias beside bounded scores or two
 // maps, is not covered.
@@ -765,7 +1195,9 @@ XL_API int xl_prefill_attention_ext(const void* q, const void* k_cache, const vo
   using namespace xl_pf;
   if (maps < 1 || maps > 2 || (maps == 2 && (!mix || shared_keys || (n_q / n_kv) % 2))) return -2;
   const int d_max = maps == 2 ? 128 : 256;
-  if (dk < 8 || dk > d_max || dk % 8 || dv < 8 || dv > d_max || dv % 8) return -3;
+  // keys that all heads share may be wider, without the other score extensions
+  const bool wide_keys = shared_keys && dk > 128 && dv <= 128 && !slopes && softcap <= 0.f && chunk <= 0 && keep_first <= 0;
+  if (dk < 8 || (dk > d_max && !wide_keys) || dk % 8 || dv < 8 || dv > d_max || dv % 8) return -3;
   if (v_pitch % 8 || (slopes && (softcap > 0.f || maps == 2))) return -3;
   if (chunk > 0 && keep_first > 0) return -2;
   if (block_size % 16 != 0 || (block_size > 64 && block_size % 64 != 0) || (block_size < 64 && 64 % block_size != 0)) return -3;
@@ -811,6 +1243,8 @@ XL_API int xl_prefill_attention_ext(const void* q, const void* k_cache, const vo
   p.window = window;
   p.status = xl_host::status_word();
   cudaStream_t st = static_cast<cudaStream_t>(stream);
+  if (wide_keys)
+    return dk > 256 ? launch_wide<8>(tq, tk, tv, p, dk, q_tiles_cap, total_q_rows, st) : launch_wide<4>(tq, tk, tv, p, dk, q_tiles_cap, total_q_rows, st);
   const bool pair = (n_q / n_kv) % 2 == 0, k2 = dk > 64, v2 = dv > 64, wide = dk > 128 || dv > 128;
 #define XL_PF_EXT(...) launch_prefill<__VA_ARGS__>(tq, tk, tv, p, q_tiles_cap, total_q_rows, st)
   if (maps == 2) {

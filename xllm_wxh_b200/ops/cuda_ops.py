@@ -807,7 +807,9 @@ def paged_attention_ext(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.T
                                        c_float(softcap), *last, _f32flag(q), _stream()), "xl_attention_simt")
         return out
     most = 256 if mix is None else 128
-    if q.dtype == torch.float32 or dk % 8 or dv % 8 or dk > most or dv > most or q.stride(1) != dk:
+    plain = slopes is None and softcap <= 0 and chunk <= 0 and keep_first <= 0
+    wide = shared_keys and dk > 128 and dv <= 128 and plain                  # kernels of their own, for keys of any width
+    if q.dtype == torch.float32 or dk % 8 or dv % 8 or (dk > most and not wide) or dv > most or q.stride(1) != dk:
         launch_count += 1
         return simt()
     hdr = getattr(inp, "header_dev", None)
@@ -822,7 +824,7 @@ def paged_attention_ext(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.T
         if window > 0:
             max_kv = min(max_kv, window + keep_first)
         max_q = max(1, inp.max_q) if inp.n_spec > 0 else 1
-        splits = decode_splits(n_dec, n_kv * -(-Hq // n_kv * max_q // 16), max_kv)
+        splits = decode_splits(n_dec, -(-Hq * max_q // 16) if wide else n_kv * -(-Hq // n_kv * max_q // 16), max_kv)
         po = pl = None
         rows = max(T, n_dec)
         if splits > 1:
