@@ -60,7 +60,7 @@ def parse():
     p.add_argument("--tp-mlp-mode", type=str, default="auto", choices=["auto", "tp", "rows"],
                    help="dense MLP under tensor parallelism: sharded weights (tp), replicated weights run by rows, or auto")
     p.add_argument("--compare-design", type=str, default="", help="instead of the serving workload: prefill and decode throughput of a "
-                   "model design's layers and its kernels, beside the closest other model at equal sizes (movolorn, falalix, babadra)")
+                   "model design's layers and its kernels, beside the closest other model at equal sizes (movolorn, falalix, babadra, govuvik)")
     p.add_argument("--seed", type=int, default=0)
     return p.parse_args()
 

@@ -637,31 +637,46 @@ prefill_attn_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_con
 
 // ---------------------------------------------------------------- one wide key head for all query heads
 // Query rows of up to hundreds of columns against one key head (scores that are mixed over the heads: the keys of all key heads lie
-// side by side), values of n_kv heads.  One CTA = (sequence, 128 query rows, query head); key tiles of 128, so that a product is
-// 128 x 128 x 16 (its issue, not its arithmetic, is what a product of this size costs).  The first QR slabs of the query rows stay in
-// shared memory, any further ones pass through the ring beside their key slabs.  The ring's units are [128 tokens or rows][64
-// columns]; they come in the order of use: K(j + 1), V(j).  Roles, softmax and waits as in the kernel above, with one softmax group.
-constexpr int WKV = 128;                       // kv tokens per tile
-constexpr int W_UNIT = 128 * 128;              // 16 KB
+// side by side), values of n_kv heads.  One CTA = (sequence, 128 query rows, query head).  A product costs nearly as much to issue as to
+// compute at these sizes, so key tiles are 256 wide (S is one 128 x 256 accumulator) and P goes back into tensor memory, from where
+// O += P V takes it as its first operand; that leaves shared memory to the query rows, whose first QR slabs stay there (further ones
+// pass through the ring beside their key slabs).  Ring units of 32 KB in the order of use, K(j + 1) ahead of V(j): [256 tokens][64
+// columns] of keys or [128 tokens][128 columns] of values.  Two softmax groups share a row: each takes half of its keys, and half of the
+// columns of O; they exchange maxima and sums through shared memory.  S(j + 1) may be issued once both have read S(j), which P V of the
+// tile before covers.  Roles and waits are those of the kernel above; a group whose wait ran out goes on without waiting, so that the
+// other one still meets it at the barriers.
+constexpr int WKV = 256;                       // kv tokens per tile
+constexpr int W_SLAB = 128 * 128;              // 16 KB: [128 rows or tokens][64 columns]
+constexpr int W_UNIT = 2 * W_SLAB;
 template <int QR> struct WideCfg {
-  static constexpr int kUnits = QR == 8 ? 4 : 8;                      // even: a pair of V units never wraps
-  static constexpr int kSmem = (QR + 2 + kUnits) * W_UNIT;            // query slabs, P, ring
-  static constexpr int kThreads = 192;
+  static constexpr int kUnits = QR == 8 ? 3 : 5;
+  static constexpr int kSmem = QR * W_SLAB + kUnits * W_UNIT;          // query slabs, ring
+  static constexpr int kThreads = 320;
 };
 struct WideBarriers {
   uint64_t q_full;
-  uint64_t full[8];
-  uint64_t empty[8];
-  uint64_t s_full[2];
-  uint64_t s_free[2];
+  uint64_t full[5];
+  uint64_t empty[5];
+  uint64_t s_full;
+  uint64_t s_free;
   uint64_t p_full;
   uint64_t pv_done;
   uint32_t tmem_base;
   int last_split;
+  float row[2][2][BQ];        // [tile parity][group][row]: maxima; at the end the sums
 };
+// D[tmem] (+)= A[tmem] * B[smem desc]: row i of A in lane i, two bf16 per column
+__device__ __forceinline__ void tc_mma_f16_ts(uint32_t tmem_d, uint32_t tmem_a, uint64_t desc_b, uint32_t idesc, uint32_t accumulate) {
+  asm volatile(
+      "{\n\t.reg .pred p;\n\t"
+      "setp.ne.b32 p, %4, 0;\n\t"
+      "tcgen05.mma.cta_group::1.kind::f16 [%0], [%1], %2, %3, p;\n\t}"
+      ::"r"(tmem_d), "r"(tmem_a), "l"(desc_b), "r"(idesc), "r"(accumulate)
+      : "memory");
+}
 
 template <int QR>
-__global__ void __launch_bounds__(192, 1)
+__global__ void __launch_bounds__(320, 1)
 prefill_attn_wide_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__ CUtensorMap tmK, const __grid_constant__ CUtensorMap tmV,
                          const Params p, const int KS) {
   constexpr int U = WideCfg<QR>::kUnits;
@@ -672,8 +687,7 @@ prefill_attn_wide_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_c
     return;
   }
   uint8_t* sQ = smem;
-  uint8_t* sP = sQ + QR * W_UNIT;
-  uint8_t* ring = sP + 2 * W_UNIT;
+  uint8_t* ring = sQ + QR * W_SLAB;
   WideBarriers* bars = reinterpret_cast<WideBarriers*>(ring + U * W_UNIT);
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const int head = blockIdx.y, vh = head / (p.n_q / p.n_kv);
@@ -700,7 +714,7 @@ prefill_attn_wide_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_c
   const int rows = min(BQ, q_len - q0);
   const int pos0 = kv_len - q_len + q0;
   const int kv_end = min(kv_len, pos0 + rows);
-  const int kv_begin = p.window > 0 ? max(0, pos0 - p.window + 1) / WKV * WKV : 0;
+  const int kv_begin = p.window > 0 ? max(0, pos0 - p.window + 1) / 64 * 64 : 0;      // boxes start at multiples of at most 64 tokens
   const int n_all = (kv_end - kv_begin + WKV - 1) / WKV;
   int n_splits = 1;
   if (p.splits > 1 && tile_ord < p.ws_tiles) n_splits = max(1, min(p.splits, n_all / p.min_tiles));
@@ -708,6 +722,8 @@ prefill_attn_wide_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_c
   const int share = (n_all + n_splits - 1) / n_splits;
   const int j_first = int(blockIdx.z) * share;
   const int n_tiles = max(0, min(n_all, j_first + share) - j_first);
+  auto tile_kv = [&](int j) { return kv_begin + (j_first + j) * WKV; };
+  auto is_half = [&](int j) { return kv_end - tile_kv(j) <= WKV / 2; };               // a last tile of at most 128 keys
   const int* bt = p.block_tables + size_t(seq) * p.max_blocks;
   if (n_tiles > 0) {
 
@@ -717,11 +733,9 @@ prefill_attn_wide_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_c
       mbar_init(&bars->full[u], 1);
       mbar_init(&bars->empty[u], 1);
     }
-    for (int b = 0; b < 2; ++b) {
-      mbar_init(&bars->s_full[b], 1);
-      mbar_init(&bars->s_free[b], 4);
-    }
-    mbar_init(&bars->p_full, 4);
+    mbar_init(&bars->s_full, 1);
+    mbar_init(&bars->s_free, 8);
+    mbar_init(&bars->p_full, 8);
     mbar_init(&bars->pv_done, 1);
     mbar_fence_init();
   }
@@ -732,106 +746,115 @@ prefill_attn_wide_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_c
   tc_fence_before();
   __syncthreads();
   tc_fence_after();
-  const uint32_t tmem_base = bars->tmem_base;             // S buffers at 0 and 128, O at 256
+  const uint32_t tmem_base = bars->tmem_base;             // S at 0, O at 256, P at 384
 
   if (warp == 0) {
     // ------------------------------------------------------------ TMA producer (whole warp: lanes share a unit's boxes)
-    const int boxes = WKV / p.box_tokens;                 // per unit: 2, 4 or 8
+    const int boxes = WKV / p.box_tokens;                 // of a whole unit: 4, 8 or 16
     if (lane == 0) {
       prefetch_tmap(&tmQ);
       prefetch_tmap(&tmK);
       prefetch_tmap(&tmV);
       const int kept = min(QR, KS);
-      mbar_arrive_expect_tx(&bars->q_full, kept * W_UNIT);
-      for (int sl = 0; sl < kept; ++sl) tma_load_3d(sQ + sl * W_UNIT, &tmQ, &bars->q_full, sl * 64, head, q_start + q0);
+      mbar_arrive_expect_tx(&bars->q_full, kept * W_SLAB);
+      for (int sl = 0; sl < kept; ++sl) tma_load_3d(sQ + sl * W_SLAB, &tmQ, &bars->q_full, sl * 64, head, q_start + q0);
     }
     auto slot_of = [&](int j) {                           // cache slot of this lane's box of tile j
       if (lane >= boxes) return 0;
-      const int tok = kv_begin + (j_first + j) * WKV + lane * p.box_tokens;
+      const int tok = tile_kv(j) + lane * p.box_tokens;
       const int bi = min(tok / p.block_size, p.max_blocks - 1);
       const long slot = long(bt[bi]) * p.block_size + tok % p.block_size;
       return slot < 0 || slot + p.box_tokens > p.num_slots ? 0 : int(slot);
     };
     int c = 0;
     bool ok = true;
-    // one unit: map 0 = query rows, 1 = keys, 2 = values
-    auto put = [&](int map, int slab, int slot) {
+    auto open = [&](int bytes) {                          // unit c may be written; it will get so many bytes
       const int u = c % U;
       if (lane == 0) {
         if (!mbar_wait(&bars->empty[u], ((c / U) & 1) ^ 1)) {
           atomicExch(p.status, XL_ERR_WAIT_EMPTY);
           ok = false;
         } else {
-          mbar_arrive_expect_tx(&bars->full[u], W_UNIT);
+          mbar_arrive_expect_tx(&bars->full[u], bytes);
         }
       }
       ok = __shfl_sync(0xffffffffu, ok, 0);
-      if (!ok) return false;
-      uint8_t* dst = ring + u * W_UNIT;
-      if (map == 0) {
-        if (lane == 0) tma_load_3d(dst, &tmQ, &bars->full[u], slab * 64, head, q_start + q0);
-      } else if (lane < boxes) {
-        tma_load_3d(dst + lane * p.box_tokens * 128, map == 1 ? &tmK : &tmV, &bars->full[u], slab * 64, map == 1 ? 0 : vh, slot);
-      }
-      __syncwarp();
-      ++c;
-      return true;
+      return ok;
     };
     int slot = slot_of(0), slot_v = 0;
     for (int j = 0; j <= n_tiles && ok; ++j) {
       const int next = j + 1 < n_tiles ? slot_of(j + 1) : 0;
-      if (j < n_tiles)
-        for (int s = 0; s < KS && ok; ++s) {
-          if (s >= QR && !put(0, s, 0)) break;
-          put(1, s, slot);
+      if (j < n_tiles) {
+        const int n = is_half(j) ? boxes / 2 : boxes;
+        for (int s = 0; s < KS; ++s) {
+          if (s >= QR) {
+            if (!open(W_SLAB)) break;
+            if (lane == 0) tma_load_3d(ring + (c % U) * W_UNIT, &tmQ, &bars->full[c % U], s * 64, head, q_start + q0);
+            __syncwarp();
+            ++c;
+          }
+          if (!open(n * p.box_tokens * 128)) break;
+          if (lane < n) tma_load_3d(ring + (c % U) * W_UNIT + lane * p.box_tokens * 128, &tmK, &bars->full[c % U], s * 64, 0, slot);
+          __syncwarp();
+          ++c;
         }
-      if (j > 0 && ok && put(2, 0, slot_v)) put(2, 1, slot_v);
+      }
+      if (j > 0 && ok) {
+        const int per = boxes / 2;                        // boxes per 64-column slab of 128 tokens
+        for (int h = 0; h < (is_half(j - 1) ? 1 : 2); ++h) {
+          if (!open(W_UNIT)) break;
+          const int z = __shfl_sync(0xffffffffu, slot_v, h * per + lane % per);
+          if (lane < boxes)
+            tma_load_3d(ring + (c % U) * W_UNIT + lane / per * W_SLAB + lane % per * p.box_tokens * 128, &tmV, &bars->full[c % U], lane / per * 64, vh, z);
+          __syncwarp();
+          ++c;
+        }
+      }
       slot_v = slot;
       slot = next;
     }
   } else if (warp == 1) {
     // ------------------------------------------------------------ MMA issuer
     if (elect_one_sync()) {
-      const uint32_t idesc_s = umma_idesc_f16(BQ, WKV, 1);
       const uint32_t idesc_o = umma_idesc_f16(BQ, DV, 1) | (1u << 16);      // B operand (V) is MN-major
-      const uint32_t q_addr = smem_u32(sQ), p_addr = smem_u32(sP), r_addr = smem_u32(ring);
+      const uint32_t q_addr = smem_u32(sQ), r_addr = smem_u32(ring);
       int c = 0;
       bool ok = mbar_wait(&bars->q_full, 0);
       if (!ok) atomicExch(p.status, XL_ERR_WAIT_FULL);
-      auto take = [&](int i) -> bool {                    // unit i has arrived
-        if (mbar_wait(&bars->full[i % U], (i / U) & 1)) return true;
+      auto take = [&]() -> bool {                         // unit c has arrived
+        if (mbar_wait(&bars->full[c % U], (c / U) & 1)) return true;
         atomicExch(p.status, XL_ERR_WAIT_FULL);
         return false;
       };
       for (int j = 0; j <= n_tiles && ok; ++j) {
         if (j < n_tiles) {
-          const int b = j & 1;
-          if (!mbar_wait(&bars->s_free[b], ((j >> 1) & 1) ^ 1)) {
+          if (!mbar_wait(&bars->s_free, (j & 1) ^ 1)) {
             atomicExch(p.status, XL_ERR_WAIT_TMEM_EMPTY);
             ok = false;
             break;
           }
+          const uint32_t idesc_s = umma_idesc_f16(BQ, is_half(j) ? WKV / 2 : WKV, 1);
           tc_fence_after();
-          for (int s = 0; s < KS && ok; ++s) {
-            uint32_t a = q_addr + s * W_UNIT;
+          for (int s = 0; s < KS; ++s) {
+            uint32_t a = q_addr + s * W_SLAB;
             int cq = -1;
             if (s >= QR) {
+              if (!(ok = take())) break;
+              a = r_addr + (c % U) * W_UNIT;
               cq = c++;
-              if (!(ok = take(cq))) break;
-              a = r_addr + (cq % U) * W_UNIT;
             }
-            if (!(ok = take(c))) break;
+            if (!(ok = take())) break;
             const uint32_t k = r_addr + (c % U) * W_UNIT;
             tc_fence_after();
 #pragma unroll
             for (int i = 0; i < 4; ++i)
-              tc_mma_f16(tmem_base + b * 128, umma_desc_sw128(a, i * 32), umma_desc_sw128(k, i * 32), idesc_s, (s | i) != 0);
+              tc_mma_f16(tmem_base, umma_desc_sw128(a, i * 32), umma_desc_sw128(k, i * 32), idesc_s, (s | i) != 0);
             if (cq >= 0) tc_commit(&bars->empty[cq % U]);
             tc_commit(&bars->empty[c % U]);
             ++c;
           }
           if (!ok) break;
-          tc_commit(&bars->s_full[b]);
+          tc_commit(&bars->s_full);
         }
         if (j > 0) {
           if (!mbar_wait(&bars->p_full, (j - 1) & 1)) {
@@ -839,26 +862,29 @@ prefill_attn_wide_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_c
             ok = false;
             break;
           }
-          if (!(ok = take(c) && take(c + 1))) break;
-          tc_fence_after();
-          const uint32_t v = r_addr + (c % U) * W_UNIT;   // two units side by side
+          const int halves = is_half(j - 1) ? 1 : 2;
+          for (int h = 0; h < halves; ++h) {
+            if (!(ok = take())) break;
+            tc_fence_after();
+            const uint32_t v = r_addr + (c % U) * W_UNIT;
 #pragma unroll
-          for (int i = 0; i < WKV / 16; ++i)
-            tc_mma_f16(tmem_base + 256, umma_desc_sw128(p_addr + (i >> 2) * W_UNIT, (i & 3) * 32), umma_desc_sw128_mn(v + i * 2048, W_UNIT, 1024),
-                       idesc_o, ((j - 1) | i) != 0);
-          tc_commit(&bars->pv_done);
-          tc_commit(&bars->empty[c % U]);
-          tc_commit(&bars->empty[(c + 1) % U]);
-          c += 2;
+            for (int i = 0; i < 8; ++i)
+              tc_mma_f16_ts(tmem_base + 256, tmem_base + 384 + h * 64 + i * 8, umma_desc_sw128_mn(v + i * 2048, W_SLAB, 1024), idesc_o,
+                            ((j - 1) | h | i) != 0);
+            if (h == halves - 1) tc_commit(&bars->pv_done);
+            tc_commit(&bars->empty[c % U]);
+            ++c;
+          }
         }
       }
     }
   } else {
-    // ------------------------------------------------------------ softmax / correction / epilogue: one row per thread
+    // ------------------------------------------------------------ softmax / correction / epilogue: half a row per thread
+    const int g = (warp - 2) >> 2;                           // which half of the keys (and of the columns of O)
     const int q = warp & 3;
     const int r = q * 32 + lane;
-    const uint32_t t_s = tmem_base + (uint32_t(q * 32) << 16);
-    const uint32_t t_o = t_s + 256;
+    const uint32_t t_lane = tmem_base + (uint32_t(q * 32) << 16);
+    const uint32_t t_s = t_lane + g * 128, t_o = t_lane + 256 + g * 64, t_p = t_lane + 384 + g * 64;
     const int pos = pos0 + r;
     const int hi = min(pos, kv_len - 1);
     const int lo = p.window > 0 ? max(0, pos - p.window + 1) : 0;
@@ -866,24 +892,25 @@ prefill_attn_wide_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_c
     const float sc = p.scale_log2;
     float m_ref = -INFINITY, l_run = 0.f;
     bool ok = true;
-    for (int j = 0; j < n_tiles && ok; ++j) {
-      const int b = j & 1;
-      if (!__all_sync(0xffffffffu, mbar_wait(&bars->s_full[b], (j >> 1) & 1))) {
-        if (lane == 0) atomicExch(p.status, XL_ERR_WAIT_TMEM_FULL);
+    auto wait = [&](uint64_t* bar, uint32_t parity, int code) {              // once a wait ran out there are no more
+      if (ok && !__all_sync(0xffffffffu, mbar_wait(bar, parity))) {
+        if (lane == 0) atomicExch(p.status, code);
         ok = false;
-        break;
       }
+    };
+    for (int j = 0; j < n_tiles; ++j) {
+      wait(&bars->s_full, j & 1, XL_ERR_WAIT_TMEM_FULL);
       tc_fence_after();
       uint32_t raw[4][32];
 #pragma unroll
-      for (int i = 0; i < 4; ++i) tmem_ld_32x32(t_s + b * 128 + i * 32, raw[i]);
+      for (int i = 0; i < 4; ++i) tmem_ld_32x32(t_s + i * 32, raw[i]);
       tc_wait_ld();
       tc_fence_before();
       __syncwarp();
-      if (lane == 0) mbar_arrive(&bars->s_free[b]);
+      if (lane == 0) mbar_arrive(&bars->s_free);
       float (&v)[128] = *reinterpret_cast<float (*)[128]>(raw);
-      const int kv0 = kv_begin + (j_first + j) * WKV;
-      if (kv0 + WKV - 1 > pos0 || kv0 + WKV > kv_len || kv0 < lo_win) {
+      const int kv0 = tile_kv(j) + g * 128;
+      if (kv0 + 127 > pos0 || kv0 + 128 > kv_len || kv0 < lo_win) {
 #pragma unroll
         for (int c = 0; c < 128; ++c)
           if (kv0 + c > hi || kv0 + c < lo) v[c] = -INFINITY;
@@ -893,7 +920,10 @@ prefill_attn_wide_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_c
       for (int i = 0; i < 8; ++i) mx8[i] = v[i];
 #pragma unroll
       for (int c = 8; c < 128; ++c) mx8[c & 7] = fmaxf(mx8[c & 7], v[c]);
-      const float mx = fmaxf(fmaxf(fmaxf(mx8[0], mx8[1]), fmaxf(mx8[2], mx8[3])), fmaxf(fmaxf(mx8[4], mx8[5]), fmaxf(mx8[6], mx8[7])));
+      float mx = fmaxf(fmaxf(fmaxf(mx8[0], mx8[1]), fmaxf(mx8[2], mx8[3])), fmaxf(fmaxf(mx8[4], mx8[5]), fmaxf(mx8[6], mx8[7])));
+      bars->row[j & 1][g][r] = mx;
+      softmax_warps_sync();
+      mx = fmaxf(mx, bars->row[j & 1][g ^ 1][r]);
       const bool had = m_ref != -INFINITY;
       const bool grow = (mx - m_ref) * sc > 8.f || (!had && mx != -INFINITY);
       const float m_new = grow ? mx : m_ref;
@@ -902,24 +932,20 @@ prefill_attn_wide_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_c
       m_ref = m_new;
       const float mneg = (m_ref == -INFINITY) ? 0.f : -m_ref * sc;
       float sum4[4] = {0.f, 0.f, 0.f, 0.f};
-      uint32_t pk[64];
+      uint32_t pk[2][32];
 #pragma unroll
       for (int c = 0; c < 128; c += 2) {
         const float e0 = fast_exp2(fmaf(v[c], sc, mneg)), e1 = fast_exp2(fmaf(v[c + 1], sc, mneg));
         sum4[(c >> 1) & 3] += e0 + e1;
-        pk[c >> 1] = pack_bf16x2(e0, e1);
+        pk[c >> 6][(c >> 1) & 31] = pack_bf16x2(e0, e1);
       }
       l_run = l_run * alpha + ((sum4[0] + sum4[1]) + (sum4[2] + sum4[3]));
       // P and O are touched only after P V of the previous tile has finished
-      if (j > 0 && !__all_sync(0xffffffffu, mbar_wait(&bars->pv_done, (j - 1) & 1))) {
-        if (lane == 0) atomicExch(p.status, XL_ERR_WAIT_TMEM_EMPTY);
-        ok = false;
-        break;
-      }
+      if (j > 0) wait(&bars->pv_done, (j - 1) & 1, XL_ERR_WAIT_TMEM_EMPTY);
       tc_fence_after();
       if (j > 0 && __any_sync(0xffffffffu, rescale)) {
 #pragma unroll
-        for (int c = 0; c < DV; c += 32) {
+        for (int c = 0; c < DV / 2; c += 32) {
           uint32_t o[32];
           tmem_ld_32x32(t_o + c, o);
           tc_wait_ld();
@@ -927,31 +953,25 @@ prefill_attn_wide_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_c
           for (int i = 0; i < 32; ++i) o[i] = __float_as_uint(__uint_as_float(o[i]) * alpha);
           tmem_st_32x32(t_o + c, o);
         }
-        tc_wait_st();
       }
-#pragma unroll
-      for (int g = 0; g < 2; ++g) {
-        uint8_t* prow = sP + g * W_UNIT + r * 128;
-#pragma unroll
-        for (int c = 0; c < 8; ++c)
-          *reinterpret_cast<uint4*>(prow + ((c ^ (r & 7)) << 4)) =
-              make_uint4(pk[g * 32 + 4 * c], pk[g * 32 + 4 * c + 1], pk[g * 32 + 4 * c + 2], pk[g * 32 + 4 * c + 3]);
-      }
-      fence_proxy_async_smem();
+      tmem_st_32x32(t_p, pk[0]);
+      tmem_st_32x32(t_p + 32, pk[1]);
+      tc_wait_st();
       tc_fence_before();
       __syncwarp();
       if (lane == 0) mbar_arrive(&bars->p_full);
     }
-    if (ok && !__all_sync(0xffffffffu, mbar_wait(&bars->pv_done, (n_tiles - 1) & 1))) {
-      if (lane == 0) atomicExch(p.status, XL_ERR_WAIT_TMEM_EMPTY);
-      ok = false;
-    }
+    wait(&bars->pv_done, (n_tiles - 1) & 1, XL_ERR_WAIT_TMEM_EMPTY);
+    // the row's sum; the buffer of the last tile but one has been read by both groups
+    bars->row[n_tiles & 1][g][r] = l_run;
+    softmax_warps_sync();
+    l_run += bars->row[n_tiles & 1][g ^ 1][r];
+    tc_fence_after();
     if (ok && n_splits > 1) {
-      tc_fence_after();
       const size_t unit = size_t(tile_ord) * gridDim.y + blockIdx.y;
-      float4* wo = reinterpret_cast<float4*>(p.ws_o) + (unit * p.splits + blockIdx.z) * (DV / 4) * BQ;
+      float4* wo = reinterpret_cast<float4*>(p.ws_o) + ((unit * p.splits + blockIdx.z) * (DV / 4) + g * 16) * BQ;
 #pragma unroll
-      for (int c = 0; c < DV; c += 32) {
+      for (int c = 0; c < DV / 2; c += 32) {
         uint32_t o[32];
         tmem_ld_32x32(t_o + c, o);
         tc_wait_ld();
@@ -960,15 +980,14 @@ prefill_attn_wide_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_c
           wo[size_t(c / 4 + i) * BQ + r] = make_float4(__uint_as_float(o[4 * i]), __uint_as_float(o[4 * i + 1]),
                                                        __uint_as_float(o[4 * i + 2]), __uint_as_float(o[4 * i + 3]));
       }
-      p.ws_ml[(unit * p.splits + blockIdx.z) * BQ + r] = make_float2(m_ref == -INFINITY ? -INFINITY : m_ref * sc, l_run);
+      if (g == 0) p.ws_ml[(unit * p.splits + blockIdx.z) * BQ + r] = make_float2(m_ref == -INFINITY ? -INFINITY : m_ref * sc, l_run);
       __threadfence();
     } else if (ok) {
-      tc_fence_after();
       if (p.sinks && m_ref != -INFINITY) l_run += fast_exp2(p.sinks[head] * 1.4426950408889634f - m_ref * sc);
       const float inv = l_run > 0.f ? 1.f / l_run : 0.f;
       __nv_bfloat16* dst = p.out + size_t(q_start + q0 + r) * (size_t(p.n_q) * p.dv) + size_t(head) * p.dv;
 #pragma unroll
-      for (int c = 0; c < DV; c += 32) {
+      for (int c = 0; c < DV / 2; c += 32) {
         uint32_t o[32];
         tmem_ld_32x32(t_o + c, o);
         tc_wait_ld();
@@ -979,7 +998,8 @@ prefill_attn_wide_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_c
 #pragma unroll
             for (int e = 0; e < 4; ++e)
               w[e] = pack_bf16x2(__uint_as_float(o[8 * i + 2 * e]) * inv, __uint_as_float(o[8 * i + 2 * e + 1]) * inv);
-            if (c + 8 * i < p.dv) *reinterpret_cast<uint4*>(dst + c + 8 * i) = make_uint4(w[0], w[1], w[2], w[3]);
+            const int col = g * 64 + c + 8 * i;
+            if (col < p.dv) *reinterpret_cast<uint4*>(dst + col) = make_uint4(w[0], w[1], w[2], w[3]);
           }
         }
       }
@@ -1000,7 +1020,7 @@ prefill_attn_wide_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_c
     if (prev == n_splits - 1) *cnt = 0;
   }
   __syncthreads();
-  if (!bars->last_split || warp < 2) return;
+  if (!bars->last_split || warp < 2 || warp > 5) return;
   __threadfence();
   const int r = (warp & 3) * 32 + lane;
   const int n_valid = (n_all + share - 1) / share;          // splits that had keys to look at
@@ -1121,7 +1141,7 @@ static int launch_wide(const CUtensorMap* tq, const CUtensorMap* tk, const CUten
     set = true;
   }
   Params p = p_in;
-  plan_splits(p, 1, 128, 6, q_tiles_cap, total_q_rows, stream);
+  plan_splits(p, 1, 128, 3, q_tiles_cap, total_q_rows, stream);
   prefill_attn_wide_kernel<QR><<<dim3(q_tiles_cap, p.n_q, p.splits), WideCfg<QR>::kThreads, smem, stream>>>(*tq, *tk, *tv, p, (dk + 127) / 128 * 2);
   return cudaGetLastError() == cudaSuccess ? 0 : -1;
 }

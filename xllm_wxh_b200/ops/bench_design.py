@@ -1,4 +1,4 @@
-"""A model design beside the framework's closest other one at equal layer sizes (`bench.py --compare-design movolorn|falalix|babadra`):
+"""A model design beside the framework's closest other one at equal layer sizes (`bench.py --compare-design movolorn|falalix|babadra|govuvik`):
 tokens per second of the decoder layers in prefill and decode, and the design's own kernels beside the like kernels with their
 distance from the roofline.  Random weights; kernel and layer times come from CUDA-graph replay between CUDA events, with
 weights, caches and activations rotated through (or larger than) more memory than L2 holds."""
@@ -14,7 +14,7 @@ import torch
 
 from ..framework.step_input import StepInput, make_layout
 from ..models.args import ModelArgs, QuantArgs, preset
-from ..models.layer_spec import AttentionSpec, LatentAttentionSpec, ParallelSpec, RotarySpec, SelectiveScanSpec
+from ..models.layer_spec import AttentionSpec, LatentAttentionSpec, MatrixMemorySpec, ParallelSpec, RotarySpec, SelectiveScanSpec
 from ..models.registry import get_model_class
 from . import cuda_ops as c
 from . import moe_cuda
@@ -25,9 +25,12 @@ DEV = "cuda:0"
 PAIRS = {"movolorn": [("movolorn-8b", "qwen3-8b", ""), ("movolorn-30b-a3b", "qwen3-30b-a3b", "")],
          "falalix": [("falalix-8b", "qwen3-8b", "parallel"), ("falalix-8b", "qwen3-8b", "scan"), ("falalix-8b", "qwen3-8b", "")],
          "babadra": [("babadra-8b", "deepseek-8b", "latent"), ("babadra-8b", "qwen3-8b", "two-map"),
-                     ("babadra-30b-a3b", "qwen3-30b-a3b", "two-map")]}
+                     ("babadra-30b-a3b", "qwen3-30b-a3b", "two-map")],
+         "govuvik": [("govuvik-30b-a3b", "qwen3-30b-a3b", "parallel"), ("govuvik-30b-a3b", "qwen3-30b-a3b", "memory"),
+                     ("govuvik-30b-a3b", "qwen3-30b-a3b", "")]}
 KINDS = {"parallel": lambda m: isinstance(m, ParallelSpec), "scan": lambda m: isinstance(m, SelectiveScanSpec),
-         "latent": lambda m: isinstance(m, LatentAttentionSpec), "two-map": lambda m: getattr(m, "maps", 1) == 2}
+         "latent": lambda m: isinstance(m, LatentAttentionSpec), "two-map": lambda m: getattr(m, "maps", 1) == 2,
+         "memory": lambda m: isinstance(m, MatrixMemorySpec)}
 
 
 def args_of(name: str) -> ModelArgs:
@@ -125,11 +128,11 @@ class Rows:
         self.pk = peaks()
         self.rows = []
 
-    def add(self, what, ours, like, bytes_ours=0.0, bytes_like=0.0, flops=0.0, flops_like=None):
-        def frac(us, nbytes, ops):
-            bound = max(nbytes / (self.pk["hbm_gbs"] * 1e3), ops / (self.pk["bf16_tflops"] * 1e6))
+    def add(self, what, ours, like, bytes_ours=0.0, bytes_like=0.0, flops=0.0, flops_like=None, fma=0.0, fma_like=0.0):
+        def frac(us, nbytes, ops, fp32):
+            bound = max(nbytes / (self.pk["hbm_gbs"] * 1e3), ops / (self.pk["bf16_tflops"] * 1e6), fp32 / FMA_RATE * 1e6)
             return bound / us
-        fo, fl = frac(ours, bytes_ours, flops), frac(like, bytes_like, flops if flops_like is None else flops_like)
+        fo, fl = frac(ours, bytes_ours, flops, fma), frac(like, bytes_like, flops if flops_like is None else flops_like, fma_like)
         self.rows.append({"what": what, "us": round(ours, 1), "like_us": round(like, 1), "roofline": round(fo, 3), "like_roofline": round(fl, 3),
                           "farther_by": round(fl / fo, 2)})
 
@@ -422,7 +425,116 @@ def babadra_kernels() -> List[Dict]:
     return R.rows
 
 
-KERNELS = {"movolorn": movolorn_kernels, "falalix": falalix_kernels, "babadra": babadra_kernels}
+@torch.inference_mode()
+def govuvik_kernels() -> List[Dict]:
+    R = Rows()
+    add, alone = R.add, R.add_alone
+    W, heads, G, d, window = 2048, 32, 4, 128, 4096
+    # ---- attention with mixed scores and sinks, beside attention with the same window
+    sinks = torch.zeros(heads, device=DEV)
+    for kind, seqs, q_len, kv in STEPS:
+        inp = step_input(seqs, q_len, kv, 16, 1000)
+        nb, T, row = seqs * (-(-kv // 16)) + 1, seqs * q_len, (heads + 2 * G) * d
+        cache_bytes = 2.0 * seqs * (kv if kind == "prefill" else min(kv, window)) * G * d * 2
+        sets = _rotated(lambda: (_bf(T, heads * G * d, std=0.1), _bf(nb, 16, G, d), _bf(nb, 16, G, d), _bf(T, row)), cache_bytes + T * row * 2)[:8]
+        o = time_graph([lambda s=s: c.paged_attention_ext(s[0].view(T, heads, G * d), s[1].view(nb, 16, 1, G * d), s[2], inp, d ** -0.5, window,
+                                                          sinks=sinks) for s in sets])
+        k = time_graph([lambda s=s: c.paged_attention(s[3][:, :heads * d].unflatten(1, (heads, d)), s[1], s[2], inp, d ** -0.5, window) for s in sets])
+        pairs = sum(min(p + 1, window) for p in range(kv - q_len, kv)) * seqs
+        fk = 4.0 * heads * d * pairs
+        io = T * heads * d * 2.0
+        # ours: scores, their mix, sums of the values; q enters with the columns of every key head
+        add(f"attention {kind} {seqs} x {q_len} of {kv}, window {window}, {heads}/{G} heads", o, k, cache_bytes + io * (1 + G), cache_bytes + 2 * io,
+            fk + 2.0 * heads * heads * pairs if kind == "prefill" else 0.0, fk if kind == "prefill" else 0.0)
+        del sets
+    # ---- norms, cache write, convolutions
+    cs, t64 = torch.randn(8192, 128, device=DEV), torch.randn(8192, 64, device=DEV)
+    mix, w, w128 = torch.eye(heads, device=DEV) + 0.1, _bf(W), _bf(128)
+    qw, kw, emb = _bf(heads * d), _bf(G * d), _bf(30000, W)
+    for T in (8192, 256):
+        inp, row = step_input(1, T, T, 16, 1000), (heads + 2 * G) * d
+        new = step_input(T, 1, 1152, 16, 1000) if T == 256 else step_input(1, T, T, 16, 1000)
+        sets = _rotated(lambda: (_bf(T, row), _bf(T // 16 + 1, 16, G, d), _bf(T // 16 + 1, 16, G, d)), T * row * 2.0)[:24]
+        rot = (t64, inp.positions, False)
+        o = time_graph([lambda s=s: c.qknorm_all_kvwrite(s[0], inp.slots, qw, kw, 1e-6, s[1], s[2], heads, G, rot, mix) for s in sets])
+        k = time_graph([lambda s=s: c.rope_qknorm_kvwrite(s[0], inp.positions, inp.slots, cs, w128, w128, 1e-6, s[1], s[2], heads, G, d) for s in sets])
+        add(f"q / k norm + rotation + score mix + cache write, {T} tokens", o, k, T * (heads * (1.0 + G) + 4 * G) * d * 2 + T * 256.0,
+            T * (2.0 * heads + 4 * G) * d * 2 + T * 512.0, fma=1.0 * T * heads * heads * d)
+        slots = T if T == 256 else 1
+        for what, C in (("input", W), ("q, k, v", row)):
+            sets = _rotated(lambda: (_bf(T, C), _bf(4, C), _bf(C), _bf(slots + 1, 3, C)), T * C * 4.0)[:16]
+            o = time_graph([lambda s=s: c.causal_conv(s[0], s[1], None, s[3], new, "none", C == W) for s in sets])
+            k = time_graph([lambda s=s: c.causal_conv(s[0], s[1], s[2], s[3], new, "silu") for s in sets])
+            b = T * C * 4.0 + (2 * T * 3 * C * 2.0 if T == 256 else 0)
+            add(f"convolution on {what}, {T} x {C}", o, k, b, b)
+        sets = _rotated(lambda: (_bf(T, W), torch.randn(T, W, device=DEV), _bf(T, W)), T * W * 10.0)
+        o = time_graph([lambda s=s: c.branches_post_norm_add_norm(s[0], s[2], w, w, 0.5, s[1], w, w, 1e-6) for s in sets])
+        k = time_graph([lambda s=s: c.post_norm_add_norm(s[0], s[1], w, w, 1e-6) for s in sets])
+        add(f"two branch norms + norm + residual + norm, {T} x {W}", o, k, T * W * 14.0, T * W * 12.0)
+        ids = torch.randint(0, 30000, (T,), device=DEV).int()
+        o = time_graph([lambda: c.embed_rms_norm(ids, emb, 1.0, w, 1e-6, w_rows=w)] * 8)
+        k = time_graph([lambda: c.rms_norm(c.embedding(ids, emb), w, 1e-6)] * 8)
+        add(f"embedding + its norm + first norm, {T} x {W}", o, k, T * W * 8.0, T * W * 8.0)
+    # ---- matrix states beside time mixing, per element of the state the same work
+    for kind, seqs, q_len, kv in STEPS[:3]:
+        T = seqs * q_len
+        inp = step_input(seqs, q_len, kv, 16, 1000)
+        passes = 1 if kv == q_len else 2
+        n, hd = 4096, 64
+        u, w0, nw = torch.randn(n // hd, hd, device=DEV), torch.randn(n, device=DEV) - 3, _bf(n)
+        sets = [(_bf(T, n), _bf(T, n), _bf(T, n), torch.randn(T, n, device=DEV), _bf(T, n), torch.empty(T, n, device=DEV, dtype=torch.bfloat16),
+                 torch.zeros(seqs + 1, n // hd, hd, hd, device=DEV)) for _ in range(3)]
+        k = time_graph([lambda s=s: c.time_mix(s[0], s[1], s[2], s[3], w0, u, s[4], nw, 0.5, 1e-6, s[6], inp, s[5]) for s in sets])
+        kb, kf = T * n * 14.0 + passes * seqs * n * hd * 4.0, 3.0 * T * n * hd
+        del sets
+        H, dk, dv = 16, 64, 128
+        row = H * (2 * dk + 2 * dv)
+        cut = lambda x: (x[:, :H * dk], x[:, H * dk:2 * H * dk], x[:, 2 * H * dk:2 * H * dk + H * dv])
+        bias, nw = torch.randn(H * dk, device=DEV) + 2, _bf(dv)
+        sets = [(_bf(T, row), torch.randn(T, H * dk, device=DEV), torch.zeros(seqs + 1, H, dk, dv, device=DEV)) for _ in range(4)]
+        o = time_graph([lambda s=s: c.gated_memory(*cut(s[0]), s[1], bias, 1 / 16, s[0][:, -H * dv:], nw, 1e-6, s[2], inp) for s in sets])
+        add(f"gated linear attention, {kind} {seqs} x {q_len}, {H} heads of {dk} x {dv}", o, k,
+            T * (row * 2.0 + H * dk * 4 + H * dv * 2) + passes * seqs * H * dk * dv * 4.0, kb, fma=3.0 * T * H * dk * dv, fma_like=kf)
+        del sets
+        H = 32
+        row = H * (2 * dk + 2 * dv)
+        bias, nw = torch.randn(2 * H, device=DEV) + 2, _bf(H * dv)
+        sets = [(_bf(T, row), torch.randn(T, 2 * H, device=DEV), torch.zeros(seqs + 1, H, dk * dv + dk, device=DEV), torch.zeros(seqs + 1, H, device=DEV))
+                for _ in range(4)]
+        o = time_graph([lambda s=s: c.matrix_memory(*cut(s[0]), s[1], bias, 15.0, s[0][:, -H * dv:], nw, 1e-6, s[2], s[3], inp) for s in sets])
+        add(f"matrix memory, {kind} {seqs} x {q_len}, {H} heads of {dk} x {dv}", o, k,
+            T * (row * 2.0 + H * 8 + H * dv * 2) + passes * seqs * H * dk * dv * 4.0, kb, fma=3.0 * T * H * dk * dv, fma_like=kf)
+        del sets
+    # ---- router and mixture: experts without gates, of as many weights
+    E, top, ff, I = 128, 8, 1152, 768
+    wr = _bf(E, W, std=0.02)
+    up, down = _bf(E, ff, W, std=0.02), _bf(E, W, ff, std=0.02)
+    w13, w2 = _bf(E, 2 * I, W, std=0.02), _bf(E, W, I, std=0.02)
+    moe_cuda.interleave_w13(w13)
+    for T in (8192, 256):
+        sets = _rotated(lambda: (_bf(T, W), torch.randn(T, W, device=DEV), _bf(T, W)), T * W * 10.0)[:16]
+        o = time_graph([lambda s=s: c.moe_router(c.linear_f32(s[0], wr), top, "softmax_chosen") for s in sets])
+        k = time_graph([lambda s=s: c.moe_router(c.linear(s[0], wr), top, "softmax", True) for s in sets])
+        b = T * W * 2.0 + E * W * 2.0 + T * 64.0
+        add(f"router product + choice, {T} x {E}", o, k, b, b, 2.0 * T * E * W)
+        wts, idx = c.moe_router(c.linear(sets[0][0], wr), top, "softmax", True)
+
+        def ours_mix(s):
+            y, dst = moe_cuda.expert_rows(s[0], up, down, idx, "relu2")
+            return moe_cuda.combine_post_norm_add_norm(y, dst, idx, wts, s[0], None, E, s[1], w, w, 1e-6)
+        o = time_graph([lambda s=s: ours_mix(s) for s in sets])
+        k = time_graph([lambda s=s: c.add_rms_norm(moe_cuda.moe_experts(s[0], w13, w2, wts, idx, 0, True), s[2], w, 1e-6) for s in sets])
+        b = 3.0 * E * I * W * 2
+        add(f"mixture to the next sublayer's input, {T} tokens", o, k, b + T * W * 12.0, b + T * W * 8.0, 6.0 * T * top * I * W)
+    # ---- small products
+    h, a1 = _bf(8192, W), _bf(8192, 16)
+    gw, a2 = _bf(64, W, std=0.02), _bf(1024, 16)
+    alone("gates of the matrix memory, 8192 x 64 x 2048", time_graph([lambda: c.linear_f32(h, gw)] * 4), 8192 * (W * 2.0 + 256))
+    alone("decay's second factor, 8192 x 1024 x 16", time_graph([lambda: c.linear_f32(a1, a2)] * 4), 8192 * (32.0 + 4096))
+    return R.rows
+
+
+KERNELS = {"movolorn": movolorn_kernels, "falalix": falalix_kernels, "babadra": babadra_kernels, "govuvik": govuvik_kernels}
 
 
 def run(design: str, layers: int = 4, block: int = 16) -> Dict:
