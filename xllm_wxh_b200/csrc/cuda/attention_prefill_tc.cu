@@ -651,7 +651,7 @@ constexpr int W_UNIT = 2 * W_SLAB;
 template <int QR> struct WideCfg {
   static constexpr int kUnits = QR == 8 ? 3 : 5;
   static constexpr int kSmem = QR * W_SLAB + kUnits * W_UNIT;          // query slabs, ring
-  static constexpr int kThreads = 320;
+  static constexpr int kThreads = 384;
 };
 struct WideBarriers {
   uint64_t q_full;
@@ -676,7 +676,7 @@ __device__ __forceinline__ void tc_mma_f16_ts(uint32_t tmem_d, uint32_t tmem_a, 
 }
 
 template <int QR>
-__global__ void __launch_bounds__(320, 1)
+__global__ void __launch_bounds__(384, 1)
 prefill_attn_wide_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__ CUtensorMap tmK, const __grid_constant__ CUtensorMap tmV,
                          const Params p, const int KS) {
   constexpr int U = WideCfg<QR>::kUnits;
@@ -748,10 +748,12 @@ prefill_attn_wide_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_c
   tc_fence_after();
   const uint32_t tmem_base = bars->tmem_base;             // S at 0, O at 256, P at 384
 
-  if (warp == 0) {
-    // ------------------------------------------------------------ TMA producer (whole warp: lanes share a unit's boxes)
+  if (warp == 0 || warp >= 10) {
+    // ------------------------------------------------------------ TMA producers: a warp issues one copy at a time, so three share a unit's
+    // boxes; the first one also announces the unit's bytes
+    const int part = warp == 0 ? 0 : warp - 9;
     const int boxes = WKV / p.box_tokens;                 // of a whole unit: 4, 8 or 16
-    if (lane == 0) {
+    if (lane == 0 && part == 0) {
       prefetch_tmap(&tmQ);
       prefetch_tmap(&tmK);
       prefetch_tmap(&tmV);
@@ -774,13 +776,14 @@ prefill_attn_wide_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_c
         if (!mbar_wait(&bars->empty[u], ((c / U) & 1) ^ 1)) {
           atomicExch(p.status, XL_ERR_WAIT_EMPTY);
           ok = false;
-        } else {
+        } else if (part == 0) {
           mbar_arrive_expect_tx(&bars->full[u], bytes);
         }
       }
       ok = __shfl_sync(0xffffffffu, ok, 0);
       return ok;
     };
+    auto mine = [&](int n) { return lane < n && lane % 3 == part; };
     int slot = slot_of(0), slot_v = 0;
     for (int j = 0; j <= n_tiles && ok; ++j) {
       const int next = j + 1 < n_tiles ? slot_of(j + 1) : 0;
@@ -789,12 +792,12 @@ prefill_attn_wide_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_c
         for (int s = 0; s < KS; ++s) {
           if (s >= QR) {
             if (!open(W_SLAB)) break;
-            if (lane == 0) tma_load_3d(ring + (c % U) * W_UNIT, &tmQ, &bars->full[c % U], s * 64, head, q_start + q0);
+            if (lane == 0 && part == 0) tma_load_3d(ring + (c % U) * W_UNIT, &tmQ, &bars->full[c % U], s * 64, head, q_start + q0);
             __syncwarp();
             ++c;
           }
           if (!open(n * p.box_tokens * 128)) break;
-          if (lane < n) tma_load_3d(ring + (c % U) * W_UNIT + lane * p.box_tokens * 128, &tmK, &bars->full[c % U], s * 64, 0, slot);
+          if (mine(n)) tma_load_3d(ring + (c % U) * W_UNIT + lane * p.box_tokens * 128, &tmK, &bars->full[c % U], s * 64, 0, slot);
           __syncwarp();
           ++c;
         }
@@ -804,7 +807,7 @@ prefill_attn_wide_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_c
         for (int h = 0; h < (is_half(j - 1) ? 1 : 2); ++h) {
           if (!open(W_UNIT)) break;
           const int z = __shfl_sync(0xffffffffu, slot_v, h * per + lane % per);
-          if (lane < boxes)
+          if (mine(boxes))
             tma_load_3d(ring + (c % U) * W_UNIT + lane / per * W_SLAB + lane % per * p.box_tokens * 128, &tmV, &bars->full[c % U], lane / per * 64, vh, z);
           __syncwarp();
           ++c;
