@@ -413,54 +413,68 @@ __global__ void __launch_bounds__(160) decode_attn_tma_kernel(const __grid_const
 }
 
 // ---------------------------------------------------------------- one wide key head for all query heads
-// One CTA handles one (sequence, block of 16 query rows, KV split); a row is (token, query head), so the rows of a block may belong to
-// several value heads.  Keys and values pass through a ring of [64 tokens][64 columns] slabs: the slabs of a tile's keys, whose
+// One CTA handles one (sequence, block of 16 MT query rows, KV split); a row is (token, query head), so the rows of a block may belong to
+// several value heads.  Keys and values pass through a ring of [128 tokens][64 columns] slabs: the slabs of a tile's keys, whose
 // products add up to S, then those of the value heads that the block's rows need; P is zero in the rows of other value heads, so all of
-// them accumulate into one O.
-constexpr int kWideSlabs = 10;
+// them accumulate into one O.  Eight consumer warps take 16 tokens of every slab each.
+constexpr int kWideTile = 128, kWideSlab = kWideTile * 128;
+constexpr int kWideMost = 12, kWideProducers = 2, kWideConsumers = 8, kWideThreads = 32 * (kWideConsumers + kWideProducers);
 struct WideDecBarriers {
-  uint64_t full[kWideSlabs];
-  uint64_t empty[kWideSlabs];
+  uint64_t full[kWideMost];
+  uint64_t empty[kWideMost];
+};
+// Place in a ring of n slabs and how often it has gone round.
+struct RingPos {
+  int slot = 0;
+  uint32_t phase = 0;
+  __device__ __forceinline__ void next(int n) {
+    if (++slot == n) {
+      slot = 0;
+      phase ^= 1;
+    }
+  }
 };
 
-template <int DV>
-__global__ void __launch_bounds__(160) decode_attn_wide_kernel(const __grid_constant__ CUtensorMap tmK, const __grid_constant__ CUtensorMap tmV,
-                                                               const DecParams p, const int KS) {
-  constexpr int VH = DV / 64;
-  constexpr int SLAB = kTile * 128;
+template <int MT, int DV>
+__global__ void __launch_bounds__(kWideThreads, 1) decode_attn_wide_kernel(const __grid_constant__ CUtensorMap tmK,
+                                                                           const __grid_constant__ CUtensorMap tmV, const DecParams p, const int KS,
+                                                                           const int n_slabs) {
+  constexpr int VH = DV / 64, ROWS = 16 * MT, CW = kWideConsumers;
   constexpr float kL2e = 1.4426950408889634f;
   extern __shared__ uint8_t smem_raw[];
   uint8_t* ring = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(smem_raw) + 1023) & ~uintptr_t(1023));
-  uint8_t* sQ = ring + kWideSlabs * SLAB;                        // 16 x 64 KS bf16, 16-byte-chunk XOR swizzle
-  WideDecBarriers* bars = reinterpret_cast<WideDecBarriers*>(sQ + 16 * KS * 128);
+  uint8_t* sQ = ring + n_slabs * kWideSlab;                      // ROWS x 64 KS bf16, 16-byte-chunk XOR swizzle
+  WideDecBarriers* bars = reinterpret_cast<WideDecBarriers*>(sQ + ROWS * KS * 128);
+  float* sM = reinterpret_cast<float*>(bars + 1);                // [CW][ROWS] maxima, then sums
+  float* sL = sM + CW * ROWS;
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
-  const int seq = p.seq_begin + blockIdx.x, row0 = blockIdx.y * 16, split = blockIdx.z;
+  const int seq = p.seq_begin + blockIdx.y, row0 = blockIdx.x * ROWS, split = blockIdx.z;
   const int group = p.n_q / p.n_kv, dk = p.dk, dv = p.dv;
   if (seq >= (p.dyn_end ? *p.dyn_end : p.seq_end)) return;
   const int q_start = p.q_cu[seq];
   const int q_len = p.q_cu[seq + 1] - q_start;
   const int kv_len = p.kv_lens[seq];
   if (q_len <= 0) return;
-  const int rows = min(16, q_len * p.n_q - row0);
+  const int rows = min(ROWS, q_len * p.n_q - row0);
   if (rows <= 0) return;
   // value heads of the rows: consecutive ones, all of them when the block reaches into the next token
   const int h_first = row0 % p.n_q, h_last = h_first + rows - 1;
   const int v_first = h_last >= p.n_q ? 0 : h_first / group, v_last = h_last >= p.n_q ? p.n_kv - 1 : h_last / group;
   const int* bt = p.block_tables + size_t(seq) * p.max_blocks;
-  const int r_begin = p.window > 0 ? max(0, kv_len - q_len - p.window + 1) / kTile * kTile : 0;
-  const int all_tiles = (kv_len - r_begin + kTile - 1) / kTile;
+  const int r_begin = p.window > 0 ? max(0, kv_len - q_len - p.window + 1) / kTile * kTile : 0;     // a multiple of the boxes' tokens
+  const int all_tiles = (kv_len - r_begin + kWideTile - 1) / kWideTile;
   const int per_split = (all_tiles + p.num_splits - 1) / p.num_splits;
   const int t_first = split * per_split;
   const int n_tiles = max(0, min(all_tiles, t_first + per_split) - t_first);
 
   if (threadIdx.x == 0) {
-    for (int s = 0; s < kWideSlabs; ++s) {
+    for (int s = 0; s < n_slabs; ++s) {
       mbar_init(&bars->full[s], 1);
-      mbar_init(&bars->empty[s], 4);
+      mbar_init(&bars->empty[s], CW);
     }
     mbar_fence_init();
   }
-  for (int i = threadIdx.x; i < 16 * KS * 8; i += blockDim.x) {
+  for (int i = threadIdx.x; i < ROWS * KS * 8; i += blockDim.x) {
     const int r = i / (KS * 8), c = i % (KS * 8);
     const bool ok = r < rows && c * 8 < dk;
     const int m = ok ? row0 + r : 0;
@@ -471,25 +485,31 @@ __global__ void __launch_bounds__(160) decode_attn_wide_kernel(const __grid_cons
   cp_async_wait_all();
   __syncthreads();
 
-  float o[DV / 8][4];
+  float o[MT][DV / 8][4];
+  float m_run[MT][2], l_run[MT][2];
 #pragma unroll
-  for (int i = 0; i < DV / 8; ++i) o[i][0] = o[i][1] = o[i][2] = o[i][3] = 0.f;
-  float m_run[2] = {-INFINITY, -INFINITY}, l_run[2] = {0.f, 0.f};
-  const int row_a = lane >> 2, row_b = row_a + 8;
+  for (int mt = 0; mt < MT; ++mt) {
+    m_run[mt][0] = m_run[mt][1] = -INFINITY;
+    l_run[mt][0] = l_run[mt][1] = 0.f;
+#pragma unroll
+    for (int i = 0; i < DV / 8; ++i) o[mt][i][0] = o[mt][i][1] = o[mt][i][2] = o[mt][i][3] = 0.f;
+  }
 
-  if (warp == 4) {
-    // ------------------------------------------------------------ producer: lanes share a slab's boxes
-    const int bt_tok = p.box_tokens;
+  RingPos at;
+  if (warp >= CW) {
+    // ------------------------------------------------------------ producers: a warp issues one copy at a time, so they share a slab's
+    // boxes; the first one also announces the slab's bytes
+    const int part = warp - CW, bt_tok = p.box_tokens;
     if (lane == 0) {
       prefetch_tmap(&tmK);
       prefetch_tmap(&tmV);
     }
     const int per_tile = KS + (v_last - v_first + 1) * VH;
-    int c = 0;
+    int issued = 0;
     bool ok = true;
     for (int t = 0; t < n_tiles && ok; ++t) {
-      const int base = r_begin + (t_first + t) * kTile;
-      const int n_boxes = (min(kTile, kv_len - base) + bt_tok - 1) / bt_tok;
+      const int base = r_begin + (t_first + t) * kWideTile;
+      const int n_boxes = (min(kWideTile, kv_len - base) + bt_tok - 1) / bt_tok;
       int z = 0;
       if (lane < n_boxes) {
         const int tok = base + lane * bt_tok;
@@ -497,82 +517,102 @@ __global__ void __launch_bounds__(160) decode_attn_wide_kernel(const __grid_cons
         if (blk < 0 || blk >= p.num_blocks_total) blk = 0;
         z = blk * p.block_size + tok % p.block_size;
       }
-      for (int i = 0; i < per_tile && ok; ++i, ++c) {
-        const int s = c % kWideSlabs;
+      for (int i = 0; i < per_tile; ++i) {
         if (lane == 0) {
-          if (!mbar_wait(&bars->empty[s], ((c / kWideSlabs) & 1) ^ 1)) {
+          if (!mbar_wait(&bars->empty[at.slot], at.phase ^ 1)) {
             atomicExch(p.status, XL_ERR_WAIT_EMPTY);
             ok = false;
-          } else {
-            mbar_arrive_expect_tx(&bars->full[s], uint32_t(n_boxes) * bt_tok * 128);
+          } else if (part == 0) {
+            mbar_arrive_expect_tx(&bars->full[at.slot], uint32_t(n_boxes) * bt_tok * 128);
           }
         }
         ok = __shfl_sync(0xffffffffu, ok, 0);
-        if (ok && lane < n_boxes) {
-          uint8_t* dst = ring + s * SLAB + lane * bt_tok * 128;
-          if (i < KS) tma_load_3d(dst, &tmK, &bars->full[s], i * 64, 0, z);
-          else tma_load_3d(dst, &tmV, &bars->full[s], (i - KS) % VH * 64, v_first + (i - KS) / VH, z);
+        if (!ok) break;
+        if (lane < n_boxes && lane % kWideProducers == part) {
+          uint8_t* dst = ring + at.slot * kWideSlab + lane * bt_tok * 128;
+          if (i < KS) tma_load_3d(dst, &tmK, &bars->full[at.slot], i * 64, 0, z);
+          else tma_load_3d(dst, &tmV, &bars->full[at.slot], (i - KS) % VH * 64, v_first + (i - KS) / VH, z);
         }
         __syncwarp();
+        at.next(n_slabs);
+        ++issued;
       }
     }
-    if (!ok && lane == 0)    // let the copies already issued land (bounded) before the CTA retires
-      for (int j = max(0, c - kWideSlabs); j < c - 1; ++j) mbar_wait(&bars->full[j % kWideSlabs], (j / kWideSlabs) & 1);
+    if (!ok && lane == 0) {  // let the copies already issued land (bounded) before the CTA retires
+      for (int back = min(issued, n_slabs); back > 0; --back) {
+        const int j = issued - back;
+        mbar_wait(&bars->full[j % n_slabs], (j / n_slabs) & 1);
+      }
+    }
   } else {
     // ------------------------------------------------------------ consumers
-    const int m_a = row0 + (row_a < rows ? row_a : 0), m_b = row0 + (row_b < rows ? row_b : 0);
-    const int lim_a = kv_len - q_len + m_a / p.n_q, lim_b = kv_len - q_len + m_b / p.n_q;
-    const int vh_a = m_a % p.n_q / group, vh_b = m_b % p.n_q / group;
+    const int row_a = lane >> 2;
+    int lim[MT][2], vh[MT][2];
+#pragma unroll
+    for (int mt = 0; mt < MT; ++mt)
+#pragma unroll
+      for (int e = 0; e < 2; ++e) {
+        const int r = mt * 16 + row_a + 8 * e, m = row0 + (r < rows ? r : 0);
+        lim[mt][e] = kv_len - q_len + m / p.n_q;
+        vh[mt][e] = r < rows ? m % p.n_q / group : -1;
+      }
     const int rk = (lane & 7) + (lane >> 4) * 8;           // K fragment row (token) of this lane
-    const int rv = (lane & 7) + ((lane >> 3) & 1) * 8;     // V fragment row (token) of this lane
-    const int rq = (lane & 7) + ((lane >> 3) & 1) * 8;     // Q fragment row
-    const uint32_t q_row = smem_u32(sQ + uint32_t(rq) * (KS * 128)), ring_u = smem_u32(ring);
-    int c = 0;
+    const int rv = (lane & 7) + ((lane >> 3) & 1) * 8;     // V fragment row (token), and Q fragment row
+    const uint32_t q_row = smem_u32(sQ + uint32_t(rv) * (KS * 128)), ring_u = smem_u32(ring) + warp * 2048;
     bool ok = true;
     auto take = [&]() -> bool {
-      if (mbar_wait(&bars->full[c % kWideSlabs], (c / kWideSlabs) & 1)) return true;
+      if (mbar_wait(&bars->full[at.slot], at.phase)) return true;
       if (lane == 0) atomicExch(p.status, XL_ERR_WAIT_FULL);
       return false;
     };
     auto give = [&]() {
       __syncwarp();
-      if (lane == 0) mbar_arrive(&bars->empty[c % kWideSlabs]);
-      ++c;
+      if (lane == 0) mbar_arrive(&bars->empty[at.slot]);
+      at.next(n_slabs);
     };
     for (int t = 0; t < n_tiles && ok; ++t) {
-      const int base = r_begin + (t_first + t) * kTile + warp * 16;
+      const int base = r_begin + (t_first + t) * kWideTile + warp * 16;
       const bool mine = base < kv_len;
-      float sc[2][4];
+      float sc[MT][2][4];
 #pragma unroll
-      for (int i = 0; i < 2; ++i) sc[i][0] = sc[i][1] = sc[i][2] = sc[i][3] = 0.f;
+      for (int mt = 0; mt < MT; ++mt)
+#pragma unroll
+        for (int i = 0; i < 2; ++i) sc[mt][i][0] = sc[mt][i][1] = sc[mt][i][2] = sc[mt][i][3] = 0.f;
       for (int ks = 0; ks < KS; ++ks) {
         if (!(ok = take())) break;
         if (mine) {
-          const uint32_t tK = ring_u + (c % kWideSlabs) * SLAB + warp * 2048 + rk * 128;
+          const uint32_t tK = ring_u + at.slot * kWideSlab + rk * 128;
 #pragma unroll
           for (int i = 0; i < 4; ++i) {
-            uint32_t b0, b1, b2, b3, a[4];
+            uint32_t b0, b1, b2, b3;
             ldsm_x4(tK + (((i * 2 + ((lane >> 3) & 1)) ^ (rk & 7)) << 4), b0, b1, b2, b3);
-            ldsm_x4(q_row + (uint32_t((ks * 8 + i * 2 + (lane >> 4)) ^ (rq & 7)) << 4), a[0], a[1], a[2], a[3]);
-            mma_bf16_16816(sc[0], a, b0, b1);
-            mma_bf16_16816(sc[1], a, b2, b3);
+#pragma unroll
+            for (int mt = 0; mt < MT; ++mt) {
+              uint32_t a[4];
+              ldsm_x4(q_row + mt * 16 * KS * 128 + (uint32_t((ks * 8 + i * 2 + (lane >> 4)) ^ (rv & 7)) << 4), a[0], a[1], a[2], a[3]);
+              mma_bf16_16816(sc[mt][0], a, b0, b1);
+              mma_bf16_16816(sc[mt][1], a, b2, b3);
+            }
           }
         }
         give();
       }
       if (!ok) break;
-      uint32_t pa[4] = {0, 0, 0, 0};
-      if (mine) {
+      uint32_t pa[MT][4];
+#pragma unroll
+      for (int mt = 0; mt < MT; ++mt) {
+        pa[mt][0] = pa[mt][1] = pa[mt][2] = pa[mt][3] = 0;
+        if (!mine) continue;
         float mx[2] = {-INFINITY, -INFINITY};
 #pragma unroll
         for (int i = 0; i < 2; ++i) {
 #pragma unroll
           for (int e = 0; e < 4; ++e) {
             const int tok = base + i * 8 + (lane & 3) * 2 + (e & 1);
-            const int lim = (e < 2) ? lim_a : lim_b;
-            const bool see = tok <= lim && tok < kv_len && (p.window <= 0 || tok > lim - p.window);
-            sc[i][e] = see ? sc[i][e] * p.scale_log2 : -INFINITY;
-            mx[e >> 1] = fmaxf(mx[e >> 1], sc[i][e]);
+            const int l = lim[mt][e >> 1];
+            const bool see = tok <= l && tok < kv_len && (p.window <= 0 || tok > l - p.window);
+            sc[mt][i][e] = see ? sc[mt][i][e] * p.scale_log2 : -INFINITY;
+            mx[e >> 1] = fmaxf(mx[e >> 1], sc[mt][i][e]);
           }
         }
         float alpha[2];
@@ -580,47 +620,60 @@ __global__ void __launch_bounds__(160) decode_attn_wide_kernel(const __grid_cons
         for (int h = 0; h < 2; ++h) {
           mx[h] = fmaxf(mx[h], __shfl_xor_sync(0xffffffffu, mx[h], 1));
           mx[h] = fmaxf(mx[h], __shfl_xor_sync(0xffffffffu, mx[h], 2));
-          const float m_new = fmaxf(m_run[h], mx[h]);
-          alpha[h] = (m_new == -INFINITY) ? 1.f : exp2f(m_run[h] - m_new);
-          m_run[h] = m_new;
+          const float m_new = fmaxf(m_run[mt][h], mx[h]);
+          alpha[h] = (m_new == -INFINITY) ? 1.f : exp2f(m_run[mt][h] - m_new);
+          m_run[mt][h] = m_new;
         }
         float rs[2] = {0.f, 0.f};
 #pragma unroll
         for (int i = 0; i < 2; ++i) {
 #pragma unroll
           for (int e = 0; e < 4; ++e) {
-            const float m = m_run[e >> 1];
-            sc[i][e] = (m == -INFINITY) ? 0.f : exp2f(sc[i][e] - m);
-            rs[e >> 1] += sc[i][e];
+            const float m = m_run[mt][e >> 1];
+            sc[mt][i][e] = (m == -INFINITY) ? 0.f : exp2f(sc[mt][i][e] - m);
+            rs[e >> 1] += sc[mt][i][e];
           }
         }
-        l_run[0] = l_run[0] * alpha[0] + rs[0];
-        l_run[1] = l_run[1] * alpha[1] + rs[1];
-        pa[0] = pack_bf16x2(sc[0][0], sc[0][1]);
-        pa[1] = pack_bf16x2(sc[0][2], sc[0][3]);
-        pa[2] = pack_bf16x2(sc[1][0], sc[1][1]);
-        pa[3] = pack_bf16x2(sc[1][2], sc[1][3]);
+        l_run[mt][0] = l_run[mt][0] * alpha[0] + rs[0];
+        l_run[mt][1] = l_run[mt][1] * alpha[1] + rs[1];
+        pa[mt][0] = pack_bf16x2(sc[mt][0][0], sc[mt][0][1]);
+        pa[mt][1] = pack_bf16x2(sc[mt][0][2], sc[mt][0][3]);
+        pa[mt][2] = pack_bf16x2(sc[mt][1][0], sc[mt][1][1]);
+        pa[mt][3] = pack_bf16x2(sc[mt][1][2], sc[mt][1][3]);
         if (alpha[0] != 1.f || alpha[1] != 1.f) {
 #pragma unroll
           for (int i = 0; i < DV / 8; ++i) {
-            o[i][0] *= alpha[0]; o[i][1] *= alpha[0]; o[i][2] *= alpha[1]; o[i][3] *= alpha[1];
+            o[mt][i][0] *= alpha[0]; o[mt][i][1] *= alpha[0]; o[mt][i][2] *= alpha[1]; o[mt][i][3] *= alpha[1];
           }
         }
       }
       for (int v = v_first; v <= v_last && ok; ++v) {
-        const bool ua = vh_a == v, ub = vh_b == v;
-        const uint32_t pv[4] = {ua ? pa[0] : 0u, ub ? pa[1] : 0u, ua ? pa[2] : 0u, ub ? pa[3] : 0u};
+        uint32_t pv[MT][4];
+        bool any[MT];
+#pragma unroll
+        for (int mt = 0; mt < MT; ++mt) {
+          const bool ua = vh[mt][0] == v, ub = vh[mt][1] == v;
+          any[mt] = __any_sync(0xffffffffu, ua || ub);
+          pv[mt][0] = ua ? pa[mt][0] : 0u;
+          pv[mt][1] = ub ? pa[mt][1] : 0u;
+          pv[mt][2] = ua ? pa[mt][2] : 0u;
+          pv[mt][3] = ub ? pa[mt][3] : 0u;
+        }
 #pragma unroll
         for (int vs = 0; vs < VH; ++vs) {
           if (!(ok = take())) break;
           if (mine) {
-            const uint32_t tV = ring_u + (c % kWideSlabs) * SLAB + warp * 2048 + rv * 128;
+            const uint32_t tV = ring_u + at.slot * kWideSlab + rv * 128;
 #pragma unroll
             for (int d = 0; d < 4; ++d) {
               uint32_t b0, b1, b2, b3;
               ldsm_x4_t(tV + (((d * 2 + (lane >> 4)) ^ (rv & 7)) << 4), b0, b1, b2, b3);
-              mma_bf16_16816(o[vs * 8 + 2 * d], pv, b0, b1);
-              mma_bf16_16816(o[vs * 8 + 2 * d + 1], pv, b2, b3);
+#pragma unroll
+              for (int mt = 0; mt < MT; ++mt) {
+                if (!any[mt]) continue;
+                mma_bf16_16816(o[mt][vs * 8 + 2 * d], pv[mt], b0, b1);
+                mma_bf16_16816(o[mt][vs * 8 + 2 * d + 1], pv[mt], b2, b3);
+              }
             }
           }
           give();
@@ -628,37 +681,41 @@ __global__ void __launch_bounds__(160) decode_attn_wide_kernel(const __grid_cons
       }
     }
 #pragma unroll
-    for (int h = 0; h < 2; ++h) {
-      l_run[h] += __shfl_xor_sync(0xffffffffu, l_run[h], 1);
-      l_run[h] += __shfl_xor_sync(0xffffffffu, l_run[h], 2);
-    }
+    for (int mt = 0; mt < MT; ++mt)
+#pragma unroll
+      for (int h = 0; h < 2; ++h) {
+        l_run[mt][h] += __shfl_xor_sync(0xffffffffu, l_run[mt][h], 1);
+        l_run[mt][h] += __shfl_xor_sync(0xffffffffu, l_run[mt][h], 2);
+      }
   }
   __syncthreads();   // ring no longer needed: reuse it for the merge
 
-  float* sO = reinterpret_cast<float*>(ring);     // [4][16][DV]
-  float* sM = sO + 4 * 16 * DV;                   // [4][16]
-  float* sL = sM + 64;
-  if (warp < 4) {
+  float* sO = reinterpret_cast<float*>(ring);     // [CW][ROWS][DV]
+  if (warp < CW) {
 #pragma unroll
-    for (int i = 0; i < DV / 8; ++i) {
-      const int col = i * 8 + (lane & 3) * 2;
-      *reinterpret_cast<float2*>(sO + (warp * 16 + row_a) * DV + col) = make_float2(o[i][0], o[i][1]);
-      *reinterpret_cast<float2*>(sO + (warp * 16 + row_b) * DV + col) = make_float2(o[i][2], o[i][3]);
-    }
-    if ((lane & 3) == 0) {
-      sM[warp * 16 + row_a] = m_run[0]; sL[warp * 16 + row_a] = l_run[0];
-      sM[warp * 16 + row_b] = m_run[1]; sL[warp * 16 + row_b] = l_run[1];
-    }
+    for (int mt = 0; mt < MT; ++mt)
+#pragma unroll
+      for (int h = 0; h < 2; ++h) {
+        const int r = mt * 16 + (lane >> 2) + 8 * h;
+        float* dst = sO + (warp * ROWS + r) * DV + (lane & 3) * 2;
+#pragma unroll
+        for (int i = 0; i < DV / 8; ++i) *reinterpret_cast<float2*>(dst + i * 8) = make_float2(o[mt][i][2 * h], o[mt][i][2 * h + 1]);
+        if ((lane & 3) == 0) {
+          sM[warp * ROWS + r] = m_run[mt][h];
+          sL[warp * ROWS + r] = l_run[mt][h];
+        }
+      }
   }
   __syncthreads();
-  if (warp == 4) return;
-  for (int r = warp; r < rows; r += 4) {
-    const float m = fmaxf(fmaxf(sM[r], sM[16 + r]), fmaxf(sM[32 + r], sM[48 + r]));
-    float w[4], l = 0.f;
+  if (warp >= CW) return;
+  for (int r = warp; r < rows; r += CW) {
+    float m = -INFINITY, w[CW], l = 0.f;
 #pragma unroll
-    for (int j = 0; j < 4; ++j) {
-      w[j] = sM[16 * j + r] == -INFINITY ? 0.f : exp2f(sM[16 * j + r] - m);
-      l += w[j] * sL[16 * j + r];
+    for (int j = 0; j < CW; ++j) m = fmaxf(m, sM[j * ROWS + r]);
+#pragma unroll
+    for (int j = 0; j < CW; ++j) {
+      w[j] = sM[j * ROWS + r] == -INFINITY ? 0.f : exp2f(sM[j * ROWS + r] - m);
+      l += w[j] * sL[j * ROWS + r];
     }
     const int hq = (row0 + r) % p.n_q;
     float den = l;                                // the sink joins once: here, or in the merge of the splits
@@ -668,9 +725,10 @@ __global__ void __launch_bounds__(160) decode_attn_wide_kernel(const __grid_cons
     for (int col = lane * 2; col < dv; col += 64) {
       float a = 0.f, b = 0.f;
 #pragma unroll
-      for (int j = 0; j < 4; ++j) {
-        a += w[j] * sO[(16 * j + r) * DV + col];
-        b += w[j] * sO[(16 * j + r) * DV + col + 1];
+      for (int j = 0; j < CW; ++j) {
+        const float2 f = *reinterpret_cast<const float2*>(sO + (j * ROWS + r) * DV + col);
+        a += w[j] * f.x;
+        b += w[j] * f.y;
       }
       if (p.num_splits == 1)
         *reinterpret_cast<uint32_t*>(p.out + tok * (size_t(p.n_q) * dv) + hq * dv + col) = pack_bf16x2(a * inv, b * inv);
@@ -682,15 +740,29 @@ __global__ void __launch_bounds__(160) decode_attn_wide_kernel(const __grid_cons
   }
 }
 
-template <int DV>
+// 1 (launched nothing): the query rows and the merge do not fit shared memory
+template <int MT, int DV>
 static int launch_wide(const CUtensorMap* tk, const CUtensorMap* tv, const DecParams& p, int max_q, cudaStream_t st) {
   const int KS = (p.dk + 63) / 64;
-  const size_t smem = size_t(kWideSlabs) * kTile * 128 + size_t(16) * KS * 128 + sizeof(WideDecBarriers) + 1024;
-  if (smem > 227 * 1024) return -3;
-  cudaFuncSetAttribute(decode_attn_wide_kernel<DV>, cudaFuncAttributeMaxDynamicSharedMemorySize, int(smem));
-  const dim3 grid(p.seq_end - p.seq_begin, (p.n_q * max_q + 15) / 16, p.num_splits);
-  decode_attn_wide_kernel<DV><<<grid, 160, smem, st>>>(*tk, *tv, p, KS);
+  const size_t rest = size_t(16 * MT) * KS * 128 + sizeof(WideDecBarriers) + size_t(2) * kWideConsumers * 16 * MT * 4 + 1024;
+  const size_t merge = size_t(kWideConsumers) * 16 * MT * DV * 4, room = size_t(227) * 1024;
+  if (rest + merge > room) return 1;
+  int n = int((room - rest) / kWideSlab);
+  if (n > kWideMost) n = kWideMost;
+  if (size_t(n) * kWideSlab < merge || n < 2) return 1;
+  const size_t smem = rest + size_t(n) * kWideSlab;
+  const dim3 grid((p.n_q * max_q + 16 * MT - 1) / (16 * MT), p.seq_end - p.seq_begin, p.num_splits);   // a sequence's blocks side by side
+  if (grid.y > 65535) return -3;
+  cudaFuncSetAttribute(decode_attn_wide_kernel<MT, DV>, cudaFuncAttributeMaxDynamicSharedMemorySize, int(smem));
+  decode_attn_wide_kernel<MT, DV><<<grid, kWideThreads, smem, st>>>(*tk, *tv, p, KS, n);
   return cudaGetLastError() == cudaSuccess ? 0 : -1;
+}
+template <int DV>
+static int launch_wide_rows(const CUtensorMap* tk, const CUtensorMap* tv, const DecParams& p, int max_q, cudaStream_t st) {
+  int rc = 1;
+  if (p.n_q * max_q > 16) rc = launch_wide<2, DV>(tk, tv, p, max_q, st);
+  if (rc == 1) rc = launch_wide<1, DV>(tk, tv, p, max_q, st);
+  return rc == 1 ? -3 : rc;
 }
 
 }  // namespace xl_dec
@@ -1004,7 +1076,7 @@ XL_API int xl_decode_attention_ext(const void* q, const void* k_cache, const voi
   cudaStream_t st = static_cast<cudaStream_t>(stream);
   const dim3 grid(seq_end - seq_begin, n_kv * p.row_blocks, p.num_splits);
   int rc;
-  if (wide_keys) rc = dv > 64 ? launch_wide<128>(tk, tv, p, max_q < 1 ? 1 : max_q, st) : launch_wide<64>(tk, tv, p, max_q < 1 ? 1 : max_q, st);
+  if (wide_keys) rc = dv > 64 ? launch_wide_rows<128>(tk, tv, p, max_q < 1 ? 1 : max_q, st) : launch_wide_rows<64>(tk, tv, p, max_q < 1 ? 1 : max_q, st);
   else if (dv > 128) rc = launch_ext<256, 256>(tk, tv, p, grid, st);
   else if (dk > 128) rc = launch_ext<256, 128>(tk, tv, p, grid, st);
   else if (dk > 64) rc = dv > 64 ? launch_ext<128, 128>(tk, tv, p, grid, st) : launch_ext<128, 64>(tk, tv, p, grid, st);

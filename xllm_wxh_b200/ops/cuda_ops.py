@@ -824,7 +824,9 @@ def paged_attention_ext(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.T
         if window > 0:
             max_kv = min(max_kv, window + keep_first)
         max_q = max(1, inp.max_q) if inp.n_spec > 0 else 1
-        splits = decode_splits(n_dec, -(-Hq * max_q // 16) if wide else n_kv * -(-Hq // n_kv * max_q // 16), max_kv)
+        splits = decode_splits(n_dec, n_kv * -(-Hq // n_kv * max_q // 16), max_kv)
+        if wide:                    # one CTA of up to 32 query rows per SM
+            splits = max(1, min(sm_count() // max(1, n_dec * -(-Hq * max_q // 32)), max_kv // 512, 16))
         po = pl = None
         rows = max(T, n_dec)
         if splits > 1:
