@@ -576,49 +576,64 @@ struct AllNorm {
   const float* mix;
 };
 
-// q of one token in shared memory (fp32) -> its rows for every query head; a thread keeps V columns of the query heads of one key head
-// in registers (GROUP of them; 0: any number, read again for every row).
-template <typename T, int V, int GROUP>
-__device__ __forceinline__ void mix_rows(const float* q, const float* mix, T* __restrict__ out, int n_q, int n_k, int dk) {
-  const int width = n_k * dk, group = GROUP > 0 ? GROUP : n_q / n_k;
-  for (int c = threadIdx.x * V; c < width; c += blockDim.x * V) {
-    const int j = c / dk, d = c % dk;
-    const float* src = q + size_t(j) * group * dk + d;
-    float qv[GROUP > 0 ? GROUP : 1][V];
-    if (GROUP > 0) {
+// q of one token in shared memory (fp32) -> its rows for every query head.  A thread keeps four columns of the query heads of one key
+// head in registers as pairs (GROUP heads) and makes every n-th row, where threads are left over.  `twice`: the matrix in shared
+// memory, every element twice.
+template <typename T, int GROUP>
+__device__ __forceinline__ void mix_rows4(const float* q, const float* twice, T* __restrict__ out, int n_q, int n_k, int dk) {
+  const int width = n_k * dk, chunks = width / 4;
+  const int parts = chunks < int(blockDim.x) ? int(blockDim.x) / chunks : 1;
+  const int part = parts > 1 ? int(threadIdx.x) / chunks : 0;
+  if (part >= parts) return;
+  for (int i = parts > 1 ? threadIdx.x % chunks : threadIdx.x; i < chunks; i += blockDim.x) {
+    const int c = i * 4, j = c / dk;
+    const float* src = q + size_t(j) * GROUP * dk + c % dk;
+    ulonglong2 qv[GROUP];
 #pragma unroll
-      for (int g = 0; g < GROUP; ++g)
-#pragma unroll
-        for (int e = 0; e < V; ++e) qv[g][e] = src[g * dk + e];
-    }
+    for (int g = 0; g < GROUP; ++g) qv[g] = *reinterpret_cast<const ulonglong2*>(src + g * dk);
+    const uint64_t* row = reinterpret_cast<const uint64_t*>(twice) + j * GROUP;
 #pragma unroll 2
-    for (int h = 0; h < n_q; ++h) {
-      const float* m = mix + size_t(h) * n_q + j * group;
-      float a[V] = {};
-      if (GROUP > 0) {
+    for (int h = part; h < n_q; h += parts) {
+      const uint64_t* m = row + size_t(h) * n_q;
+      uint64_t a0 = 0, a1 = 0;
 #pragma unroll
-        for (int g = 0; g < GROUP; ++g)
-#pragma unroll
-          for (int e = 0; e < V; ++e) a[e] = fmaf(m[g], qv[GROUP > 0 ? g : 0][e], a[e]);
-      } else {
-        for (int g = 0; g < group; ++g)
-#pragma unroll
-          for (int e = 0; e < V; ++e) a[e] = fmaf(m[g], src[g * dk + e], a[e]);
+      for (int g = 0; g < GROUP; g += 2) {
+        ulonglong2 mm;
+        if (GROUP % 2 == 0) {
+          mm = *reinterpret_cast<const ulonglong2*>(m + g);      // n_q and j * GROUP are even
+        } else {
+          mm.x = m[g];
+          mm.y = 0;
+        }
+        a0 = fma2(mm.x, qv[g].x, a0);
+        a1 = fma2(mm.x, qv[g].y, a1);
+        if (GROUP % 2 == 0) {
+          a0 = fma2(mm.y, qv[GROUP > 1 ? g + 1 : 0].x, a0);
+          a1 = fma2(mm.y, qv[GROUP > 1 ? g + 1 : 0].y, a1);
+        }
       }
+      const float2 x = unpack2(a0), y = unpack2(a1);
       T* dst = out + size_t(h) * width + c;
-      if constexpr (V == 4 && sizeof(T) == 2) {
-        *reinterpret_cast<uint2*>(dst) = make_uint2(pack_bf16x2(a[0], a[1]), pack_bf16x2(a[2], a[3]));
-      } else if constexpr (V == 4) {
-        *reinterpret_cast<float4*>(dst) = make_float4(a[0], a[1], a[2], a[3]);
-      } else {
-        from_f32(dst, a[0]);
-      }
+      if constexpr (sizeof(T) == 2) *reinterpret_cast<uint2*>(dst) = make_uint2(pack_bf16x2(x.x, x.y), pack_bf16x2(y.x, y.y));
+      else *reinterpret_cast<float4*>(dst) = make_float4(x.x, x.y, y.x, y.y);
     }
   }
 }
+// The same for any sizes, an element at a time; element (h, g) of the matrix at mix[(h * n_q + g) * step].
+template <typename T>
+__device__ __forceinline__ void mix_rows_any(const float* q, const float* mix, int step, T* __restrict__ out, int n_q, int n_k, int dk) {
+  const int width = n_k * dk, group = n_q / n_k;
+  for (int i = threadIdx.x; i < n_q * width; i += blockDim.x) {
+    const int h = i / width, c = i % width, j = c / dk;
+    const float *src = q + size_t(j) * group * dk + c % dk, *m = mix + (size_t(h) * n_q + j * group) * step;
+    float a = 0.f;
+    for (int g = 0; g < group; ++g) a = fmaf(m[g * step], src[g * dk], a);
+    from_f32(out + i, a);
+  }
+}
 
-template <typename T, int V, bool MIX>
-__global__ void __launch_bounds__(256) qknorm_all_kernel(T* __restrict__ qkv, const int* __restrict__ slots, const T* __restrict__ q_w,
+template <typename T, int V, bool MIX, bool TURN>
+__global__ void __launch_bounds__(256, MIX ? 4 : 1) qknorm_all_kernel(T* __restrict__ qkv, const int* __restrict__ slots, const T* __restrict__ q_w,
                                                          const T* __restrict__ k_w, T* __restrict__ k_cache, T* __restrict__ v_cache,
                                                          T* __restrict__ wide, const AllNorm a, const Rotation rot, int mix_smem) {
   extern __shared__ __align__(16) float s_row[];       // MIX or rotation: normed q and k of the row; MIX: then the mixing matrix
@@ -642,7 +657,8 @@ __global__ void __launch_bounds__(256) qknorm_all_kernel(T* __restrict__ qkv, co
   const float rq = rsqrtf(block_sum(sq, red_q) / float(nq) + a.eps), rk = rsqrtf(block_sum(sk, red_k) / float(nk) + a.eps);
   const int slot = slots[t];
   const bool in = slot >= 0 && slot < a.cache_slots;
-  const bool turned = rot.table != nullptr;
+  constexpr bool turned = TURN;
+  const bool direct = V == 8 && turned && !rot.interleaved && rot.dims % 16 == 0 && a.dk % 8 == 0 && !(reinterpret_cast<uintptr_t>(rot.table) & 15);
   for (int c = threadIdx.x * V; c < nq + nk + nv; c += blockDim.x * V) {
     load(row + c, f);
     if (c < nq + nk) {
@@ -650,9 +666,22 @@ __global__ void __launch_bounds__(256) qknorm_all_kernel(T* __restrict__ qkv, co
       load(c < nq ? q_w + c : k_w + (c - nq), w);
 #pragma unroll
       for (int e = 0; e < V; ++e) f[e] = f[e] * r * w[e];
-      if (turned || (MIX && c < nq)) {
+      if constexpr (V == 8 && TURN) {
+        const int at = c % a.dk;
+        if (direct && at < rot.dims) {                     // turned here: the other elements of the eight pairs lie half away
+          const int half = rot.dims / 2, away = at < half ? half : -half, j = at < half ? at : at - half;
+          const float* tab = rot.table + size_t(clamp_id(rot.positions[t], rot.rows)) * rot.dims;
+          float g[8], wg[8], cs[8], sn[8];
+          load8(row + c + away, g);
+          load8((c < nq ? q_w + c : k_w + (c - nq)) + away, wg);
+          load8(tab + j, cs);
+          load8(tab + half + j, sn);
 #pragma unroll
-        for (int e = 0; e < V; ++e) s_row[c + e] = f[e];
+          for (int e = 0; e < 8; ++e) f[e] = fmaf(at < half ? -sn[e] : sn[e], g[e] * r * wg[e], f[e] * cs[e]);
+        }
+      }
+      if ((turned && !MIX) || (MIX && c < nq) || (turned && !direct)) {
+        if constexpr (V == 8) store8(s_row + c, f); else s_row[c] = f[0];
       } else if (c < nq) {
         store(row + c, f);
       } else if (in) {
@@ -665,9 +694,9 @@ __global__ void __launch_bounds__(256) qknorm_all_kernel(T* __restrict__ qkv, co
   if (!turned && !MIX) return;
   float* s_mix = s_row + (nq + nk + 3) / 4 * 4;
   if (MIX && mix_smem)
-    for (int i = threadIdx.x; i < a.n_q * a.n_q; i += blockDim.x) s_mix[i] = a.mix[i];
+    for (int i = threadIdx.x; i < a.n_q * a.n_q; i += blockDim.x) reinterpret_cast<float2*>(s_mix)[i] = make_float2(a.mix[i], a.mix[i]);
   __syncthreads();
-  if (turned) {
+  if (turned && !direct) {
     const float* cs = rot.table + size_t(clamp_id(rot.positions[t], rot.rows)) * rot.dims;
     const int half = rot.dims / 2;
     for (int i = threadIdx.x; i < (a.n_q + a.n_k) * half; i += blockDim.x) {
@@ -678,6 +707,8 @@ __global__ void __launch_bounds__(256) qknorm_all_kernel(T* __restrict__ qkv, co
       head[y] = rot_one(rot, cs, y, v, u);
     }
     __syncthreads();
+  }
+  if (turned && (!MIX || !direct)) {
     for (int c = (MIX ? nq : 0) + threadIdx.x * V; c < nq + nk; c += blockDim.x * V) {
 #pragma unroll
       for (int e = 0; e < V; ++e) f[e] = s_row[c + e];
@@ -687,15 +718,17 @@ __global__ void __launch_bounds__(256) qknorm_all_kernel(T* __restrict__ qkv, co
   }
   if constexpr (MIX) {
     T* out = wide + size_t(t) * a.n_q * nk;
-    const float* m = mix_smem ? s_mix : a.mix;
-    constexpr int W = V == 8 ? 4 : 1;
-    switch (a.n_q / a.n_k) {
-      case 1: mix_rows<T, W, 1>(s_row, m, out, a.n_q, a.n_k, a.dk); break;
-      case 2: mix_rows<T, W, 2>(s_row, m, out, a.n_q, a.n_k, a.dk); break;
-      case 4: mix_rows<T, W, 4>(s_row, m, out, a.n_q, a.n_k, a.dk); break;
-      case 8: mix_rows<T, W, 8>(s_row, m, out, a.n_q, a.n_k, a.dk); break;
-      default: mix_rows<T, W, 0>(s_row, m, out, a.n_q, a.n_k, a.dk); break;
+    if constexpr (V == 8) {
+      if (mix_smem) {
+        switch (a.n_q / a.n_k) {
+          case 1: mix_rows4<T, 1>(s_row, s_mix, out, a.n_q, a.n_k, a.dk); return;
+          case 2: mix_rows4<T, 2>(s_row, s_mix, out, a.n_q, a.n_k, a.dk); return;
+          case 4: mix_rows4<T, 4>(s_row, s_mix, out, a.n_q, a.n_k, a.dk); return;
+          case 8: mix_rows4<T, 8>(s_row, s_mix, out, a.n_q, a.n_k, a.dk); return;
+        }
+      }
     }
+    mix_rows_any(s_row, mix_smem ? s_mix : a.mix, mix_smem ? 2 : 1, out, a.n_q, a.n_k, a.dk);
   }
 }
 template <typename T>
@@ -709,17 +742,19 @@ static int launch_qknorm_all(void* qkv, const void* slots, const void* q_w, cons
                    (!a.mix || (a.dk % 8 == 0 && al16(wide)));
   constexpr size_t kMost = 160 * 1024;
   size_t smem = a.mix || rot.table ? size_t(nq + nk + 3) / 4 * 16 : 0;
-  const int mix_smem = a.mix && smem + size_t(a.n_q) * a.n_q * 4 <= kMost;
-  if (mix_smem) smem += size_t(a.n_q) * a.n_q * 4;
+  const int mix_smem = a.mix && smem + size_t(a.n_q) * a.n_q * 8 <= kMost;
+  if (mix_smem) smem += size_t(a.n_q) * a.n_q * 8;
   if (smem > kMost) return -2;
-#define XL_ALL(V, MIX)                                                                                                                 \
+#define XL_ALL(V, MIX, TURN)                                                                                                           \
   do {                                                                                                                                 \
     static bool set = false;                                                                                                           \
-    if (!set) { cudaFuncSetAttribute(qknorm_all_kernel<T, V, MIX>, cudaFuncAttributeMaxDynamicSharedMemorySize, int(kMost)); set = true; } \
-    qknorm_all_kernel<T, V, MIX><<<rows, 256, smem, st>>>(x, s, qw, kw, kc, vc, o, a, rot, mix_smem);                                  \
+    if (!set) { cudaFuncSetAttribute(qknorm_all_kernel<T, V, MIX, TURN>, cudaFuncAttributeMaxDynamicSharedMemorySize, int(kMost)); set = true; } \
+    qknorm_all_kernel<T, V, MIX, TURN><<<rows, 256, smem, st>>>(x, s, qw, kw, kc, vc, o, a, rot, mix_smem);                            \
   } while (0)
-  if (a.mix) { if (vec) XL_ALL(8, true); else XL_ALL(1, true); }
-  else { if (vec) XL_ALL(8, false); else XL_ALL(1, false); }
+#define XL_ALL_TURN(V, MIX) do { if (rot.table) XL_ALL(V, MIX, true); else XL_ALL(V, MIX, false); } while (0)
+  if (a.mix) { if (vec) XL_ALL_TURN(8, true); else XL_ALL_TURN(1, true); }
+  else { if (vec) XL_ALL_TURN(8, false); else XL_ALL_TURN(1, false); }
+#undef XL_ALL_TURN
 #undef XL_ALL
   return cudaGetLastError() == cudaSuccess ? 0 : -1;
 }
