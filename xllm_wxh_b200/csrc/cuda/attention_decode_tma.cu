@@ -469,7 +469,7 @@ __global__ void __launch_bounds__(kWideThreads, 1) decode_attn_wide_kernel(const
 
   if (threadIdx.x == 0) {
     for (int s = 0; s < n_slabs; ++s) {
-      mbar_init(&bars->full[s], 1);
+      mbar_init(&bars->full[s], kWideProducers);
       mbar_init(&bars->empty[s], CW);
     }
     mbar_fence_init();
@@ -524,6 +524,8 @@ __global__ void __launch_bounds__(kWideThreads, 1) decode_attn_wide_kernel(const
             ok = false;
           } else if (part == 0) {
             mbar_arrive_expect_tx(&bars->full[at.slot], uint32_t(n_boxes) * bt_tok * 128);
+          } else {
+            mbar_arrive(&bars->full[at.slot]);             // also without a box of its own: no producer falls a round behind
           }
         }
         ok = __shfl_sync(0xffffffffu, ok, 0);

@@ -648,10 +648,11 @@ prefill_attn_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_con
 constexpr int WKV = 256;                       // kv tokens per tile
 constexpr int W_SLAB = 128 * 128;              // 16 KB: [128 rows or tokens][64 columns]
 constexpr int W_UNIT = 2 * W_SLAB;
+constexpr int kWideProducers = 3;
 template <int QR> struct WideCfg {
   static constexpr int kUnits = QR == 8 ? 3 : 5;
   static constexpr int kSmem = QR * W_SLAB + kUnits * W_UNIT;          // query slabs, ring
-  static constexpr int kThreads = 384;
+  static constexpr int kThreads = 288 + 32 * kWideProducers;
 };
 struct WideBarriers {
   uint64_t q_full;
@@ -676,7 +677,7 @@ __device__ __forceinline__ void tc_mma_f16_ts(uint32_t tmem_d, uint32_t tmem_a, 
 }
 
 template <int QR>
-__global__ void __launch_bounds__(384, 1)
+__global__ void __launch_bounds__(WideCfg<QR>::kThreads, 1)
 prefill_attn_wide_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__ CUtensorMap tmK, const __grid_constant__ CUtensorMap tmV,
                          const Params p, const int KS) {
   constexpr int U = WideCfg<QR>::kUnits;
@@ -730,7 +731,7 @@ prefill_attn_wide_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_c
   if (threadIdx.x == 0) {
     mbar_init(&bars->q_full, 1);
     for (int u = 0; u < U; ++u) {
-      mbar_init(&bars->full[u], 1);
+      mbar_init(&bars->full[u], kWideProducers);
       mbar_init(&bars->empty[u], 1);
     }
     mbar_init(&bars->s_full, 1);
@@ -778,12 +779,14 @@ prefill_attn_wide_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_c
           ok = false;
         } else if (part == 0) {
           mbar_arrive_expect_tx(&bars->full[u], bytes);
+        } else {
+          mbar_arrive(&bars->full[u]);                    // also without a box of its own: no producer falls a round behind
         }
       }
       ok = __shfl_sync(0xffffffffu, ok, 0);
       return ok;
     };
-    auto mine = [&](int n) { return lane < n && lane % 3 == part; };
+    auto mine = [&](int n) { return lane < n && lane % kWideProducers == part; };
     int slot = slot_of(0), slot_v = 0;
     for (int j = 0; j <= n_tiles && ok; ++j) {
       const int next = j + 1 < n_tiles ? slot_of(j + 1) : 0;
