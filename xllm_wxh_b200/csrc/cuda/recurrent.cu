@@ -322,7 +322,7 @@ struct MixParams {
 };
 template <int KIND, typename T>
 __device__ __forceinline__ size_t record_size(const MixParams<T>& p) {
-  return size_t(p.dk) * p.dv + (KIND == MIX_MEMORY ? p.dk : 0);
+  return size_t(p.dk) * (KIND == MIX_BONUS ? p.dk : p.dv) + (KIND == MIX_MEMORY ? p.dk : 0);
 }
 template <int KIND, typename T>
 __device__ __forceinline__ float decay_of(const MixParams<T>& p, float z) {
@@ -467,7 +467,7 @@ matrix_segment_kernel(const MixParams<T> p, int v8, int g8, int s4) {
   }
   const int slot = record_of(p.q, seq);
   if (slot < 0) return;
-  const int h = blockIdx.y, dk = p.dk, dv = p.dv, tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
+  const int h = blockIdx.y, dk = p.dk, dv = BONUS ? dk : p.dv, tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
   const int kg = tid % KG, vg = tid / KG;
   const int start = p.q.q_cu[seq], len = p.q.q_cu[seq + 1] - start;
   const int t0 = start + seg * p.L, n = min(p.L, len - seg * p.L);
@@ -516,10 +516,9 @@ matrix_segment_kernel(const MixParams<T> p, int v8, int g8, int s4) {
   float prod[PR];                                         // !OUT: decay of keys `tid`, `tid` + NT ... over the segment
 #pragma unroll
   for (int i = 0; i < PR; ++i) prod[i] = 1.f;
-  // Rows are finished by vectors of 8 columns: LR lanes per row, RP rows per warp and pass; LK lanes per row for its keys.
+  // Rows are finished (and their bonus is prepared) by vectors of 8 columns: LR lanes per row, RP rows per warp and pass.
   constexpr int LR = DV / 8, RP = 32 / LR, PASSES = kMixRows / (NT / 32 * RP);
-  constexpr int LK = DK / 8, RK = 32 / LK;
-  static_assert(PASSES >= 1, "rows per pass");
+  static_assert(PASSES >= 1 && (!BONUS || DK == DV), "rows per pass; the bonus takes keys and values of one size");
   const int fr_row = warp * RP + lane / LR, fr_c = lane % LR * 8;
   if (OUT) {                                              // visible behind the first tile's barrier
     for (int c = tid; c < DV; c += NT) sNw[OUT ? c : 0] = c < dv ? to_f32(p.norm_w[h * p.norm_step + c]) * p.scale : 0.f;
@@ -548,10 +547,11 @@ matrix_segment_kernel(const MixParams<T> p, int v8, int g8, int s4) {
         } else {
           fz[i].load(p.z + t * (size_t(p.H) * dk) + size_t(h) * dk + c);
         }
+        if (BONUS) fv[BONUS ? i : 0].load(p.v + at);        // keys and values are of one size
       }
     }
 #pragma unroll
-    for (int i = 0; i < NV; ++i) {
+    for (int i = 0; i < (BONUS ? 0 : NV); ++i) {
       const int e = i * NT + tid, row = e / (DV / 8), c = e % (DV / 8) * 8;
       if (row < m && c < dv) fv[i].load(p.v + size_t(t0 + b + row) * p.ld + size_t(h) * dv + c);
     }
@@ -566,11 +566,12 @@ matrix_segment_kernel(const MixParams<T> p, int v8, int g8, int s4) {
       for (int i = 0; i < NK; ++i) {
         const int e = i * NT + tid, row = e / (DK / 8), c = e % (DK / 8) * 8;
         if (EK % NT && e >= EK) break;
-        float k[8] = {}, r[8] = {}, w[8];
+        float k[8] = {}, r[8] = {}, w[8], vv[8] = {};
 #pragma unroll
         for (int j = 0; j < 8; ++j) w[j] = 1.f;
         if (row < m && c < dk) {
           fk[i].get(k);
+          if (BONUS) fv[BONUS ? i : 0].get(vv);
           if (OUT) fr[OUT ? i : 0].get(r);
           if constexpr (MEMORY) {
 #pragma unroll
@@ -592,10 +593,11 @@ matrix_segment_kernel(const MixParams<T> p, int v8, int g8, int s4) {
         }
         store_keys<DK>(sK[row], c, k);
         store_keys<DK>(sW[row], c, w);
+        if (BONUS) store8(&sV[BONUS ? row : 0][BONUS ? c : 0], vv);
         if (OUT) store_keys<DK>(sR[row], c, r);
       }
 #pragma unroll
-      for (int i = 0; i < NV; ++i) {
+      for (int i = 0; i < (BONUS ? 0 : NV); ++i) {
         const int e = i * NT + tid, row = e / (DV / 8), c = e % (DV / 8) * 8;
         if (EV % NT && e >= EV) break;
         float v[8] = {};
@@ -634,24 +636,22 @@ matrix_segment_kernel(const MixParams<T> p, int v8, int g8, int s4) {
 #pragma unroll
       for (int q = 0; q < PASSES; ++q) {
         const int row = q * (NT / 32 * RP) + fr_row;
-        if (row < m && g8 && fr_c < dv) gate[OUT ? q : 0].load(p.gate + size_t(t0 + b + row) * p.ldg + size_t(h) * dv + fr_c);
-      }
-      if (BONUS) {
-#pragma unroll
-        for (int q = 0; q < kMixRows; q += NT / 32 * RK) {
-          const int row = q + warp * RK + lane / LK, c = lane % LK * 8;
-          float s = 0.f;
-          if (row < m) {
+        float s = 0.f;
+        if (row < m) {
+          if (g8 && fr_c < dv) gate[OUT ? q : 0].load(p.gate + size_t(t0 + b + row) * p.ldg + size_t(h) * dv + fr_c);
+          if constexpr (BONUS) {
             float r[8], k[8], u[8];
-            load_keys<DK>(sR[row], c, r);
-            load_keys<DK>(sK[row], c, k);
-            load8(&sU[c], u);
+            load_keys<DK>(sR[row], fr_c, r);
+            load_keys<DK>(sK[row], fr_c, k);
+            load8(&sU[fr_c], u);
 #pragma unroll
             for (int j = 0; j < 8; ++j) s = fmaf(r[j] * u[j], k[j], s);
           }
+        }
+        if constexpr (BONUS) {
 #pragma unroll
-          for (int o = LK / 2; o > 0; o >>= 1) s += __shfl_xor_sync(0xffffffffu, s, o);
-          if (lane % LK == 0 && row < m) sRow[row] = s;    // read behind the next barrier
+          for (int o = LR / 2; o > 0; o >>= 1) s += __shfl_xor_sync(0xffffffffu, s, o);
+          if (lane % LR == 0 && row < m) sRow[row] = s;    // read behind the next barrier
         }
       }
     } else {
@@ -862,7 +862,7 @@ template <typename T, int KIND>
 __global__ void __launch_bounds__(kMixThreads) matrix_single_kernel(const MixParams<T> p) {
   constexpr bool BONUS = KIND == MIX_BONUS, MEMORY = KIND == MIX_MEMORY;
   extern __shared__ __align__(16) float sm[];
-  const int seq = blockIdx.x, h = blockIdx.y, dk = p.dk, dv = p.dv, tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
+  const int seq = blockIdx.x, h = blockIdx.y, dk = p.dk, dv = BONUS ? dk : p.dv, tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
   const int t = p.q.q_cu[seq], len = p.q.q_cu[seq + 1] - t;
   if (len != 1) return;
   const int slot = record_of(p.q, seq);
@@ -882,6 +882,16 @@ __global__ void __launch_bounds__(kMixThreads) matrix_single_kernel(const MixPar
 #pragma unroll
     for (int i = 0; i < kAhead; ++i)
       if (kq + i * groups < dk) s[i] = rec[size_t(kq + i * groups) * quads + vq];
+  }
+  constexpr int kCols = 4;                                  // columns per thread: dv <= 4 * kMixThreads
+  T vals[kCols], gates[kCols];
+#pragma unroll
+  for (int i = 0; i < kCols; ++i) {
+    const int c = i * kMixThreads + tid;
+    if (c < dv) {
+      vals[i] = p.v[size_t(t) * p.ld + size_t(h) * dv + c];
+      gates[i] = p.gate[size_t(t) * p.ldg + size_t(h) * dv + c];
+    }
   }
   TokenGates g = {};
   if (MEMORY) g = token_gates(p, t, h, cont ? p.top[size_t(slot) * p.H + h] : 0.f);
@@ -904,7 +914,9 @@ __global__ void __launch_bounds__(kMixThreads) matrix_single_kernel(const MixPar
     sR[c] = r;
     sK[c] = k;
   }
-  for (int c = tid; c < dv; c += kMixThreads) sV[c] = to_f32(p.v[size_t(t) * p.ld + size_t(h) * dv + c]);
+#pragma unroll
+  for (int i = 0; i < kCols; ++i)
+    if (i * kMixThreads + tid < dv) sV[i * kMixThreads + tid] = to_f32(vals[i]);
   dot = warp_sum(dot);
   if (lane == 0) red[0][warp] = dot;
   __syncthreads();
@@ -955,9 +967,13 @@ __global__ void __launch_bounds__(kMixThreads) matrix_single_kernel(const MixPar
 #pragma unroll
   for (int i = 0; i < kMixThreads / 32; ++i) ss += red[1][i];
   const float inv = rsqrtf(ss / float(dv) + p.eps) * p.scale;
-  for (int c = tid; c < dv; c += kMixThreads)
-    from_f32(p.out + size_t(t) * p.ldo + size_t(h) * dv + c,
-             sO[c] * inv * to_f32(p.norm_w[h * p.norm_step + c]) * out_gate<KIND>(to_f32(p.gate[size_t(t) * p.ldg + size_t(h) * dv + c])));
+#pragma unroll
+  for (int i = 0; i < kCols; ++i) {
+    const int c = i * kMixThreads + tid;
+    if (c < dv)
+      from_f32(p.out + size_t(t) * p.ldo + size_t(h) * dv + c,
+               sO[c] * inv * to_f32(p.norm_w[h * p.norm_step + c]) * out_gate<KIND>(to_f32(gates[i])));
+  }
 }
 
 // Any head sizes, any number of rows: the state stays in memory, one thread per value column.
@@ -1066,16 +1082,17 @@ static int launch_matrix(MixParams<T> p, int seg_cap, int has_long, int has_sing
       matrix_any_kernel<T, KIND><<<by_seq, 256, any_smem, st>>>(p, 2, 1 << 30);
     } else {
 #define XL_MIX(DK, DV) return launch_segments<T, KIND, DK, DV>(p, seg_cap, v8, g8, s4, st)
-      if (KIND == MIX_BONUS) {                                         // keys and values of one size
+      if constexpr (KIND == MIX_BONUS) {                               // keys and values of one size
         if (dk <= 32) XL_MIX(32, 32);
         if (dk <= 64) XL_MIX(64, 64);
         XL_MIX(128, 128);
-      }
+      } else {
       if (dk <= 32) { if (dv <= 32) XL_MIX(32, 32); if (dv <= 64) XL_MIX(32, 64); XL_MIX(32, 128); }
       if (dk <= 64) { if (dv <= 32) XL_MIX(64, 32); if (dv <= 64) XL_MIX(64, 64); XL_MIX(64, 128); }
       if (dv <= 32) XL_MIX(128, 32);
       if (dv <= 64) XL_MIX(128, 64);
       XL_MIX(128, 128);
+      }
 #undef XL_MIX
     }
   }

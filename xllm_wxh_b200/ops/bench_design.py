@@ -289,7 +289,7 @@ def falalix_kernels() -> List[Dict]:
         alone(f"token shift, {kind} {seqs} x {q_len}", time_graph([lambda s=s: c.token_shift(s[0], s[1], s[2], inp) for s in sets]), T * H * 12.0)
         del sets
         sets = [(_bf(T, 2 * C), _bf(taps, C), _bf(C), _bf(seqs + 1, taps - 1, C)) for _ in range(4 if kind == "prefill" else 16)]
-        alone(f"convolution, {kind} {seqs} x {q_len}", time_graph([lambda s=s: c.conv_silu(s[0][:, :C], s[1], s[2], s[3], inp) for s in sets]),
+        alone(f"convolution, {kind} {seqs} x {q_len}", time_graph([lambda s=s: c.causal_conv(s[0][:, :C], s[1], s[2], s[3], inp, "silu") for s in sets]),
               T * C * 4.0 + (0 if new else 2) * seqs * 3 * C * 2.0)
         del sets
         A = -torch.rand(C, N, device=DEV)
