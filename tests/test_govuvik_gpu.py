@@ -141,13 +141,13 @@ def test_long_and_many_portions(rows, monkeypatch):
     qq, kk, vv = (rg.take(x, rows) for x in (q, k, v))
     vv = torch.cat([qq, kk, vv], 1)
     qq, kk, vv = vv[:, :H * d], vv[:, H * d:2 * H * d], vv[:, 2 * H * d:]
-    a_ = ops.gated_memory(qq, kk, vv, rg.take(z, rows), bias.to(DEV), 1 / 16, rg.take(gate, rows), torch.ones(dv, device=DEV), 1e-5, state, inp)
+    a_ = ops.gated_memory(qq, kk, vv, rg.take(z, rows), bias.to(DEV), 1 / 20, rg.take(gate, rows), torch.ones(dv, device=DEV), 1e-5, state, inp)
     b_ = ops.matrix_memory(qq, kk, vv, rg.take(zi, rows), ibias.to(DEV), 9.0, rg.take(gate, rows), torch.ones(H * dv, device=DEV), 1e-5, mem, top, inp)
     at = 0
     for i, a, b in rows:
         if lens[i] > 8 or i % 7 == 0:
             Q, K, V = (x[i].double().view(-1, H, w) for x, w in ((q, d), (k, d), (v, dv)))
-            o = O.gated_linear_core(Q * d ** -0.5, K, V, O.channel_decay(z[i].double() + bias.double(), 16.0).view(-1, H, d))
+            o = O.gated_linear_core(Q * d ** -0.5, K, V, O.channel_decay(z[i].double() + bias.double(), 20.0).view(-1, H, d))
             assert rel(a_[at:at + b - a], O.rms_norm(o, 1.0, 1e-5).flatten(1) * O.silu(gate[i].double())) < 2e-5, lens[i]
             li, f = O.soft_bound(zi[i].double() + ibias.double(), 9.0).split(H, -1)
             o = O.matrix_memory_core(Q * d ** -0.5, K, V, li, O.log_sigmoid(f))
@@ -206,7 +206,7 @@ def test_attention(heads, size, block, pad, dtype):
 
 
 @pytest.mark.parametrize("dtype", DTYPES)
-@pytest.mark.parametrize("heads", [(4, 2, 64, 64), (8, 4, 128, 128), (8, 4, 96, 64)])
+@pytest.mark.parametrize("heads", [(6, 2, 64, 40), (8, 4, 128, 128), (8, 4, 96, 64)])
 @pytest.mark.parametrize("size", [40, 64, 33, 128])
 def test_one_key_just_inside_or_outside(size, heads, dtype):
     """One key stands out by far (its value too): rows that see it come out large, all others small; it lies at block and tile
@@ -227,7 +227,7 @@ def test_one_key_just_inside_or_outside(size, heads, dtype):
 
 
 def test_a_sink_that_takes_most_of_the_weight():
-    for heads in ((4, 2, 64, 64), (8, 4, 128, 128)):
+    for heads in ((6, 2, 64, 40), (8, 4, 128, 128)):
         got, want = attention_case(SPANS, *heads, 50, 16, torch.bfloat16, sinks=12.0)
         assert rel(got, want) < 1e-2
 
@@ -297,7 +297,7 @@ def test_norm_kernels(H, dtype):
     assert rel(xd, want) < 1e-6 and rel(h, O.rms_norm(want, d[5], 1e-6)) < tol
 
 
-@pytest.mark.parametrize("T,W,ff,E,top", [(1, 64, 96, 8, 4), (300, 256, 128, 16, 3), (37, 72, 40, 5, 2), (33, 67, 45, 7, 1), (9, 128, 64, 1, 1), (64, 2048, 1152, 12, 6)])
+@pytest.mark.parametrize("T,W,ff,E,top", [(1, 64, 80, 10, 4), (300, 256, 128, 16, 3), (37, 72, 40, 5, 2), (33, 67, 45, 7, 1), (9, 128, 64, 1, 1), (64, 2048, 1152, 12, 6)])
 @pytest.mark.parametrize("dtype", DTYPES)
 def test_experts_without_a_gate(T, W, ff, E, top, dtype):
     g = torch.Generator().manual_seed(T + W)
@@ -323,10 +323,10 @@ def test_experts_without_a_gate(T, W, ff, E, top, dtype):
 def models(tmp_path_factory):
     out = {}
     wide = M.config([
-        (M.parallel(heads=8, kv_heads=4, dim=128, vdim=128, window=70, conv=4, rot=64, g_heads=4, g_dim=64, g_vdim=128, tau=16.0), M.moe(ff=256, experts=16, top=4)),
-        (M.memory(heads=4, dim=64, vdim=128, cap=15.0), M.moe(ff=128, experts=8, top=2)),
-        (M.parallel(heads=4, kv_heads=2, dim=64, vdim=64, window=150, rot=16, g_heads=6, g_dim=32, g_vdim=64), None)],
-        width=256, vocab=1024, taps=4, softcap=30.0)
+        (M.parallel(heads=8, kv_heads=4, dim=128, vdim=128, window=70, conv=4, rot=64, g_heads=4, g_dim=64, g_vdim=128, tau=12.0), M.moe(ff=256, experts=16, top=4)),
+        (M.memory(heads=3, dim=64, vdim=128, cap=11.0), M.moe(ff=128, experts=10, top=2)),
+        (M.parallel(heads=6, kv_heads=2, dim=56, vdim=48, window=150, rot=32, g_heads=5, g_dim=32, g_vdim=96), None)],
+        width=320, vocab=1000, taps=4, softcap=22.0)
     for name, cfg in (("mixed", M.mixed_config()), ("odd", M.odd_config()), ("wide", wide)):
         sd = M.weights(cfg, 5)
         out[name] = cfg, {k: v.double() for k, v in sd.items()}, M.save(cfg, sd, tmp_path_factory.mktemp(name))

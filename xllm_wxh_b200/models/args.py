@@ -543,9 +543,9 @@ def preset(name: str) -> ModelArgs:
         mlp = FeedForwardSpec(ff=1152, act="relu2", experts=128, top_k=8, scoring="softmax_chosen")
         par = LayerSpec(ParallelSpec(AttentionSpec(heads=32, kv_heads=4, dim=128, vdim=128, scale=128 ** -0.5, window=4096, conv=4,
                                                    mixed_scores=True, learned_sink=True, qk_norm_all=True,
-                                                   rot=RotarySpec(64, 1e6, False, 8.0, 8192.0, 4.0, 1.0, True)),
+                                                   rot=RotarySpec(64, 5e5, False, 8.0, 8192.0, 4.0, 1.0, True)),
                                      GatedLinearSpec(heads=16, dim=64, vdim=128, tau=16.0), 0.5, 0.5, branch_norm=True), mlp)
         mem = LayerSpec(MatrixMemorySpec(heads=32, dim=64, vdim=128, gate_cap=15.0), mlp)
         return args_from_layer_list([par, par, par, mem] * 12, run_order(48), model_type="govuvik", vocab_size=151936, hidden_size=2048,
-                                    max_position_embeddings=40960, input_conv=4, logit_softcap=30.0)
+                                    max_position_embeddings=40960, input_conv=4, logit_softcap=20.0)
     raise KeyError(name)
